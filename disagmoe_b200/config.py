@@ -7,7 +7,7 @@ layers) and what the Blackwell kernels need to know.
 from __future__ import annotations
 
 from dataclasses import dataclass, field, replace
-from typing import List, Optional
+from typing import List, Optional, Union
 
 import torch
 
@@ -79,6 +79,101 @@ class ModelConfig:
         return replace(self, **changes)
 
 
+# ---- decoders described layer by layer --------------------------------------------------------------------------------
+# A layer = one token mixer (attention or a linear recurrence) and an optional feed-forward, each between a norm before it
+# and a norm after it. Mixers carry their own sizes, so layers of one model may differ in everything but the width.
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary embedding on the first ``dims`` dimensions of a head (pairs i, i + dims / 2); ``factor`` != None: YaRN."""
+    dims: int
+    base: float
+    factor: Optional[float] = None
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Softmax attention with per-head query / key norm. ``window``: a token sees itself and the window - 1 tokens before
+    it (None: all). ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[RotarySpec] = None
+    window: Optional[int] = None
+    softcap: Optional[float] = None
+    kv_from: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Gated linear attention: decay sigmoid(z)^(1 / tau) per key channel, ``rank`` = inner size of the map to z."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 16
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """Gated delta rule with one decay per head and key channel and short convolutions of ``conv`` taps on q, k and v;
+    ``rank`` / ``gate_rank`` = inner sizes of the maps to the decay and to the output gate."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    rank: int = 16
+    gate_rank: int = 16
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Union[AttentionSpec, GatedLinearSpec, ChannelDeltaSpec]
+    ff: Optional[int] = None                    # width of the gated feed-forward, None = the layer has none
+
+
+@dataclass
+class LayerListConfig(ModelConfig):
+    """A decoder given as a list of :class:`LayerSpec`. The MoE fields of the base class stay at zero: everything is on
+    the attention side, so only the single-GPU engines serve it."""
+    layers: List[LayerSpec] = field(default_factory=list)
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    architecture: str = ""
+
+    def is_dense_layer(self, layer_id: int) -> bool:
+        return True
+
+    def __post_init__(self):
+        super().__post_init__()
+        assert self.num_layers == len(self.layers)
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            if isinstance(m, GatedLinearSpec):
+                continue
+            if m.heads % m.kv_heads:
+                raise ValueError(f"layer {i}: {m.heads} heads do not share {m.kv_heads} key / value heads evenly")
+            src = getattr(m, "kv_from", None)
+            if src is not None:
+                s = self.layers[src].mixer if 0 <= src < i else None
+                if not isinstance(s, AttentionSpec) or s.kv_from is not None or \
+                        (s.kv_heads, s.dim, s.vdim) != (m.kv_heads, m.dim, m.vdim):
+                    raise ValueError(f"layer {i} cannot read the keys and values of layer {src}")
+
+    @classmethod
+    def make(cls, width: int, vocab: int, layers: List[LayerSpec], dtype=torch.bfloat16, **kw) -> "LayerListConfig":
+        heads = max(l.mixer.heads for l in layers)
+        kw = {**dict(rms_norm_eps=1e-6, head_dim=max(l.mixer.dim for l in layers)), **kw}
+        return cls(hidden_size=width, num_layers=len(layers), num_heads=heads, num_kv_heads=heads, num_experts=0,
+                   intermediate_size=max((l.ff or 0) for l in layers), dtype=dtype, ep_size=1, top_k=0, vocab_size=vocab,
+                   layers=list(layers), **kw)
+
+
 @dataclass
 class CacheConfig:
     """Paged KV cache configuration (field names of vLLM's CacheConfig as used at disagmoe/config.py:41-61)."""
@@ -133,7 +228,24 @@ tiny_config = ModelConfig(
     dtype=torch.float32, ep_size=1, top_k=2, vocab_size=1024, head_dim=64, rope_theta=1e4, name="tiny-moe",
 )
 
+# Rurunex design at the size of a small production model (random weights): two recurrences for every attention layer.
+def _rurunex_layers(groups: int, heads: int, dim: int, ff: int) -> List[LayerSpec]:
+    gla = GatedLinearSpec(heads, dim, dim, tau=16.0, rank=16)
+    delta = ChannelDeltaSpec(heads, heads, dim, dim, conv=4, rank=dim, gate_rank=dim)
+    out: List[LayerSpec] = []
+    for g in range(groups):
+        attn = AttentionSpec(heads, max(1, heads // 4), dim, dim, scale=dim ** -0.5, window=1024, softcap=30.0,
+                             rot=RotarySpec(dim, 1e6, factor=4.0, original=8192),
+                             kv_from=len(out) - 1 if g % 2 else None)
+        out += [LayerSpec(gla, ff), LayerSpec(delta, ff), LayerSpec(attn, ff)]
+    return out
+
+
+rurunex_config = LayerListConfig.make(2048, 32000, _rurunex_layers(6, 16, 128, 5632), max_seq_len=8192, embed_scale=45.25,
+                                      logit_scale=0.25, architecture="Rurunex", name="rurunex-18l")
+
 PRESETS = {
+    "rurunex": rurunex_config,
     "mixtral": mixtral_config, "mixtral-8x7b": mixtral_config, "duo": duo_expert_mixtral,
     "qwen-moe": qwen_moe_config, "deepseek-v2-lite": deepseek_v2_lite_config, "tiny": tiny_config,
 }

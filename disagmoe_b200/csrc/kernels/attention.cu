@@ -79,6 +79,22 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// Options of the EXT instantiations of both kernels (plain ones compile without them):
+//   window > 0: a query at position p sees only keys in (p - window, p];
+//   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap).
+// The EXT kernels also keep the softmax weights at fp32 accuracy in the P V product: P = hi + lo, both bf16, two MMAs.
+struct AttnExt {
+  int window;
+  float cap_in, cap_log2;
+};
+// raw q.k -> score in base-2 units. tanh(x) = 1 - 2 / (exp(2x) + 1), good to ~1e-7 absolute.
+template <bool EXT>
+__device__ __forceinline__ float attn_score(float raw, float scale_log2, const AttnExt& x) {
+  if (EXT && x.cap_log2 > 0.f) return x.cap_log2 * (1.f - __fdividef(2.f, exp2f(raw * x.cap_in) + 1.f));
+  return raw * scale_log2;
+}
+__device__ __forceinline__ float bf16_rest(float v) { return v - __bfloat162float(__float2bfloat16(v)); }
+
 constexpr int kAttnStages = 3;     // cp.async ring depth, per warp
 constexpr int kAttnStageTok = 16;  // cached tokens per stage and warp (block_size must be a multiple of it)
 constexpr int kAttnWarps = kAttnThreads / 32;
@@ -87,13 +103,13 @@ constexpr int kAttnWarps = kAttnThreads / 32;
 // Each warp owns every 4th chunk of 16 cached tokens and streams them through its private cp.async ring
 // (swizzled so that ldmatrix is bank-conflict free): S = Q K^T (2 n-tiles), online softmax on the accumulator
 // fragments, P re-used in place as the A operand of O += P V (V read with ldmatrix.trans).
-template <int HD, int GQ>
+template <int HD, int GQ, bool EXT>
 __global__ void __launch_bounds__(kAttnThreads)
 paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ kcache,
                   const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_blocks,
                   const int* __restrict__ bt_row, const int* __restrict__ ctx_len, int block_size, int n_kv,
                   float scale_log2, int splits, __nv_bfloat16* __restrict__ out, long long ld_out,
-                  float* __restrict__ part_o, float* __restrict__ part_lse) {
+                  float* __restrict__ part_o, float* __restrict__ part_lse, AttnExt ext) {
   static_assert(GQ <= 8, "the query group must fit the first 8 rows of the MMA tile");
   constexpr int ROWB = HD * 2;                       // bytes of one cached row of one kv head
   constexpr int NCH = HD / 8;                        // 16-byte chunks per row
@@ -117,10 +133,14 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
   const int len = ctx_len[t];
   const int row = bt_row != nullptr ? bt_row[t] : t;
   const int* bt = block_tables + static_cast<long long>(row) * max_blocks;
-  const int nblk = (len + block_size - 1) / block_size;
+  // first visible token, and its block: the blocks from there on are dealt out to the splits
+  const int vis0 = EXT && ext.window > 0 ? max(0, len - ext.window) : 0;
+  const int blk0 = vis0 / block_size;
+  const int nblk = (len + block_size - 1) / block_size - blk0;
   const int blk_per = (nblk + splits - 1) / splits;
-  const int c0 = min(len, split * blk_per * block_size);
-  const int c1 = min(len, (split + 1) * blk_per * block_size);
+  int c0 = min(len, (blk0 + split * blk_per) * block_size);
+  const int c1 = min(len, (blk0 + (split + 1) * blk_per) * block_size);
+  if (EXT) c0 = max(c0, vis0 / kAttnStageTok * kAttnStageTok);
   const int nchunk = (c1 - c0 + kAttnStageTok - 1) / kAttnStageTok;
   const int my_chunks = nchunk > warp ? (nchunk - warp + kAttnWarps - 1) / kAttnWarps : 0;
   const long long tok_stride = static_cast<long long>(n_kv) * HD;
@@ -189,14 +209,15 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
     }
     // row g: tokens tok0 + 2 tq + {0, 1} (s0) and tok0 + 8 + 2 tq + {0, 1} (s1)
     const int tk = tok0 + 2 * tq;
-    float p00 = tk < c1 ? s0[0] * scale_log2 : -INFINITY;
-    float p01 = tk + 1 < c1 ? s0[1] * scale_log2 : -INFINITY;
-    float p10 = tk + 8 < c1 ? s1[0] * scale_log2 : -INFINITY;
-    float p11 = tk + 9 < c1 ? s1[1] * scale_log2 : -INFINITY;
+    auto seen = [&](int j) { return j < c1 && (!EXT || j >= vis0); };
+    float p00 = seen(tk) ? attn_score<EXT>(s0[0], scale_log2, ext) : -INFINITY;
+    float p01 = seen(tk + 1) ? attn_score<EXT>(s0[1], scale_log2, ext) : -INFINITY;
+    float p10 = seen(tk + 8) ? attn_score<EXT>(s1[0], scale_log2, ext) : -INFINITY;
+    float p11 = seen(tk + 9) ? attn_score<EXT>(s1[1], scale_log2, ext) : -INFINITY;
     float mx = fmaxf(fmaxf(p00, p01), fmaxf(p10, p11));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-    const float mn = fmaxf(m, mx);                     // finite: token tok0 itself is always valid
+    const float mn = fmaxf(m, mx);                     // finite: every chunk holds a visible token
     const float corr = exp2f(m - mn);
     p00 = exp2f(p00 - mn); p01 = exp2f(p01 - mn); p10 = exp2f(p10 - mn); p11 = exp2f(p11 - mn);
     float ls = p00 + p01 + p10 + p11;
@@ -207,6 +228,7 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
 #pragma unroll
     for (int i = 0; i < NT; ++i) { o[i][0] *= corr; o[i][1] *= corr; }
     uint32_t pa[4] = {pack_bf16(p00, p01), 0u, pack_bf16(p10, p11), 0u};
+    const uint32_t pl[4] = {pack_bf16(bf16_rest(p00), bf16_rest(p01)), 0u, pack_bf16(bf16_rest(p10), bf16_rest(p11)), 0u};
     {
       const int r = (lm_mi & 1) * 8 + lm_r;
 #pragma unroll
@@ -216,6 +238,10 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
         ldmatrix_x4_trans(vb + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
         mma_bf16_16816(o[2 * dp], pa, b0, b1);
         mma_bf16_16816(o[2 * dp + 1], pa, b2, b3);
+        if (EXT) {
+          mma_bf16_16816(o[2 * dp], pl, b0, b1);
+          mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
+        }
       }
     }
     __syncwarp();   // every lane is done with this ring slot before it is refilled
@@ -295,12 +321,12 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
 constexpr int kPreKeys = 64;       // keys per pipeline stage
 constexpr int kPreRows = 64;       // query rows per CTA (4 warps x 16)
 
-template <int HD, int GQ>
+template <int HD, int GQ, bool EXT>
 __global__ void __launch_bounds__(128)
 prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ kcache,
                     const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_blocks,
                     const int4* __restrict__ tiles, int block_size, int n_kv, float scale_log2,
-                    __nv_bfloat16* __restrict__ out, long long ld_out) {
+                    __nv_bfloat16* __restrict__ out, long long ld_out, AttnExt ext) {
   constexpr int ROWB = HD * 2;
   constexpr int NCH = HD / 8;                       // 16-byte chunks per K / V row
   constexpr int TILEB = kPreKeys * ROWB;
@@ -318,6 +344,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   const int* bt = block_tables + static_cast<long long>(tile.z) * max_blocks;
   const int kmax = pos0 + ntok;                     // keys [0, kmax) exist for the last token of the tile
   const int nkb = (kmax + kPreKeys - 1) / kPreKeys;
+  const int kb0 = EXT && ext.window > 0 ? max(0, pos0 - ext.window + 1) / kPreKeys : 0;   // first block anyone sees
   const long long tok_stride = static_cast<long long>(n_kv) * HD;
   const uint32_t sbase = smem_u32(s_pre);
 
@@ -342,7 +369,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
     }
     cp_async_commit();
   };
-  issue(0);
+  issue(kb0);
 
   // Q fragments: this warp's rows R0 = warp * 16 + g and R0 + 8; row R = (token R / GQ, head R % GQ)
   const int R0 = warp * 16 + g, R1 = R0 + 8;
@@ -368,15 +395,19 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   const int lm_mi = lane >> 3, lm_r = lane & 7;
   // the warp's last query position: key blocks entirely behind it are skipped by this warp (causal)
   const int wlast = pos0 + min(ntok - 1, (warp * 16 + 15) / GQ);
+  // and, with a window, those entirely before the reach of its first query; a row's first visible key
+  const int wfirst = EXT && ext.window > 0 ? pos0 + warp * 16 / GQ - ext.window + 1 : 0;
+  const int lo0 = EXT && ext.window > 0 ? qpos0 - ext.window + 1 : 0;
+  const int lo1 = EXT && ext.window > 0 ? qpos1 - ext.window + 1 : 0;
 
-  for (int kb = 0; kb < nkb; ++kb) {
+  for (int kb = kb0; kb < nkb; ++kb) {
     issue(kb + 1);
     cp_async_wait<1>();
     __syncthreads();
     const uint32_t kbuf = sbase + (kb & 1) * STAGEB;
     const uint32_t vbuf = kbuf + TILEB;
     const int key0 = kb * kPreKeys;
-    if (key0 <= wlast && warp * 16 / GQ < ntok) {
+    if (key0 <= wlast && warp * 16 / GQ < ntok && (!EXT || key0 + kPreKeys > wfirst)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
@@ -397,10 +428,12 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         const int k0 = key0 + nt * 8 + 2 * tq;
-        s[nt][0] = (v0 && k0 <= qpos0) ? s[nt][0] * scale_log2 : -INFINITY;
-        s[nt][1] = (v0 && k0 + 1 <= qpos0) ? s[nt][1] * scale_log2 : -INFINITY;
-        s[nt][2] = (v1 && k0 <= qpos1) ? s[nt][2] * scale_log2 : -INFINITY;
-        s[nt][3] = (v1 && k0 + 1 <= qpos1) ? s[nt][3] * scale_log2 : -INFINITY;
+        const bool a0 = v0 && k0 <= qpos0 && (!EXT || k0 >= lo0), a1 = v0 && k0 + 1 <= qpos0 && (!EXT || k0 + 1 >= lo0);
+        const bool b0 = v1 && k0 <= qpos1 && (!EXT || k0 >= lo1), b1 = v1 && k0 + 1 <= qpos1 && (!EXT || k0 + 1 >= lo1);
+        s[nt][0] = a0 ? attn_score<EXT>(s[nt][0], scale_log2, ext) : -INFINITY;
+        s[nt][1] = a1 ? attn_score<EXT>(s[nt][1], scale_log2, ext) : -INFINITY;
+        s[nt][2] = b0 ? attn_score<EXT>(s[nt][2], scale_log2, ext) : -INFINITY;
+        s[nt][3] = b1 ? attn_score<EXT>(s[nt][3], scale_log2, ext) : -INFINITY;
         mx0 = fmaxf(mx0, fmaxf(s[nt][0], s[nt][1]));
         mx1 = fmaxf(mx1, fmaxf(s[nt][2], s[nt][3]));
       }
@@ -435,6 +468,13 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
       for (int kg = 0; kg < 4; ++kg) {
         const uint32_t pa[4] = {pack_bf16(s[2 * kg][0], s[2 * kg][1]), pack_bf16(s[2 * kg][2], s[2 * kg][3]),
                                 pack_bf16(s[2 * kg + 1][0], s[2 * kg + 1][1]), pack_bf16(s[2 * kg + 1][2], s[2 * kg + 1][3])};
+        uint32_t pl[4] = {0u, 0u, 0u, 0u};
+        if (EXT) {
+          pl[0] = pack_bf16(bf16_rest(s[2 * kg][0]), bf16_rest(s[2 * kg][1]));
+          pl[1] = pack_bf16(bf16_rest(s[2 * kg][2]), bf16_rest(s[2 * kg][3]));
+          pl[2] = pack_bf16(bf16_rest(s[2 * kg + 1][0]), bf16_rest(s[2 * kg + 1][1]));
+          pl[3] = pack_bf16(bf16_rest(s[2 * kg + 1][2]), bf16_rest(s[2 * kg + 1][3]));
+        }
         const int r = kg * 16 + (lm_mi & 1) * 8 + lm_r;
 #pragma unroll
         for (int dp = 0; dp < NT / 2; ++dp) {
@@ -443,6 +483,10 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
           ldmatrix_x4_trans(vbuf + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
           mma_bf16_16816(o[2 * dp], pa, b0, b1);
           mma_bf16_16816(o[2 * dp + 1], pa, b2, b3);
+          if (EXT) {
+            mma_bf16_16816(o[2 * dp], pl, b0, b1);
+            mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
+          }
         }
       }
     }
@@ -465,43 +509,52 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   }
 }
 
-template <int HD, int GQ>
+// Options of a launch as the kernels take them (softcap <= 0: none; window <= 0: every key).
+static AttnExt make_ext(float scale, int window, float softcap) {
+  AttnExt x;
+  x.window = window > 0 ? window : 0;
+  x.cap_in = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
+  x.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  return x;
+}
+
+template <int HD, int GQ, bool EXT>
 static int launch_prefill(const void* q, long long ld_q, const void* kc, const void* vc, const int* bt, int max_blocks,
                           const void* tiles, int n_tiles, int block_size, int n_kv, float scale, void* out,
-                          long long ld_out, cudaStream_t stream) {
+                          long long ld_out, AttnExt ext, cudaStream_t stream) {
   const size_t smem = 2 * 2 * static_cast<size_t>(kPreKeys) * HD * 2;
   static PerDeviceOnce configured;
   const int crc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(prefill_attn_kernel<HD, GQ>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return static_cast<int>(cudaFuncSetAttribute(prefill_attn_kernel<HD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  96 * 1024));
   });
   if (crc != 0) return crc;
   dim3 grid(n_tiles, n_kv);
-  prefill_attn_kernel<HD, GQ><<<grid, 128, smem, stream>>>(
+  prefill_attn_kernel<HD, GQ, EXT><<<grid, 128, smem, stream>>>(
       static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kc),
       static_cast<const __nv_bfloat16*>(vc), bt, max_blocks, static_cast<const int4*>(tiles), block_size, n_kv,
-      scale * 1.4426950408889634f, static_cast<__nv_bfloat16*>(out), ld_out);
+      scale * 1.4426950408889634f, static_cast<__nv_bfloat16*>(out), ld_out, ext);
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int HD, int GQ>
+template <int HD, int GQ, bool EXT>
 static int launch_attn(const void* q, long long ld_q, const void* kc, const void* vc, const int* bt, int max_blocks,
                        const int* bt_row, const int* ctx_len, int block_size, int T, int n_kv, float scale, int splits,
-                       void* out, long long ld_out, float* part_o, float* part_lse, cudaStream_t stream) {
+                       void* out, long long ld_out, float* part_o, float* part_lse, AttnExt ext, cudaStream_t stream) {
   const size_t merge_b = static_cast<size_t>(kAttnWarps) * GQ * HD * sizeof(float);
   const size_t ring_b = static_cast<size_t>(kAttnWarps) * kAttnStages * 2 * kAttnStageTok * HD * 2;
   const size_t smem = merge_b > ring_b ? merge_b : ring_b;
   static PerDeviceOnce configured;
   const int crc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(paged_attn_kernel<HD, GQ>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return static_cast<int>(cudaFuncSetAttribute(paged_attn_kernel<HD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  160 * 1024));
   });
   if (crc != 0) return crc;
   dim3 grid(T, n_kv, splits);
-  cudaError_t e = launch_kernel(paged_attn_kernel<HD, GQ>, grid, dim3(kAttnThreads), smem, stream,
+  cudaError_t e = launch_kernel(paged_attn_kernel<HD, GQ, EXT>, grid, dim3(kAttnThreads), smem, stream,
       static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kc),
       static_cast<const __nv_bfloat16*>(vc), bt, max_blocks, bt_row, ctx_len, block_size, n_kv,
-      scale * 1.4426950408889634f, splits, static_cast<__nv_bfloat16*>(out), ld_out, part_o, part_lse);
+      scale * 1.4426950408889634f, splits, static_cast<__nv_bfloat16*>(out), ld_out, part_o, part_lse, ext);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (splits > 1) {
     dim3 g2(T, n_kv * GQ);
@@ -521,20 +574,21 @@ extern "C" long long dmoe_paged_attention_workspace_floats(int T, int n_q, int h
   return static_cast<long long>(T) * n_q * splits * (hd + 1);
 }
 
-extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, const void* vcache,
-                                    const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
-                                    int block_size, int T, int n_q, int n_kv, int hd, float scale, int splits, void* out,
-                                    long long ld_out, float* workspace, void* stream_) {
-  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+// Instantiations by head size, query group and options; -11: no tensor-core kernel for this shape.
+template <bool EXT>
+static int attn_dispatch(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
+                         int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
+                         int hd, float scale, int splits, void* out, long long ld_out, float* workspace, AttnExt ext,
+                         cudaStream_t stream) {
   if (T == 0) return 0;
   if (n_kv < 1 || n_q % n_kv != 0 || splits < 1 || splits > 65535 || n_kv > 65535 || block_size % kAttnStageTok != 0) return -10;
   if (splits > 1 && workspace == nullptr) return -12;
   const int gq = n_q / n_kv;
   float* part_o = workspace;
   float* part_lse = workspace != nullptr ? workspace + static_cast<long long>(T) * n_q * splits * hd : nullptr;
-#define DMOE_ATTN(HD_, GQ_)                                                                                        \
-  return launch_attn<HD_, GQ_>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, \
-                               n_kv, scale, splits, out, ld_out, part_o, part_lse, stream)
+#define DMOE_ATTN(HD_, GQ_)                                                                                             \
+  return launch_attn<HD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, \
+                                    n_kv, scale, splits, out, ld_out, part_o, part_lse, ext, stream)
   if (hd == 128) {
     switch (gq) {
       case 1: DMOE_ATTN(128, 1);
@@ -554,6 +608,26 @@ extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* k
   return -11;
 }
 
+extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, const void* vcache,
+                                    const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
+                                    int block_size, int T, int n_q, int n_kv, int hd, float scale, int splits, void* out,
+                                    long long ld_out, float* workspace, void* stream_) {
+  return attn_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
+                              hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0.f),
+                              static_cast<cudaStream_t>(stream_));
+}
+
+// The same with a sliding window and a score soft cap (0 = without).
+extern "C" int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
+                                        const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
+                                        int block_size, int T, int n_q, int n_kv, int hd, float scale, int window,
+                                        float softcap, int splits, void* out, long long ld_out, float* workspace,
+                                        void* stream_) {
+  return attn_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
+                             hd, scale, splits, out, ld_out, workspace, make_ext(scale, window, softcap),
+                             static_cast<cudaStream_t>(stream_));
+}
+
 // Tokens per tile of dmoe_prefill_attention for a query group of n_q / n_kv heads.
 extern "C" int dmoe_prefill_tile_tokens(int n_q, int n_kv) {
   if (n_kv < 1 || n_q % n_kv != 0) return 0;
@@ -561,17 +635,16 @@ extern "C" int dmoe_prefill_tile_tokens(int n_q, int n_kv) {
   return (gq == 1 || gq == 2 || gq == 4 || gq == 8) ? kPreRows / gq : 0;
 }
 
-extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void* kcache, const void* vcache,
-                                      const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
-                                      int block_size, int n_q, int n_kv, int hd, float scale, void* out, long long ld_out,
-                                      void* stream_) {
-  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+template <bool EXT>
+static int prefill_dispatch(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
+                            int max_blocks, const void* tiles, int n_tiles, int block_size, int n_q, int n_kv, int hd,
+                            float scale, void* out, long long ld_out, AttnExt ext, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   if (n_kv < 1 || n_q % n_kv != 0 || n_kv > 65535 || n_tiles < 0 || block_size < 1 || tiles == nullptr) return -10;
   const int gq = n_q / n_kv;
-#define DMOE_PRE(HD_, GQ_)                                                                                     \
-  return launch_prefill<HD_, GQ_>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, \
-                                  n_kv, scale, out, ld_out, stream)
+#define DMOE_PRE(HD_, GQ_)                                                                                          \
+  return launch_prefill<HD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, \
+                                       n_kv, scale, out, ld_out, ext, stream)
   if (hd == 128) {
     switch (gq) {
       case 1: DMOE_PRE(128, 1);
@@ -589,4 +662,113 @@ extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void*
   }
 #undef DMOE_PRE
   return -11;
+}
+
+extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void* kcache, const void* vcache,
+                                      const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
+                                      int block_size, int n_q, int n_kv, int hd, float scale, void* out, long long ld_out,
+                                      void* stream_) {
+  return prefill_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
+                                 hd, scale, out, ld_out, make_ext(scale, 0, 0.f), static_cast<cudaStream_t>(stream_));
+}
+
+extern "C" int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
+                                          const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
+                                          int block_size, int n_q, int n_kv, int hd, float scale, int window,
+                                          float softcap, void* out, long long ld_out, void* stream_) {
+  return prefill_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
+                                hd, scale, out, ld_out, make_ext(scale, window, softcap),
+                                static_cast<cudaStream_t>(stream_));
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Attention of any shape in fp32 arithmetic on the CUDA cores (key size, value size and query group free; bf16 or fp32
+// cache): the fp32 configuration, and head shapes without a tensor-core kernel. One CTA per (token, query head) walks
+// the visible keys 128 at a time: one score per thread, online softmax, then one value column per thread.
+namespace dmoe {
+
+constexpr int kAnyKeys = 128;
+
+template <typename T>
+__global__ void __launch_bounds__(kAnyKeys)
+any_attn_kernel(const T* __restrict__ q, long long ld_q, const T* __restrict__ kcache, const T* __restrict__ vcache,
+                const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ bt_row,
+                const int* __restrict__ ctx_len, int block_size, int n_q, int n_kv, int dk, int dv, float scale, int window,
+                float softcap, T* __restrict__ out, long long ld_out) {
+  extern __shared__ float s_any[];          // q [dk] | acc [dv]
+  __shared__ float s_p[kAnyKeys];
+  __shared__ long long s_slot[kAnyKeys];
+  __shared__ float s_red[2][kAnyKeys / 32];
+  float* s_q = s_any;
+  float* s_acc = s_any + dk;
+  const int t = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+  const int hkv = head / (n_q / n_kv);
+  const int len = ctx_len[t];
+  const int* bt = block_tables + static_cast<long long>(bt_row != nullptr ? bt_row[t] : t) * max_blocks;
+  for (int d = tid; d < dk; d += kAnyKeys) s_q[d] = static_cast<float>(q[t * ld_q + head * dk + d]);
+  for (int d = tid; d < dv; d += kAnyKeys) s_acc[d] = 0.f;
+  __syncthreads();
+  float m = -INFINITY, l = 0.f;
+  for (int j0 = window > 0 ? max(0, len - window) : 0; j0 < len; j0 += kAnyKeys) {
+    const int n = min(kAnyKeys, len - j0);
+    float s = -INFINITY;
+    if (tid < n) {
+      const int j = j0 + tid;
+      const long long slot = static_cast<long long>(bt[j / block_size]) * block_size + j % block_size;
+      const T* kr = kcache + (slot * n_kv + hkv) * dk;
+      float acc = 0.f;
+      for (int d = 0; d < dk; ++d) acc += s_q[d] * static_cast<float>(kr[d]);
+      s = acc * scale;
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      s_slot[tid] = slot;
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    if ((tid & 31) == 0) s_red[0][tid >> 5] = mx;
+    __syncthreads();
+    mx = fmaxf(fmaxf(s_red[0][0], s_red[0][1]), fmaxf(s_red[0][2], s_red[0][3]));
+    const float mn = fmaxf(m, mx);           // finite: a tile has at least one key
+    const float p = tid < n ? expf(s - mn) : 0.f;
+    s_p[tid] = p;
+    float ps = p;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+    if ((tid & 31) == 0) s_red[1][tid >> 5] = ps;
+    __syncthreads();
+    const float corr = expf(m - mn);
+    l = l * corr + (s_red[1][0] + s_red[1][1] + s_red[1][2] + s_red[1][3]);
+    m = mn;
+    for (int d = tid; d < dv; d += kAnyKeys) {
+      float acc = s_acc[d] * corr;
+      for (int j = 0; j < n; ++j) acc += s_p[j] * static_cast<float>(vcache[(s_slot[j] * n_kv + hkv) * dv + d]);
+      s_acc[d] = acc;
+    }
+    __syncthreads();
+  }
+  for (int d = tid; d < dv; d += kAnyKeys)
+    out[t * ld_out + head * dv + d] = static_cast<T>(l > 0.f ? s_acc[d] / l : 0.f);
+}
+
+}  // namespace dmoe
+
+extern "C" int dmoe_any_attention(int is_f32, const void* q, long long ld_q, const void* kcache, const void* vcache,
+                                  const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
+                                  int block_size, int T, int n_q, int n_kv, int dk, int dv, float scale, int window,
+                                  float softcap, void* out, long long ld_out, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (T == 0) return 0;
+  if (n_kv < 1 || n_q % n_kv != 0 || n_q > 65535 || block_size < 1 || dk < 1 || dv < 1 || dk + dv > 8192) return -10;
+  const dim3 grid(T, n_q);
+  const size_t smem = static_cast<size_t>(dk + dv) * sizeof(float);
+  if (is_f32)
+    any_attn_kernel<float><<<grid, kAnyKeys, smem, stream>>>(
+        static_cast<const float*>(q), ld_q, static_cast<const float*>(kcache), static_cast<const float*>(vcache), block_tables,
+        max_blocks, bt_row, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, softcap, static_cast<float*>(out), ld_out);
+  else
+    any_attn_kernel<__nv_bfloat16><<<grid, kAnyKeys, smem, stream>>>(
+        static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kcache),
+        static_cast<const __nv_bfloat16*>(vcache), block_tables, max_blocks, bt_row, ctx_len, block_size, n_q, n_kv, dk, dv,
+        scale, window, softcap, static_cast<__nv_bfloat16*>(out), ld_out);
+  return static_cast<int>(cudaGetLastError());
 }

@@ -108,6 +108,22 @@ int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, cons
                          int T, int n_q, int n_kv, int hd, float scale, int splits, void* out, long long ld_out,
                          float* workspace, void* stream);
 
+// With a sliding window (a query sees the last `window` tokens, itself included; 0 = all) and a score soft cap
+// (cap * tanh(score / cap); 0 = none).
+int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
+                             int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
+                             int hd, float scale, int window, float softcap, int splits, void* out, long long ld_out,
+                             float* workspace, void* stream);
+int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
+                               const int* block_tables, int max_blocks, const void* tiles, int n_tiles, int block_size,
+                               int n_q, int n_kv, int hd, float scale, int window, float softcap, void* out,
+                               long long ld_out, void* stream);
+// Any key / value size and query group, bf16 or fp32 cache, fp32 arithmetic on the CUDA cores.
+int dmoe_any_attention(int is_f32, const void* q, long long ld_q, const void* kcache, const void* vcache,
+                       const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T,
+                       int n_q, int n_kv, int dk, int dv, float scale, int window, float softcap, void* out,
+                       long long ld_out, void* stream);
+
 // Tiled causal attention for prompt tokens: CTA column i handles tiles[i] = int4 {first row in q / out, tokens
 // (<= dmoe_prefill_tile_tokens), block-table row, position of the first token}; the tokens of a tile are consecutive
 // rows at consecutive positions of one sequence, whose K / V (own tokens included) are already in the paged cache.
@@ -115,6 +131,59 @@ int dmoe_prefill_tile_tokens(int n_q, int n_kv);
 int dmoe_prefill_attention(const void* q, long long ld_q, const void* kcache, const void* vcache,
                            const int* block_tables, int max_blocks, const void* tiles, int n_tiles, int block_size,
                            int n_q, int n_kv, int hd, float scale, void* out, long long ld_out, void* stream);
+
+// ---- fp32-residual decoders (layer_ops.cu); is_f32: fp32 activations instead of bf16 -----------------------
+// out[t] = table[ids[t]] * scale (fp32)
+int dmoe_embed_f32(const int* ids, const void* table, int is_f32, float scale, float* out, int T, int W, int vocab, void* stream);
+// x = resid[r] + norm(y[r]) * post (y may be NULL: x = resid[r]); resid[r] = x unless a row table picks r = rows[i];
+// h[i] = norm(x) * pre * out_scale (h may be NULL); norm(v) = v / sqrt(mean(v^2) + eps). resid fp32 [.., W].
+int dmoe_resid_norm(int is_f32, float* resid, const void* y, long long ld_y, const float* post, const float* pre,
+                    float out_scale, float eps, const int* rows, void* h, long long ld_h, int n, int W, void* stream);
+// float2 table [max_pos][half] = (cos, sin)(pos * freq[i]) * mscale, freq in double on the device
+int dmoe_rope_freq_table(void* table, int max_pos, int half, const double* freq, float mscale, void* stream);
+// Per-head RMS norm of q and k, rotation of pairs (i, i + rot / 2), i < rot / 2, q in place, k / v into the paged caches.
+int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots, void* kcache,
+                      void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, const void* table, int max_pos,
+                      const float* qw, const float* kw, float eps, void* stream);
+int dmoe_silu_mul(int is_f32, const void* gu, long long ld, void* out, long long ld_out, int T, int I, void* stream);
+// Y = X W^T on the CUDA cores in fp32 arithmetic: fp32 operands, or bf16 operands of any alignment.
+int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y, long long ldy,
+                     int T, int F, int K, void* stream);
+
+// ---- linear recurrences with a matrix state per head (recurrent.cu) ---------------------------------------
+typedef struct DmoeRecur {
+  const void* q;            // [rows, kv_heads * dim], row stride ldq; raw projections where taps > 0
+  const void* k;
+  const void* v;            // [rows, heads * vdim]
+  const void* gate;         // [rows, heads * vdim] output gate before its activation
+  const void* beta;         // delta: [rows, heads] write strength before its sigmoid
+  const float* z;           // [rows, heads * dim] decay logits without their bias
+  const float* z_bias;      // [heads * dim]
+  const float* a_log;       // [heads], decay_kind 1
+  const float* conv_w;      // [2 kv_heads dim + heads vdim, taps], last column = current token
+  void* ring;               // [n_slots, taps, channels]: the last inputs of the convolution, by position modulo taps
+  const void* segs;         // int4 {first row, tokens, slot, first position}; NULL (decode step): segment i is row i at
+  const int* positions;     // position positions[i] of the sequence in slot rows[i], skipped where kv_slots[i] < 0
+  const int* rows;
+  const long long* kv_slots;
+  float* state;             // [n_slots, heads, dim, vdim]
+  const float* norm_w;      // [vdim]
+  void* out;                // [rows, heads * vdim]
+  float* raw;               // read-outs before norm and gate
+  long long ldq, ldk, ldv, ldg, ldb, ldz, ldo, ldraw;
+  int n_segs, n_slots, heads, kv_heads, dim, vdim, taps;
+  int delta;                // 0: plain write, 1: delta rule (q and k are made unit vectors)
+  int decay_kind;           // 0: log a = log sigmoid(z + b) * inv_tau, 1: log a = -exp(a_log) softplus(z + b)
+  int gate_kind;            // 0: silu, 1: sigmoid
+  int is_f32;
+  float qscale, inv_tau, eps;
+} DmoeRecur;
+int dmoe_recur_value_tile(int dim, int vdim);
+int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream);
+int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw, const void* gate,
+                   long long ldg, const float* norm_w, float eps, int gate_kind, void* out, long long ldo, int heads, int V,
+                   void* stream);
+int dmoe_conv_chunks(const DmoeRecur* a, const void* chunks, int n_chunks, void* out, long long ldo, void* stream);
 
 // ---- routing (moe.cu) -------------------------------------------------------------------------------
 // (RMSNorm ->) gate -> softmax -> top-k (-> renormalise); counts[e] += tokens routed to e (may be NULL).

@@ -1,0 +1,148 @@
+"""Whole-iteration executor of layer-list decoders (:class:`disagmoe_b200.config.LayerListConfig`).
+
+    embed * scale -> per layer [ norm -> mixer -> norm + add (-> norm -> gated feed-forward -> norm + add) ]
+                  -> norm -> head -> argmax
+
+The residual stream is fp32; the norm after a sublayer, the residual add and the norm before the next sublayer are one
+launch. Two kinds of per-sequence memory: KV pages for the attention layers that have keys and values of their own (layers
+that read another layer's have none), and for recurrent layers one state slot per sequence, numbered like its row of the
+block table, so the block manager's row allocation is the slot allocation. As in the MoE executor, a decode iteration is
+one chain of launches captured per batch-size bucket, prompts run eagerly, and CPU tensors run the PyTorch restatements.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Optional, Tuple
+
+import torch
+
+from ..config import AttentionSpec
+from ..models import weights as W
+from ..models.mixers import GatedFeedForward, StepMeta, make_mixer
+from ..ops import functional as F
+from ..ops import gemm
+from ..ops.recurrent import MAX_TAPS, RecurrentState, SegmentTables, build_segments, decode_segments
+from .step import StepExecutor, TokenBuffers
+
+
+class LayerListBuffers(TokenBuffers):
+    def __init__(self, cfg, cap: int, device, logit_rows: int):
+        super().__init__(cfg, cap, device, logit_rows)
+        self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=device)
+        self.segments: Optional[SegmentTables] = None        # None: decode step, every row its own segment
+        self.prefill_tiles: Dict[int, Tuple[torch.Tensor, int]] = {}    # tokens per tile -> (table, tiles)
+        self.ctx_len_decode: Optional[torch.Tensor] = None
+        self.n_untiled = 0
+
+
+class LayerListExecutor(StepExecutor):
+    def _load(self, state_dict: Optional[W.StateDict]) -> None:
+        cfg, dev, dt = self.cfg, self.device, self.dtype
+        assert self.layer_ids == list(range(cfg.num_layers)), "a layer-list decoder runs whole"
+        if any(getattr(l.mixer, "conv", 0) > MAX_TAPS for l in cfg.layers):
+            raise ValueError(f"short convolutions longer than {MAX_TAPS} taps are not supported")
+        # without a checkpoint: seeded random weights, created on the device tensor by tensor
+        sd = state_dict if state_dict is not None else W.init_state_dict(cfg, dev, dt)
+        one_plus = lambda n: (1.0 + sd[n].to(device=dev, dtype=torch.float32)).contiguous()
+        self.embed_w = sd["embed"].to(device=dev, dtype=dt).contiguous()
+        self.head_w = sd["head"].to(device=dev, dtype=dt).contiguous()
+        self.final_norm = one_plus("final.norm")
+        self.mixers, self.ffs, self.norms = [], [], []
+        for i, layer in enumerate(cfg.layers):
+            m = make_mixer(cfg, i, dev, dt)
+            m.load_weights(sd)
+            self.mixers.append(m)
+            self.ffs.append(GatedFeedForward(sd, f"l{i}.mlp.", dev, dt) if layer.ff else None)
+            self.norms.append({n: one_plus(f"l{i}.{n}") for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.ff else ())})
+
+    # ---- cache and state ------------------------------------------------------------------------------------------
+    def _owns_kv(self, i: int) -> bool:
+        m = self.cfg.layers[i].mixer
+        return isinstance(m, AttentionSpec) and m.kv_from is None
+
+    def _cache_bytes_per_block(self) -> int:
+        el = torch.empty((), dtype=self.dtype).element_size()
+        return sum(self.block_size * m.kv_heads * (m.dim + m.vdim) * el
+                   for i, m in enumerate(l.mixer for l in self.cfg.layers) if self._owns_kv(i))
+
+    def _allocate_cache(self) -> None:
+        z = lambda *s: torch.zeros(*s, dtype=self.dtype, device=self.device)
+        self.kv: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
+        self.states: Dict[int, RecurrentState] = {}
+        for i, layer in enumerate(self.cfg.layers):
+            m = layer.mixer
+            if self._owns_kv(i):
+                self.kv[i] = tuple(z(self.num_blocks, self.block_size, m.kv_heads, d) for d in (m.dim, m.vdim))
+            elif isinstance(m, AttentionSpec):
+                self.kv[i] = self.kv[m.kv_from]
+            else:
+                self.states[i] = self.mixers[i].recur.new_state(self.max_batch_size, self.dtype, self.device)
+
+    def state_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for s in self.states.values() for t in s.tensors())
+
+    def export_sequence(self, blocks: List[int], row: int) -> dict:
+        idx = torch.tensor(blocks, device=self.device)
+        return dict(pages=[t[idx].cpu() for i in sorted(self.kv) if self._owns_kv(i) for t in self.kv[i]],
+                    state=[t[row].cpu() for i in sorted(self.states) for t in self.states[i].tensors()])
+
+    def import_sequence(self, blocks: List[int], row: int, data: dict) -> None:
+        caches = [t for i in sorted(self.kv) if self._owns_kv(i) for t in self.kv[i]]
+        for t, p in zip(caches, data["pages"]):
+            n = min(p.shape[0], len(blocks))
+            t[torch.tensor(blocks[:n], device=self.device)] = p[:n].to(self.device)
+        for t, s in zip((t for i in sorted(self.states) for t in self.states[i].tensors()), data["state"]):
+            t[row] = s.to(self.device)
+
+    def _make_buffers(self, cap: int) -> LayerListBuffers:
+        # prompts sample one row per sequence; a step that wants more rows allocates its logits
+        return LayerListBuffers(self.cfg, cap, self.device, min(cap, self.max_batch_size))
+
+    # ---- one iteration ----------------------------------------------------------------------------------------------
+    def _begin_prefill(self, buf: LayerListBuffers, T: int, positions, ctx_len, bt_row) -> None:
+        buf.segments = build_segments(bt_row, positions, self.device)
+        buf.prefill_tiles, buf.ctx_len_decode, buf.n_untiled = {}, None, T
+        if self.device.type != "cuda":
+            return
+        for m in (l.mixer for l in self.cfg.layers):
+            if not isinstance(m, AttentionSpec) or not F.attention_on_tensor_cores(self.dtype, m.heads, m.kv_heads, m.dim, m.vdim):
+                continue
+            n = F.prefill_tile_tokens(m.heads, m.kv_heads)
+            if n in buf.prefill_tiles:
+                continue
+            tiles, covered = F.build_prefill_tiles(bt_row, positions, n)
+            if len(tiles):
+                buf.prefill_tiles[n] = (tiles.to(self.device), len(tiles))
+                cd = torch.as_tensor(ctx_len).clone()
+                cd[covered] = 0              # which rows are tiled does not depend on the tile size
+                buf.ctx_len_decode, buf.n_untiled = cd.to(self.device), int((~covered).sum())
+
+    def _end_prefill(self, buf: LayerListBuffers) -> None:
+        buf.segments, buf.prefill_tiles, buf.ctx_len_decode = None, {}, None
+
+    def _forward(self, buf: LayerListBuffers, T: int, max_ctx: int, want_logits: bool):
+        cfg, eps, dt = self.cfg, self.cfg.rms_norm_eps, self.dtype
+        pos, slots, rows = buf.positions[:T], buf.slots[:T], buf.bt_row[:T]
+        segs = buf.segments if buf.segments is not None else decode_segments(pos, rows, slots)
+        meta = StepMeta(pos, slots, self.block_tables, rows, buf.ctx_len[:T], max_ctx=max_ctx,
+                        num_decode_tokens=buf.n_untiled if buf.segments is not None else T,
+                        prefill_tiles=buf.prefill_tiles if buf.segments is not None else None,
+                        ctx_len_decode=buf.ctx_len_decode, segments=segs)
+        resid = buf.resid[:T]
+        F.embed_f32(buf.ids[:T], self.embed_w, cfg.embed_scale, resid)
+        h = F.resid_norm(resid, None, None, self.norms[0]["norm1"], eps, dt)
+        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
+            last = i + 1 == len(self.mixers)
+            y, post = mixer(h, self.states[i] if i in self.states else self.kv[i], meta), n["norm1b"]
+            if ff is not None:
+                h = F.resid_norm(resid, y, post, n["norm2"], eps, dt)
+                y, post = ff(h), n["norm2b"]
+            if last:
+                # the head's input carries the logit scale; only the rows that are sampled get that far
+                h = F.resid_norm(resid, y, post, self.final_norm, eps, dt, out_scale=cfg.logit_scale, rows=buf.out_rows)
+            else:
+                h = F.resid_norm(resid, y, post, self.norms[i + 1]["norm1"], eps, dt)
+        n_out = h.shape[0]
+        logits = gemm.linear(h, self.head_w, out=buf.logits[:n_out] if n_out <= buf.logits.shape[0] else None,
+                             out_dtype=torch.float32)
+        F.argmax(logits, out=buf.next_ids[:n_out])
+        return buf.next_ids[:n_out], (logits if want_logits else None)

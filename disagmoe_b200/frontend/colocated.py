@@ -1,8 +1,9 @@
 """Single-GPU serving engine: every layer's attention and experts colocated on one device.
 
 The in-process counterpart of a one-worker ``ColocatePlacement`` deployment (reference: disagmoe/utils/placement.py:
-467-508, disagmoe/frontend/engine.py:873-904): continuous batching over the whole-iteration executor
-(:class:`disagmoe_b200.executor.fused.FusedModelExecutor`), the native paged-KV ``BlockManager`` with a
+467-508, disagmoe/frontend/engine.py:873-904): continuous batching over the whole-iteration executor that the model
+registry picks for the configuration (MoE decoders: :class:`disagmoe_b200.executor.fused.FusedModelExecutor`, layer-list
+decoders: :class:`disagmoe_b200.executor.layer_list.LayerListExecutor`), the native paged-KV ``BlockManager`` with a
 device-resident block table that is patched incrementally, pinned host staging for the per-step inputs and a
 device->host read of the sampled ids (the sampler lives on the host, as in the reference).
 """
@@ -10,13 +11,13 @@ from __future__ import annotations
 
 import time
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
 from .. import disagmoe_c as C
 from ..config import CacheConfig, ModelConfig
-from ..executor.fused import FusedModelExecutor
+from ..models.registry import make_executor
 from ..utils.constants import EOS_TOKEN_ID
 
 
@@ -41,15 +42,16 @@ class ColocatedEngine:
         self.device = torch.device(device)
         self.max_batch_size = max_batch_size
         self.ignore_eos = ignore_eos
-        self.executor = FusedModelExecutor(cfg, self.cache_cfg, device=device, dtype=dtype, max_batch_size=max_batch_size,
-                                           max_prefill_tokens=max_prefill_tokens, state_dict=state_dict,
-                                           num_blocks=num_blocks, enable_cuda_graph=enable_cuda_graph)
+        self.executor = make_executor(cfg, self.cache_cfg, device=device, dtype=dtype, max_batch_size=max_batch_size,
+                                      max_prefill_tokens=max_prefill_tokens, state_dict=state_dict,
+                                      num_blocks=num_blocks, enable_cuda_graph=enable_cuda_graph)
         self.block_size = self.cache_cfg.block_size
         self.block_mgr = C.BlockManager(self.block_size, self.executor.num_blocks - self.cache_cfg.num_reserved_blocks,
                                         self.cache_cfg.num_reserved_blocks, max_batch_size)
         self.waiting: List[_Seq] = []
         self.running: Dict[int, _Seq] = {}    # insertion ordered
         self.finished: Dict[int, _Seq] = {}
+        self.fed: Dict[int, int] = {}         # sequences driven by feed(): tokens cached so far
         pin = self.device.type == "cuda"
         B = max(max_batch_size, max_prefill_tokens)
         mk = lambda dt: torch.zeros(B, dtype=dt, pin_memory=pin)
@@ -96,6 +98,70 @@ class ColocatedEngine:
         return 3 * 8 * n
 
     # ---- steps --------------------------------------------------------------------------------------------------
+    def _execute(self, ids, pos, rows, slots, out_rows: Optional[List[int]] = None, decode_only: bool = False,
+                 want_logits: bool = False):
+        """One pass of the executor over a batch of rows (token ids, positions, block-table rows, KV slots): staging,
+        block-table patches, then the decode path (one token per sequence) or the general one. Returns device tensors
+        (next ids, logits or None) of ``out_rows``, or of every row."""
+        T = len(ids)
+        h2d = self._apply_block_table_patches()
+        self._h_ids.numpy()[:T] = ids
+        self._h_pos.numpy()[:T] = pos
+        self._h_ctx.numpy()[:T] = self._h_pos.numpy()[:T] + 1
+        self._h_row.numpy()[:T] = rows
+        self._h_slots.numpy()[:T] = slots
+        self.h2d_bytes_last += h2d + T * 24
+        args = (self._h_ids[:T], self._h_pos[:T], self._h_slots[:T], self._h_ctx[:T], self._h_row[:T])
+        if not decode_only:
+            return self.executor.prefill(*args, want_logits=want_logits, out_rows=out_rows)
+        nxt, logits = self.executor.decode(*args, want_logits=want_logits)
+        if out_rows is None or out_rows == list(range(T)):
+            return nxt, logits
+        pick = torch.tensor(out_rows, dtype=torch.long, device=nxt.device)
+        return nxt[pick], (logits[pick] if logits is not None else None)
+
+    def _slots(self, req_id: int, start: int, n: int) -> List[int]:
+        """KV slots of positions start .. start + n - 1 of a sequence."""
+        blocks, bs = self.block_mgr.get_seq_block_list(req_id), self.block_size
+        return [blocks[p // bs] * bs + p % bs for p in range(start, start + n)]
+
+    def feed(self, entries: Sequence[Tuple[int, Sequence[int], Sequence[int]]]) -> torch.Tensor:
+        """One engine step over given tokens instead of sampled ones: ``entries`` = (sequence id, its next tokens, places
+        among them whose logits are wanted); all entries run as one batch, portions of prompts beside single decode tokens,
+        from what earlier steps left in the cache and the state. Sequences are admitted at their first entry and hold their
+        pages and slot until :meth:`end_fed`. Returns the wanted logits [n, vocab] in the order of entries and places."""
+        if len(set(self.fed) | {sid for sid, _, _ in entries}) > self.max_batch_size:
+            raise ValueError(f"more than {self.max_batch_size} live sequences")
+        ids, pos, rows, slots, want = [], [], [], [], []
+        for sid, tokens, places in entries:
+            n, start = len(tokens), self.fed.get(sid)
+            if n == 0:
+                continue
+            if start is None:
+                start = 0
+                self.block_mgr.allocate(sid, n)
+            else:
+                self.block_mgr.append_tokens(sid, start, n)
+            want += [len(ids) + p for p in places]
+            ids += tokens
+            pos += range(start, start + n)
+            rows += [self.block_mgr.row_of(sid)] * n
+            slots += self._slots(sid, start, n)
+            self.fed[sid] = start + n
+        if not ids:
+            return torch.empty(0, self.cfg.vocab_size)
+        decode_only = all(len(tokens) <= 1 for _, tokens, _ in entries)
+        _, logits = self._execute(ids, pos, rows, slots, out_rows=want or [0], decode_only=decode_only, want_logits=True)
+        if self.device.type == "cuda":
+            torch.cuda.current_stream().synchronize()      # the staging buffers are free again
+        return logits[:len(want)]
+
+    def end_fed(self, seq_ids: Sequence[int]) -> None:
+        """Gives back the pages and slots of sequences driven by :meth:`feed`."""
+        for sid in seq_ids:
+            if self.fed.pop(sid, None) is not None:
+                self.block_mgr.release(sid)
+
     def _blocks(self, tokens: int) -> int:
         return (tokens + self.block_size - 1) // self.block_size
 
@@ -119,28 +185,24 @@ class ColocatedEngine:
             total += len(s.prompt)
         if not batch:
             return []
-        h2d = self._apply_block_table_patches()
-        i = 0
-        ends = []
+        ids, pos, rows, slots, ends = [], [], [], [], []
         for s in batch:
-            row = self.block_mgr.row_of(s.req_id)
-            for p, tok in enumerate(s.prompt):
-                self._h_ids[i], self._h_pos[i], self._h_ctx[i], self._h_row[i] = tok, p, p + 1, row
-                self._h_slots[i] = self.block_mgr.slot_of(s.req_id, p)
-                i += 1
-            ends.append(i - 1)
-        T = i
-        nxt, _ = ex.prefill(self._h_ids[:T], self._h_pos[:T], self._h_slots[:T], self._h_ctx[:T], self._h_row[:T])
+            n = len(s.prompt)
+            ids += s.prompt
+            pos += range(n)
+            rows += [self.block_mgr.row_of(s.req_id)] * n
+            slots += self._slots(s.req_id, 0, n)
+            ends.append(len(ids) - 1)
+        nxt, _ = self._execute(ids, pos, rows, slots, out_rows=ends)
         out = nxt.cpu()
         res = []
         now = time.time()
-        for s, e in zip(batch, ends):
+        for i, s in enumerate(batch):
             s.length = len(s.prompt)
-            tok = int(out[e])
+            tok = int(out[i])
             self._record(s, tok, now)
             res.append((s.req_id, tok))
-        self.h2d_bytes_last += h2d + T * 24
-        self.d2h_bytes_last += T * 4
+        self.d2h_bytes_last += len(batch) * 4
         return res
 
     def _record(self, s: _Seq, tok: int, now: float) -> None:
@@ -162,17 +224,11 @@ class ColocatedEngine:
             return []
         lens = [s.length for s in seqs]
         rs = self.block_mgr.step_decode([s.req_id for s in seqs], lens)
-        self._h_ids.numpy()[:B] = [s.last_token for s in seqs]
-        self._h_pos.numpy()[:B] = lens
-        self._h_ctx.numpy()[:B] = [l + 1 for l in lens]
-        self._h_row.numpy()[:B] = rs[:B]
-        self._h_slots.numpy()[:B] = rs[B:]
         ev = None
         if self.profile_events and self.device.type == "cuda":
             ev = (torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True))
             ev[0].record()
-        h2d = self._apply_block_table_patches()
-        nxt, _ = self.executor.decode(self._h_ids[:B], self._h_pos[:B], self._h_slots[:B], self._h_ctx[:B], self._h_row[:B])
+        nxt, _ = self._execute([s.last_token for s in seqs], lens, rs[:B], rs[B:], decode_only=True)
         self._h_out[:B].copy_(nxt, non_blocking=True)
         if ev is not None:
             ev[1].record()
@@ -186,7 +242,6 @@ class ColocatedEngine:
             s.length += 1
             self._record(s, tok, now)
             res.append((s.req_id, tok))
-        self.h2d_bytes_last += h2d + B * 24
         self.d2h_bytes_last += B * 4
         return res
 
@@ -208,14 +263,14 @@ class ColocatedEngine:
 
     # ---- serving-state snapshot ----------------------------------------------------------------------------------
     def save_state(self, path: str) -> None:
-        """Writes the request table and the KV pages of every live sequence (between two steps). A new engine with the
+        """Writes the request table and the KV pages (and recurrent state) of every live sequence (between two steps). A new engine with the
         same weights continues from it with :meth:`load_state` and produces the same tokens."""
         seqs = []
         for s in self.running.values():
             blocks = self.block_mgr.get_seq_block_list(s.req_id)
-            pages = self.executor.kv_cache[:, :, torch.tensor(blocks, device=self.device)].cpu()
+            cached = self.executor.export_sequence(blocks, self.block_mgr.row_of(s.req_id))
             seqs.append(dict(req_id=s.req_id, prompt=s.prompt, max_new_tokens=s.max_new_tokens, length=s.length,
-                             last_token=s.last_token, outputs=list(s.outputs), pages=pages))
+                             last_token=s.last_token, outputs=list(s.outputs), cached=cached))
         waiting = [dict(req_id=s.req_id, prompt=s.prompt, max_new_tokens=s.max_new_tokens) for s in self.waiting]
         finished = {r: list(s.outputs) for r, s in self.finished.items()}
         tmp = path + ".tmp"
@@ -231,8 +286,7 @@ class ColocatedEngine:
                      outputs=list(d["outputs"]), t_arrival=time.time())
             self.block_mgr.allocate(s.req_id, s.length + 1)
             blocks = self.block_mgr.get_seq_block_list(s.req_id)
-            n = d["pages"].shape[2]
-            self.executor.kv_cache[:, :, torch.tensor(blocks[:n], device=self.device)] = d["pages"].to(self.device)
+            self.executor.import_sequence(blocks, self.block_mgr.row_of(s.req_id), d["cached"])
             self.running[s.req_id] = s
         for d in st["waiting"]:
             self.add_request(d["req_id"], d["prompt"], d["max_new_tokens"])

@@ -60,21 +60,19 @@ class MixedBatchEngine(ColocatedEngine):
         T = len(p)
         if T == 0:
             return []
-        h2d = self._apply_block_table_patches()
-        self._h_ids.numpy()[:T] = p.ids
-        self._h_pos.numpy()[:T] = p.pos
-        self._h_ctx.numpy()[:T] = [x + 1 for x in p.pos]
-        self._h_row.numpy()[:T] = p.rows
-        self._h_slots.numpy()[:T] = p.slots
         decode_only = all(row >= 0 and grown == 1 and s.length >= len(s.prompt) for row, s, grown in p.emit)
-        args = (self._h_ids[:T], self._h_pos[:T], self._h_slots[:T], self._h_ctx[:T], self._h_row[:T])
-        nxt, _ = self.executor.decode(*args) if decode_only else self.executor.prefill(*args)
-        self._h_out[:T].copy_(nxt[:T], non_blocking=True)
+        # the rows that sample: a prompt portion that is not the last one has none
+        emit = [row for row, _, _ in p.emit if row >= 0]
+        nxt, _ = self._execute(p.ids, p.pos, p.rows, p.slots, out_rows=emit or [0], decode_only=decode_only)
+        n = len(emit)
+        self._h_out[:n].copy_(nxt[:n], non_blocking=True)
         if self.device.type == "cuda":
             torch.cuda.current_stream().synchronize()
-        out = self.sched.commit(plans, [self._h_out[:T].tolist()], time.time())
-        self.h2d_bytes_last += h2d + T * 24
-        self.d2h_bytes_last += T * 4
+        toks = [0] * T
+        for row, tok in zip(emit, self._h_out[:n].tolist()):
+            toks[row] = tok
+        out = self.sched.commit(plans, [toks], time.time())
+        self.d2h_bytes_last += n * 4
         return out
 
     def run_until_done(self, max_steps: int = 1 << 30) -> Dict[int, List[int]]:
@@ -87,15 +85,15 @@ class MixedBatchEngine(ColocatedEngine):
     # ---- serving-state snapshot ----------------------------------------------------------------------------------
     def save_state(self, path: str) -> None:
         """Request table (running sequences with their prefill progress, waiting and finished requests) and the KV
-        pages of every running sequence, taken between two steps. ``load_state`` on a fresh engine with the same weights
+        pages and recurrent state of every running sequence, taken between two steps. ``load_state`` on a fresh engine with the same weights
         continues with identical tokens."""
         import os
         running = []
         for s in self.sched.running[0].values():
             blocks = self.block_mgr.get_seq_block_list(s.req_id)
-            pages = self.executor.kv_cache[:, :, torch.tensor(blocks, device=self.device)].cpu()
+            cached = self.executor.export_sequence(blocks, self.block_mgr.row_of(s.req_id))
             running.append(dict(req_id=s.req_id, prompt=s.prompt, max_new_tokens=s.max_new_tokens, length=s.length,
-                                last_token=s.last_token, outputs=list(s.outputs), t_arrival=s.t_arrival, pages=pages))
+                                last_token=s.last_token, outputs=list(s.outputs), t_arrival=s.t_arrival, cached=cached))
         waiting = [dict(req_id=s.req_id, prompt=s.prompt, max_new_tokens=s.max_new_tokens, t_arrival=s.t_arrival)
                    for s in self.sched.waiting]
         finished = {r: list(s.outputs) for r, s in self.sched.finished.items()}
@@ -113,8 +111,7 @@ class MixedBatchEngine(ColocatedEngine):
             # the same reservation a fresh admission makes: room for the whole prompt, the rest grows step by step
             self.block_mgr.allocate(s.req_id, max(len(s.prompt), s.length) + 1)
             blocks = self.block_mgr.get_seq_block_list(s.req_id)
-            n = min(d["pages"].shape[2], len(blocks))
-            self.executor.kv_cache[:, :, torch.tensor(blocks[:n], device=self.device)] = d["pages"][:, :, :n].to(self.device)
+            self.executor.import_sequence(blocks, self.block_mgr.row_of(s.req_id), d["cached"])
             self.sched.restore_running(0, s)
         for d in st["waiting"]:
             self.sched.add_request(d["req_id"], d["prompt"], d["max_new_tokens"], d["t_arrival"])

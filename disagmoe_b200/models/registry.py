@@ -1,0 +1,95 @@
+"""Model registry: which configuration reader, checkpoint layout and executor serve an architecture.
+
+``load_model(path)`` reads a checkpoint folder (config.json + model.safetensors) and picks the architecture by the
+``architecture`` key of config.json; ``make_executor`` builds the whole-iteration executor of a configuration, whether it
+comes from a folder or from a preset.
+"""
+from __future__ import annotations
+
+import json
+import os
+from dataclasses import dataclass
+from typing import Any, Callable, Dict, Optional, Tuple
+
+import torch
+
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, LayerSpec, ModelConfig, PRESETS,
+                      RotarySpec, get_preset)
+from . import weights as W
+
+
+# ---- Rurunex: gated linear attention, channel-wise gated delta rule and windowed attention in any order -----------------
+def _rotary(rot: Optional[dict]) -> Optional[RotarySpec]:
+    if not rot:
+        return None
+    sc = rot.get("scaling") or {}
+    return RotarySpec(int(rot["dims"]), float(rot["base"]), **{k: float(v) for k, v in sc.items()})
+
+
+def _rurunex_layer(i: int, layer: dict, shapes: Dict[str, Tuple[int, ...]]) -> LayerSpec:
+    m, kind = layer["mixer"], layer["type"]
+    rank = lambda name: shapes[f"l{i}.mix.{name}"][0] if f"l{i}.mix.{name}" in shapes else 16
+    if kind == "gla":
+        mixer = GatedLinearSpec(m["heads"], m["dim"], m["vdim"], float(m["tau"]), rank("a1"))
+    elif kind == "channel_delta":
+        mixer = ChannelDeltaSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"], rank("a1"), rank("g1"))
+    elif kind == "attention":
+        mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), _rotary(m.get("rot")),
+                              (m.get("mask") or {}).get("size"), m.get("softcap"), m.get("kv_from"))
+    else:
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    mlp = layer.get("mlp")
+    if mlp is not None and mlp.get("kind") != "dense":
+        raise ValueError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
+    return LayerSpec(mixer, None if mlp is None else mlp["ff"])
+
+
+def rurunex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, ...]], **kw) -> LayerListConfig:
+    """``shapes``: tensor name -> shape of the checkpoint, the only place that has the ranks of the low-rank maps."""
+    layers = [_rurunex_layer(i, l, shapes) for i, l in enumerate(raw["layers"])]
+    return LayerListConfig.make(raw["width"], raw["vocab"], layers, rms_norm_eps=float(raw["norm"]["eps"]),
+                                embed_scale=float(raw["embedding"]["scale"]), logit_scale=float(raw["logit_scale"]),
+                                architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
+
+
+@dataclass(frozen=True)
+class Architecture:
+    config_from_json: Callable[..., ModelConfig]
+
+
+ARCHITECTURES: Dict[str, Architecture] = {
+    "Rurunex": Architecture(rurunex_config_from_json),
+}
+
+
+def load_model(path: str, dtype: Optional[torch.dtype] = None, **kw) -> Tuple[ModelConfig, W.StateDict]:
+    """(configuration, weights on the CPU as stored) of a checkpoint folder. ``kw``: further configuration fields."""
+    with open(os.path.join(path, "config.json")) as f:
+        raw = json.load(f)
+    name = raw.get("architecture")
+    if name not in ARCHITECTURES:
+        raise ValueError(f"unknown architecture {name!r}; known: {sorted(ARCHITECTURES)}")
+    sd = W.load_safetensors(os.path.join(path, "model.safetensors"))
+    cfg = ARCHITECTURES[name].config_from_json(raw, {n: tuple(t.shape) for n, t in sd.items()},
+                                               dtype=dtype or torch.bfloat16, **kw)
+    bad = W.check_state_dict(cfg, sd)
+    if bad:
+        raise ValueError(f"{path}: tensors missing or of the wrong shape: {', '.join(bad[:8])}")
+    return cfg, sd
+
+
+def resolve_model(name_or_path: str, dtype: Optional[torch.dtype] = None, **kw) -> Tuple[ModelConfig, Optional[W.StateDict]]:
+    """A preset name -> (its configuration, None: random weights); a checkpoint folder -> :func:`load_model`."""
+    if name_or_path in PRESETS:
+        return get_preset(name_or_path, **({"dtype": dtype} if dtype else {}), **kw), None
+    if os.path.isdir(name_or_path):
+        return load_model(name_or_path, dtype, **kw)
+    raise ValueError(f"{name_or_path!r} is neither a preset ({', '.join(sorted(PRESETS))}) nor a checkpoint folder")
+
+
+def make_executor(cfg: ModelConfig, cache_cfg, **kw):
+    """The whole-iteration executor that runs ``cfg`` on one device."""
+    from ..executor.fused import FusedModelExecutor
+    from ..executor.layer_list import LayerListExecutor
+    cls = LayerListExecutor if isinstance(cfg, LayerListConfig) else FusedModelExecutor
+    return cls(cfg, cache_cfg, **kw)

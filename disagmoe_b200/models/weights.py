@@ -23,17 +23,69 @@ into the runtime layout ``w13 [E, 2 I, H]`` / ``w2 [E, H, I]`` (:func:`to_runtim
 """
 from __future__ import annotations
 
+import json
 import os
+import struct
 from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
-from ..config import ModelConfig
+from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, ModelConfig
 
 StateDict = Dict[str, torch.Tensor]
 
 
+def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
+    """Names and shapes of a layer-list checkpoint: ``l<i>.norm1 / norm1b / norm2 / norm2b`` around the sublayers,
+    ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward; linear weights [out, in]."""
+    H = cfg.hidden_size
+    out: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab_size, H)}
+    for i, layer in enumerate(cfg.layers):
+        p, m = f"l{i}.", layer.mixer
+        x = p + "mix."
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.ff else ()):
+            out[p + n] = (H,)
+        vs = m.heads * m.vdim
+        if isinstance(m, GatedLinearSpec):
+            ks = m.heads * m.dim
+            out.update({x + "q": (ks, H), x + "k": (ks, H), x + "v": (vs, H), x + "g": (vs, H), x + "norm": (m.vdim,),
+                        x + "a1": (m.rank, H), x + "a2": (ks, m.rank), x + "a2.b": (ks,)})
+        elif isinstance(m, ChannelDeltaSpec):
+            ks, zs = m.kv_heads * m.dim, m.heads * m.dim
+            for n, c in (("q", ks), ("k", ks), ("v", vs)):
+                out.update({x + n: (c, H), x + n + ".conv": (c, m.conv)})
+            out.update({x + "b": (m.heads, H), x + "A_log": (m.heads,), x + "norm": (m.vdim,), x + "a1": (m.rank, H),
+                        x + "a2": (zs, m.rank), x + "dt_bias": (zs,), x + "g1": (m.gate_rank, H),
+                        x + "g2": (vs, m.gate_rank)})
+        else:
+            out.update({x + "q": (m.heads * m.dim, H), x + "q.norm": (m.dim,)})
+            if m.kv_from is None:
+                out.update({x + "k": (m.kv_heads * m.dim, H), x + "v": (m.kv_heads * m.vdim, H), x + "k.norm": (m.dim,)})
+        out[x + "o"] = (H, vs)
+        if layer.ff:
+            out.update({p + "mlp.gate": (layer.ff, H), p + "mlp.up": (layer.ff, H), p + "mlp.down": (H, layer.ff)})
+    out.update({"final.norm": (H,), "head": (cfg.vocab_size, H)})
+    return out
+
+
+def _init_layer_list_tensor(name: str, shape: Tuple[int, ...], gen, device) -> torch.Tensor:
+    """Random values of the order a trained model has: weights of unit gain, norms near one, slow decays."""
+    r = torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
+    leaf = name.split(".mix.")[-1]
+    if len(shape) == 2:
+        return r * (0.02 if name == "embed" else shape[1] ** -0.5)
+    if leaf == "A_log":
+        return r * 0.3
+    if leaf == "dt_bias":
+        return r * 0.5 - 4.0
+    if leaf == "a2.b":
+        return r + 2.0
+    return 1.0 + 0.05 * r if ".mix." in name else 0.05 * r
+
+
 def param_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
+    if isinstance(cfg, LayerListConfig):
+        return layer_list_shapes(cfg)
     H, hd = cfg.hidden_size, cfg.head_dim
     shapes: Dict[str, Tuple[int, ...]] = {
         "embed_tokens.weight": (cfg.vocab_size, H),
@@ -86,6 +138,8 @@ def init_tensor(cfg: ModelConfig, name: str, shape: Tuple[int, ...], device="cpu
         return torch.stack([init_tensor(cfg, f"{name}.{e}", tuple(shape[1:]), device, dtype) for e in range(shape[0])])
     gen = torch.Generator(device=device)
     gen.manual_seed(_name_seed(cfg.seed, name))
+    if isinstance(cfg, LayerListConfig):
+        return _init_layer_list_tensor(name, shape, gen, device).to(dtype)
     t = torch.empty(shape, dtype=torch.float32 if torch.device(device).type == "cpu" else dtype, device=device)
     t.normal_(0.0, cfg.init_std, generator=gen)
     return t.to(dtype)
@@ -159,6 +213,49 @@ def save_state_dict(sd: StateDict, path: str) -> None:
 def load_state_dict(path: str, device="cpu", dtype=None) -> StateDict:
     sd = torch.load(path, map_location="cpu", weights_only=True)
     return {k: v.to(device=device, dtype=dtype or v.dtype) for k, v in sd.items()}
+
+
+_SAFETENSORS_DTYPES = {"BF16": torch.bfloat16, "F32": torch.float32, "F16": torch.float16, "I32": torch.int32,
+                       "I64": torch.int64}
+
+
+def load_safetensors(path: str) -> StateDict:
+    """Reads a safetensors file: 8-byte little-endian header length, a JSON header name -> dtype, shape, data_offsets, then
+    the data. Tensors keep their stored dtype and own their memory."""
+    out: StateDict = {}
+    with open(path, "rb") as f:
+        n = struct.unpack("<Q", f.read(8))[0]
+        header = json.loads(f.read(n))
+        for name, e in header.items():
+            if name == "__metadata__":
+                continue
+            if e["dtype"] not in _SAFETENSORS_DTYPES:
+                raise ValueError(f"{path}: tensor {name} has unsupported dtype {e['dtype']}")
+            a, b = e["data_offsets"]
+            f.seek(8 + n + a)
+            data = bytearray(f.read(b - a))
+            dt = _SAFETENSORS_DTYPES[e["dtype"]]
+            t = torch.frombuffer(data, dtype=dt) if data else torch.empty(0, dtype=dt)
+            out[name] = t.reshape(e["shape"])
+    return out
+
+
+def save_safetensors(sd: StateDict, path: str) -> None:
+    """Writes tensors in the format :func:`load_safetensors` reads."""
+    names = {v: k for k, v in _SAFETENSORS_DTYPES.items()}
+    header, pos, blobs = {}, 0, []
+    for name, t in sd.items():
+        t = t.detach().cpu().contiguous()
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes()
+        header[name] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [pos, pos + len(raw)]}
+        pos += len(raw)
+        blobs.append(raw)
+    head = json.dumps(header).encode()
+    head += b" " * (-len(head) % 8)
+    tmp = path + ".tmp"
+    with open(tmp, "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head + b"".join(blobs))
+    os.replace(tmp, path)
 
 
 def check_state_dict(cfg: ModelConfig, sd: StateDict) -> List[str]:

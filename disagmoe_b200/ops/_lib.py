@@ -64,6 +64,15 @@ class DmoeRouteDispatch(ctypes.Structure):
                                   "region_cap", "n_wait", "ret_rank", "ret_rank_set")]
 
 
+class DmoeRecur(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("q", "k", "v", "gate", "beta", "z", "z_bias", "a_log", "conv_w", "ring", "segs",
+                                   "positions", "rows", "kv_slots", "state", "norm_w", "out", "raw")] + \
+               [(n, _ll) for n in ("ldq", "ldk", "ldv", "ldg", "ldb", "ldz", "ldo", "ldraw")] + \
+               [(n, _i) for n in ("n_segs", "n_slots", "heads", "kv_heads", "dim", "vdim", "taps", "delta", "decay_kind",
+                                  "gate_kind", "is_f32")] + \
+               [(n, _f) for n in ("qscale", "inv_tau", "eps")]
+
+
 def lib_path() -> str:
     return _LIB_PATH
 

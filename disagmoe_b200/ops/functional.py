@@ -96,20 +96,38 @@ def pick_attn_splits(T: int, n_kv: int, max_ctx: int, block_size: int) -> int:
 _attn_ws = {}
 
 
+def attention_on_tensor_cores(dtype, n_q: int, n_kv: int, hd: int, vd: int) -> bool:
+    """Shapes of the tensor-core attention kernels; the others (and fp32) run on the CUDA cores."""
+    return dtype == torch.bfloat16 and hd == vd and hd in (64, 128) and n_q % n_kv == 0 and n_q // n_kv in (1, 2, 4, 8)
+
+
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
-                    out: Optional[torch.Tensor] = None, splits: int = 1, scale: Optional[float] = None) -> torch.Tensor:
-    """out[t] = softmax(q[t] K^T * scale) V over the first ctx_len[t] cached tokens of block-table row bt_row[t]."""
+                    out: Optional[torch.Tensor] = None, splits: int = 1, scale: Optional[float] = None,
+                    window: Optional[int] = None, softcap: Optional[float] = None, fp32_weights: bool = False) -> torch.Tensor:
+    """out[t] = softmax(q[t] K^T * scale) V over the first ctx_len[t] cached tokens of block-table row bt_row[t], or the
+    last ``window`` of them; ``softcap``: scores are soft-capped, cap * tanh(score / cap). ``fp32_weights`` keeps the
+    softmax weights at fp32 accuracy in the product with V (implied by the two options before). Value heads may have
+    another size than key heads (``vcache.shape[-1]``)."""
     if not q.is_cuda:
-        o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale)
+        o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale, window, softcap)
         if out is not None:
             out.copy_(o)
             return out
         return o
     T = q.shape[0]
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
+    vd = vcache.shape[-1]
     if out is None:
-        out = torch.empty(T, n_q * hd, dtype=torch.bfloat16, device=q.device)
+        out = torch.empty(T, n_q * vd, dtype=q.dtype, device=q.device)
+    if not attention_on_tensor_cores(q.dtype, n_q, n_kv, hd, vd):
+        assert q.dtype == kcache.dtype == vcache.dtype == out.dtype
+        _lib.check(_lib.lib().dmoe_any_attention(
+            c_int(int(q.dtype == torch.float32)), _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables),
+            c_int(block_tables.stride(0)), _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q),
+            c_int(n_kv), c_int(hd), c_int(vd), c_float(scale), c_int(window or 0), c_float(softcap or 0.0), _vp(out),
+            c_ll(out.stride(0)), _st()), "dmoe_any_attention")
+        return out
     assert block_tables.dtype == torch.int32 and ctx_len.dtype == torch.int32 and block_tables.stride(1) == 1
     ws = None
     if splits > 1:
@@ -119,6 +137,13 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         if ws is None or ws.numel() < need:
             ws = torch.empty(max(need, 1 << 22), dtype=torch.float32, device=q.device)
             _attn_ws[key] = ws
+    if window or softcap or fp32_weights:
+        _lib.check(_lib.lib().dmoe_paged_attention_ext(
+            _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
+            _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_float(scale),
+            c_int(window or 0), c_float(softcap or 0.0), c_int(splits), _vp(out), c_ll(out.stride(0)), _vp(ws), _st()),
+            "dmoe_paged_attention_ext")
+        return out
     _lib.check(_lib.lib().dmoe_paged_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
         _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd),
@@ -334,6 +359,16 @@ def prefill_tile_tokens(n_q: int, n_kv: int) -> int:
     return 64 // gq if n_q % n_kv == 0 and gq in (1, 2, 4, 8) else 0
 
 
+def token_runs(bt_row, positions):
+    """(first row, end row) of every run of consecutive rows of one sequence at consecutive positions."""
+    import numpy as np
+    rows, pos = np.asarray(bt_row, dtype=np.int64), np.asarray(positions, dtype=np.int64)
+    if len(rows) == 0:
+        return []
+    brk = np.nonzero((rows[1:] != rows[:-1]) | (pos[1:] != pos[:-1] + 1))[0] + 1
+    return list(zip([0] + brk.tolist(), brk.tolist() + [len(rows)]))
+
+
 def build_prefill_tiles(bt_row, positions, tile_tokens: int, min_len: int = 8):
     """Finds the prompt segments of a flat token batch on the host and cuts them into attention tiles.
 
@@ -349,10 +384,7 @@ def build_prefill_tiles(bt_row, positions, tile_tokens: int, min_len: int = 8):
     tiles = []
     if T == 0 or tile_tokens <= 0:
         return torch.zeros(0, 4, dtype=torch.int32), torch.from_numpy(covered)
-    brk = np.nonzero((rows[1:] != rows[:-1]) | (pos[1:] != pos[:-1] + 1))[0] + 1
-    starts = np.concatenate([[0], brk])
-    ends = np.concatenate([brk, [T]])
-    for a, b in zip(starts.tolist(), ends.tolist()):
+    for a, b in token_runs(rows, pos):
         if b - a < min_len:
             continue
         covered[a:b] = True
@@ -364,7 +396,8 @@ def build_prefill_tiles(bt_row, positions, tile_tokens: int, min_len: int = 8):
 
 def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                       tiles: torch.Tensor, n_tiles: int, n_q: int, n_kv: int, hd: int, out: torch.Tensor,
-                      scale: Optional[float] = None) -> torch.Tensor:
+                      scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
+                      fp32_weights: bool = False) -> torch.Tensor:
     """Causal attention of the prompt tokens named by ``tiles`` (device int32 [>= n_tiles, 4], see
     :func:`build_prefill_tiles`) over the paged cache, which already holds their own K / V; writes their rows of
     ``out``. Every tile streams its sequence's K / V once (the per-token kernel streams it once per row)."""
@@ -372,8 +405,107 @@ def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
         return out
     assert q.is_cuda and tiles.is_cuda and tiles.dtype == torch.int32 and tiles.is_contiguous()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
+    if window or softcap or fp32_weights:
+        _lib.check(_lib.lib().dmoe_prefill_attention_ext(
+            _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
+            _vp(tiles), c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_float(scale),
+            c_int(window or 0), c_float(softcap or 0.0), _vp(out), c_ll(out.stride(0)), _st()), "dmoe_prefill_attention_ext")
+        return out
     _lib.check(_lib.lib().dmoe_prefill_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(tiles),
         c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_float(scale), _vp(out),
         c_ll(out.stride(0)), _st()), "dmoe_prefill_attention")
     return out
+
+
+# ---- decoders with an fp32 residual stream (csrc/kernels/layer_ops.cu) ------------------------------------------------
+def _f32(dtype) -> c_int:
+    assert dtype in (torch.float32, torch.bfloat16)
+    return c_int(int(dtype == torch.float32))
+
+
+def embed_f32(ids: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor) -> torch.Tensor:
+    """out (fp32) = table[ids] * scale."""
+    if not table.is_cuda:
+        out.copy_(table[ids.long()].float() * scale)
+        return out
+    assert ids.dtype == torch.int32 and table.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32
+    _lib.check(_lib.lib().dmoe_embed_f32(_vp(ids), _vp(table), _f32(table.dtype), c_float(scale), _vp(out),
+                                         c_int(ids.shape[0]), c_int(table.shape[1]), c_int(table.shape[0]), _st()),
+               "dmoe_embed_f32")
+    return out
+
+
+def resid_norm(resid: torch.Tensor, y: Optional[torch.Tensor], post: Optional[torch.Tensor], pre: Optional[torch.Tensor],
+               eps: float, dtype: torch.dtype, out_scale: float = 1.0, rows: Optional[torch.Tensor] = None
+               ) -> Optional[torch.Tensor]:
+    """One step of a residual stream kept in fp32: resid += norm(y) * post (where y is given), then returns
+    norm(resid) * pre * out_scale in ``dtype`` (None where pre is None). ``rows`` (int32) picks the rows to return; resid
+    itself is then left as it is. post / pre: fp32 weights as multiplied (offsets from one already added)."""
+    if not resid.is_cuda:
+        return reference.resid_norm(resid, y, post, pre, eps, dtype, out_scale, rows)
+    n, W = (resid.shape[0] if rows is None else rows.shape[0]), resid.shape[1]
+    h = torch.empty(n, W, dtype=dtype, device=resid.device) if pre is not None else None
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and (y is None or (y.dtype == dtype and y.stride(1) == 1))
+    assert rows is None or rows.dtype == torch.int32
+    _lib.check(_lib.lib().dmoe_resid_norm(
+        _f32(dtype), _vp(resid), _vp(y), c_ll(y.stride(0) if y is not None else 0), _vp(post), _vp(pre), c_float(out_scale),
+        c_float(eps), _vp(rows), _vp(h), c_ll(W), c_int(n), c_int(W), _st()), "dmoe_resid_norm")
+    return h
+
+
+def rope_frequencies(dims: int, base: float, factor: Optional[float] = None, original: float = 0.0, fast: float = 32.0,
+                     slow: float = 1.0):
+    """(list of dims / 2 inverse frequencies, factor on cos and sin). With ``factor``: YaRN (Peng et al., "YaRN: Efficient
+    Context Window Extension of Large Language Models"): dimensions that turn more than ``fast`` times over the original
+    context keep their frequency, those below ``slow`` turns are slowed down by ``factor``, a linear ramp in between."""
+    f = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if factor is None:
+        return f, 1.0
+    turn_dim = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(turn_dim(fast)), 0), min(math.ceil(turn_dim(slow)), dims - 1)
+    width = max(hi - lo, 0.001)
+    ramp = [min(max((i - lo) / width, 0.0), 1.0) for i in range(dims // 2)]
+    return [x / factor * r + x * (1.0 - r) for x, r in zip(f, ramp)], 0.1 * math.log(factor) + 1.0
+
+
+_freq_tables = {}
+
+
+def rope_freq_table(spec, max_pos: int, device) -> Optional[torch.Tensor]:
+    """fp32 [max_pos, dims / 2, 2] = (cos, sin) of a :class:`disagmoe_b200.config.RotarySpec`, from double-precision
+    angles; cached per (device, positions, spec)."""
+    if spec is None:
+        return None
+    device = torch.device(device)
+    key = (device.type, device.index or 0, max_pos, spec)
+    if key not in _freq_tables:
+        f, m = rope_frequencies(spec.dims, spec.base, spec.factor, spec.original, spec.fast, spec.slow)
+        freq = torch.tensor(f, dtype=torch.float64, device=device)
+        if device.type == "cuda":
+            t = torch.empty(max_pos, len(f), 2, dtype=torch.float32, device=device)
+            _lib.check(_lib.lib().dmoe_rope_freq_table(_vp(t), c_int(max_pos), c_int(len(f)), _vp(freq), c_float(m), _st()),
+                       "dmoe_rope_freq_table")
+            torch.cuda.current_stream().synchronize()     # `freq` may be freed from here on
+        else:
+            ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * freq
+            t = (torch.stack([ang.cos(), ang.sin()], -1) * m).float()
+        _freq_tables[key] = t
+    return _freq_tables[key]
+
+
+def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: Optional[torch.Tensor],
+                 vcache: Optional[torch.Tensor], n_q: int, n_kv: int, dk: int, dv: int, table: Optional[torch.Tensor],
+                 qw: torch.Tensor, kw: Optional[torch.Tensor], eps: float) -> None:
+    """RMS norm of every q / k head (weights fp32 [dk]) and rotation by ``table`` (:func:`rope_freq_table`, None: no
+    rotation) on rows [q | k | v]; q in place, k and v to the paged caches at ``slots``. n_kv = 0: q only (a layer that
+    reads another layer's cache)."""
+    if not qkv.is_cuda:
+        return reference.qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps)
+    assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and qkv.stride(1) == 1
+    assert n_kv == 0 or (kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == qkv.dtype)
+    rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
+    _lib.check(_lib.lib().dmoe_qk_norm_rope(
+        _f32(qkv.dtype), _vp(qkv), c_ll(qkv.stride(0)), _vp(positions), _vp(slots), _vp(kcache), _vp(vcache),
+        c_int(qkv.shape[0]), c_int(n_q), c_int(n_kv), c_int(dk), c_int(dv), c_int(rot), _vp(table), c_int(max_pos), _vp(qw),
+        _vp(kw), c_float(eps), _st()), "dmoe_qk_norm_rope")

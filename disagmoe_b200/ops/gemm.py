@@ -7,7 +7,8 @@
                     row (and GPU) it came from                         -- reference: disagmoe/frontend/engine.py:731-734
 
 Weights are K-contiguous ``[groups, out, in]``. CPU tensors take a plain PyTorch path (used by the fp32 CPU
-configuration and as the numerical reference); CUDA tensors always run the sm_100a kernel.
+configuration and as the numerical reference); CUDA tensors always run the sm_100a kernels: bf16 the tcgen05 kernel, fp32
+operands (and bf16 operands whose rows are not 16-byte aligned) the CUDA-core kernel of ``csrc/kernels/layer_ops.cu``.
 """
 from __future__ import annotations
 
@@ -234,6 +235,27 @@ def _launch(W, X, Y, R, offs, recs, bases, G, T, F, K, epi, bn, splitk, ldy, y_f
     _lib.check(_lib.lib().dmoe_gemm(ctypes.byref(d), _lib.stream_ptr()), "dmoe_gemm")
 
 
+def _tma_ok(x, w) -> bool:
+    """Can the tcgen05 kernel's TMA address these operands (16-byte rows and base addresses)?"""
+    return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
+
+
+def _simt_linear(x, w, out, out_dtype):
+    """fp32 operands (true fp32 arithmetic), or bf16 operands that TMA cannot address: the CUDA-core GEMM."""
+    T, K = x.shape
+    F = w.shape[0]
+    assert w.is_contiguous() and w.dtype == x.dtype and w.shape[1] == K and x.stride(1) == 1
+    f32 = x.dtype == torch.float32
+    if out is None:
+        out = torch.empty(T, F, dtype=out_dtype or x.dtype, device=x.device)
+    assert out.stride(1) == 1 and (out.dtype == torch.float32 or not f32)
+    v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+    _lib.check(_lib.lib().dmoe_simt_linear(
+        i(int(f32)), i(int(out.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), ll(K),
+        v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), v(_lib.stream_ptr())), "dmoe_simt_linear")
+    return out
+
+
 def _check_x(x):
     assert x.dim() == 2 and x.stride(1) == 1 and x.dtype == torch.bfloat16, "x must be [T, K] bf16, K contiguous"
     assert x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0, "x rows must be 16-byte aligned"
@@ -255,6 +277,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
             out.copy_(y)
             return out
         return y
+    if x.dtype == torch.float32 or (comm is None and residual is None and not _tma_ok(x, w)):
+        assert comm is None and residual is None
+        return _simt_linear(x, w, out, out_dtype)
     _check_x(x)
     assert w.is_contiguous() and w.dtype == torch.bfloat16 and w.shape[1] == K
     odt = out_dtype or torch.bfloat16
@@ -436,6 +461,15 @@ def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor
             out.copy_(y)
             return out
         return y
+    if x.dtype == torch.float32 or not _tma_ok(x, w13):
+        gu = _simt_linear(x, w13, None, None)
+        if out is None:
+            out = torch.empty(T, I, dtype=x.dtype, device=x.device)
+        v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+        _lib.check(_lib.lib().dmoe_silu_mul(i(int(x.dtype == torch.float32)), v(gu.data_ptr()), ll(gu.stride(0)),
+                                            v(out.data_ptr()), ll(out.stride(0)), i(T), i(I), v(_lib.stream_ptr())),
+                   "dmoe_silu_mul")
+        return out
     _check_x(x)
     assert w13.is_contiguous() and w13.dtype == torch.bfloat16
     if out is None:

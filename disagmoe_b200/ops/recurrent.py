@@ -1,0 +1,200 @@
+"""Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``): gated linear attention and the gated
+delta rule, with one decay per head and key channel. CUDA tensors run the kernels, CPU tensors the PyTorch restatements.
+
+A step's rows fall into segments (consecutive rows of one sequence). One-token segments (decoding) take one launch from
+the projections to the gated, normalised output; longer ones (prompts and portions of prompts) are convolved and then run
+chunk by chunk on the tensor cores, or token by token where fp32 is asked for or the head shape has no chunk kernel.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _lib, reference
+from .functional import token_runs
+from .gemm import num_sms
+
+CHUNK = 64          # tokens of a chunk
+MAX_TAPS = 8        # longest short convolution
+
+
+@dataclass
+class SegmentTables:
+    """Segments of one step. ``singles`` / ``multi``: int32 [n, 4] = (first row, tokens, slot, first position); ``chunks``:
+    int32 [n, 4] = (first row, tokens, index into ``multi``, number in the segment). ``singles`` None with n_single > 0:
+    every row is a segment of its own (decode step), described by ``positions``, ``rows`` (slots) and ``kv_slots``."""
+    n_single: int = 0
+    n_multi: int = 0
+    n_chunks: int = 0
+    max_multi: int = 0                              # tokens of the longest segment
+    singles: Optional[torch.Tensor] = None
+    multi: Optional[torch.Tensor] = None
+    chunks: Optional[torch.Tensor] = None
+    positions: Optional[torch.Tensor] = None
+    rows: Optional[torch.Tensor] = None
+    kv_slots: Optional[torch.Tensor] = None
+
+
+def build_segments(bt_row, positions, device) -> SegmentTables:
+    """Tables of a batch given on the host (rows of one sequence are consecutive, as every scheduler emits them)."""
+    rows, pos = torch.as_tensor(bt_row).tolist(), torch.as_tensor(positions).tolist()
+    singles, multi, chunks = [], [], []
+    for a, b in token_runs(rows, pos):
+        if b - a == 1:
+            singles.append((a, 1, rows[a], pos[a]))
+            continue
+        for i, c in enumerate(range(a, b, CHUNK)):
+            chunks.append((c, min(CHUNK, b - c), len(multi), i))
+        multi.append((a, b - a, rows[a], pos[a]))
+    table = torch.tensor(singles + multi + chunks, dtype=torch.int32).reshape(-1, 4)
+    if torch.device(device).type == "cuda":
+        table = table.to(device)
+    s, m = len(singles), len(multi)
+    return SegmentTables(s, m, len(chunks), max((x[1] for x in multi), default=0), table[:s], table[s:s + m], table[s + m:])
+
+
+def decode_segments(positions: torch.Tensor, rows: torch.Tensor, kv_slots: torch.Tensor) -> SegmentTables:
+    """Every row one token (padding rows have kv_slots < 0); no host work, so a captured graph can hold it."""
+    return SegmentTables(n_single=positions.shape[0], positions=positions, rows=rows, kv_slots=kv_slots)
+
+
+@dataclass
+class RecurrentState:
+    """Per-layer state pool: S fp32 [slots, heads, dim, vdim] and, with a short convolution, the ring of its last inputs
+    [slots, taps, channels]. A slot needs no clearing: a segment at position 0 starts from zero."""
+    S: torch.Tensor
+    ring: Optional[torch.Tensor] = None
+
+    def tensors(self):
+        return [self.S] + ([self.ring] if self.ring is not None else [])
+
+
+@dataclass
+class Recurrence:
+    """Constants of one recurrent layer (weights fp32). ``delta``: the gated delta rule with unit-norm q / k and
+    log a = -exp(a_log) softplus(z + z_bias); otherwise the plain write with log a = log sigmoid(z + z_bias) / tau."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    delta: bool
+    z_bias: torch.Tensor
+    norm_w: torch.Tensor
+    eps: float
+    a_log: Optional[torch.Tensor] = None
+    tau: float = 1.0
+    conv_w: Optional[torch.Tensor] = None            # [2 kv_heads dim + heads vdim, taps]
+    sigmoid_gate: bool = False
+
+    @property
+    def taps(self) -> int:
+        return 0 if self.conv_w is None else self.conv_w.shape[1]
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def new_state(self, slots: int, dtype, device) -> RecurrentState:
+        S = torch.zeros(slots, self.heads, self.dim, self.vdim, dtype=torch.float32, device=device)
+        ring = torch.zeros(slots, self.taps, self.channels, dtype=dtype, device=device) if self.taps else None
+        return RecurrentState(S, ring)
+
+
+def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) -> _lib.DmoeRecur:
+    d = _lib.DmoeRecur()
+    for name, t in (("q", q), ("k", k), ("v", v), ("gate", gate), ("beta", beta), ("z", z)):
+        assert t is None or (t.stride(1) == 1 and t.dtype == (torch.float32 if name == "z" else q.dtype))
+        setattr(d, name, _lib.ptr(t))
+    for name, t in (("ldq", q), ("ldk", k), ("ldv", v), ("ldg", gate), ("ldb", beta), ("ldz", z)):
+        setattr(d, name, 0 if t is None else t.stride(0))
+    d.z_bias, d.a_log, d.norm_w = _lib.ptr(r.z_bias), _lib.ptr(r.a_log), _lib.ptr(r.norm_w)
+    d.state, d.n_slots = _lib.ptr(state.S), state.S.shape[0]
+    d.heads, d.kv_heads, d.dim, d.vdim = r.heads, r.kv_heads, r.dim, r.vdim
+    d.delta, d.decay_kind, d.gate_kind = int(r.delta), int(r.delta), int(r.sigmoid_gate)
+    d.is_f32 = int(q.dtype == torch.float32)
+    d.qscale, d.inv_tau, d.eps = r.dim ** -0.5, 1.0 / r.tau, r.eps
+    return d
+
+
+def _gate_norm(r: Recurrence, table, n, max_tokens, raw, gate, out) -> None:
+    v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+    _lib.check(_lib.lib().dmoe_gate_norm(
+        i(int(out.dtype == torch.float32)), v(_lib.ptr(table)), i(n), i(max_tokens), v(raw.data_ptr()), ll(raw.stride(0)),
+        v(gate.data_ptr()), ll(gate.stride(0)), v(r.norm_w.data_ptr()), ctypes.c_float(r.eps), i(int(r.sigmoid_gate)),
+        v(out.data_ptr()), ll(out.stride(0)), i(r.heads), i(r.vdim), v(_lib.stream_ptr())), "dmoe_gate_norm")
+
+
+def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, segs: SegmentTables) -> torch.Tensor:
+    """q, k [T, kv_heads dim], v, gate [T, heads vdim], beta [T, heads] (delta) straight from the projections (columns of
+    one wider matrix are fine), z fp32 [T, heads dim]. Returns [T, heads vdim]: the recurrence's read-outs, normalised per
+    head, weighed and gated. Convolution inputs and states of the segments' slots are updated."""
+    if not q.is_cuda:
+        return _reference(r, q, k, v, gate, beta, z, state, segs)
+    T = q.shape[0]
+    lib, st = _lib.lib(), ctypes.c_void_p(_lib.stream_ptr())
+    out = torch.empty(T, r.heads * r.vdim, dtype=q.dtype, device=q.device)
+    vt = lib.dmoe_recur_value_tile(r.dim, r.vdim)
+    assert vt > 0, "head too large for the recurrence kernels"
+    raw = None
+    if segs.n_single:
+        d = _descriptor(r, q, k, v, gate, beta, z, state)
+        if r.taps:
+            d.conv_w, d.ring, d.taps = r.conv_w.data_ptr(), state.ring.data_ptr(), r.taps
+        d.segs, d.n_segs = _lib.ptr(segs.singles), segs.n_single
+        d.positions, d.rows, d.kv_slots = _lib.ptr(segs.positions), _lib.ptr(segs.rows), _lib.ptr(segs.kv_slots)
+        svt = vt
+        # few heads in flight: deal the value columns to more CTAs, at the price of a second (norm) launch
+        while svt >= 32 and svt % 8 == 0 and segs.n_single * r.heads * ((r.vdim + svt - 1) // svt) < num_sms(q.device):
+            svt //= 2
+        if svt >= r.vdim:
+            d.out, d.ldo = out.data_ptr(), out.stride(0)
+        else:
+            raw = torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=q.device)
+            d.raw, d.ldraw = raw.data_ptr(), raw.stride(0)
+        _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(svt), st), "dmoe_recur_step")
+        if svt < r.vdim:
+            _gate_norm(r, segs.singles, segs.n_single, 1, raw, gate, out)
+    if segs.n_multi:
+        if raw is None:
+            raw = torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=q.device)
+        qs, vs = r.kv_heads * r.dim, r.heads * r.vdim
+        if r.taps:
+            act = torch.empty(T, r.channels, dtype=q.dtype, device=q.device)
+            d = _descriptor(r, q, k, v, None, None, None, state)
+            d.conv_w, d.ring, d.taps = r.conv_w.data_ptr(), state.ring.data_ptr(), r.taps
+            d.segs, d.n_segs = segs.multi.data_ptr(), segs.n_multi
+            _lib.check(lib.dmoe_conv_chunks(ctypes.byref(d), ctypes.c_void_p(segs.chunks.data_ptr()),
+                                            ctypes.c_int(segs.n_chunks), ctypes.c_void_p(act.data_ptr()),
+                                            ctypes.c_longlong(act.stride(0)), st), "dmoe_conv_chunks")
+            q, k, v = act[:, :qs], act[:, qs:2 * qs], act[:, 2 * qs:]
+        d = _descriptor(r, q, k, v, gate, beta, z, state)
+        d.segs, d.n_segs = segs.multi.data_ptr(), segs.n_multi
+        d.raw, d.ldraw = raw.data_ptr(), raw.stride(0)
+        _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(vt), st), "dmoe_recur_step")
+        _gate_norm(r, segs.chunks, segs.n_chunks, CHUNK, raw, gate, out)
+    return out
+
+
+def _reference(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, segs: SegmentTables) -> torch.Tensor:
+    T, H, G, D, V = q.shape[0], r.heads, r.kv_heads, r.dim, r.vdim
+    if segs.singles is None and segs.n_single:
+        table = [(i, 1, int(segs.rows[i]), int(segs.positions[i])) for i in range(segs.n_single) if segs.kv_slots[i] >= 0]
+    else:
+        table = segs.singles.tolist() + segs.multi.tolist()
+    zb = z.float() + r.z_bias
+    logd = (-torch.exp(r.a_log)[:, None] * torch.nn.functional.softplus(zb).view(T, H, D)) if r.delta else \
+        torch.nn.functional.logsigmoid(zb).view(T, H, D) / r.tau
+    out = torch.zeros(T, H * V, dtype=q.dtype)
+    for a, n, slot, pos0 in table:
+        x = torch.cat([q[a:a + n], k[a:a + n], v[a:a + n]], 1)
+        if r.taps:
+            x = reference.conv_segment(x, r.conv_w, state.ring[slot], pos0)
+        qq, kk = (x[:, j * G * D:(j + 1) * G * D].view(n, G, D).repeat_interleave(H // G, 1) for j in (0, 1))
+        o = reference.recur_segment(qq, kk, x[:, 2 * G * D:].view(n, H, V), None if beta is None else beta[a:a + n],
+                                    logd[a:a + n], state.S[slot], pos0, r.delta, D ** -0.5)
+        o = reference.gate_norm(o, gate[a:a + n].view(n, H, V), r.norm_w, r.eps, r.sigmoid_gate)
+        out[a:a + n] = o.reshape(n, H * V).to(q.dtype)
+    return out

@@ -58,12 +58,15 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slots: Optional[t
 
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
-                    scale: Optional[float] = None) -> torch.Tensor:
-    """Token t attends to the first ctx_len[t] cached tokens of block-table row bt_row[t] (default t)."""
+                    scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None
+                    ) -> torch.Tensor:
+    """Token t attends to the first ctx_len[t] cached tokens of block-table row bt_row[t] (default t), or to the last
+    ``window`` of them; ``softcap``: scores become cap * tanh(score / cap)."""
     T = q.shape[0]
     block_size = kcache.shape[1]
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
-    out = torch.zeros(T, n_q * hd, dtype=torch.float32, device=q.device)
+    vd = vcache.shape[-1]
+    out = torch.zeros(T, n_q * vd, dtype=torch.float32, device=q.device)
     gq = n_q // n_kv
     for t in range(T):
         L = int(ctx_len[t])
@@ -73,9 +76,13 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         nb = (L + block_size - 1) // block_size
         blocks = block_tables[row, :nb].long()
         k = kcache[blocks].reshape(nb * block_size, n_kv, hd)[:L].float()
-        v = vcache[blocks].reshape(nb * block_size, n_kv, hd)[:L].float()
+        v = vcache[blocks].reshape(nb * block_size, n_kv, vd)[:L].float()
+        if window:
+            k, v = k[-window:], v[-window:]
         qt = q[t].float().view(n_kv, gq, hd)
         s = torch.einsum("kgd,lkd->kgl", qt, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         p = torch.softmax(s, dim=-1)
         o = torch.einsum("kgl,lkd->kgd", p, v)
         out[t] = o.reshape(-1)
@@ -149,3 +156,83 @@ def permute_rows(src: torch.Tensor, mapping: torch.Tensor, repeat: int = 1, gath
     ok = m >= 0
     out[m[ok]] = src[idx[ok]]
     return out
+
+
+# ---- decoders with an fp32 residual stream ---------------------------------------------------------------------------
+def _rms_scale(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def resid_norm(resid, y, post, pre, eps, dtype, out_scale=1.0, rows=None):
+    """resid (+)= norm(y) * post; returns norm(resid) * pre * out_scale (of ``rows`` only, resid untouched)."""
+    if rows is not None:
+        resid, y = resid[rows.long()], (y[rows.long()] if y is not None else None)
+    x = resid
+    if y is not None:
+        x = resid + _rms_scale(y.float(), eps) * post
+        if rows is None:
+            resid.copy_(x)
+    return None if pre is None else (_rms_scale(x, eps) * pre * out_scale).to(dtype)
+
+
+def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps) -> None:
+    """Per-head norm + partial rotation of q (in place) and k, K / V append at slots >= 0."""
+    T = qkv.shape[0]
+
+    def turn(x, w):
+        x = _rms_scale(x.float(), eps) * w
+        if table is None:
+            return x
+        half = table.shape[1]
+        c, s = (table[positions.long()][:, None, :, j] for j in (0, 1))
+        u, v = x[..., :half], x[..., half:2 * half]
+        return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
+
+    qs, ks = n_q * dk, n_kv * dk
+    q = turn(qkv[:, :qs].reshape(T, n_q, dk), qw).to(qkv.dtype)
+    if n_kv:
+        k = turn(qkv[:, qs:qs + ks].reshape(T, n_kv, dk), kw).to(qkv.dtype)
+        ok = slots >= 0
+        kcache.view(-1, n_kv, dk)[slots[ok]] = k[ok]
+        vcache.view(-1, n_kv, dv)[slots[ok]] = qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
+    qkv[:, :qs] = q.reshape(T, qs)
+
+
+# ---- linear recurrences ----------------------------------------------------------------------------------------------
+def conv_segment(x: torch.Tensor, w: torch.Tensor, ring: Optional[torch.Tensor], pos0: int) -> torch.Tensor:
+    """Causal depthwise convolution + silu of one segment's rows x [n, C] that start at position pos0; ``ring`` [taps, C]
+    holds earlier inputs at their position modulo taps and takes this segment's last ones."""
+    n, taps = x.shape[0], w.shape[1]
+    hist = [ring[(pos0 - j) % taps] if pos0 - j >= 0 else torch.zeros_like(x[0]) for j in range(taps - 1, 0, -1)]
+    full = torch.cat([torch.stack(hist), x]) if hist else x
+    acc = sum(full[j:j + n].float() * w[:, j] for j in range(taps))
+    for j in range(max(0, n - taps + 1), n):
+        ring[(pos0 + j) % taps] = x[j]
+    return torch.nn.functional.silu(acc).to(x.dtype)
+
+
+def recur_segment(q, k, v, beta, logd, state: torch.Tensor, pos0: int, delta: bool, qscale: float) -> torch.Tensor:
+    """Token-by-token recurrence of one segment: q, k, logd [n, H, D], v [n, H, V], beta [n, H] (delta); ``state``
+    [H, D, V] is read (zero where pos0 = 0) and updated. Returns fp32 read-outs [n, H, V]."""
+    q, k, v = q.float(), k.float(), v.float()
+    if delta:
+        q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6)
+        k = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+    q = q * qscale
+    S = state.clone() if pos0 > 0 else torch.zeros_like(state)
+    out = []
+    for t in range(q.shape[0]):
+        S = S * torch.exp(logd[t])[..., None]
+        u = v[t]
+        if delta:
+            u = torch.sigmoid(beta[t].float())[:, None] * (u - torch.einsum("hdv,hd->hv", S, k[t]))
+        S = S + k[t][..., None] * u[:, None, :]
+        out.append(torch.einsum("hdv,hd->hv", S, q[t]))
+    state.copy_(S)
+    return torch.stack(out)
+
+
+def gate_norm(o: torch.Tensor, gate: torch.Tensor, norm_w: torch.Tensor, eps: float, sigmoid_gate: bool) -> torch.Tensor:
+    """o [n, H, V] fp32 -> norm over V * norm_w * (sigmoid | silu)(gate)."""
+    g = gate.float()
+    return _rms_scale(o, eps) * norm_w * (torch.sigmoid(g) if sigmoid_gate else torch.nn.functional.silu(g))
