@@ -26,8 +26,9 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
 from benchmark.utils import get_parser_base
 from benchmark.workload import Workload, get_generator
-from disagmoe_b200.config import CacheConfig, SamplingConfig, get_preset
+from disagmoe_b200.config import CacheConfig, LayerListConfig, SamplingConfig
 from disagmoe_b200.frontend.datatypes import SloStat
+from disagmoe_b200.models.registry import resolve_model
 from disagmoe_b200.utils.placement import ClusterConfig, get_model_placement
 
 
@@ -79,8 +80,21 @@ def analyze_results(results: List[SloStat], arrivals: Dict[int, float], duration
         ttft_mean_ms=float(np.mean(ttft)) * ms, ttft_p99_ms=float(np.percentile(ttft, 99)) * ms)
 
 
+def model_from_args(args):
+    """(configuration, weights or None for random ones) of --model: a preset or a checkpoint folder."""
+    cfg, weights = resolve_model(args.model)
+    if isinstance(cfg, LayerListConfig):
+        if args.backend != "colocated":
+            raise SystemExit(f"{cfg.name} has no routed experts to place on other GPUs: use --backend colocated")
+        longest = args.max_input_len + args.max_output_len
+        return cfg.clone(max_seq_len=(longest + 15) // 16 * 16, graph_stride=args.graph_stride), weights
+    return model_config_from_args(args), weights
+
+
 def model_config_from_args(args):
-    cfg = get_preset(args.model)
+    cfg, _ = resolve_model(args.model)
+    if isinstance(cfg, LayerListConfig):
+        return model_from_args(args)[0]
     if args.model in ("mixtral", "duo"):
         cfg = cfg.clone(num_layers=args.num_layers, num_experts=args.num_experts, top_k=args.topk)
     return cfg.clone(ep_size=args.ep_size, tp_size=args.tp_size, dp_size=args.dp_size,
@@ -145,7 +159,7 @@ def run_benchmark_controller(master, cfg, wl: Workload, args):
     return stats, arrivals, time.time() - t0
 
 
-def run_benchmark_colocated(cfg, wl: Workload, args):
+def run_benchmark_colocated(cfg, wl: Workload, args, weights=None):
     """One GPU, fused executor: the driver loop admits arrived requests and steps the engine."""
     import torch
     from disagmoe_b200.frontend.colocated import ColocatedEngine
@@ -159,7 +173,7 @@ def run_benchmark_colocated(cfg, wl: Workload, args):
                                   num_gpu_blocks=args.num_blocks), device=args.device,
                  max_batch_size=args.max_batch_size_attn,
                  max_prefill_tokens=max(args.max_input_len, args.max_batch_size_attn, 2048) + (budget if budget > 0 else 0),
-                 enable_cuda_graph=args.cuda_graph_attn,
+                 enable_cuda_graph=args.cuda_graph_attn, state_dict=weights,
                  dtype=torch.float32 if args.device == "cpu" else None, **kw)
     if args.cuda_graph_attn:
         eng.executor.capture()
@@ -273,8 +287,8 @@ def main(argv=None):
     prefix = os.path.join(os.path.dirname(os.path.abspath(args.file)), "")
     try:
         if args.backend == "colocated":
-            cfg = model_config_from_args(args)
-            stats, arrivals, dur = run_benchmark_colocated(cfg, wl, args)
+            cfg, weights = model_from_args(args)
+            stats, arrivals, dur = run_benchmark_colocated(cfg, wl, args, weights)
             sampler_steps, queueing = [], {}
         else:
             master, cfg = launch(args)

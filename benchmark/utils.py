@@ -25,7 +25,8 @@ def get_parser_base() -> ArgumentParser:
     p.add_argument("--seed", type=int, default=0)
     p.add_argument("--duration", type=float, default=0, help="generate requests for this many seconds instead of -n")
     # model
-    p.add_argument("--model", type=str, default="mixtral", help="preset: mixtral | qwen-moe | deepseek-v2-lite | tiny")
+    p.add_argument("--model", type=str, default="mixtral", help="preset: mixtral | qwen-moe | deepseek-v2-lite | tiny | rurunex, or a checkpoint folder with config.json "
+                        "and model.safetensors (colocated backend)")
     p.add_argument("-ca", "--cuda-graph-attn", action="store_true", default=False)
     p.add_argument("-N", "--num-nodes", type=int, default=1)
     p.add_argument("-g", "--num-gpus", type=int, default=4)

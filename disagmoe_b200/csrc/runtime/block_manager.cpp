@@ -3,12 +3,11 @@
 namespace dmoe {
 
 BlockManager::BlockManager(int block_size, int num_blocks, int reserved_blocks, int max_rows)
-    : block_size_(block_size), num_blocks_(num_blocks), reserved_blocks_(reserved_blocks) {
+    : block_size_(block_size), num_blocks_(num_blocks), reserved_blocks_(reserved_blocks), max_rows_(max_rows) {
   DMOE_CHECK(block_size > 0 && num_blocks >= 0 && reserved_blocks >= 0, "bad block manager sizes");
   const int total = num_blocks + reserved_blocks;
   free_.reserve(total);
   for (int b = total - 1; b >= 0; --b) free_.push_back(b);  // block 0 is handed out first
-  (void)max_rows;
 }
 
 int BlockManager::num_free_blocks() {
@@ -46,6 +45,7 @@ void BlockManager::allocate(int seq_id, int seq_len) {
     s.row = free_rows_.back();
     free_rows_.pop_back();
   } else {
+    DMOE_CHECK(max_rows_ <= 0 || next_row_ < max_rows_, "all " << max_rows_ << " sequence rows are in use");
     s.row = next_row_++;
   }
   s.blocks.reserve(need);

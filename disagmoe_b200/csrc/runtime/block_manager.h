@@ -1,5 +1,7 @@
 // Paged-KV block allocator of an attention worker.
 //
+// A row also numbers the sequence's slot in the state pools of recurrent layers; max_rows > 0 bounds the rows in use.
+//
 // Blocks are handed out from a LIFO free list (recently released blocks are still warm in L2). Every sequence
 // also owns one ROW of the device-resident block table; the manager records each (row, column, block) change so
 // that the executor can patch the device table incrementally instead of re-uploading it every step.
@@ -57,7 +59,7 @@ class BlockManager {
     std::vector<int> blocks;
     int row;
   };
-  int block_size_, num_blocks_, reserved_blocks_;
+  int block_size_, num_blocks_, reserved_blocks_, max_rows_;
   std::mutex mu_;
   std::vector<int> free_;       // LIFO
   std::vector<int> free_rows_;  // LIFO
