@@ -1,0 +1,141 @@
+"""Prefill and decode throughput of layer-list decoders (Rurunex design) beside a dense decoder of equal size.
+
+    python bench.py --layer-list [--steps K --warmup W]
+
+Both run through the same engine classes with random weights: the layer-list model repeats (gated linear attention,
+channel-wise delta rule, windowed attention), every layer with a gated feed-forward; the dense model is the MoE decoder
+with a dense feed-forward in every layer, full attention, the same width, heads, feed-forward and number of layers.
+Prints one JSON line per (size, phase, model): tokens/s from device-timed steps (CUDA events, inputs larger than L2 for
+the larger sizes, L2 flushed between steps otherwise), and one per (size, phase) with the device time per kernel.
+"""
+from __future__ import annotations
+
+import json
+import statistics
+from typing import Dict, List
+
+import torch
+
+from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, LayerSpec,
+                                  ModelConfig, RotarySpec)
+from disagmoe_b200.frontend.colocated import ColocatedEngine
+from disagmoe_b200.ops import _lib, gemm
+
+# name: width, heads, kv heads, head size, feed-forward, layers
+SIZES = {"1024": (1024, 8, 2, 128, 2816, 6), "2048": (2048, 16, 4, 128, 5632, 6), "4096": (4096, 32, 8, 128, 11264, 6)}
+VOCAB = 32000
+
+
+def hybrid_config(size: str, window: int = 1024, max_seq_len: int = 8192) -> LayerListConfig:
+    W, H, G, D, ff, n = SIZES[size]
+    layers: List[LayerSpec] = []
+    for i in range(0, n, 3):
+        attn = AttentionSpec(H, G, D, D, D ** -0.5, RotarySpec(D, 1e6, 4.0, 8192), window, 30.0, 2 if i else None)
+        layers += [LayerSpec(GatedLinearSpec(H, D, D, 16.0, 16), ff), LayerSpec(ChannelDeltaSpec(H, H, D, D, 4, D, D), ff),
+                   LayerSpec(attn, ff)]
+    return LayerListConfig.make(W, VOCAB, layers, max_seq_len=max_seq_len, embed_scale=32.0, name="rurunex-" + size)
+
+
+def dense_config(size: str, max_seq_len: int = 8192) -> ModelConfig:
+    W, H, G, D, ff, n = SIZES[size]
+    return ModelConfig(hidden_size=W, num_layers=n, num_heads=H, num_kv_heads=G, num_experts=1, intermediate_size=ff,
+                       dtype=torch.bfloat16, ep_size=1, top_k=1, vocab_size=VOCAB, head_dim=D, rope_theta=1e6,
+                       first_k_dense=n, dense_intermediate_size=ff, max_seq_len=max_seq_len, name="dense-" + size)
+
+
+def make_engine(cfg, batch: int, prompt_tokens: int, ctx: int, steps: int) -> ColocatedEngine:
+    blocks = max(batch * ((ctx + steps + 32) // 16 + 1), prompt_tokens // 16 + 64)
+    eng = ColocatedEngine(cfg, CacheConfig(block_size=16), device="cuda", max_batch_size=batch,
+                          max_prefill_tokens=max(batch, prompt_tokens), num_blocks=blocks)
+    ex = eng.executor
+    if hasattr(ex, "kv_cache"):
+        ex.kv_cache.normal_(0, 0.5)
+    else:
+        for k, v in ex.kv.values():
+            k.normal_(0, 0.5), v.normal_(0, 0.5)
+        for s in ex.states.values():
+            s.S.normal_(0, 0.1)
+    ex.capture([batch])
+    return eng
+
+
+class Flush:
+    """Overwrites a buffer larger than L2 between timed steps."""
+
+    def __init__(self):
+        self.buf = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def __call__(self):
+        self.buf.zero_()
+
+
+def timed(fn, steps: int, warmup: int, flush) -> float:
+    """Median device milliseconds of fn."""
+    out = []
+    for i in range(warmup + steps):
+        flush()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= warmup:
+            out.append(a.elapsed_time(b))
+    return statistics.median(out)
+
+
+def kernel_times(fn) -> Dict[str, list]:
+    fn()
+    torch.cuda.synchronize()
+    _lib.start_timeline()
+    fn()
+    return {k: [n, round(ms, 4)] for k, (n, ms) in sorted(_lib.stop_timeline().items(), key=lambda kv: -kv[1][1])}
+
+
+def rows_of(n_seqs: int, length: int, block: int = 16):
+    """Host tensors of n_seqs prompts of one length, each in its own pages and row."""
+    pos = torch.arange(length, dtype=torch.int32).repeat(n_seqs)
+    row = torch.arange(n_seqs, dtype=torch.int32).repeat_interleave(length)
+    per = (length + block - 1) // block * block
+    slots = row.long() * per + pos.long()
+    ids = torch.randint(0, VOCAB, (n_seqs * length,), generator=torch.Generator().manual_seed(0), dtype=torch.int32)
+    return ids, pos, slots, pos + 1, row, per // block
+
+
+def main(args) -> int:
+    flush = Flush()
+    for size in (args.layer_list_sizes or "1024,2048,4096").split(","):
+        for phase, n, length in (("prefill", 1, 4096), ("prefill", 4, 2048), ("decode", 16, 2048), ("decode", 256, 1024)):
+            for cfg in (hybrid_config(size), dense_config(size)):
+                B = n if phase == "decode" else 8
+                eng = make_engine(cfg, B, n * length if phase == "prefill" else B, length if phase == "decode" else 16, 8)
+                ex = eng.executor
+                if phase == "prefill":
+                    ids, pos, slots, ctx, row, nb = rows_of(n, length)
+                    for r in range(n):
+                        ex.set_block_table_row(r, list(range(r * nb, (r + 1) * nb)))
+                    ends = [(r + 1) * length - 1 for r in range(n)]
+                    step = eager = lambda: ex.prefill(ids, pos, slots, ctx, row, out_rows=ends)
+                else:
+                    nb = length // 16 + 1
+                    for r in range(n):
+                        ex.set_block_table_row(r, list(range(r * nb, (r + 1) * nb)))
+                    pos = torch.full((n,), length - 1, dtype=torch.int32)
+                    row = torch.arange(n, dtype=torch.int32)
+                    slots = row.long() * nb * 16 + length - 1
+                    ids = torch.zeros(n, dtype=torch.int32)
+                    step = lambda: ex.decode(ids, pos, slots, pos + 1, row)
+
+                    def eager():
+                        sizes, ex.graph_sizes = ex.graph_sizes, []
+                        ex.decode(ids, pos, slots, pos + 1, row)
+                        ex.graph_sizes = sizes
+                ms = timed(step, max(3, args.steps), max(3, args.warmup), flush)
+                toks = n * length if phase == "prefill" else n
+                print(json.dumps({"model": cfg.name, "phase": phase, "sequences": n, "length": length, "ms": round(ms, 3),
+                                  "tokens_per_s": round(toks / ms * 1e3, 1), "launches": ex.graph_launches.get(n),
+                                  "kernel_status": gemm.check_status("cuda")}), flush=True)
+                print(json.dumps({"kernels_ms": kernel_times(eager)}), flush=True)
+                del eng, ex, step, eager
+                torch.cuda.empty_cache()
+    return 0

@@ -17,7 +17,7 @@
 // Reference behaviour covered: vLLM paged attention / flash_attn_with_kvcache reached from
 // disagmoe/models/attention.py:150-155,219 with metadata built at disagmoe/frontend/engine.py:429-485.
 #include "dmoe_kernels.h"
-#include "sm100.cuh"
+#include "mma_sync.cuh"
 
 namespace dmoe {
 
@@ -37,11 +37,6 @@ __device__ __forceinline__ void cvt8(const bf16x8a& p, float* f) {
   }
 }
 
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
-  // src-size 0 zero-fills the 16 destination bytes (rows past the end of the context)
-  const int sz = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
-}
 // The decode kernel reads every K / V byte once per step: an evict-first L2 policy keeps that stream from pushing the
 // small hot tensors of the neighbouring kernels (residual rows, norm and gate weights, staged activations) out of L2.
 __device__ __forceinline__ uint64_t l2_stream_policy() {
@@ -54,31 +49,6 @@ __device__ __forceinline__ void cp_async16_stream(uint32_t dst, const void* src,
   asm volatile("cp.async.cg.shared.global.L2::cache_hint [%0], [%1], 16, %2, %3;" ::"r"(dst), "l"(src), "r"(sz), "l"(policy)
                : "memory");
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-// D (16x8 fp32) += A (16x16 bf16, row) * B (16x8 bf16, col)
-__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
-
 // Options of the EXT instantiations of both kernels (plain ones compile without them):
 //   window > 0: a query at position p sees only keys in (p - window, p];
 //   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap).
@@ -93,7 +63,6 @@ __device__ __forceinline__ float attn_score(float raw, float scale_log2, const A
   if (EXT && x.cap_log2 > 0.f) return x.cap_log2 * (1.f - __fdividef(2.f, exp2f(raw * x.cap_in) + 1.f));
   return raw * scale_log2;
 }
-__device__ __forceinline__ float bf16_rest(float v) { return v - __bfloat162float(__float2bfloat16(v)); }
 
 constexpr int kAttnStages = 3;     // cp.async ring depth, per warp
 constexpr int kAttnStageTok = 16;  // cached tokens per stage and warp (block_size must be a multiple of it)

@@ -183,6 +183,10 @@ int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream);
 int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw, const void* gate,
                    long long ldg, const float* norm_w, float eps, int gate_kind, void* out, long long ldo, int heads, int V,
                    void* stream);
+// The same recurrence chunk by chunk on the tensor cores (recurrent_chunk.cu), bf16 activations, for segments of any length.
+int dmoe_recur_chunk_ok(int dim, int vdim);
+long long dmoe_recur_chunk_bytes(int dim, int vdim, int delta, int n_chunks);
+int dmoe_recur_chunks(const DmoeRecur* a, const void* chunks, int n_chunks, void* ws, long long ws_bytes, void* stream);
 int dmoe_conv_chunks(const DmoeRecur* a, const void* chunks, int n_chunks, void* out, long long ldo, void* stream);
 
 // ---- routing (moe.cu) -------------------------------------------------------------------------------

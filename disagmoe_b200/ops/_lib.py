@@ -92,6 +92,7 @@ def lib():
         _LIB.dmoe_gemm.argtypes = [ctypes.POINTER(DmoeGemm), ctypes.c_void_p]
         _LIB.dmoe_gemm.restype = ctypes.c_int
         _LIB.dmoe_gemm_workspace_bytes.restype = ctypes.c_longlong
+        _LIB.dmoe_recur_chunk_bytes.restype = ctypes.c_longlong
         _LIB.dmoe_norm_gather.argtypes = [ctypes.POINTER(DmoeNormGather), ctypes.c_void_p]
         _LIB.dmoe_route_dispatch.argtypes = [ctypes.POINTER(DmoeRouteDispatch), ctypes.c_void_p]
         _LIB.dmoe_set_flag_wait_cycles.argtypes = [ctypes.c_longlong]

@@ -1,4 +1,4 @@
-"""Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``): gated linear attention and the gated
+"""Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``, ``recurrent_chunk.cu``): gated linear attention and the gated
 delta rule, with one decay per head and key channel. CUDA tensors run the kernels, CPU tensors the PyTorch restatements.
 
 A step's rows fall into segments (consecutive rows of one sequence). One-token segments (decoding) take one launch from
@@ -19,6 +19,7 @@ from .gemm import num_sms
 
 CHUNK = 64          # tokens of a chunk
 MAX_TAPS = 8        # longest short convolution
+WORKSPACE = 512 << 20   # bytes of scratch the chunked kernels may use; more heads than fit run in groups
 
 
 @dataclass
@@ -173,7 +174,14 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
         d = _descriptor(r, q, k, v, gate, beta, z, state)
         d.segs, d.n_segs = segs.multi.data_ptr(), segs.n_multi
         d.raw, d.ldraw = raw.data_ptr(), raw.stride(0)
-        _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(vt), st), "dmoe_recur_step")
+        if q.dtype == torch.bfloat16 and lib.dmoe_recur_chunk_ok(r.dim, r.vdim):
+            per_head = lib.dmoe_recur_chunk_bytes(r.dim, r.vdim, int(r.delta), segs.n_chunks)
+            ws = torch.empty(max(per_head, min(per_head * r.heads, WORKSPACE)), dtype=torch.uint8, device=q.device)
+            _lib.check(lib.dmoe_recur_chunks(ctypes.byref(d), ctypes.c_void_p(segs.chunks.data_ptr()),
+                                             ctypes.c_int(segs.n_chunks), ctypes.c_void_p(ws.data_ptr()),
+                                             ctypes.c_longlong(ws.numel()), st), "dmoe_recur_chunks")
+        else:
+            _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(vt), st), "dmoe_recur_step")
         _gate_norm(r, segs.chunks, segs.n_chunks, CHUNK, raw, gate, out)
     return out
 
