@@ -1,0 +1,78 @@
+"""Recurrent layers alone: prompts (chunked kernels) and decode steps, gated linear attention and the channel-wise delta rule.
+
+    python -m benchmark.ops.recurrence [--heads 16] [--dim 128] [--tokens 4096] [--batch 256]
+
+Device time (CUDA events, L2 flushed in between) beside the bytes the operation has to move: projections in, output out and,
+for a decode step, every state read and written once.
+"""
+import argparse
+import json
+import os
+import statistics
+import sys
+
+import torch
+
+sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))))
+
+from disagmoe_b200.ops.recurrent import Recurrence, build_segments, decode_segments, recurrent_attention
+
+
+def layer(kind, H, D, V, dev="cuda"):
+    r = lambda *s: torch.randn(*s, device=dev)
+    if kind == "gla":
+        return Recurrence(H, H, D, V, False, r(H * D) + 2.0, 1 + 0.1 * r(V), 1e-6, tau=16.0)
+    return Recurrence(H, H, D, V, True, 0.5 * r(H * D) - 4.0, 1 + 0.1 * r(V), 1e-6, a_log=0.3 * r(H),
+                      conv_w=0.5 * r(2 * H * D + H * V, 4), sigmoid_gate=True)
+
+
+def main():
+    p = argparse.ArgumentParser()
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--dim", type=int, default=128)
+    p.add_argument("--tokens", type=int, default=4096, help="prompt tokens")
+    p.add_argument("--prompts", type=int, default=1)
+    p.add_argument("--batch", type=int, default=256, help="decoding sequences")
+    p.add_argument("--iters", type=int, default=10)
+    p.add_argument("--only", default="", help="prompt | decode")
+    a = p.parse_args()
+    H, D = a.heads, a.dim
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    peak = json.load(open("MEASURED_PEAKS.json"))["hbm_gbs"] if os.path.exists("MEASURED_PEAKS.json") else 6650.0
+    for kind in ("gla", "delta"):
+        r = layer(kind, H, D, D)
+        for phase in ("prompt", "decode"):
+            if a.only not in ("", phase):
+                continue
+            T = a.tokens if phase == "prompt" else a.batch
+            b = lambda n: torch.randn(T, n, device="cuda").bfloat16()
+            x = b(4 * H * D + H)
+            q, k, v, gate, beta = (x[:, i * H * D:(i + 1) * H * D] for i in range(4)), None, None, None, x[:, 4 * H * D:]
+            q, k, v, gate = q
+            z = torch.randn(T, H * D, device="cuda")
+            state = r.new_state(a.batch if phase == "decode" else a.prompts, torch.bfloat16, "cuda")
+            if phase == "prompt":
+                n = T // a.prompts
+                segs = build_segments(torch.arange(a.prompts).repeat_interleave(n), torch.arange(n).repeat(a.prompts), "cuda")
+            else:
+                i = torch.arange(T, device="cuda")
+                segs = decode_segments(torch.full((T,), 100, dtype=torch.int32, device="cuda"), i.int(), i)
+            fn = lambda: recurrent_attention(r, q, k, v, gate, beta if kind == "delta" else None, z, state, segs)
+            ms = []
+            for it in range(a.iters + 3):
+                flush.zero_()
+                e = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+                e[0].record()
+                fn()
+                e[1].record()
+                torch.cuda.synchronize()
+                ms.append(e[0].elapsed_time(e[1]))
+            t = statistics.median(ms[3:])
+            moved = T * H * D * (2 * 5 + 4) + (2 * state.S.numel() * 4 if phase == "decode" else 0)
+            print(json.dumps({"kind": kind, "phase": phase, "tokens": T, "heads": H, "dim": D, "us": round(t * 1e3, 1),
+                              "MB": round(moved / 1e6, 1), "GB_s": round(moved / t / 1e6), "of_measured_copy": round(moved / t / 1e6 / peak, 3)}),
+                  flush=True)
+
+
+if __name__ == "__main__":
+    main()

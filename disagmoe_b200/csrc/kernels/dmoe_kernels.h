@@ -176,7 +176,9 @@ typedef struct DmoeRecur {
   int decay_kind;           // 0: log a = log sigmoid(z + b) * inv_tau, 1: log a = -exp(a_log) softplus(z + b)
   int gate_kind;            // 0: silu, 1: sigmoid
   int is_f32;
+  int one_token;            // dmoe_recur_step: every segment has one token
   float qscale, inv_tau, eps;
+  int* status;              // optional device status word: non-zero after a bounded wait gave up
 } DmoeRecur;
 int dmoe_recur_value_tile(int dim, int vdim);
 int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream);

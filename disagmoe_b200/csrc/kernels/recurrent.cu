@@ -11,8 +11,8 @@
 // Work is described by tables that the host builds once per step:
 //   segs    int4 {first row, tokens, slot, position of the first token}; a segment = consecutive rows of one sequence
 //   chunks  int4 {first row, tokens <= 64, segment, chunk number in the segment}
-// Segments of one token (decoding) take step_kernel, which does everything from the raw projections to the gated,
-// normalised output in one launch. Longer ones are convolved by conv_chunk_kernel and then run either through the chunked
+// Segments of one token (decoding) take stream_step_kernel or step_kernel, which do everything from the raw projections to
+// the gated, normalised output in one launch. Longer ones are convolved by conv_chunk_kernel and then run either through the chunked
 // tensor-core kernels of recurrent_chunk.cu or, token by token in fp32 arithmetic, through step_kernel.
 #include "dmoe_kernels.h"
 #include "recurrent.cuh"
@@ -22,28 +22,84 @@ namespace dmoe {
 constexpr int kStepThreads = 256;
 constexpr int kStepRows = 16;        // state rows a thread holds in registers
 
+// Decay factor, q and k of the token's key channels and its values -> shared memory (convolved and activated with CONV).
+template <typename T, bool DELTA, bool CONV>
+__device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, int pos, int slot, int h, int hk, int v0, int nv,
+                                             float decay_scale, float4* s_gqk, float* s_v) {
+  const int D = a.dim, V = a.vdim, group = a.heads / a.kv_heads;
+  for (int i = threadIdx.x; i < D + nv; i += blockDim.x) {
+    if (i < D) {
+      const float z = a.z[row * a.ldz + h * D + i] + a.z_bias[h * D + i];
+      float q, k;
+      if (CONV) {
+        ConvInputs<T> xq, xk;
+        xq.load(a, row, pos, slot, hk * D + i, a.q, a.ldq, hk * D + i);
+        xk.load(a, row, pos, slot, (a.kv_heads + hk) * D + i, a.k, a.ldk, hk * D + i);
+        const bool writes = h % group == 0 && v0 == 0;
+        q = xq.finish(a, pos, slot, hk * D + i, writes);
+        k = xk.finish(a, pos, slot, (a.kv_heads + hk) * D + i, writes);
+      } else {
+        q = static_cast<float>(static_cast<const T*>(a.q)[row * a.ldq + hk * D + i]);
+        k = static_cast<float>(static_cast<const T*>(a.k)[row * a.ldk + hk * D + i]);
+      }
+      s_gqk[i] = make_float4(expf(log_decay(a.decay_kind, z, decay_scale)), q, k, 0.f);
+    } else {
+      const int c = h * V + v0 + i - D;
+      if (CONV) {
+        ConvInputs<T> xv;
+        xv.load(a, row, pos, slot, 2 * a.kv_heads * D + c, a.v, a.ldv, c);
+        s_v[i - D] = xv.finish(a, pos, slot, 2 * a.kv_heads * D + c, true);
+      } else {
+        s_v[i - D] = static_cast<float>(static_cast<const T*>(a.v)[row * a.ldv + c]);
+      }
+    }
+  }
+}
+
+// Factors that turn the raw rows into q (scaled, unit) and k (unit), and q.k of the raw rows; every warp on its own.
+struct RowFactors {
+  float fq, fk, qk;
+};
+template <bool DELTA>
+__device__ __forceinline__ RowFactors row_factors(const DmoeRecur& a, const float4* s_gqk) {
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int d = threadIdx.x & 31; d < a.dim; d += 32) {
+    const float4 x = s_gqk[d];
+    qq += x.y * x.y;
+    kk += x.z * x.z;
+    qk += x.y * x.z;
+  }
+  RowFactors f;
+  f.qk = warp_sum(qk);
+  f.fq = a.qscale;
+  f.fk = 1.f;
+  if (DELTA) {
+    f.fq *= 1.f / sqrtf(warp_sum(qq) + 1e-6f);
+    f.fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+  }
+  return f;
+}
+
 // One CTA: one segment, one head, `vt` value columns. Threads form a grid of (vt / VEC) column groups x rpp row groups;
 // a thread keeps rows rg, rg + rpp, ... of its VEC columns in registers for the whole segment. Per token the read-outs
 // of the decayed state at k and at q are reduced together, and o = (a S)^T q + (k.q) u gives the read-out after the
 // write without a second pass.
 template <typename T, bool DELTA, bool CONV, int VEC>
-__global__ void __launch_bounds__(kStepThreads)
+__global__ void __launch_bounds__(kStepThreads, 2)
 step_kernel(const DmoeRecur a, int vt) {
-  extern __shared__ float s_mem[];
+  extern __shared__ __align__(16) float s_mem[];
   const int tid = threadIdx.x, lane = tid & 31;
   const int4 seg = a.segs != nullptr ? static_cast<const int4*>(a.segs)[blockIdx.x] : row_segment(a, blockIdx.x);
   const int row0 = seg.x, ntok = seg.y, slot = seg.z, pos0 = seg.w;
   if (ntok <= 0 || slot < 0 || slot >= a.n_slots) return;
   const int h = blockIdx.y, D = a.dim, V = a.vdim;
-  const int hk = DELTA ? h / (a.heads / a.kv_heads) : h;
+  const int group = a.heads / a.kv_heads, hk = DELTA ? h / group : h;
   const int v0 = blockIdx.z * vt, nv = min(vt, V - v0);
   const int vq = vt / VEC, rpp = kStepThreads / vq;
   const int cg = tid % vq, rg = tid / vq;
   const bool mine = rg < rpp && cg * VEC < nv;
-  float* s_q = s_mem;                  // [D]
-  float* s_k = s_q + D;                // [D]
-  float* s_g = s_k + D;                // [D] decay factors
-  float* s_v = s_g + D;                // [vt]
+  float4* s_gqk = reinterpret_cast<float4*>(s_mem);    // [D] decay factor, q, k of the token
+  float* s_v = s_mem + 4 * D;          // [vt]
   float* s_u = s_v + vt;               // [vt]
   float* s_o = s_u + vt;               // [vt]
   float* s_red = s_o + vt;             // [DELTA ? 2 : 1][rpp][vt]
@@ -62,41 +118,20 @@ step_kernel(const DmoeRecur a, int vt) {
   for (int t = 0; t < ntok; ++t) {
     const long long row = row0 + t;
     const int pos = pos0 + t;
-    for (int i = tid; i < D + nv; i += kStepThreads) {
-      if (i < D) {
-        float q, k;
-        if (CONV) {
-          q = conv_step<T>(a, row, pos, slot, hk * D + i, a.q, a.ldq, hk * D + i, h % (a.heads / a.kv_heads) == 0 && v0 == 0);
-          k = conv_step<T>(a, row, pos, slot, (a.kv_heads + hk) * D + i, a.k, a.ldk, hk * D + i,
-                           h % (a.heads / a.kv_heads) == 0 && v0 == 0);
-        } else {
-          q = static_cast<float>(static_cast<const T*>(a.q)[row * a.ldq + hk * D + i]);
-          k = static_cast<float>(static_cast<const T*>(a.k)[row * a.ldk + hk * D + i]);
-        }
-        s_q[i] = q;
-        s_k[i] = k;
-        s_g[i] = expf(log_decay(a.decay_kind, a.z[row * a.ldz + h * D + i] + a.z_bias[h * D + i], decay_scale));
-      } else {
-        const int c = h * V + v0 + i - D;
-        s_v[i - D] = CONV ? conv_step<T>(a, row, pos, slot, 2 * a.kv_heads * D + c, a.v, a.ldv, c, true)
-                          : static_cast<float>(static_cast<const T*>(a.v)[row * a.ldv + c]);
-      }
+    // what the end of the step needs, requested before anything waits
+    const bool fused = a.raw == nullptr;
+    const int oc = min(tid, nv - 1);
+    float beta = 0.f, gate = 0.f, weight = 0.f;
+    if (DELTA) beta = static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h]);
+    if (fused) {
+      gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + oc]);
+      weight = a.norm_w[oc];
     }
+    token_inputs<T, DELTA, CONV>(a, row, pos, slot, h, hk, v0, nv, decay_scale, s_gqk, s_v);
     __syncthreads();
-    // every warp: |q|^2, |k|^2 and q.k of the raw rows
-    float qq = 0.f, kk = 0.f, qk = 0.f;
-    for (int d = lane; d < D; d += 32) {
-      const float q = s_q[d], k = s_k[d];
-      qq += q * q;
-      kk += k * k;
-      qk += q * k;
-    }
-    qk = warp_sum(qk);
-    float fq = a.qscale, fk = 1.f;     // factors of the raw rows
-    if (DELTA) {
-      fq *= 1.f / sqrtf(warp_sum(qq) + 1e-6f);
-      fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
-    }
+    const RowFactors f = row_factors<DELTA>(a, s_gqk);
+    const float fq = f.fq, fk = f.fk, qk = f.qk;
+    if (DELTA) beta = 1.f / (1.f + expf(-beta));
     float rq[VEC], rk[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) rq[e] = rk[e] = 0.f;
@@ -105,37 +140,32 @@ step_kernel(const DmoeRecur a, int vt) {
       for (int i = 0; i < kStepRows; ++i) {
         const int d = rg + i * rpp;
         if (d < D) {
-          const float g = s_g[d], q = s_q[d], k = s_k[d];
+          const float4 x = s_gqk[d];
 #pragma unroll
           for (int e = 0; e < VEC; ++e) {
-            S[i][e] *= g;
-            rq[e] += S[i][e] * q;
-            if (DELTA) rk[e] += S[i][e] * k;
+            S[i][e] *= x.x;
+            rq[e] += S[i][e] * x.y;
+            if (DELTA) rk[e] += S[i][e] * x.z;
           }
         }
       }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        s_red[rg * vt + cg * VEC + e] = rq[e];
-        if (DELTA) s_red[(rpp + rg) * vt + cg * VEC + e] = rk[e];
-      }
+      store_vec<VEC>(s_red + rg * vt + cg * VEC, rq);
+      if (DELTA) store_vec<VEC>(s_red + (rpp + rg) * vt + cg * VEC, rk);
     }
     __syncthreads();
     for (int c = tid; c < nv; c += kStepThreads) {
       float oq = 0.f, ok = 0.f;
+#pragma unroll 4
       for (int r = 0; r < rpp; ++r) {
         oq += s_red[r * vt + c];
         if (DELTA) ok += s_red[(rpp + r) * vt + c];
       }
       float u = s_v[c];
-      if (DELTA) {
-        const float beta = 1.f / (1.f + expf(-static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h])));
-        u = beta * (u - ok * fk);
-      }
+      if (DELTA) u = beta * (u - ok * fk);
       s_u[c] = u * fk;
       const float o = oq * fq + qk * fq * fk * u;
-      if (a.raw != nullptr) a.raw[row * a.ldraw + h * V + v0 + c] = o;
-      else s_o[c] = o;
+      if (fused) s_o[c] = o;
+      else a.raw[row * a.ldraw + h * V + v0 + c] = o;
     }
     __syncthreads();
     if (mine) {
@@ -146,34 +176,139 @@ step_kernel(const DmoeRecur a, int vt) {
       for (int i = 0; i < kStepRows; ++i) {
         const int d = rg + i * rpp;
         if (d < D) {
-          const float k = s_k[d];
+          const float k = s_gqk[d].z;
 #pragma unroll
           for (int e = 0; e < VEC; ++e) S[i][e] += k * u[e];
+          if (t + 1 == ntok) store_vec<VEC>(sp + static_cast<long long>(d) * V, S[i]);
         }
       }
     }
-    if (a.raw == nullptr) {
+    if (fused) {
       // the CTA holds the whole head: normalise over the value columns, weigh and gate
       float ss = 0.f;
       for (int c = lane; c < V; c += 32) ss += s_o[c] * s_o[c];
       const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + a.eps);
       for (int c = tid; c < V; c += kStepThreads) {
-        const float g = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
-        static_cast<T*>(a.out)[row * a.ldo + h * V + c] = static_cast<T>(s_o[c] * inv * a.norm_w[c] * gate_value(a.gate_kind, g));
+        if (c != tid) {                // heads wider than the CTA
+          gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
+          weight = a.norm_w[c];
+        }
+        static_cast<T*>(a.out)[row * a.ldo + h * V + c] = static_cast<T>(s_o[c] * inv * weight * gate_value(a.gate_kind, gate));
       }
     }
-    if (t + 1 < ntok) __syncthreads();   // s_k, s_v, s_o are rewritten
+    if (t + 1 < ntok) __syncthreads();   // s_gqk, s_v, s_o are rewritten
   }
+}
+
+// Decode steps at full bandwidth: one CTA per (sequence, head), the head's state fetched by one bulk copy into shared memory
+// while the token's inputs are prepared (three CTAs per SM keep copies in flight), updated from there straight back to
+// global memory. One-token segments, whole heads, vdim a multiple of 4.
+template <typename T, bool DELTA, bool CONV>
+__global__ void __launch_bounds__(kStepThreads, 3)
+stream_step_kernel(const DmoeRecur a) {
+  extern __shared__ __align__(128) float s_stream[];
+  __shared__ __align__(8) unsigned long long s_bar;
+  __shared__ int s_abort;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int4 seg = a.segs != nullptr ? static_cast<const int4*>(a.segs)[blockIdx.x] : row_segment(a, blockIdx.x);
+  const int slot = seg.z, pos = seg.w, h = blockIdx.y, D = a.dim, V = a.vdim;
+  if (seg.y <= 0 || slot < 0 || slot >= a.n_slots) return;
+  const long long row = seg.x;
+  const int hk = DELTA ? h / (a.heads / a.kv_heads) : h;
+  float* s_S = s_stream;                                            // [D][V]
+  float4* s_gqk = reinterpret_cast<float4*>(s_S + D * V);        // [D]
+  float* s_v = reinterpret_cast<float*>(s_gqk + D);              // [V]
+  float* s_red = s_v + V;                                        // [DELTA ? 2 : 1][rpp][V]
+  float* s_u = s_v;                                              // column c of v and of the sums is read by the thread
+  float* s_o = s_red;                                            // that then writes u and o there
+  float* sp = a.state + (static_cast<long long>(slot) * a.heads + h) * D * V;
+  const uint32_t bar = smem_u32(&s_bar);
+  if (tid == 0) {
+    s_abort = 0;
+    mbar_init(bar, 1);
+    mbar_fence_init();
+    if (pos > 0) {
+      const uint32_t bytes = static_cast<uint32_t>(D) * V * 4;
+      mbar_expect_tx(bar, bytes);
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(s_S)),
+                   "l"(sp), "r"(bytes), "r"(bar) : "memory");
+    }
+  }
+  const int vq = V / 4, rpp = kStepThreads / vq, cg = tid % vq, rg = tid / vq;
+  const bool mine = rg < rpp;
+  float beta = 0.f, gate = 0.f, weight = 0.f;
+  if (DELTA) beta = static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h]);
+  if (tid < V) {
+    gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + tid]);
+    weight = a.norm_w[tid];
+  }
+  token_inputs<T, DELTA, CONV>(a, row, pos, slot, h, hk, 0, V, a.decay_kind == 0 ? a.inv_tau : expf(a.a_log[h]), s_gqk, s_v);
+  __syncthreads();                                               // the inputs, and the barrier's initialisation
+  const RowFactors f = row_factors<DELTA>(a, s_gqk);
+  if (DELTA) beta = 1.f / (1.f + expf(-beta));
+  if (pos > 0 && !mbar_wait(bar, 0, &s_abort) && tid == 0 && a.status != nullptr) atomicExch(a.status, kStatusBarrierTimeout);
+  float rq[4] = {0.f, 0.f, 0.f, 0.f}, rk[4] = {0.f, 0.f, 0.f, 0.f};
+  if (mine) {
+    if (pos > 0) {
+#pragma unroll 8
+      for (int d = rg; d < D; d += rpp) {
+        const float4 x = s_gqk[d];
+        const float4 s = *reinterpret_cast<const float4*>(s_S + d * V + cg * 4);
+        const float sv[4] = {s.x * x.x, s.y * x.x, s.z * x.x, s.w * x.x};
 #pragma unroll
-  for (int i = 0; i < kStepRows; ++i) {
-    const int d = rg + i * rpp;
-    if (mine && d < D) store_vec<VEC>(sp + static_cast<long long>(d) * V, S[i]);
+        for (int e = 0; e < 4; ++e) {
+          rq[e] += sv[e] * x.y;
+          if (DELTA) rk[e] += sv[e] * x.z;
+        }
+      }
+    }
+    store_vec<4>(s_red + rg * V + cg * 4, rq);
+    if (DELTA) store_vec<4>(s_red + (rpp + rg) * V + cg * 4, rk);
+  }
+  __syncthreads();
+  if (s_abort) {                                                 // the copy never came: leave state and output alone
+    for (int i = 0; i < (1 << 20) && !mbar_try_wait(bar, 0); ++i) {}
+    return;
+  }
+  for (int c = tid; c < V; c += kStepThreads) {
+    float oq = 0.f, ok = 0.f;
+#pragma unroll 4
+    for (int r = 0; r < rpp; ++r) {
+      oq += s_red[r * V + c];
+      if (DELTA) ok += s_red[(rpp + r) * V + c];
+    }
+    float u = s_v[c];
+    if (DELTA) u = beta * (u - ok * f.fk);
+    s_u[c] = u * f.fk;
+    s_o[c] = oq * f.fq + f.qk * f.fq * f.fk * u;
+  }
+  __syncthreads();
+  if (mine) {
+    const float4 u = *reinterpret_cast<const float4*>(s_u + cg * 4);
+#pragma unroll 8
+    for (int d = rg; d < D; d += rpp) {
+      const float4 x = s_gqk[d];
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (pos > 0) s = *reinterpret_cast<const float4*>(s_S + d * V + cg * 4);
+      *reinterpret_cast<float4*>(sp + static_cast<long long>(d) * V + cg * 4) =
+          make_float4(s.x * x.x + x.z * u.x, s.y * x.x + x.z * u.y, s.z * x.x + x.z * u.z, s.w * x.x + x.z * u.w);
+    }
+  }
+  float ss = 0.f;
+  for (int c = lane; c < V; c += 32) ss += s_o[c] * s_o[c];
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + a.eps);
+  for (int c = tid; c < V; c += kStepThreads) {
+    if (c != tid) {                                              // heads wider than the CTA
+      gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
+      weight = a.norm_w[c];
+    }
+    static_cast<T*>(a.out)[row * a.ldo + h * V + c] = static_cast<T>(s_o[c] * inv * weight * gate_value(a.gate_kind, gate));
   }
 }
 
 // out[row, h, :] = raw / sqrt(mean(raw^2) + eps) * norm_w * gate for the rows of a table (segs or chunks; NULL: entry i is
-// row i); one warp per (row, head)
-template <typename T>
+// row i); one warp per (row, head), VEC consecutive columns per lane and pass
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, long long ldraw, const T* __restrict__ gate,
                  long long ldg, const float* __restrict__ norm_w, float eps, int gate_kind, T* __restrict__ out,
@@ -184,24 +319,47 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
     const long long row = e.x + i / heads;
     const int h = i % heads;
     const float* r = raw + row * ldraw + h * V;
+    const T* gp = gate + row * ldg + h * V;
+    float x[VEC], gv[VEC], w[VEC];
     float ss = 0.f;
-    for (int c = lane; c < V; c += 32) ss += r[c] * r[c];
+    const int c0 = lane * VEC;
+    if (c0 < V) {                          // the first pass stays in registers (all of it where V <= 32 VEC)
+      load_vec<VEC>(r + c0, x);
+      load_any<VEC>(gp + c0, gv);
+      load_vec<VEC>(norm_w + c0, w);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ss += x[k] * x[k];
+    }
+    for (int c = c0 + 32 * VEC; c < V; c += 32 * VEC) {
+      float y[VEC];
+      load_vec<VEC>(r + c, y);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ss += y[k] * y[k];
+    }
     const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
-    for (int c = lane; c < V; c += 32)
-      out[row * ldo + h * V + c] =
-          static_cast<T>(r[c] * inv * norm_w[c] * gate_value(gate_kind, static_cast<float>(gate[row * ldg + h * V + c])));
+    for (int c = c0; c < V; c += 32 * VEC) {
+      if (c != c0) {
+        load_vec<VEC>(r + c, x);
+        load_any<VEC>(gp + c, gv);
+        load_vec<VEC>(norm_w + c, w);
+      }
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) x[k] *= inv * w[k] * gate_value(gate_kind, gv[k]);
+      store_any<VEC>(out + row * ldo + h * V + c, x);
+    }
   }
 }
 
-// Causal depthwise convolution + silu of the q | k | v projections of one chunk of a segment. The taps before the
-// segment's first row come from the ring: ring[slot][p % taps][channel] = projection at position p.
-template <typename T>
+// Causal depthwise convolution + silu of the q | k | v projections of one chunk of a segment, VEC neighbouring channels per
+// thread. The taps before the segment's first row come from the ring: ring[slot][p % taps][channel] = projection at p.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(128)
 conv_chunk_kernel(const DmoeRecur a, const int4* __restrict__ chunks, T* __restrict__ out, long long ldo) {
+  constexpr int HIST = kMaxTaps - 1, STEP = 8;
   const int4 ck = chunks[blockIdx.x];
   const int4 seg = static_cast<const int4*>(a.segs)[ck.z];
   const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
   if (c >= C || seg.z < 0 || seg.z >= a.n_slots) return;
   const int R = a.taps, qc = a.kv_heads * a.dim;
   const T* src;
@@ -210,26 +368,45 @@ conv_chunk_kernel(const DmoeRecur a, const int4* __restrict__ chunks, T* __restr
   else if (c < 2 * qc) { src = static_cast<const T*>(a.k) + c - qc; ld = a.ldk; }
   else { src = static_cast<const T*>(a.v) + c - 2 * qc; ld = a.ldv; }
   const T* ring = static_cast<const T*>(a.ring) + static_cast<long long>(seg.z) * R * C + c;
-  float w[kMaxTaps], x[kMaxTaps];      // x[j]: input j tokens back
-#pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) {
-    w[j] = j < R ? a.conv_w[static_cast<long long>(c) * R + R - 1 - j] : 0.f;
-    x[j] = 0.f;
-  }
+  float w[kMaxTaps][VEC];               // w[j]: weight of the input j tokens back
+  float x[HIST + STEP][VEC];            // x[HIST + i]: input of row i of the step
   const int pos0 = seg.w + (ck.x - seg.x);     // position of the chunk's first row
 #pragma unroll
-  for (int j = 1; j < kMaxTaps; ++j) {
+  for (int j = 0; j < kMaxTaps; ++j)
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) w[j][e] = j < R ? a.conv_w[static_cast<long long>(c + e) * R + R - 1 - j] : 0.f;
+#pragma unroll
+  for (int j = 1; j <= HIST; ++j) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[HIST - j][e] = 0.f;
     if (j < R && pos0 - j >= 0)
-      x[j] = static_cast<float>(ck.x - j >= seg.x ? src[(ck.x - j) * ld] : ring[static_cast<long long>((pos0 - j) % R) * C]);
+      load_any<VEC>(ck.x - j >= seg.x ? src + (ck.x - j) * ld : ring + static_cast<long long>((pos0 - j) % R) * C, x[HIST - j]);
   }
-  for (int t = 0; t < ck.y; ++t) {
-    x[0] = static_cast<float>(src[(ck.x + t) * ld]);
-    float acc = 0.f;
+  for (int t = 0; t < ck.y; t += STEP) {
 #pragma unroll
-    for (int j = kMaxTaps - 1; j >= 0; --j) acc += w[j] * x[j];
-    out[(ck.x + t) * ldo + c] = static_cast<T>(silu(acc));
+    for (int i = 0; i < STEP; ++i) {
 #pragma unroll
-    for (int j = kMaxTaps - 1; j > 0; --j) x[j] = x[j - 1];
+      for (int e = 0; e < VEC; ++e) x[HIST + i][e] = 0.f;
+      if (t + i < ck.y) load_any<VEC>(src + (ck.x + t + i) * ld, x[HIST + i]);
+    }
+#pragma unroll
+    for (int i = 0; i < STEP; ++i) {
+      if (t + i < ck.y) {
+        float acc[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          acc[e] = 0.f;
+#pragma unroll
+          for (int j = kMaxTaps - 1; j >= 0; --j) acc[e] += w[j][e] * x[HIST + i - j][e];
+          acc[e] = silu(acc[e]);
+        }
+        store_any<VEC>(out + (ck.x + t + i) * ldo + c, acc);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < HIST; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[j][e] = x[STEP + j][e];
   }
 }
 
@@ -260,10 +437,34 @@ static int check_recur(const DmoeRecur* a) {
   return 0;
 }
 
+constexpr int kStreamSmem = 76400;       // three CTAs per SM
+
+// Shared memory of stream_step_kernel, or 0 where it does not apply: whole heads of a multiple of 4 value columns whose
+// state leaves room for three CTAs per SM.
+static size_t stream_smem(const DmoeRecur& a) {
+  if (a.raw != nullptr || a.vdim % 4 != 0 || a.vdim > 4 * kStepThreads || (reinterpret_cast<uintptr_t>(a.state) & 15) != 0)
+    return 0;
+  const int rpp = kStepThreads / (a.vdim / 4);
+  const size_t b = (static_cast<size_t>(a.dim) * a.vdim + 4 * a.dim + a.vdim + static_cast<size_t>(a.delta ? 2 : 1) * rpp * a.vdim) * 4;
+  return b <= kStreamSmem ? b : 0;
+}
+
+template <typename T, bool DELTA, bool CONV>
+static int launch_stream(const DmoeRecur& a, size_t smem, cudaStream_t stream) {
+  static PerDeviceOnce configured;
+  const int rc = configured.run([] {
+    return static_cast<int>(cudaFuncSetAttribute(stream_step_kernel<T, DELTA, CONV>,
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, kStreamSmem));
+  });
+  if (rc != 0) return rc;
+  return static_cast<int>(launch_kernel(stream_step_kernel<T, DELTA, CONV>, dim3(a.n_segs, a.heads), dim3(kStepThreads), smem,
+                                        stream, a));
+}
+
 template <typename T, bool DELTA, bool CONV, int VEC>
 static int launch_step(const DmoeRecur& a, int vt, cudaStream_t stream) {
   const int vq = vt / VEC, rpp = kStepThreads / vq;
-  const size_t smem = (3 * static_cast<size_t>(a.dim) + 3 * vt + static_cast<size_t>(DELTA ? 2 : 1) * rpp * vt) * sizeof(float);
+  const size_t smem = (4 * static_cast<size_t>(a.dim) + 3 * vt + static_cast<size_t>(DELTA ? 2 : 1) * rpp * vt) * sizeof(float);
   if (smem > 48 * 1024) return -13;
   const dim3 grid(a.n_segs, a.heads, (a.vdim + vt - 1) / vt);
   return static_cast<int>(launch_kernel(step_kernel<T, DELTA, CONV, VEC>, grid, dim3(kStepThreads), smem, stream, a, vt));
@@ -272,6 +473,11 @@ static int launch_step(const DmoeRecur& a, int vt, cudaStream_t stream) {
 template <typename T>
 static int step_dispatch(const DmoeRecur& a, int vt, bool vec, cudaStream_t stream) {
   const bool conv = a.taps > 0;
+  const size_t smem = a.one_token ? stream_smem(a) : 0;
+  if (smem > 0) {
+    if (!a.delta) return conv ? -12 : launch_stream<T, false, false>(a, smem, stream);
+    return conv ? launch_stream<T, true, true>(a, smem, stream) : launch_stream<T, true, false>(a, smem, stream);
+  }
   if (!a.delta) {
     if (conv) return -12;
     return vec ? launch_step<T, false, false, 4>(a, vt, stream) : launch_step<T, false, false, 1>(a, vt, stream);
@@ -320,14 +526,20 @@ extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_toke
   long long by = (static_cast<long long>(max_tokens) * heads + 31) / 32;     // about four (row, head) pairs per warp
   if (by > 1024) by = 1024;
   const dim3 grid(n, static_cast<unsigned>(by));
-  if (is_f32)
-    gate_norm_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const int4*>(table), raw, ldraw,
-                                                      static_cast<const float*>(gate), ldg, norm_w, eps, gate_kind,
-                                                      static_cast<float*>(out), ldo, heads, V);
-  else
-    gate_norm_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(
-        static_cast<const int4*>(table), raw, ldraw, static_cast<const __nv_bfloat16*>(gate), ldg, norm_w, eps, gate_kind,
-        static_cast<__nv_bfloat16*>(out), ldo, heads, V);
+  const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = V % 4 == 0 && ldraw % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(raw) && al(gate) && al(out) && al(norm_w);
+#define DMOE_GATE_NORM(T_, VEC_)                                                                                       \
+  gate_norm_kernel<T_, VEC_><<<grid, 256, 0, stream>>>(static_cast<const int4*>(table), raw, ldraw,                    \
+                                                       static_cast<const T_*>(gate), ldg, norm_w, eps, gate_kind,      \
+                                                       static_cast<T_*>(out), ldo, heads, V)
+  if (is_f32) {
+    if (vec) DMOE_GATE_NORM(float, 4);
+    else DMOE_GATE_NORM(float, 1);
+  } else {
+    if (vec) DMOE_GATE_NORM(__nv_bfloat16, 4);
+    else DMOE_GATE_NORM(__nv_bfloat16, 1);
+  }
+#undef DMOE_GATE_NORM
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -339,13 +551,18 @@ extern "C" int dmoe_conv_chunks(const DmoeRecur* a, const void* chunks, int n_ch
   if (n_chunks == 0 || a->n_segs == 0) return 0;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   const int C = 2 * a->kv_heads * a->dim + a->heads * a->vdim;
-  const dim3 g1(n_chunks, (C + 127) / 128), g2(a->n_segs, (C + 255) / 256);
+  const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 3) == 0; };
+  const bool pairs = !a->is_f32 && (a->kv_heads * a->dim) % 2 == 0 && C % 2 == 0 && a->ldq % 2 == 0 && a->ldk % 2 == 0 &&
+                     a->ldv % 2 == 0 && ldo % 2 == 0 && al(a->q) && al(a->k) && al(a->v) && al(out) && al(a->ring);
+  const int per = pairs ? 256 : 128;
+  const dim3 g1(n_chunks, (C + per - 1) / per), g2(a->n_segs, (C + 255) / 256);
+  const int4* ck = static_cast<const int4*>(chunks);
   if (a->is_f32) {
-    conv_chunk_kernel<float><<<g1, 128, 0, stream>>>(*a, static_cast<const int4*>(chunks), static_cast<float*>(out), ldo);
+    conv_chunk_kernel<float, 1><<<g1, 128, 0, stream>>>(*a, ck, static_cast<float*>(out), ldo);
     ring_update_kernel<float><<<g2, 256, 0, stream>>>(*a);
   } else {
-    conv_chunk_kernel<__nv_bfloat16><<<g1, 128, 0, stream>>>(*a, static_cast<const int4*>(chunks),
-                                                             static_cast<__nv_bfloat16*>(out), ldo);
+    if (pairs) conv_chunk_kernel<__nv_bfloat16, 2><<<g1, 128, 0, stream>>>(*a, ck, static_cast<__nv_bfloat16*>(out), ldo);
+    else conv_chunk_kernel<__nv_bfloat16, 1><<<g1, 128, 0, stream>>>(*a, ck, static_cast<__nv_bfloat16*>(out), ldo);
     ring_update_kernel<__nv_bfloat16><<<g2, 256, 0, stream>>>(*a);
   }
   return static_cast<int>(cudaGetLastError());

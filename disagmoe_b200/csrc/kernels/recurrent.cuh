@@ -41,22 +41,89 @@ __device__ __forceinline__ void store_vec(float* p, const float* f) {
   else p[0] = f[0];
 }
 
-// Convolution + silu of one channel of a one-token segment at position pos, from the raw projection `src` and the ring of
-// earlier inputs (ring[slot][p % taps][channel]); the one writing thread of a channel stores the new input. Slot
-// pos % taps is not among the taps - 1 positions that are read, so readers in other CTAs do not race with it.
-template <typename T>
-__device__ __forceinline__ float conv_step(const DmoeRecur& a, long long row, int pos, int slot, int channel,
-                                           const void* src, long long ld, int src_col, bool writes) {
-  const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim, R = a.taps;
-  T* ring = static_cast<T*>(a.ring) + static_cast<long long>(slot) * R * C + channel;
-  const float* w = a.conv_w + static_cast<long long>(channel) * R;
-  const T x = static_cast<const T*>(src)[row * ld + src_col];
-  float acc = 0.f;
-  for (int j = R - 1; j >= 1; --j)
-    if (pos - j >= 0) acc += w[R - 1 - j] * static_cast<float>(ring[static_cast<long long>((pos - j) % R) * C]);
-  acc += w[R - 1] * static_cast<float>(x);
-  if (writes && R > 1) ring[static_cast<long long>(pos % R) * C] = x;
-  return static_cast<float>(static_cast<T>(silu(acc)));
+// VEC consecutive values of either type as floats (one access; VEC is 1, 2 or 4)
+template <int VEC>
+__device__ __forceinline__ void load_any(const float* p, float* f) {
+  if (VEC == 4) load_vec<VEC>(p, f);
+  else
+    for (int i = 0; i < VEC; ++i) f[i] = p[i];
 }
+template <int VEC>
+__device__ __forceinline__ void load_any(const __nv_bfloat16* p, float* f) {
+  if (VEC == 1) {
+    f[0] = __bfloat162float(p[0]);
+    return;
+  }
+  uint32_t r[2];
+  if (VEC == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    r[0] = v.x;
+    r[1] = v.y;
+  } else {
+    r[0] = r[1] = *reinterpret_cast<const uint32_t*>(p);
+  }
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r[i / 2]));
+    f[i] = i % 2 ? v.y : v.x;
+  }
+}
+template <int VEC>
+__device__ __forceinline__ void store_any(float* p, const float* f) {
+  if (VEC == 4) store_vec<VEC>(p, f);
+  else
+    for (int i = 0; i < VEC; ++i) p[i] = f[i];
+}
+template <int VEC>
+__device__ __forceinline__ void store_any(__nv_bfloat16* p, const float* f) {
+  if (VEC == 1) {
+    p[0] = __float2bfloat16(f[0]);
+    return;
+  }
+  uint32_t r[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(f[VEC == 4 ? 2 * i : 0], f[VEC == 4 ? 2 * i + 1 : VEC - 1]);
+    r[i] = *reinterpret_cast<const uint32_t*>(&v);
+  }
+  if (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(r[0], r[1]);
+  else *reinterpret_cast<uint32_t*>(p) = r[0];
+}
+
+// Convolution + silu of one channel of a one-token segment at position pos, from the raw projection and the ring of earlier
+// inputs (ring[slot][p % taps][channel]). load() requests everything, finish() combines it and, in the one writing thread
+// of a channel, stores the new input. Slot pos % taps is not among the taps - 1 positions that are read, so readers in
+// other CTAs do not race with it.
+template <typename T>
+struct ConvInputs {
+  T x[kMaxTaps];
+  float w[kMaxTaps];
+  __device__ __forceinline__ static T* ring_of(const DmoeRecur& a, int slot, int channel) {
+    const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim;
+    return static_cast<T*>(a.ring) + static_cast<long long>(slot) * a.taps * C + channel;
+  }
+  __device__ __forceinline__ void load(const DmoeRecur& a, long long row, int pos, int slot, int channel, const void* src,
+                                       long long ld, int src_col) {
+    const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim, R = a.taps;
+    const T* ring = ring_of(a, slot, channel);
+    const float* wp = a.conv_w + static_cast<long long>(channel) * R + R - 1;
+    x[0] = static_cast<const T*>(src)[row * ld + src_col];
+    w[0] = wp[0];
+#pragma unroll
+    for (int j = 1; j < kMaxTaps; ++j) {
+      const bool on = j < R && pos - j >= 0;
+      x[j] = on ? ring[static_cast<long long>((pos - j) % R) * C] : static_cast<T>(0.f);
+      w[j] = on ? wp[-j] : 0.f;
+    }
+  }
+  __device__ __forceinline__ float finish(const DmoeRecur& a, int pos, int slot, int channel, bool writes) {
+    float acc = 0.f;
+#pragma unroll
+    for (int j = kMaxTaps - 1; j >= 0; --j) acc += w[j] * static_cast<float>(x[j]);
+    const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim;
+    if (writes && a.taps > 1) ring_of(a, slot, channel)[static_cast<long long>(pos % a.taps) * C] = x[0];
+    return static_cast<float>(static_cast<T>(silu(acc)));
+  }
+};
 
 }  // namespace dmoe

@@ -28,14 +28,37 @@ constexpr float kMaxShift = 60.f;          // log2 units
 constexpr int kMid = 31;
 constexpr int kPs = kChunk + 8;            // row stride (elements) of 64-column bf16 tiles in shared memory
 
-// Workspace of one (chunk, head), in bytes.
+// Workspace of one (chunk, head), in bytes. The left operands of the scan's products (q e^b, (k e^(b_end - b))^T, P, W) are
+// stored as mma.sync A fragments: per 16 x 16 tile and plane (hi, lo) one uint4 per lane, so that a warp fetches a tile
+// with one coalesced 512-byte load straight into registers. Tile order: q, P, W by (row tile, k tile), k by (channel
+// tile, token tile); planes innermost.
 template <int DP>
 struct ChunkWs {
-  static constexpr long long kPlane = 2ll * kChunk * DP;          // one bf16 plane [64][DP]
-  static constexpr long long kQ = 0, kK = 2 * kPlane, kP = 4 * kPlane, kDec = kP + 4ll * kChunk * kChunk;
-  static constexpr long long kW = kDec + 4ll * DP, kU = kW + 2 * kPlane;
+  static constexpr long long kMat = 2ll * 2 * kChunk * DP;        // both planes of a [64][DP] matrix
+  static constexpr long long kQ = 0, kK = kMat, kP = 2 * kMat, kDec = kP + 2ll * 2 * kChunk * kChunk;
+  static constexpr long long kW = kDec + 4ll * DP, kU = kW + kMat;
   static long long bytes(bool delta, int V) { return delta ? kU + 4ll * kChunk * V : kW; }
 };
+constexpr int kFrag = 512;                 // bytes of one fragment tile of one plane
+
+__device__ __forceinline__ void store_frag(uint8_t* tile, int lane, const uint32_t (&f)[4]) {
+  reinterpret_cast<uint4*>(tile)[lane] = make_uint4(f[0], f[1], f[2], f[3]);
+}
+// Issued where it stands (not moved towards its use): the scan prefetches the next chunk's fragments with it.
+__device__ __forceinline__ void load_frag(const uint8_t* tile, int lane, uint32_t (&f)[4]) {
+  asm volatile("ld.global.v4.u32 {%0, %1, %2, %3}, [%4];"
+               : "=r"(f[0]), "=r"(f[1]), "=r"(f[2]), "=r"(f[3]) : "l"(tile + lane * 16));
+}
+// Two neighbouring accumulator tiles (16 x 8 each) as one A fragment, split into planes.
+__device__ __forceinline__ void store_acc_frag(uint8_t* tile, int lane, const float* a, const float* b) {
+  uint32_t h[4], l[4];
+  split2(a[0], a[1], h[0], l[0]);
+  split2(a[2], a[3], h[1], l[1]);
+  split2(b[0], b[1], h[2], l[2]);
+  split2(b[2], b[3], h[3], l[3]);
+  store_frag(tile, lane, h);
+  store_frag(tile + kFrag, lane, l);
+}
 
 template <int N>
 __device__ __forceinline__ void load_bf16(const __nv_bfloat16* p, float* f) {
@@ -116,7 +139,7 @@ struct PrepSmem {
   static constexpr int kKs = DP + 8;
   static constexpr int kKn = 2 * kChunk * kKs * 2, kTX = DELTA ? 4 * kChunk * kPs * 2 : 0;
   static constexpr int kRegion = kKn > kTX ? kKn : kTX;
-  static constexpr int kBytes = 4 * kChunk * DP + 4 * 4 * kChunk + kRegion + (DELTA ? 2 * 4 * kChunk * (kChunk + 1) : 0) + 16;
+  static constexpr int kBytes = 4 * kChunk * DP + 3 * 4 * kChunk + kRegion + (DELTA ? 2 * 4 * kChunk * (kChunk + 1) : 0) + 16;
 };
 
 template <int DP, bool DELTA>
@@ -124,19 +147,17 @@ __global__ void __launch_bounds__(kChunkThreads, 2)
 chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* __restrict__ ws, long long ws_stride, int h0) {
   using L = ChunkWs<DP>;
   using SM = PrepSmem<DP, DELTA>;
-  constexpr int PL = DP / 32, KS = DP / 16, LDA = kChunk + 1;
+  constexpr int PL = DP / 32, KS = DP / 16, MT = DP / 16, LDA = kChunk + 1, ROWS = kChunk / 8;
   extern __shared__ __align__(16) uint8_t s_raw[];
   float* s_b = reinterpret_cast<float*>(s_raw);                 // [64][DP] running log2 decay
-  float* s_fq = s_b + kChunk * DP;                              // [64] factor of the raw q row
+  float* s_fq = s_b + kChunk * DP;                              // [64] factors of the raw q and k rows
   float* s_fk = s_fq + kChunk;
   float* s_beta = s_fk + kChunk;
-  float* s_tot = s_beta + kChunk;                               // [64], unused slack
-  uint8_t* region = reinterpret_cast<uint8_t*>(s_tot + kChunk);
-  __nv_bfloat16* s_kh = reinterpret_cast<__nv_bfloat16*>(region);          // k e^(m - b), hi then lo plane
+  uint8_t* region = reinterpret_cast<uint8_t*>(s_beta + kChunk);
+  __nv_bfloat16* s_kh = reinterpret_cast<__nv_bfloat16*>(region);          // scaled k rows, hi then lo plane
   __nv_bfloat16* s_kl = s_kh + kChunk * SM::kKs;
   float* s_A = reinterpret_cast<float*>(region + SM::kRegion);
   float* s_T = s_A + kChunk * LDA;
-  (void)s_tot;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int lm_mi = lane >> 3, lm_r = lane & 7;
@@ -147,39 +168,76 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + row0 * a.ldq + hk * D;
   const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k) + row0 * a.ldk + hk * D;
   uint8_t* w = ws + (static_cast<long long>(blockIdx.x) * gridDim.y + blockIdx.y) * ws_stride;
-  __nv_bfloat16* w_q = reinterpret_cast<__nv_bfloat16*>(w + L::kQ);
-  __nv_bfloat16* w_k = reinterpret_cast<__nv_bfloat16*>(w + L::kK);
-  __nv_bfloat16* w_p = reinterpret_cast<__nv_bfloat16*>(w + L::kP);
 
-  // ---- log2 decays and their running sums
+  // ---- this warp's rows of k (and q, for its norm); loads first, they are used below
+  const int t0 = warp * ROWS, d0 = lane * PL;
+  float k[ROWS][PL];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+#pragma unroll
+    for (int e = 0; e < PL; ++e) k[i][e] = 0.f;
+    if (t0 + i < n && d0 < D) load_bf16<PL>(kp + (t0 + i) * a.ldk + d0, k[i]);
+  }
+  // ---- log2 decays and their running sums; a thread keeps one channel
   {
+    constexpr int NG = kChunkThreads / DP, LEN = kChunk / NG;
     const float scale = a.decay_kind == 0 ? a.inv_tau : expf(a.a_log[h]);
-    for (int i = tid; i < kChunk * DP; i += kChunkThreads) {
-      const int t = i / DP, d = i % DP;
-      s_b[i] = t < n && d < D
-                   ? kLog2e * log_decay(a.decay_kind, a.z[(row0 + t) * a.ldz + h * D + d] + a.z_bias[h * D + d], scale)
-                   : 0.f;
+    const int d = tid % DP, gi = tid / DP;
+    const float bias = d < D ? a.z_bias[h * D + d] : 0.f;
+    const float* zp = a.z + row0 * a.ldz + h * D + d;
+    float run = 0.f;
+#pragma unroll
+    for (int t8 = 0; t8 < LEN; t8 += 8) {
+      float z[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = gi * LEN + t8 + j;
+        z[j] = t < n && d < D ? zp[t * a.ldz] : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = gi * LEN + t8 + j;
+        if (t < n && d < D) run += kLog2e * log_decay(a.decay_kind, z[j] + bias, scale);
+        s_b[t * DP + d] = run;
+      }
     }
     if (tid < kChunk)
       s_beta[tid] = DELTA && tid < n
                         ? 1.f / (1.f + expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + tid) * a.ldb + h])))
                         : 0.f;
     __syncthreads();
-    constexpr int NG = kChunkThreads / DP, LEN = kChunk / NG;
-    const int d = tid % DP, gi = tid / DP;
-    float run = 0.f;
-#pragma unroll 8
-    for (int t = gi * LEN; t < (gi + 1) * LEN; ++t) {
-      run += s_b[t * DP + d];
-      s_b[t * DP + d] = run;
-    }
-    __syncthreads();
     float before = 0.f;
     for (int j = 0; j < gi; ++j) before += s_b[((j + 1) * LEN - 1) * DP + d];
     __syncthreads();
-    for (int t = gi * LEN; t < (gi + 1) * LEN; ++t) s_b[t * DP + d] += before;
-    __syncthreads();
+    if (gi > 0) {
+#pragma unroll 8
+      for (int t = gi * LEN; t < (gi + 1) * LEN; ++t) s_b[t * DP + d] += before;
+    }
   }
+  // ---- factors of the rows: scale and unit norms
+  if (DELTA) {
+    float q[ROWS][PL];
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+#pragma unroll
+      for (int e = 0; e < PL; ++e) q[i][e] = 0.f;
+      if (t0 + i < n && d0 < D) load_bf16<PL>(qp + (t0 + i) * a.ldq + d0, q[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+      float qq = 0.f, kk = 0.f;
+#pragma unroll
+      for (int e = 0; e < PL; ++e) { qq += q[i][e] * q[i][e]; kk += k[i][e] * k[i][e]; }
+      const float fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f), fq = a.qscale / sqrtf(warp_sum(qq) + 1e-6f);
+      if (lane == 0) { s_fq[t0 + i] = fq; s_fk[t0 + i] = fk; }
+#pragma unroll
+      for (int e = 0; e < PL; ++e) k[i][e] *= fk;
+    }
+  } else if (lane < ROWS) {
+    s_fq[t0 + lane] = a.qscale;
+    s_fk[t0 + lane] = 1.f;
+  }
+  __syncthreads();
   bool wide = false;
   if (tid < DP) {
     const float m = s_b[kMid * DP + tid];
@@ -188,45 +246,36 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   }
   const bool slow = __syncthreads_or(wide);
 
-  // ---- rows: unit norms, k e^(m - b) to shared memory, q e^b and k e^(b_end - b) to the workspace
-  for (int t = warp; t < kChunk; t += kChunkThreads / 32) {
-    const int d0 = lane * PL;
-    float q[PL], k[PL];
+  // ---- k e^(b_end - b): through shared memory into transposed fragments
+  auto stage_k = [&](int ref) {                      // k e^(b_ref - b)
 #pragma unroll
-    for (int e = 0; e < PL; ++e) q[e] = k[e] = 0.f;
-    if (t < n && d0 < D) {
-      load_bf16<PL>(qp + t * a.ldq + d0, q);
-      load_bf16<PL>(kp + t * a.ldk + d0, k);
-    }
-    float fq = a.qscale, fk = 1.f;
-    if (DELTA) {
-      float qq = 0.f, kk = 0.f;
+    for (int i = 0; i < ROWS; ++i) {
+      float x[PL];
 #pragma unroll
-      for (int e = 0; e < PL; ++e) { qq += q[e] * q[e]; kk += k[e] * k[e]; }
-      fq *= 1.f / sqrtf(warp_sum(qq) + 1e-6f);
-      fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+      for (int e = 0; e < PL; ++e) x[e] = k[i][e] * exp2f(s_b[ref * DP + d0 + e] - s_b[(t0 + i) * DP + d0 + e]);
+      store_split<PL>(s_kh + (t0 + i) * SM::kKs + d0, s_kl + (t0 + i) * SM::kKs + d0, x);
     }
-    if (lane == 0) { s_fq[t] = fq; s_fk[t] = fk; }
-    float x[PL], y[PL], z[PL];
-#pragma unroll
-    for (int e = 0; e < PL; ++e) {
-      const float b = s_b[t * DP + d0 + e];
-      const float kv = k[e] * fk;
-      x[e] = kv * exp2f(s_b[kMid * DP + d0 + e] - b);
-      y[e] = kv * exp2f(s_b[(kChunk - 1) * DP + d0 + e] - b);
-      z[e] = q[e] * fq * exp2f(b);
-    }
-    if (!slow) store_split<PL>(s_kh + t * SM::kKs + d0, s_kl + t * SM::kKs + d0, x);
-    store_split<PL>(w_k + t * DP + d0, w_k + kChunk * DP + t * DP + d0, y);
-    store_split<PL>(w_q + t * DP + d0, w_q + kChunk * DP + t * DP + d0, z);
+  };
+  stage_k(kChunk - 1);
+  __syncthreads();
+  for (int i = warp; i < MT * 4; i += kChunkThreads / 32) {
+    const int mt = i / 4, ks = i % 4;
+    const uint32_t off = ((ks * 16 + (lm_mi >> 1) * 8 + lm_r) * SM::kKs + mt * 16 + (lm_mi & 1) * 8) * 2;
+    uint32_t f[4];
+    ldmatrix_x4_trans(smem_u32(s_kh) + off, f[0], f[1], f[2], f[3]);
+    store_frag(w + L::kK + i * 2 * kFrag, lane, f);
+    ldmatrix_x4_trans(smem_u32(s_kl) + off, f[0], f[1], f[2], f[3]);
+    store_frag(w + L::kK + (i * 2 + 1) * kFrag, lane, f);
   }
   __syncthreads();
+  if (!slow) stage_k(kMid);                     // now k e^(m - b): right operand of P and A
+  __syncthreads();
 
-  // ---- P (warps 0-3) and A (warps 4-7)
-  if (!slow) {
+  // ---- P and the fragments of q e^b (warps 0-3), A (warps 4-7)
+  {
     const int mi = warp & 3;
     const bool second = warp >= 4;
-    if (DELTA || !second) {
+    if (!second || (DELTA && !slow)) {
       const int r0 = mi * 16 + g, r1 = r0 + 8;
       const __nv_bfloat16* src = second ? kp : qp;
       const long long ld = second ? a.ldk : a.ldq;
@@ -236,47 +285,73 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
       for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
       const uint32_t bh = smem_u32(s_kh), bl = smem_u32(s_kl);
 #pragma unroll
-      for (int ks = 0; ks < KS; ++ks) {
-        uint32_t ah[4], al[4];
+      for (int kb = 0; kb < KS; kb += 4) {           // raw values of up to four k tiles in flight
+        uint32_t raw[4][4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int r = j & 1 ? r1 : r0, c = ks * 16 + 2 * tq + (j >> 1) * 8;
-          float x[2] = {0.f, 0.f};
-          if (r < n && c < D) load_bf16<2>(src + r * ld + c, x);
-          const float f = j & 1 ? f1 : f0;
-          const float2 b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
-          const float2 m = *reinterpret_cast<const float2*>(s_b + kMid * DP + c);
-          split2(x[0] * f * exp2f(b.x - m.x), x[1] * f * exp2f(b.y - m.y), ah[j], al[j]);
-        }
+        for (int kk = 0; kk < 4 && kb + kk < KS; ++kk)
 #pragma unroll
-        for (int kg = 0; kg < 4; ++kg) {
-          if (kg <= mi) {
-            const uint32_t off = ((kg * 16 + (lm_mi >> 1) * 8 + lm_r) * SM::kKs + ks * 16 + (lm_mi & 1) * 8) * 2;
-            uint32_t h0_, h1_, h2_, h3_, l0_, l1_, l2_, l3_;
-            ldmatrix_x4(bh + off, h0_, h1_, h2_, h3_);
-            ldmatrix_x4(bl + off, l0_, l1_, l2_, l3_);
-            mma_split(acc[2 * kg], ah, al, h0_, h1_, l0_, l1_);
-            mma_split(acc[2 * kg + 1], ah, al, h2_, h3_, l2_, l3_);
+          for (int j = 0; j < 4; ++j) {
+            const int r = j & 1 ? r1 : r0, c = (kb + kk) * 16 + 2 * tq + (j >> 1) * 8;
+            raw[kk][j] = r < n && c < D ? *reinterpret_cast<const uint32_t*>(src + r * ld + c) : 0u;
+          }
+#pragma unroll
+        for (int kk = 0; kk < 4 && kb + kk < KS; ++kk) {
+          const int ks = kb + kk;
+          uint32_t ah[4], al[4], zh[4], zl[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int r = j & 1 ? r1 : r0, c = ks * 16 + 2 * tq + (j >> 1) * 8;
+            const float f = j & 1 ? f1 : f0;
+            float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[kk][j]));
+            x.x *= f;
+            x.y *= f;
+            const float2 b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
+            const float2 m = *reinterpret_cast<const float2*>(s_b + kMid * DP + c);
+            split2(x.x * exp2f(b.x - m.x), x.y * exp2f(b.y - m.y), ah[j], al[j]);
+            if (!second) split2(x.x * exp2f(b.x), x.y * exp2f(b.y), zh[j], zl[j]);
+          }
+          if (!second) {
+            store_frag(w + L::kQ + (mi * KS + ks) * 2 * kFrag, lane, zh);
+            store_frag(w + L::kQ + ((mi * KS + ks) * 2 + 1) * kFrag, lane, zl);
+          }
+          if (slow) continue;
+#pragma unroll
+          for (int kg = 0; kg < 4; ++kg) {
+            if (kg <= mi) {
+              const uint32_t off = ((kg * 16 + (lm_mi >> 1) * 8 + lm_r) * SM::kKs + ks * 16 + (lm_mi & 1) * 8) * 2;
+              uint32_t h0_, h1_, h2_, h3_, l0_, l1_, l2_, l3_;
+              ldmatrix_x4(bh + off, h0_, h1_, h2_, h3_);
+              ldmatrix_x4(bl + off, l0_, l1_, l2_, l3_);
+              mma_split(acc[2 * kg], ah, al, h0_, h1_, l0_, l1_);
+              mma_split(acc[2 * kg + 1], ah, al, h2_, h3_, l2_, l3_);
+            }
           }
         }
       }
+      if (!slow) {
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const int c = nt * 8 + 2 * tq;
+        for (int nt = 0; nt < 8; ++nt) {
+          const int c = nt * 8 + 2 * tq, edge = second ? -1 : 0;        // A is strictly below the diagonal
+          if (c > r0 + edge) acc[nt][0] = 0.f;
+          if (c + 1 > r0 + edge) acc[nt][1] = 0.f;
+          if (c > r1 + edge) acc[nt][2] = 0.f;
+          if (c + 1 > r1 + edge) acc[nt][3] = 0.f;
+          if (DELTA && second) {
+            s_A[r0 * LDA + c] = acc[nt][0] * s_beta[r0];
+            s_A[r0 * LDA + c + 1] = acc[nt][1] * s_beta[r0];
+            s_A[r1 * LDA + c] = acc[nt][2] * s_beta[r1];
+            s_A[r1 * LDA + c + 1] = acc[nt][3] * s_beta[r1];
+          }
+        }
         if (!second) {
-          const float v[4] = {c <= r0 ? acc[nt][0] : 0.f, c + 1 <= r0 ? acc[nt][1] : 0.f, c <= r1 ? acc[nt][2] : 0.f,
-                              c + 1 <= r1 ? acc[nt][3] : 0.f};
-          store_split<2>(w_p + r0 * kChunk + c, w_p + kChunk * kChunk + r0 * kChunk + c, v);
-          store_split<2>(w_p + r1 * kChunk + c, w_p + kChunk * kChunk + r1 * kChunk + c, v + 2);
-        } else if (DELTA) {
-          s_A[r0 * LDA + c] = c < r0 ? acc[nt][0] * s_beta[r0] : 0.f;
-          s_A[r0 * LDA + c + 1] = c + 1 < r0 ? acc[nt][1] * s_beta[r0] : 0.f;
-          s_A[r1 * LDA + c] = c < r1 ? acc[nt][2] * s_beta[r1] : 0.f;
-          s_A[r1 * LDA + c + 1] = c + 1 < r1 ? acc[nt][3] * s_beta[r1] : 0.f;
+#pragma unroll
+          for (int kg = 0; kg < 4; ++kg)
+            store_acc_frag(w + L::kP + (mi * 4 + kg) * 2 * kFrag, lane, acc[2 * kg], acc[2 * kg + 1]);
         }
       }
     }
-  } else {
+  }
+  if (slow) {
     for (int i = tid; i < kChunk * kChunk; i += kChunkThreads) {
       const int t = i / kChunk, j = i % kChunk;
       float p = 0.f, kk = 0.f;
@@ -287,8 +362,12 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
           if (DELTA) kk += __bfloat162float(kp[t * a.ldk + d]) * e;
         }
       }
+      // place of element (t, j) in the fragment tiles
       const float pv = p * s_fq[t];
-      store_split<1>(w_p + i, w_p + kChunk * kChunk + i, &pv);
+      const int r = t % 16, c = j % 16;
+      __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(w + L::kP + (t / 16 * 4 + j / 16) * 2 * kFrag) +
+                         ((r % 8) * 4 + c % 8 / 2) * 8 + ((r >= 8) + 2 * (c >= 8)) * 2 + c % 2;
+      store_split<1>(e, e + kFrag / 2, &pv);
       if (DELTA) s_A[t * LDA + j] = j < t ? kk * s_fk[t] * s_beta[t] : 0.f;
     }
   }
@@ -300,31 +379,44 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   __nv_bfloat16* s_tl = s_th + kChunk * kPs;
   __nv_bfloat16* s_xh = s_tl + kChunk * kPs;
   __nv_bfloat16* s_xl = s_xh + kChunk * kPs;
+  const int nd = (DP + 63) / 64, nv = (V + 63) / 64;
+  const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.v) + row0 * a.ldv + h * V;
+  float* w_u = reinterpret_cast<float*>(w + L::kU);
+  const int mi = warp & 3, nh = warp >> 2;
+  uint32_t raw[8];                                   // the next 64-column tile of k or v: rows tid / 32 + 8 i
+  auto fetch = [&](int x) {
+    const bool keys = x < nd;
+    const int cc = (keys ? x : x - nd) * 64 + tid % 32 * 2;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int t = tid / 32 + 8 * i;
+      raw[i] = t < n && cc < (keys ? D : V)
+                   ? *reinterpret_cast<const uint32_t*>(keys ? kp + t * a.ldk + cc : vp + t * a.ldv + cc) : 0u;
+    }
+  };
+  fetch(0);
   invert_unit_lower(s_A, s_T, reinterpret_cast<float*>(s_xh));
   for (int i = tid; i < kChunk * kChunk / 2; i += kChunkThreads) {
     const int t = i / (kChunk / 2), c = i % (kChunk / 2) * 2;
     const float v[2] = {s_T[t * LDA + c], s_T[t * LDA + c + 1]};
     store_split<2>(s_th + t * kPs + c, s_tl + t * kPs + c, v);
   }
-  const int nd = (DP + 63) / 64, nv = (V + 63) / 64;
-  const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.v) + row0 * a.ldv + h * V;
-  __nv_bfloat16* w_w = reinterpret_cast<__nv_bfloat16*>(w + L::kW);
-  float* w_u = reinterpret_cast<float*>(w + L::kU);
-  const int mi = warp & 3, nh = warp >> 2;
   for (int x = 0; x < nd + nv; ++x) {
     const bool keys = x < nd;
     const int c0 = (keys ? x : x - nd) * 64;
-    for (int i = tid; i < kChunk * 32; i += kChunkThreads) {
-      const int t = i / 32, c = i % 32 * 2, cc = c0 + c;
-      float v[2] = {0.f, 0.f};
-      if (t < n && cc < (keys ? D : V)) {
-        load_bf16<2>(keys ? kp + t * a.ldk + cc : vp + t * a.ldv + cc, v);
-        const float f = keys ? -s_beta[t] * s_fk[t] : s_beta[t];
-        v[0] *= f * (keys ? exp2f(s_b[t * DP + cc]) : 1.f);
-        v[1] *= f * (keys ? exp2f(s_b[t * DP + cc + 1]) : 1.f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int t = tid / 32 + 8 * i, c = tid % 32 * 2, cc = c0 + c;
+      const float2 r = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[i]));
+      float v[2] = {r.x * s_beta[t], r.y * s_beta[t]};
+      if (keys) {
+        const float f = -s_fk[t];
+        v[0] *= cc < DP ? f * exp2f(s_b[t * DP + cc]) : 0.f;
+        v[1] *= cc < DP ? f * exp2f(s_b[t * DP + cc + 1]) : 0.f;
       }
       store_split<2>(s_xh + t * kPs + c, s_xl + t * kPs + c, v);
     }
+    if (x + 1 < nd + nv) fetch(x + 1);
     __syncthreads();
     float acc[4][4];
 #pragma unroll
@@ -347,48 +439,39 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
         }
       }
     }
+    if (keys) {
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
-      const int c = c0 + nh * 32 + nt * 8 + 2 * tq, r0 = mi * 16 + g, r1 = r0 + 8;
-      if (keys) {
-        if (c < DP) {
-          store_split<2>(w_w + r0 * DP + c, w_w + kChunk * DP + r0 * DP + c, acc[nt]);
-          store_split<2>(w_w + r1 * DP + c, w_w + kChunk * DP + r1 * DP + c, acc[nt] + 2);
+      for (int p = 0; p < 2; ++p) {
+        const int ks = (c0 + nh * 32) / 16 + p;      // k tile of W
+        if (ks < KS) store_acc_frag(w + L::kW + (mi * KS + ks) * 2 * kFrag, lane, acc[2 * p], acc[2 * p + 1]);
+      }
+    } else {
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) {
+        const int c = c0 + nh * 32 + nt * 8 + 2 * tq, r0 = mi * 16 + g, r1 = r0 + 8;
+        if (c < V) {
+          *reinterpret_cast<float2*>(w_u + r0 * V + c) = make_float2(acc[nt][0], acc[nt][1]);
+          *reinterpret_cast<float2*>(w_u + r1 * V + c) = make_float2(acc[nt][2], acc[nt][3]);
         }
-      } else if (c < V) {
-        *reinterpret_cast<float2*>(w_u + r0 * V + c) = make_float2(acc[nt][0], acc[nt][1]);
-        *reinterpret_cast<float2*>(w_u + r1 * V + c) = make_float2(acc[nt][2], acc[nt][3]);
       }
     }
     __syncthreads();
   }
 }
 
-template <int DP, int VT, bool DELTA>
-struct ScanSmem {
-  static constexpr int kKs = DP + 8, kVs = VT + 8;
-  static constexpr int kRows = kChunk * kKs * 2, kPb = kChunk * kPs * 2, kS = DP * kVs * 2, kUb = kChunk * kVs * 2;
-  static constexpr int kBytes = (DELTA ? 6 : 4) * kRows + 2 * kPb + 2 * kS + 2 * kUb;
-};
-
 // Chunks of one segment in order. Warps 4-7 own 16 rows each of the read-outs, warps 0-3 of u (delta), warps 0 .. DP / 16
-// - 1 sixteen key channels each of the state. The tiles of the next chunk are fetched while the current one computes:
-// q e^b and W during the state update, k e^(b_end - b) and P (and v) during the products with the old state.
+// - 1 sixteen key channels each of the state. Left operands come straight from the workspace into registers, fetched half a
+// chunk ahead: q e^b and W while the state is updated, (k e^(b_end - b))^T and P while the old state is multiplied. Only
+// the state and u, the right operands that every warp shares, go through shared memory.
 template <int DP, int VT, bool DELTA>
-__global__ void __launch_bounds__(kChunkThreads)
+__global__ void __launch_bounds__(kChunkThreads, 1)
 chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long ws_stride, int h0, int n_heads) {
   using L = ChunkWs<DP>;
-  using SM = ScanSmem<DP, VT, DELTA>;
-  constexpr int NT = VT / 8, KS = DP / 16, MT = DP / 16;
-  extern __shared__ __align__(16) uint8_t s_raw[];
-  const uint32_t s_q = smem_u32(s_raw);                          // planes hi, lo
-  const uint32_t s_k = s_q + 2 * SM::kRows;
-  const uint32_t s_w = s_k + 2 * SM::kRows;
-  const uint32_t s_p = s_w + (DELTA ? 2 : 0) * SM::kRows;
-  const uint32_t s_s = s_p + 2 * SM::kPb;
-  const uint32_t s_u = s_s + 2 * SM::kS;
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_raw + (s_s - s_q));
-  __nv_bfloat16* p_u = reinterpret_cast<__nv_bfloat16*>(s_raw + (s_u - s_q));
+  constexpr int NT = VT / 8, KS = DP / 16, MT = DP / 16, VS = VT + 8;
+  __shared__ __align__(16) __nv_bfloat16 p_s[2][DP * VS];        // state, planes hi / lo
+  __shared__ __align__(16) __nv_bfloat16 p_u[DELTA ? 2 : 1][kChunk * VS];
+  const uint32_t s_s = smem_u32(p_s), s_u = smem_u32(p_u);
+  constexpr uint32_t kSPlane = DP * VS * 2, kUPlane = kChunk * VS * 2;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int lm_mi = lane >> 3, lm_r = lane & 7;
@@ -402,148 +485,182 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
   for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
   const int nc = (seg.y + kChunk - 1) / kChunk;
   const int hl = blockIdx.y, h = h0 + hl, D = a.dim, V = a.vdim, v0 = blockIdx.z * VT;
+  const int mi = warp & 3, r0 = mi * 16 + g, r1 = r0 + 8;
+  const bool reads = warp >= 4, updates = warp < MT;
+  const int d0 = warp * 16 + g, d1 = d0 + 8;
 
   auto base = [&](int c) { return ws + (static_cast<long long>(before + c) * n_heads + hl) * ws_stride; };
-  auto copy_rows = [&](uint32_t dst, const uint8_t* src) {       // two planes [64][DP]
-    for (int i = tid; i < 2 * kChunk * (DP / 8); i += kChunkThreads) {
-      const int r = i / (DP / 8), c = i % (DP / 8);
-      cp_async16(dst + r * (SM::kKs * 2) + c * 16, src + i * 16, true);
+  uint32_t fa[KS][2][4];                                         // q e^b (warps 4-7) or W (warps 0-3)
+  uint32_t fk[4][2][4], fp[4][2][4];
+  float u0[NT][4], dec0 = 0.f, dec1 = 0.f;
+  uint4 vnext = make_uint4(0u, 0u, 0u, 0u);                      // plain write: this thread's 8 values of the next v tile
+  auto fetch_a = [&](int c) {
+    if (reads || DELTA) {
+      const uint8_t* p = base(c) + (reads ? L::kQ : L::kW) + mi * KS * 2 * kFrag;
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) {
+        load_frag(p + ks * 2 * kFrag, lane, fa[ks][0]);
+        load_frag(p + (ks * 2 + 1) * kFrag, lane, fa[ks][1]);
+      }
     }
-  };
-  auto load_a = [&](int c) {
-    copy_rows(s_q, base(c) + L::kQ);
-    if (DELTA) copy_rows(s_w, base(c) + L::kW);
-  };
-  auto load_b = [&](int c) {
-    copy_rows(s_k, base(c) + L::kK);
-    const uint8_t* src = base(c) + L::kP;
-    for (int i = tid; i < 2 * kChunk * 8; i += kChunkThreads)
-      cp_async16(s_p + i / 8 * (kPs * 2) + i % 8 * 16, src + i * 16, true);
-    if (!DELTA) {                                                // u = v
-      const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.v);
-      for (int i = tid; i < kChunk * NT; i += kChunkThreads) {
-        const int t = i / NT, cc = v0 + i % NT * 8;
-        const bool ok = c * kChunk + t < seg.y && cc < V;
-        const long long off = ok ? static_cast<long long>(seg.x + c * kChunk + t) * a.ldv + h * V + cc : 0;
-        cp_async16(s_u + t * (SM::kVs * 2) + i % NT * 16, vp + off, ok);
+    if (DELTA && !reads) {
+      const float* up = reinterpret_cast<const float*>(base(c) + L::kU);
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const int cc = v0 + nt * 8 + 2 * tq;
+        float2 x = make_float2(0.f, 0.f), y = x;
+        if (cc < V) {
+          x = *reinterpret_cast<const float2*>(up + r0 * V + cc);
+          y = *reinterpret_cast<const float2*>(up + r1 * V + cc);
+        }
+        u0[nt][0] = x.x; u0[nt][1] = x.y; u0[nt][2] = y.x; u0[nt][3] = y.y;
       }
     }
   };
-  load_a(0);
-  cp_async_commit();
-  load_b(0);
-  cp_async_commit();
+  auto fetch_b = [&](int c) {
+    if (updates) {
+      const uint8_t* p = base(c) + L::kK + warp * 4 * 2 * kFrag;
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        load_frag(p + ks * 2 * kFrag, lane, fk[ks][0]);
+        load_frag(p + (ks * 2 + 1) * kFrag, lane, fk[ks][1]);
+      }
+      const float* dp = reinterpret_cast<const float*>(base(c) + L::kDec);
+      dec0 = dp[d0];
+      dec1 = dp[d1];
+    }
+    if (reads) {
+      const uint8_t* p = base(c) + L::kP + mi * 4 * 2 * kFrag;
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        if (ks <= mi) {
+          load_frag(p + ks * 2 * kFrag, lane, fp[ks][0]);
+          load_frag(p + (ks * 2 + 1) * kFrag, lane, fp[ks][1]);
+        }
+      }
+    }
+  };
+  auto fetch_v = [&](int c) {
+    if (!DELTA && tid < kChunk * NT) {
+      const int t = tid / NT, cc = v0 + tid % NT * 8;
+      vnext = make_uint4(0u, 0u, 0u, 0u);
+      if (c * kChunk + t < seg.y && cc < V)
+        vnext = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) +
+                                                static_cast<long long>(seg.x + c * kChunk + t) * a.ldv + h * V + cc);
+    }
+  };
+  fetch_a(0);
+  fetch_b(0);
+  fetch_v(0);
 
   // the state tile: rows d = warp * 16 + g (+ 8), columns v0 + nt * 8 + 2 tq (+ 1)
   float* sp = a.state + (static_cast<long long>(slot) * a.heads + h) * D * V;
-  const int d0 = warp * 16 + g, d1 = d0 + 8;
   float sacc[NT][4];
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt) {
     sacc[nt][0] = sacc[nt][1] = sacc[nt][2] = sacc[nt][3] = 0.f;
     const int cc = v0 + nt * 8 + 2 * tq;
-    if (warp < MT && seg.w > 0 && cc < V) {
+    if (updates && seg.w > 0 && cc < V) {
       if (d0 < D) { const float2 x = *reinterpret_cast<const float2*>(sp + d0 * V + cc); sacc[nt][0] = x.x; sacc[nt][1] = x.y; }
       if (d1 < D) { const float2 x = *reinterpret_cast<const float2*>(sp + d1 * V + cc); sacc[nt][2] = x.x; sacc[nt][3] = x.y; }
     }
   }
   auto publish = [&] {                                           // state -> hi / lo planes in shared memory
-    if (warp < MT) {
+    if (updates) {
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
-        const int o0 = d0 * SM::kVs + nt * 8 + 2 * tq, o1 = d1 * SM::kVs + nt * 8 + 2 * tq;
-        store_split<2>(p_s + o0, p_s + DP * SM::kVs + o0, sacc[nt]);
-        store_split<2>(p_s + o1, p_s + DP * SM::kVs + o1, sacc[nt] + 2);
+        const int o0 = d0 * VS + nt * 8 + 2 * tq, o1 = d1 * VS + nt * 8 + 2 * tq;
+        store_split<2>(p_s[0] + o0, p_s[1] + o0, sacc[nt]);
+        store_split<2>(p_s[0] + o1, p_s[1] + o1, sacc[nt] + 2);
       }
     }
   };
   publish();
-  cp_async_wait<1>();
   __syncthreads();
 
-  const int mi = warp & 3, r0 = mi * 16 + g, r1 = r0 + 8;
   for (int c = 0; c < nc; ++c) {
-    float dec0 = 0.f, dec1 = 0.f;
-    if (warp < MT) {
-      const float* dp = reinterpret_cast<const float*>(base(c) + L::kDec);
-      dec0 = dp[d0];
-      dec1 = dp[d1];
+    if (!DELTA && tid < kChunk * NT) {                           // u = v
+      *reinterpret_cast<uint4*>(p_u[0] + tid / NT * VS + tid % NT * 8) = vnext;
+      if (c + 1 < nc) fetch_v(c + 1);
     }
-    // products with the old state
-    float acc[NT][4];
+    // products with the old state; hi hi and the cross terms in separate accumulators (shorter dependency chains)
+    float acc[NT][4], cross[NT][4];
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
-    if (DELTA && warp < 4) {
-      const float* up = reinterpret_cast<const float*>(base(c) + L::kU);
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        const int cc = v0 + nt * 8 + 2 * tq;
-        if (cc < V) {
-          const float2 x = *reinterpret_cast<const float2*>(up + r0 * V + cc), y = *reinterpret_cast<const float2*>(up + r1 * V + cc);
-          acc[nt][0] = x.x; acc[nt][1] = x.y; acc[nt][2] = y.x; acc[nt][3] = y.y;
-        }
+      for (int e = 0; e < 4; ++e) {
+        acc[nt][e] = DELTA && !reads ? u0[nt][e] : 0.f;
+        cross[nt][e] = 0.f;
       }
-    }
-    if (DELTA || warp >= 4) {
-      const uint32_t src = warp >= 4 ? s_q : s_w;
+    if (DELTA || reads) {
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks) {
-        const uint32_t ao = ((mi * 16 + (lm_mi & 1) * 8 + lm_r) * SM::kKs + ks * 16 + (lm_mi >> 1) * 8) * 2;
-        uint32_t ah[4], al[4];
-        ldmatrix_x4(src + ao, ah[0], ah[1], ah[2], ah[3]);
-        ldmatrix_x4(src + SM::kRows + ao, al[0], al[1], al[2], al[3]);
 #pragma unroll
         for (int p = 0; p < NT / 2; ++p) {
-          const uint32_t bo = ((ks * 16 + (lm_mi & 1) * 8 + lm_r) * SM::kVs + p * 16 + (lm_mi >> 1) * 8) * 2;
+          const uint32_t bo = ((ks * 16 + (lm_mi & 1) * 8 + lm_r) * VS + p * 16 + (lm_mi >> 1) * 8) * 2;
           uint32_t h0_, h1_, h2_, h3_, l0_, l1_, l2_, l3_;
           ldmatrix_x4_trans(s_s + bo, h0_, h1_, h2_, h3_);
-          ldmatrix_x4_trans(s_s + SM::kS + bo, l0_, l1_, l2_, l3_);
-          mma_split(acc[2 * p], ah, al, h0_, h1_, l0_, l1_);
-          mma_split(acc[2 * p + 1], ah, al, h2_, h3_, l2_, l3_);
+          ldmatrix_x4_trans(s_s + kSPlane + bo, l0_, l1_, l2_, l3_);
+          mma_bf16_16816(acc[2 * p], fa[ks][0], h0_, h1_);
+          mma_bf16_16816(acc[2 * p + 1], fa[ks][0], h2_, h3_);
+          mma_bf16_16816(cross[2 * p], fa[ks][0], l0_, l1_);
+          mma_bf16_16816(cross[2 * p + 1], fa[ks][0], l2_, l3_);
+          mma_bf16_16816(cross[2 * p], fa[ks][1], h0_, h1_);
+          mma_bf16_16816(cross[2 * p + 1], fa[ks][1], h2_, h3_);
         }
       }
     }
-    if (DELTA && warp < 4) {
+    if (c + 1 < nc) fetch_a(c + 1);
+    if (DELTA && !reads) {
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
-        const int o0 = r0 * SM::kVs + nt * 8 + 2 * tq, o1 = r1 * SM::kVs + nt * 8 + 2 * tq;
-        store_split<2>(p_u + o0, p_u + kChunk * SM::kVs + o0, acc[nt]);
-        store_split<2>(p_u + o1, p_u + kChunk * SM::kVs + o1, acc[nt] + 2);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[nt][e] += cross[nt][e];
+        const int o0 = r0 * VS + nt * 8 + 2 * tq, o1 = r1 * VS + nt * 8 + 2 * tq;
+        store_split<2>(p_u[0] + o0, p_u[DELTA ? 1 : 0] + o0, acc[nt]);
+        store_split<2>(p_u[0] + o1, p_u[DELTA ? 1 : 0] + o1, acc[nt] + 2);
       }
     }
-    cp_async_wait<0>();
     __syncthreads();
-    if (c + 1 < nc) load_a(c + 1);
-    cp_async_commit();
 
-    // read-outs: + P u
-    if (warp >= 4) {
+    // state: decay, then + (k e^(b_end - b))^T u; read-outs: + P u
+    if (updates) {
 #pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
-        if (ks <= mi) {
-          const uint32_t ao = ((mi * 16 + (lm_mi & 1) * 8 + lm_r) * kPs + ks * 16 + (lm_mi >> 1) * 8) * 2;
-          uint32_t ah[4], al[4];
-          ldmatrix_x4(s_p + ao, ah[0], ah[1], ah[2], ah[3]);
-          ldmatrix_x4(s_p + SM::kPb + ao, al[0], al[1], al[2], al[3]);
+      for (int nt = 0; nt < NT; ++nt) { sacc[nt][0] *= dec0; sacc[nt][1] *= dec0; sacc[nt][2] *= dec1; sacc[nt][3] *= dec1; }
+    }
 #pragma unroll
-          for (int p = 0; p < NT / 2; ++p) {
-            const uint32_t bo = ((ks * 16 + (lm_mi & 1) * 8 + lm_r) * SM::kVs + p * 16 + (lm_mi >> 1) * 8) * 2;
-            uint32_t h0_, h1_, h2_, h3_;
-            ldmatrix_x4_trans(s_u + bo, h0_, h1_, h2_, h3_);
-            if (DELTA) {
-              uint32_t l0_, l1_, l2_, l3_;
-              ldmatrix_x4_trans(s_u + SM::kUb + bo, l0_, l1_, l2_, l3_);
-              mma_split(acc[2 * p], ah, al, h0_, h1_, l0_, l1_);
-              mma_split(acc[2 * p + 1], ah, al, h2_, h3_, l2_, l3_);
-            } else {                                             // v is exact in bf16
-              mma_bf16_16816(acc[2 * p], ah, h0_, h1_);
-              mma_bf16_16816(acc[2 * p], al, h0_, h1_);
-              mma_bf16_16816(acc[2 * p + 1], ah, h2_, h3_);
-              mma_bf16_16816(acc[2 * p + 1], al, h2_, h3_);
-            }
+    for (int ks = 0; ks < 4; ++ks) {
+#pragma unroll
+      for (int p = 0; p < NT / 2; ++p) {
+        const uint32_t bo = ((ks * 16 + (lm_mi & 1) * 8 + lm_r) * VS + p * 16 + (lm_mi >> 1) * 8) * 2;
+        uint32_t h0_, h1_, h2_, h3_, l0_ = 0u, l1_ = 0u, l2_ = 0u, l3_ = 0u;
+        ldmatrix_x4_trans(s_u + bo, h0_, h1_, h2_, h3_);
+        if (DELTA) ldmatrix_x4_trans(s_u + kUPlane + bo, l0_, l1_, l2_, l3_);   // (v is exact in bf16)
+        if (updates) {
+          mma_bf16_16816(sacc[2 * p], fk[ks][0], h0_, h1_);
+          mma_bf16_16816(sacc[2 * p + 1], fk[ks][0], h2_, h3_);
+          mma_bf16_16816(sacc[2 * p], fk[ks][1], h0_, h1_);
+          mma_bf16_16816(sacc[2 * p + 1], fk[ks][1], h2_, h3_);
+          if (DELTA) {
+            mma_bf16_16816(sacc[2 * p], fk[ks][0], l0_, l1_);
+            mma_bf16_16816(sacc[2 * p + 1], fk[ks][0], l2_, l3_);
+          }
+        }
+        if (reads && ks <= mi) {
+          mma_bf16_16816(acc[2 * p], fp[ks][0], h0_, h1_);
+          mma_bf16_16816(acc[2 * p + 1], fp[ks][0], h2_, h3_);
+          mma_bf16_16816(cross[2 * p], fp[ks][1], h0_, h1_);
+          mma_bf16_16816(cross[2 * p + 1], fp[ks][1], h2_, h3_);
+          if (DELTA) {
+            mma_bf16_16816(cross[2 * p], fp[ks][0], l0_, l1_);
+            mma_bf16_16816(cross[2 * p + 1], fp[ks][0], l2_, l3_);
           }
         }
       }
+    }
+    if (c + 1 < nc) fetch_b(c + 1);
+    publish();
+    if (reads) {
       const int t0 = c * kChunk + r0, t1 = c * kChunk + r1;
       float* o0 = a.raw + static_cast<long long>(seg.x + t0) * a.ldraw + h * V;
       float* o1 = a.raw + static_cast<long long>(seg.x + t1) * a.ldraw + h * V;
@@ -551,47 +668,14 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
       for (int nt = 0; nt < NT; ++nt) {
         const int cc = v0 + nt * 8 + 2 * tq;
         if (cc < V) {
-          if (t0 < seg.y) *reinterpret_cast<float2*>(o0 + cc) = make_float2(acc[nt][0], acc[nt][1]);
-          if (t1 < seg.y) *reinterpret_cast<float2*>(o1 + cc) = make_float2(acc[nt][2], acc[nt][3]);
+          if (t0 < seg.y) *reinterpret_cast<float2*>(o0 + cc) = make_float2(acc[nt][0] + cross[nt][0], acc[nt][1] + cross[nt][1]);
+          if (t1 < seg.y) *reinterpret_cast<float2*>(o1 + cc) = make_float2(acc[nt][2] + cross[nt][2], acc[nt][3] + cross[nt][3]);
         }
       }
     }
-    // state: decay, then + (k e^(b_end - b))^T u
-    if (warp < MT) {
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt) { sacc[nt][0] *= dec0; sacc[nt][1] *= dec0; sacc[nt][2] *= dec1; sacc[nt][3] *= dec1; }
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
-        const uint32_t ao = ((ks * 16 + (lm_mi >> 1) * 8 + lm_r) * SM::kKs + warp * 16 + (lm_mi & 1) * 8) * 2;
-        uint32_t ah[4], al[4];
-        ldmatrix_x4_trans(s_k + ao, ah[0], ah[1], ah[2], ah[3]);
-        ldmatrix_x4_trans(s_k + SM::kRows + ao, al[0], al[1], al[2], al[3]);
-#pragma unroll
-        for (int p = 0; p < NT / 2; ++p) {
-          const uint32_t bo = ((ks * 16 + (lm_mi & 1) * 8 + lm_r) * SM::kVs + p * 16 + (lm_mi >> 1) * 8) * 2;
-          uint32_t h0_, h1_, h2_, h3_;
-          ldmatrix_x4_trans(s_u + bo, h0_, h1_, h2_, h3_);
-          if (DELTA) {
-            uint32_t l0_, l1_, l2_, l3_;
-            ldmatrix_x4_trans(s_u + SM::kUb + bo, l0_, l1_, l2_, l3_);
-            mma_split(sacc[2 * p], ah, al, h0_, h1_, l0_, l1_);
-            mma_split(sacc[2 * p + 1], ah, al, h2_, h3_, l2_, l3_);
-          } else {
-            mma_bf16_16816(sacc[2 * p], ah, h0_, h1_);
-            mma_bf16_16816(sacc[2 * p], al, h0_, h1_);
-            mma_bf16_16816(sacc[2 * p + 1], ah, h2_, h3_);
-            mma_bf16_16816(sacc[2 * p + 1], al, h2_, h3_);
-          }
-        }
-      }
-    }
-    publish();
-    cp_async_wait<0>();
     __syncthreads();
-    if (c + 1 < nc) load_b(c + 1);
-    cp_async_commit();
   }
-  if (warp < MT) {
+  if (updates) {
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int cc = v0 + nt * 8 + 2 * tq;
@@ -620,15 +704,8 @@ static int launch_prep(const DmoeRecur& a, const void* chunks, int n_chunks, uin
 
 template <int DP, int VT, bool DELTA>
 static int launch_scan(const DmoeRecur& a, const uint8_t* ws, long long stride, int h0, int hn, cudaStream_t stream) {
-  using SM = ScanSmem<DP, VT, DELTA>;
-  static PerDeviceOnce configured;
-  const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(chunk_scan_kernel<DP, VT, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                                 SM::kBytes));
-  });
-  if (rc != 0) return rc;
   const dim3 grid(a.n_segs, hn, (a.vdim + VT - 1) / VT);
-  chunk_scan_kernel<DP, VT, DELTA><<<grid, kChunkThreads, SM::kBytes, stream>>>(a, ws, stride, h0, hn);
+  chunk_scan_kernel<DP, VT, DELTA><<<grid, kChunkThreads, 0, stream>>>(a, ws, stride, h0, hn);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -69,8 +69,8 @@ class DmoeRecur(ctypes.Structure):
                                    "positions", "rows", "kv_slots", "state", "norm_w", "out", "raw")] + \
                [(n, _ll) for n in ("ldq", "ldk", "ldv", "ldg", "ldb", "ldz", "ldo", "ldraw")] + \
                [(n, _i) for n in ("n_segs", "n_slots", "heads", "kv_heads", "dim", "vdim", "taps", "delta", "decay_kind",
-                                  "gate_kind", "is_f32")] + \
-               [(n, _f) for n in ("qscale", "inv_tau", "eps")]
+                                  "gate_kind", "is_f32", "one_token")] + \
+               [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp)]
 
 
 def lib_path() -> str:

@@ -15,7 +15,7 @@ import torch
 
 from . import _lib, reference
 from .functional import token_runs
-from .gemm import num_sms
+from .gemm import num_sms, scratch
 
 CHUNK = 64          # tokens of a chunk
 MAX_TAPS = 8        # longest short convolution
@@ -117,6 +117,7 @@ def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) ->
     d.delta, d.decay_kind, d.gate_kind = int(r.delta), int(r.delta), int(r.sigmoid_gate)
     d.is_f32 = int(q.dtype == torch.float32)
     d.qscale, d.inv_tau, d.eps = r.dim ** -0.5, 1.0 / r.tau, r.eps
+    d.status = scratch(q.device).status.data_ptr()
     return d
 
 
@@ -144,7 +145,7 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
         d = _descriptor(r, q, k, v, gate, beta, z, state)
         if r.taps:
             d.conv_w, d.ring, d.taps = r.conv_w.data_ptr(), state.ring.data_ptr(), r.taps
-        d.segs, d.n_segs = _lib.ptr(segs.singles), segs.n_single
+        d.segs, d.n_segs, d.one_token = _lib.ptr(segs.singles), segs.n_single, 1
         d.positions, d.rows, d.kv_slots = _lib.ptr(segs.positions), _lib.ptr(segs.rows), _lib.ptr(segs.kv_slots)
         svt = vt
         # few heads in flight: deal the value columns to more CTAs, at the price of a second (norm) launch

@@ -69,18 +69,18 @@ def short_conv(x, taps):
     return sum(pad[j:j + x.shape[0]] * taps[:, j] for j in range(n))
 
 
-def gla_recurrence(q, k, v, log_decay):
-    """q, k, log_decay [T, H, D], v [T, H, V] -> read-outs [T, H, V]."""
+def gla_recurrence(q, k, v, log_decay, with_state=False):
+    """q, k, log_decay [T, H, D], v [T, H, V] -> read-outs [T, H, V] (and the state after the last token)."""
     T, H, D = q.shape
     S = torch.zeros(H, D, v.shape[-1], dtype=q.dtype)
     out = []
     for t in range(T):
         S = torch.exp(log_decay[t])[..., None] * S + k[t][..., None] * v[t][:, None, :]
         out.append((S * q[t][..., None]).sum(1))
-    return torch.stack(out)
+    return (torch.stack(out), S) if with_state else torch.stack(out)
 
 
-def delta_recurrence(q, k, v, log_decay, beta):
+def delta_recurrence(q, k, v, log_decay, beta, with_state=False):
     """As above, but what is written is the error of the read-out at k, scaled by beta [T, H]."""
     T, H, D = q.shape
     S = torch.zeros(H, D, v.shape[-1], dtype=q.dtype)
@@ -90,7 +90,7 @@ def delta_recurrence(q, k, v, log_decay, beta):
         u = beta[t][:, None] * (v[t] - (S * k[t][..., None]).sum(1))
         S = S + k[t][..., None] * u[:, None, :]
         out.append((S * q[t][..., None]).sum(1))
-    return torch.stack(out)
+    return (torch.stack(out), S) if with_state else torch.stack(out)
 
 
 def gla(h, w, p, m, eps):

@@ -180,12 +180,13 @@ class Recur:
         z = (d(self.z) + d(zb)).view(T, H, D)
         if kind == "delta":
             unit = lambda x: (x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(H // G, 1)
-            o = oracle.delta_recurrence(unit(q) * D ** -0.5, unit(k), v, -torch.exp(d(alog))[:, None] * oracle.softplus(z),
-                                        oracle.sigmoid(d(self.beta)))
+            o, S = oracle.delta_recurrence(unit(q) * D ** -0.5, unit(k), v, -torch.exp(d(alog))[:, None] * oracle.softplus(z),
+                                           oracle.sigmoid(d(self.beta)), with_state=True)
             g = oracle.sigmoid(d(self.gate))
         else:
-            o = oracle.gla_recurrence(q * D ** -0.5, k, v, oracle.log_sigmoid(z) / self.r.tau)
+            o, S = oracle.gla_recurrence(q * D ** -0.5, k, v, oracle.log_sigmoid(z) / self.r.tau, with_state=True)
             g = oracle.silu(d(self.gate))
+        self.state = S
         self.want = ((oracle.rms(o, 1e-5) * d(nw)).reshape(T, -1) * g)
 
     def rows(self, a, b):
@@ -193,10 +194,10 @@ class Recur:
         return [cut(t) for t in (self.q, self.k, self.v, self.gate, self.beta, self.z)]
 
 
-def run_steps(seqs, schedule, n_slots, slots, implicit=False):
+def run_steps(seqs, schedule, n_slots, slots, implicit=False, state=None):
     """``schedule``: steps of (sequence, tokens); returns each sequence's outputs. Sequence i lives in slot slots[i]."""
     r0 = seqs[0]
-    state = r0.r.new_state(n_slots, r0.dtype, DEV)
+    state = state or r0.r.new_state(n_slots, r0.dtype, DEV)
     for t in state.tensors():
         t.fill_(7.0)                        # a slot that was used before
     at, out = [0] * len(seqs), [[] for _ in seqs]
@@ -233,6 +234,20 @@ def test_recurrence_cuts(kind, H, G, D, V, taps, dtype):
         assert sum(cuts) == 150
         got, = run_steps([s], [[(0, n)] for n in cuts], 3, [1])
         close(got, s.want, tol(dtype, 2e-4, 6e-2))
+
+
+@BOTH
+@pytest.mark.parametrize("kind,H,G,D,V,taps", [h for h in HEADS if h[5] == 0] + [("delta", 4, 2, 32, 64, 0), ("delta", 2, 2, 128, 128, 0),
+                                              ("delta", 1, 1, 96, 40, 0), ("delta", 2, 2, 8, 8, 0)])
+@pytest.mark.parametrize("decay", [0.05, 1.0, 20.0])
+def test_state_is_fp32(kind, H, G, D, V, taps, decay, dtype):
+    """The state after prompts, portions and single tokens, with inputs that are exact in both formats: fp32 accuracy also
+    where the activations are bf16."""
+    s = Recur(kind, H, G, D, V, taps, 200, dtype, seed=5, decay=decay)
+    for cuts in ([200], [129, 1, 70], [1] * 30 + [100, 2, 68]):
+        state = s.r.new_state(2, dtype, DEV)
+        run_steps([s], [[(0, n)] for n in cuts], 2, [1], state=state)
+        close(state.S[1], s.state, 3e-4)
 
 
 @pytest.mark.parametrize("kind,H,G,D,V,taps", HEADS)
