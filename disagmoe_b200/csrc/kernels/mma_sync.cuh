@@ -38,8 +38,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // operands give fp32-like accuracy on the bf16 tensor cores.
 __device__ __forceinline__ float bf16_rest(float v) { return v - __bfloat162float(__float2bfloat16(v)); }
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(x, y);
-  lo = pack_bf16(bf16_rest(x), bf16_rest(y));
+  hi = pack_bf16(x, y);                  // the halves are the upper 16 bits of their fp32 values
+  lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 __device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0,
                                           uint32_t bh1, uint32_t bl0, uint32_t bl1) {

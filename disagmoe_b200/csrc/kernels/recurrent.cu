@@ -351,11 +351,11 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
 }
 
 // Causal depthwise convolution + silu of the q | k | v projections of one chunk of a segment, VEC neighbouring channels per
-// thread. The taps before the segment's first row come from the ring: ring[slot][p % taps][channel] = projection at p.
-template <typename T, int VEC>
+// thread (TAPS: bound of the number of taps). The taps before the segment's first row come from the ring: ring[slot][p % taps][channel] = projection at p.
+template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(128)
 conv_chunk_kernel(const DmoeRecur a, const int4* __restrict__ chunks, T* __restrict__ out, long long ldo) {
-  constexpr int HIST = kMaxTaps - 1, STEP = 8;
+  constexpr int HIST = TAPS - 1, STEP = 8;
   const int4 ck = chunks[blockIdx.x];
   const int4 seg = static_cast<const int4*>(a.segs)[ck.z];
   const int C = 2 * a.kv_heads * a.dim + a.heads * a.vdim;
@@ -368,11 +368,11 @@ conv_chunk_kernel(const DmoeRecur a, const int4* __restrict__ chunks, T* __restr
   else if (c < 2 * qc) { src = static_cast<const T*>(a.k) + c - qc; ld = a.ldk; }
   else { src = static_cast<const T*>(a.v) + c - 2 * qc; ld = a.ldv; }
   const T* ring = static_cast<const T*>(a.ring) + static_cast<long long>(seg.z) * R * C + c;
-  float w[kMaxTaps][VEC];               // w[j]: weight of the input j tokens back
+  float w[TAPS][VEC];               // w[j]: weight of the input j tokens back
   float x[HIST + STEP][VEC];            // x[HIST + i]: input of row i of the step
   const int pos0 = seg.w + (ck.x - seg.x);     // position of the chunk's first row
 #pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j)
+  for (int j = 0; j < TAPS; ++j)
 #pragma unroll
     for (int e = 0; e < VEC; ++e) w[j][e] = j < R ? a.conv_w[static_cast<long long>(c + e) * R + R - 1 - j] : 0.f;
 #pragma unroll
@@ -397,8 +397,8 @@ conv_chunk_kernel(const DmoeRecur a, const int4* __restrict__ chunks, T* __restr
         for (int e = 0; e < VEC; ++e) {
           acc[e] = 0.f;
 #pragma unroll
-          for (int j = kMaxTaps - 1; j >= 0; --j) acc[e] += w[j][e] * x[HIST + i - j][e];
-          acc[e] = silu(acc[e]);
+          for (int j = TAPS - 1; j >= 0; --j) acc[e] += w[j][e] * x[HIST + i - j][e];
+          acc[e] = sizeof(T) == 2 ? __fdividef(acc[e], 1.f + __expf(-acc[e])) : silu(acc[e]);
         }
         store_any<VEC>(out + (ck.x + t + i) * ldo + c, acc);
       }
@@ -557,13 +557,15 @@ extern "C" int dmoe_conv_chunks(const DmoeRecur* a, const void* chunks, int n_ch
   const int per = pairs ? 256 : 128;
   const dim3 g1(n_chunks, (C + per - 1) / per), g2(a->n_segs, (C + 255) / 256);
   const int4* ck = static_cast<const int4*>(chunks);
-  if (a->is_f32) {
-    conv_chunk_kernel<float, 1><<<g1, 128, 0, stream>>>(*a, ck, static_cast<float*>(out), ldo);
-    ring_update_kernel<float><<<g2, 256, 0, stream>>>(*a);
-  } else {
-    if (pairs) conv_chunk_kernel<__nv_bfloat16, 2><<<g1, 128, 0, stream>>>(*a, ck, static_cast<__nv_bfloat16*>(out), ldo);
-    else conv_chunk_kernel<__nv_bfloat16, 1><<<g1, 128, 0, stream>>>(*a, ck, static_cast<__nv_bfloat16*>(out), ldo);
-    ring_update_kernel<__nv_bfloat16><<<g2, 256, 0, stream>>>(*a);
-  }
+#define DMOE_CONV(T_, VEC_)                                                                                       \
+  do {                                                                                                           \
+    if (a->taps <= 4) conv_chunk_kernel<T_, VEC_, 4><<<g1, 128, 0, stream>>>(*a, ck, static_cast<T_*>(out), ldo); \
+    else conv_chunk_kernel<T_, VEC_, kMaxTaps><<<g1, 128, 0, stream>>>(*a, ck, static_cast<T_*>(out), ldo);      \
+    ring_update_kernel<T_><<<g2, 256, 0, stream>>>(*a);                                                          \
+  } while (0)
+  if (a->is_f32) DMOE_CONV(float, 1);
+  else if (pairs) DMOE_CONV(__nv_bfloat16, 2);
+  else DMOE_CONV(__nv_bfloat16, 1);
+#undef DMOE_CONV
   return static_cast<int>(cudaGetLastError());
 }

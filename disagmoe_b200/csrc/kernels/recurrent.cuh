@@ -13,7 +13,19 @@ __device__ __forceinline__ float warp_sum(float v) {
   return v;
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// log(1 + e) for 0 <= e <= 1 as 2 atanh(e / (2 + e)): the odd series in s <= 1/3, to full fp32 accuracy also for tiny e
+__device__ __forceinline__ float log1p_unit(float e) {
+  const float s = __fdividef(e, 2.f + e), q = s * s;
+  float p = 1.f / 15.f;
+  p = p * q + 1.f / 13.f;
+  p = p * q + 1.f / 11.f;
+  p = p * q + 1.f / 9.f;
+  p = p * q + 1.f / 7.f;
+  p = p * q + 1.f / 5.f;
+  p = p * q + 1.f / 3.f;
+  return 2.f * (s + s * q * p);
+}
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1p_unit(expf(-fabsf(x))); }
 // log of the decay of one key channel: kind 0: log sigmoid(z) * scale, kind 1: -scale * softplus(z)
 __device__ __forceinline__ float log_decay(int kind, float z, float scale) {
   return kind == 0 ? -softplus(-z) * scale : -scale * softplus(z);

@@ -120,13 +120,17 @@ __device__ __forceinline__ void invert_unit_lower(const float* A, float* T, floa
     for (int I = dist; I < 4; ++I) {
       const int J = I - dist;
       float s = 0.f;
-      for (int k = 16 * J; k < 16 * I; ++k) s += A[(16 * I + i) * LD + k] * T[k * LD + 16 * J + j];
+      for (int K = J; K < I; ++K) {
+#pragma unroll
+        for (int k = 0; k < 16; ++k) s += A[(16 * I + i) * LD + 16 * K + k] * T[(16 * K + k) * LD + 16 * J + j];
+      }
       m[(J * 16 + i) * 17 + j] = s;
     }
     __syncthreads();
     for (int I = dist; I < 4; ++I) {
       const int J = I - dist;
       float s = 0.f;
+#pragma unroll
       for (int k = 0; k < 16; ++k) s -= T[(16 * I + i) * LD + 16 * I + k] * m[(J * 16 + k) * 17 + j];
       T[(16 * I + i) * LD + 16 * J + j] = s;
     }
@@ -247,16 +251,20 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   const bool slow = __syncthreads_or(wide);
 
   // ---- k e^(b_end - b): through shared memory into transposed fragments
-  auto stage_k = [&](int ref) {                      // k e^(b_ref - b)
+  auto stage_k = [&] {
 #pragma unroll
-    for (int i = 0; i < ROWS; ++i) {
-      float x[PL];
-#pragma unroll
-      for (int e = 0; e < PL; ++e) x[e] = k[i][e] * exp2f(s_b[ref * DP + d0 + e] - s_b[(t0 + i) * DP + d0 + e]);
-      store_split<PL>(s_kh + (t0 + i) * SM::kKs + d0, s_kl + (t0 + i) * SM::kKs + d0, x);
-    }
+    for (int i = 0; i < ROWS; ++i)
+      store_split<PL>(s_kh + (t0 + i) * SM::kKs + d0, s_kl + (t0 + i) * SM::kKs + d0, k[i]);
   };
-  stage_k(kChunk - 1);
+  float to_mid[PL];                                  // e^(m - b_end)
+#pragma unroll
+  for (int e = 0; e < PL; ++e) {
+    const float end = s_b[(kChunk - 1) * DP + d0 + e];
+    to_mid[e] = slow ? 0.f : exp2f(s_b[kMid * DP + d0 + e] - end);
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) k[i][e] *= exp2f(end - s_b[(t0 + i) * DP + d0 + e]);
+  }
+  stage_k();
   __syncthreads();
   for (int i = warp; i < MT * 4; i += kChunkThreads / 32) {
     const int mt = i / 4, ks = i % 4;
@@ -268,7 +276,13 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
     store_frag(w + L::kK + (i * 2 + 1) * kFrag, lane, f);
   }
   __syncthreads();
-  if (!slow) stage_k(kMid);                     // now k e^(m - b): right operand of P and A
+  if (!slow) {                                       // now k e^(m - b): right operand of P and A
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i)
+#pragma unroll
+      for (int e = 0; e < PL; ++e) k[i][e] *= to_mid[e];
+    stage_k();
+  }
   __syncthreads();
 
   // ---- P and the fragments of q e^b (warps 0-3), A (warps 4-7)

@@ -11,6 +11,7 @@ import ctypes
 from dataclasses import dataclass
 from typing import Optional
 
+import numpy as np
 import torch
 
 from . import _lib, reference
@@ -41,15 +42,15 @@ class SegmentTables:
 
 def build_segments(bt_row, positions, device) -> SegmentTables:
     """Tables of a batch given on the host (rows of one sequence are consecutive, as every scheduler emits them)."""
-    rows, pos = torch.as_tensor(bt_row).tolist(), torch.as_tensor(positions).tolist()
+    rows, pos = np.asarray(bt_row), np.asarray(positions)
     singles, multi, chunks = [], [], []
     for a, b in token_runs(rows, pos):
+        seg = (a, b - a, int(rows[a]), int(pos[a]))
         if b - a == 1:
-            singles.append((a, 1, rows[a], pos[a]))
+            singles.append(seg)
             continue
-        for i, c in enumerate(range(a, b, CHUNK)):
-            chunks.append((c, min(CHUNK, b - c), len(multi), i))
-        multi.append((a, b - a, rows[a], pos[a]))
+        chunks += [(c, min(CHUNK, b - c), len(multi), i) for i, c in enumerate(range(a, b, CHUNK))]
+        multi.append(seg)
     table = torch.tensor(singles + multi + chunks, dtype=torch.int32).reshape(-1, 4)
     if torch.device(device).type == "cuda":
         table = table.to(device)
