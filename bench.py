@@ -170,7 +170,7 @@ def main():
 
     import torch
     import torch.distributed as dist
-    from disagmoe_b200.config import CacheConfig, get_preset
+    from disagmoe_b200.config import CacheConfig, LayerListConfig, get_preset
 
     world = int(os.environ.get("WORLD_SIZE", "1"))
     rank = int(os.environ.get("RANK", "0"))
@@ -181,6 +181,8 @@ def main():
     W = max(args.warmup, 3)
     K = args.steps
     cfg = get_preset(args.model)
+    if isinstance(cfg, LayerListConfig):
+        raise SystemExit(f"{cfg.name} is not an MoE model: use --layer-list")
     if args.layers:
         cfg = cfg.clone(num_layers=args.layers)
     cfg.max_seq_len = max(4096, (args.ctx_max + K + W + args.timeline + 2 + 15) // 16 * 16)

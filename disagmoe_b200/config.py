@@ -95,8 +95,8 @@ class RotarySpec:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Softmax attention with per-head query / key norm. ``window``: a token sees itself and the window - 1 tokens before
-    it (None: all). ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none)."""
+    """Softmax attention with per-head query / key norm. ``window``: how many of the latest tokens, its own included, a
+    query attends to (None: all). ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none)."""
     heads: int
     kv_heads: int
     dim: int

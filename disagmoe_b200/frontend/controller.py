@@ -234,6 +234,8 @@ class Controller:
     def init_engine(self, placement: ModelPlacement, model_config: ModelConfig, cache_config: Optional[CacheConfig] = None,
                     sampling_config: Optional[SamplingConfig] = None, state_dict_path: Optional[str] = None,
                     keep_logits: bool = False, dtype=None, ignore_eos: bool = True) -> None:
+        from ..models.registry import require_experts
+        require_experts(model_config)
         self.placement, self.model_config = placement, model_config
         self._init_args = (placement, model_config, cache_config, sampling_config, state_dict_path, keep_logits, dtype,
                            ignore_eos)

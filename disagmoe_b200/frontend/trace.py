@@ -4,7 +4,7 @@
 
 DIR is a checkpoint folder (config.json, model.safetensors). Every input line is one engine step,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["b"]}
+    {"step": 7, "entries": [{"id": "q1", "tokens": [311, 8], "want": [1]}, {"id": "q2", "tokens": [42], "want": [0]}], "end": ["q2"]}
 
 whose entries run as one batch (portions of prompts beside single tokens) from the cache and state that earlier steps
 left; ``want`` are the places among an entry's tokens whose logits are written, in order, to ``<out>/<step>.f32``

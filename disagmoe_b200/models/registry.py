@@ -87,6 +87,12 @@ def resolve_model(name_or_path: str, dtype: Optional[torch.dtype] = None, **kw) 
     raise ValueError(f"{name_or_path!r} is neither a preset ({', '.join(sorted(PRESETS))}) nor a checkpoint folder")
 
 
+def require_experts(cfg: ModelConfig) -> None:
+    """The disaggregated paths place routed experts on GPUs of their own; a model without any is refused there."""
+    if isinstance(cfg, LayerListConfig):
+        raise ValueError(f"{cfg.name} has no routed experts: serve it with the single-GPU engines (--backend colocated)")
+
+
 def make_executor(cfg: ModelConfig, cache_cfg, **kw):
     """The whole-iteration executor that runs ``cfg`` on one device."""
     from ..executor.fused import FusedModelExecutor

@@ -266,7 +266,9 @@ class FusedServingRank:
         sharing inside a TP group, scheduling, result collection) then runs as plain CPU processes."""
         import torch.distributed as dist
         from .. import disagmoe_c as C
+        from ..models.registry import require_experts
         from ..ops import _lib, gemm
+        require_experts(cfg)
         from .disagg import AttentionRank, DisaggShape, ExpertRank, build_layout
         from .peer import PeerArena
         self.dist, self._lib, self._gemm = dist, _lib, gemm

@@ -191,3 +191,13 @@ def test_serving_command_line_from_a_checkpoint_folder(tmp_path, budget):
         from benchmark.benchmark_serving import model_from_args
         from benchmark.utils import get_parser_base
         model_from_args(get_parser_base().parse_args(argv + ["--backend", "controller"]))
+
+
+def test_disaggregated_paths_refuse_models_without_experts():
+    from disagmoe_b200.frontend.controller import init_controller
+    from disagmoe_b200.parallel.serving import FusedServingRank
+    cfg = get_preset("rurunex")
+    with pytest.raises(ValueError, match="no routed experts"):
+        FusedServingRank(cfg, 2, 0, 0, 1)
+    with pytest.raises(ValueError, match="no routed experts"):
+        init_controller(1, 2, device="cpu").init_engine(None, cfg)
