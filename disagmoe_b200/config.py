@@ -79,24 +79,32 @@ class ModelConfig:
         return replace(self, **changes)
 
 
+ACTIVATIONS = ("silu", "gelu_tanh")             # of gated feed-forwards
+
+
 # ---- decoders described layer by layer --------------------------------------------------------------------------------
-# A layer = one token mixer (attention or a linear recurrence) and an optional feed-forward, each between a norm before it
-# and a norm after it. Mixers carry their own sizes, so layers of one model may differ in everything but the width.
+# A layer = one token mixer (attention or a linear recurrence) and an optional feed-forward, dense or routed to experts.
+# Mixers carry their own sizes, so layers of one model may differ in everything but the width. How the two sublayers sit on
+# the residual stream is the model's ``block``.
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary embedding on the first ``dims`` dimensions of a head (pairs i, i + dims / 2); ``factor`` != None: YaRN."""
+    """Rotary embedding on the first ``dims`` dimensions of a head: pairs (i, i + dims / 2), or (2i, 2i + 1) where
+    ``interleaved``; ``factor`` != None: YaRN."""
     dims: int
     base: float
     factor: Optional[float] = None
     original: float = 0.0
     fast: float = 32.0
     slow: float = 1.0
+    interleaved: bool = False
 
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Softmax attention with per-head query / key norm. ``window``: how many of the latest tokens, its own included, a
-    query attends to (None: all). ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none)."""
+    """Softmax attention. ``window``: how many of the latest tokens, its own included, a query attends to (None: all).
+    ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none). ``qk_norm``: RMS norm
+    of every query and key head. ``sink``: a learned number per head enters the softmax denominator. ``v_mix``: the values
+    are mixed with those that the first such layer computed for the same token."""
     heads: int
     kv_heads: int
     dim: int
@@ -106,6 +114,24 @@ class AttentionSpec:
     window: Optional[int] = None
     softcap: Optional[float] = None
     kv_from: Optional[int] = None
+    qk_norm: bool = True
+    sink: bool = False
+    v_mix: bool = False
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Softmax attention whose keys and values are linear maps of one latent vector of ``kv_rank`` numbers per token; beside
+    it every token has one rotated key part of ``rot_dim`` numbers that all heads share. The cache holds those two."""
+    heads: int
+    dim: int                                    # unrotated query / key size per head
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: Optional[RotarySpec] = None
+    window: Optional[int] = None
+    sink: bool = False
 
 
 @dataclass(frozen=True)
@@ -132,29 +158,56 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class RoutedSpec:
+    """Feed-forward of ``experts`` gated feed-forwards of width ``ff``; a token uses the ``top`` ones with the largest
+    softmax scores, weighted by these scores (``renormalize``: divided by their sum)."""
+    experts: int
+    top: int
+    ff: int
+    act: str = "silu"
+    renormalize: bool = False
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, GatedLinearSpec, ChannelDeltaSpec]
-    ff: Optional[int] = None                    # width of the gated feed-forward, None = the layer has none
+    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, ChannelDeltaSpec]
+    ff: Optional[int] = None                    # width of the dense gated feed-forward, None = the layer has none
+    act: str = "silu"                           # of the dense feed-forward: silu or gelu_tanh
+    routed: Optional[RoutedSpec] = None         # experts instead of a dense feed-forward
 
 
 @dataclass
 class LayerListConfig(ModelConfig):
-    """A decoder given as a list of :class:`LayerSpec`. The MoE fields of the base class stay at zero: everything is on
-    the attention side, so only the single-GPU engines serve it."""
+    """A decoder given as a list of :class:`LayerSpec`. The MoE fields of the base class stay at zero: experts, where
+    layers have some, run beside the attention, and only the single-GPU engines serve these models.
+
+    ``block``: how a layer's sublayers sit on the residual stream x.
+      "sandwich"  x += post(mixer(pre(x))), then x += post(ff(pre(x))); RMS norms whose stored weight is an offset from one
+      "parallel"  h = norm(x); x += mixer(h) + ff(h); layer norms (mean taken off) with a plain weight
+    """
     layers: List[LayerSpec] = field(default_factory=list)
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     architecture: str = ""
+    block: str = "sandwich"
 
     def is_dense_layer(self, layer_id: int) -> bool:
         return True
 
     def __post_init__(self):
         super().__post_init__()
-        assert self.num_layers == len(self.layers)
+        assert self.num_layers == len(self.layers) and self.block in ("sandwich", "parallel")
         for i, layer in enumerate(self.layers):
-            m = layer.mixer
-            if isinstance(m, GatedLinearSpec):
+            m, r = layer.mixer, layer.routed
+            if layer.act not in ACTIVATIONS or (r is not None and r.act not in ACTIVATIONS):
+                raise ValueError(f"layer {i}: unknown activation (known: {', '.join(ACTIVATIONS)})")
+            if r is not None and (layer.ff or self.block == "sandwich" or not 1 <= r.top <= r.experts):
+                raise ValueError(f"layer {i}: experts need a parallel block, no dense feed-forward beside them and 1 <= top "
+                                 f"<= experts")
+            rot = getattr(m, "rot", None)
+            if rot is not None and (rot.dims % 2 or rot.dims > (m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim)):
+                raise ValueError(f"layer {i}: {rot.dims} rotated dimensions do not fit the head")
+            if isinstance(m, (GatedLinearSpec, LatentAttentionSpec)):
                 continue
             if m.heads % m.kv_heads:
                 raise ValueError(f"layer {i}: {m.heads} heads do not share {m.kv_heads} key / value heads evenly")
@@ -164,13 +217,23 @@ class LayerListConfig(ModelConfig):
                 if not isinstance(s, AttentionSpec) or s.kv_from is not None or \
                         (s.kv_heads, s.dim, s.vdim) != (m.kv_heads, m.dim, m.vdim):
                     raise ValueError(f"layer {i} cannot read the keys and values of layer {src}")
+            first = self.first_v_mix
+            if getattr(m, "v_mix", False):
+                f = self.layers[first].mixer
+                if m.kv_from is not None or (f.kv_heads, f.vdim) != (m.kv_heads, m.vdim):
+                    raise ValueError(f"layer {i} cannot mix its values with those of layer {first}")
+
+    @property
+    def first_v_mix(self) -> Optional[int]:
+        """The layer whose values the later value-mixing layers mix in."""
+        return next((i for i, l in enumerate(self.layers) if getattr(l.mixer, "v_mix", False)), None)
 
     @classmethod
     def make(cls, width: int, vocab: int, layers: List[LayerSpec], dtype=torch.bfloat16, **kw) -> "LayerListConfig":
         heads = max(l.mixer.heads for l in layers)
         kw = {**dict(rms_norm_eps=1e-6, head_dim=max(l.mixer.dim for l in layers)), **kw}
         return cls(hidden_size=width, num_layers=len(layers), num_heads=heads, num_kv_heads=heads, num_experts=0,
-                   intermediate_size=max((l.ff or 0) for l in layers), dtype=dtype, ep_size=1, top_k=0, vocab_size=vocab,
+                   intermediate_size=max((l.routed.ff if l.routed else l.ff or 0) for l in layers), dtype=dtype, ep_size=1, top_k=0, vocab_size=vocab,
                    layers=list(layers), **kw)
 
 
@@ -244,7 +307,25 @@ def _rurunex_layers(groups: int, heads: int, dim: int, ff: int) -> List[LayerSpe
 rurunex_config = LayerListConfig.make(2048, 32000, _rurunex_layers(6, 16, 128, 5632), max_seq_len=8192, embed_scale=45.25,
                                       logit_scale=0.25, architecture="Rurunex", name="rurunex-18l")
 
+# Supinex design at the size of a small production model (random weights): grouped-query attention over the whole context
+# and windowed latent attention in turn; experts in every layer but the first.
+def _supinex_layers(groups: int, heads: int, dim: int, rank: int, ff: int, experts: RoutedSpec, window: int) -> List[LayerSpec]:
+    rot, half = RotarySpec(dim, 5e5, interleaved=True), dim // 2
+    attn = AttentionSpec(heads, max(1, heads // 4), dim, dim, scale=dim ** -0.5, rot=rot, qk_norm=False, sink=True, v_mix=True)
+    latent = LatentAttentionSpec(heads, dim, half, dim, rank, scale=(dim + half) ** -0.5, window=window, sink=True,
+                                 rot=RotarySpec(half, 1e6, factor=4.0, original=8192, interleaved=True))
+    out: List[LayerSpec] = []
+    for g in range(groups):
+        out += [LayerSpec(attn, routed=experts) if g else LayerSpec(attn, ff, "gelu_tanh"), LayerSpec(latent, routed=experts)]
+    return out
+
+
+supinex_config = LayerListConfig.make(
+    2048, 32000, _supinex_layers(8, 16, 128, 512, 5632, RoutedSpec(64, 6, 1408), 1024), max_seq_len=8192, block="parallel",
+    architecture="Supinex", name="supinex-16l")
+
 PRESETS = {
+    "supinex": supinex_config,
     "rurunex": rurunex_config,
     "mixtral": mixtral_config, "mixtral-8x7b": mixtral_config, "duo": duo_expert_mixtral,
     "qwen-moe": qwen_moe_config, "deepseek-v2-lite": deepseek_v2_lite_config, "tiny": tiny_config,

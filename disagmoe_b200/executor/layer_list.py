@@ -1,23 +1,27 @@
 """Whole-iteration executor of layer-list decoders (:class:`disagmoe_b200.config.LayerListConfig`).
 
-    embed * scale -> per layer [ norm -> mixer -> norm + add (-> norm -> gated feed-forward -> norm + add) ]
-                  -> norm -> head -> argmax
+    sandwich  embed * scale -> per layer [ norm -> mixer -> norm + add (-> norm -> gated feed-forward -> norm + add) ]
+    parallel  embed * scale -> per layer [ norm (+ router) -> mixer, feed-forward or experts on the same rows -> add both ]
+              -> norm -> head -> argmax
 
-The residual stream is fp32; the norm after a sublayer, the residual add and the norm before the next sublayer are one
-launch. Two kinds of per-sequence memory: KV pages for the attention layers that have keys and values of their own (layers
-that read another layer's have none), and for recurrent layers one state slot per sequence, numbered like its row of the
-block table, so the block manager's row allocation is the slot allocation. As in the MoE executor, a decode iteration is
-one chain of launches captured per batch-size bucket, prompts run eagerly, and CPU tensors run the PyTorch restatements.
+The residual stream is fp32; what stands between two sublayers (norm after, residual add, norm before, and the router of a
+layer with experts) is one launch. Two kinds of per-sequence memory: pages for the attention layers that have keys and values
+of their own (layers that read another layer's have none; latent attention keeps one latent row per token), and for recurrent
+layers one state slot per sequence, numbered like its row of the block table, so the block manager's row allocation is the
+slot allocation. As in the MoE executor, a decode iteration is one chain of launches captured per batch-size bucket, prompts
+run eagerly, and CPU tensors run the PyTorch restatements.
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec
+from ..config import AttentionSpec, LatentAttentionSpec
 from ..models import weights as W
-from ..models.mixers import GatedFeedForward, StepMeta, make_mixer
+from ..models.mixers import (GatedFeedForward, LatentTables, RoutedBuffers, RoutedFeedForward, ScatterRows, StepMeta,
+                             make_mixer)
 from ..ops import functional as F
 from ..ops import gemm
 from ..ops.recurrent import MAX_TAPS, RecurrentState, SegmentTables, build_segments, decode_segments
@@ -25,8 +29,15 @@ from .step import StepExecutor, TokenBuffers
 
 
 class LayerListBuffers(TokenBuffers):
-    def __init__(self, cfg, cap: int, device, logit_rows: int):
+    def __init__(self, cfg, cap: int, device, dtype, logit_rows: int, mixers):
         super().__init__(cfg, cap, device, logit_rows)
+        self.routed: Dict[Tuple[int, int], RoutedBuffers] = {}
+        for r in {(l.routed.experts, l.routed.top) for l in cfg.layers if l.routed}:
+            self.routed[r] = RoutedBuffers(cap, cfg.hidden_size, *r, device, dtype)
+        self.latent_out: Dict[int, ScatterRows] = {}
+        for size in {m.lay.heads * m.lay.vdimp for m in mixers if hasattr(m, "lay")}:
+            self.latent_out[size] = ScatterRows(cap, size, device, dtype)
+        self.latent: Dict[Tuple, LatentTables] = {}          # of a prefill step
         self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=device)
         self.segments: Optional[SegmentTables] = None        # None: decode step, every row its own segment
         self.prefill_tiles: Dict[int, Tuple[torch.Tensor, int]] = {}    # tokens per tile -> (table, tiles)
@@ -42,36 +53,42 @@ class LayerListExecutor(StepExecutor):
             raise ValueError(f"short convolutions longer than {MAX_TAPS} taps are not supported")
         # without a checkpoint: seeded random weights, created on the device tensor by tensor
         sd = state_dict if state_dict is not None else W.init_state_dict(cfg, dev, dt)
-        one_plus = lambda n: (1.0 + sd[n].to(device=dev, dtype=torch.float32)).contiguous()
+        # sandwich norms are stored as offsets from one
+        plus = 0.0 if cfg.block == "parallel" else 1.0
+        norm = lambda n: (plus + sd[n].to(device=dev, dtype=torch.float32)).contiguous()
         self.embed_w = sd["embed"].to(device=dev, dtype=dt).contiguous()
         self.head_w = sd["head"].to(device=dev, dtype=dt).contiguous()
-        self.final_norm = one_plus("final.norm")
+        self.final_norm = norm("final.norm")
         self.mixers, self.ffs, self.norms = [], [], []
         for i, layer in enumerate(cfg.layers):
             m = make_mixer(cfg, i, dev, dt)
             m.load_weights(sd)
             self.mixers.append(m)
-            self.ffs.append(GatedFeedForward(sd, f"l{i}.mlp.", dev, dt) if layer.ff else None)
-            self.norms.append({n: one_plus(f"l{i}.{n}") for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.ff else ())})
+            p = f"l{i}.mlp."
+            self.ffs.append(RoutedFeedForward(sd, p, layer.routed, dev, dt) if layer.routed else
+                            GatedFeedForward(sd, p, layer.ff, layer.act, dev, dt) if layer.ff else None)
+            self.norms.append({n: norm(f"l{i}.{n}") for n in W.layer_norm_names(cfg, i)})
+        self.latent_specs = {LatentTables.key(l.mixer): l.mixer for l in cfg.layers if isinstance(l.mixer, LatentAttentionSpec)}
+        self.decode_tables: Dict[int, Dict[Tuple, LatentTables]] = {}
 
     # ---- cache and state ------------------------------------------------------------------------------------------
     def _owns_kv(self, i: int) -> bool:
         m = self.cfg.layers[i].mixer
-        return isinstance(m, AttentionSpec) and m.kv_from is None
+        return isinstance(m, LatentAttentionSpec) or isinstance(m, AttentionSpec) and m.kv_from is None
 
     def _cache_bytes_per_block(self) -> int:
         el = torch.empty((), dtype=self.dtype).element_size()
-        return sum(self.block_size * m.kv_heads * (m.dim + m.vdim) * el
-                   for i, m in enumerate(l.mixer for l in self.cfg.layers) if self._owns_kv(i))
+        return sum(self.block_size * math.prod(s) * el for i, m in enumerate(self.mixers) if self._owns_kv(i)
+                   for s in m.kv_shapes())
 
     def _allocate_cache(self) -> None:
         z = lambda *s: torch.zeros(*s, dtype=self.dtype, device=self.device)
-        self.kv: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
+        self.kv: Dict[int, Tuple[torch.Tensor, ...]] = {}
         self.states: Dict[int, RecurrentState] = {}
         for i, layer in enumerate(self.cfg.layers):
             m = layer.mixer
             if self._owns_kv(i):
-                self.kv[i] = tuple(z(self.num_blocks, self.block_size, m.kv_heads, d) for d in (m.dim, m.vdim))
+                self.kv[i] = tuple(z(self.num_blocks, self.block_size, *s) for s in self.mixers[i].kv_shapes())
             elif isinstance(m, AttentionSpec):
                 self.kv[i] = self.kv[m.kv_from]
             else:
@@ -95,16 +112,17 @@ class LayerListExecutor(StepExecutor):
 
     def _make_buffers(self, cap: int) -> LayerListBuffers:
         # prompts sample one row per sequence; a step that wants more rows allocates its logits
-        return LayerListBuffers(self.cfg, cap, self.device, min(cap, self.max_batch_size))
+        return LayerListBuffers(self.cfg, cap, self.device, self.dtype, min(cap, self.max_batch_size), self.mixers)
 
     # ---- one iteration ----------------------------------------------------------------------------------------------
     def _begin_prefill(self, buf: LayerListBuffers, T: int, positions, ctx_len, bt_row) -> None:
         buf.segments = build_segments(bt_row, positions, self.device)
         buf.prefill_tiles, buf.ctx_len_decode, buf.n_untiled = {}, None, T
-        if self.device.type != "cuda":
-            return
-        for m in (l.mixer for l in self.cfg.layers):
-            if not isinstance(m, AttentionSpec) or not F.attention_on_tensor_cores(self.dtype, m.heads, m.kv_heads, m.dim, m.vdim):
+        buf.latent = {k: LatentTables.prefill(m, bt_row, positions, self.device, self.dtype)
+                      for k, m in self.latent_specs.items()}
+        for mixer in self.mixers:
+            m = mixer.spec
+            if not isinstance(m, AttentionSpec) or not mixer.tiled():
                 continue
             n = F.prefill_tile_tokens(m.heads, m.kv_heads)
             if n in buf.prefill_tiles:
@@ -117,32 +135,57 @@ class LayerListExecutor(StepExecutor):
                 buf.ctx_len_decode, buf.n_untiled = cd.to(self.device), int((~covered).sum())
 
     def _end_prefill(self, buf: LayerListBuffers) -> None:
-        buf.segments, buf.prefill_tiles, buf.ctx_len_decode = None, {}, None
+        buf.segments, buf.prefill_tiles, buf.ctx_len_decode, buf.latent = None, {}, None, {}
+
+    def _decode_tables(self, T: int) -> Dict[Tuple, LatentTables]:
+        """Made once per batch size: graphs replay on them."""
+        if T not in self.decode_tables:
+            self.decode_tables[T] = {k: LatentTables.decode(m, T, self.device) for k, m in self.latent_specs.items()}
+        return self.decode_tables[T]
 
     def _forward(self, buf: LayerListBuffers, T: int, max_ctx: int, want_logits: bool):
-        cfg, eps, dt = self.cfg, self.cfg.rms_norm_eps, self.dtype
+        cfg = self.cfg
         pos, slots, rows = buf.positions[:T], buf.slots[:T], buf.bt_row[:T]
         segs = buf.segments if buf.segments is not None else decode_segments(pos, rows, slots)
+        prompts = buf.segments is not None
         meta = StepMeta(pos, slots, self.block_tables, rows, buf.ctx_len[:T], max_ctx=max_ctx,
-                        num_decode_tokens=buf.n_untiled if buf.segments is not None else T,
-                        prefill_tiles=buf.prefill_tiles if buf.segments is not None else None,
-                        ctx_len_decode=buf.ctx_len_decode, segments=segs)
+                        num_decode_tokens=buf.n_untiled if prompts else T,
+                        prefill_tiles=buf.prefill_tiles if prompts else None,
+                        ctx_len_decode=buf.ctx_len_decode, segments=segs,
+                        latent=buf.latent if prompts else self._decode_tables(T), latent_out=buf.latent_out)
         resid = buf.resid[:T]
         F.embed_f32(buf.ids[:T], self.embed_w, cfg.embed_scale, resid)
-        h = F.resid_norm(resid, None, None, self.norms[0]["norm1"], eps, dt)
-        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
-            last = i + 1 == len(self.mixers)
-            y, post = mixer(h, self.states[i] if i in self.states else self.kv[i], meta), n["norm1b"]
-            if ff is not None:
-                h = F.resid_norm(resid, y, post, n["norm2"], eps, dt)
-                y, post = ff(h), n["norm2b"]
-            if last:
-                # the head's input carries the logit scale; only the rows that are sampled get that far
-                h = F.resid_norm(resid, y, post, self.final_norm, eps, dt, out_scale=cfg.logit_scale, rows=buf.out_rows)
-            else:
-                h = F.resid_norm(resid, y, post, self.norms[i + 1]["norm1"], eps, dt)
+        h = (self._parallel_blocks if cfg.block == "parallel" else self._sandwich_blocks)(buf, resid, meta)
         n_out = h.shape[0]
         logits = gemm.linear(h, self.head_w, out=buf.logits[:n_out] if n_out <= buf.logits.shape[0] else None,
                              out_dtype=torch.float32)
         F.argmax(logits, out=buf.next_ids[:n_out])
         return buf.next_ids[:n_out], (logits if want_logits else None)
+
+    def _memory(self, i: int):
+        return self.states[i] if i in self.states else self.kv[i]
+
+    def _sandwich_blocks(self, buf: LayerListBuffers, resid: torch.Tensor, meta: StepMeta) -> torch.Tensor:
+        """All layers; returns the head's input rows."""
+        cfg, eps, dt = self.cfg, self.cfg.rms_norm_eps, self.dtype
+        h = F.resid_norm(resid, None, None, self.norms[0]["norm1"], eps, dt)
+        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
+            y, post = mixer(h, self._memory(i), meta), n["norm1b"]
+            if ff is not None:
+                h = F.resid_norm(resid, y, post, n["norm2"], eps, dt)
+                y, post = ff(h), n["norm2b"]
+            if i + 1 == len(self.mixers):
+                # the head's input carries the logit scale; only the rows that are sampled get that far
+                return F.resid_norm(resid, y, post, self.final_norm, eps, dt, out_scale=cfg.logit_scale, rows=buf.out_rows)
+            h = F.resid_norm(resid, y, post, self.norms[i + 1]["norm1"], eps, dt)
+
+    def _parallel_blocks(self, buf: LayerListBuffers, resid: torch.Tensor, meta: StepMeta) -> torch.Tensor:
+        eps, dt = self.cfg.rms_norm_eps, self.dtype
+        y = z = None
+        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
+            r = self.cfg.layers[i].routed
+            rb = buf.routed[r.experts, r.top] if r else None
+            h, ids, weights = F.sum_norm(resid, y, z, n["norm1"], eps, dt, True, router=ff.router(rb) if r else None)
+            y = mixer(h, self._memory(i), meta)
+            z = ff(h, ids, weights, rb) if r else ff(h) if ff is not None else None
+        return F.sum_norm(resid, y, z, self.final_norm, eps, dt, True, rows=buf.out_rows)[0]

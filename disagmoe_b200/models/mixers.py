@@ -1,4 +1,4 @@
-"""Token mixers and the gated feed-forward of layer-list decoders (:class:`disagmoe_b200.config.LayerListConfig`).
+"""Token mixers and feed-forwards of layer-list decoders (:class:`disagmoe_b200.config.LayerListConfig`).
 
 Each module loads its tensors by the checkpoint's names, fuses the projections that read the same rows into one weight
 (row blocks padded to multiples of 8, so that every block of the output can be the TMA operand of a following GEMM) and
@@ -7,23 +7,101 @@ keep their state in the slot pool (:class:`disagmoe_b200.ops.recurrent.Recurrent
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig
+from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig
 from ..ops import functional as F
 from ..ops import gemm
 from ..ops.recurrent import Recurrence, RecurrentState, SegmentTables, recurrent_attention
 from .attention import AttnMeta
+from .experts import ExpertStack
 from .weights import StateDict
 
 
 @dataclass
 class StepMeta(AttnMeta):
-    """Attention metadata of a step plus the segments the recurrent layers run over."""
+    """Attention metadata of a step plus the segments the recurrent layers run over, the row tables of the latent attention
+    layers and the values that value-mixing layers mix in (set by the first of them)."""
     segments: Optional[SegmentTables] = None
+    latent: Dict[Tuple, "LatentTables"] = field(default_factory=dict)
+    latent_out: Dict[int, "ScatterRows"] = field(default_factory=dict)      # by row size
+    v_first: Optional[torch.Tensor] = None
+
+
+class ScatterRows:
+    """Rows that a combine epilogue scatters to, and the device table of their address (made once: graphs replay on it)."""
+
+    def __init__(self, cap: int, size: int, device, dtype):
+        self.rows = torch.zeros(cap, size, dtype=dtype, device=device)
+        self.base = torch.tensor([self.rows.data_ptr()], dtype=torch.int64, device=device)
+
+
+@dataclass
+class LatentTables:
+    """How one step's rows go through latent attention layers of one kind: prompt runs long enough to expand the latents of
+    their visible keys are tiled, the other ("loose") rows attend over the latents."""
+    n_loose: int
+    loose: Optional[torch.Tensor] = None      # int32 [T]: place of a row among the loose ones, -1 = tiled; None: all are loose
+    rows: Optional[torch.Tensor] = None       # int32 [n_loose]: the batch rows of the loose ones; None: the identity
+    offs: Optional[torch.Tensor] = None       # int32 [heads + 1]: row groups (heads) of the per-head GEMMs
+    recs: Optional[torch.Tensor] = None       # int32 [heads * n_loose, 4]: where their output rows go, see ops.gemm
+    tiles: Optional[torch.Tensor] = None      # int32 [n_tiles, 4], see ops.functional.build_prefill_tiles
+    base: Optional[torch.Tensor] = None       # int32 [n_tiles]: workspace row of position 0 of the tile's sequence
+    n_tiles: int = 0
+    keys: Optional[torch.Tensor] = None       # int32 [n_keys, 2] = (block-table row, position) of every workspace row
+    n_keys: int = 0
+
+    @staticmethod
+    def key(m: LatentAttentionSpec) -> Tuple:
+        return m.heads, m.window, latent_layout(m).min_run()
+
+    @staticmethod
+    def _per_head(rows: torch.Tensor, heads: int, device):
+        """Tables of the per-head GEMMs over [heads, n, .] rows whose outputs go to rows (batch row, head)."""
+        n = len(rows)
+        recs = torch.zeros(heads * n, 4, dtype=torch.int32)
+        recs[:, 1] = (rows[None].long() * heads + torch.arange(heads)[:, None]).reshape(-1).int()
+        recs[:, 2] = torch.ones(1).view(torch.int32)
+        return (torch.arange(heads + 1, dtype=torch.int32) * n).to(device), recs.to(device)
+
+    @classmethod
+    def decode(cls, m: LatentAttentionSpec, T: int, device) -> "LatentTables":
+        return cls(T, None, None, *cls._per_head(torch.arange(T), m.heads, device))
+
+    @classmethod
+    def prefill(cls, m: LatentAttentionSpec, bt_row, positions, device, dtype) -> "LatentTables":
+        lay, T = latent_layout(m), len(positions)
+        if not (device.type == "cuda" and lay.tiled(dtype)):
+            return cls.decode(m, T, device)
+        tiles, covered = F.build_prefill_tiles(bt_row, positions, 64, lay.min_run())
+        if len(tiles) == 0:
+            return cls.decode(m, T, device)
+        rows = (~covered).nonzero()[:, 0].int()
+        loose = torch.full((T,), -1, dtype=torch.int32)
+        loose[rows.long()] = torch.arange(len(rows), dtype=torch.int32)
+        base, keys, at, prev = [], [], 0, (-1, -1)
+        for r0, n, row, pos in tiles.tolist():
+            if (row, pos) != prev:              # a new run: its keys start a window before its first token
+                lo = max(0, pos - m.window + 1) if m.window else 0
+                off = at - lo
+                hi = lo
+            grow = torch.arange(hi, pos + n, dtype=torch.int32)
+            keys.append(torch.stack([torch.full_like(grow, row), grow], 1))
+            at, hi, prev = at + len(grow), pos + n, (row, pos + n)
+            base.append(off)
+        keys = torch.cat(keys)
+        t = cls(len(rows), loose.to(device), rows.to(device), None, None, tiles.to(device),
+                torch.tensor(base, dtype=torch.int32).to(device), len(tiles), keys.to(device), len(keys))
+        if len(rows):
+            t.offs, t.recs = cls._per_head(rows, m.heads, device)
+        return t
+
+
+def latent_layout(m: LatentAttentionSpec) -> F.LatentLayout:
+    return F.LatentLayout(m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank)
 
 
 def _pad8(n: int) -> int:
@@ -32,6 +110,21 @@ def _pad8(n: int) -> int:
 
 def _pad_rows(w: torch.Tensor, rows: int) -> torch.Tensor:
     return w if w.shape[0] == rows else torch.cat([w, w.new_zeros(rows - w.shape[0], w.shape[1])])
+
+
+def _pad_heads(w: torch.Tensor, heads: int, sizes: List[Tuple[int, int]]) -> torch.Tensor:
+    """Rows of w are ``heads`` blocks with parts of the given (size, padded size): zero rows fill every part up."""
+    w = w.reshape(heads, -1, w.shape[1])
+    parts, at = [], 0
+    for n, full in sizes:
+        parts += [w[:, at:at + n], w.new_zeros(heads, full - n, w.shape[2])]
+        at += n
+    return torch.cat(parts, 1).reshape(-1, w.shape[2])
+
+
+def _pad_head_cols(w: torch.Tensor, heads: int, n: int, full: int) -> torch.Tensor:
+    """The same for the columns of a map from concatenated heads of size n."""
+    return w if n == full else _pad_heads(w.T.contiguous(), heads, [(n, full)]).T
 
 
 def _pad_cols(w: torch.Tensor, cols: int) -> torch.Tensor:
@@ -98,28 +191,51 @@ class RecurrentMixer(Mixer):
         return gemm.linear(o, self.o)
 
 
-class NormedAttention(Mixer):
-    """Softmax attention with per-head query / key norm, partial rotation, optional window and score soft cap, over the
-    layer's own paged cache or, with ``kv_from``, an earlier layer's."""
+class SoftmaxAttention(Mixer):
+    """Softmax attention over the layer's own paged cache or, with ``kv_from``, an earlier layer's: optional per-head query /
+    key norm, rotation, window, score soft cap, sink and value mixing. Head sizes without a tensor-core kernel are kept
+    padded with zeros to those of the next one (not where heads are normed)."""
+
+    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
+        super().__init__(cfg, layer_id, device, dtype)
+        m = self.spec
+        self.dk, self.dv = (m.dim, m.vdim) if m.qk_norm or m.kv_from is not None else \
+            F.attention_tile(dtype, self.device, m.heads, m.kv_heads, m.dim, m.vdim)
+
+    def kv_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        """Per token: shapes of what the layer caches."""
+        return (self.spec.kv_heads, self.dk), (self.spec.kv_heads, self.dv)
+
+    def tiled(self) -> bool:
+        return self.device.type == "cuda" and \
+            F.attention_on_tensor_cores(self.dtype, self.spec.heads, self.spec.kv_heads, self.dk, self.dv)
 
     def load_weights(self, sd: StateDict) -> None:
         m = self.spec
         own = m.kv_from is None
         # contiguous head blocks [q | k | v]: the norm + rotation kernel walks them as one row of heads
-        self.proj = FusedProjection([(n, self._get(sd, n)) for n in (("q", "k", "v") if own else ("q",))], pad=False)
-        self.o = self._get(sd, "o")
-        self.q_norm = self._get(sd, "q.norm", torch.float32)
-        self.k_norm = self._get(sd, "k.norm", torch.float32) if own else None
+        parts = [("q", m.heads, m.dim, self.dk)] + ([("k", m.kv_heads, m.dim, self.dk), ("v", m.kv_heads, m.vdim, self.dv)] if own else [])
+        self.proj = FusedProjection([(n, _pad_heads(self._get(sd, n), h, [(d, p)])) for n, h, d, p in parts], pad=False)
+        self.o = _pad_head_cols(self._get(sd, "o"), m.heads, m.vdim, self.dv).contiguous()
+        self.q_norm = self._get(sd, "q.norm", torch.float32) if m.qk_norm else None
+        self.k_norm = self._get(sd, "k.norm", torch.float32) if m.qk_norm and own else None
+        self.sink = self._get(sd, "sink", torch.float32) if m.sink else None
+        mixes = m.v_mix and self.layer_id != self.cfg.first_v_mix
+        self.v_lambda = float(sd[f"l{self.layer_id}.mix.vmix"].float()) if mixes else None
         self.rope = F.rope_freq_table(m.rot, self.cfg.max_seq_len, self.device)
 
     def forward(self, h: torch.Tensor, kv: Tuple[torch.Tensor, torch.Tensor], meta: StepMeta) -> torch.Tensor:
         m, (kc, vc) = self.spec, kv
+        n_kv = 0 if m.kv_from is not None else m.kv_heads
         qkv = self.proj(h)
-        F.qk_norm_rope(qkv, meta.positions, meta.slots, kc, vc, m.heads, 0 if m.kv_from is not None else m.kv_heads, m.dim,
-                       m.vdim, self.rope, self.q_norm, self.k_norm, self.eps)
-        q = qkv[:, :m.heads * m.dim]
-        opt = dict(scale=m.scale, window=m.window, softcap=m.softcap, fp32_weights=True)
-        cuda = q.is_cuda and F.attention_on_tensor_cores(q.dtype, m.heads, m.kv_heads, m.dim, m.vdim)
+        first = meta.v_first if self.v_lambda is not None else None
+        F.qk_norm_rope(qkv, meta.positions, meta.slots, kc, vc, m.heads, n_kv, self.dk, self.dv, self.rope, self.q_norm,
+                       self.k_norm, self.eps, m.rot is not None and m.rot.interleaved, first, self.v_lambda or 0.0)
+        if m.v_mix and self.v_lambda is None:
+            meta.v_first = qkv[:, (m.heads + n_kv) * self.dk:].view(-1, n_kv, self.dv)
+        q = qkv[:, :m.heads * self.dk]
+        opt = dict(scale=m.scale, window=m.window, softcap=m.softcap, fp32_weights=True, sink=self.sink)
+        cuda = self.tiled()
         tiles, n_tiles = meta.prefill_tiles.get(F.prefill_tile_tokens(m.heads, m.kv_heads), (None, 0)) \
             if cuda and meta.prefill_tiles else (None, 0)
         splits = 1
@@ -129,30 +245,124 @@ class NormedAttention(Mixer):
         attn = None
         if n_tiles == 0 or meta.num_decode_tokens > 0:
             attn = F.paged_attention(q, kc, vc, meta.block_tables, meta.bt_row,
-                                     meta.ctx_len_decode if n_tiles else meta.ctx_len, m.heads, m.kv_heads, m.dim,
+                                     meta.ctx_len_decode if n_tiles else meta.ctx_len, m.heads, m.kv_heads, self.dk,
                                      splits=splits, **opt)
         if n_tiles:
             if attn is None:
-                attn = torch.empty(q.shape[0], m.heads * m.vdim, dtype=q.dtype, device=q.device)
-            F.prefill_attention(q, kc, vc, meta.block_tables, tiles, n_tiles, m.heads, m.kv_heads, m.dim, attn, **opt)
+                attn = torch.empty(q.shape[0], m.heads * self.dv, dtype=q.dtype, device=q.device)
+            F.prefill_attention(q, kc, vc, meta.block_tables, tiles, n_tiles, m.heads, m.kv_heads, self.dk, attn, **opt)
         return gemm.linear(attn, self.o)
 
 
-class GatedFeedForward:
-    """down(silu(gate h) * (up h)); the inner width is padded to a multiple of 8 with zero rows / columns."""
+class LatentAttention(Mixer):
+    """Attention over cached latents. Rows on their own (decoding, short portions) multiply the key map into the query and
+    attend over the latents themselves, one shared key and value head; long prompt runs expand the latents of their visible
+    keys into per-head keys and values first, which is cheaper from some tens of queries per key on."""
 
-    def __init__(self, sd: StateDict, prefix: str, device, dtype):
-        get = lambda n: sd[prefix + n].to(device=device, dtype=dtype)
-        gate, up, down = get("gate"), get("up"), get("down")
-        n = _pad8(gate.shape[0])
-        self.w13 = torch.cat([_pad_rows(gate, n), _pad_rows(up, n)]).contiguous()
-        self.w2 = _pad_cols(down, n).contiguous()
+    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
+        super().__init__(cfg, layer_id, device, dtype)
+        self.lay = latent_layout(self.spec)
+
+    def kv_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        return ((self.lay.row,),)
+
+    def load_weights(self, sd: StateDict) -> None:
+        m, lay = self.spec, self.lay
+        H = m.heads
+        q = _pad_heads(self._get(sd, "q"), H, [(m.dim, lay.dimp), (m.rot_dim, lay.rotp)])
+        dkv = _pad_heads(self._get(sd, "dkv"), 1, [(m.kv_rank, lay.rankp), (m.rot_dim, lay.rotp)])
+        self.proj = FusedProjection([("q", q), ("dkv", dkv)])
+        uk = _pad_cols(_pad_heads(self._get(sd, "uk"), H, [(m.dim, lay.dimp)]), lay.rankp).view(H, lay.dimp, lay.rankp)
+        uv = _pad_cols(_pad_heads(self._get(sd, "uv"), H, [(m.vdim, lay.vdimp)]), lay.rankp).view(H, lay.vdimp, lay.rankp)
+        self.absorb, self.expand_v = uk.transpose(1, 2).contiguous(), uv.contiguous()
+        self.expand = torch.cat([uk, uv], 1).reshape(-1, lay.rankp).contiguous() if lay.tiled(self.dtype) and \
+            self.device.type == "cuda" else None
+        self.o = _pad_head_cols(self._get(sd, "o"), H, m.vdim, lay.vdimp).contiguous()
+        self.norm = self._get(sd, "dkv.norm", torch.float32)
+        self.sink = self._get(sd, "sink", torch.float32) if m.sink else None
+        self.rope = F.rope_freq_table(m.rot, self.cfg.max_seq_len, self.device)
+
+    def forward(self, h: torch.Tensor, kv: Tuple[torch.Tensor], meta: StepMeta) -> torch.Tensor:
+        m, lay, cache = self.spec, self.lay, kv[0]
+        T, t = h.shape[0], meta.latent[LatentTables.key(m)]
+        y = self.proj(h)
+        xq, qa = F.latent_prep(y, meta.positions, meta.slots, cache, lay, self.rope, self.norm, self.eps, t.loose, t.n_loose,
+                               m.rot is not None and m.rot.interleaved)
+        out = meta.latent_out[m.heads * lay.vdimp]
+        attn = out.rows[:T]
+        if t.n_loose:
+            gemm.grouped_linear(xq.view(-1, lay.dimp), self.absorb, t.offs, out=qa.view(-1, lay.row)[:, :lay.rankp])
+            o = F.latent_attention(qa, cache, meta.block_tables, meta.bt_row, meta.ctx_len, t.rows, lay, m.scale, m.window,
+                                   self.sink, meta.max_ctx)
+            gemm.grouped_combine(o.view(-1, lay.rankp), self.expand_v, t.offs, t.recs, out.base, lay.vdimp,
+                                 outs=[attn.view(-1, lay.vdimp)])
+        if t.n_tiles:
+            lat = F.latent_gather(cache, meta.block_tables, t.keys, t.n_keys)
+            kvx = gemm.linear(lat[:, :lay.rankp], self.expand)
+            F.latent_prefill(y, kvx, lat, t.tiles, t.base, t.n_tiles, lay, m.scale, m.window, self.sink, attn)
+        return gemm.linear(attn, self.o)
+
+
+def _gated_stack(sd: StateDict, prefixes: List[str], ff: int, device, dtype) -> Tuple[torch.Tensor, torch.Tensor]:
+    """(w13 [n, 2 I, H], w2 [n, H, I]) of gated feed-forwards; the inner width I is ff padded to a multiple of 8 with zero
+    rows / columns."""
+    I = _pad8(ff)
+    get = lambda p, n: sd[p + n].to(device=device, dtype=dtype)
+    H = sd[prefixes[0] + "down"].shape[0]
+    w13 = torch.zeros(len(prefixes), 2 * I, H, dtype=dtype, device=device)
+    w2 = torch.zeros(len(prefixes), H, I, dtype=dtype, device=device)
+    for i, p in enumerate(prefixes):
+        w13[i, :ff], w13[i, I:I + ff], w2[i, :, :ff] = get(p, "gate"), get(p, "up"), get(p, "down")
+    return w13, w2
+
+
+class GatedFeedForward:
+    """down(act(gate h) * (up h))"""
+
+    def __init__(self, sd: StateDict, prefix: str, ff: int, act: str, device, dtype):
+        w13, w2 = _gated_stack(sd, [prefix], ff, device, dtype)
+        self.w13, self.w2, self.act = w13[0], w2[0], act
 
     def __call__(self, h: torch.Tensor) -> torch.Tensor:
-        return gemm.linear(gemm.swiglu_linear(h, self.w13), self.w2)
+        return gemm.linear(gemm.swiglu_linear(h, self.w13, act=self.act), self.w2)
 
 
-MIXERS = {AttentionSpec: NormedAttention, GatedLinearSpec: RecurrentMixer, ChannelDeltaSpec: RecurrentMixer}
+class RoutedBuffers:
+    """Activations of the routed feed-forwards of one shape for up to ``cap`` tokens, shared by the layers that have it:
+    dispatched rows and the weighted output rows [cap, top, width] of the chosen experts."""
+
+    def __init__(self, cap: int, H: int, experts: int, top: int, device, dtype):
+        self.dispatch = F.DispatchBuffers(cap * top, H, experts, device, dtype)
+        self.out = ScatterRows(cap * top, H, device, dtype)
+        self.parts = self.out.rows.view(cap, top, H)
+
+
+class RoutedFeedForward:
+    """Experts on the device that has the attention: sort by expert, grouped GEMMs, weighted rows per (token, choice)."""
+
+    def __init__(self, sd: StateDict, prefix: str, spec, device, dtype):
+        if spec.experts > F.Router.MAX_EXPERTS or spec.top > F.Router.MAX_TOP:
+            raise ValueError(f"more than {F.Router.MAX_EXPERTS} experts or {F.Router.MAX_TOP} per token are not supported")
+        w13, w2 = _gated_stack(sd, [f"{prefix}e{e}." for e in range(spec.experts)], spec.ff, device, dtype)
+        self.spec = spec
+        self.stack = ExpertStack(spec.experts, w2.shape[1], w2.shape[2], device, dtype, spec.act)
+        self.stack.set_weights(w13, w2)
+        self.router_w = sd[prefix + "router"].to(device=device, dtype=dtype).contiguous()
+
+    def router(self, buf: RoutedBuffers) -> F.Router:
+        return F.Router(self.router_w, self.spec.top, self.spec.renormalize, buf.dispatch.counts)
+
+    def __call__(self, h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, buf: RoutedBuffers) -> torch.Tensor:
+        """Output rows [T, top, width], to be summed over the choices."""
+        T, d = h.shape[0], buf.dispatch
+        F.dispatch_local(h, ids, weights, d)
+        n, H = T * self.spec.top, h.shape[1]
+        self.stack.forward_combine(n, d.xs[:n], d.offs, d.recs[:n], buf.out.base, H, outs=[buf.out.rows])
+        return buf.parts[:T]
+
+
+MIXERS = {AttentionSpec: SoftmaxAttention, LatentAttentionSpec: LatentAttention, GatedLinearSpec: RecurrentMixer,
+          ChannelDeltaSpec: RecurrentMixer}
 
 
 def make_mixer(cfg: LayerListConfig, layer_id: int, device, dtype) -> Mixer:

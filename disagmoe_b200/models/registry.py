@@ -13,19 +13,23 @@ from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
 
-from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, LayerSpec, ModelConfig, PRESETS,
-                      RotarySpec, get_preset)
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, LayerSpec,
+                      ModelConfig, PRESETS, RotarySpec, RoutedSpec, get_preset)
 from . import weights as W
 
 
-# ---- Rurunex: gated linear attention, channel-wise gated delta rule and windowed attention in any order -----------------
-def _rotary(rot: Optional[dict]) -> Optional[RotarySpec]:
+def _rotary(rot: Optional[dict], interleaved: bool = False) -> Optional[RotarySpec]:
     if not rot:
         return None
     sc = rot.get("scaling") or {}
-    return RotarySpec(int(rot["dims"]), float(rot["base"]), **{k: float(v) for k, v in sc.items()})
+    return RotarySpec(int(rot["dims"]), float(rot["base"]), interleaved=interleaved, **{k: float(v) for k, v in sc.items()})
 
 
+def _window(mixer: dict) -> Optional[int]:
+    return (mixer.get("mask") or {}).get("size")
+
+
+# ---- Rurunex: gated linear attention, channel-wise gated delta rule and windowed attention in any order -----------------
 def _rurunex_layer(i: int, layer: dict, shapes: Dict[str, Tuple[int, ...]]) -> LayerSpec:
     m, kind = layer["mixer"], layer["type"]
     rank = lambda name: shapes[f"l{i}.mix.{name}"][0] if f"l{i}.mix.{name}" in shapes else 16
@@ -35,7 +39,7 @@ def _rurunex_layer(i: int, layer: dict, shapes: Dict[str, Tuple[int, ...]]) -> L
         mixer = ChannelDeltaSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"], rank("a1"), rank("g1"))
     elif kind == "attention":
         mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), _rotary(m.get("rot")),
-                              (m.get("mask") or {}).get("size"), m.get("softcap"), m.get("kv_from"))
+                              _window(m), m.get("softcap"), m.get("kv_from"))
     else:
         raise ValueError(f"layer {i}: unknown mixer {kind!r}")
     mlp = layer.get("mlp")
@@ -52,6 +56,34 @@ def rurunex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, .
                                 architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
 
 
+# ---- Supinex: attention over everything and windowed latent attention in any order, dense or routed feed-forwards, both
+# sublayers of a layer on one norm -----------------------------------------------------------------------------------------
+def _supinex_layer(i: int, layer: dict) -> LayerSpec:
+    m, kind, mlp = layer["mixer"], layer["type"], layer.get("mlp")
+    rot = _rotary(m.get("rot"), interleaved=True)
+    if kind == "latent_attention":
+        mixer = LatentAttentionSpec(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], float(m["scale"]), rot,
+                                    _window(m), sink=True)
+    elif kind == "attention":
+        mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), rot, _window(m),
+                              qk_norm=False, sink=True, v_mix=bool(m.get("v_mix")))
+    else:
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    if mlp is None:
+        return LayerSpec(mixer)
+    if mlp["kind"] == "dense":
+        return LayerSpec(mixer, mlp["ff"], "gelu_tanh")
+    if mlp["kind"] != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    return LayerSpec(mixer, routed=RoutedSpec(mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]))
+
+
+def supinex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, ...]], **kw) -> LayerListConfig:
+    layers = [_supinex_layer(i, l) for i, l in enumerate(raw["layers"])]
+    return LayerListConfig.make(raw["width"], raw["vocab"], layers, rms_norm_eps=float(raw["norm"]["eps"]), block="parallel",
+                                architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
+
+
 @dataclass(frozen=True)
 class Architecture:
     config_from_json: Callable[..., ModelConfig]
@@ -59,6 +91,7 @@ class Architecture:
 
 ARCHITECTURES: Dict[str, Architecture] = {
     "Rurunex": Architecture(rurunex_config_from_json),
+    "Supinex": Architecture(supinex_config_from_json),
 }
 
 
@@ -88,9 +121,11 @@ def resolve_model(name_or_path: str, dtype: Optional[torch.dtype] = None, **kw) 
 
 
 def require_experts(cfg: ModelConfig) -> None:
-    """The disaggregated paths place routed experts on GPUs of their own; a model without any is refused there."""
+    """The disaggregated paths place the MoE decoder's routed experts on GPUs of their own; layer-list models, which have
+    none or keep them beside the attention, are refused there."""
     if isinstance(cfg, LayerListConfig):
-        raise ValueError(f"{cfg.name} has no routed experts: serve it with the single-GPU engines (--backend colocated)")
+        why = "keeps its experts beside the attention" if any(l.routed for l in cfg.layers) else "has no routed experts"
+        raise ValueError(f"{cfg.name} {why}: serve it with the single-GPU engines (--backend colocated)")
 
 
 def make_executor(cfg: ModelConfig, cache_cfg, **kw):

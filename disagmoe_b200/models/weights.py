@@ -30,20 +30,28 @@ from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, ModelConfig
+from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, ModelConfig
 
 StateDict = Dict[str, torch.Tensor]
 
 
+def layer_norm_names(cfg: LayerListConfig, i: int) -> Tuple[str, ...]:
+    """The residual-stream norms of layer i."""
+    if cfg.block == "parallel":
+        return ("norm1",)
+    return ("norm1", "norm1b") + (("norm2", "norm2b") if cfg.layers[i].ff else ())
+
+
 def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
-    """Names and shapes of a layer-list checkpoint: ``l<i>.norm1 / norm1b / norm2 / norm2b`` around the sublayers,
-    ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward; linear weights [out, in]."""
+    """Names and shapes of a layer-list checkpoint: ``l<i>.norm1 / norm1b / norm2 / norm2b`` around the sublayers (parallel
+    blocks have ``norm1`` alone), ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward, with ``e<j>.`` in front of an
+    expert's tensors; linear weights [out, in]."""
     H = cfg.hidden_size
     out: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab_size, H)}
     for i, layer in enumerate(cfg.layers):
         p, m = f"l{i}.", layer.mixer
         x = p + "mix."
-        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.ff else ()):
+        for n in layer_norm_names(cfg, i):
             out[p + n] = (H,)
         vs = m.heads * m.vdim
         if isinstance(m, GatedLinearSpec):
@@ -57,18 +65,33 @@ def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
             out.update({x + "b": (m.heads, H), x + "A_log": (m.heads,), x + "norm": (m.vdim,), x + "a1": (m.rank, H),
                         x + "a2": (zs, m.rank), x + "dt_bias": (zs,), x + "g1": (m.gate_rank, H),
                         x + "g2": (vs, m.gate_rank)})
+        elif isinstance(m, LatentAttentionSpec):
+            out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.kv_rank + m.rot_dim, H),
+                        x + "dkv.norm": (m.kv_rank,), x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (vs, m.kv_rank)})
         else:
-            out.update({x + "q": (m.heads * m.dim, H), x + "q.norm": (m.dim,)})
-            if m.kv_from is None:
-                out.update({x + "k": (m.kv_heads * m.dim, H), x + "v": (m.kv_heads * m.vdim, H), x + "k.norm": (m.dim,)})
+            own = m.kv_from is None
+            out[x + "q"] = (m.heads * m.dim, H)
+            if own:
+                out.update({x + "k": (m.kv_heads * m.dim, H), x + "v": (m.kv_heads * m.vdim, H)})
+            if m.qk_norm:
+                out.update({x + n + ".norm": (m.dim,) for n in (("q", "k") if own else ("q",))})
+            if m.v_mix:
+                out[x + "vmix"] = ()
+        if getattr(m, "sink", False):
+            out[x + "sink"] = (m.heads,)
         out[x + "o"] = (H, vs)
+        gated = lambda q, ff: {q + "gate": (ff, H), q + "up": (ff, H), q + "down": (H, ff)}
         if layer.ff:
-            out.update({p + "mlp.gate": (layer.ff, H), p + "mlp.up": (layer.ff, H), p + "mlp.down": (H, layer.ff)})
+            out.update(gated(p + "mlp.", layer.ff))
+        if layer.routed:
+            for e in range(layer.routed.experts):
+                out.update(gated(f"{p}mlp.e{e}.", layer.routed.ff))
+            out[p + "mlp.router"] = (layer.routed.experts, H)
     out.update({"final.norm": (H,), "head": (cfg.vocab_size, H)})
     return out
 
 
-def _init_layer_list_tensor(name: str, shape: Tuple[int, ...], gen, device) -> torch.Tensor:
+def _init_layer_list_tensor(cfg: LayerListConfig, name: str, shape: Tuple[int, ...], gen, device) -> torch.Tensor:
     """Random values of the order a trained model has: weights of unit gain, norms near one, slow decays."""
     r = torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
     leaf = name.split(".mix.")[-1]
@@ -80,7 +103,12 @@ def _init_layer_list_tensor(name: str, shape: Tuple[int, ...], gen, device) -> t
         return r * 0.5 - 4.0
     if leaf == "a2.b":
         return r + 2.0
-    return 1.0 + 0.05 * r if ".mix." in name else 0.05 * r
+    if leaf == "vmix":
+        return 0.5 + 0.1 * r
+    if leaf == "sink":
+        return r
+    # norms of the residual stream: the sandwich block stores offsets from one
+    return 1.0 + 0.05 * r if ".mix." in name or cfg.block == "parallel" else 0.05 * r
 
 
 def param_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
@@ -139,7 +167,7 @@ def init_tensor(cfg: ModelConfig, name: str, shape: Tuple[int, ...], device="cpu
     gen = torch.Generator(device=device)
     gen.manual_seed(_name_seed(cfg.seed, name))
     if isinstance(cfg, LayerListConfig):
-        return _init_layer_list_tensor(name, shape, gen, device).to(dtype)
+        return _init_layer_list_tensor(cfg, name, shape, gen, device).to(dtype)
     t = torch.empty(shape, dtype=torch.float32 if torch.device(device).type == "cpu" else dtype, device=device)
     t.normal_(0.0, cfg.init_std, generator=gen)
     return t.to(dtype)

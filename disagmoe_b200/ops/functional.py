@@ -6,6 +6,7 @@ from __future__ import annotations
 
 import ctypes
 import math
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -96,21 +97,52 @@ def pick_attn_splits(T: int, n_kv: int, max_ctx: int, block_size: int) -> int:
 _attn_ws = {}
 
 
+# (key size, value size) of the tensor-core kernels over the paged cache: with options (window, soft cap, sink, fp32 softmax
+# weights) for query groups of any size up to 64 heads, without for equal sizes and groups of 1, 2, 4 or 8.
+ATTN_TILES = ((64, 32), (64, 64), (128, 64), (128, 128))
+
+
 def attention_on_tensor_cores(dtype, n_q: int, n_kv: int, hd: int, vd: int) -> bool:
     """Shapes of the tensor-core attention kernels; the others (and fp32) run on the CUDA cores."""
-    return dtype == torch.bfloat16 and hd == vd and hd in (64, 128) and n_q % n_kv == 0 and n_q // n_kv in (1, 2, 4, 8)
+    return dtype == torch.bfloat16 and (hd, vd) in ATTN_TILES and n_q % n_kv == 0 and n_q // n_kv <= 64
+
+
+def attention_tile(dtype, device, n_q: int, n_kv: int, hd: int, vd: int) -> Tuple[int, int]:
+    """Head sizes to keep queries / keys and values in: those of the smallest tensor-core kernel that holds them (the rest of
+    a head is zeros), or (hd, vd) where there is none."""
+    if torch.device(device).type == "cuda":
+        for k, v in ATTN_TILES:
+            if hd <= k and vd <= v and attention_on_tensor_cores(dtype, n_q, n_kv, k, v):
+                return k, v
+    return hd, vd
+
+
+def _attn_workspace(device, need: int) -> torch.Tensor:
+    key = device.index or 0
+    ws = _attn_ws.get(key)
+    if ws is None or ws.numel() < need:
+        ws = torch.empty(max(need, 1 << 22), dtype=torch.float32, device=device)
+        _attn_ws[key] = ws
+    return ws
+
+
+def _check_sink(sink, n_q: int) -> None:
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_q and sink.is_contiguous())
 
 
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
                     out: Optional[torch.Tensor] = None, splits: int = 1, scale: Optional[float] = None,
-                    window: Optional[int] = None, softcap: Optional[float] = None, fp32_weights: bool = False) -> torch.Tensor:
+                    window: Optional[int] = None, softcap: Optional[float] = None, fp32_weights: bool = False,
+                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = softmax(q[t] K^T * scale) V over the first ctx_len[t] cached tokens of block-table row bt_row[t], or the
-    last ``window`` of them; ``softcap``: scores are soft-capped, cap * tanh(score / cap). ``fp32_weights`` keeps the
-    softmax weights at fp32 accuracy in the product with V (implied by the two options before). Value heads may have
-    another size than key heads (``vcache.shape[-1]``)."""
+    last ``window`` of them; ``softcap``: scores are soft-capped, cap * tanh(score / cap); ``sink`` (fp32 [n_q]): the softmax
+    denominator has exp(sink) of the head in addition. ``fp32_weights`` keeps the softmax weights at fp32 accuracy in the
+    product with V (implied by the options before). Value heads may have another size than key heads
+    (``vcache.shape[-1]``)."""
     if not q.is_cuda:
-        o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale, window, softcap)
+        o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale, window, softcap,
+                                      sink)
         if out is not None:
             out.copy_(o)
             return out
@@ -120,34 +152,39 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     vd = vcache.shape[-1]
     if out is None:
         out = torch.empty(T, n_q * vd, dtype=q.dtype, device=q.device)
+    _check_sink(sink, n_q)
     if not attention_on_tensor_cores(q.dtype, n_q, n_kv, hd, vd):
-        assert q.dtype == kcache.dtype == vcache.dtype == out.dtype
-        _lib.check(_lib.lib().dmoe_any_attention(
-            c_int(int(q.dtype == torch.float32)), _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables),
-            c_int(block_tables.stride(0)), _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q),
-            c_int(n_kv), c_int(hd), c_int(vd), c_float(scale), c_int(window or 0), c_float(softcap or 0.0), _vp(out),
-            c_ll(out.stride(0)), _st()), "dmoe_any_attention")
-        return out
+        return _any_attention(q, hd, q.stride(0), kcache, vcache, block_tables, bt_row, None, ctx_len, T, n_q, n_kv, hd, vd,
+                              scale, window, softcap, sink, out, vd, out.stride(0))
     assert block_tables.dtype == torch.int32 and ctx_len.dtype == torch.int32 and block_tables.stride(1) == 1
-    ws = None
-    if splits > 1:
-        need = T * n_q * splits * (hd + 1)
-        key = q.device.index or 0
-        ws = _attn_ws.get(key)
-        if ws is None or ws.numel() < need:
-            ws = torch.empty(max(need, 1 << 22), dtype=torch.float32, device=q.device)
-            _attn_ws[key] = ws
-    if window or softcap or fp32_weights:
+    ws = _attn_workspace(q.device, T * n_q * splits * (vd + 1)) if splits > 1 else None
+    if window or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
         _lib.check(_lib.lib().dmoe_paged_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
-            _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_float(scale),
-            c_int(window or 0), c_float(softcap or 0.0), c_int(splits), _vp(out), c_ll(out.stride(0)), _vp(ws), _st()),
-            "dmoe_paged_attention_ext")
+            _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd),
+            c_float(scale), c_int(window or 0), c_float(softcap or 0.0), _vp(sink), c_int(splits), _vp(out),
+            c_ll(out.stride(0)), _vp(ws), _st()), "dmoe_paged_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_paged_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
         _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd),
         c_float(scale), c_int(splits), _vp(out), c_ll(out.stride(0)), _vp(ws), _st()), "dmoe_paged_attention")
+    return out
+
+
+def _any_attention(q, q_head, q_row, kcache, vcache, block_tables, bt_row, rows, ctx_len, T, n_q, n_kv, hd, vd, scale, window,
+                   softcap, sink, out, o_head, o_row):
+    """CUDA-core attention with free strides: query t of head h at q + t * q_row + h * q_head, likewise the output; the
+    cached heads of a token are contiguous, tokens ``stride(1)`` apart. Query t has the context of batch row rows[t]
+    (None: t)."""
+    assert q.dtype == kcache.dtype == vcache.dtype == out.dtype
+    assert kcache.stride(0) == kcache.shape[1] * kcache.stride(1) and vcache.stride(0) == vcache.shape[1] * vcache.stride(1)
+    _lib.check(_lib.lib().dmoe_any_attention(
+        c_int(int(q.dtype == torch.float32)), _vp(q), c_ll(q_head), c_ll(q_row), _vp(kcache), c_ll(kcache.stride(1)),
+        _vp(vcache), c_ll(vcache.stride(1)), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows),
+        _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
+        c_int(window or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(o_head), c_ll(o_row), _st()),
+        "dmoe_any_attention")
     return out
 
 
@@ -243,7 +280,8 @@ def route(x: torch.Tensor, norm_w: Optional[torch.Tensor], eps: float, gate_w: t
 
 
 class DispatchBuffers:
-    """Device buffers of the local (single GPU) expert dispatch: sorted rows, token records, offsets, scratch."""
+    """Device buffers of the local (single GPU) expert dispatch: sorted rows, token records, offsets, scratch. Rows are bf16
+    of a size that is a multiple of 16 bytes, or anything else of 2 or 4 bytes per element."""
 
     def __init__(self, capacity: int, H: int, E: int, device, dtype=torch.bfloat16):
         self.capacity, self.H, self.E = capacity, H, E
@@ -275,8 +313,14 @@ def dispatch_local(y: torch.Tensor, topk_ids: torch.Tensor, topk_w: torch.Tensor
         buf.recs[pos, 3] = topk_ids.reshape(-1)
         buf.counts.zero_()
         return
-    assert T * K <= buf.capacity
+    assert T * K <= buf.capacity and y.dtype == buf.xs.dtype
     s = scratch(y.device)
+    if y.dtype != torch.bfloat16 or buf.H % 8 or y.stride(0) % 8:
+        _lib.check(_lib.lib().dmoe_dispatch_local_any(
+            c_int(y.element_size()), _vp(y), c_ll(y.stride(0)), _vp(topk_ids), _vp(topk_w), c_int(T), c_int(K), c_int(buf.H),
+            c_int(buf.E), _vp(buf.ws), _vp(buf.offs), _vp(buf.x_bases), c_ll(buf.xs.stride(0)), _vp(buf.rec_bases),
+            c_int(buf.capacity), _vp(s.status), _st()), "dmoe_dispatch_local_any")
+        return
     _lib.check(_lib.lib().dmoe_dispatch_local(
         _vp(y), c_ll(y.stride(0)), _vp(topk_ids), _vp(topk_w), c_int(T), c_int(K), c_int(buf.H), c_int(buf.E),
         c_int(buf.E), c_int(0), _vp(buf.ws), _vp(buf.offs), _vp(buf.x_bases), c_ll(buf.xs.stride(0)),
@@ -355,8 +399,7 @@ def wait_flags(flags: torch.Tensor, n: int, epoch: torch.Tensor, status: Optiona
 # ---- tiled causal attention for prompt tokens (csrc/kernels/attention.cu: prefill_attn_kernel) -----------------------
 def prefill_tile_tokens(n_q: int, n_kv: int) -> int:
     """Prompt tokens per tile of :func:`prefill_attention` (64 query rows = tokens x query heads per kv head)."""
-    gq = n_q // n_kv
-    return 64 // gq if n_q % n_kv == 0 and gq in (1, 2, 4, 8) else 0
+    return 64 // (n_q // n_kv) if n_q % n_kv == 0 else 0
 
 
 def token_runs(bt_row, positions):
@@ -397,7 +440,7 @@ def build_prefill_tiles(bt_row, positions, tile_tokens: int, min_len: int = 8):
 def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                       tiles: torch.Tensor, n_tiles: int, n_q: int, n_kv: int, hd: int, out: torch.Tensor,
                       scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
-                      fp32_weights: bool = False) -> torch.Tensor:
+                      fp32_weights: bool = False, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the prompt tokens named by ``tiles`` (device int32 [>= n_tiles, 4], see
     :func:`build_prefill_tiles`) over the paged cache, which already holds their own K / V; writes their rows of
     ``out``. Every tile streams its sequence's K / V once (the per-token kernel streams it once per row)."""
@@ -405,11 +448,14 @@ def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
         return out
     assert q.is_cuda and tiles.is_cuda and tiles.dtype == torch.int32 and tiles.is_contiguous()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
-    if window or softcap or fp32_weights:
+    vd = vcache.shape[-1]
+    _check_sink(sink, n_q)
+    if window or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
         _lib.check(_lib.lib().dmoe_prefill_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
-            _vp(tiles), c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_float(scale),
-            c_int(window or 0), c_float(softcap or 0.0), _vp(out), c_ll(out.stride(0)), _st()), "dmoe_prefill_attention_ext")
+            _vp(tiles), c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
+            c_int(window or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()),
+            "dmoe_prefill_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_prefill_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(tiles),
@@ -454,6 +500,56 @@ def resid_norm(resid: torch.Tensor, y: Optional[torch.Tensor], post: Optional[to
     return h
 
 
+@dataclass
+class Router:
+    """Softmax router over rows that are already normalised: ``weight`` [experts, width] in the activations' dtype, the
+    ``top`` largest scores as weights (``renormalize``: divided by their sum); ``counts`` (int32 [experts]) is the histogram
+    that :func:`dispatch_local` reads and clears."""
+    weight: torch.Tensor
+    top: int
+    renormalize: bool = False
+    counts: Optional[torch.Tensor] = None
+
+    MAX_EXPERTS, MAX_TOP = 256, 32
+
+
+def sum_norm(resid: torch.Tensor, y: Optional[torch.Tensor], parts: Optional[torch.Tensor], w: torch.Tensor, eps: float,
+             dtype: torch.dtype, centred: bool, rows: Optional[torch.Tensor] = None, router: Optional[Router] = None):
+    """One step of a residual stream kept in fp32 whose sublayers share a norm: resid += y + parts.sum(1) (y [T, W], parts
+    [T, P, W] or [T, W], each may be None), then h = norm(resid) * w in ``dtype``; ``centred``: layer norm, otherwise RMS
+    norm. ``rows`` (int32) picks the rows to return; resid itself is then left as it is. Returns (h, expert ids [T, top],
+    weights [T, top]), the last two None without a ``router``, which sees h."""
+    if not resid.is_cuda:
+        h = reference.sum_norm(resid, y, parts, w, eps, dtype, centred, rows)
+        if router is None:
+            return h, None, None
+        _, ids, wts, _ = reference.route(h, None, eps, router.weight, router.top, router.renormalize)
+        if router.counts is not None:
+            router.counts += torch.bincount(ids.reshape(-1).long(), minlength=router.weight.shape[0]).int()
+        return h, ids, wts
+    n, W = (resid.shape[0] if rows is None else rows.shape[0]), resid.shape[1]
+    if parts is not None and parts.dim() == 2:
+        parts = parts.unsqueeze(1)
+    h = torch.empty(n, W, dtype=dtype, device=resid.device)
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and w.dtype == torch.float32
+    assert all(a is None or (a.dtype == dtype and a.stride(-1) == 1) for a in (y, parts)) and (rows is None or rows.dtype == torch.int32)
+    ids = wts = None
+    E = K = 0
+    if router is not None:
+        E, K = router.weight.shape[0], router.top
+        assert rows is None and router.weight.dtype == dtype and router.weight.is_contiguous()
+        ids = torch.empty(n, K, dtype=torch.int32, device=resid.device)
+        wts = torch.empty(n, K, dtype=torch.float32, device=resid.device)
+    _lib.check(_lib.lib().dmoe_sum_norm(
+        _f32(dtype), _vp(resid), _vp(y), c_ll(y.stride(0) if y is not None else 0), _vp(parts),
+        c_int(parts.shape[1] if parts is not None else 0), c_ll(parts.stride(0) if parts is not None else 0),
+        c_ll(parts.stride(1) if parts is not None else 0), _vp(w), c_int(int(centred)), c_float(eps), _vp(rows), _vp(h), c_ll(W),
+        c_int(n), c_int(W), _vp(router.weight if router else None), c_int(E), c_int(K),
+        c_int(int(bool(router and router.renormalize))), _vp(ids), _vp(wts), _vp(router.counts if router else None), _st()),
+        "dmoe_sum_norm")
+    return h, ids, wts
+
+
 def rope_frequencies(dims: int, base: float, factor: Optional[float] = None, original: float = 0.0, fast: float = 32.0,
                      slow: float = 1.0):
     """(list of dims / 2 inverse frequencies, factor on cos and sin). With ``factor``: YaRN (Peng et al., "YaRN: Efficient
@@ -496,16 +592,159 @@ def rope_freq_table(spec, max_pos: int, device) -> Optional[torch.Tensor]:
 
 def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: Optional[torch.Tensor],
                  vcache: Optional[torch.Tensor], n_q: int, n_kv: int, dk: int, dv: int, table: Optional[torch.Tensor],
-                 qw: torch.Tensor, kw: Optional[torch.Tensor], eps: float) -> None:
-    """RMS norm of every q / k head (weights fp32 [dk]) and rotation by ``table`` (:func:`rope_freq_table`, None: no
-    rotation) on rows [q | k | v]; q in place, k and v to the paged caches at ``slots``. n_kv = 0: q only (a layer that
-    reads another layer's cache)."""
+                 qw: Optional[torch.Tensor], kw: Optional[torch.Tensor], eps: float, interleaved: bool = False,
+                 v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0) -> None:
+    """RMS norm of every q / k head (weights fp32 [dk]; None: no norm) and rotation by ``table`` (:func:`rope_freq_table`,
+    None: no rotation; ``interleaved``: of neighbouring dimensions) on rows [q | k | v]; q in place, k and v to the paged
+    caches at ``slots``. n_kv = 0: q only (a layer that reads another layer's cache). ``v_first`` [T, n_kv, >= dv]: the
+    values become (1 - v_lambda) v + v_lambda v_first on their way to the cache."""
     if not qkv.is_cuda:
-        return reference.qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps)
+        return reference.qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps,
+                                      interleaved, v_first, v_lambda)
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and qkv.stride(1) == 1
     assert n_kv == 0 or (kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == qkv.dtype)
     rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
     _lib.check(_lib.lib().dmoe_qk_norm_rope(
         _f32(qkv.dtype), _vp(qkv), c_ll(qkv.stride(0)), _vp(positions), _vp(slots), _vp(kcache), _vp(vcache),
-        c_int(qkv.shape[0]), c_int(n_q), c_int(n_kv), c_int(dk), c_int(dv), c_int(rot), _vp(table), c_int(max_pos), _vp(qw),
-        _vp(kw), c_float(eps), _st()), "dmoe_qk_norm_rope")
+        c_int(qkv.shape[0]), c_int(n_q), c_int(n_kv), c_int(dk), c_int(dv), c_int(rot), c_int(int(interleaved)), _vp(table),
+        c_int(max_pos), _vp(qw), _vp(kw), c_float(eps), _vp(v_first), c_ll(v_first.stride(0) if v_first is not None else 0),
+        c_int(v_first.stride(1) if v_first is not None else 0), c_float(v_lambda), _st()), "dmoe_qk_norm_rope")
+
+
+# ---- latent attention (csrc/kernels/latent_attention.cu) ---------------------------------------------------------------
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class LatentLayout:
+    """Sizes of a latent attention layer as its kernels see them: every part of a row is padded to a multiple of 8 (zeros).
+
+    projection row   [heads x (q unrotated | q rotated) | latent | rotated key part]
+    cache row        [latent | rotated key part]
+    """
+    heads: int
+    dim: int
+    rot: int
+    vdim: int
+    rank: int
+
+    @property
+    def dimp(self) -> int:
+        return _pad8(self.dim)
+
+    @property
+    def rotp(self) -> int:
+        return _pad8(self.rot)
+
+    @property
+    def vdimp(self) -> int:
+        return _pad8(self.vdim)
+
+    @property
+    def rankp(self) -> int:
+        return _pad8(self.rank)
+
+    @property
+    def qd(self) -> int:
+        return self.dimp + self.rotp
+
+    @property
+    def row(self) -> int:
+        return self.rankp + self.rotp
+
+    def min_run(self) -> int:
+        """Prompt tokens from which expanding the latents of all visible keys pays: it costs rank * (dim + vdim) per key and
+        head once, and saves 2 rank + rot - (dim + rot + vdim) per key, head and query."""
+        saves = max(1, 2 * self.rank + self.rot - (self.dim + self.rot + self.vdim))
+        return min(128, max(16, self.rank * (self.dim + self.vdim) // saves))
+
+    def tiled(self, dtype) -> bool:
+        """Is there a prompt kernel for these head sizes?"""
+        return dtype == torch.bfloat16 and any(self.qd <= k and self.vdimp <= v for k, v in LATENT_TILES)
+
+
+LATENT_TILES = ((96, 64), (128, 128), (192, 128))     # (key, value) sizes of the prompt kernel
+LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 640            # of the tensor-core kernel over the latent cache
+
+
+def latent_prep(y: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, lay: LatentLayout,
+                table: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float, loose: Optional[torch.Tensor], n_loose: int,
+                interleaved: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
+    """From projection rows y (:class:`LatentLayout`): RMS norm of the latent (weight fp32 [rank]), rotation of the shared
+    key part, both to the paged ``cache`` [blocks, block_size, row] at ``slots``; rotation of the queries, in place. Rows with
+    loose[t] = i >= 0 (None: row t is i = t) are attended over the latents themselves, so their queries are also written
+    head by head: returns (unrotated part [heads, n_loose, dimp], [heads, n_loose, row] with the rotated part in place and
+    the latent part still to be filled)."""
+    if not y.is_cuda:
+        return reference.latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved)
+    assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and y.stride(1) == 1 and cache.is_contiguous()
+    assert y.shape[1] == lay.heads * lay.qd + lay.row and cache.dtype == y.dtype and norm_w.dtype == torch.float32
+    xq = torch.empty(lay.heads, n_loose, lay.dimp, dtype=y.dtype, device=y.device)
+    qa = torch.empty(lay.heads, n_loose, lay.row, dtype=y.dtype, device=y.device)
+    rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
+    _lib.check(_lib.lib().dmoe_latent_prep(
+        _f32(y.dtype), _vp(y), c_ll(y.stride(0)), _vp(positions), _vp(slots), _vp(cache), c_int(y.shape[0]), c_int(lay.heads),
+        c_int(lay.dim), c_int(lay.rot), c_int(lay.rank), c_int(rot), c_int(int(interleaved)), _vp(table), c_int(max_pos),
+        _vp(norm_w), c_float(eps), _vp(loose), c_int(n_loose), _vp(xq), _vp(qa), _st()), "dmoe_latent_prep")
+    return xq, qa
+
+
+def latent_attention(qa: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, bt_row: torch.Tensor,
+                     ctx_len: torch.Tensor, rows: Optional[torch.Tensor], lay: LatentLayout, scale: float,
+                     window: Optional[int] = None, sink: Optional[torch.Tensor] = None, max_ctx: int = 1 << 30) -> torch.Tensor:
+    """Attention over the cached latents: queries qa [heads, n, row] (latent part already multiplied by the key map), values
+    are the latents. Query i belongs to batch row rows[i] (None: i). Returns [heads, n, rankp]."""
+    H, n, row = qa.shape
+    k3 = cache.unsqueeze(2)
+    if not qa.is_cuda:
+        idx = slice(None) if rows is None else rows.long()
+        o = reference.paged_attention(qa.transpose(0, 1).reshape(n, H * row), k3, k3[..., :lay.rankp], block_tables,
+                                      bt_row[idx], ctx_len[idx], H, 1, row, scale, window, None, sink)
+        return o.view(n, H, lay.rankp).transpose(0, 1).contiguous()
+    out = torch.empty(H, n, lay.rankp, dtype=qa.dtype, device=qa.device)
+    _check_sink(sink, H)
+    if qa.dtype == torch.float32 or lay.rankp > LATENT_MAX_RANK or lay.row > LATENT_MAX_ROW:
+        return _any_attention(qa, n * row, row, k3, k3[..., :lay.rankp], block_tables, bt_row, rows, ctx_len, n, H, 1, row,
+                              lay.rankp, scale, window, None, sink, out, n * lay.rankp, lay.rankp)
+    reach = min(max_ctx, window or max_ctx)
+    splits = pick_latent_splits(n, H, reach)
+    ws = _attn_workspace(qa.device, H * n * splits * (lay.rankp + 1)) if splits > 1 else None
+    _lib.check(_lib.lib().dmoe_latent_attention(
+        _vp(qa), _vp(cache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows), _vp(ctx_len),
+        c_int(cache.shape[1]), c_int(n), c_int(H), c_int(lay.rankp), c_int(row), c_float(scale), c_int(window or 0), _vp(sink),
+        c_int(splits), _vp(out), _vp(ws), _st()), "dmoe_latent_attention")
+    return out
+
+
+def pick_latent_splits(n: int, heads: int, reach: int) -> int:
+    """Key ranges per (query token, group of up to 32 heads) of :func:`latent_attention`: enough CTAs for all SMs, never
+    fewer than 128 keys each."""
+    from .gemm import num_sms
+    sms, ctas = num_sms(), max(1, n * ((heads + 31) // 32))
+    return max(1, min((2 * sms + ctas - 1) // ctas, (reach + 127) // 128, 64)) if ctas < 2 * sms else 1
+
+
+def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, keys: torch.Tensor, n_keys: int) -> torch.Tensor:
+    """Rows [n_keys, row] of the cached tokens named by ``keys`` (int32 [>= n_keys, 2] = block-table row, position)."""
+    out = torch.empty(n_keys, cache.shape[2], dtype=cache.dtype, device=cache.device)
+    assert keys.dtype == torch.int32 and keys.is_contiguous() and cache.shape[2] % 8 == 0 and cache.dtype == torch.bfloat16
+    _lib.check(_lib.lib().dmoe_latent_gather(_vp(cache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(keys),
+                                             c_int(n_keys), c_int(cache.shape[1]), c_int(cache.shape[2]), _vp(out), _st()),
+               "dmoe_latent_gather")
+    return out
+
+
+def latent_prefill(q: torch.Tensor, kv: torch.Tensor, lat: torch.Tensor, tiles: torch.Tensor, base: torch.Tensor, n_tiles: int,
+                   lay: LatentLayout, scale: float, window: Optional[int], sink: Optional[torch.Tensor],
+                   out: torch.Tensor) -> torch.Tensor:
+    """Causal attention of the prompt tokens named by ``tiles`` over expanded keys and values: kv [keys, heads x (key
+    unrotated | value)], rotated key parts in the gathered cache rows ``lat`` [keys, row]; the key at position p of tile i's
+    sequence is row base[i] + p. q: projection rows with rotated queries. Writes the tokens' rows of out [T, heads x vdimp]."""
+    _check_sink(sink, lay.heads)
+    assert tiles.dtype == base.dtype == torch.int32 and kv.stride(1) == lat.stride(1) == 1
+    _lib.check(_lib.lib().dmoe_latent_prefill(
+        _vp(q), c_ll(q.stride(0)), _vp(kv), c_ll(kv.stride(0)), _vp(lat), c_ll(lat.stride(0)), _vp(tiles), _vp(base),
+        c_int(n_tiles), c_int(lay.heads), c_int(lay.dimp), c_int(lay.rotp), c_int(lay.rankp), c_int(lay.vdimp), c_float(scale),
+        c_int(window or 0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()), "dmoe_latent_prefill")
+    return out

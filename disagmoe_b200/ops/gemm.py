@@ -2,6 +2,7 @@
 
 ``linear``          y = x @ w.T (+ residual)                         -- reference: disagmoe/models/linear.py:131-136
 ``grouped_swiglu``  act = silu(x @ w13[g][:I].T) * (x @ w13[g][I:].T)   -- reference: disagmoe/models/experts.py:84-88
+                    (or the tanh form of gelu in place of silu)
 ``grouped_linear``  y = x @ w2[g].T per expert group                   -- reference: disagmoe/models/experts.py:89
 ``grouped_combine`` the same GEMM whose epilogue scales each row by its router weight and scatters it to the
                     row (and GPU) it came from                         -- reference: disagmoe/frontend/engine.py:731-734
@@ -17,8 +18,9 @@ from typing import Optional
 
 import torch
 
-from . import _lib
+from . import _lib, reference
 
+ACTS = {"silu": 0, "gelu_tanh": 1}
 EPI_PLAIN, EPI_SWIGLU, EPI_COMBINE = 0, 1, 2
 STREAM_K = True      # default work distribution of every GEMM launched without an explicit split (tests may turn it off)
 TRACE = None         # profiling aid: an int64 [8] CUDA tensor that CTA 0 of every launch fills with nanosecond stamps
@@ -210,10 +212,10 @@ def rope_table(max_pos: int, hd: int, theta: float, device) -> torch.Tensor:
 
 
 def _launch(W, X, Y, R, offs, recs, bases, G, T, F, K, epi, bn, splitk, ldy, y_f32, comm: Optional[GemmComm] = None,
-            streamk: bool = False, pair: bool = False, w_blocked: bool = False):
+            streamk: bool = False, pair: bool = False, w_blocked: bool = False, act: str = "silu"):
     s = scratch(X.device)
     d = _lib.DmoeGemm()
-    d.w_blocked = int(w_blocked)
+    d.w_blocked, d.act = int(w_blocked), ACTS[act]
     d.trace = TRACE.data_ptr() if TRACE is not None else None
     d.streamk, d.n_counters = int(streamk and splitk <= 1 and not pair), s.counters.numel()
     d.pair = int(pair)
@@ -253,6 +255,30 @@ def _simt_linear(x, w, out, out_dtype):
     _lib.check(_lib.lib().dmoe_simt_linear(
         i(int(f32)), i(int(out.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), ll(K),
         v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), v(_lib.stream_ptr())), "dmoe_simt_linear")
+    return out
+
+
+def _simt_grouped(x, w, offs, out, recs=None, base=None, ld_out=0):
+    """The CUDA-core GEMM over row groups: rows offs[g] .. offs[g + 1] of x times w[g].T, into ``out`` or, with ``recs``
+    (combine), scaled and scattered to rows of the buffer at ``base[0]`` in x's dtype."""
+    T, K = x.shape
+    G, F, _ = w.shape
+    assert w.is_contiguous() and w.dtype == x.dtype and w.shape[2] == K and x.stride(1) == 1
+    assert offs.dtype == torch.int32 and (out is None or out.dtype == x.dtype)
+    v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+    _lib.check(_lib.lib().dmoe_simt_grouped(
+        i(int(x.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), v(offs.data_ptr()), i(G),
+        v(_lib.ptr(out)), ll(out.stride(0) if out is not None else ld_out), v(_lib.ptr(recs)), v(_lib.ptr(base)), i(T), i(F),
+        i(K), v(_lib.stream_ptr())), "dmoe_simt_grouped")
+    return out
+
+
+def _gate_mul(gu, out, I: int, act: str):
+    """out = act(gu[:, :I]) * gu[:, I:]"""
+    v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+    _lib.check(_lib.lib().dmoe_gate_mul(i(int(gu.dtype == torch.float32)), i(ACTS[act]), v(gu.data_ptr()), ll(gu.stride(0)),
+                                        v(out.data_ptr()), ll(out.stride(0)), i(gu.shape[0]), i(I), v(_lib.stream_ptr())),
+               "dmoe_gate_mul")
     return out
 
 
@@ -312,7 +338,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
     return out
 
 
-def _grouped_ref(x, w, offs, swiglu):
+def _grouped_ref(x, w, offs, swiglu, act="silu"):
     offs = offs.tolist()
     G = w.shape[0]
     F = w.shape[1] // 2 if swiglu else w.shape[1]
@@ -323,24 +349,27 @@ def _grouped_ref(x, w, offs, swiglu):
             continue
         h = x[a:b].float() @ w[g].float().T
         if swiglu:
-            h = torch.nn.functional.silu(h[:, :F]) * h[:, F:]
+            h = reference.swiglu(h, act)
         y[a:b] = h
     return y
 
 
 def grouped_swiglu(x: torch.Tensor, w13: torch.Tensor, offs: Optional[torch.Tensor], out: Optional[torch.Tensor] = None,
                    bn: int = 0, comm: Optional[GemmComm] = None, streamk: Optional[bool] = None,
-                   pair: bool = False, w_blocked: bool = False) -> torch.Tensor:
-    """act[T, I] = silu(x @ w13[g, :I].T) * (x @ w13[g, I:].T) for the rows of group g; w13 is [G, 2I, K]."""
+                   pair: bool = False, w_blocked: bool = False, act: str = "silu") -> torch.Tensor:
+    """y[T, I] = act(x @ w13[g, :I].T) * (x @ w13[g, I:].T) for the rows of group g; w13 is [G, 2I, K]."""
     T, K = x.shape
     G, F2, _ = w13.shape
     I = F2 // 2
     if not x.is_cuda:
-        y = _grouped_ref(x, w13, offs, True).to(x.dtype)
+        y = _grouped_ref(x, w13, offs, True, act).to(x.dtype)
         if out is not None:
             out.copy_(y)
             return out
         return y
+    if x.dtype == torch.float32 or (comm is None and not w_blocked and not _tma_ok(x, w13)):
+        gu = _simt_grouped(x, w13, offs, torch.empty(T, F2, dtype=x.dtype, device=x.device))
+        return _gate_mul(gu, torch.empty(T, I, dtype=x.dtype, device=x.device) if out is None else out, I, act)
     _check_x(x)
     assert w13.is_contiguous() and w13.dtype == torch.bfloat16
     assert comm is not None or (offs.dtype == torch.int32 and offs.is_cuda)
@@ -353,7 +382,7 @@ def grouped_swiglu(x: torch.Tensor, w13: torch.Tensor, offs: Optional[torch.Tens
         bn = max(bn, 128)
     sk = want_streamk(EPI_SWIGLU, I, G, T, bn, num_sms(x.device)) if streamk is None else streamk
     _launch(w13, x, out, None, offs, None, None, G, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False, comm,
-            streamk=sk, pair=pair, w_blocked=w_blocked)
+            streamk=sk, pair=pair, w_blocked=w_blocked, act=act)
     return out
 
 
@@ -369,6 +398,8 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, out: Op
             out.copy_(y)
             return out
         return y
+    if x.dtype == torch.float32 or (not w_blocked and not _tma_ok(x, w)):
+        return _simt_grouped(x, w, offs, torch.empty(T, F, dtype=x.dtype, device=x.device) if out is None else out)
     _check_x(x)
     assert w.is_contiguous() and w.dtype == torch.bfloat16 and offs.dtype == torch.int32 and offs.is_cuda
     if out is None:
@@ -431,12 +462,13 @@ def grouped_combine(x: torch.Tensor, w: torch.Tensor, offs: Optional[torch.Tenso
     T, K = x.shape
     G, F, _ = w.shape
     if not x.is_cuda:
-        y = _grouped_ref(x, w, offs, False)
-        wts = recs[:, 2].contiguous().view(torch.float32)
-        for t in range(T):
-            r, row = int(recs[t, 0]), int(recs[t, 1])
-            if row >= 0:
-                outs[r][row] = (y[t] * wts[t]).to(outs[r].dtype)
+        y = _grouped_ref(x, w, offs, False) * recs[:, 2].contiguous().view(torch.float32)[:, None]
+        for r, o in enumerate(outs):
+            mine = (recs[:, 0] == r) & (recs[:, 1] >= 0)
+            o[recs[mine, 1].long()] = y[mine].to(o.dtype)
+        return
+    if x.dtype == torch.float32 or (comm is None and not w_blocked and not _tma_ok(x, w)):
+        _simt_grouped(x, w, offs, None, recs, bases, ld_out)
         return
     _check_x(x)
     assert recs.dtype == torch.int32 and recs.is_contiguous() and recs.shape[1] == 4 and bases.dtype == torch.int64
@@ -450,26 +482,20 @@ def grouped_combine(x: torch.Tensor, w: torch.Tensor, offs: Optional[torch.Tenso
             pair=pair, w_blocked=w_blocked)
 
 
-def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor] = None, bn: int = 0) -> torch.Tensor:
-    """Dense SwiGLU up-projection: silu(x @ w13[:I].T) * (x @ w13[I:].T); w13 is [2I, K] (a one-group grouped_swiglu)."""
+def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor] = None, bn: int = 0,
+                  act: str = "silu") -> torch.Tensor:
+    """Dense gated up-projection: act(x @ w13[:I].T) * (x @ w13[I:].T); w13 is [2I, K] (a one-group grouped_swiglu)."""
     T, K = x.shape
     I = w13.shape[0] // 2
     if not x.is_cuda:
-        h = x.float() @ w13.float().T
-        y = (torch.nn.functional.silu(h[:, :I]) * h[:, I:]).to(x.dtype)
+        y = reference.swiglu(x.float() @ w13.float().T, act).to(x.dtype)
         if out is not None:
             out.copy_(y)
             return out
         return y
     if x.dtype == torch.float32 or not _tma_ok(x, w13):
         gu = _simt_linear(x, w13, None, None)
-        if out is None:
-            out = torch.empty(T, I, dtype=x.dtype, device=x.device)
-        v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
-        _lib.check(_lib.lib().dmoe_silu_mul(i(int(x.dtype == torch.float32)), v(gu.data_ptr()), ll(gu.stride(0)),
-                                            v(out.data_ptr()), ll(out.stride(0)), i(T), i(I), v(_lib.stream_ptr())),
-                   "dmoe_silu_mul")
-        return out
+        return _gate_mul(gu, torch.empty(T, I, dtype=x.dtype, device=x.device) if out is None else out, I, act)
     _check_x(x)
     assert w13.is_contiguous() and w13.dtype == torch.bfloat16
     if out is None:
@@ -477,5 +503,6 @@ def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor
     if T == 0:
         return out
     bn = bn or pick_bn(T, EPI_SWIGLU)
-    _launch(w13, x, out, None, None, None, None, 1, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False)
+    _launch(w13, x, out, None, None, None, None, 1, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False,
+            act=act)
     return out

@@ -58,10 +58,11 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slots: Optional[t
 
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
-                    scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None
-                    ) -> torch.Tensor:
+                    scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
+                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Token t attends to the first ctx_len[t] cached tokens of block-table row bt_row[t] (default t), or to the last
-    ``window`` of them; ``softcap``: scores become cap * tanh(score / cap)."""
+    ``window`` of them; ``softcap``: scores become cap * tanh(score / cap); ``sink`` [n_q]: the softmax denominator has
+    exp(sink) in addition."""
     T = q.shape[0]
     block_size = kcache.shape[1]
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
@@ -83,7 +84,9 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         s = torch.einsum("kgd,lkd->kgl", qt, k) * scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
-        p = torch.softmax(s, dim=-1)
+        if sink is not None:
+            s = torch.cat([s, sink.view(n_kv, gq, 1).to(s.dtype)], -1)
+        p = torch.softmax(s, dim=-1)[..., :k.shape[0]]
         o = torch.einsum("kgl,lkd->kgd", p, v)
         out[t] = o.reshape(-1)
     return out.to(q.dtype)
@@ -120,9 +123,11 @@ def sort_by_expert(topk_ids: torch.Tensor) -> torch.Tensor:
     return pos.int()
 
 
-def swiglu(h: torch.Tensor) -> torch.Tensor:
+def swiglu(h: torch.Tensor, act: str = "silu") -> torch.Tensor:
     I = h.shape[-1] // 2
-    return torch.nn.functional.silu(h[..., :I].float()) * h[..., I:].float()
+    g = h[..., :I].float()
+    g = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+    return g * h[..., I:].float()
 
 
 def moe_experts(y: torch.Tensor, topk_ids: torch.Tensor, topk_w: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor
@@ -175,18 +180,43 @@ def resid_norm(resid, y, post, pre, eps, dtype, out_scale=1.0, rows=None):
     return None if pre is None else (_rms_scale(x, eps) * pre * out_scale).to(dtype)
 
 
-def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps) -> None:
-    """Per-head norm + partial rotation of q (in place) and k, K / V append at slots >= 0."""
+def sum_norm(resid, y, parts, w, eps, dtype, centred, rows=None):
+    """resid += y + parts.sum(1) (either may be None; ``rows``: only these rows are returned, resid untouched); returns the
+    RMS norm of resid times w, or with ``centred`` its layer norm (mean taken off) times w."""
+    x = resid if rows is None else resid[rows.long()]
+    for a in (y, parts):
+        if a is not None:
+            a = a if rows is None else a[rows.long()]
+            x = x + (a.float() if a.dim() == 2 else a.float().sum(1))
+    if rows is None:
+        resid.copy_(x)
+    if centred:
+        x = x - x.mean(-1, keepdim=True)
+    return (_rms_scale(x, eps) * w).to(dtype)
+
+
+def _turn(x, table, positions, interleaved):
+    """Rotation of the leading dimensions of x [T, heads, d] by (cos, sin) rows of ``table``."""
+    if table is None:
+        return x
+    rot = 2 * table.shape[1]
+    c, s = (table[positions.long()][:, None, :, j] for j in (0, 1))
+    if interleaved:
+        u, v = x[..., 0:rot:2], x[..., 1:rot:2]
+        return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., rot:]], -1)
+    u, v = x[..., :rot // 2], x[..., rot // 2:rot]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., rot:]], -1)
+
+
+def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps, interleaved=False,
+                 v_first=None, v_lambda=0.0) -> None:
+    """Per-head norm (where weights are given) + partial rotation of q (in place) and k, K / V append at slots >= 0; with
+    ``v_first`` [T, n_kv, >= dv] the values appended are (1 - v_lambda) v + v_lambda v_first."""
     T = qkv.shape[0]
 
     def turn(x, w):
-        x = _rms_scale(x.float(), eps) * w
-        if table is None:
-            return x
-        half = table.shape[1]
-        c, s = (table[positions.long()][:, None, :, j] for j in (0, 1))
-        u, v = x[..., :half], x[..., half:2 * half]
-        return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
+        x = x.float() if w is None else _rms_scale(x.float(), eps) * w
+        return _turn(x, table, positions, interleaved)
 
     qs, ks = n_q * dk, n_kv * dk
     q = turn(qkv[:, :qs].reshape(T, n_q, dk), qw).to(qkv.dtype)
@@ -194,8 +224,32 @@ def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table
         k = turn(qkv[:, qs:qs + ks].reshape(T, n_kv, dk), kw).to(qkv.dtype)
         ok = slots >= 0
         kcache.view(-1, n_kv, dk)[slots[ok]] = k[ok]
-        vcache.view(-1, n_kv, dv)[slots[ok]] = qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
+        v = qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
+        if v_first is not None:
+            v = ((1.0 - v_lambda) * v.float() + v_lambda * v_first[ok][..., :dv].float()).to(v.dtype)
+        vcache.view(-1, n_kv, dv)[slots[ok]] = v
     qkv[:, :qs] = q.reshape(T, qs)
+
+
+def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved):
+    """See :func:`disagmoe_b200.ops.functional.latent_prep`."""
+    T, H = y.shape[0], lay.heads
+    q = y[:, :H * lay.qd].reshape(T, H, lay.qd)
+    d = y[:, H * lay.qd:]
+    c = (_rms_scale(d[:, :lay.rank].float(), eps) * norm_w).to(y.dtype)
+    kr = _turn(d[:, None, lay.rank:lay.rank + lay.rot].float(), table, positions, interleaved)[:, 0].to(y.dtype)
+    ok = slots >= 0
+    flat = cache.view(-1, lay.row)
+    flat[slots[ok], :lay.rank] = c[ok]
+    flat[slots[ok], lay.rankp:lay.rankp + lay.rot] = kr[ok]
+    qr = _turn(q[..., lay.dimp:lay.dimp + lay.rot].float(), table, positions, interleaved).to(y.dtype)
+    xq, qa = y.new_zeros(H, n_loose, lay.dimp), y.new_zeros(H, n_loose, lay.row)
+    idx = torch.arange(T) if loose is None else loose.long()
+    on = idx >= 0
+    xq[:, idx[on]] = q[on][..., :lay.dimp].transpose(0, 1)
+    qa[:, idx[on], lay.rankp:lay.rankp + lay.rot] = qr[on].transpose(0, 1)
+    y[:, :H * lay.qd] = torch.cat([q[..., :lay.dimp], qr, q[..., lay.dimp + lay.rot:]], -1).reshape(T, -1)
+    return xq, qa
 
 
 # ---- linear recurrences ----------------------------------------------------------------------------------------------
