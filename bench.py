@@ -146,9 +146,9 @@ def main():
                          "continuous batching; prints output tokens/s with p50 / p99 time per output token per rate")
     ap.add_argument("--rates", default="2,8,16,32")
     ap.add_argument("--duration", type=float, default=60.0)
-    ap.add_argument("--layer-list", action="store_true",
-                    help="1 GPU: prefill and decode throughput of layer-list decoders beside a dense decoder of equal size "
-                         "(benchmark/layer_list.py) instead of the headline workload")
+    ap.add_argument("--layer-list", nargs="?", const="rurunex", choices=["rurunex", "supinex"],
+                    help="1 GPU: prefill and decode throughput of layer-list decoders of this design beside the closest "
+                         "decoder of equal size (benchmark/layer_list.py) instead of the headline workload")
     ap.add_argument("--layer-list-sizes", default="", help="comma-separated widths for --layer-list")
     args = ap.parse_args()
     if args.layer_list:
@@ -182,7 +182,7 @@ def main():
     K = args.steps
     cfg = get_preset(args.model)
     if isinstance(cfg, LayerListConfig):
-        raise SystemExit(f"{cfg.name} is not an MoE model: use --layer-list")
+        raise SystemExit(f"{cfg.name} is a layer-list decoder: use --layer-list")
     if args.layers:
         cfg = cfg.clone(num_layers=args.layers)
     cfg.max_seq_len = max(4096, (args.ctx_max + K + W + args.timeline + 2 + 15) // 16 * 16)

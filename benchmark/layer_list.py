@@ -1,12 +1,15 @@
-"""Prefill and decode throughput of layer-list decoders (Rurunex design) beside a dense decoder of equal size.
+"""Prefill and decode throughput of layer-list decoders beside the closest decoder of the package at equal size.
 
-    python bench.py --layer-list [--steps K --warmup W]
+    python bench.py --layer-list [rurunex | supinex] [--steps K --warmup W]
 
-Both run through the same engine classes with random weights: the layer-list model repeats (gated linear attention,
-channel-wise delta rule, windowed attention), every layer with a gated feed-forward; the dense model is the MoE decoder
-with a dense feed-forward in every layer, full attention, the same width, heads, feed-forward and number of layers.
-Prints one JSON line per (size, phase, model): tokens/s from device-timed steps (CUDA events, inputs larger than L2 for
-the larger sizes, L2 flushed between steps otherwise), and one per (size, phase) with the device time per kernel.
+Both run through the same engine classes with random weights.
+  rurunex  repeats (gated linear attention, channel-wise delta rule, windowed attention), every layer with a gated
+           feed-forward; beside the MoE decoder with a dense feed-forward in every layer and full attention: same width, heads,
+           feed-forward and number of layers
+  supinex  repeats (attention over everything, windowed latent attention), experts in every layer but the first; beside the MoE
+           decoder with the same width, heads, experts and number of layers
+Prints one JSON line per (size, phase, model): tokens/s from device-timed steps (CUDA events, L2 flushed between steps), and
+one per (size, phase) with the device time per kernel.
 """
 from __future__ import annotations
 
@@ -16,13 +19,16 @@ from typing import Dict, List
 
 import torch
 
-from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, LayerListConfig, LayerSpec,
-                                  ModelConfig, RotarySpec)
+from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec,
+                                  LayerListConfig, LayerSpec, ModelConfig, RotarySpec, RoutedSpec)
 from disagmoe_b200.frontend.colocated import ColocatedEngine
 from disagmoe_b200.ops import _lib, gemm
 
 # name: width, heads, kv heads, head size, feed-forward, layers
 SIZES = {"1024": (1024, 8, 2, 128, 2816, 6), "2048": (2048, 16, 4, 128, 5632, 6), "4096": (4096, 32, 8, 128, 11264, 6)}
+# the same, then: latent rank, experts, experts per token (the feed-forward is an expert's; the dense first layer has 4 of them)
+MOE_SIZES = {"1024": (1024, 8, 2, 128, 768, 6, 256, 32, 4), "2048": (2048, 16, 4, 128, 1408, 6, 512, 64, 6),
+             "4096": (4096, 32, 8, 128, 4096, 6, 512, 16, 2)}
 VOCAB = 32000
 
 
@@ -43,6 +49,24 @@ def dense_config(size: str, max_seq_len: int = 8192) -> ModelConfig:
                        first_k_dense=n, dense_intermediate_size=ff, max_seq_len=max_seq_len, name="dense-" + size)
 
 
+def parallel_config(size: str, window: int = 1024, max_seq_len: int = 8192) -> LayerListConfig:
+    W, H, G, D, ff, n, rank, E, K = MOE_SIZES[size]
+    attn = AttentionSpec(H, G, D, D, D ** -0.5, RotarySpec(D, 5e5, interleaved=True), qk_norm=False, sink=True, v_mix=True)
+    lat = LatentAttentionSpec(H, D, D // 2, D, rank, (D + D // 2) ** -0.5, window=window, sink=True,
+                              rot=RotarySpec(D // 2, 1e6, 4.0, 8192, interleaved=True))
+    moe = RoutedSpec(E, K, ff)
+    layers = [LayerSpec(attn if i % 2 == 0 else lat, routed=moe) if i else LayerSpec(attn, 4 * ff, "gelu_tanh") for i in range(n)]
+    return LayerListConfig.make(W, VOCAB, layers, max_seq_len=max_seq_len, block="parallel", name="supinex-" + size)
+
+
+def moe_config(size: str, max_seq_len: int = 8192) -> ModelConfig:
+    W, H, G, D, ff, n, _, E, K = MOE_SIZES[size]
+    return ModelConfig(hidden_size=W, num_layers=n, num_heads=H, num_kv_heads=G, num_experts=E, intermediate_size=ff,
+                       dtype=torch.bfloat16, ep_size=1, top_k=K, vocab_size=VOCAB, head_dim=D, rope_theta=5e5,
+                       norm_topk_prob=False, first_k_dense=1, dense_intermediate_size=4 * ff, max_seq_len=max_seq_len,
+                       name="moe-" + size)
+
+
 def make_engine(cfg, batch: int, prompt_tokens: int, ctx: int, steps: int) -> ColocatedEngine:
     blocks = max(batch * ((ctx + steps + 32) // 16 + 1), prompt_tokens // 16 + 64)
     eng = ColocatedEngine(cfg, CacheConfig(block_size=16), device="cuda", max_batch_size=batch,
@@ -51,8 +75,8 @@ def make_engine(cfg, batch: int, prompt_tokens: int, ctx: int, steps: int) -> Co
     if hasattr(ex, "kv_cache"):
         ex.kv_cache.normal_(0, 0.5)
     else:
-        for k, v in ex.kv.values():
-            k.normal_(0, 0.5), v.normal_(0, 0.5)
+        for t in (t for kv in ex.kv.values() for t in kv):
+            t.normal_(0, 0.5)
         for s in ex.states.values():
             s.S.normal_(0, 0.1)
     ex.capture([batch])
@@ -106,7 +130,8 @@ def main(args) -> int:
     flush = Flush()
     for size in (args.layer_list_sizes or "1024,2048,4096").split(","):
         for phase, n, length in (("prefill", 1, 4096), ("prefill", 4, 2048), ("decode", 16, 2048), ("decode", 256, 1024)):
-            for cfg in (hybrid_config(size), dense_config(size)):
+            for cfg in (hybrid_config(size), dense_config(size)) if args.layer_list == "rurunex" else \
+                    (parallel_config(size), moe_config(size)):
                 B = n if phase == "decode" else 8
                 eng = make_engine(cfg, B, n * length if phase == "prefill" else B, length if phase == "decode" else 16, 8)
                 ex = eng.executor

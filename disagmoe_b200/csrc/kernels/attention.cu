@@ -51,12 +51,24 @@ __device__ __forceinline__ void cp_async16_stream(uint32_t dst, const void* src,
 }
 // Options of the EXT instantiations of both kernels (plain ones compile without them):
 //   window > 0: a query at position p sees only keys in (p - window, p];
-//   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap).
+//   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap);
+//   sink != NULL: exp(sink[head]) enters the softmax denominator (no key, no value);
+//   gq: query heads per kv head where the instantiation leaves it open (GQ = 0).
 // The EXT kernels also keep the softmax weights at fp32 accuracy in the P V product: P = hi + lo, both bf16, two MMAs.
 struct AttnExt {
   int window;
   float cap_in, cap_log2;
+  const float* sink;
+  int gq;
 };
+constexpr float kLog2e = 1.4426950408889634f;
+// 16-byte chunk c of tile row r in shared memory: rows of 128 bytes and more permute their chunks by groups of eight, rows of
+// 64 bytes (two to a 128-byte line) by groups of four; either way eight rows of one column meet no bank twice.
+template <int NCH>
+__device__ __forceinline__ int swz(int c, int r) {
+  static_assert(NCH == 4 || NCH % 8 == 0, "row size");
+  return NCH == 4 ? c ^ ((r >> 1) & 3) : c ^ (r & 7);
+}
 // raw q.k -> score in base-2 units. tanh(x) = 1 - 2 / (exp(2x) + 1), good to ~1e-7 absolute.
 template <bool EXT>
 __device__ __forceinline__ float attn_score(float raw, float scale_log2, const AttnExt& x) {
@@ -72,7 +84,8 @@ constexpr int kAttnWarps = kAttnThreads / 32;
 // Each warp owns every 4th chunk of 16 cached tokens and streams them through its private cp.async ring
 // (swizzled so that ldmatrix is bank-conflict free): S = Q K^T (2 n-tiles), online softmax on the accumulator
 // fragments, P re-used in place as the A operand of O += P V (V read with ldmatrix.trans).
-template <int HD, int GQ, bool EXT>
+// VD: value size. GQ = 0: groups of ext.gq heads, at most 8 of which go to one CTA.
+template <int HD, int VD, int GQ, bool EXT>
 __global__ void __launch_bounds__(kAttnThreads)
 paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ kcache,
                   const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_blocks,
@@ -80,24 +93,27 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
                   float scale_log2, int splits, __nv_bfloat16* __restrict__ out, long long ld_out,
                   float* __restrict__ part_o, float* __restrict__ part_lse, AttnExt ext) {
   static_assert(GQ <= 8, "the query group must fit the first 8 rows of the MMA tile");
-  constexpr int ROWB = HD * 2;                       // bytes of one cached row of one kv head
-  constexpr int NCH = HD / 8;                        // 16-byte chunks per row
-  constexpr int TILEB = kAttnStageTok * ROWB;        // K (or V) tile of one stage
-  constexpr int STAGEB = 2 * TILEB;
+  constexpr int ROWB = HD * 2, ROWBV = VD * 2;       // bytes of one cached key / value row of one kv head
+  constexpr int NCH = HD / 8, NCHV = VD / 8;         // 16-byte chunks per row
+  constexpr int TILEB = kAttnStageTok * ROWB;        // K tile of one stage
+  constexpr int STAGEB = TILEB + kAttnStageTok * ROWBV;
   constexpr int WARPB = kAttnStages * STAGEB;
-  constexpr int CPL = kAttnStageTok * NCH / 32;      // 16-byte copies per lane per tile
+  constexpr int CPL = kAttnStageTok * NCH / 32, CPLV = kAttnStageTok * NCHV / 32;   // 16-byte copies per lane per tile
   constexpr int KS = HD / 16;                        // k-steps of Q K^T
-  constexpr int NT = HD / 8;                         // n-tiles of the output
+  constexpr int NT = VD / 8;                         // n-tiles of the output
   __shared__ float s_m[kAttnWarps][8];
   __shared__ float s_l[kAttnWarps][8];
-  extern __shared__ __align__(128) uint8_t s_dyn[];  // per-warp rings; reused as [warps][GQ][HD] floats at the end
+  extern __shared__ __align__(128) uint8_t s_dyn[];  // per-warp rings; reused as [warps][heads][VD] floats at the end
 
   pdl_trigger();
   pdl_wait();      // q, the new K / V rows and the sequence tables come from the kernels before this one
-  const int t = blockIdx.x, hkv = blockIdx.y, split = blockIdx.z;
+  const int gq = GQ > 0 ? GQ : ext.gq, nsub = GQ > 0 ? 1 : (gq + 7) / 8;
+  const int t = blockIdx.x, hkv = blockIdx.y / nsub, split = blockIdx.z;
+  const int sub0 = (blockIdx.y % nsub) * 8;          // this CTA's heads of the group: sub0 .. sub0 + gn - 1
+  const int gn = GQ > 0 ? GQ : min(8, gq - sub0), head0 = hkv * gq + sub0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tq = lane & 3;            // accumulator row / column-pair of this lane
-  const int n_q = n_kv * GQ;
+  const int n_q = n_kv * gq;
 
   const int len = ctx_len[t];
   const int row = bt_row != nullptr ? bt_row[t] : t;
@@ -112,7 +128,6 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
   if (EXT) c0 = max(c0, vis0 / kAttnStageTok * kAttnStageTok);
   const int nchunk = (c1 - c0 + kAttnStageTok - 1) / kAttnStageTok;
   const int my_chunks = nchunk > warp ? (nchunk - warp + kAttnWarps - 1) / kAttnWarps : 0;
-  const long long tok_stride = static_cast<long long>(n_kv) * HD;
   const uint32_t ring = smem_u32(s_dyn) + warp * WARPB;
   const uint64_t stream_policy = l2_stream_policy();
 
@@ -127,10 +142,19 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
         const int id = lane + i * 32;
         const int r = id / NCH, c = id % NCH;
         const bool valid = tok0 + r < c1;
-        const long long off = valid ? (slot0 + r) * tok_stride + hkv * HD + c * 8 : 0;
-        const uint32_t d = dst0 + r * ROWB + ((c ^ (r & 7)) << 4);
-        cp_async16_stream(d, kcache + off, valid, stream_policy);
-        cp_async16_stream(d + TILEB, vcache + off, valid, stream_policy);
+        const long long off = valid ? ((slot0 + r) * n_kv + hkv) * HD + c * 8 : 0;
+        cp_async16_stream(dst0 + r * ROWB + (swz<NCH>(c, r) << 4), kcache + off, valid, stream_policy);
+        if (HD == VD) cp_async16_stream(dst0 + TILEB + r * ROWBV + (swz<NCHV>(c, r) << 4), vcache + off, valid, stream_policy);
+      }
+      if (HD != VD) {
+#pragma unroll
+        for (int i = 0; i < CPLV; ++i) {
+          const int id = lane + i * 32;
+          const int r = id / NCHV, c = id % NCHV;
+          const bool valid = tok0 + r < c1;
+          const long long off = valid ? ((slot0 + r) * n_kv + hkv) * VD + c * 8 : 0;
+          cp_async16_stream(dst0 + TILEB + r * ROWBV + (swz<NCHV>(c, r) << 4), vcache + off, valid, stream_policy);
+        }
       }
     }
     cp_async_commit();
@@ -138,14 +162,14 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
 #pragma unroll
   for (int j = 0; j < kAttnStages - 1; ++j) issue(j);
 
-  // Q fragments (rows >= GQ are zero)
+  // Q fragments (rows >= gn are zero)
   uint32_t qa[KS][4];
   {
-    const __nv_bfloat16* qp = q + static_cast<long long>(t) * ld_q + (hkv * GQ + g) * HD;
+    const __nv_bfloat16* qp = q + static_cast<long long>(t) * ld_q + (head0 + g) * HD;
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
-      qa[ks][0] = g < GQ ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * tq) : 0u;
-      qa[ks][2] = g < GQ ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 8 + 2 * tq) : 0u;
+      qa[ks][0] = g < gn ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * tq) : 0u;
+      qa[ks][2] = g < gn ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 8 + 2 * tq) : 0u;
       qa[ks][1] = 0u;
       qa[ks][3] = 0u;
     }
@@ -171,7 +195,7 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
       for (int ks = 0; ks < KS; ++ks) {
         const int c = 2 * ks + (lm_mi & 1);
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4(kb + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
+        ldmatrix_x4(kb + r * ROWB + (swz<NCH>(c, r) << 4), b0, b1, b2, b3);
         mma_bf16_16816(s0, qa[ks], b0, b1);
         mma_bf16_16816(s1, qa[ks], b2, b3);
       }
@@ -204,7 +228,7 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
       for (int dp = 0; dp < NT / 2; ++dp) {
         const int c = 2 * dp + (lm_mi >> 1);
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(vb + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
+        ldmatrix_x4_trans(vb + r * ROWBV + (swz<NCHV>(c, r) << 4), b0, b1, b2, b3);
         mma_bf16_16816(o[2 * dp], pa, b0, b1);
         mma_bf16_16816(o[2 * dp + 1], pa, b2, b3);
         if (EXT) {
@@ -219,44 +243,47 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
   __syncthreads();
 
   // merge the warps' partial states
-  float* s_acc = reinterpret_cast<float*>(s_dyn);   // [warps][GQ][HD]
-  if (g < GQ) {
+  float* s_acc = reinterpret_cast<float*>(s_dyn);   // [warps][gn][VD]
+  if (g < gn) {
     if (tq == 0) { s_m[warp][g] = m; s_l[warp][g] = l; }
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
-      s_acc[(warp * GQ + g) * HD + i * 8 + 2 * tq] = o[i][0];
-      s_acc[(warp * GQ + g) * HD + i * 8 + 2 * tq + 1] = o[i][1];
+      s_acc[(warp * gn + g) * VD + i * 8 + 2 * tq] = o[i][0];
+      s_acc[(warp * gn + g) * VD + i * 8 + 2 * tq + 1] = o[i][1];
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < GQ * HD; idx += kAttnThreads) {
-    const int gg = idx / HD, d = idx % HD;
+  for (int idx = threadIdx.x; idx < gn * VD; idx += kAttnThreads) {
+    const int gg = idx / VD, d = idx % VD;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kAttnWarps; ++w) M = fmaxf(M, s_m[w][gg]);
-    float L = 0.f, O = 0.f;
+    const int head = head0 + gg;
+    const bool sunk = EXT && ext.sink != nullptr && split == 0;      // one split carries the sink
+    const float sk = sunk ? ext.sink[head] * kLog2e : -INFINITY;
+    M = fmaxf(M, sk);
+    float L = sunk ? exp2f(sk - M) : 0.f, O = 0.f;
     if (M > -INFINITY) {
 #pragma unroll
       for (int w = 0; w < kAttnWarps; ++w) {
         const float wgt = exp2f(s_m[w][gg] - M);
         L += s_l[w][gg] * wgt;
-        O += s_acc[(w * GQ + gg) * HD + d] * wgt;
+        O += s_acc[(w * gn + gg) * VD + d] * wgt;
       }
     }
     const float val = L > 0.f ? O / L : 0.f;
-    const int head = hkv * GQ + gg;
     if (splits == 1) {
-      out[static_cast<long long>(t) * ld_out + head * HD + d] = __float2bfloat16(val);
+      out[static_cast<long long>(t) * ld_out + head * VD + d] = __float2bfloat16(val);
     } else {
       const long long pi = (static_cast<long long>(t) * n_q + head) * splits + split;
-      part_o[pi * HD + d] = val;
+      part_o[pi * VD + d] = val;
       if (d == 0) part_lse[pi] = L > 0.f ? M + log2f(L) : -INFINITY;
     }
   }
 }
 
 // out[t, head] = sum_s softmax_s(lse) * part_o[t, head, s]
-template <int HD>
+template <int VD>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, int splits,
                                   int n_q, __nv_bfloat16* __restrict__ out, long long ld_out) {
   const int t = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
@@ -268,10 +295,10 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     for (int s = 0; s < splits; ++s) {
       const float w = exp2f(part_lse[pi + s] - M);
       L += w;
-      O += w * part_o[(pi + s) * HD + d];
+      O += w * part_o[(pi + s) * VD + d];
     }
   }
-  out[static_cast<long long>(t) * ld_out + head * HD + d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
+  out[static_cast<long long>(t) * ld_out + head * VD + d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -290,31 +317,36 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
 constexpr int kPreKeys = 64;       // keys per pipeline stage
 constexpr int kPreRows = 64;       // query rows per CTA (4 warps x 16)
 
-template <int HD, int GQ, bool EXT>
+// 1 / denominator of a row with running maximum m (base 2) and sum l, the sink included; 0 for a row that saw nothing.
+__device__ __forceinline__ float sink_inverse(float m, float l, float sink) {
+  const float sk = sink * kLog2e, M = fmaxf(m, sk), f = exp2f(m - M);
+  return f / (l * f + exp2f(sk - M));
+}
+
+template <int HD, int VD, int GQ, bool EXT>
 __global__ void __launch_bounds__(128)
 prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ kcache,
                     const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_blocks,
                     const int4* __restrict__ tiles, int block_size, int n_kv, float scale_log2,
                     __nv_bfloat16* __restrict__ out, long long ld_out, AttnExt ext) {
-  constexpr int ROWB = HD * 2;
-  constexpr int NCH = HD / 8;                       // 16-byte chunks per K / V row
+  constexpr int ROWB = HD * 2, ROWBV = VD * 2;
+  constexpr int NCH = HD / 8, NCHV = VD / 8;        // 16-byte chunks per K / V row
   constexpr int TILEB = kPreKeys * ROWB;
-  constexpr int STAGEB = 2 * TILEB;                 // K tile then V tile
-  constexpr int CPT = kPreKeys * NCH / 128;         // 16-byte copies per thread per tile
+  constexpr int STAGEB = TILEB + kPreKeys * ROWBV;  // K tile then V tile
+  constexpr int CPT = kPreKeys * NCH / 128, CPTV = kPreKeys * NCHV / 128;   // 16-byte copies per thread per tile
   constexpr int KS = HD / 16;                       // k-steps of Q K^T
-  constexpr int NT = HD / 8;                        // n-tiles of the output
+  constexpr int NT = VD / 8;                        // n-tiles of the output
   extern __shared__ __align__(128) uint8_t s_pre[];
 
   const int4 tile = tiles[blockIdx.x];
   const int row0 = tile.x, ntok = tile.y, pos0 = tile.w;
-  const int hkv = blockIdx.y;
+  const int hkv = blockIdx.y, gq = GQ > 0 ? GQ : ext.gq;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tq = lane & 3;
   const int* bt = block_tables + static_cast<long long>(tile.z) * max_blocks;
   const int kmax = pos0 + ntok;                     // keys [0, kmax) exist for the last token of the tile
   const int nkb = (kmax + kPreKeys - 1) / kPreKeys;
   const int kb0 = EXT && ext.window > 0 ? max(0, pos0 - ext.window + 1) / kPreKeys : 0;   // first block anyone sees
-  const long long tok_stride = static_cast<long long>(n_kv) * HD;
   const uint32_t sbase = smem_u32(s_pre);
 
   auto issue = [&](int kb) {
@@ -329,26 +361,41 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
         long long off = 0;
         if (valid) {
           const long long blk = bt[key / block_size];
-          off = (blk * block_size + key % block_size) * tok_stride + hkv * HD + c * 8;
+          off = ((blk * block_size + key % block_size) * n_kv + hkv) * HD + c * 8;
         }
-        const uint32_t d = dst0 + r * ROWB + ((c ^ (r & 7)) << 4);
-        cp_async16(d, kcache + off, valid);
-        cp_async16(d + TILEB, vcache + off, valid);
+        cp_async16(dst0 + r * ROWB + (swz<NCH>(c, r) << 4), kcache + off, valid);
+        if (HD == VD) cp_async16(dst0 + TILEB + r * ROWBV + (swz<NCHV>(c, r) << 4), vcache + off, valid);
+      }
+      if (HD != VD) {
+#pragma unroll
+        for (int i = 0; i < CPTV; ++i) {
+          const int id = threadIdx.x + i * 128;
+          const int r = id / NCHV, c = id % NCHV;
+          const int key = kb * kPreKeys + r;
+          const bool valid = key < kmax;
+          long long off = 0;
+          if (valid) {
+            const long long blk = bt[key / block_size];
+            off = ((blk * block_size + key % block_size) * n_kv + hkv) * VD + c * 8;
+          }
+          cp_async16(dst0 + TILEB + r * ROWBV + (swz<NCHV>(c, r) << 4), vcache + off, valid);
+        }
       }
     }
     cp_async_commit();
   };
   issue(kb0);
 
-  // Q fragments: this warp's rows R0 = warp * 16 + g and R0 + 8; row R = (token R / GQ, head R % GQ)
+  // Q fragments: this warp's rows R0 = warp * 16 + g and R0 + 8; row R = (token R / gq, head R % gq)
   const int R0 = warp * 16 + g, R1 = R0 + 8;
-  const int t0 = R0 / GQ, t1 = R1 / GQ;
+  const int t0 = R0 / gq, t1 = R1 / gq;
+  const int head0 = hkv * gq + R0 % gq, head1 = hkv * gq + R1 % gq;
   const bool v0 = t0 < ntok, v1 = t1 < ntok;
   const int qpos0 = pos0 + t0, qpos1 = pos0 + t1;
   uint32_t qa[KS][4];
   {
-    const __nv_bfloat16* q0 = q + static_cast<long long>(row0 + t0) * ld_q + (hkv * GQ + R0 % GQ) * HD;
-    const __nv_bfloat16* q1 = q + static_cast<long long>(row0 + t1) * ld_q + (hkv * GQ + R1 % GQ) * HD;
+    const __nv_bfloat16* q0 = q + static_cast<long long>(row0 + t0) * ld_q + head0 * HD;
+    const __nv_bfloat16* q1 = q + static_cast<long long>(row0 + t1) * ld_q + head1 * HD;
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
       qa[ks][0] = v0 ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16 + 2 * tq) : 0u;
@@ -363,9 +410,9 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   const int lm_mi = lane >> 3, lm_r = lane & 7;
   // the warp's last query position: key blocks entirely behind it are skipped by this warp (causal)
-  const int wlast = pos0 + min(ntok - 1, (warp * 16 + 15) / GQ);
+  const int wlast = pos0 + min(ntok - 1, (warp * 16 + 15) / gq);
   // and, with a window, those entirely before the reach of its first query; a row's first visible key
-  const int wfirst = EXT && ext.window > 0 ? pos0 + warp * 16 / GQ - ext.window + 1 : 0;
+  const int wfirst = EXT && ext.window > 0 ? pos0 + warp * 16 / gq - ext.window + 1 : 0;
   const int lo0 = EXT && ext.window > 0 ? qpos0 - ext.window + 1 : 0;
   const int lo1 = EXT && ext.window > 0 ? qpos1 - ext.window + 1 : 0;
 
@@ -376,7 +423,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
     const uint32_t kbuf = sbase + (kb & 1) * STAGEB;
     const uint32_t vbuf = kbuf + TILEB;
     const int key0 = kb * kPreKeys;
-    if (key0 <= wlast && warp * 16 / GQ < ntok && (!EXT || key0 + kPreKeys > wfirst)) {
+    if (key0 <= wlast && warp * 16 / gq < ntok && (!EXT || key0 + kPreKeys > wfirst)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
@@ -387,7 +434,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
         for (int ks = 0; ks < KS; ++ks) {
           const int c = 2 * ks + (lm_mi & 1);
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(kbuf + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
+          ldmatrix_x4(kbuf + r * ROWB + (swz<NCH>(c, r) << 4), b0, b1, b2, b3);
           mma_bf16_16816(s[2 * kg], qa[ks], b0, b1);
           mma_bf16_16816(s[2 * kg + 1], qa[ks], b2, b3);
         }
@@ -449,7 +496,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
         for (int dp = 0; dp < NT / 2; ++dp) {
           const int c = 2 * dp + (lm_mi >> 1);
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(vbuf + r * ROWB + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
+          ldmatrix_x4_trans(vbuf + r * ROWBV + (swz<NCHV>(c, r) << 4), b0, b1, b2, b3);
           mma_bf16_16816(o[2 * dp], pa, b0, b1);
           mma_bf16_16816(o[2 * dp + 1], pa, b2, b3);
           if (EXT) {
@@ -463,15 +510,19 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   }
   cp_async_wait<0>();
 
-  const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  if (EXT && ext.sink != nullptr) {
+    inv0 = sink_inverse(m0, l0, ext.sink[head0]);
+    inv1 = sink_inverse(m1, l1, ext.sink[head1]);
+  }
   if (v0) {
-    __nv_bfloat16* op = out + static_cast<long long>(row0 + t0) * ld_out + (hkv * GQ + R0 % GQ) * HD;
+    __nv_bfloat16* op = out + static_cast<long long>(row0 + t0) * ld_out + head0 * VD;
 #pragma unroll
     for (int i = 0; i < NT; ++i)
       *reinterpret_cast<uint32_t*>(op + i * 8 + 2 * tq) = pack_bf16(o[i][0] * inv0, o[i][1] * inv0);
   }
   if (v1) {
-    __nv_bfloat16* op = out + static_cast<long long>(row0 + t1) * ld_out + (hkv * GQ + R1 % GQ) * HD;
+    __nv_bfloat16* op = out + static_cast<long long>(row0 + t1) * ld_out + head1 * VD;
 #pragma unroll
     for (int i = 0; i < NT; ++i)
       *reinterpret_cast<uint32_t*>(op + i * 8 + 2 * tq) = pack_bf16(o[i][2] * inv1, o[i][3] * inv1);
@@ -479,55 +530,58 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
 }
 
 // Options of a launch as the kernels take them (softcap <= 0: none; window <= 0: every key).
-static AttnExt make_ext(float scale, int window, float softcap) {
+static AttnExt make_ext(float scale, int window, float softcap, const float* sink, int gq) {
   AttnExt x;
+  x.sink = sink;
+  x.gq = gq;
   x.window = window > 0 ? window : 0;
   x.cap_in = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
   x.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   return x;
 }
 
-template <int HD, int GQ, bool EXT>
+template <int HD, int VD, int GQ, bool EXT>
 static int launch_prefill(const void* q, long long ld_q, const void* kc, const void* vc, const int* bt, int max_blocks,
                           const void* tiles, int n_tiles, int block_size, int n_kv, float scale, void* out,
                           long long ld_out, AttnExt ext, cudaStream_t stream) {
-  const size_t smem = 2 * 2 * static_cast<size_t>(kPreKeys) * HD * 2;
+  const size_t smem = 2 * static_cast<size_t>(kPreKeys) * (HD + VD) * 2;
   static PerDeviceOnce configured;
   const int crc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(prefill_attn_kernel<HD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return static_cast<int>(cudaFuncSetAttribute(prefill_attn_kernel<HD, VD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  96 * 1024));
   });
   if (crc != 0) return crc;
   dim3 grid(n_tiles, n_kv);
-  prefill_attn_kernel<HD, GQ, EXT><<<grid, 128, smem, stream>>>(
+  prefill_attn_kernel<HD, VD, GQ, EXT><<<grid, 128, smem, stream>>>(
       static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kc),
       static_cast<const __nv_bfloat16*>(vc), bt, max_blocks, static_cast<const int4*>(tiles), block_size, n_kv,
       scale * 1.4426950408889634f, static_cast<__nv_bfloat16*>(out), ld_out, ext);
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int HD, int GQ, bool EXT>
+template <int HD, int VD, int GQ, bool EXT>
 static int launch_attn(const void* q, long long ld_q, const void* kc, const void* vc, const int* bt, int max_blocks,
                        const int* bt_row, const int* ctx_len, int block_size, int T, int n_kv, float scale, int splits,
                        void* out, long long ld_out, float* part_o, float* part_lse, AttnExt ext, cudaStream_t stream) {
-  const size_t merge_b = static_cast<size_t>(kAttnWarps) * GQ * HD * sizeof(float);
-  const size_t ring_b = static_cast<size_t>(kAttnWarps) * kAttnStages * 2 * kAttnStageTok * HD * 2;
+  const int gq = GQ > 0 ? GQ : ext.gq, nsub = (gq + 7) / 8;
+  const size_t merge_b = static_cast<size_t>(kAttnWarps) * (gq < 8 ? gq : 8) * VD * sizeof(float);
+  const size_t ring_b = static_cast<size_t>(kAttnWarps) * kAttnStages * kAttnStageTok * (HD + VD) * 2;
   const size_t smem = merge_b > ring_b ? merge_b : ring_b;
   static PerDeviceOnce configured;
   const int crc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(paged_attn_kernel<HD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return static_cast<int>(cudaFuncSetAttribute(paged_attn_kernel<HD, VD, GQ, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  160 * 1024));
   });
   if (crc != 0) return crc;
-  dim3 grid(T, n_kv, splits);
-  cudaError_t e = launch_kernel(paged_attn_kernel<HD, GQ, EXT>, grid, dim3(kAttnThreads), smem, stream,
+  dim3 grid(T, n_kv * nsub, splits);
+  cudaError_t e = launch_kernel(paged_attn_kernel<HD, VD, GQ, EXT>, grid, dim3(kAttnThreads), smem, stream,
       static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kc),
       static_cast<const __nv_bfloat16*>(vc), bt, max_blocks, bt_row, ctx_len, block_size, n_kv,
       scale * 1.4426950408889634f, splits, static_cast<__nv_bfloat16*>(out), ld_out, part_o, part_lse, ext);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (splits > 1) {
-    dim3 g2(T, n_kv * GQ);
-    attn_merge_kernel<HD><<<g2, HD, 0, stream>>>(part_o, part_lse, splits, n_kv * GQ,
+    dim3 g2(T, n_kv * gq);
+    attn_merge_kernel<VD><<<g2, VD, 0, stream>>>(part_o, part_lse, splits, n_kv * gq,
                                                   static_cast<__nv_bfloat16*>(out), ld_out);
     e = cudaGetLastError();
   }
@@ -543,34 +597,41 @@ extern "C" long long dmoe_paged_attention_workspace_floats(int T, int n_q, int h
   return static_cast<long long>(T) * n_q * splits * (hd + 1);
 }
 
-// Instantiations by head size, query group and options; -11: no tensor-core kernel for this shape.
+// Instantiations: without options by head size and query group, with options by key and value size; -11: no tensor-core
+// kernel for this shape.
 template <bool EXT>
 static int attn_dispatch(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
                          int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
-                         int hd, float scale, int splits, void* out, long long ld_out, float* workspace, AttnExt ext,
+                         int hd, int vd, float scale, int splits, void* out, long long ld_out, float* workspace, AttnExt ext,
                          cudaStream_t stream) {
   if (T == 0) return 0;
-  if (n_kv < 1 || n_q % n_kv != 0 || splits < 1 || splits > 65535 || n_kv > 65535 || block_size % kAttnStageTok != 0) return -10;
+  if (n_kv < 1 || n_q % n_kv != 0 || splits < 1 || splits > 65535 || n_q > 65535 || block_size % kAttnStageTok != 0) return -10;
   if (splits > 1 && workspace == nullptr) return -12;
   const int gq = n_q / n_kv;
   float* part_o = workspace;
-  float* part_lse = workspace != nullptr ? workspace + static_cast<long long>(T) * n_q * splits * hd : nullptr;
-#define DMOE_ATTN(HD_, GQ_)                                                                                             \
-  return launch_attn<HD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, \
-                                    n_kv, scale, splits, out, ld_out, part_o, part_lse, ext, stream)
-  if (hd == 128) {
+  float* part_lse = workspace != nullptr ? workspace + static_cast<long long>(T) * n_q * splits * vd : nullptr;
+#define DMOE_ATTN(HD_, VD_, GQ_)                                                                                             \
+  return launch_attn<HD_, VD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, \
+                                         n_kv, scale, splits, out, ld_out, part_o, part_lse, ext, stream)
+  if constexpr (EXT) {
+    if (gq > 64) return -11;
+    if (hd == 128 && vd == 128) DMOE_ATTN(128, 128, 0);
+    if (hd == 128 && vd == 64) DMOE_ATTN(128, 64, 0);
+    if (hd == 64 && vd == 64) DMOE_ATTN(64, 64, 0);
+    if (hd == 64 && vd == 32) DMOE_ATTN(64, 32, 0);
+  } else if (hd == 128) {
     switch (gq) {
-      case 1: DMOE_ATTN(128, 1);
-      case 2: DMOE_ATTN(128, 2);
-      case 4: DMOE_ATTN(128, 4);
-      case 8: DMOE_ATTN(128, 8);
+      case 1: DMOE_ATTN(128, 128, 1);
+      case 2: DMOE_ATTN(128, 128, 2);
+      case 4: DMOE_ATTN(128, 128, 4);
+      case 8: DMOE_ATTN(128, 128, 8);
     }
   } else if (hd == 64) {
     switch (gq) {
-      case 1: DMOE_ATTN(64, 1);
-      case 2: DMOE_ATTN(64, 2);
-      case 4: DMOE_ATTN(64, 4);
-      case 8: DMOE_ATTN(64, 8);
+      case 1: DMOE_ATTN(64, 64, 1);
+      case 2: DMOE_ATTN(64, 64, 2);
+      case 4: DMOE_ATTN(64, 64, 4);
+      case 8: DMOE_ATTN(64, 64, 8);
     }
   }
 #undef DMOE_ATTN
@@ -582,51 +643,58 @@ extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* k
                                     int block_size, int T, int n_q, int n_kv, int hd, float scale, int splits, void* out,
                                     long long ld_out, float* workspace, void* stream_) {
   return attn_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                              hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0.f),
+                              hd, hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0.f, nullptr, 0),
                               static_cast<cudaStream_t>(stream_));
 }
 
-// The same with a sliding window and a score soft cap (0 = without).
+// The same with a sliding window, a score soft cap (0 = without) and a sink per head (NULL = without), value heads of another
+// size than key heads, and query groups of up to 64 heads.
 extern "C" int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                         const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
-                                        int block_size, int T, int n_q, int n_kv, int hd, float scale, int window,
-                                        float softcap, int splits, void* out, long long ld_out, float* workspace,
-                                        void* stream_) {
+                                        int block_size, int T, int n_q, int n_kv, int hd, int vd, float scale, int window,
+                                        float softcap, const float* sink, int splits, void* out, long long ld_out,
+                                        float* workspace, void* stream_) {
+  if (n_kv < 1) return -10;
   return attn_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                             hd, scale, splits, out, ld_out, workspace, make_ext(scale, window, softcap),
+                             hd, vd, scale, splits, out, ld_out, workspace, make_ext(scale, window, softcap, sink, n_q / n_kv),
                              static_cast<cudaStream_t>(stream_));
 }
 
 // Tokens per tile of dmoe_prefill_attention for a query group of n_q / n_kv heads.
 extern "C" int dmoe_prefill_tile_tokens(int n_q, int n_kv) {
   if (n_kv < 1 || n_q % n_kv != 0) return 0;
-  const int gq = n_q / n_kv;
-  return (gq == 1 || gq == 2 || gq == 4 || gq == 8) ? kPreRows / gq : 0;
+  return kPreRows / (n_q / n_kv);
 }
 
 template <bool EXT>
 static int prefill_dispatch(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
-                            int max_blocks, const void* tiles, int n_tiles, int block_size, int n_q, int n_kv, int hd,
+                            int max_blocks, const void* tiles, int n_tiles, int block_size, int n_q, int n_kv, int hd, int vd,
                             float scale, void* out, long long ld_out, AttnExt ext, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   if (n_kv < 1 || n_q % n_kv != 0 || n_kv > 65535 || n_tiles < 0 || block_size < 1 || tiles == nullptr) return -10;
   const int gq = n_q / n_kv;
-#define DMOE_PRE(HD_, GQ_)                                                                                          \
-  return launch_prefill<HD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, \
-                                       n_kv, scale, out, ld_out, ext, stream)
-  if (hd == 128) {
+#define DMOE_PRE(HD_, VD_, GQ_)                                                                                          \
+  return launch_prefill<HD_, VD_, GQ_, EXT>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, \
+                                            n_kv, scale, out, ld_out, ext, stream)
+  if constexpr (EXT) {
+    if (gq > kPreRows) return -11;
+    if (hd == 128 && vd == 128) DMOE_PRE(128, 128, 0);
+    if (hd == 128 && vd == 64) DMOE_PRE(128, 64, 0);
+    if (hd == 64 && vd == 64) DMOE_PRE(64, 64, 0);
+    if (hd == 64 && vd == 32) DMOE_PRE(64, 32, 0);
+  } else if (hd == 128) {
     switch (gq) {
-      case 1: DMOE_PRE(128, 1);
-      case 2: DMOE_PRE(128, 2);
-      case 4: DMOE_PRE(128, 4);
-      case 8: DMOE_PRE(128, 8);
+      case 1: DMOE_PRE(128, 128, 1);
+      case 2: DMOE_PRE(128, 128, 2);
+      case 4: DMOE_PRE(128, 128, 4);
+      case 8: DMOE_PRE(128, 128, 8);
     }
   } else if (hd == 64) {
     switch (gq) {
-      case 1: DMOE_PRE(64, 1);
-      case 2: DMOE_PRE(64, 2);
-      case 4: DMOE_PRE(64, 4);
-      case 8: DMOE_PRE(64, 8);
+      case 1: DMOE_PRE(64, 64, 1);
+      case 2: DMOE_PRE(64, 64, 2);
+      case 4: DMOE_PRE(64, 64, 4);
+      case 8: DMOE_PRE(64, 64, 8);
     }
   }
 #undef DMOE_PRE
@@ -638,15 +706,17 @@ extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void*
                                       int block_size, int n_q, int n_kv, int hd, float scale, void* out, long long ld_out,
                                       void* stream_) {
   return prefill_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                 hd, scale, out, ld_out, make_ext(scale, 0, 0.f), static_cast<cudaStream_t>(stream_));
+                                 hd, hd, scale, out, ld_out, make_ext(scale, 0, 0.f, nullptr, 0),
+                                 static_cast<cudaStream_t>(stream_));
 }
 
 extern "C" int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                           const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
-                                          int block_size, int n_q, int n_kv, int hd, float scale, int window,
-                                          float softcap, void* out, long long ld_out, void* stream_) {
+                                          int block_size, int n_q, int n_kv, int hd, int vd, float scale, int window,
+                                          float softcap, const float* sink, void* out, long long ld_out, void* stream_) {
+  if (n_kv < 1) return -10;
   return prefill_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                hd, scale, out, ld_out, make_ext(scale, window, softcap),
+                                hd, vd, scale, out, ld_out, make_ext(scale, window, softcap, sink, n_q / n_kv),
                                 static_cast<cudaStream_t>(stream_));
 }
 
@@ -660,21 +730,24 @@ constexpr int kAnyKeys = 128;
 
 template <typename T>
 __global__ void __launch_bounds__(kAnyKeys)
-any_attn_kernel(const T* __restrict__ q, long long ld_q, const T* __restrict__ kcache, const T* __restrict__ vcache,
-                const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ bt_row,
-                const int* __restrict__ ctx_len, int block_size, int n_q, int n_kv, int dk, int dv, float scale, int window,
-                float softcap, T* __restrict__ out, long long ld_out) {
+any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, const T* __restrict__ kcache, long long k_tok,
+                const T* __restrict__ vcache, long long v_tok, const int* __restrict__ block_tables, int max_blocks,
+                const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len, int block_size,
+                int n_q, int n_kv, int dk, int dv, float scale, int window, float softcap, const float* __restrict__ sink,
+                T* __restrict__ out, long long o_head, long long o_row) {
   extern __shared__ float s_any[];          // q [dk] | acc [dv]
   __shared__ float s_p[kAnyKeys];
   __shared__ long long s_slot[kAnyKeys];
   __shared__ float s_red[2][kAnyKeys / 32];
   float* s_q = s_any;
   float* s_acc = s_any + dk;
-  const int t = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+  const int head = blockIdx.y, tid = threadIdx.x;
+  const int t = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;      // batch row whose context the query has
+  const T* qp = q + blockIdx.x * q_row + head * q_head;
   const int hkv = head / (n_q / n_kv);
   const int len = ctx_len[t];
   const int* bt = block_tables + static_cast<long long>(bt_row != nullptr ? bt_row[t] : t) * max_blocks;
-  for (int d = tid; d < dk; d += kAnyKeys) s_q[d] = static_cast<float>(q[t * ld_q + head * dk + d]);
+  for (int d = tid; d < dk; d += kAnyKeys) s_q[d] = static_cast<float>(qp[d]);
   for (int d = tid; d < dv; d += kAnyKeys) s_acc[d] = 0.f;
   __syncthreads();
   float m = -INFINITY, l = 0.f;
@@ -684,7 +757,7 @@ any_attn_kernel(const T* __restrict__ q, long long ld_q, const T* __restrict__ k
     if (tid < n) {
       const int j = j0 + tid;
       const long long slot = static_cast<long long>(bt[j / block_size]) * block_size + j % block_size;
-      const T* kr = kcache + (slot * n_kv + hkv) * dk;
+      const T* kr = kcache + slot * k_tok + hkv * dk;
       float acc = 0.f;
       for (int d = 0; d < dk; ++d) acc += s_q[d] * static_cast<float>(kr[d]);
       s = acc * scale;
@@ -710,21 +783,28 @@ any_attn_kernel(const T* __restrict__ q, long long ld_q, const T* __restrict__ k
     m = mn;
     for (int d = tid; d < dv; d += kAnyKeys) {
       float acc = s_acc[d] * corr;
-      for (int j = 0; j < n; ++j) acc += s_p[j] * static_cast<float>(vcache[(s_slot[j] * n_kv + hkv) * dv + d]);
+      for (int j = 0; j < n; ++j) acc += s_p[j] * static_cast<float>(vcache[s_slot[j] * v_tok + hkv * dv + d]);
       s_acc[d] = acc;
     }
     __syncthreads();
   }
+  float f = 1.f;
+  if (sink != nullptr && len > 0) {
+    const float mn = fmaxf(m, sink[head]);
+    f = expf(m - mn);
+    l = l * f + expf(sink[head] - mn);
+  }
   for (int d = tid; d < dv; d += kAnyKeys)
-    out[t * ld_out + head * dv + d] = static_cast<T>(l > 0.f ? s_acc[d] / l : 0.f);
+    out[blockIdx.x * o_row + head * o_head + d] = static_cast<T>(l > 0.f ? s_acc[d] * f / l : 0.f);
 }
 
 }  // namespace dmoe
 
-extern "C" int dmoe_any_attention(int is_f32, const void* q, long long ld_q, const void* kcache, const void* vcache,
-                                  const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
-                                  int block_size, int T, int n_q, int n_kv, int dk, int dv, float scale, int window,
-                                  float softcap, void* out, long long ld_out, void* stream_) {
+extern "C" int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_row, const void* kcache,
+                                  long long k_tok, const void* vcache, long long v_tok, const int* block_tables, int max_blocks,
+                                  const int* bt_row, const int* rows, const int* ctx_len, int block_size, int T, int n_q,
+                                  int n_kv, int dk, int dv, float scale, int window, float softcap, const float* sink, void* out,
+                                  long long o_head, long long o_row, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (T == 0) return 0;
   if (n_kv < 1 || n_q % n_kv != 0 || n_q > 65535 || block_size < 1 || dk < 1 || dv < 1 || dk + dv > 8192) return -10;
@@ -732,12 +812,13 @@ extern "C" int dmoe_any_attention(int is_f32, const void* q, long long ld_q, con
   const size_t smem = static_cast<size_t>(dk + dv) * sizeof(float);
   if (is_f32)
     any_attn_kernel<float><<<grid, kAnyKeys, smem, stream>>>(
-        static_cast<const float*>(q), ld_q, static_cast<const float*>(kcache), static_cast<const float*>(vcache), block_tables,
-        max_blocks, bt_row, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, softcap, static_cast<float*>(out), ld_out);
+        static_cast<const float*>(q), q_head, q_row, static_cast<const float*>(kcache), k_tok, static_cast<const float*>(vcache),
+        v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, softcap, sink,
+        static_cast<float*>(out), o_head, o_row);
   else
     any_attn_kernel<__nv_bfloat16><<<grid, kAnyKeys, smem, stream>>>(
-        static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(kcache),
-        static_cast<const __nv_bfloat16*>(vcache), block_tables, max_blocks, bt_row, ctx_len, block_size, n_q, n_kv, dk, dv,
-        scale, window, softcap, static_cast<__nv_bfloat16*>(out), ld_out);
+        static_cast<const __nv_bfloat16*>(q), q_head, q_row, static_cast<const __nv_bfloat16*>(kcache), k_tok,
+        static_cast<const __nv_bfloat16*>(vcache), v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv,
+        dk, dv, scale, window, softcap, sink, static_cast<__nv_bfloat16*>(out), o_head, o_row);
   return static_cast<int>(cudaGetLastError());
 }

@@ -73,6 +73,8 @@ typedef struct DmoeGemm {
   // != 0: W is stored tile by tile, [group][128-row tile][K / 64][128][64] (see ops/gemm.py: block_weight), so that
   // every 16 KB box the kernel fetches is one contiguous run of HBM; needs F % 128 == 0 and K % 64 == 0
   int w_blocked;
+  // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form)
+  int act;
   // profiling aid, normally null: 16 x uint64 of device memory that CTA 0 fills with %globaltimer stamps (entry, set-up
   // done, first TMA issued, first stage landed, last MMA committed, accumulator seen by the epilogue, epilogue done,
   // tear-down reached, then five points inside the first epilogue chunk and three inside the producer's start)
@@ -108,21 +110,46 @@ int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, cons
                          int T, int n_q, int n_kv, int hd, float scale, int splits, void* out, long long ld_out,
                          float* workspace, void* stream);
 
-// With a sliding window (a query sees the last `window` tokens, itself included; 0 = all) and a score soft cap
-// (cap * tanh(score / cap); 0 = none).
+// With a sliding window (a query sees the last `window` tokens, itself included; 0 = all), a score soft cap
+// (cap * tanh(score / cap); 0 = none) and a sink (exp(sink[head]) enters the softmax denominator; NULL = none); value heads
+// of size vd. (hd, vd) = (64, 32), (64, 64), (128, 64), (128, 128), up to 64 query heads per kv head.
 int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
                              int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
-                             int hd, float scale, int window, float softcap, int splits, void* out, long long ld_out,
-                             float* workspace, void* stream);
+                             int hd, int vd, float scale, int window, float softcap, const float* sink, int splits, void* out,
+                             long long ld_out, float* workspace, void* stream);
 int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                const int* block_tables, int max_blocks, const void* tiles, int n_tiles, int block_size,
-                               int n_q, int n_kv, int hd, float scale, int window, float softcap, void* out,
-                               long long ld_out, void* stream);
-// Any key / value size and query group, bf16 or fp32 cache, fp32 arithmetic on the CUDA cores.
-int dmoe_any_attention(int is_f32, const void* q, long long ld_q, const void* kcache, const void* vcache,
-                       const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T,
-                       int n_q, int n_kv, int dk, int dv, float scale, int window, float softcap, void* out,
-                       long long ld_out, void* stream);
+                               int n_q, int n_kv, int hd, int vd, float scale, int window, float softcap, const float* sink,
+                               void* out, long long ld_out, void* stream);
+// Any key / value size and query group, bf16 or fp32 cache, fp32 arithmetic on the CUDA cores. Query i of head h starts at
+// q + i * q_row + h * q_head (output likewise) and has the context of batch row rows[i] (NULL: i); the heads of a cached token
+// are contiguous, tokens k_tok / v_tok elements apart.
+int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_row, const void* kcache, long long k_tok,
+                       const void* vcache, long long v_tok, const int* block_tables, int max_blocks, const int* bt_row,
+                       const int* rows, const int* ctx_len, int block_size, int T, int n_q, int n_kv, int dk, int dv,
+                       float scale, int window, float softcap, const float* sink, void* out, long long o_head, long long o_row,
+                       void* stream);
+
+// ---- latent attention (latent_attention.cu): the cache has one row [latent rankp | rotated key part rotp] per token ---------
+// Projection rows y = [heads x (q dimp | rotp) | latent rankp | key part rotp] (every part padded to a multiple of 8): RMS norm
+// of the latent, rotation of the key part, both to cache rows at slots (< 0: skip); rotation of the queries in place, and for
+// rows with loose[t] = i >= 0 (NULL: i = t) to xq [heads, n_loose, dimp] and columns rankp.. of qa [heads, n_loose, row].
+int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
+                     int heads, int dim, int rot_dim, int rank, int rot, int interleaved, const void* table, int max_pos,
+                     const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa, void* stream);
+// Queries qa [heads, n, row] over cache rows (keys: all of a row, values: its first rankp columns), out [heads, n, rankp];
+// rankp <= 512, row <= 640. workspace: heads * n * splits * (rankp + 1) floats where splits > 1.
+int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
+                          const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale,
+                          int window, const float* sink, int splits, void* out, float* workspace, void* stream);
+// out[i] = cache row of position keys[i].y of block-table row keys[i].x
+int dmoe_latent_gather(const void* cache, const int* block_tables, int max_blocks, const void* keys, int n, int block_size,
+                       int row, void* out, void* stream);
+// Prompt tiles over expanded keys and values: tile i's key at position p is row base[i] + p of kv [heads x (dimp | vdimp)] and
+// of lat (columns rankp ..: its rotated part).
+int dmoe_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
+                        const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp, int vdimp,
+                        float scale, int window, const float* sink, void* out, long long ld_out, void* stream);
 
 // Tiled causal attention for prompt tokens: CTA column i handles tiles[i] = int4 {first row in q / out, tokens
 // (<= dmoe_prefill_tile_tokens), block-table row, position of the first token}; the tokens of a tile are consecutive
@@ -141,14 +168,29 @@ int dmoe_resid_norm(int is_f32, float* resid, const void* y, long long ld_y, con
                     float out_scale, float eps, const int* rows, void* h, long long ld_h, int n, int W, void* stream);
 // float2 table [max_pos][half] = (cos, sin)(pos * freq[i]) * mscale, freq in double on the device
 int dmoe_rope_freq_table(void* table, int max_pos, int half, const double* freq, float mscale, void* stream);
-// Per-head RMS norm of q and k, rotation of pairs (i, i + rot / 2), i < rot / 2, q in place, k / v into the paged caches.
+// Per-head RMS norm of q and k (qw, kw; NULL: none), rotation of pairs (i, i + rot / 2), i < rot / 2, or (2i, 2i + 1) where
+// interleaved; q in place, k / v into the paged caches, v as (1 - v_lambda) v + v_lambda v_first where that is given
+// (row stride ld_first, head stride first_head).
 int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots, void* kcache,
-                      void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, const void* table, int max_pos,
-                      const float* qw, const float* kw, float eps, void* stream);
-int dmoe_silu_mul(int is_f32, const void* gu, long long ld, void* out, long long ld_out, int T, int I, void* stream);
+                      void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved, const void* table,
+                      int max_pos, const float* qw, const float* kw, float eps, const void* v_first, long long ld_first,
+                      int first_head, float v_lambda, void* stream);
+// x = resid[r] + y[r] + sum of n_parts rows of parts (both may be NULL); resid[r] = x unless a row table picks r = rows[i];
+// h[i] = norm(x) * w, RMS norm or with `centred` layer norm. With gate_w [E, W] also softmax router over h: the K largest
+// scores (renorm: divided by their sum) and, where counts is given, the histogram of the chosen experts. E <= 256, K <= 32.
+int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
+                  long long part_row, long long part_stride, const float* w, int centred, float eps, const int* rows, void* h,
+                  long long ld_h, int n, int W, const void* gate_w, int E, int K, int renorm, int* ids, float* wts, int* counts,
+                  void* stream);
+// out[t, i] = act(gu[t, i]) * gu[t, I + i]; act 0: silu, 1: gelu (tanh form)
+int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I, void* stream);
 // Y = X W^T on the CUDA cores in fp32 arithmetic: fp32 operands, or bf16 operands of any alignment.
 int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y, long long ldy,
                      int T, int F, int K, void* stream);
+// The same over row groups: rows offs[g] .. offs[g + 1] of X with W[g] [F, K]; recs / bases (may be NULL): row t goes, scaled,
+// where recs[t] says (see DmoeGemm), in X's type.
+int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y, long long ldy,
+                      const void* recs, const void* bases, int T, int F, int K, void* stream);
 
 // ---- linear recurrences with a matrix state per head (recurrent.cu) ---------------------------------------
 typedef struct DmoeRecur {
@@ -204,6 +246,10 @@ int dmoe_route_ex(const void* x, long long ld_x, const void* norm_w, float eps, 
 int dmoe_dispatch_local(const void* y, long long ld_y, const int* topk_ids, const float* topk_w, int T, int K, int H,
                         int E, int experts_per_rank, int my_rank, int* ws, int* offs, const void* x_bases,
                         long long ld_dst, const void* rec_bases, int dst_capacity, int* status, void* stream);
+// The same on one device for rows of H elements of elem_bytes (2 or 4) without alignment.
+int dmoe_dispatch_local_any(int elem_bytes, const void* y, long long ld_y, const int* topk_ids, const float* topk_w, int T, int K,
+                            int H, int E, int* ws, int* offs, const void* x_bases, long long ld_dst, const void* rec_bases,
+                            int dst_capacity, int* status, void* stream);
 
 // ---- peer-memory dispatch (comm.cu) -----------------------------------------------------------------
 // Stores every routed (token, k) row of this attention rank into its region on the expert GPU that owns the

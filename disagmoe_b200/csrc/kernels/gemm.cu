@@ -96,6 +96,7 @@ struct GemmArgs {
   // w_blocked: the weights are stored tile by tile ([group][128-row tile][K block][128][64], every 16 KB TMA box one
   // contiguous run of HBM) instead of row-major [group][row][K]
   int w_blocked;
+  int act;      // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form)
   // optional [16] nanosecond stamps written by CTA 0 (a profiling aid, null in normal launches): 0 entry, 1 set-up done,
   // 2 first TMA issued, 3 first stage landed, 4 last MMA committed, 5 accumulator seen by the epilogue, 6 epilogue done,
   // 7 tear-down reached; 8-12 inside the first epilogue chunk: TMEM read done, staged to shared memory, barrier passed,
@@ -137,6 +138,12 @@ __device__ __forceinline__ void trace_stamp(const GemmArgs& a, int i) {
     asm volatile("mov.u64 %0, %globaltimer;" : "=l"(t));
     a.trace[i] = t;
   }
+}
+
+// silu(g) = g sigmoid(g); the tanh form of gelu is g sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3))
+__device__ __forceinline__ float gate_act(float g, int act) {
+  const float z = act == 0 ? g : 1.5957691216057308f * (g + 0.044715f * g * g * g);
+  return g / (1.f + __expf(-z));
 }
 
 __device__ __forceinline__ int ld_acquire_sys(const int* p) {
@@ -504,7 +511,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
           }
           if (EPI == EPI_SWIGLU) {
 #pragma unroll
-            for (int j = 0; j < 32; ++j) acc[j] = (acc[j] / (1.f + __expf(-acc[j]))) * up[j];
+            for (int j = 0; j < 32; ++j) acc[j] = gate_act(acc[j], a.act) * up[j];
           }
         } else {
           uint32_t v[32];
@@ -518,7 +525,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
             for (int j = 0; j < 32; ++j) {
               const float g = __uint_as_float(v[j]);
               const float up = __uint_as_float(uu[j]);
-              acc[j] = (g / (1.f + __expf(-g))) * up;
+              acc[j] = gate_act(g, a.act) * up;
             }
           } else {
             tmem_ld_wait();
@@ -1001,6 +1008,7 @@ extern "C" int dmoe_gemm(const DmoeGemm* d, void* stream_) {
   const long long ldx = d->ldx > 0 ? d->ldx : d->K;
   a.trace = static_cast<unsigned long long*>(d->trace);
   a.w_blocked = d->w_blocked != 0;
+  a.act = d->act;
   if (a.w_blocked) {
     // whole 128-row tiles and whole 64-element K blocks only; row coordinates must stay below 2^31
     const long long rows = static_cast<long long>(d->G) * a.w_rows * (d->K / kBK);

@@ -1,0 +1,628 @@
+// Latent attention for sm_100a: keys and values of all heads are linear maps of one cached latent vector per token, plus one
+// rotated key part that the heads share. Cache row = [latent (rankp) | rotated key part (rotp)], bf16 (fp32 in fp32 runs).
+//
+//   latent_prep_kernel     norm of the latent, rotations, cache append, queries head by head for the rows below
+//   latent_attn_kernel     rows on their own (decoding, short portions): the key map is already multiplied into the query, so
+//                          all heads attend over the cached rows themselves (key = the row, value = its first rankp columns)
+//   latent_gather_kernel   cached rows of a prompt run's visible keys, packed for the GEMM that expands them to heads
+//   latent_prefill_kernel  prompt runs: causal attention over expanded keys and values
+#include "dmoe_kernels.h"
+#include "mma_sync.cuh"
+
+namespace dmoe {
+
+typedef __nv_bfloat16 bf16;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int pad8(int n) { return (n + 7) / 8 * 8; }
+
+// One CTA per row. A row of y is [heads x (dimp | rotp) | rankp | rotp], parts padded with zeros to multiples of 8.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
+                   T* __restrict__ cache, int heads, int dimp, int rotp, int rank, int rankp, int rot, int interleaved,
+                   const float2* __restrict__ table, int max_pos, const float* __restrict__ norm_w, float eps,
+                   const int* __restrict__ loose, int n_loose, T* __restrict__ xq, T* __restrict__ qa) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int half = rot / 2, qd = dimp + rotp, row = rankp + rotp;
+  const int pos = min(max(positions[t], 0), max_pos - 1);
+  const long long slot = slots[t];
+  const int li = loose != nullptr ? loose[t] : static_cast<int>(t);
+  const float2* tab = table + static_cast<long long>(pos) * half;
+  T* yr = y + t * ld;
+  const T* c = yr + static_cast<long long>(heads) * qd;
+
+  // rotated part of a head (or of the key): pairs turn, what is not rotated passes
+  auto turn = [&](const T* p, T* dst, int first, int step) {
+    for (int i = first; i < half; i += step) {
+      const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
+      const float u = static_cast<float>(p[a]), v = static_cast<float>(p[b]);
+      const float2 cs = tab[i];
+      dst[a] = static_cast<T>(u * cs.x - v * cs.y);
+      dst[b] = static_cast<T>(v * cs.x + u * cs.y);
+    }
+    if (p != dst)
+      for (int d = rot + first; d < rotp; d += step) dst[d] = p[d];
+  };
+
+  if (slot >= 0) {
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < rank; d += blockDim.x) {
+      const float x = static_cast<float>(c[d]);
+      ss += x * x;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) ss += red[w];
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(rank) + eps);
+    T* dst = cache + slot * row;
+    for (int d = threadIdx.x; d < rank; d += blockDim.x) dst[d] = static_cast<T>(static_cast<float>(c[d]) * inv * norm_w[d]);
+    turn(c + rankp, dst + rankp, threadIdx.x, blockDim.x);
+  }
+  for (int h = warp; h < heads; h += blockDim.x >> 5) {
+    T* q = yr + static_cast<long long>(h) * qd;
+    if (li < 0) {
+      turn(q + dimp, q + dimp, lane, 32);
+      continue;
+    }
+    const long long at = static_cast<long long>(h) * n_loose + li;
+    constexpr int V = 16 / sizeof(T);
+    const uint4* src = reinterpret_cast<const uint4*>(q);
+    uint4* dst = reinterpret_cast<uint4*>(xq + at * dimp);
+    for (int v = lane; v < dimp / V; v += 32) dst[v] = src[v];
+    turn(q + dimp, qa + at * row + rankp, lane, 32);
+  }
+}
+
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_tables, int max_blocks,
+                     const int2* __restrict__ keys, int n, int block_size, int units, uint4* __restrict__ out) {
+  const int lane = threadIdx.x & 31;
+  const long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (i >= n) return;
+  const int2 k = keys[i];
+  const long long slot = static_cast<long long>(block_tables[static_cast<long long>(k.x) * max_blocks + k.y / block_size]) * block_size + k.y % block_size;
+  for (int v = lane; v < units; v += 32) out[i * units + v] = cache[slot * units + v];
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Attention over the cached rows. A CTA of eight warps has one query token, 16 MT heads (the rows of its MMA tiles) and one
+// range of keys, which come 64 at a time through a double-buffered cp.async ring. Per 64 keys: every warp computes the scores of
+// all heads with 8 keys (S = Q K^T over the whole row), the warps agree on the running maxima through shared memory, the softmax
+// weights go there as hi + lo bf16 pairs, and every warp accumulates 8 NT value columns (O += P V, V = the same rows).
+constexpr int kLatKeys = 64, kLatThreads = 256, kLatWarps = 8;
+
+struct LatentSmem {      // bytes
+  int pitch, q, p, m, total;
+};
+__host__ __device__ inline LatentSmem latent_smem(int row, int mt) {
+  LatentSmem s;
+  s.pitch = (row + 31) / 32 * 64 + 16;        // an odd number of 16-byte units: ldmatrix meets no bank twice
+  s.q = 2 * kLatKeys * s.pitch;
+  s.p = s.q + 16 * mt * s.pitch;
+  s.m = s.p + 2 * 16 * mt * (kLatKeys * 2 + 16);
+  s.total = s.m + 16 * mt * kLatWarps * 4;
+  return s;
+}
+
+template <int NT, int MT>
+__global__ void __launch_bounds__(kLatThreads)
+latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, const int* __restrict__ block_tables,
+                   int max_blocks, const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len,
+                   int block_size, int n, int heads, int rankp, int row, float scale_log2, int window,
+                   const float* __restrict__ sink, int splits, bf16* __restrict__ out, float* __restrict__ part_o,
+                   float* __restrict__ part_lse) {
+  constexpr int PP = kLatKeys * 2 + 16;         // pitch of a row of P
+  extern __shared__ __align__(128) uint8_t smem[];
+  const LatentSmem L = latent_smem(row, MT);
+  const int i = blockIdx.x, h0 = blockIdx.y * 16 * MT, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = lane >> 2, tq = lane & 3;
+  const int b = rows != nullptr ? rows[i] : i;
+  const int len = ctx_len[b];
+  const int* bt = block_tables + static_cast<long long>(bt_row != nullptr ? bt_row[b] : b) * max_blocks;
+  const int lo = window > 0 ? max(0, len - window) : 0;
+  const int per = ((len - lo + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
+  const int c0 = min(len, lo + split * per), c1 = min(len, c0 + per);
+  const int ntile = (c1 - c0 + kLatKeys - 1) / kLatKeys;
+  const int nch = row / 8, k32 = (row + 31) / 32;
+  const uint32_t sb = smem_u32(smem), sq = sb + L.q, sp = sb + L.p;
+  float* s_m = reinterpret_cast<float*>(smem + L.m);      // [16 MT][warps]
+
+  // zeros where no copy ever writes: columns row .. 32 k32 of the keys and of the queries, and absent heads
+  const int tail = k32 * 4 - nch;                         // 16-byte units
+  for (int r = threadIdx.x; r < 2 * kLatKeys + 16 * MT; r += kLatThreads)
+    for (int c = 0; c < tail; ++c)
+      *reinterpret_cast<uint4*>(smem + r * L.pitch + (nch + c) * 16) = make_uint4(0, 0, 0, 0);
+  for (int r = warp; r < 16 * MT; r += kLatWarps) {
+    const bf16* src = q + (static_cast<long long>(h0 + r) * n + i) * row;
+    for (int c = lane; c < nch; c += 32)
+      *reinterpret_cast<uint4*>(smem + L.q + r * L.pitch + c * 16) =
+          h0 + r < heads ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
+  }
+
+  auto issue = [&](int j) {
+    if (j < ntile) {
+      const int tok0 = c0 + j * kLatKeys;
+      const uint32_t dst0 = sb + (j & 1) * kLatKeys * L.pitch;
+      // a warp fetches rows 8 warp .. 8 warp + 7; lane r < 8 looks up the slot of row r
+      long long slot = 0;
+      const int key = tok0 + warp * 8 + (lane & 7);
+      if (key < c1) slot = static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
+      int r = 0, c = lane;
+      while (c >= nch) { c -= nch; ++r; }
+      for (int x = lane; x - lane < 8 * nch; x += 32) {   // the whole warp iterates: the shuffle needs every lane
+        const int rr = r < 8 ? r : 7;
+        const long long s = __shfl_sync(0xffffffffu, slot, rr);
+        if (x < 8 * nch)
+          cp_async16(dst0 + (warp * 8 + r) * L.pitch + c * 16, cache + s * row + c * 8, tok0 + warp * 8 + r < c1);
+        c += 32;
+        while (c >= nch) { c -= nch; ++r; }
+      }
+    }
+    cp_async_commit();
+  };
+  issue(0);
+
+  float o[MT][NT][4];
+  float m[MT][2], l[MT][2];
+#pragma unroll
+  for (int t = 0; t < MT; ++t) {
+    m[t][0] = m[t][1] = -INFINITY;
+    l[t][0] = l[t][1] = 0.f;
+#pragma unroll
+    for (int x = 0; x < NT; ++x) o[t][x][0] = o[t][x][1] = o[t][x][2] = o[t][x][3] = 0.f;
+  }
+  const int lm_mi = lane >> 3, lm_r = lane & 7;
+  const int col0 = warp * NT * 8;                         // this warp's value columns
+
+  for (int j = 0; j < ntile; ++j) {
+    cp_async_wait<0>();
+    __syncthreads();                    // tile j has landed; everyone is done with tile j - 1
+    issue(j + 1);
+    const uint32_t kb = sb + (j & 1) * kLatKeys * L.pitch;
+    float s[MT][4];
+#pragma unroll
+    for (int t = 0; t < MT; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
+    const uint32_t kaddr = kb + (warp * 8 + lm_r) * L.pitch + lm_mi * 16;
+    const uint32_t qaddr = sq + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
+#pragma unroll 2
+    for (int k = 0; k < k32; ++k) {
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
+#pragma unroll
+      for (int t = 0; t < MT; ++t) {
+        uint32_t a0[4], a1[4];
+        ldmatrix_x4(qaddr + t * 16 * L.pitch + k * 64, a0[0], a0[1], a0[2], a0[3]);
+        ldmatrix_x4(qaddr + t * 16 * L.pitch + k * 64 + 32, a1[0], a1[1], a1[2], a1[3]);
+        mma_bf16_16816(s[t], a0, b0, b1);
+        mma_bf16_16816(s[t], a1, b2, b3);
+      }
+    }
+    const int key = c0 + j * kLatKeys + warp * 8 + 2 * tq;
+    const bool v0 = key < c1, v1 = key + 1 < c1;
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+      s[t][0] = v0 ? s[t][0] * scale_log2 : -INFINITY;
+      s[t][1] = v1 ? s[t][1] * scale_log2 : -INFINITY;
+      s[t][2] = v0 ? s[t][2] * scale_log2 : -INFINITY;
+      s[t][3] = v1 ? s[t][3] * scale_log2 : -INFINITY;
+      float x0 = fmaxf(s[t][0], s[t][1]), x1 = fmaxf(s[t][2], s[t][3]);
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+      if (tq == 0) {
+        s_m[(t * 16 + g) * kLatWarps + warp] = x0;
+        s_m[(t * 16 + g + 8) * kLatWarps + warp] = x1;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float4* pm = reinterpret_cast<const float4*>(s_m + (t * 16 + g + 8 * e) * kLatWarps);
+        const float4 x = pm[0], z = pm[1];
+        // finite: the first key of the tile is visible
+        const float mn = fmaxf(m[t][e], fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(z.x, z.y), fmaxf(z.z, z.w))));
+        const float corr = exp2f(m[t][e] - mn);
+        m[t][e] = mn;
+        const float p0 = exp2f(s[t][2 * e] - mn), p1 = exp2f(s[t][2 * e + 1] - mn);
+        l[t][e] = l[t][e] * corr + p0 + p1;               // of this lane's keys; the lanes add up at the end
+        uint32_t hi, lo2;
+        split2(p0, p1, hi, lo2);
+        uint8_t* pr = smem + L.p + (t * 16 + g + 8 * e) * PP + (warp * 8 + 2 * tq) * 2;
+        *reinterpret_cast<uint32_t*>(pr) = hi;
+        *reinterpret_cast<uint32_t*>(pr + 16 * MT * PP) = lo2;
+#pragma unroll
+        for (int x2 = 0; x2 < NT; ++x2) { o[t][x2][2 * e] *= corr; o[t][x2][2 * e + 1] *= corr; }
+      }
+    }
+    __syncthreads();
+    if (col0 < rankp) {
+#pragma unroll
+      for (int ks = 0; ks < kLatKeys / 16; ++ks) {
+        uint32_t ph[MT][4], pl[MT][4];
+#pragma unroll
+        for (int t = 0; t < MT; ++t) {
+          const uint32_t pa = sp + (t * 16 + lm_r + (lm_mi & 1) * 8) * PP + ks * 32 + (lm_mi >> 1) * 16;
+          ldmatrix_x4(pa, ph[t][0], ph[t][1], ph[t][2], ph[t][3]);
+          ldmatrix_x4(pa + 16 * MT * PP, pl[t][0], pl[t][1], pl[t][2], pl[t][3]);
+        }
+        const uint32_t va = kb + (ks * 16 + (lm_mi & 1) * 8 + lm_r) * L.pitch + col0 * 2 + (lm_mi >> 1) * 16;
+#pragma unroll
+        for (int dp = 0; dp < NT / 2; ++dp) {
+          if (col0 + dp * 16 < rankp) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(va + dp * 32, b0, b1, b2, b3);
+#pragma unroll
+            for (int t = 0; t < MT; ++t) {
+              mma_bf16_16816(o[t][2 * dp], ph[t], b0, b1);
+              mma_bf16_16816(o[t][2 * dp + 1], ph[t], b2, b3);
+              mma_bf16_16816(o[t][2 * dp], pl[t], b0, b1);
+              mma_bf16_16816(o[t][2 * dp + 1], pl[t], b2, b3);
+            }
+          }
+        }
+      }
+    }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // denominators: lanes of a row, then warps
+#pragma unroll
+  for (int t = 0; t < MT; ++t)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float x = l[t][e];
+      x += __shfl_xor_sync(0xffffffffu, x, 1);
+      x += __shfl_xor_sync(0xffffffffu, x, 2);
+      if (tq == 0) s_m[(t * 16 + g + 8 * e) * kLatWarps + warp] = x;
+    }
+  __syncthreads();
+#pragma unroll
+  for (int t = 0; t < MT; ++t)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int head = h0 + t * 16 + g + 8 * e;
+      if (head >= heads) continue;
+      float den = 0.f;
+#pragma unroll
+      for (int w = 0; w < kLatWarps; ++w) den += s_m[(t * 16 + g + 8 * e) * kLatWarps + w];
+      float mm = m[t][e], f = 1.f;
+      if (sink != nullptr && split == 0 && len > 0) {     // one split carries the sink
+        const float sk = sink[head] * kLog2e, mn = fmaxf(mm, sk);
+        f = exp2f(mm - mn);
+        den = den * f + exp2f(sk - mn);
+        mm = mn;
+      }
+      f = den > 0.f ? f / den : 0.f;
+      const long long at = static_cast<long long>(head) * n + i;
+#pragma unroll
+      for (int x = 0; x < NT; ++x) {
+        const int col = col0 + x * 8 + 2 * tq;
+        if (col >= rankp) continue;
+        const float a = o[t][x][2 * e] * f, c = o[t][x][2 * e + 1] * f;
+        if (splits == 1) *reinterpret_cast<uint32_t*>(out + at * rankp + col) = pack_bf16(a, c);
+        else *reinterpret_cast<float2*>(part_o + (at * splits + split) * rankp + col) = make_float2(a, c);
+      }
+      if (splits > 1 && warp == 0 && tq == 0) part_lse[at * splits + split] = den > 0.f ? mm + log2f(den) : -INFINITY;
+    }
+}
+
+// out[at] = sum over splits of its softmax(lse)-weighted parts, at = (head, query)
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, int splits, int rankp,
+                    bf16* __restrict__ out) {
+  const long long at = blockIdx.x;
+  float M = -INFINITY;
+  for (int s = 0; s < splits; ++s) M = fmaxf(M, part_lse[at * splits + s]);
+  float L = 0.f;
+  if (M > -INFINITY)
+    for (int s = 0; s < splits; ++s) L += exp2f(part_lse[at * splits + s] - M);
+  const float inv = L > 0.f ? 1.f / L : 0.f;
+  for (int d = threadIdx.x * 2; d < rankp; d += blockDim.x * 2) {
+    float x = 0.f, y = 0.f;
+    if (L > 0.f)
+      for (int s = 0; s < splits; ++s) {
+        const float w = exp2f(part_lse[at * splits + s] - M);
+        if (w == 0.f) continue;
+        const float2 v = *reinterpret_cast<const float2*>(part_o + (at * splits + s) * rankp + d);
+        x += w * v.x;
+        y += w * v.y;
+      }
+    *reinterpret_cast<uint32_t*>(out + at * rankp + d) = pack_bf16(x * inv, y * inv);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Prompt runs over expanded keys and values: a CTA of four warps has 64 consecutive tokens of one head (16 per warp as MMA
+// rows), keys 64 at a time, double buffered. KD / VD: key (unrotated + rotated) and value sizes rounded up to the tile's.
+constexpr int kLpKeys = 64;
+
+template <int KD, int VD>
+__global__ void __launch_bounds__(128)
+latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __restrict__ kv, long long ld_kv,
+                      const bf16* __restrict__ lat, long long ld_lat, const int4* __restrict__ tiles, const int* __restrict__ base,
+                      int dimp, int rotp, int rankp, int vdimp, float scale_log2, int window, const float* __restrict__ sink,
+                      bf16* __restrict__ out, long long ld_out) {
+  constexpr int KP = KD * 2 + 16, VP = VD * 2 + 16;       // row pitches: odd numbers of 16-byte units
+  constexpr int STAGE = kLpKeys * (KP + VP);
+  constexpr int KS = KD / 16, NT = VD / 8;
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int4 tile = tiles[blockIdx.x];
+  const int row0 = tile.x, ntok = tile.y, pos0 = tile.w, head = blockIdx.y;
+  const long long kbase = base[blockIdx.x];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = lane >> 2, tq = lane & 3;
+  const int kmax = pos0 + ntok, klo = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int kb0 = klo / kLpKeys, nkb = (kmax + kLpKeys - 1) / kLpKeys;
+  const int qd = dimp + rotp, hw = dimp + vdimp;
+  const uint32_t sbase = smem_u32(smem);
+
+  auto issue = [&](int kb) {
+    if (kb < nkb) {
+      const uint32_t dst = sbase + (kb & 1) * STAGE;
+      for (int id = threadIdx.x; id < kLpKeys * (KD / 8); id += 128) {
+        const int r = id / (KD / 8), c = id % (KD / 8) * 8;
+        const int key = kb * kLpKeys + r;
+        const bool valid = key >= klo && key < kmax && c < qd;
+        const long long kr = valid ? kbase + key : 0;
+        const bf16* src = c < dimp ? kv + kr * ld_kv + head * hw + c : lat + kr * ld_lat + rankp + (valid ? c - dimp : 0);
+        cp_async16(dst + r * KP + c * 2, src, valid);
+      }
+      for (int id = threadIdx.x; id < kLpKeys * (VD / 8); id += 128) {
+        const int r = id / (VD / 8), c = id % (VD / 8) * 8;
+        const int key = kb * kLpKeys + r;
+        const bool valid = key >= klo && key < kmax && c < vdimp;
+        const long long kr = valid ? kbase + key : 0;
+        cp_async16(dst + kLpKeys * KP + r * VP + c * 2, kv + kr * ld_kv + head * hw + dimp + (valid ? c : 0), valid);
+      }
+    }
+    cp_async_commit();
+  };
+  issue(kb0);
+
+  // rows R0 and R0 + 8 of this warp's tile are tokens t0, t1
+  const int t0 = warp * 16 + g, t1 = t0 + 8;
+  const bool v0 = t0 < ntok, v1 = t1 < ntok;
+  const int qpos0 = pos0 + t0, qpos1 = pos0 + t1;
+  uint32_t qa[KS][4];
+  {
+    const bf16* q0 = q + static_cast<long long>(row0 + t0) * ld_q + head * qd;
+    const bf16* q1 = q + static_cast<long long>(row0 + t1) * ld_q + head * qd;
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+      const int c = ks * 16 + 2 * tq;
+      qa[ks][0] = v0 && c < qd ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
+      qa[ks][1] = v1 && c < qd ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
+      qa[ks][2] = v0 && c + 8 < qd ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
+      qa[ks][3] = v1 && c + 8 < qd ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+    }
+  }
+  float o[NT][4];
+#pragma unroll
+  for (int x = 0; x < NT; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const int lm_mi = lane >> 3, lm_r = lane & 7;
+  const int wlast = pos0 + min(ntok - 1, warp * 16 + 15);           // last query of the warp, first key of its first query
+  const int wfirst = window > 0 ? pos0 + warp * 16 - window + 1 : 0;
+  const int lo0 = window > 0 ? qpos0 - window + 1 : 0, lo1 = window > 0 ? qpos1 - window + 1 : 0;
+
+  for (int kb = kb0; kb < nkb; ++kb) {
+    issue(kb + 1);
+    cp_async_wait<1>();
+    __syncthreads();
+    const uint32_t kbuf = sbase + (kb & 1) * STAGE, vbuf = kbuf + kLpKeys * KP;
+    const int key0 = kb * kLpKeys;
+    if (key0 <= wlast && warp * 16 < ntok && key0 + kLpKeys > wfirst) {
+      float s[8][4];
+#pragma unroll
+      for (int x = 0; x < 8; ++x) s[x][0] = s[x][1] = s[x][2] = s[x][3] = 0.f;
+#pragma unroll
+      for (int kg = 0; kg < 4; ++kg) {
+        const uint32_t ka = kbuf + (kg * 16 + (lm_mi >> 1) * 8 + lm_r) * KP + (lm_mi & 1) * 16;
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(ka + ks * 32, b0, b1, b2, b3);
+          mma_bf16_16816(s[2 * kg], qa[ks], b0, b1);
+          mma_bf16_16816(s[2 * kg + 1], qa[ks], b2, b3);
+        }
+      }
+      float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        const int k0 = key0 + x * 8 + 2 * tq, k1 = k0 + 1;
+        s[x][0] = v0 && k0 <= qpos0 && k0 >= lo0 ? s[x][0] * scale_log2 : -INFINITY;
+        s[x][1] = v0 && k1 <= qpos0 && k1 >= lo0 ? s[x][1] * scale_log2 : -INFINITY;
+        s[x][2] = v1 && k0 <= qpos1 && k0 >= lo1 ? s[x][2] * scale_log2 : -INFINITY;
+        s[x][3] = v1 && k1 <= qpos1 && k1 >= lo1 ? s[x][3] * scale_log2 : -INFINITY;
+        mx0 = fmaxf(mx0, fmaxf(s[x][0], s[x][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[x][2], s[x][3]));
+      }
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+      const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+      // a row with nothing visible yet keeps -inf: subtract 0 instead so that exp2 gives 0, not NaN
+      const float sub0 = mn0 == -INFINITY ? 0.f : mn0, sub1 = mn1 == -INFINITY ? 0.f : mn1;
+      const float corr0 = exp2f(m0 - sub0), corr1 = exp2f(m1 - sub1);
+      float ls0 = 0.f, ls1 = 0.f;
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        s[x][0] = exp2f(s[x][0] - sub0); s[x][1] = exp2f(s[x][1] - sub0);
+        s[x][2] = exp2f(s[x][2] - sub1); s[x][3] = exp2f(s[x][3] - sub1);
+        ls0 += s[x][0] + s[x][1];
+        ls1 += s[x][2] + s[x][3];
+      }
+      ls0 += __shfl_xor_sync(0xffffffffu, ls0, 1);
+      ls0 += __shfl_xor_sync(0xffffffffu, ls0, 2);
+      ls1 += __shfl_xor_sync(0xffffffffu, ls1, 1);
+      ls1 += __shfl_xor_sync(0xffffffffu, ls1, 2);
+      l0 = l0 * corr0 + ls0;
+      l1 = l1 * corr1 + ls1;
+      m0 = mn0;
+      m1 = mn1;
+#pragma unroll
+      for (int x = 0; x < NT; ++x) { o[x][0] *= corr0; o[x][1] *= corr0; o[x][2] *= corr1; o[x][3] *= corr1; }
+#pragma unroll
+      for (int kg = 0; kg < 4; ++kg) {
+        uint32_t ph[4], pl[4];
+        split2(s[2 * kg][0], s[2 * kg][1], ph[0], pl[0]);
+        split2(s[2 * kg][2], s[2 * kg][3], ph[1], pl[1]);
+        split2(s[2 * kg + 1][0], s[2 * kg + 1][1], ph[2], pl[2]);
+        split2(s[2 * kg + 1][2], s[2 * kg + 1][3], ph[3], pl[3]);
+        const uint32_t va = vbuf + (kg * 16 + (lm_mi & 1) * 8 + lm_r) * VP + (lm_mi >> 1) * 16;
+#pragma unroll
+        for (int dp = 0; dp < NT / 2; ++dp) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(va + dp * 32, b0, b1, b2, b3);
+          mma_bf16_16816(o[2 * dp], ph, b0, b1);
+          mma_bf16_16816(o[2 * dp + 1], ph, b2, b3);
+          mma_bf16_16816(o[2 * dp], pl, b0, b1);
+          mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
+        }
+      }
+    }
+    __syncthreads();   // every warp is done with this stage before it is refilled
+  }
+  cp_async_wait<0>();
+  float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  if (sink != nullptr) {
+    const float sk = sink[head] * kLog2e;
+    const float M0 = fmaxf(m0, sk), M1 = fmaxf(m1, sk), f0 = exp2f(m0 - M0), f1 = exp2f(m1 - M1);
+    inv0 = f0 / (l0 * f0 + exp2f(sk - M0));
+    inv1 = f1 / (l1 * f1 + exp2f(sk - M1));
+  }
+  bf16* o0 = out + static_cast<long long>(row0 + t0) * ld_out + head * vdimp;
+  bf16* o1 = out + static_cast<long long>(row0 + t1) * ld_out + head * vdimp;
+#pragma unroll
+  for (int x = 0; x < NT; ++x) {
+    const int col = x * 8 + 2 * tq;
+    if (col >= vdimp) continue;
+    if (v0) *reinterpret_cast<uint32_t*>(o0 + col) = pack_bf16(o[x][0] * inv0, o[x][1] * inv0);
+    if (v1) *reinterpret_cast<uint32_t*>(o1 + col) = pack_bf16(o[x][2] * inv1, o[x][3] * inv1);
+  }
+}
+
+template <int NT, int MT>
+static int launch_latent(const void* q, const void* cache, const int* bt, int max_blocks, const int* bt_row, const int* rows,
+                         const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale, int window,
+                         const float* sink, int splits, void* out, float* ws, cudaStream_t stream) {
+  static PerDeviceOnce configured;
+  const int rc = configured.run([] {
+    return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+  });
+  if (rc != 0) return rc;
+  const int smem = latent_smem(row, MT).total;
+  if (smem > 227 * 1024) return -11;
+  const long long at = static_cast<long long>(heads) * n;
+  float* part_lse = ws != nullptr ? ws + at * splits * rankp : nullptr;
+  latent_attn_kernel<NT, MT><<<dim3(n, (heads + 16 * MT - 1) / (16 * MT), splits), kLatThreads, smem, stream>>>(
+      static_cast<const bf16*>(q), static_cast<const bf16*>(cache), bt, max_blocks, bt_row, rows, ctx_len, block_size, n, heads,
+      rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse);
+  if (splits > 1)
+    latent_merge_kernel<<<static_cast<unsigned>(at), 128, 0, stream>>>(ws, part_lse, splits, rankp, static_cast<bf16*>(out));
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int KD, int VD>
+static int launch_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
+                                 const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp,
+                                 int vdimp, float scale, int window, const float* sink, void* out, long long ld_out,
+                                 cudaStream_t stream) {
+  constexpr int smem = 2 * kLpKeys * (KD * 2 + VD * 2 + 32);
+  static PerDeviceOnce configured;
+  const int rc = configured.run([] {
+    return static_cast<int>(cudaFuncSetAttribute(latent_prefill_kernel<KD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  });
+  if (rc != 0) return rc;
+  latent_prefill_kernel<KD, VD><<<dim3(n_tiles, heads), 128, smem, stream>>>(
+      static_cast<const bf16*>(q), ld_q, static_cast<const bf16*>(kv), ld_kv, static_cast<const bf16*>(lat), ld_lat,
+      static_cast<const int4*>(tiles), base, dimp, rotp, rankp, vdimp, scale * kLog2e, window, sink, static_cast<bf16*>(out), ld_out);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace dmoe
+
+using namespace dmoe;
+
+extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
+                                int heads, int dim, int rot_dim, int rank, int rot, int interleaved, const void* table,
+                                int max_pos, const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa,
+                                void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (heads < 1 || dim < 1 || rot_dim < 0 || rank < 1 || rot < 0 || rot % 2 != 0 || rot > rot_dim || (rot > 0 && table == nullptr)) return -10;
+  const int align = is_f32 ? 4 : 8;
+  if (ld % align != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 || (loose == nullptr && n_loose < T)) return -10;
+  if (T == 0) return 0;
+  const int dimp = pad8(dim), rotp = pad8(rot_dim), rankp = pad8(rank);
+  if (is_f32)
+    latent_prep_kernel<float><<<T, 256, 0, stream>>>(
+        static_cast<float*>(y), ld, positions, slots, static_cast<float*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,
+        static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<float*>(xq), static_cast<float*>(qa));
+  else
+    latent_prep_kernel<bf16><<<T, 256, 0, stream>>>(
+        static_cast<bf16*>(y), ld, positions, slots, static_cast<bf16*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,
+        static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<bf16*>(xq), static_cast<bf16*>(qa));
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
+                                     const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row,
+                                     float scale, int window, const float* sink, int splits, void* out, float* workspace,
+                                     void* stream_) {
+  if (heads < 1 || heads > 65535 || rankp < 8 || rankp % 8 != 0 || row % 8 != 0 || row < rankp || rankp > 512 || row > 640) return -10;
+  if (block_size < 1 || splits < 1 || splits > 65535 || (splits > 1 && workspace == nullptr)) return -10;
+  if (n == 0) return 0;
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+#define DMOE_LAT(NT_, MT_)                                                                                              \
+  return launch_latent<NT_, MT_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, \
+                                 row, scale, window, sink, splits, out, workspace, stream)
+  if (heads <= 16) {
+    if (rankp <= 128) DMOE_LAT(2, 1);
+    if (rankp <= 256) DMOE_LAT(4, 1);
+    DMOE_LAT(8, 1);
+  }
+  if (rankp <= 128) DMOE_LAT(2, 2);
+  if (rankp <= 256) DMOE_LAT(4, 2);
+  DMOE_LAT(8, 2);
+#undef DMOE_LAT
+}
+
+extern "C" int dmoe_latent_gather(const void* cache, const int* block_tables, int max_blocks, const void* keys, int n,
+                                  int block_size, int row, void* out, void* stream) {
+  if (row < 8 || row % 8 != 0 || block_size < 1) return -10;
+  if (n == 0) return 0;
+  latent_gather_kernel<<<(n + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(cache), block_tables, max_blocks, static_cast<const int2*>(keys), n, block_size, row / 8,
+      static_cast<uint4*>(out));
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dmoe_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
+                                   const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp,
+                                   int vdimp, float scale, int window, const float* sink, void* out, long long ld_out,
+                                   void* stream_) {
+  if (n_tiles == 0) return 0;
+  if (n_tiles < 0 || heads < 1 || heads > 65535 || dimp % 8 != 0 || rotp % 8 != 0 || rankp % 8 != 0 || vdimp % 8 != 0) return -10;
+  if (ld_q % 8 != 0 || ld_kv % 8 != 0 || ld_lat % 8 != 0 || ld_out % 8 != 0 || tiles == nullptr || base == nullptr) return -10;
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  const int kd = dimp + rotp;
+#define DMOE_LP(KD_, VD_)                                                                                               \
+  if (kd <= KD_ && vdimp <= VD_)                                                                                        \
+    return launch_latent_prefill<KD_, VD_>(q, ld_q, kv, ld_kv, lat, ld_lat, tiles, base, n_tiles, heads, dimp, rotp, rankp, \
+                                           vdimp, scale, window, sink, out, ld_out, stream)
+  DMOE_LP(96, 64);
+  DMOE_LP(128, 128);
+  DMOE_LP(192, 128);
+#undef DMOE_LP
+  return -11;
+}

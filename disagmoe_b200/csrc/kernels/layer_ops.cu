@@ -1,7 +1,8 @@
 // Row kernels of decoders whose residual stream is kept in fp32, for bf16 and fp32 activations: scaled embedding,
-// post-norm + residual add + pre-norm in one pass, per-head query / key norm + partial rotary embedding + paged KV
-// append, rotary table from arbitrary frequencies, silu(gate) * up, and a CUDA-core GEMM for fp32 operands (and for bf16
-// shapes the tcgen05 kernel's TMA cannot address).
+// post-norm + residual add + pre-norm in one pass, residual sum + norm + softmax router in one pass, per-head query / key
+// norm + partial rotary embedding + value mixing + paged KV append, rotary table from arbitrary frequencies, act(gate) * up,
+// and a CUDA-core GEMM, dense or over row groups, for fp32 operands (and for bf16 shapes the tcgen05 kernel's TMA cannot
+// address).
 #include "dmoe_kernels.h"
 #include "sm100.cuh"
 
@@ -145,6 +146,169 @@ resid_norm_kernel(float* __restrict__ resid, const T* __restrict__ y, long long 
   }
 }
 
+// Residual sum, norm and (optionally) router of blocks whose sublayers share a norm, TPC rows per CTA of 256 threads:
+//   x = resid[r] + y[r] + sum_p parts[r, p];  resid[r] = x (unless a row table picks the rows);  h = norm(x) * w
+//   router: logits = gate_w h, softmax, the K largest (lowest index first among equals).
+// The rows stay in shared memory (fp32) from the sum on; with several rows per CTA the router's weights are fetched once for
+// all of them.
+struct SumNormArgs {
+  float* resid;
+  const void* y;
+  long long ld_y;
+  const void* parts;
+  int n_parts;
+  long long part_row, part_stride;
+  const float* w;
+  int centred;
+  float eps;
+  const int* rows;
+  void* h;
+  long long ld_h;
+  int n, W;
+  const void* gate_w;
+  int E, K, renorm;
+  int* ids;
+  float* wts;
+  int* counts;
+};
+constexpr int kSumThreads = 256, kSumWarps = kSumThreads / 32;
+constexpr int kMaxExperts = 256, kMaxTop = 32;
+
+template <typename T, int VEC, int TPC>
+__global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs a) {
+  constexpr int G = kSumThreads / TPC, GW = G / 32;       // threads / warps per row
+  extern __shared__ __align__(16) float s_row[];          // [TPC][W]
+  __shared__ float red[kSumWarps];
+  __shared__ float slog[TPC][kMaxExperts];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j = threadIdx.x / G, tid = threadIdx.x % G;
+  const int W = a.W, nvec = W / VEC;
+  const long long i = static_cast<long long>(blockIdx.x) * TPC + j;
+  const bool valid = i < a.n;
+  const long long r = !valid ? 0 : a.rows != nullptr ? a.rows[i] : i;
+  float* row = s_row + static_cast<long long>(j) * W;
+  const T* y = static_cast<const T*>(a.y);
+  const T* parts = static_cast<const T*>(a.parts);
+  auto group_sum = [&](float v) {       // over the threads of one row; all threads of the CTA call it
+    v = warp_sum(v);
+    if (GW == 1) return v;
+    __syncthreads();
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int k = 0; k < GW; ++k) t += red[j * GW + k];
+    return t;
+  };
+
+  float sum = 0.f;
+  if (valid) {
+    for (int v = tid; v < nvec; v += G) {
+      float x[VEC], t[VEC];
+      Pack<float, VEC>::load(a.resid + r * W + v * VEC, x);
+      if (y != nullptr) {
+        Pack<T, VEC>::load(y + r * a.ld_y + v * VEC, t);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += t[e];
+      }
+      for (int p = 0; p < a.n_parts; ++p) {
+        Pack<T, VEC>::load(parts + r * a.part_row + p * a.part_stride + v * VEC, t);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += t[e];
+      }
+      if (a.rows == nullptr && (y != nullptr || a.n_parts > 0)) Pack<float, VEC>::store(a.resid + r * W + v * VEC, x);
+      Pack<float, VEC>::store(row + v * VEC, x);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum += x[e];
+    }
+  }
+  const float mean = a.centred ? group_sum(sum) / static_cast<float>(W) : 0.f;
+  float ss = 0.f;
+  if (valid)
+    for (int v = tid; v < nvec; v += G)        // every thread reads back what it wrote itself
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float d = row[v * VEC + e] - mean;
+        ss += d * d;
+      }
+  const float inv = 1.f / sqrtf(group_sum(ss) / static_cast<float>(W) + a.eps);
+  if (valid)
+    for (int v = tid; v < nvec; v += G) {
+      float x[VEC], w[VEC];
+      Pack<float, VEC>::load(row + v * VEC, x);
+      Pack<float, VEC>::load(a.w + v * VEC, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = (x[e] - mean) * inv * w[e];
+      Pack<T, VEC>::store(static_cast<T*>(a.h) + i * a.ld_h + v * VEC, x);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = static_cast<float>(static_cast<T>(x[e]));
+      Pack<float, VEC>::store(row + v * VEC, x);
+    }
+  if (a.gate_w == nullptr) return;
+  __syncthreads();
+
+  const T* gate = static_cast<const T*>(a.gate_w);
+  for (int e = warp; e < a.E; e += kSumWarps) {
+    float acc[TPC] = {};
+    for (int v = lane; v < nvec; v += 32) {
+      float g[VEC];
+      Pack<T, VEC>::load(gate + static_cast<long long>(e) * W + v * VEC, g);
+#pragma unroll
+      for (int t = 0; t < TPC; ++t) {
+        float x[VEC];
+        Pack<float, VEC>::load(s_row + static_cast<long long>(t) * W + v * VEC, x);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) acc[t] += g[k] * x[k];
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < TPC; ++t) {
+      const float z = warp_sum(acc[t]);
+      if (lane == 0) slog[t][e] = z;
+    }
+  }
+  __syncthreads();
+  const long long tok = static_cast<long long>(blockIdx.x) * TPC + warp;
+  if (warp >= TPC || tok >= a.n) return;
+  float* lg = slog[warp];
+  float mx = -INFINITY;
+  for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, lg[e]);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  float den = 0.f;
+  for (int e = lane; e < a.E; e += 32) den += expf(lg[e] - mx);
+  den = warp_sum(den);
+  int my_id = -1;           // lane k keeps the k-th choice
+  float my_w = 0.f, total = 0.f;
+  for (int k = 0; k < a.K; ++k) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < a.E; e += 32)
+      if (lg[e] > best) { best = lg[e]; bi = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    float s = expf(best - mx) / den;
+    if (bi >= a.E) {        // no finite logit left: the lowest expert not chosen yet, so that the ids stay valid
+      for (bi = 0; __any_sync(0xffffffffu, my_id == bi);) ++bi;
+      s = 0.f;
+    }
+    if (lane == k) { my_id = bi; my_w = s; }
+    total += s;
+    __syncwarp();
+    if (lane == 0) lg[bi] = -INFINITY;
+    __syncwarp();
+  }
+  if (lane < a.K) {
+    a.ids[tok * a.K + lane] = my_id;
+    a.wts[tok * a.K + lane] = a.renorm && total > 0.f ? my_w / total : my_w;
+    if (a.counts != nullptr) atomicAdd(&a.counts[my_id], 1);
+  }
+}
+
 // table[pos][i] = (cos, sin)(pos * freq[i]) * mscale, angles and functions in double precision
 __global__ void rope_freq_table_kernel(float2* __restrict__ table, int max_pos, int half, const double* __restrict__ freq,
                                        float mscale) {
@@ -155,15 +319,17 @@ __global__ void rope_freq_table_kernel(float2* __restrict__ table, int max_pos, 
   table[i] = make_float2(static_cast<float>(c * mscale), static_cast<float>(s * mscale));
 }
 
-// rows [q heads | k heads | v heads] (the last two only where n_kv > 0): RMS norm over each q / k head with its weight,
-// rotation of the pairs (i, i + rot / 2), i < rot / 2, q written back in place, k and v appended to the paged caches
-// ([blocks, block_size, n_kv, dk] and [.., dv]) at slots[t] (< 0: skip). One warp per head.
+// rows [q heads | k heads | v heads] (the last two only where n_kv > 0): RMS norm over each q / k head with its weight (qw !=
+// NULL), rotation of the pairs (i, i + rot / 2) or, interleaved, (2i, 2i + 1), i < rot / 2, q written back in place, k and v
+// appended to the paged caches ([blocks, block_size, n_kv, dk] and [.., dv]) at slots[t] (< 0: skip). v_first != NULL: what is
+// appended is (1 - lambda) v + lambda v_first (head size first_head in memory). One warp per head.
 template <typename T>
 __global__ void __launch_bounds__(256)
 qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ positions,
                     const long long* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache, int n_q, int n_kv,
-                    int dk, int dv, int rot, const float2* __restrict__ table, int max_pos, const float* __restrict__ qw,
-                    const float* __restrict__ kw, float eps) {
+                    int dk, int dv, int rot, int interleaved, const float2* __restrict__ table, int max_pos,
+                    const float* __restrict__ qw, const float* __restrict__ kw, float eps, const T* __restrict__ v_first,
+                    long long ld_first, int first_head, float v_lambda) {
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int half = rot / 2;
@@ -177,53 +343,85 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
     if (!is_q && slot < 0) continue;
     const float* w = is_q ? qw : kw;
     T* dst = is_q ? p : kcache + (slot * n_kv + (head - n_q)) * dk;
-    float ss = 0.f;
-    for (int d = lane; d < dk; d += 32) {
-      const float x = static_cast<float>(p[d]);
-      ss += x * x;
+    float inv = 1.f;
+    if (w != nullptr) {
+      float ss = 0.f;
+      for (int d = lane; d < dk; d += 32) {
+        const float x = static_cast<float>(p[d]);
+        ss += x * x;
+      }
+      inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(dk) + eps);
     }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(dk) + eps);
     for (int i = lane; i < half; i += 32) {
-      const float u = static_cast<float>(p[i]) * inv * w[i], v = static_cast<float>(p[i + half]) * inv * w[i + half];
+      const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
+      float u = static_cast<float>(p[a]), v = static_cast<float>(p[b]);
+      if (w != nullptr) { u *= inv * w[a]; v *= inv * w[b]; }
       const float2 cs = tab[i];
-      dst[i] = static_cast<T>(u * cs.x - v * cs.y);
-      dst[i + half] = static_cast<T>(v * cs.x + u * cs.y);
+      dst[a] = static_cast<T>(u * cs.x - v * cs.y);
+      dst[b] = static_cast<T>(v * cs.x + u * cs.y);
     }
-    for (int d = rot + lane; d < dk; d += 32) dst[d] = static_cast<T>(static_cast<float>(p[d]) * inv * w[d]);
+    if (w == nullptr && is_q) continue;         // the rest of the head is in place
+    for (int d = rot + lane; d < dk; d += 32) {
+      const float x = static_cast<float>(p[d]);
+      dst[d] = static_cast<T>(w != nullptr ? x * inv * w[d] : x);
+    }
   }
   if (slot >= 0) {
     const T* src = row + static_cast<long long>(n_q + n_kv) * dk;
     T* dst = vcache + slot * n_kv * dv;
-    for (int i = threadIdx.x; i < n_kv * dv; i += blockDim.x) dst[i] = src[i];
+    for (int i = threadIdx.x; i < n_kv * dv; i += blockDim.x) {
+      if (v_first == nullptr) { dst[i] = src[i]; continue; }
+      const int d = i % dv;
+      const float first = d < first_head ? static_cast<float>(v_first[t * ld_first + i / dv * first_head + d]) : 0.f;
+      dst[i] = static_cast<T>((1.f - v_lambda) * static_cast<float>(src[i]) + v_lambda * first);
+    }
   }
 }
 
-// out[t, i] = silu(gu[t, i]) * gu[t, I + i]
+// out[t, i] = act(gu[t, i]) * gu[t, I + i]
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ld_out, int I) {
+__global__ void gate_mul_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ld_out, int I, int act) {
   const long long t = blockIdx.y;
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= I) return;
   const float g = static_cast<float>(gu[t * ld + i]), u = static_cast<float>(gu[t * ld + I + i]);
-  out[t * ld_out + i] = static_cast<T>(g / (1.f + expf(-g)) * u);
+  const float v = act == 0 ? g / (1.f + expf(-g))
+                           : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+  out[t * ld_out + i] = static_cast<T>(v * u);
 }
 
-// Y[t, f] = sum_k X[t, k] W[f, k] with fp32 multiply-adds: 64 x 64 tiles, 4 x 4 outputs per thread.
+// Y[t, f] = sum_k X[t, k] W[f, k] with fp32 multiply-adds: 64 x 64 tiles, 4 x 4 outputs per thread. With offs, W is a stack of
+// G matrices [F, K] and group g has rows offs[g] .. offs[g + 1] (blockIdx.y counts row tiles group after group); with recs, row
+// t is scaled and stored where its record {buffer, row or < 0, weight bits, -} says.
 constexpr int kSgTile = 64, kSgK = 16;
 
 template <typename T, typename TY>
 __global__ void __launch_bounds__(256)
 simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw, TY* __restrict__ Y,
-                 long long ldy, int M, int F, int K) {
+                 long long ldy, int M, int F, int K, const int* __restrict__ offs, int G, const int4* __restrict__ recs,
+                 void* const* __restrict__ bases) {
   __shared__ float sx[kSgK][kSgTile + 4], sw[kSgK][kSgTile + 4];
-  const int t0 = blockIdx.y * kSgTile, f0 = blockIdx.x * kSgTile;
+  int t0 = blockIdx.y * kSgTile, t1 = M;
+  const int f0 = blockIdx.x * kSgTile;
+  if (offs != nullptr) {
+    int left = blockIdx.y, g = 0;
+    for (; g < G; ++g) {
+      const int tiles = (offs[g + 1] - offs[g] + kSgTile - 1) / kSgTile;
+      if (left < tiles) break;
+      left -= tiles;
+    }
+    if (g == G) return;
+    t0 = offs[g] + left * kSgTile;
+    t1 = min(M, offs[g + 1]);
+    W += static_cast<long long>(g) * F * ldw;
+  }
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kSgK) {
     for (int i = threadIdx.x; i < kSgTile * kSgK; i += 256) {
       const int r = i / kSgK, k = i % kSgK;
       const bool in_k = k0 + k < K;
-      sx[k][r] = in_k && t0 + r < M ? static_cast<float>(X[(t0 + r) * ldx + k0 + k]) : 0.f;
+      sx[k][r] = in_k && t0 + r < t1 ? static_cast<float>(X[(t0 + r) * ldx + k0 + k]) : 0.f;
       sw[k][r] = in_k && f0 + r < F ? static_cast<float>(W[(f0 + r) * ldw + k0 + k]) : 0.f;
     }
     __syncthreads();
@@ -242,11 +440,19 @@ simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int t = t0 + ty * 4 + i;
-    if (t >= M) continue;
+    if (t >= t1) continue;
+    TY* dst = Y + t * ldy;
+    float scale = 1.f;
+    if (recs != nullptr) {
+      const int4 rec = recs[t];
+      if (rec.y < 0) continue;
+      dst = static_cast<TY*>(bases[rec.x]) + rec.y * ldy;
+      scale = __int_as_float(rec.z);
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int f = f0 + tx * 4 + j;
-      if (f < F) Y[t * ldy + f] = static_cast<TY>(acc[i][j]);
+      if (f < F) dst[f] = static_cast<TY>(acc[i][j] * scale);
     }
   }
 }
@@ -269,6 +475,29 @@ static int launch_resid_norm(float* resid, const void* y, long long ld_y, const 
   else
     resid_norm_kernel<T, 1><<<n, threads, 0, stream>>>(resid, static_cast<const T*>(y), ld_y, post, pre, out_scale, eps, rows,
                                                        static_cast<T*>(h), ld_h, W);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int VEC>
+static int launch_sum_norm(const SumNormArgs& a, cudaStream_t stream) {
+  // rows per CTA: one until there are rows for all SMs; more where a router's weights are read for every CTA
+  const bool routed = a.gate_w != nullptr;
+  int tpc = !routed || a.n < 160 ? 1 : a.n < 640 ? 2 : 8;
+  while (tpc > 1 && static_cast<long long>(tpc) * a.W * 4 > 160 * 1024) tpc = tpc == 8 ? 2 : 1;
+  const size_t smem = static_cast<size_t>(tpc) * a.W * 4;
+  if (smem > 160 * 1024) return -10;
+  static PerDeviceOnce configured;
+  const int rc = configured.run([] {
+    int e = static_cast<int>(cudaFuncSetAttribute(sum_norm_kernel<T, VEC, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    if (e == 0) e = static_cast<int>(cudaFuncSetAttribute(sum_norm_kernel<T, VEC, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    if (e == 0) e = static_cast<int>(cudaFuncSetAttribute(sum_norm_kernel<T, VEC, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    return e;
+  });
+  if (rc != 0) return rc;
+  const unsigned grid = static_cast<unsigned>((a.n + tpc - 1) / tpc);
+  if (tpc == 8) sum_norm_kernel<T, VEC, 8><<<grid, kSumThreads, smem, stream>>>(a);
+  else if (tpc == 2) sum_norm_kernel<T, VEC, 2><<<grid, kSumThreads, smem, stream>>>(a);
+  else sum_norm_kernel<T, VEC, 1><<<grid, kSumThreads, smem, stream>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -307,39 +536,60 @@ extern "C" int dmoe_rope_freq_table(void* table, int max_pos, int half, const do
   return static_cast<int>(cudaGetLastError());
 }
 
+extern "C" int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
+                             long long part_row, long long part_stride, const float* w, int centred, float eps, const int* rows,
+                             void* h, long long ld_h, int n, int W, const void* gate_w, int E, int K, int renorm, int* ids,
+                             float* wts, int* counts, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (W < 1 || resid == nullptr || h == nullptr || w == nullptr || n_parts < 0) return -10;
+  if (gate_w != nullptr && (E < 1 || E > kMaxExperts || K < 1 || K > kMaxTop || K > E || ids == nullptr || wts == nullptr)) return -10;
+  if (n == 0) return 0;
+  if (parts == nullptr) n_parts = 0;
+  const SumNormArgs a{resid, y, ld_y, parts, n_parts, part_row, part_stride, w, centred, eps, rows, h, ld_h, n, W, gate_w, E, K,
+                      renorm, ids, wts, counts};
+  const bool vec = W % 8 == 0 && ld_y % 8 == 0 && ld_h % 8 == 0 && part_row % 8 == 0 && part_stride % 8 == 0 && aligned16(resid) &&
+                   aligned16(y) && aligned16(parts) && aligned16(w) && aligned16(h) && aligned16(gate_w);
+  if (is_f32) return vec ? launch_sum_norm<float, 8>(a, stream) : launch_sum_norm<float, 1>(a, stream);
+  return vec ? launch_sum_norm<bf16, 8>(a, stream) : launch_sum_norm<bf16, 1>(a, stream);
+}
+
 extern "C" int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots,
-                                 void* kcache, void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot,
-                                 const void* table, int max_pos, const float* qw, const float* kw, float eps, void* stream_) {
+                                 void* kcache, void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved,
+                                 const void* table, int max_pos, const float* qw, const float* kw, float eps,
+                                 const void* v_first, long long ld_first, int first_head, float v_lambda, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (n_q < 1 || n_kv < 0 || dk < 1 || rot < 0 || rot % 2 != 0 || rot > dk || (rot > 0 && table == nullptr)) return -10;
-  if (n_kv > 0 && (kcache == nullptr || vcache == nullptr || kw == nullptr)) return -10;
+  if (n_kv > 0 && (kcache == nullptr || vcache == nullptr || (qw != nullptr && kw == nullptr))) return -10;
+  if (v_first != nullptr && first_head < 1) return -10;
   if (T == 0) return 0;
   int threads = (n_q + n_kv) * 32;
   if (threads > 256) threads = 256;
   if (is_f32)
     qk_norm_rope_kernel<float><<<T, threads, 0, stream>>>(
         static_cast<float*>(qkv), ld, positions, slots, static_cast<float*>(kcache), static_cast<float*>(vcache), n_q, n_kv,
-        dk, dv, rot, static_cast<const float2*>(table), max_pos, qw, kw, eps);
+        dk, dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const float*>(v_first),
+        ld_first, first_head, v_lambda);
   else
     qk_norm_rope_kernel<bf16><<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk,
-        dv, rot, static_cast<const float2*>(table), max_pos, qw, kw, eps);
+        dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const bf16*>(v_first),
+        ld_first, first_head, v_lambda);
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int dmoe_silu_mul(int is_f32, const void* gu, long long ld, void* out, long long ld_out, int T, int I,
+extern "C" int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I,
                              void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (I < 1) return -10;
+  if (I < 1 || act < 0 || act > 1) return -10;
   for (int t0 = 0; t0 < T; t0 += 65535) {      // grid.y limit
     const int n = T - t0 < 65535 ? T - t0 : 65535;
     const dim3 grid((I + 255) / 256, n);
     if (is_f32)
-      silu_mul_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(gu) + t0 * ld, ld,
-                                                       static_cast<float*>(out) + t0 * ld_out, ld_out, I);
+      gate_mul_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(gu) + t0 * ld, ld,
+                                                       static_cast<float*>(out) + t0 * ld_out, ld_out, I, act);
     else
-      silu_mul_kernel<bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(gu) + t0 * ld, ld,
-                                                      static_cast<bf16*>(out) + t0 * ld_out, ld_out, I);
+      gate_mul_kernel<bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(gu) + t0 * ld, ld,
+                                                      static_cast<bf16*>(out) + t0 * ld_out, ld_out, I, act);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -354,12 +604,31 @@ extern "C" int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long l
   const dim3 grid((F + kSgTile - 1) / kSgTile, static_cast<unsigned>(ty));
   if (x_f32)
     simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W),
-                                                             ldw, static_cast<float*>(Y), ldy, T, F, K);
+                                                             ldw, static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
   else if (y_f32)
     simt_gemm_kernel<bf16, float><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                            static_cast<float*>(Y), ldy, T, F, K);
+                                                            static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
   else
     simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                           static_cast<bf16*>(Y), ldy, T, F, K);
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y,
+                                 long long ldy, const void* recs, const void* bases, int T, int F, int K, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (F < 1 || K < 1 || G < 1 || offs == nullptr || (recs == nullptr && Y == nullptr) || (recs != nullptr && bases == nullptr)) return -10;
+  if (T == 0) return 0;
+  const long long ty = (T + kSgTile - 1) / kSgTile + G;      // every group may end in a partial tile
+  if (ty > 65535) return -10;
+  const dim3 grid((F + kSgTile - 1) / kSgTile, static_cast<unsigned>(ty));
+  const int4* r = static_cast<const int4*>(recs);
+  void* const* b = static_cast<void* const*>(bases);
+  if (is_f32)
+    simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W), K,
+                                                             static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b);
+  else
+    simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), K,
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, offs, G, r, b);
   return static_cast<int>(cudaGetLastError());
 }

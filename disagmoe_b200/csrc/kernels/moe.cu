@@ -202,9 +202,11 @@ route_kernel(const __nv_bfloat16* __restrict__ x, long long ld_x, const __nv_bfl
 // Row placement: row_base[e] + slot, where row_base[e] is the exclusive prefix of counts restricted to the
 // experts of the same destination rank (so every rank's buffer is packed from row 0) -- when `rank_packed` --
 // or the global exclusive prefix otherwise.
+// A row is `units` elements of U (16-byte vectors, or single elements where rows are not aligned); ld_y / ld_dst count U.
+template <typename U>
 __global__ void __launch_bounds__(256)
-dispatch_kernel(const __nv_bfloat16* __restrict__ y, long long ld_y, const int* __restrict__ topk_ids,
-                const float* __restrict__ topk_w, int T, int K, int H, int E, int experts_per_rank, int my_rank,
+dispatch_kernel(const U* __restrict__ y, long long ld_y, const int* __restrict__ topk_ids,
+                const float* __restrict__ topk_w, int T, int K, int units, int E, int experts_per_rank, int my_rank,
                 int* __restrict__ ws, int* __restrict__ offs, void* const* __restrict__ x_bases, long long ld_dst,
                 void* const* __restrict__ rec_bases, int dst_capacity, int* __restrict__ status) {
   __shared__ int s_base[kMaxExperts + 1];
@@ -228,7 +230,6 @@ dispatch_kernel(const __nv_bfloat16* __restrict__ y, long long ld_y, const int* 
       offs[E] = run;
     }
   }
-  const int nvec = H / 8;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int npairs = T * K;
   for (int p = blockIdx.x * nw + warp; p < npairs; p += gridDim.x * nw) {
@@ -247,9 +248,9 @@ dispatch_kernel(const __nv_bfloat16* __restrict__ y, long long ld_y, const int* 
       continue;
     }
     const int t = p / K;
-    const bf16x8m* sp = reinterpret_cast<const bf16x8m*>(y + static_cast<long long>(t) * ld_y);
-    bf16x8m* dp = reinterpret_cast<bf16x8m*>(static_cast<__nv_bfloat16*>(x_bases[rank]) + static_cast<long long>(row) * ld_dst);
-    for (int v = lane; v < nvec; v += 32) dp[v] = sp[v];
+    const U* sp = y + static_cast<long long>(t) * ld_y;
+    U* dp = static_cast<U*>(x_bases[rank]) + static_cast<long long>(row) * ld_dst;
+    for (int v = lane; v < units; v += 32) dp[v] = sp[v];
     if (lane == 0) {
       int4 rec;
       rec.x = my_rank;
@@ -317,17 +318,36 @@ extern "C" int dmoe_route_ex(const void* x, long long ld_x, const void* norm_w, 
   return static_cast<int>(cudaGetLastError());
 }
 
+static int dispatch_grid(int npairs) {      // one warp per (token, choice), up to four CTAs per SM
+  const int grid = (npairs + 7) / 8, cap = device_num_sms() * 4;
+  return grid < cap ? grid : cap;
+}
+
 extern "C" int dmoe_dispatch_local(const void* y, long long ld_y, const int* topk_ids, const float* topk_w, int T, int K,
                                    int H, int E, int experts_per_rank, int my_rank, int* ws, int* offs,
                                    const void* x_bases, long long ld_dst, const void* rec_bases, int dst_capacity,
                                    int* status, void* stream) {
-  if (H % 8 != 0 || E > kMaxExperts || experts_per_rank < 1) return -10;
+  if (H % 8 != 0 || ld_y % 8 != 0 || ld_dst % 8 != 0 || E > kMaxExperts || experts_per_rank < 1) return -10;
   if (T == 0) return 0;
-  const int npairs = T * K;
-  int grid = (npairs + 7) / 8;
-  if (grid > device_num_sms() * 4) grid = device_num_sms() * 4;
-  dispatch_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const __nv_bfloat16*>(y), ld_y, topk_ids, topk_w, T, K, H, E, experts_per_rank, my_rank, ws, offs,
-      static_cast<void* const*>(x_bases), ld_dst, static_cast<void* const*>(rec_bases), dst_capacity, status);
+  dispatch_kernel<uint4><<<dispatch_grid(T * K), 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(y), ld_y / 8, topk_ids, topk_w, T, K, H / 8, E, experts_per_rank, my_rank, ws, offs,
+      static_cast<void* const*>(x_bases), ld_dst / 8, static_cast<void* const*>(rec_bases), dst_capacity, status);
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dmoe_dispatch_local_any(int elem_bytes, const void* y, long long ld_y, const int* topk_ids, const float* topk_w,
+                                       int T, int K, int H, int E, int* ws, int* offs, const void* x_bases, long long ld_dst,
+                                       const void* rec_bases, int dst_capacity, int* status, void* stream_) {
+  if (H < 1 || E < 1 || E > kMaxExperts || (elem_bytes != 2 && elem_bytes != 4)) return -10;
+  if (T == 0) return 0;
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (elem_bytes == 4)
+    dispatch_kernel<uint32_t><<<dispatch_grid(T * K), 256, 0, stream>>>(
+        static_cast<const uint32_t*>(y), ld_y, topk_ids, topk_w, T, K, H, E, E, 0, ws, offs,
+        static_cast<void* const*>(x_bases), ld_dst, static_cast<void* const*>(rec_bases), dst_capacity, status);
+  else
+    dispatch_kernel<uint16_t><<<dispatch_grid(T * K), 256, 0, stream>>>(
+        static_cast<const uint16_t*>(y), ld_y, topk_ids, topk_w, T, K, H, E, E, 0, ws, offs,
+        static_cast<void* const*>(x_bases), ld_dst, static_cast<void* const*>(rec_bases), dst_capacity, status);
   return static_cast<int>(cudaGetLastError());
 }

@@ -228,7 +228,7 @@ def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table
         if v_first is not None:
             v = ((1.0 - v_lambda) * v.float() + v_lambda * v_first[ok][..., :dv].float()).to(v.dtype)
         vcache.view(-1, n_kv, dv)[slots[ok]] = v
-    qkv[:, :qs] = q.reshape(T, qs)
+    qkv[:, :qs] = q.reshape(T, qs).clone()
 
 
 def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved):
@@ -237,7 +237,7 @@ def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_lo
     q = y[:, :H * lay.qd].reshape(T, H, lay.qd)
     d = y[:, H * lay.qd:]
     c = (_rms_scale(d[:, :lay.rank].float(), eps) * norm_w).to(y.dtype)
-    kr = _turn(d[:, None, lay.rank:lay.rank + lay.rot].float(), table, positions, interleaved)[:, 0].to(y.dtype)
+    kr = _turn(d[:, None, lay.rankp:lay.rankp + lay.rot].float(), table, positions, interleaved)[:, 0].to(y.dtype)
     ok = slots >= 0
     flat = cache.view(-1, lay.row)
     flat[slots[ok], :lay.rank] = c[ok]

@@ -168,7 +168,7 @@ def random_weights(config, seed=0):
     g = torch.Generator().manual_seed(seed)
     out = {}
     for n, s in shapes(config).items():
-        r = torch.randn(*s, generator=g)
+        r = torch.randn(s, generator=g)
         leaf = n.rsplit(".", 1)[-1]
         if leaf == "vmix":
             t = 0.5 + 0.3 * r
