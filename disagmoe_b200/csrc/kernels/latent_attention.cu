@@ -16,7 +16,8 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr int pad8(int n) { return (n + 7) / 8 * 8; }
 
 // One CTA per row. A row of y is [heads x (dimp | rotp) | rankp | rotp], parts padded with zeros to multiples of 8.
-template <typename T>
+// VEC: the rotation is interleaved, covers all of rotp and moves in 16-byte units.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
                    T* __restrict__ cache, int heads, int dimp, int rotp, int rank, int rankp, int rot, int interleaved,
@@ -63,6 +64,32 @@ latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ posi
     for (int d = threadIdx.x; d < rank; d += blockDim.x) dst[d] = static_cast<T>(static_cast<float>(c[d]) * inv * norm_w[d]);
     turn(c + rankp, dst + rankp, threadIdx.x, blockDim.x);
   }
+  if (VEC) {
+    // units of all heads dealt out to the threads: what is copied, what turns in place and what turns on its way out
+    constexpr int V = 16 / sizeof(T);
+    const int un = dimp / V, ur = rotp / V, first = li < 0 ? un : 0;
+    for (int x = threadIdx.x; x < heads * (un + ur - first); x += blockDim.x) {
+      const int h = x / (un + ur - first), u = first + x % (un + ur - first);
+      const long long at = static_cast<long long>(h) * n_loose + li;
+      T* src = yr + static_cast<long long>(h) * qd + u * V;
+      if (u < un) {
+        *reinterpret_cast<uint4*>(xq + at * dimp + u * V) = *reinterpret_cast<const uint4*>(src);
+        continue;
+      }
+      alignas(16) T v[V];
+      *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(src);
+#pragma unroll
+      for (int e = 0; e < V / 2; ++e) {
+        const float2 cs = tab[(u - un) * (V / 2) + e];
+        const float p = static_cast<float>(v[2 * e]), w = static_cast<float>(v[2 * e + 1]);
+        v[2 * e] = static_cast<T>(p * cs.x - w * cs.y);
+        v[2 * e + 1] = static_cast<T>(w * cs.x + p * cs.y);
+      }
+      T* dst = li < 0 ? src : qa + at * row + rankp + (u - un) * V;
+      *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(v);
+    }
+    return;
+  }
   for (int h = warp; h < heads; h += blockDim.x >> 5) {
     T* q = yr + static_cast<long long>(h) * qd;
     if (li < 0) {
@@ -90,36 +117,38 @@ latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ bl
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Attention over the cached rows. A CTA of eight warps has one query token, 16 MT heads (the rows of its MMA tiles) and one
-// range of keys, which come 64 at a time through a double-buffered cp.async ring. Per 64 keys: every warp computes the scores of
-// all heads with 8 keys (S = Q K^T over the whole row), the warps agree on the running maxima through shared memory, the softmax
-// weights go there as hi + lo bf16 pairs, and every warp accumulates 8 NT value columns (O += P V, V = the same rows).
+// Attention over the cached rows. A CTA of eight warps has one query token, 16 heads (the rows of its MMA tiles, whose A
+// fragments stay in registers) and one range of keys, which come 64 at a time through a double-buffered cp.async ring. Per 64
+// keys: every warp computes the scores of all heads with 8 keys (S = Q K^T over the whole row) and leaves them in shared memory;
+// after one barrier every warp takes the whole 16 x 64 score tile back as its own A fragments, does the online softmax (all
+// warps the same one) and accumulates 8 NT value columns (O += P V, V = the same rows, P = hi + lo bf16).
 constexpr int kLatKeys = 64, kLatThreads = 256, kLatWarps = 8;
+constexpr int kLatSp = kLatKeys + 8;        // pitch of a score row, floats: 64-bit reads of a fragment meet no bank twice
 
 struct LatentSmem {      // bytes
-  int pitch, q, p, m, total;
+  int pitch, q, s, total;
 };
-__host__ __device__ inline LatentSmem latent_smem(int row, int mt) {
+__host__ __device__ inline LatentSmem latent_smem(int row) {
   LatentSmem s;
   s.pitch = (row + 31) / 32 * 64 + 16;        // an odd number of 16-byte units: ldmatrix meets no bank twice
   s.q = 2 * kLatKeys * s.pitch;
-  s.p = s.q + 16 * mt * s.pitch;
-  s.m = s.p + 2 * 16 * mt * (kLatKeys * 2 + 16);
-  s.total = s.m + 16 * mt * kLatWarps * 4;
+  s.s = s.q + 16 * s.pitch;
+  s.total = s.s + 16 * kLatSp * 4;
   return s;
 }
 
-template <int NT, int MT>
+// NT: 8-column tiles of the output per warp (rankp <= 64 NT); K32: most 32-wide steps of a row (row <= 32 K32)
+template <int NT, int K32>
 __global__ void __launch_bounds__(kLatThreads)
 latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, const int* __restrict__ block_tables,
                    int max_blocks, const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len,
-                   int block_size, int n, int heads, int rankp, int row, float scale_log2, int window,
+                   int block_size, int n, int heads, int groups, int rankp, int row, float scale_log2, int window,
                    const float* __restrict__ sink, int splits, bf16* __restrict__ out, float* __restrict__ part_o,
                    float* __restrict__ part_lse) {
-  constexpr int PP = kLatKeys * 2 + 16;         // pitch of a row of P
   extern __shared__ __align__(128) uint8_t smem[];
-  const LatentSmem L = latent_smem(row, MT);
-  const int i = blockIdx.x, h0 = blockIdx.y * 16 * MT, split = blockIdx.z;
+  const LatentSmem L = latent_smem(row);
+  // the head groups of a token are neighbours: they read the same rows at about the same time
+  const int i = blockIdx.x / groups, h0 = blockIdx.x % groups * 16, split = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tq = lane & 3;
   const int b = rows != nullptr ? rows[i] : i;
@@ -130,36 +159,23 @@ latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, c
   const int c0 = min(len, lo + split * per), c1 = min(len, c0 + per);
   const int ntile = (c1 - c0 + kLatKeys - 1) / kLatKeys;
   const int nch = row / 8, k32 = (row + 31) / 32;
-  const uint32_t sb = smem_u32(smem), sq = sb + L.q, sp = sb + L.p;
-  float* s_m = reinterpret_cast<float*>(smem + L.m);      // [16 MT][warps]
+  const uint32_t sb = smem_u32(smem);
+  float* s_s = reinterpret_cast<float*>(smem + L.s);      // [16][kLatSp] scores, base-2 units
 
-  // zeros where no copy ever writes: columns row .. 32 k32 of the keys and of the queries, and absent heads
-  const int tail = k32 * 4 - nch;                         // 16-byte units
-  for (int r = threadIdx.x; r < 2 * kLatKeys + 16 * MT; r += kLatThreads)
-    for (int c = 0; c < tail; ++c)
-      *reinterpret_cast<uint4*>(smem + r * L.pitch + (nch + c) * 16) = make_uint4(0, 0, 0, 0);
-  for (int r = warp; r < 16 * MT; r += kLatWarps) {
-    const bf16* src = q + (static_cast<long long>(h0 + r) * n + i) * row;
-    for (int c = lane; c < nch; c += 32)
-      *reinterpret_cast<uint4*>(smem + L.q + r * L.pitch + c * 16) =
-          h0 + r < heads ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
-  }
-
+  // copies of a warp: rows 8 warp .. 8 warp + 7, in 16-byte units; lane l takes units l, l + 32, ... of the 8 nch
   auto issue = [&](int j) {
     if (j < ntile) {
-      const int tok0 = c0 + j * kLatKeys;
-      const uint32_t dst0 = sb + (j & 1) * kLatKeys * L.pitch;
-      // a warp fetches rows 8 warp .. 8 warp + 7; lane r < 8 looks up the slot of row r
-      long long slot = 0;
-      const int key = tok0 + warp * 8 + (lane & 7);
-      if (key < c1) slot = static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
+      const int tok0 = c0 + j * kLatKeys + warp * 8;
+      const uint32_t dst0 = sb + ((j & 1) * kLatKeys + warp * 8) * L.pitch;
+      const int key = tok0 + (lane & 7);                  // lanes look up the slots of the eight rows
+      int slot = 0;
+      if (key < c1) slot = bt[key / block_size] * block_size + key % block_size;
       int r = 0, c = lane;
       while (c >= nch) { c -= nch; ++r; }
-      for (int x = lane; x - lane < 8 * nch; x += 32) {   // the whole warp iterates: the shuffle needs every lane
-        const int rr = r < 8 ? r : 7;
-        const long long s = __shfl_sync(0xffffffffu, slot, rr);
-        if (x < 8 * nch)
-          cp_async16(dst0 + (warp * 8 + r) * L.pitch + c * 16, cache + s * row + c * 8, tok0 + warp * 8 + r < c1);
+#pragma unroll 4
+      for (int x = 0; x < 8 * nch; x += 32) {             // the whole warp iterates: the shuffle needs every lane
+        const long long s = __shfl_sync(0xffffffffu, slot, r & 7);
+        if (r < 8) cp_async16(dst0 + r * L.pitch + c * 16, cache + s * row + c * 8, tok0 + r < c1);
         c += 32;
         while (c >= nch) { c -= nch; ++r; }
       }
@@ -168,16 +184,31 @@ latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, c
   };
   issue(0);
 
-  float o[MT][NT][4];
-  float m[MT][2], l[MT][2];
-#pragma unroll
-  for (int t = 0; t < MT; ++t) {
-    m[t][0] = m[t][1] = -INFINITY;
-    l[t][0] = l[t][1] = 0.f;
-#pragma unroll
-    for (int x = 0; x < NT; ++x) o[t][x][0] = o[t][x][1] = o[t][x][2] = o[t][x][3] = 0.f;
+  // zeros where no copy ever writes: columns row .. 32 k32 of the keys and of the queries, and absent heads
+  const int tail = k32 * 4 - nch;                         // 16-byte units
+  for (int r = threadIdx.x; r < 2 * kLatKeys + 16; r += kLatThreads)
+    for (int c = 0; c < tail; ++c)
+      *reinterpret_cast<uint4*>(smem + r * L.pitch + (nch + c) * 16) = make_uint4(0, 0, 0, 0);
+  for (int r = warp; r < 16; r += kLatWarps) {
+    const bf16* src = q + (static_cast<long long>(h0 + r) * n + i) * row;
+    for (int c = lane; c < nch; c += 32)
+      *reinterpret_cast<uint4*>(smem + L.q + r * L.pitch + c * 16) =
+          h0 + r < heads ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
   }
+  __syncthreads();
   const int lm_mi = lane >> 3, lm_r = lane & 7;
+  uint32_t qa[2 * K32][4];
+  {
+    const uint32_t qaddr = sb + L.q + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
+#pragma unroll
+    for (int k = 0; k < 2 * K32; ++k)
+      if (k < 2 * k32) ldmatrix_x4(qaddr + k * 32, qa[k][0], qa[k][1], qa[k][2], qa[k][3]);
+  }
+
+  float o[NT][4];
+#pragma unroll
+  for (int x = 0; x < NT; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const int col0 = warp * NT * 8;                         // this warp's value columns
 
   for (int j = 0; j < ntile; ++j) {
@@ -185,134 +216,102 @@ latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, c
     __syncthreads();                    // tile j has landed; everyone is done with tile j - 1
     issue(j + 1);
     const uint32_t kb = sb + (j & 1) * kLatKeys * L.pitch;
-    float s[MT][4];
+    {
+      float s[4][4] = {};               // four independent sums: an MMA does not wait for the one before it
+      const uint32_t kaddr = kb + (warp * 8 + lm_r) * L.pitch + lm_mi * 16;
 #pragma unroll
-    for (int t = 0; t < MT; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
-    const uint32_t kaddr = kb + (warp * 8 + lm_r) * L.pitch + lm_mi * 16;
-    const uint32_t qaddr = sq + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
-#pragma unroll 2
-    for (int k = 0; k < k32; ++k) {
-      uint32_t b0, b1, b2, b3;
-      ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
-#pragma unroll
-      for (int t = 0; t < MT; ++t) {
-        uint32_t a0[4], a1[4];
-        ldmatrix_x4(qaddr + t * 16 * L.pitch + k * 64, a0[0], a0[1], a0[2], a0[3]);
-        ldmatrix_x4(qaddr + t * 16 * L.pitch + k * 64 + 32, a1[0], a1[1], a1[2], a1[3]);
-        mma_bf16_16816(s[t], a0, b0, b1);
-        mma_bf16_16816(s[t], a1, b2, b3);
-      }
-    }
-    const int key = c0 + j * kLatKeys + warp * 8 + 2 * tq;
-    const bool v0 = key < c1, v1 = key + 1 < c1;
-#pragma unroll
-    for (int t = 0; t < MT; ++t) {
-      s[t][0] = v0 ? s[t][0] * scale_log2 : -INFINITY;
-      s[t][1] = v1 ? s[t][1] * scale_log2 : -INFINITY;
-      s[t][2] = v0 ? s[t][2] * scale_log2 : -INFINITY;
-      s[t][3] = v1 ? s[t][3] * scale_log2 : -INFINITY;
-      float x0 = fmaxf(s[t][0], s[t][1]), x1 = fmaxf(s[t][2], s[t][3]);
-      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
-      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
-      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
-      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-      if (tq == 0) {
-        s_m[(t * 16 + g) * kLatWarps + warp] = x0;
-        s_m[(t * 16 + g + 8) * kLatWarps + warp] = x1;
-      }
-    }
-    __syncthreads();
-#pragma unroll
-    for (int t = 0; t < MT; ++t) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float4* pm = reinterpret_cast<const float4*>(s_m + (t * 16 + g + 8 * e) * kLatWarps);
-        const float4 x = pm[0], z = pm[1];
-        // finite: the first key of the tile is visible
-        const float mn = fmaxf(m[t][e], fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(z.x, z.y), fmaxf(z.z, z.w))));
-        const float corr = exp2f(m[t][e] - mn);
-        m[t][e] = mn;
-        const float p0 = exp2f(s[t][2 * e] - mn), p1 = exp2f(s[t][2 * e + 1] - mn);
-        l[t][e] = l[t][e] * corr + p0 + p1;               // of this lane's keys; the lanes add up at the end
-        uint32_t hi, lo2;
-        split2(p0, p1, hi, lo2);
-        uint8_t* pr = smem + L.p + (t * 16 + g + 8 * e) * PP + (warp * 8 + 2 * tq) * 2;
-        *reinterpret_cast<uint32_t*>(pr) = hi;
-        *reinterpret_cast<uint32_t*>(pr + 16 * MT * PP) = lo2;
-#pragma unroll
-        for (int x2 = 0; x2 < NT; ++x2) { o[t][x2][2 * e] *= corr; o[t][x2][2 * e + 1] *= corr; }
-      }
+      for (int k = 0; k < K32; ++k)
+        if (k < k32) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
+          mma_bf16_16816(s[(2 * k) & 3], qa[2 * k], b0, b1);
+          mma_bf16_16816(s[(2 * k + 1) & 3], qa[2 * k + 1], b2, b3);
+        }
+      const int key = c0 + j * kLatKeys + warp * 8 + 2 * tq;
+      const bool v0 = key < c1, v1 = key + 1 < c1;
+      auto fin = [&](int e, bool v) { return v ? ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * scale_log2 : -INFINITY; };
+      float* dst = s_s + g * kLatSp + warp * 8 + 2 * tq;
+      *reinterpret_cast<float2*>(dst) = make_float2(fin(0, v0), fin(1, v1));
+      *reinterpret_cast<float2*>(dst + 8 * kLatSp) = make_float2(fin(2, v0), fin(3, v1));
     }
     __syncthreads();
     if (col0 < rankp) {
+      float p[2][16];                   // rows g, g + 8; columns 8 y + 2 tq + {0, 1}, y = 0 .. 7
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float* src = s_s + (g + 8 * e) * kLatSp + 2 * tq;
+        float mx = m[e];
+#pragma unroll
+        for (int y = 0; y < 8; ++y) {
+          const float2 v = *reinterpret_cast<const float2*>(src + 8 * y);
+          p[e][2 * y] = v.x;
+          p[e][2 * y + 1] = v.y;
+          mx = fmaxf(mx, fmaxf(v.x, v.y));
+        }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));      // finite: the first key of the tile is visible
+        const float corr = exp2f(m[e] - mx);
+        m[e] = mx;
+        float sum = 0.f;
+#pragma unroll
+        for (int y = 0; y < 16; ++y) {
+          p[e][y] = exp2f(p[e][y] - mx);
+          sum += p[e][y];
+        }
+        l[e] = l[e] * corr + sum;       // of this lane's keys; the four lanes of a row add up at the end
+#pragma unroll
+        for (int x = 0; x < NT; ++x) { o[x][2 * e] *= corr; o[x][2 * e + 1] *= corr; }
+      }
 #pragma unroll
       for (int ks = 0; ks < kLatKeys / 16; ++ks) {
-        uint32_t ph[MT][4], pl[MT][4];
-#pragma unroll
-        for (int t = 0; t < MT; ++t) {
-          const uint32_t pa = sp + (t * 16 + lm_r + (lm_mi & 1) * 8) * PP + ks * 32 + (lm_mi >> 1) * 16;
-          ldmatrix_x4(pa, ph[t][0], ph[t][1], ph[t][2], ph[t][3]);
-          ldmatrix_x4(pa + 16 * MT * PP, pl[t][0], pl[t][1], pl[t][2], pl[t][3]);
-        }
+        uint32_t ph[4], pl[4];
+        split2(p[0][4 * ks], p[0][4 * ks + 1], ph[0], pl[0]);
+        split2(p[1][4 * ks], p[1][4 * ks + 1], ph[1], pl[1]);
+        split2(p[0][4 * ks + 2], p[0][4 * ks + 3], ph[2], pl[2]);
+        split2(p[1][4 * ks + 2], p[1][4 * ks + 3], ph[3], pl[3]);
         const uint32_t va = kb + (ks * 16 + (lm_mi & 1) * 8 + lm_r) * L.pitch + col0 * 2 + (lm_mi >> 1) * 16;
 #pragma unroll
         for (int dp = 0; dp < NT / 2; ++dp) {
           if (col0 + dp * 16 < rankp) {
             uint32_t b0, b1, b2, b3;
             ldmatrix_x4_trans(va + dp * 32, b0, b1, b2, b3);
-#pragma unroll
-            for (int t = 0; t < MT; ++t) {
-              mma_bf16_16816(o[t][2 * dp], ph[t], b0, b1);
-              mma_bf16_16816(o[t][2 * dp + 1], ph[t], b2, b3);
-              mma_bf16_16816(o[t][2 * dp], pl[t], b0, b1);
-              mma_bf16_16816(o[t][2 * dp + 1], pl[t], b2, b3);
-            }
+            mma_bf16_16816(o[2 * dp], ph, b0, b1);
+            mma_bf16_16816(o[2 * dp + 1], ph, b2, b3);
+            mma_bf16_16816(o[2 * dp], pl, b0, b1);
+            mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
           }
         }
       }
     }
   }
   cp_async_wait<0>();
-  __syncthreads();
-  // denominators: lanes of a row, then warps
+  if (col0 >= rankp) return;
 #pragma unroll
-  for (int t = 0; t < MT; ++t)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      float x = l[t][e];
-      x += __shfl_xor_sync(0xffffffffu, x, 1);
-      x += __shfl_xor_sync(0xffffffffu, x, 2);
-      if (tq == 0) s_m[(t * 16 + g + 8 * e) * kLatWarps + warp] = x;
+  for (int e = 0; e < 2; ++e) {
+    float den = l[e];
+    den += __shfl_xor_sync(0xffffffffu, den, 1);
+    den += __shfl_xor_sync(0xffffffffu, den, 2);
+    const int head = h0 + g + 8 * e;
+    if (head >= heads) continue;
+    float mm = m[e], f = 1.f;
+    if (sink != nullptr && split == 0 && len > 0) {       // one split carries the sink
+      const float sk = sink[head] * kLog2e, mn = fmaxf(mm, sk);
+      f = exp2f(mm - mn);
+      den = den * f + exp2f(sk - mn);
+      mm = mn;
     }
-  __syncthreads();
+    f = den > 0.f ? f / den : 0.f;
+    const long long at = static_cast<long long>(head) * n + i;
 #pragma unroll
-  for (int t = 0; t < MT; ++t)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int head = h0 + t * 16 + g + 8 * e;
-      if (head >= heads) continue;
-      float den = 0.f;
-#pragma unroll
-      for (int w = 0; w < kLatWarps; ++w) den += s_m[(t * 16 + g + 8 * e) * kLatWarps + w];
-      float mm = m[t][e], f = 1.f;
-      if (sink != nullptr && split == 0 && len > 0) {     // one split carries the sink
-        const float sk = sink[head] * kLog2e, mn = fmaxf(mm, sk);
-        f = exp2f(mm - mn);
-        den = den * f + exp2f(sk - mn);
-        mm = mn;
-      }
-      f = den > 0.f ? f / den : 0.f;
-      const long long at = static_cast<long long>(head) * n + i;
-#pragma unroll
-      for (int x = 0; x < NT; ++x) {
-        const int col = col0 + x * 8 + 2 * tq;
-        if (col >= rankp) continue;
-        const float a = o[t][x][2 * e] * f, c = o[t][x][2 * e + 1] * f;
-        if (splits == 1) *reinterpret_cast<uint32_t*>(out + at * rankp + col) = pack_bf16(a, c);
-        else *reinterpret_cast<float2*>(part_o + (at * splits + split) * rankp + col) = make_float2(a, c);
-      }
-      if (splits > 1 && warp == 0 && tq == 0) part_lse[at * splits + split] = den > 0.f ? mm + log2f(den) : -INFINITY;
+    for (int x = 0; x < NT; ++x) {
+      const int col = col0 + x * 8 + 2 * tq;
+      if (col >= rankp) continue;
+      const float a = o[x][2 * e] * f, c = o[x][2 * e + 1] * f;
+      if (splits == 1) *reinterpret_cast<uint32_t*>(out + at * rankp + col) = pack_bf16(a, c);
+      else *reinterpret_cast<float2*>(part_o + (at * splits + split) * rankp + col) = make_float2(a, c);
     }
+    if (splits > 1 && warp == 0 && tq == 0) part_lse[at * splits + split] = den > 0.f ? mm + log2f(den) : -INFINITY;
+  }
 }
 
 // out[at] = sum over splits of its softmax(lse)-weighted parts, at = (head, query)
@@ -512,22 +511,22 @@ latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __
   }
 }
 
-template <int NT, int MT>
+template <int NT, int K32>
 static int launch_latent(const void* q, const void* cache, const int* bt, int max_blocks, const int* bt_row, const int* rows,
                          const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale, int window,
                          const float* sink, int splits, void* out, float* ws, cudaStream_t stream) {
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT, K32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
   });
   if (rc != 0) return rc;
-  const int smem = latent_smem(row, MT).total;
-  if (smem > 227 * 1024) return -11;
-  const long long at = static_cast<long long>(heads) * n;
+  const int smem = latent_smem(row).total, groups = (heads + 15) / 16;
+  const long long at = static_cast<long long>(heads) * n, ctas = static_cast<long long>(groups) * n;
+  if (smem > 227 * 1024 || ctas > 0x7fffffffll) return -11;
   float* part_lse = ws != nullptr ? ws + at * splits * rankp : nullptr;
-  latent_attn_kernel<NT, MT><<<dim3(n, (heads + 16 * MT - 1) / (16 * MT), splits), kLatThreads, smem, stream>>>(
+  latent_attn_kernel<NT, K32><<<dim3(static_cast<unsigned>(ctas), splits), kLatThreads, smem, stream>>>(
       static_cast<const bf16*>(q), static_cast<const bf16*>(cache), bt, max_blocks, bt_row, rows, ctx_len, block_size, n, heads,
-      rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse);
+      groups, rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse);
   if (splits > 1)
     latent_merge_kernel<<<static_cast<unsigned>(at), 128, 0, stream>>>(ws, part_lse, splits, rankp, static_cast<bf16*>(out));
   return static_cast<int>(cudaGetLastError());
@@ -564,14 +563,16 @@ extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* po
   if (ld % align != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 || (loose == nullptr && n_loose < T)) return -10;
   if (T == 0) return 0;
   const int dimp = pad8(dim), rotp = pad8(rot_dim), rankp = pad8(rank);
-  if (is_f32)
-    latent_prep_kernel<float><<<T, 256, 0, stream>>>(
-        static_cast<float*>(y), ld, positions, slots, static_cast<float*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,
-        static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<float*>(xq), static_cast<float*>(qa));
-  else
-    latent_prep_kernel<bf16><<<T, 256, 0, stream>>>(
-        static_cast<bf16*>(y), ld, positions, slots, static_cast<bf16*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,
-        static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<bf16*>(xq), static_cast<bf16*>(qa));
+  const bool vec = interleaved && rot == rotp && rot > 0;
+#define DMOE_PREP(T_, VEC_)                                                                                                  \
+  latent_prep_kernel<T_, VEC_><<<T, 256, 0, stream>>>(                                                                       \
+      static_cast<T_*>(y), ld, positions, slots, static_cast<T_*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,  \
+      static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<T_*>(xq), static_cast<T_*>(qa))
+  if (is_f32 && vec) DMOE_PREP(float, true);
+  else if (is_f32) DMOE_PREP(float, false);
+  else if (vec) DMOE_PREP(bf16, true);
+  else DMOE_PREP(bf16, false);
+#undef DMOE_PREP
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -583,17 +584,13 @@ extern "C" int dmoe_latent_attention(const void* qa, const void* cache, const in
   if (block_size < 1 || splits < 1 || splits > 65535 || (splits > 1 && workspace == nullptr)) return -10;
   if (n == 0) return 0;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-#define DMOE_LAT(NT_, MT_)                                                                                              \
-  return launch_latent<NT_, MT_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, \
-                                 row, scale, window, sink, splits, out, workspace, stream)
-  if (heads <= 16) {
-    if (rankp <= 128) DMOE_LAT(2, 1);
-    if (rankp <= 256) DMOE_LAT(4, 1);
-    DMOE_LAT(8, 1);
-  }
-  if (rankp <= 128) DMOE_LAT(2, 2);
-  if (rankp <= 256) DMOE_LAT(4, 2);
-  DMOE_LAT(8, 2);
+#define DMOE_LAT(NT_, K_)                                                                                              \
+  return launch_latent<NT_, K_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, \
+                                row, scale, window, sink, splits, out, workspace, stream)
+  if (rankp <= 128 && row <= 192) DMOE_LAT(2, 6);
+  if (rankp <= 256 && row <= 320) DMOE_LAT(4, 10);
+  if (row <= 576) DMOE_LAT(8, 18);
+  DMOE_LAT(8, 20);
 #undef DMOE_LAT
 }
 

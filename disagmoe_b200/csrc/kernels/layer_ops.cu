@@ -248,24 +248,31 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
   __syncthreads();
 
   const T* gate = static_cast<const T*>(a.gate_w);
-  for (int e = warp; e < a.E; e += kSumWarps) {
-    float acc[TPC] = {};
+  constexpr int EB = TPC == 8 ? 4 : TPC;      // experts per pass of a warp: they share the reads of the rows
+  for (int e0 = warp * EB; e0 < a.E; e0 += kSumWarps * EB) {
+    float acc[EB][TPC] = {};
     for (int v = lane; v < nvec; v += 32) {
-      float g[VEC];
-      Pack<T, VEC>::load(gate + static_cast<long long>(e) * W + v * VEC, g);
+      float g[EB][VEC];
+#pragma unroll
+      for (int k = 0; k < EB; ++k)
+        Pack<T, VEC>::load(gate + static_cast<long long>(min(e0 + k, a.E - 1)) * W + v * VEC, g[k]);
 #pragma unroll
       for (int t = 0; t < TPC; ++t) {
         float x[VEC];
         Pack<float, VEC>::load(s_row + static_cast<long long>(t) * W + v * VEC, x);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) acc[t] += g[k] * x[k];
+        for (int k = 0; k < EB; ++k)
+#pragma unroll
+          for (int c = 0; c < VEC; ++c) acc[k][t] += g[k][c] * x[c];
       }
     }
 #pragma unroll
-    for (int t = 0; t < TPC; ++t) {
-      const float z = warp_sum(acc[t]);
-      if (lane == 0) slog[t][e] = z;
-    }
+    for (int k = 0; k < EB; ++k)
+#pragma unroll
+      for (int t = 0; t < TPC; ++t) {
+        const float z = warp_sum(acc[k][t]);
+        if (lane == 0 && e0 + k < a.E) slog[t][e0 + k] = z;
+      }
   }
   __syncthreads();
   const long long tok = static_cast<long long>(blockIdx.x) * TPC + warp;
@@ -375,6 +382,54 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
       const float first = d < first_head ? static_cast<float>(v_first[t * ld_first + i / dv * first_head + d]) : 0.f;
       dst[i] = static_cast<T>((1.f - v_lambda) * static_cast<float>(src[i]) + v_lambda * first);
     }
+  }
+}
+
+// The same for interleaved rotation without norms where everything moves in 16-byte units (dk, dv and rot multiples of 8):
+// the units of a row's heads are dealt out to the threads.
+__global__ void __launch_bounds__(256)
+rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
+                   bf16* __restrict__ kcache, bf16* __restrict__ vcache, int n_q, int n_kv, int dk, int dv, int rot,
+                   const float2* __restrict__ table, int max_pos, const bf16* __restrict__ v_first, long long ld_first,
+                   int first_head, float v_lambda) {
+  const long long t = blockIdx.x;
+  const int pos = min(max(positions[t], 0), max_pos - 1);
+  const long long slot = slots[t];
+  bf16* row = qkv + t * ld;
+  const float2* tab = table + static_cast<long long>(pos) * (rot / 2);
+  const int uq = n_q * dk / 8, uk = uq + (slot >= 0 ? n_kv * dk / 8 : 0);
+  for (int u = threadIdx.x; u < uk; u += blockDim.x) {
+    const int d = u * 8 % dk;
+    const bool is_q = u < uq;
+    if (is_q && d >= rot) continue;           // in place already
+    bf16* dst = is_q ? row + u * 8 : kcache + slot * n_kv * dk + (u - uq) * 8;
+    float x[8];
+    Pack<bf16, 8>::load(row + u * 8, x);
+    if (d < rot) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 cs = tab[d / 2 + e];
+        const float a = x[2 * e], b = x[2 * e + 1];
+        x[2 * e] = a * cs.x - b * cs.y;
+        x[2 * e + 1] = b * cs.x + a * cs.y;
+      }
+    }
+    Pack<bf16, 8>::store(dst, x);
+  }
+  if (slot < 0) return;
+  const bf16* src = row + static_cast<long long>(n_q + n_kv) * dk;
+  bf16* dst = vcache + slot * n_kv * dv;
+  for (int u = threadIdx.x; u < n_kv * dv / 8; u += blockDim.x) {
+    float x[8];
+    Pack<bf16, 8>::load(src + u * 8, x);
+    if (v_first != nullptr) {
+      const int h = u * 8 / dv, d = u * 8 % dv;
+      float y[8] = {};
+      if (d < first_head) Pack<bf16, 8>::load(v_first + t * ld_first + h * first_head + d, y);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = (1.f - v_lambda) * x[e] + v_lambda * y[e];
+    }
+    Pack<bf16, 8>::store(dst + u * 8, x);
   }
 }
 
@@ -564,6 +619,14 @@ extern "C" int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int*
   if (T == 0) return 0;
   int threads = (n_q + n_kv) * 32;
   if (threads > 256) threads = 256;
+  if (!is_f32 && qw == nullptr && n_kv > 0 && (interleaved || rot == 0) && dk % 8 == 0 && dv % 8 == 0 && rot % 8 == 0 &&
+      ld % 8 == 0 && first_head % 8 == 0 && ld_first % 8 == 0 && aligned16(qkv) && aligned16(kcache) && aligned16(vcache) &&
+      aligned16(v_first)) {
+    rope_append_kernel<<<T, threads, 0, stream>>>(
+        static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk, dv,
+        rot, static_cast<const float2*>(table), max_pos, static_cast<const bf16*>(v_first), ld_first, first_head, v_lambda);
+    return static_cast<int>(cudaGetLastError());
+  }
   if (is_f32)
     qk_norm_rope_kernel<float><<<T, threads, 0, stream>>>(
         static_cast<float*>(qkv), ld, positions, slots, static_cast<float*>(kcache), static_cast<float*>(vcache), n_q, n_kv,

@@ -718,11 +718,11 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, block_tables: torch.
 
 
 def pick_latent_splits(n: int, heads: int, reach: int) -> int:
-    """Key ranges per (query token, group of up to 32 heads) of :func:`latent_attention`: enough CTAs for all SMs, never
-    fewer than 128 keys each."""
+    """Key ranges per (query token, group of 16 heads) of :func:`latent_attention`, one CTA per SM each: as many waves of
+    CTAs as it takes to keep all SMs busy, never fewer than 128 keys per range."""
     from .gemm import num_sms
-    sms, ctas = num_sms(), max(1, n * ((heads + 31) // 32))
-    return max(1, min((2 * sms + ctas - 1) // ctas, (reach + 127) // 128, 64)) if ctas < 2 * sms else 1
+    sms, ctas = num_sms(), max(1, n * ((heads + 15) // 16))
+    return max(1, min((4 * sms) // ctas, (reach + 127) // 128, 64))
 
 
 def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, keys: torch.Tensor, n_keys: int) -> torch.Tensor:
