@@ -138,10 +138,11 @@ int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, co
                      int heads, int dim, int rot_dim, int rank, int rot, int interleaved, const void* table, int max_pos,
                      const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa, void* stream);
 // Queries qa [heads, n, row] over cache rows (keys: all of a row, values: its first rankp columns), out [heads, n, rankp];
-// rankp <= 512, row <= 640. workspace: heads * n * splits * (rankp + 1) floats where splits > 1.
+// rankp <= 512, row <= 640. workspace: heads * n * splits * (rankp + 1) floats where splits > 1. status (may be NULL): non-zero
+// after a bounded wait gave up.
 int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
                           const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale,
-                          int window, const float* sink, int splits, void* out, float* workspace, void* stream);
+                          int window, const float* sink, int splits, void* out, float* workspace, int* status, void* stream);
 // out[i] = cache row of position keys[i].y of block-table row keys[i].x
 int dmoe_latent_gather(const void* cache, const int* block_tables, int max_blocks, const void* keys, int n, int block_size,
                        int row, void* out, void* stream);

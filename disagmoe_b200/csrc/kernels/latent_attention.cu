@@ -117,35 +117,42 @@ latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ bl
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Attention over the cached rows. A CTA of eight warps has one query token, 16 heads (the rows of its MMA tiles, whose A
-// fragments stay in registers) and one range of keys, which come 64 at a time through a double-buffered cp.async ring. Per 64
-// keys: every warp computes the scores of all heads with 8 keys (S = Q K^T over the whole row) and leaves them in shared memory;
-// after one barrier every warp takes the whole 16 x 64 score tile back as its own A fragments, does the online softmax (all
-// warps the same one) and accumulates 8 NT value columns (O += P V, V = the same rows, P = hi + lo bf16).
-constexpr int kLatKeys = 64, kLatThreads = 256, kLatWarps = 8;
+// Attention over the cached rows. A CTA of eight warps (two CTAs per SM) has one query token, 16 heads (the rows of its MMA
+// tiles) and one range of keys, which come 32 at a time, one bulk copy per cached row, into a double buffer. Per 32 keys: a warp
+// computes the scores of all heads with 8 keys over one half of the row (S = Q K^T) and leaves them in shared memory; after one
+// barrier every warp takes the whole 16 x 32 score tile back as its own A fragments, does the online softmax (all warps the same
+// one) and accumulates 8 NT value columns (O += P V, V = the same rows, P = hi + lo bf16).
+constexpr int kLatKeys = 32, kLatThreads = 256, kLatMaxSmem = 112 * 1024;
 constexpr int kLatSp = kLatKeys + 8;        // pitch of a score row, floats: 64-bit reads of a fragment meet no bank twice
 
 struct LatentSmem {      // bytes
-  int pitch, q, s, total;
+  int pitch, q, s, bars, total;
 };
 __host__ __device__ inline LatentSmem latent_smem(int row) {
   LatentSmem s;
   s.pitch = (row + 31) / 32 * 64 + 16;        // an odd number of 16-byte units: ldmatrix meets no bank twice
   s.q = 2 * kLatKeys * s.pitch;
   s.s = s.q + 16 * s.pitch;
-  s.total = s.s + 16 * kLatSp * 4;
+  s.bars = s.s + 2 * 16 * kLatSp * 4;
+  s.total = s.bars + 32;
   return s;
 }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
-// NT: 8-column tiles of the output per warp (rankp <= 64 NT); K32: most 32-wide steps of a row (row <= 32 K32)
-template <int NT, int K32>
-__global__ void __launch_bounds__(kLatThreads)
+// NT: 8-column tiles of the output per warp (rankp <= 64 NT)
+template <int NT>
+__global__ void __launch_bounds__(kLatThreads, 2)
 latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, const int* __restrict__ block_tables,
                    int max_blocks, const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len,
                    int block_size, int n, int heads, int groups, int rankp, int row, float scale_log2, int window,
                    const float* __restrict__ sink, int splits, bf16* __restrict__ out, float* __restrict__ part_o,
-                   float* __restrict__ part_lse) {
+                   float* __restrict__ part_lse, int* __restrict__ status) {
   extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ int s_abort;
   const LatentSmem L = latent_smem(row);
   // the head groups of a token are neighbours: they read the same rows at about the same time
   const int i = blockIdx.x / groups, h0 = blockIdx.x % groups * 16, split = blockIdx.y;
@@ -158,104 +165,99 @@ latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, c
   const int per = ((len - lo + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
   const int c0 = min(len, lo + split * per), c1 = min(len, c0 + per);
   const int ntile = (c1 - c0 + kLatKeys - 1) / kLatKeys;
-  const int nch = row / 8, k32 = (row + 31) / 32;
-  const uint32_t sb = smem_u32(smem);
-  float* s_s = reinterpret_cast<float*>(smem + L.s);      // [16][kLatSp] scores, base-2 units
+  const int nch = row / 8, k32 = (row + 31) / 32, khalf = (k32 + 1) / 2;
+  const uint32_t sb = smem_u32(smem), bar = sb + L.bars;
+  float* s_s = reinterpret_cast<float*>(smem + L.s);      // [half of the row][16][kLatSp] partial scores
 
-  // copies of a warp: rows 8 warp .. 8 warp + 7, in 16-byte units; lane l takes units l, l + 32, ... of the 8 nch
-  auto issue = [&](int j) {
-    if (j < ntile) {
-      const int tok0 = c0 + j * kLatKeys + warp * 8;
-      const uint32_t dst0 = sb + ((j & 1) * kLatKeys + warp * 8) * L.pitch;
-      const int key = tok0 + (lane & 7);                  // lanes look up the slots of the eight rows
-      int slot = 0;
-      if (key < c1) slot = bt[key / block_size] * block_size + key % block_size;
-      int r = 0, c = lane;
-      while (c >= nch) { c -= nch; ++r; }
-#pragma unroll 4
-      for (int x = 0; x < 8 * nch; x += 32) {             // the whole warp iterates: the shuffle needs every lane
-        const long long s = __shfl_sync(0xffffffffu, slot, r & 7);
-        if (r < 8) cp_async16(dst0 + r * L.pitch + c * 16, cache + s * row + c * 8, tok0 + r < c1);
-        c += 32;
-        while (c >= nch) { c -= nch; ++r; }
-      }
-    }
-    cp_async_commit();
-  };
-  issue(0);
-
+  if (threadIdx.x == 0) {
+    s_abort = 0;
+    mbar_init(bar, 1);
+    mbar_init(bar + 8, 1);
+    mbar_fence_init();
+  }
   // zeros where no copy ever writes: columns row .. 32 k32 of the keys and of the queries, and absent heads
   const int tail = k32 * 4 - nch;                         // 16-byte units
   for (int r = threadIdx.x; r < 2 * kLatKeys + 16; r += kLatThreads)
     for (int c = 0; c < tail; ++c)
       *reinterpret_cast<uint4*>(smem + r * L.pitch + (nch + c) * 16) = make_uint4(0, 0, 0, 0);
-  for (int r = warp; r < 16; r += kLatWarps) {
+  for (int r = warp; r < 16; r += kLatThreads / 32) {
     const bf16* src = q + (static_cast<long long>(h0 + r) * n + i) * row;
     for (int c = lane; c < nch; c += 32)
       *reinterpret_cast<uint4*>(smem + L.q + r * L.pitch + c * 16) =
           h0 + r < heads ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
   }
   __syncthreads();
-  const int lm_mi = lane >> 3, lm_r = lane & 7;
-  uint32_t qa[2 * K32][4];
-  {
-    const uint32_t qaddr = sb + L.q + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
-#pragma unroll
-    for (int k = 0; k < 2 * K32; ++k)
-      if (k < 2 * k32) ldmatrix_x4(qaddr + k * 32, qa[k][0], qa[k][1], qa[k][2], qa[k][3]);
-  }
+
+  auto issue = [&](int j) {             // warp 0: one row per lane; rows past the end repeat the last one (their weight is 0)
+    if (warp != 0 || j >= ntile) return;
+    const uint32_t mb = bar + (j & 1) * 8;
+    if (lane == 0) mbar_expect_tx(mb, kLatKeys * row * 2);
+    const int key = min(c0 + j * kLatKeys + lane, c1 - 1);
+    const long long slot = static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
+    const uint32_t dst = sb + ((j & 1) * kLatKeys + lane) * L.pitch;
+    __syncwarp();
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
+                 "l"(cache + slot * row), "r"(row * 2), "r"(mb) : "memory");
+  };
+  issue(0);
 
   float o[NT][4];
 #pragma unroll
   for (int x = 0; x < NT; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const int lm_mi = lane >> 3, lm_r = lane & 7;
   const int col0 = warp * NT * 8;                         // this warp's value columns
+  const int kt = warp & 3, kh = warp >> 2;                // its 8 keys and its half of the row in S
+  const int ks0 = kh * khalf, ks1 = min(k32, ks0 + khalf);
+  const uint32_t qaddr = sb + L.q + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
 
+  bool gave_up = false;
   for (int j = 0; j < ntile; ++j) {
-    cp_async_wait<0>();
-    __syncthreads();                    // tile j has landed; everyone is done with tile j - 1
+    const bool ok = mbar_wait(bar + (j & 1) * 8, (j >> 1) & 1, &s_abort);
+    gave_up = __syncthreads_or(!ok);    // tile j has landed; everyone is done with tile j - 1
+    if (gave_up) break;
     issue(j + 1);
     const uint32_t kb = sb + (j & 1) * kLatKeys * L.pitch;
     {
-      float s[4][4] = {};               // four independent sums: an MMA does not wait for the one before it
-      const uint32_t kaddr = kb + (warp * 8 + lm_r) * L.pitch + lm_mi * 16;
-#pragma unroll
-      for (int k = 0; k < K32; ++k)
-        if (k < k32) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
-          mma_bf16_16816(s[(2 * k) & 3], qa[2 * k], b0, b1);
-          mma_bf16_16816(s[(2 * k + 1) & 3], qa[2 * k + 1], b2, b3);
-        }
-      const int key = c0 + j * kLatKeys + warp * 8 + 2 * tq;
-      const bool v0 = key < c1, v1 = key + 1 < c1;
-      auto fin = [&](int e, bool v) { return v ? ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * scale_log2 : -INFINITY; };
-      float* dst = s_s + g * kLatSp + warp * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(dst) = make_float2(fin(0, v0), fin(1, v1));
-      *reinterpret_cast<float2*>(dst + 8 * kLatSp) = make_float2(fin(2, v0), fin(3, v1));
+      float s[2][4] = {};
+      const uint32_t kaddr = kb + (kt * 8 + lm_r) * L.pitch + lm_mi * 16;
+#pragma unroll 3
+      for (int k = ks0; k < ks1; ++k) {
+        uint32_t b0, b1, b2, b3, a0[4], a1[4];
+        ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
+        ldmatrix_x4(qaddr + k * 64, a0[0], a0[1], a0[2], a0[3]);
+        ldmatrix_x4(qaddr + k * 64 + 32, a1[0], a1[1], a1[2], a1[3]);
+        mma_bf16_16816(s[0], a0, b0, b1);
+        mma_bf16_16816(s[1], a1, b2, b3);
+      }
+      float* dst = s_s + (kh * 16 + g) * kLatSp + kt * 8 + 2 * tq;
+      *reinterpret_cast<float2*>(dst) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
+      *reinterpret_cast<float2*>(dst + 8 * kLatSp) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
     }
     __syncthreads();
     if (col0 < rankp) {
-      float p[2][16];                   // rows g, g + 8; columns 8 y + 2 tq + {0, 1}, y = 0 .. 7
+      float p[2][8];                    // rows g, g + 8; columns 8 y + 2 tq + {0, 1}, y = 0 .. 3
+      const int seen = c1 - (c0 + j * kLatKeys) - 2 * tq;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const float* src = s_s + (g + 8 * e) * kLatSp + 2 * tq;
         float mx = m[e];
 #pragma unroll
-        for (int y = 0; y < 8; ++y) {
+        for (int y = 0; y < 4; ++y) {
           const float2 v = *reinterpret_cast<const float2*>(src + 8 * y);
-          p[e][2 * y] = v.x;
-          p[e][2 * y + 1] = v.y;
-          mx = fmaxf(mx, fmaxf(v.x, v.y));
+          const float2 w = *reinterpret_cast<const float2*>(src + 16 * kLatSp + 8 * y);
+          p[e][2 * y] = 8 * y < seen ? (v.x + w.x) * scale_log2 : -INFINITY;
+          p[e][2 * y + 1] = 8 * y + 1 < seen ? (v.y + w.y) * scale_log2 : -INFINITY;
+          mx = fmaxf(mx, fmaxf(p[e][2 * y], p[e][2 * y + 1]));
         }
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));      // finite: the first key of the tile is visible
-        const float corr = exp2f(m[e] - mx);
+        const float corr = ex2(m[e] - mx);
         m[e] = mx;
         float sum = 0.f;
 #pragma unroll
-        for (int y = 0; y < 16; ++y) {
-          p[e][y] = exp2f(p[e][y] - mx);
+        for (int y = 0; y < 8; ++y) {
+          p[e][y] = ex2(p[e][y] - mx);
           sum += p[e][y];
         }
         l[e] = l[e] * corr + sum;       // of this lane's keys; the four lanes of a row add up at the end
@@ -284,7 +286,13 @@ latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, c
       }
     }
   }
-  cp_async_wait<0>();
+  if (gave_up) {
+    // every copy that was issued is one that was waited for, or the next one: give both a last, bounded chance to land
+    if (threadIdx.x == 0 && status != nullptr) atomicExch(status, kStatusBarrierTimeout);
+    for (int p = 0; p < 2; ++p)
+      for (int x = 0; x < (1 << 20) && !(mbar_try_wait(bar + 8 * p, 0) && mbar_try_wait(bar + 8 * p, 1)); ++x) {}
+    return;
+  }
   if (col0 >= rankp) return;
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -511,22 +519,24 @@ latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __
   }
 }
 
-template <int NT, int K32>
+template <int NT>
 static int launch_latent(const void* q, const void* cache, const int* bt, int max_blocks, const int* bt_row, const int* rows,
                          const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale, int window,
-                         const float* sink, int splits, void* out, float* ws, cudaStream_t stream) {
+                         const float* sink, int splits, void* out, float* ws, int* status,
+                         cudaStream_t stream) {
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT, K32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLatMaxSmem));
   });
   if (rc != 0) return rc;
   const int smem = latent_smem(row).total, groups = (heads + 15) / 16;
   const long long at = static_cast<long long>(heads) * n, ctas = static_cast<long long>(groups) * n;
-  if (smem > 227 * 1024 || ctas > 0x7fffffffll) return -11;
+  if (smem > kLatMaxSmem || ctas > 0x7fffffffll) return -11;
   float* part_lse = ws != nullptr ? ws + at * splits * rankp : nullptr;
-  latent_attn_kernel<NT, K32><<<dim3(static_cast<unsigned>(ctas), splits), kLatThreads, smem, stream>>>(
+  latent_attn_kernel<NT><<<dim3(static_cast<unsigned>(ctas), splits), kLatThreads, smem, stream>>>(
       static_cast<const bf16*>(q), static_cast<const bf16*>(cache), bt, max_blocks, bt_row, rows, ctx_len, block_size, n, heads,
-      groups, rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse);
+      groups, rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse,
+      status);
   if (splits > 1)
     latent_merge_kernel<<<static_cast<unsigned>(at), 128, 0, stream>>>(ws, part_lse, splits, rankp, static_cast<bf16*>(out));
   return static_cast<int>(cudaGetLastError());
@@ -579,18 +589,18 @@ extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* po
 extern "C" int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
                                      const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row,
                                      float scale, int window, const float* sink, int splits, void* out, float* workspace,
-                                     void* stream_) {
+                                     int* status, void* stream_) {
   if (heads < 1 || heads > 65535 || rankp < 8 || rankp % 8 != 0 || row % 8 != 0 || row < rankp || rankp > 512 || row > 640) return -10;
+  if ((reinterpret_cast<uintptr_t>(qa) & 15) != 0 || (reinterpret_cast<uintptr_t>(cache) & 15) != 0) return -10;
   if (block_size < 1 || splits < 1 || splits > 65535 || (splits > 1 && workspace == nullptr)) return -10;
   if (n == 0) return 0;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-#define DMOE_LAT(NT_, K_)                                                                                              \
-  return launch_latent<NT_, K_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, \
-                                row, scale, window, sink, splits, out, workspace, stream)
-  if (rankp <= 128 && row <= 192) DMOE_LAT(2, 6);
-  if (rankp <= 256 && row <= 320) DMOE_LAT(4, 10);
-  if (row <= 576) DMOE_LAT(8, 18);
-  DMOE_LAT(8, 20);
+#define DMOE_LAT(NT_)                                                                                                   \
+  return launch_latent<NT_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, row, \
+                            scale, window, sink, splits, out, workspace, status, stream)
+  if (rankp <= 128) DMOE_LAT(2);
+  if (rankp <= 256) DMOE_LAT(4);
+  DMOE_LAT(8);
 #undef DMOE_LAT
 }
 

@@ -713,16 +713,17 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, block_tables: torch.
     _lib.check(_lib.lib().dmoe_latent_attention(
         _vp(qa), _vp(cache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows), _vp(ctx_len),
         c_int(cache.shape[1]), c_int(n), c_int(H), c_int(lay.rankp), c_int(row), c_float(scale), c_int(window or 0), _vp(sink),
-        c_int(splits), _vp(out), _vp(ws), _st()), "dmoe_latent_attention")
+        c_int(splits), _vp(out), _vp(ws), _vp(scratch(qa.device).status), _st()), "dmoe_latent_attention")
     return out
 
 
 def pick_latent_splits(n: int, heads: int, reach: int) -> int:
-    """Key ranges per (query token, group of 16 heads) of :func:`latent_attention`, one CTA per SM each: as many waves of
-    CTAs as it takes to keep all SMs busy, never fewer than 128 keys per range."""
+    """Key ranges per (query token, group of 16 heads) of :func:`latent_attention`: the number whose waves of CTAs (two per
+    SM), with a few tiles' worth of start and merge per CTA, are done first."""
     from .gemm import num_sms
-    sms, ctas = num_sms(), max(1, n * ((heads + 15) // 16))
-    return max(1, min((4 * sms) // ctas, (reach + 127) // 128, 64))
+    slots, ctas = 2 * num_sms(), max(1, n * ((heads + 15) // 16))
+    cost = lambda s: -(-ctas * s // slots) * (-(-reach // (32 * s)) + (3 if s == 1 else 6))
+    return min(range(1, max(1, min(64, reach // 64)) + 1), key=cost)
 
 
 def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, keys: torch.Tensor, n_keys: int) -> torch.Tensor:
