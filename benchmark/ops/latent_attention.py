@@ -65,7 +65,7 @@ def main(argv=None) -> None:
         report("latent_attention (decode)", timed(run, a.steps, 3, flush), (B * N + 2 * H * B) * lay.row * 2,
                2.0 * B * N * H * (lay.row + lay.rankp))
     if a.only in ("", "decode"):
-        y, pos = rnd(B, H * lay.qd + lay.row), ctx - 1
+        y, pos = rnd(B, H * lay.qd + lay.kd), ctx - 1
         slots, table, nw = row.long() * N, F.rope_freq_table(m.rot, N, dev), torch.ones(a.rank, device=dev)
         report("latent_prep (decode)", timed(lambda: F.latent_prep(y, pos, slots, cache, lay, table, nw, 1e-6, None, B), a.steps, 3, flush),
                B * (2 * H * lay.qd + 2 * lay.row) * 2, 0)
@@ -82,7 +82,7 @@ def main(argv=None) -> None:
         pos = torch.arange(T)
         t = LatentTables.prefill(m, torch.zeros(T, dtype=torch.int32), pos, dev, dt)
         cache, bt = rnd(T // 16, 16, lay.row), torch.arange(T // 16, dtype=torch.int32, device=dev)[None]
-        y, out = rnd(T, H * lay.qd + lay.row), torch.empty(T, H * lay.vdimp, dtype=dt, device=dev)
+        y, out = rnd(T, H * lay.qd + lay.kd), torch.empty(T, H * lay.vdimp, dtype=dt, device=dev)
         w = rnd(H * (lay.dimp + lay.vdimp), lay.rankp) * 0.05
         slots, table, nw = pos.to(dev), F.rope_freq_table(m.rot, T, dev), torch.ones(a.rank, device=dev)
         report("latent_prep (prompt)", timed(lambda: F.latent_prep(y, pos.int().to(dev), slots, cache, lay, table, nw, 1e-6, t.loose, t.n_loose), a.steps, 3, flush),

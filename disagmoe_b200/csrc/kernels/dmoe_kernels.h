@@ -130,19 +130,20 @@ int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_
                        float scale, int window, float softcap, const float* sink, void* out, long long o_head, long long o_row,
                        void* stream);
 
-// ---- latent attention (latent_attention.cu): the cache has one row [latent rankp | rotated key part rotp] per token ---------
+// ---- latent attention (latent_attention.cu): the cache has one row [latent rankp | rotated key part rotp] per token,
+// `row` elements apart ------
 // Projection rows y = [heads x (q dimp | rotp) | latent rankp | key part rotp] (every part padded to a multiple of 8): RMS norm
 // of the latent, rotation of the key part, both to cache rows at slots (< 0: skip); rotation of the queries in place, and for
 // rows with loose[t] = i >= 0 (NULL: i = t) to xq [heads, n_loose, dimp] and columns rankp.. of qa [heads, n_loose, row].
 int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
-                     int heads, int dim, int rot_dim, int rank, int rot, int interleaved, const void* table, int max_pos,
+                     int heads, int dim, int rot_dim, int rank, int row, int rot, int interleaved, const void* table, int max_pos,
                      const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa, void* stream);
-// Queries qa [heads, n, row] over cache rows (keys: all of a row, values: its first rankp columns), out [heads, n, rankp];
-// rankp <= 512, row <= 640. workspace: heads * n * splits * (rankp + 1) floats where splits > 1. status (may be NULL): non-zero
+// Queries qa [heads, n, row] over cache rows (keys: the first kd columns, values: the first rankp), out [heads, n, rankp];
+// rankp <= 512, kd <= 640, row an odd multiple of 8, block_size a multiple of 16. workspace: heads * n * splits * (rankp + 1) floats where splits > 1. status (may be NULL): non-zero
 // after a bounded wait gave up.
 int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
-                          const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale,
-                          int window, const float* sink, int splits, void* out, float* workspace, int* status, void* stream);
+                          const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int kd, int row,
+                          float scale, int window, const float* sink, int splits, void* out, float* workspace, int* status, void* stream);
 // out[i] = cache row of position keys[i].y of block-table row keys[i].x
 int dmoe_latent_gather(const void* cache, const int* block_tables, int max_blocks, const void* keys, int n, int block_size,
                        int row, void* out, void* stream);

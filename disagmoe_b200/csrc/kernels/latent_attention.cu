@@ -1,5 +1,6 @@
 // Latent attention for sm_100a: keys and values of all heads are linear maps of one cached latent vector per token, plus one
-// rotated key part that the heads share. Cache row = [latent (rankp) | rotated key part (rotp)], bf16 (fp32 in fp32 runs).
+// rotated key part that the heads share. Cache row = [latent (rankp) | rotated key part (rotp)], bf16 (fp32 in
+// fp32 runs), rows an odd number of 16-byte units apart.
 //
 //   latent_prep_kernel     norm of the latent, rotations, cache append, queries head by head for the rows below
 //   latent_attn_kernel     rows on their own (decoding, short portions): the key map is already multiplied into the query, so
@@ -20,13 +21,13 @@ constexpr int pad8(int n) { return (n + 7) / 8 * 8; }
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
-                   T* __restrict__ cache, int heads, int dimp, int rotp, int rank, int rankp, int rot, int interleaved,
-                   const float2* __restrict__ table, int max_pos, const float* __restrict__ norm_w, float eps,
+                   T* __restrict__ cache, int heads, int dimp, int rotp, int rank, int rankp, int row, int rot,
+                   int interleaved, const float2* __restrict__ table, int max_pos, const float* __restrict__ norm_w, float eps,
                    const int* __restrict__ loose, int n_loose, T* __restrict__ xq, T* __restrict__ qa) {
   __shared__ float red[8];
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int half = rot / 2, qd = dimp + rotp, row = rankp + rotp;
+  const int half = rot / 2, qd = dimp + rotp;
   const int pos = min(max(positions[t], 0), max_pos - 1);
   const long long slot = slots[t];
   const int li = loose != nullptr ? loose[t] : static_cast<int>(t);
@@ -117,25 +118,39 @@ latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ bl
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Attention over the cached rows. A CTA of eight warps (two CTAs per SM) has one query token, 16 heads (the rows of its MMA
-// tiles) and one range of keys, which come 32 at a time, one bulk copy per cached row, into a double buffer. Per 32 keys: a warp
-// computes the scores of all heads with 8 keys over one half of the row (S = Q K^T) and leaves them in shared memory; after one
-// barrier every warp takes the whole 16 x 32 score tile back as its own A fragments, does the online softmax (all warps the same
-// one) and accumulates 8 NT value columns (O += P V, V = the same rows, P = hi + lo bf16).
-constexpr int kLatKeys = 32, kLatThreads = 256, kLatMaxSmem = 112 * 1024;
+// Attention over the cached rows. A CTA (one per SM) has one query token and one range of keys, which a producer warp brings 32
+// at a time, one bulk copy per 16 cached rows (consecutive in their page), into a ring of up to 8 tiles. Two groups of eight warps
+// consume them with a softmax state and accumulators of their own: up to 16 heads (the rows of the MMA tiles) take turns with the
+// tiles and merge at the end; of more heads each group has 16 and sees every tile. Per tile a warp computes the scores of its
+// group's heads with 8 keys over one half of the row (S = Q K^T) and leaves them in shared memory; after the tile's only barrier
+// every warp takes the whole 16 x 32 score tile back as its own A fragments, does the online softmax (all the same one) and
+// accumulates 8 NT value columns (O += P V, V = the same rows, P = hi + lo bf16).
+// Cached rows are an odd number of 16-byte units apart, so that ldmatrix meets no bank twice although they are copied as they are.
+constexpr int kLatKeys = 32, kLatPiece = 16, kLatThreads = 512 + 32, kLatMaxSmem = 226 * 1024, kLatMaxStages = 8;
 constexpr int kLatSp = kLatKeys + 8;        // pitch of a score row, floats: 64-bit reads of a fragment meet no bank twice
+constexpr int kLatScores = 2 * 16 * kLatSp; // of one tile: two halves of the row x 16 heads
 
 struct LatentSmem {      // bytes
-  int pitch, q, s, bars, total;
+  int qpitch, stages, q, s, bars, total;
 };
-__host__ __device__ inline LatentSmem latent_smem(int row) {
+__host__ __device__ inline LatentSmem latent_smem(int kd, int row) {
   LatentSmem s;
-  s.pitch = (row + 31) / 32 * 64 + 16;        // an odd number of 16-byte units: ldmatrix meets no bank twice
-  s.q = 2 * kLatKeys * s.pitch;
-  s.s = s.q + 16 * s.pitch;
-  s.bars = s.s + 2 * 16 * kLatSp * 4;
-  s.total = s.bars + 32;
+  s.qpitch = (kd + 31) / 32 * 64 + 16;
+  const int fixed = 32 * s.qpitch + 4 * kLatScores * 4 + 16 * kLatMaxStages, fit = (kLatMaxSmem - fixed) / (kLatKeys * row * 2);
+  s.stages = fit > kLatMaxStages ? kLatMaxStages : fit;
+  s.q = s.stages * kLatKeys * row * 2;
+  s.s = s.q + 32 * s.qpitch;
+  s.bars = s.s + 4 * kLatScores * 4;
+  s.total = s.bars + 16 * kLatMaxStages;
   return s;
+}
+// Barrier of the 256 threads of a group; true for all of them where `flag` is set for one.
+__device__ __forceinline__ bool group_sync_or(int id, bool flag) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, %2, 256, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+      : "=r"(r) : "r"(flag ? 1u : 0u), "r"(id) : "memory");
+  return r != 0;
 }
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -143,178 +158,222 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-// NT: 8-column tiles of the output per warp (rankp <= 64 NT)
+// NT: 8-column tiles of the output per warp (rankp <= 64 NT). kd: key size; row: elements from one cached row (or query) to the next.
 template <int NT>
-__global__ void __launch_bounds__(kLatThreads, 2)
+__global__ void __launch_bounds__(kLatThreads, 1)
 latent_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, const int* __restrict__ block_tables,
                    int max_blocks, const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len,
-                   int block_size, int n, int heads, int groups, int rankp, int row, float scale_log2, int window,
+                   int block_size, int n, int heads, int groups, int rankp, int kd, int row, float scale_log2, int window,
                    const float* __restrict__ sink, int splits, bf16* __restrict__ out, float* __restrict__ part_o,
                    float* __restrict__ part_lse, int* __restrict__ status) {
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ int s_abort;
-  const LatentSmem L = latent_smem(row);
+  const LatentSmem L = latent_smem(kd, row);
+  const int pitch = row * 2;
+  const bool both = heads > 16;         // both groups see every tile, 16 heads each
   // the head groups of a token are neighbours: they read the same rows at about the same time
-  const int i = blockIdx.x / groups, h0 = blockIdx.x % groups * 16, split = blockIdx.y;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int i = blockIdx.x / groups, cta_h0 = blockIdx.x % groups * (both ? 32 : 16), split = blockIdx.y;
+  const int warp = threadIdx.x >> 5 & 7, grp = threadIdx.x >> 8, lane = threadIdx.x & 31;   // warp within its group; 2: producer
   const int g = lane >> 2, tq = lane & 3;
   const int b = rows != nullptr ? rows[i] : i;
   const int len = ctx_len[b];
   const int* bt = block_tables + static_cast<long long>(bt_row != nullptr ? bt_row[b] : b) * max_blocks;
-  const int lo = window > 0 ? max(0, len - window) : 0;
-  const int per = ((len - lo + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
-  const int c0 = min(len, lo + split * per), c1 = min(len, c0 + per);
+  const int lo = window > 0 ? max(0, len - window) : 0, first = lo / kLatPiece * kLatPiece;
+  const int per = ((len - first + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
+  const int c0 = min(len, first + split * per), c1 = min(len, c0 + per);
   const int ntile = (c1 - c0 + kLatKeys - 1) / kLatKeys;
-  const int nch = row / 8, k32 = (row + 31) / 32, khalf = (k32 + 1) / 2;
-  const uint32_t sb = smem_u32(smem), bar = sb + L.bars;
-  float* s_s = reinterpret_cast<float*>(smem + L.s);      // [half of the row][16][kLatSp] partial scores
+  const int k32 = (kd + 31) / 32, khalf = (k32 + 1) / 2;
+  const uint32_t sb = smem_u32(smem), full = sb + L.bars, empty = full + 8 * kLatMaxStages;
 
   if (threadIdx.x == 0) {
     s_abort = 0;
-    mbar_init(bar, 1);
-    mbar_init(bar + 8, 1);
+    for (int x = 0; x < L.stages; ++x) {
+      mbar_init(full + 8 * x, 1);
+      mbar_init(empty + 8 * x, both ? 16 : 8);
+    }
     mbar_fence_init();
   }
-  // zeros where no copy ever writes: columns row .. 32 k32 of the keys and of the queries, and absent heads
-  const int tail = k32 * 4 - nch;                         // 16-byte units
-  for (int r = threadIdx.x; r < 2 * kLatKeys + 16; r += kLatThreads)
-    for (int c = 0; c < tail; ++c)
-      *reinterpret_cast<uint4*>(smem + r * L.pitch + (nch + c) * 16) = make_uint4(0, 0, 0, 0);
-  for (int r = warp; r < 16; r += kLatThreads / 32) {
-    const bf16* src = q + (static_cast<long long>(h0 + r) * n + i) * row;
-    for (int c = lane; c < nch; c += 32)
-      *reinterpret_cast<uint4*>(smem + L.q + r * L.pitch + c * 16) =
-          h0 + r < heads ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
+  // queries, zeros behind them and for absent heads; zeros for rows that neither the last tile nor one before it brings
+  for (int x = threadIdx.x; x < (both ? 32 : 16) * (k32 * 4); x += kLatThreads) {
+    const int r = x / (k32 * 4), c = x % (k32 * 4);
+    const bf16* src = q + (static_cast<long long>(cta_h0 + r) * n + i) * row + c * 8;
+    *reinterpret_cast<uint4*>(smem + L.q + r * L.qpitch + c * 16) =
+        cta_h0 + r < heads && c * 8 < kd ? *reinterpret_cast<const uint4*>(src) : make_uint4(0, 0, 0, 0);
+  }
+  if (ntile > 0 && ntile <= L.stages) {
+    const int have = c1 - c0 - (ntile - 1) * kLatKeys;
+    uint4* z = reinterpret_cast<uint4*>(smem + ((ntile - 1) * kLatKeys + have) * pitch);
+    for (int x = threadIdx.x; x < (kLatKeys - have) * (row / 8); x += kLatThreads) z[x] = make_uint4(0, 0, 0, 0);
   }
   __syncthreads();
-
-  auto issue = [&](int j) {             // warp 0: one row per lane; rows past the end repeat the last one (their weight is 0)
-    if (warp != 0 || j >= ntile) return;
-    const uint32_t mb = bar + (j & 1) * 8;
-    if (lane == 0) mbar_expect_tx(mb, kLatKeys * row * 2);
-    const int key = min(c0 + j * kLatKeys + lane, c1 - 1);
-    const long long slot = static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
-    const uint32_t dst = sb + ((j & 1) * kLatKeys + lane) * L.pitch;
-    __syncwarp();
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
-                 "l"(cache + slot * row), "r"(row * 2), "r"(mb) : "memory");
-  };
-  issue(0);
 
   float o[NT][4];
 #pragma unroll
   for (int x = 0; x < NT; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  const int lm_mi = lane >> 3, lm_r = lane & 7;
   const int col0 = warp * NT * 8;                         // this warp's value columns
-  const int kt = warp & 3, kh = warp >> 2;                // its 8 keys and its half of the row in S
-  const int ks0 = kh * khalf, ks1 = min(k32, ks0 + khalf);
-  const uint32_t qaddr = sb + L.q + (lm_r + (lm_mi & 1) * 8) * L.pitch + (lm_mi >> 1) * 16;
-
   bool gave_up = false;
-  for (int j = 0; j < ntile; ++j) {
-    const bool ok = mbar_wait(bar + (j & 1) * 8, (j >> 1) & 1, &s_abort);
-    gave_up = __syncthreads_or(!ok);    // tile j has landed; everyone is done with tile j - 1
-    if (gave_up) break;
-    issue(j + 1);
-    const uint32_t kb = sb + (j & 1) * kLatKeys * L.pitch;
-    {
-      float s[2][4] = {};
-      const uint32_t kaddr = kb + (kt * 8 + lm_r) * L.pitch + lm_mi * 16;
-#pragma unroll 3
-      for (int k = ks0; k < ks1; ++k) {
-        uint32_t b0, b1, b2, b3, a0[4], a1[4];
-        ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
-        ldmatrix_x4(qaddr + k * 64, a0[0], a0[1], a0[2], a0[3]);
-        ldmatrix_x4(qaddr + k * 64 + 32, a1[0], a1[1], a1[2], a1[3]);
-        mma_bf16_16816(s[0], a0, b0, b1);
-        mma_bf16_16816(s[1], a1, b2, b3);
-      }
-      float* dst = s_s + (kh * 16 + g) * kLatSp + kt * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(dst) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
-      *reinterpret_cast<float2*>(dst + 8 * kLatSp) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
+  if (grp == 2) {
+    // producer: lane 0 and 1 have a piece of every tile
+    for (int j = 0; j < ntile; ++j) {
+      const int st = j % L.stages, key = c0 + j * kLatKeys + lane * kLatPiece;
+      const int have = lane < 2 ? min(kLatPiece, c1 - key) : 0;
+      long long slot = 0;
+      if (have > 0) slot = static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
+      if (j >= L.stages) gave_up = !mbar_wait(empty + 8 * st, (j / L.stages - 1) & 1, &s_abort);
+      if (__any_sync(0xffffffffu, gave_up)) { gave_up = true; break; }
+      if (lane == 0) mbar_expect_tx(full + 8 * st, min(kLatKeys, c1 - key) * pitch);
+      __syncwarp();
+      if (have > 0)
+        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                         sb + (st * kLatKeys + lane * kLatPiece) * pitch), "l"(cache + slot * row), "r"(have * pitch),
+                     "r"(full + 8 * st) : "memory");
     }
-    __syncthreads();
-    if (col0 < rankp) {
-      float p[2][8];                    // rows g, g + 8; columns 8 y + 2 tq + {0, 1}, y = 0 .. 3
-      const int seen = c1 - (c0 + j * kLatKeys) - 2 * tq;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float* src = s_s + (g + 8 * e) * kLatSp + 2 * tq;
-        float mx = m[e];
-#pragma unroll
-        for (int y = 0; y < 4; ++y) {
-          const float2 v = *reinterpret_cast<const float2*>(src + 8 * y);
-          const float2 w = *reinterpret_cast<const float2*>(src + 16 * kLatSp + 8 * y);
-          p[e][2 * y] = 8 * y < seen ? (v.x + w.x) * scale_log2 : -INFINITY;
-          p[e][2 * y + 1] = 8 * y + 1 < seen ? (v.y + w.y) * scale_log2 : -INFINITY;
-          mx = fmaxf(mx, fmaxf(p[e][2 * y], p[e][2 * y + 1]));
+  } else {
+    // [group][its tile & 1][half of the row][16][kLatSp] partial scores
+    float* s_s = reinterpret_cast<float*>(smem + L.s) + grp * 2 * kLatScores;
+    const int lm_mi = lane >> 3, lm_r = lane & 7;
+    const int kt = warp & 3, kh = warp >> 2;              // its 8 keys and its half of the row in S
+    const int ks0 = kh * khalf, ks1 = min(k32, ks0 + khalf);
+    const uint32_t qaddr = sb + L.q + (both ? grp * 16 * L.qpitch : 0) + (lm_r + (lm_mi & 1) * 8) * L.qpitch + (lm_mi >> 1) * 16;
+    int buf = 0;
+    for (int j = both ? 0 : grp; j < ntile; j += both ? 1 : 2) {
+      const int st = j % L.stages;
+      const bool ok = mbar_wait(full + st * 8, j / L.stages & 1, &s_abort);
+      const uint32_t kb = sb + st * kLatKeys * pitch;
+      float* sj = s_s + buf * kLatScores;
+      buf ^= 1;
+      {
+        float s[2][4] = {};
+        const uint32_t kaddr = kb + (kt * 8 + lm_r) * pitch + lm_mi * 16;
+#pragma unroll 3
+        for (int k = ks0; k < ks1; ++k) {
+          uint32_t b0, b1, b2, b3, a0[4], a1[4];
+          ldmatrix_x4(kaddr + k * 64, b0, b1, b2, b3);
+          ldmatrix_x4(qaddr + k * 64, a0[0], a0[1], a0[2], a0[3]);
+          ldmatrix_x4(qaddr + k * 64 + 32, a1[0], a1[1], a1[2], a1[3]);
+          if (k * 32 + 32 > kd) {       // what lies behind a key is not part of it
+            if (k * 32 + 8 >= kd) b1 = 0u;
+            if (k * 32 + 16 >= kd) b2 = 0u;
+            if (k * 32 + 24 >= kd) b3 = 0u;
+          }
+          mma_bf16_16816(s[0], a0, b0, b1);
+          mma_bf16_16816(s[1], a1, b2, b3);
         }
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));      // finite: the first key of the tile is visible
-        const float corr = ex2(m[e] - mx);
-        m[e] = mx;
-        float sum = 0.f;
-#pragma unroll
-        for (int y = 0; y < 8; ++y) {
-          p[e][y] = ex2(p[e][y] - mx);
-          sum += p[e][y];
-        }
-        l[e] = l[e] * corr + sum;       // of this lane's keys; the four lanes of a row add up at the end
-#pragma unroll
-        for (int x = 0; x < NT; ++x) { o[x][2 * e] *= corr; o[x][2 * e + 1] *= corr; }
+        float* dst = sj + (kh * 16 + g) * kLatSp + kt * 8 + 2 * tq;
+        *reinterpret_cast<float2*>(dst) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
+        *reinterpret_cast<float2*>(dst + 8 * kLatSp) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
       }
+      gave_up = group_sync_or(1 + grp, !ok);
+      if (gave_up) break;
+      if (col0 < rankp) {
+        float p[2][8];                  // rows g, g + 8; columns 8 y + 2 tq + {0, 1}, y = 0 .. 3
+        const int key = c0 + j * kLatKeys + 2 * tq, seen = c1 - key, from = lo - key;      // visible: from <= column < seen
 #pragma unroll
-      for (int ks = 0; ks < kLatKeys / 16; ++ks) {
-        uint32_t ph[4], pl[4];
-        split2(p[0][4 * ks], p[0][4 * ks + 1], ph[0], pl[0]);
-        split2(p[1][4 * ks], p[1][4 * ks + 1], ph[1], pl[1]);
-        split2(p[0][4 * ks + 2], p[0][4 * ks + 3], ph[2], pl[2]);
-        split2(p[1][4 * ks + 2], p[1][4 * ks + 3], ph[3], pl[3]);
-        const uint32_t va = kb + (ks * 16 + (lm_mi & 1) * 8 + lm_r) * L.pitch + col0 * 2 + (lm_mi >> 1) * 16;
+        for (int e = 0; e < 2; ++e) {
+          const float* src = sj + (g + 8 * e) * kLatSp + 2 * tq;
+          float mx = m[e];
 #pragma unroll
-        for (int dp = 0; dp < NT / 2; ++dp) {
-          if (col0 + dp * 16 < rankp) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(va + dp * 32, b0, b1, b2, b3);
-            mma_bf16_16816(o[2 * dp], ph, b0, b1);
-            mma_bf16_16816(o[2 * dp + 1], ph, b2, b3);
-            mma_bf16_16816(o[2 * dp], pl, b0, b1);
-            mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
+          for (int y = 0; y < 4; ++y) {
+            const float2 v = *reinterpret_cast<const float2*>(src + 8 * y);
+            const float2 w = *reinterpret_cast<const float2*>(src + 16 * kLatSp + 8 * y);
+            p[e][2 * y] = 8 * y < seen && 8 * y >= from ? (v.x + w.x) * scale_log2 : -INFINITY;
+            p[e][2 * y + 1] = 8 * y + 1 < seen && 8 * y + 1 >= from ? (v.y + w.y) * scale_log2 : -INFINITY;
+            mx = fmaxf(mx, fmaxf(p[e][2 * y], p[e][2 * y + 1]));
+          }
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));      // finite: every tile has a visible key
+          const float corr = ex2(m[e] - mx);
+          m[e] = mx;
+          float sum = 0.f;
+#pragma unroll
+          for (int y = 0; y < 8; ++y) {
+            p[e][y] = ex2(p[e][y] - mx);
+            sum += p[e][y];
+          }
+          l[e] = l[e] * corr + sum;     // of this lane's keys; the four lanes of a row add up at the end
+#pragma unroll
+          for (int x = 0; x < NT; ++x) { o[x][2 * e] *= corr; o[x][2 * e + 1] *= corr; }
+        }
+#pragma unroll
+        for (int ks = 0; ks < kLatKeys / 16; ++ks) {
+          uint32_t ph[4], pl[4];
+          split2(p[0][4 * ks], p[0][4 * ks + 1], ph[0], pl[0]);
+          split2(p[1][4 * ks], p[1][4 * ks + 1], ph[1], pl[1]);
+          split2(p[0][4 * ks + 2], p[0][4 * ks + 3], ph[2], pl[2]);
+          split2(p[1][4 * ks + 2], p[1][4 * ks + 3], ph[3], pl[3]);
+          const uint32_t va = kb + (ks * 16 + (lm_mi & 1) * 8 + lm_r) * pitch + col0 * 2 + (lm_mi >> 1) * 16;
+#pragma unroll
+          for (int dp = 0; dp < NT / 2; ++dp) {
+            if (col0 + dp * 16 < rankp) {
+              uint32_t b0, b1, b2, b3;
+              ldmatrix_x4_trans(va + dp * 32, b0, b1, b2, b3);
+              mma_bf16_16816(o[2 * dp], ph, b0, b1);
+              mma_bf16_16816(o[2 * dp + 1], ph, b2, b3);
+              mma_bf16_16816(o[2 * dp], pl, b0, b1);
+              mma_bf16_16816(o[2 * dp + 1], pl, b2, b3);
+            }
           }
         }
       }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(empty + 8 * st);
     }
   }
-  if (gave_up) {
-    // every copy that was issued is one that was waited for, or the next one: give both a last, bounded chance to land
+  if (__syncthreads_or(gave_up)) {
+    // copies may be in flight: give every barrier a last, bounded chance
     if (threadIdx.x == 0 && status != nullptr) atomicExch(status, kStatusBarrierTimeout);
-    for (int p = 0; p < 2; ++p)
-      for (int x = 0; x < (1 << 20) && !(mbar_try_wait(bar + 8 * p, 0) && mbar_try_wait(bar + 8 * p, 1)); ++x) {}
+    for (int p = 0; p < L.stages; ++p)
+      for (int x = 0; x < (1 << 20) && !(mbar_try_wait(full + 8 * p, 0) && mbar_try_wait(full + 8 * p, 1)); ++x) {}
     return;
   }
-  if (col0 >= rankp) return;
+  // heads that took turns: the second group leaves its state where the ring was, [16][m, sum], then accumulators as
+  // [warp][value][lane]
+  float* s_ml = reinterpret_cast<float*>(smem);
+  float* s_o = s_ml + 32 + warp * (NT * 4 * 32) + lane;
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
-    float den = l[e];
-    den += __shfl_xor_sync(0xffffffffu, den, 1);
-    den += __shfl_xor_sync(0xffffffffu, den, 2);
-    const int head = h0 + g + 8 * e;
-    if (head >= heads) continue;
-    float mm = m[e], f = 1.f;
-    if (sink != nullptr && split == 0 && len > 0) {       // one split carries the sink
-      const float sk = sink[head] * kLog2e, mn = fmaxf(mm, sk);
-      f = exp2f(mm - mn);
-      den = den * f + exp2f(sk - mn);
-      mm = mn;
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+  }
+  if (grp == 1 && !both) {
+    if (warp == 0 && tq == 0) {
+      s_ml[2 * g] = m[0]; s_ml[2 * g + 1] = l[0];
+      s_ml[2 * (g + 8)] = m[1]; s_ml[2 * (g + 8) + 1] = l[1];
     }
-    f = den > 0.f ? f / den : 0.f;
+#pragma unroll
+    for (int x = 0; x < NT; ++x)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s_o[(x * 4 + e) * 32] = o[x][e];
+  }
+  __syncthreads();
+  if (grp == 2 || (grp == 1 && !both) || col0 >= rankp) return;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int head = cta_h0 + (both ? grp * 16 : 0) + g + 8 * e;
+    if (head >= heads) continue;
+    const float m1 = both ? -INFINITY : s_ml[2 * (g + 8 * e)], l1 = both ? 0.f : s_ml[2 * (g + 8 * e) + 1];
+    const bool sunk = sink != nullptr && split == 0 && len > 0;      // one split carries the sink
+    const float sk = sunk ? sink[head] * kLog2e : -INFINITY;
+    const float mm = fmaxf(fmaxf(m[e], m1), sk);
+    float f0 = 0.f, f1 = 0.f, den = 0.f;
+    if (mm > -INFINITY) {
+      f0 = exp2f(m[e] - mm);
+      f1 = exp2f(m1 - mm);
+      den = l[e] * f0 + l1 * f1 + (sunk ? exp2f(sk - mm) : 0.f);
+      f0 /= den;
+      f1 /= den;
+    }
     const long long at = static_cast<long long>(head) * n + i;
 #pragma unroll
     for (int x = 0; x < NT; ++x) {
       const int col = col0 + x * 8 + 2 * tq;
       if (col >= rankp) continue;
-      const float a = o[x][2 * e] * f, c = o[x][2 * e + 1] * f;
+      float a = o[x][2 * e] * f0, c = o[x][2 * e + 1] * f0;
+      if (!both) {
+        a += s_o[(x * 4 + 2 * e) * 32] * f1;
+        c += s_o[(x * 4 + 2 * e + 1) * 32] * f1;
+      }
       if (splits == 1) *reinterpret_cast<uint32_t*>(out + at * rankp + col) = pack_bf16(a, c);
       else *reinterpret_cast<float2*>(part_o + (at * splits + split) * rankp + col) = make_float2(a, c);
     }
@@ -521,7 +580,7 @@ latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __
 
 template <int NT>
 static int launch_latent(const void* q, const void* cache, const int* bt, int max_blocks, const int* bt_row, const int* rows,
-                         const int* ctx_len, int block_size, int n, int heads, int rankp, int row, float scale, int window,
+                         const int* ctx_len, int block_size, int n, int heads, int rankp, int kd, int row, float scale, int window,
                          const float* sink, int splits, void* out, float* ws, int* status,
                          cudaStream_t stream) {
   static PerDeviceOnce configured;
@@ -529,13 +588,14 @@ static int launch_latent(const void* q, const void* cache, const int* bt, int ma
     return static_cast<int>(cudaFuncSetAttribute(latent_attn_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLatMaxSmem));
   });
   if (rc != 0) return rc;
-  const int smem = latent_smem(row).total, groups = (heads + 15) / 16;
+  const LatentSmem L = latent_smem(kd, row);
+  const int smem = L.total, groups = heads > 16 ? (heads + 31) / 32 : 1;
   const long long at = static_cast<long long>(heads) * n, ctas = static_cast<long long>(groups) * n;
-  if (smem > kLatMaxSmem || ctas > 0x7fffffffll) return -11;
+  if (L.stages < 2 || smem > kLatMaxSmem || ctas > 0x7fffffffll) return -11;
   float* part_lse = ws != nullptr ? ws + at * splits * rankp : nullptr;
   latent_attn_kernel<NT><<<dim3(static_cast<unsigned>(ctas), splits), kLatThreads, smem, stream>>>(
       static_cast<const bf16*>(q), static_cast<const bf16*>(cache), bt, max_blocks, bt_row, rows, ctx_len, block_size, n, heads,
-      groups, rankp, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse,
+      groups, rankp, kd, row, scale * kLog2e, window, sink, splits, static_cast<bf16*>(out), ws, part_lse,
       status);
   if (splits > 1)
     latent_merge_kernel<<<static_cast<unsigned>(at), 128, 0, stream>>>(ws, part_lse, splits, rankp, static_cast<bf16*>(out));
@@ -564,20 +624,22 @@ static int launch_latent_prefill(const void* q, long long ld_q, const void* kv, 
 using namespace dmoe;
 
 extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
-                                int heads, int dim, int rot_dim, int rank, int rot, int interleaved, const void* table,
+                                int heads, int dim, int rot_dim, int rank, int row, int rot, int interleaved, const void* table,
                                 int max_pos, const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa,
                                 void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (heads < 1 || dim < 1 || rot_dim < 0 || rank < 1 || rot < 0 || rot % 2 != 0 || rot > rot_dim || (rot > 0 && table == nullptr)) return -10;
   const int align = is_f32 ? 4 : 8;
+  if (row % align != 0 || row < pad8(rank) + pad8(rot_dim)) return -10;
   if (ld % align != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 || (loose == nullptr && n_loose < T)) return -10;
   if (T == 0) return 0;
   const int dimp = pad8(dim), rotp = pad8(rot_dim), rankp = pad8(rank);
   const bool vec = interleaved && rot == rotp && rot > 0;
 #define DMOE_PREP(T_, VEC_)                                                                                                  \
   latent_prep_kernel<T_, VEC_><<<T, 256, 0, stream>>>(                                                                       \
-      static_cast<T_*>(y), ld, positions, slots, static_cast<T_*>(cache), heads, dimp, rotp, rank, rankp, rot, interleaved,  \
-      static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<T_*>(xq), static_cast<T_*>(qa))
+      static_cast<T_*>(y), ld, positions, slots, static_cast<T_*>(cache), heads, dimp, rotp, rank, rankp, row, rot,          \
+      interleaved, static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<T_*>(xq),            \
+      static_cast<T_*>(qa))
   if (is_f32 && vec) DMOE_PREP(float, true);
   else if (is_f32) DMOE_PREP(float, false);
   else if (vec) DMOE_PREP(bf16, true);
@@ -587,17 +649,18 @@ extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* po
 }
 
 extern "C" int dmoe_latent_attention(const void* qa, const void* cache, const int* block_tables, int max_blocks, const int* bt_row,
-                                     const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int row,
+                                     const int* rows, const int* ctx_len, int block_size, int n, int heads, int rankp, int kd, int row,
                                      float scale, int window, const float* sink, int splits, void* out, float* workspace,
                                      int* status, void* stream_) {
-  if (heads < 1 || heads > 65535 || rankp < 8 || rankp % 8 != 0 || row % 8 != 0 || row < rankp || rankp > 512 || row > 640) return -10;
+  if (heads < 1 || heads > 65535 || rankp < 8 || rankp % 8 != 0 || kd % 8 != 0 || kd < rankp || row < kd || rankp > 512 || kd > 640) return -10;
+  if (row % 16 != 8 || block_size % kLatPiece != 0) return -10;
   if ((reinterpret_cast<uintptr_t>(qa) & 15) != 0 || (reinterpret_cast<uintptr_t>(cache) & 15) != 0) return -10;
-  if (block_size < 1 || splits < 1 || splits > 65535 || (splits > 1 && workspace == nullptr)) return -10;
+  if (splits < 1 || splits > 65535 || (splits > 1 && workspace == nullptr)) return -10;
   if (n == 0) return 0;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
 #define DMOE_LAT(NT_)                                                                                                   \
-  return launch_latent<NT_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, row, \
-                            scale, window, sink, splits, out, workspace, status, stream)
+  return launch_latent<NT_>(qa, cache, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n, heads, rankp, kd, \
+                            row, scale, window, sink, splits, out, workspace, status, stream)
   if (rankp <= 128) DMOE_LAT(2);
   if (rankp <= 256) DMOE_LAT(4);
   DMOE_LAT(8);

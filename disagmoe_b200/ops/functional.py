@@ -621,7 +621,8 @@ class LatentLayout:
     """Sizes of a latent attention layer as its kernels see them: every part of a row is padded to a multiple of 8 (zeros).
 
     projection row   [heads x (q unrotated | q rotated) | latent | rotated key part]
-    cache row        [latent | rotated key part]
+    cache row        [latent | rotated key part], an odd multiple of 8 elements from one row to the next: tiles that are copied
+                     to shared memory as they are read without bank conflicts
     """
     heads: int
     dim: int
@@ -650,8 +651,12 @@ class LatentLayout:
         return self.dimp + self.rotp
 
     @property
-    def row(self) -> int:
+    def kd(self) -> int:
         return self.rankp + self.rotp
+
+    @property
+    def row(self) -> int:
+        return self.kd + (8 if self.kd % 16 == 0 else 0)
 
     def min_run(self) -> int:
         """Prompt tokens from which expanding the latents of all visible keys pays: it costs rank * (dim + vdim) per key and
@@ -665,7 +670,7 @@ class LatentLayout:
 
 
 LATENT_TILES = ((96, 64), (128, 128), (192, 128))     # (key, value) sizes of the prompt kernel
-LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 640            # of the tensor-core kernel over the latent cache
+LATENT_MAX_RANK, LATENT_MAX_KEY = 512, 640            # of the tensor-core kernel over the latent cache
 
 
 def latent_prep(y: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, lay: LatentLayout,
@@ -679,13 +684,13 @@ def latent_prep(y: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, c
     if not y.is_cuda:
         return reference.latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved)
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and y.stride(1) == 1 and cache.is_contiguous()
-    assert y.shape[1] == lay.heads * lay.qd + lay.row and cache.dtype == y.dtype and norm_w.dtype == torch.float32
+    assert y.shape[1] == lay.heads * lay.qd + lay.kd and cache.dtype == y.dtype and norm_w.dtype == torch.float32
     xq = torch.empty(lay.heads, n_loose, lay.dimp, dtype=y.dtype, device=y.device)
     qa = torch.empty(lay.heads, n_loose, lay.row, dtype=y.dtype, device=y.device)
     rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
     _lib.check(_lib.lib().dmoe_latent_prep(
         _f32(y.dtype), _vp(y), c_ll(y.stride(0)), _vp(positions), _vp(slots), _vp(cache), c_int(y.shape[0]), c_int(lay.heads),
-        c_int(lay.dim), c_int(lay.rot), c_int(lay.rank), c_int(rot), c_int(int(interleaved)), _vp(table), c_int(max_pos),
+        c_int(lay.dim), c_int(lay.rot), c_int(lay.rank), c_int(lay.row), c_int(rot), c_int(int(interleaved)), _vp(table), c_int(max_pos),
         _vp(norm_w), c_float(eps), _vp(loose), c_int(n_loose), _vp(xq), _vp(qa), _st()), "dmoe_latent_prep")
     return xq, qa
 
@@ -704,25 +709,26 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, block_tables: torch.
         return o.view(n, H, lay.rankp).transpose(0, 1).contiguous()
     out = torch.empty(H, n, lay.rankp, dtype=qa.dtype, device=qa.device)
     _check_sink(sink, H)
-    if qa.dtype == torch.float32 or lay.rankp > LATENT_MAX_RANK or lay.row > LATENT_MAX_ROW:
-        return _any_attention(qa, n * row, row, k3, k3[..., :lay.rankp], block_tables, bt_row, rows, ctx_len, n, H, 1, row,
+    if qa.dtype == torch.float32 or lay.rankp > LATENT_MAX_RANK or lay.kd > LATENT_MAX_KEY or cache.shape[1] % 16:
+        return _any_attention(qa, n * row, row, k3, k3[..., :lay.rankp], block_tables, bt_row, rows, ctx_len, n, H, 1, lay.kd,
                               lay.rankp, scale, window, None, sink, out, n * lay.rankp, lay.rankp)
     reach = min(max_ctx, window or max_ctx)
     splits = pick_latent_splits(n, H, reach)
     ws = _attn_workspace(qa.device, H * n * splits * (lay.rankp + 1)) if splits > 1 else None
     _lib.check(_lib.lib().dmoe_latent_attention(
         _vp(qa), _vp(cache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows), _vp(ctx_len),
-        c_int(cache.shape[1]), c_int(n), c_int(H), c_int(lay.rankp), c_int(row), c_float(scale), c_int(window or 0), _vp(sink),
+        c_int(cache.shape[1]), c_int(n), c_int(H), c_int(lay.rankp), c_int(lay.kd), c_int(row), c_float(scale), c_int(window or 0), _vp(sink),
         c_int(splits), _vp(out), _vp(ws), _vp(scratch(qa.device).status), _st()), "dmoe_latent_attention")
     return out
 
 
 def pick_latent_splits(n: int, heads: int, reach: int) -> int:
-    """Key ranges per (query token, group of 16 heads) of :func:`latent_attention`: the number whose waves of CTAs (two per
-    SM), with a few tiles' worth of start and merge per CTA, are done first."""
+    """Key ranges per (query token, group of heads) of :func:`latent_attention`: the number whose waves of CTAs (one per SM, 16
+    heads and 64 keys at a time, or 32 and 32), with some start and merge per CTA, are done first."""
     from .gemm import num_sms
-    slots, ctas = 2 * num_sms(), max(1, n * ((heads + 15) // 16))
-    cost = lambda s: -(-ctas * s // slots) * (-(-reach // (32 * s)) + (3 if s == 1 else 6))
+    slots, ctas = num_sms(), max(1, n * ((heads + 31) // 32))
+    keys = 64 if heads <= 16 else 32
+    cost = lambda s: -(-ctas * s // slots) * (-(-reach // (keys * s)) + (3 if s == 1 else 5))
     return min(range(1, max(1, min(64, reach // 64)) + 1), key=cost)
 
 

@@ -215,7 +215,7 @@ def test_latent_attention(window, H, D, R, V, K, dtype):
     qq = torch.cat([q[..., :D].double(), oracle.rotate_pairs(q[..., D:].double(), spec)], -1)
     want = attend(qq, key, (c @ uv.double().T).view(T, H, V), m.scale, sink, window)
     # rows as the projection leaves them
-    y = torch.zeros(T, H * lay.qd + lay.row, dtype=dtype)
+    y = torch.zeros(T, H * lay.qd + lay.kd, dtype=dtype)
     yq = y[:, :H * lay.qd].view(T, H, lay.qd)
     yq[..., :D], yq[..., lay.dimp:lay.dimp + R] = q[..., :D], q[..., D:]
     y[:, H * lay.qd:H * lay.qd + K], y[:, H * lay.qd + lay.rankp:H * lay.qd + lay.rankp + R] = d[:, :K], d[:, K:]
