@@ -85,7 +85,8 @@ def main(argv=None) -> None:
         y, out = rnd(T, H * lay.qd + lay.kd), torch.empty(T, H * lay.vdimp, dtype=dt, device=dev)
         w = rnd(H * (lay.dimp + lay.vdimp), lay.rankp) * 0.05
         slots, table, nw = pos.to(dev), F.rope_freq_table(m.rot, T, dev), torch.ones(a.rank, device=dev)
-        report("latent_prep (prompt)", timed(lambda: F.latent_prep(y, pos.int().to(dev), slots, cache, lay, table, nw, 1e-6, t.loose, t.n_loose), a.steps, 3, flush),
+        pos = pos.int().to(dev)
+        report("latent_prep (prompt)", timed(lambda: F.latent_prep(y, pos, slots, cache, lay, table, nw, 1e-6, t.loose, t.n_loose), a.steps, 3, flush),
                T * (2 * H * lay.rotp + 2 * lay.row) * 2, 0)
         lat = F.latent_gather(cache, bt, t.keys, t.n_keys)
         report("latent_gather", timed(lambda: F.latent_gather(cache, bt, t.keys, t.n_keys), a.steps, 3, flush), 2 * T * lay.row * 2, 0)

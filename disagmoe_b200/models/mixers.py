@@ -10,6 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
+import numpy as np
 import torch
 
 from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig
@@ -82,19 +83,21 @@ class LatentTables:
         rows = (~covered).nonzero()[:, 0].int()
         loose = torch.full((T,), -1, dtype=torch.int32)
         loose[rows.long()] = torch.arange(len(rows), dtype=torch.int32)
-        base, keys, at, prev = [], [], 0, (-1, -1)
-        for r0, n, row, pos in tiles.tolist():
-            if (row, pos) != prev:              # a new run: its keys start a window before its first token
-                lo = max(0, pos - m.window + 1) if m.window else 0
-                off = at - lo
-                hi = lo
-            grow = torch.arange(hi, pos + n, dtype=torch.int32)
-            keys.append(torch.stack([torch.full_like(grow, row), grow], 1))
-            at, hi, prev = at + len(grow), pos + n, (row, pos + n)
-            base.append(off)
-        keys = torch.cat(keys)
+        # runs of tiles: the keys of a run start a window before its first token and end with its last
+        tl = tiles.numpy()
+        n, row, pos = tl[:, 1], tl[:, 2], tl[:, 3]
+        begins = np.nonzero(np.r_[True, (row[1:] != row[:-1]) | (pos[1:] != pos[:-1] + n[:-1])])[0]
+        ends = np.r_[begins[1:], len(tl)] - 1
+        lo = np.maximum(0, pos[begins] - m.window + 1) if m.window else np.zeros_like(begins)
+        hi = pos[ends] + n[ends]
+        at = np.r_[0, np.cumsum(hi - lo)]
+        keys = np.empty((at[-1], 2), dtype=np.int32)
+        for i, (a, b) in enumerate(zip(at[:-1], at[1:])):
+            keys[a:b, 0], keys[a:b, 1] = row[begins[i]], np.arange(lo[i], hi[i])
+        base = torch.from_numpy(np.repeat(at[:-1] - lo, ends - begins + 1).astype(np.int32))
+        keys = torch.from_numpy(keys)
         t = cls(len(rows), loose.to(device), rows.to(device), None, None, tiles.to(device),
-                torch.tensor(base, dtype=torch.int32).to(device), len(tiles), keys.to(device), len(keys))
+                base.to(device), len(tiles), keys.to(device), len(keys))
         if len(rows):
             t.offs, t.recs = cls._per_head(rows, m.heads, device)
         return t
