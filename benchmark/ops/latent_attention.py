@@ -71,11 +71,11 @@ def main(argv=None) -> None:
                B * (2 * H * lay.qd + 2 * lay.row) * 2, 0)
         t = LatentTables.decode(m, B, dev)
         xq, w = rnd(H * B, lay.dimp), rnd(H, lay.rankp, lay.dimp)
-        report("key map into the query (grouped GEMM)", timed(lambda: gemm.grouped_linear(xq, w, t.offs, out=qa.view(-1, lay.row)[:, :lay.rankp]), a.steps, 3, flush),
+        report("key map into the query (grouped GEMM)", timed(lambda: gemm.grouped_linear(xq, w, t.offs, out=qa.view(-1, lay.row)[:, :lay.rankp], bn=gemm.pick_even_bn(B, lay.rankp, H)), a.steps, 3, flush),
                (xq.numel() + w.numel() + H * B * lay.rankp) * 2, 2.0 * H * B * lay.dimp * lay.rankp)
         o, wv, out = rnd(H * B, lay.rankp), rnd(H, lay.vdimp, lay.rankp), rnd(B, H * lay.vdimp)
         base = torch.tensor([out.data_ptr()], dtype=torch.int64, device=dev)
-        report("value map of the outputs (grouped GEMM)", timed(lambda: gemm.grouped_combine(o, wv, t.offs, t.recs, base, lay.vdimp), a.steps, 3, flush),
+        report("value map of the outputs (grouped GEMM)", timed(lambda: gemm.grouped_combine(o, wv, t.offs, t.recs, base, lay.vdimp, bn=gemm.pick_even_bn(B, lay.vdimp, H)), a.steps, 3, flush),
                (o.numel() + wv.numel() + out.numel()) * 2, 2.0 * H * B * lay.vdimp * lay.rankp)
     if a.only in ("", "prefill"):
         T = a.prompt

@@ -294,11 +294,13 @@ class LatentAttention(Mixer):
         out = meta.latent_out[m.heads * lay.vdimp]
         attn = out.rows[:T]
         if t.n_loose:
-            gemm.grouped_linear(xq.view(-1, lay.dimp), self.absorb, t.offs, out=qa.view(-1, lay.row)[:, :lay.rankp])
+            bn = lambda F_: gemm.pick_even_bn(t.n_loose, F_, m.heads) if h.is_cuda else 0
+            gemm.grouped_linear(xq.view(-1, lay.dimp), self.absorb, t.offs, out=qa.view(-1, lay.row)[:, :lay.rankp],
+                                bn=bn(lay.rankp))
             o = F.latent_attention(qa, cache, meta.block_tables, meta.bt_row, meta.ctx_len, t.rows, lay, m.scale, m.window,
                                    self.sink, meta.max_ctx)
             gemm.grouped_combine(o.view(-1, lay.rankp), self.expand_v, t.offs, t.recs, out.base, lay.vdimp,
-                                 outs=[attn.view(-1, lay.vdimp)])
+                                 bn=bn(lay.vdimp), outs=[attn.view(-1, lay.vdimp)])
         if t.n_tiles:
             lat = F.latent_gather(cache, meta.block_tables, t.keys, t.n_keys)
             kvx = gemm.linear(lat[:, :lay.rankp], self.expand)

@@ -120,6 +120,15 @@ def pick_bn(tokens_per_group: int, epi: int) -> int:
     return bn
 
 
+def pick_even_bn(tokens: int, F: int, G: int, sms: int = 0) -> int:
+    """Token tile of a grouped GEMM whose G groups have ``tokens`` rows each (the per-head maps of latent attention): the
+    smallest one whose tiles fit one wave of CTAs; below a wave short loops and epilogues count for more than weight re-reads."""
+    for bn in (32, 64, 128):
+        if (F + 127) // 128 * G * ((tokens + bn - 1) // bn) <= (sms or num_sms()):
+            return bn
+    return 256
+
+
 def want_streamk(epi: int, F: int, G: int, T: int, bn: int, sms: int) -> bool:
     """Work distribution of a grouped GEMM, from measurements on B200 (benchmark/ops/grouped_gemm.py): the stream-K
     tail pays off when the expected tile count fills the last wave of CTAs badly (few experts with long K loops, the
