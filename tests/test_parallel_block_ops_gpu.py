@@ -180,6 +180,38 @@ def test_attention_with_sinks(window, H, G, D, V, dtype):
         assert bool((out[-1] == 7.0).all())
 
 
+@BOTH
+@pytest.mark.parametrize("H,G,D,V", [(4, 2, 64, 32), (6, 2, 128, 64)])
+def test_one_far_key_takes_the_weight(H, G, D, V, dtype):
+    """Of 700 keys, one far back (first, at a page's first and last place) stands out for some late queries: single rows with
+    and without splits, and prompt portions."""
+    T, bs = 700, 16
+    q, k, v = rnd(T, H, D, seed=1, dtype=dtype), rnd(T, G, D, seed=2, dtype=dtype), rnd(T, G, V, seed=3, dtype=dtype)
+    pairs = [(699, 0), (650, 31), (500, 32), (497, 255), (300, 1)]
+    for i, j in pairs:
+        k[j] = (4 * q[i].view(G, -1, D)[:, 0].float()).to(dtype)
+    sink = rnd(H, seed=4)
+    want = attend(q, k, v, D ** -0.5, sink, None)
+    for i, j in pairs:
+        assert float((want[i, 0] - v[j, 0].double()).abs().max()) < 0.05      # what a missed key would change
+    blocks = pages(T, bs)
+    kc, vc = torch.zeros(len(blocks), bs, G, D, dtype=dtype), torch.zeros(len(blocks), bs, G, V, dtype=dtype)
+    t = torch.arange(T)
+    kc[blocks[t // bs].long(), t % bs], vc[blocks[t // bs].long(), t % bs] = k, v
+    kc, vc, bt = kc.to(DEV), vc.to(DEV), blocks[None].to(DEV)
+    opt = dict(fp32_weights=True, sink=sink.to(DEV))
+    late = torch.tensor([i for i, _ in pairs])
+    for splits in (1, 5):
+        got = F.paged_attention(q[late].reshape(len(late), -1).to(DEV), kc, vc, bt, torch.zeros(len(late), dtype=torch.int32, device=DEV),
+                                (late + 1).int().to(DEV), H, G, D, splits=splits, **opt)
+        heads_close(got.view(-1, H, V), want[late], tol(dtype, 1e-4))
+    if F.attention_on_tensor_cores(dtype, H, G, D, V):
+        tiles, _ = F.build_prefill_tiles([0] * 210, range(490, T), F.prefill_tile_tokens(H, G))
+        out = torch.zeros(210, H * V, dtype=dtype, device=DEV)
+        F.prefill_attention(q[490:].reshape(210, -1).to(DEV), kc, vc, bt, tiles.to(DEV), len(tiles), H, G, D, out, **opt)
+        heads_close(out.view(-1, H, V), want[490:], tol(dtype, 1e-4))
+
+
 LATENT = [(4, 32, 16, 48, 32), (6, 64, 32, 64, 64), (16, 128, 64, 128, 512), (35, 16, 8, 16, 264), (5, 9, 6, 11, 21), (2, 16, 2, 24, 130)]
 
 
