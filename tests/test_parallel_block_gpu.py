@@ -95,8 +95,8 @@ def test_mixed_batches_reuse_pages(name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_long_decoding_over_windows_and_pages(dtype):
-    raw = model(128, 200, [attn(4, 2, 64, 32, moe(4, 2, 48)), latent(4, 32, 16, 32, 48, 33, dense(96)),
-                           attn(4, 2, 64, 32, None), latent(4, 32, 16, 32, 48, 48, moe(4, 2, 48))])
+    raw = model(128, 200, [attn(4, 1, 64, 32, moe(4, 2, 48)), latent(4, 32, 16, 32, 48, 33, dense(96)),
+                           attn(4, 1, 64, 32, None), latent(4, 32, 16, 32, 48, 48, moe(4, 2, 48))])
     w = oracle.random_weights(raw, seed=8)
     toks = tokens(400, raw["vocab"], 2)
     want = oracle.run(raw, w, toks)[0]
