@@ -102,9 +102,11 @@ class RotarySpec:
 @dataclass(frozen=True)
 class AttentionSpec:
     """Softmax attention. ``window``: how many of the latest tokens, its own included, a query attends to (None: all).
+    ``chunk``: positions fall into chunks of that size, counted from 0, and a query attends to its own chunk only.
     ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none). ``qk_norm``: RMS norm
     of every query and key head. ``sink``: a learned number per head enters the softmax denominator. ``v_mix``: the values
-    are mixed with those that the first such layer computed for the same token."""
+    are mixed with those that the first such layer computed for the same token. ``tied_values``: the values are the keys before
+    their rotation (vdim = dim, no map of their own)."""
     heads: int
     kv_heads: int
     dim: int
@@ -117,12 +119,15 @@ class AttentionSpec:
     qk_norm: bool = True
     sink: bool = False
     v_mix: bool = False
+    chunk: Optional[int] = None
+    tied_values: bool = False
 
 
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Softmax attention whose keys and values are linear maps of one latent vector of ``kv_rank`` numbers per token; beside
-    it every token has one rotated key part of ``rot_dim`` numbers that all heads share. The cache holds those two."""
+    it every token has one rotated key part of ``rot_dim`` numbers that all heads share. The cache holds those two. ``gate``:
+    every head's output is scaled by the sigmoid of a linear map of the layer's input."""
     heads: int
     dim: int                                    # unrotated query / key size per head
     rot_dim: int
@@ -132,6 +137,7 @@ class LatentAttentionSpec:
     rot: Optional[RotarySpec] = None
     window: Optional[int] = None
     sink: bool = False
+    gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -158,22 +164,49 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class WkvSpec:
+    """RWKV-style time mixing: every projection reads a mix of its own of the row and the row before it; state of ``dim`` x
+    ``dim`` numbers per head with decays exp(-exp(.)) per key channel, read before the token's own write, which enters with a
+    bonus per channel. ``rank`` = inner size of the map to the decays."""
+    heads: int
+    dim: int
+    rank: int = 16
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+
+@dataclass(frozen=True)
 class RoutedSpec:
     """Feed-forward of ``experts`` gated feed-forwards of width ``ff``; a token uses the ``top`` ones with the largest
-    softmax scores, weighted by these scores (``renormalize``: divided by their sum)."""
+    scores, weighted by these scores (``renormalize``: divided by their sum) times ``scale``. ``scoring``: "softmax", or
+    "sigmoid" of every logit; ``correction``: a stored number per expert is added for the choice alone (sigmoid scores);
+    ``groups`` / ``keep``: experts form equal groups of neighbours and only those of the ``keep`` groups whose two best choice
+    scores have the largest sum can be chosen (sigmoid scores)."""
     experts: int
     top: int
     ff: int
     act: str = "silu"
     renormalize: bool = False
+    scoring: str = "softmax"
+    correction: bool = False
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, ChannelDeltaSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, ChannelDeltaSpec, WkvSpec]
     ff: Optional[int] = None                    # width of the dense gated feed-forward, None = the layer has none
     act: str = "silu"                           # of the dense feed-forward: silu or gelu_tanh
     routed: Optional[RoutedSpec] = None         # experts instead of a dense feed-forward
+    weights_of: Optional[int] = None            # the layer whose tensors this one uses, with a cache or state of its own
 
 
 @dataclass
@@ -184,31 +217,44 @@ class LayerListConfig(ModelConfig):
     ``block``: how a layer's sublayers sit on the residual stream x.
       "sandwich"  x += post(mixer(pre(x))), then x += post(ff(pre(x))); RMS norms whose stored weight is an offset from one
       "parallel"  h = norm(x); x += mixer(h) + ff(h); layer norms (mean taken off) with a plain weight
+      "prenorm"   x += m mixer(pre(x)), then x += m ff(pre(x)), m = ``residual_mult``; RMS norms as in "sandwich"
     """
     layers: List[LayerSpec] = field(default_factory=list)
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     architecture: str = ""
     block: str = "sandwich"
+    residual_mult: float = 1.0
 
     def is_dense_layer(self, layer_id: int) -> bool:
         return True
 
     def __post_init__(self):
         super().__post_init__()
-        assert self.num_layers == len(self.layers) and self.block in ("sandwich", "parallel")
+        assert self.num_layers == len(self.layers) and self.block in ("sandwich", "parallel", "prenorm")
         for i, layer in enumerate(self.layers):
             m, r = layer.mixer, layer.routed
             if layer.act not in ACTIVATIONS or (r is not None and r.act not in ACTIVATIONS):
                 raise ValueError(f"layer {i}: unknown activation (known: {', '.join(ACTIVATIONS)})")
             if r is not None and (layer.ff or self.block == "sandwich" or not 1 <= r.top <= r.experts):
-                raise ValueError(f"layer {i}: experts need a parallel block, no dense feed-forward beside them and 1 <= top "
-                                 f"<= experts")
+                raise ValueError(f"layer {i}: experts need a parallel or pre-norm block, no dense feed-forward beside them and "
+                                 f"1 <= top <= experts")
+            if r is not None and r.scoring not in ("softmax", "sigmoid"):
+                raise ValueError(f"layer {i}: unknown expert scores {r.scoring!r}")
+            if r is not None and (r.experts % r.groups or not 1 <= r.keep <= r.groups or r.top > r.experts // r.groups * r.keep):
+                raise ValueError(f"layer {i}: {r.top} experts of {r.keep} out of {r.groups} groups of {r.experts}")
+            if r is not None and r.scoring != "sigmoid" and (r.correction or r.groups > 1):
+                raise ValueError(f"layer {i}: corrections and groups of experts need sigmoid scores")
+            if layer.weights_of is not None and replace(layer, weights_of=None) != \
+                    replace(self.layers[self.weight_layer(i)], weights_of=None):
+                raise ValueError(f"layer {i} cannot use the weights of layer {layer.weights_of}")
             rot = getattr(m, "rot", None)
             if rot is not None and (rot.dims % 2 or rot.dims > (m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim)):
                 raise ValueError(f"layer {i}: {rot.dims} rotated dimensions do not fit the head")
-            if isinstance(m, (GatedLinearSpec, LatentAttentionSpec)):
+            if isinstance(m, (GatedLinearSpec, LatentAttentionSpec, WkvSpec)):
                 continue
+            if getattr(m, "tied_values", False) and (m.vdim != m.dim or m.v_mix or m.kv_from is not None or m.qk_norm):
+                raise ValueError(f"layer {i}: values tied to the keys have their size and no norm, mixing or sharing")
             if m.heads % m.kv_heads:
                 raise ValueError(f"layer {i}: {m.heads} heads do not share {m.kv_heads} key / value heads evenly")
             src = getattr(m, "kv_from", None)
@@ -222,6 +268,16 @@ class LayerListConfig(ModelConfig):
                 f = self.layers[first].mixer
                 if m.kv_from is not None or (f.kv_heads, f.vdim) != (m.kv_heads, m.vdim):
                     raise ValueError(f"layer {i} cannot mix its values with those of layer {first}")
+
+    def weight_layer(self, i: int) -> int:
+        """The layer whose tensors layer i uses."""
+        seen = {i}
+        while self.layers[i].weights_of is not None:
+            i = self.layers[i].weights_of
+            if not 0 <= i < len(self.layers) or i in seen:
+                raise ValueError(f"weights_of names no layer with weights: {i}")
+            seen.add(i)
+        return i
 
     @property
     def first_v_mix(self) -> Optional[int]:

@@ -51,17 +51,24 @@ __device__ __forceinline__ void cp_async16_stream(uint32_t dst, const void* src,
 }
 // Options of the EXT instantiations of both kernels (plain ones compile without them):
 //   window > 0: a query at position p sees only keys in (p - window, p];
+//   chunk > 0: it sees only keys of its own chunk of `chunk` positions, counted from position 0;
 //   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap);
 //   sink != NULL: exp(sink[head]) enters the softmax denominator (no key, no value);
 //   gq: query heads per kv head where the instantiation leaves it open (GQ = 0).
 // The EXT kernels also keep the softmax weights at fp32 accuracy in the P V product: P = hi + lo, both bf16, two MMAs.
 struct AttnExt {
-  int window;
+  int window, chunk;
   float cap_in, cap_log2;
   const float* sink;
   int gq;
 };
 constexpr float kLog2e = 1.4426950408889634f;
+// first key that a query at position p sees
+__device__ __forceinline__ int first_key(int p, int window, int chunk) {
+  int lo = window > 0 ? max(0, p - window + 1) : 0;
+  if (chunk > 0) lo = max(lo, p / chunk * chunk);
+  return lo;
+}
 // 16-byte chunk c of tile row r in shared memory: rows of 128 bytes and more permute their chunks by groups of eight, rows of
 // 64 bytes (two to a 128-byte line) by groups of four; either way eight rows of one column meet no bank twice.
 template <int NCH>
@@ -119,7 +126,7 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
   const int row = bt_row != nullptr ? bt_row[t] : t;
   const int* bt = block_tables + static_cast<long long>(row) * max_blocks;
   // first visible token, and its block: the blocks from there on are dealt out to the splits
-  const int vis0 = EXT && ext.window > 0 ? max(0, len - ext.window) : 0;
+  const int vis0 = EXT && len > 0 ? first_key(len - 1, ext.window, ext.chunk) : 0;
   const int blk0 = vis0 / block_size;
   const int nblk = (len + block_size - 1) / block_size - blk0;
   const int blk_per = (nblk + splits - 1) / splits;
@@ -346,7 +353,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   const int* bt = block_tables + static_cast<long long>(tile.z) * max_blocks;
   const int kmax = pos0 + ntok;                     // keys [0, kmax) exist for the last token of the tile
   const int nkb = (kmax + kPreKeys - 1) / kPreKeys;
-  const int kb0 = EXT && ext.window > 0 ? max(0, pos0 - ext.window + 1) / kPreKeys : 0;   // first block anyone sees
+  const int kb0 = EXT ? first_key(pos0, ext.window, ext.chunk) / kPreKeys : 0;   // first block anyone sees
   const uint32_t sbase = smem_u32(s_pre);
 
   auto issue = [&](int kb) {
@@ -411,10 +418,10 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   const int lm_mi = lane >> 3, lm_r = lane & 7;
   // the warp's last query position: key blocks entirely behind it are skipped by this warp (causal)
   const int wlast = pos0 + min(ntok - 1, (warp * 16 + 15) / gq);
-  // and, with a window, those entirely before the reach of its first query; a row's first visible key
-  const int wfirst = EXT && ext.window > 0 ? pos0 + warp * 16 / gq - ext.window + 1 : 0;
-  const int lo0 = EXT && ext.window > 0 ? qpos0 - ext.window + 1 : 0;
-  const int lo1 = EXT && ext.window > 0 ? qpos1 - ext.window + 1 : 0;
+  // and, with a window or chunks, those entirely before the reach of its first query; a row's first visible key
+  const int wfirst = EXT ? first_key(pos0 + warp * 16 / gq, ext.window, ext.chunk) : 0;
+  const int lo0 = EXT ? first_key(qpos0, ext.window, ext.chunk) : 0;
+  const int lo1 = EXT ? first_key(qpos1, ext.window, ext.chunk) : 0;
 
   for (int kb = kb0; kb < nkb; ++kb) {
     issue(kb + 1);
@@ -529,12 +536,13 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   }
 }
 
-// Options of a launch as the kernels take them (softcap <= 0: none; window <= 0: every key).
-static AttnExt make_ext(float scale, int window, float softcap, const float* sink, int gq) {
+// Options of a launch as the kernels take them (softcap <= 0: none; window, chunk <= 0: every key).
+static AttnExt make_ext(float scale, int window, int chunk, float softcap, const float* sink, int gq) {
   AttnExt x;
   x.sink = sink;
   x.gq = gq;
   x.window = window > 0 ? window : 0;
+  x.chunk = chunk > 0 ? chunk : 0;
   x.cap_in = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
   x.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   return x;
@@ -643,20 +651,20 @@ extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* k
                                     int block_size, int T, int n_q, int n_kv, int hd, float scale, int splits, void* out,
                                     long long ld_out, float* workspace, void* stream_) {
   return attn_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                              hd, hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0.f, nullptr, 0),
+                              hd, hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0, 0.f, nullptr, 0),
                               static_cast<cudaStream_t>(stream_));
 }
 
-// The same with a sliding window, a score soft cap (0 = without) and a sink per head (NULL = without), value heads of another
+// The same with a sliding window, chunks of positions that see no other chunk (0 = without), a score soft cap (0 = without) and a sink per head (NULL = without), value heads of another
 // size than key heads, and query groups of up to 64 heads.
 extern "C" int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                         const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
                                         int block_size, int T, int n_q, int n_kv, int hd, int vd, float scale, int window,
-                                        float softcap, const float* sink, int splits, void* out, long long ld_out,
+                                        int chunk, float softcap, const float* sink, int splits, void* out, long long ld_out,
                                         float* workspace, void* stream_) {
   if (n_kv < 1) return -10;
   return attn_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                             hd, vd, scale, splits, out, ld_out, workspace, make_ext(scale, window, softcap, sink, n_q / n_kv),
+                             hd, vd, scale, splits, out, ld_out, workspace, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv),
                              static_cast<cudaStream_t>(stream_));
 }
 
@@ -706,17 +714,17 @@ extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void*
                                       int block_size, int n_q, int n_kv, int hd, float scale, void* out, long long ld_out,
                                       void* stream_) {
   return prefill_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                 hd, hd, scale, out, ld_out, make_ext(scale, 0, 0.f, nullptr, 0),
+                                 hd, hd, scale, out, ld_out, make_ext(scale, 0, 0, 0.f, nullptr, 0),
                                  static_cast<cudaStream_t>(stream_));
 }
 
 extern "C" int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                           const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
                                           int block_size, int n_q, int n_kv, int hd, int vd, float scale, int window,
-                                          float softcap, const float* sink, void* out, long long ld_out, void* stream_) {
+                                          int chunk, float softcap, const float* sink, void* out, long long ld_out, void* stream_) {
   if (n_kv < 1) return -10;
   return prefill_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                hd, vd, scale, out, ld_out, make_ext(scale, window, softcap, sink, n_q / n_kv),
+                                hd, vd, scale, out, ld_out, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv),
                                 static_cast<cudaStream_t>(stream_));
 }
 
@@ -733,7 +741,7 @@ __global__ void __launch_bounds__(kAnyKeys)
 any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, const T* __restrict__ kcache, long long k_tok,
                 const T* __restrict__ vcache, long long v_tok, const int* __restrict__ block_tables, int max_blocks,
                 const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len, int block_size,
-                int n_q, int n_kv, int dk, int dv, float scale, int window, float softcap, const float* __restrict__ sink,
+                int n_q, int n_kv, int dk, int dv, float scale, int window, int chunk, float softcap, const float* __restrict__ sink,
                 T* __restrict__ out, long long o_head, long long o_row) {
   extern __shared__ float s_any[];          // q [dk] | acc [dv]
   __shared__ float s_p[kAnyKeys];
@@ -751,7 +759,7 @@ any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, cons
   for (int d = tid; d < dv; d += kAnyKeys) s_acc[d] = 0.f;
   __syncthreads();
   float m = -INFINITY, l = 0.f;
-  for (int j0 = window > 0 ? max(0, len - window) : 0; j0 < len; j0 += kAnyKeys) {
+  for (int j0 = len > 0 ? first_key(len - 1, window, chunk) : 0; j0 < len; j0 += kAnyKeys) {
     const int n = min(kAnyKeys, len - j0);
     float s = -INFINITY;
     if (tid < n) {
@@ -803,7 +811,7 @@ any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, cons
 extern "C" int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_row, const void* kcache,
                                   long long k_tok, const void* vcache, long long v_tok, const int* block_tables, int max_blocks,
                                   const int* bt_row, const int* rows, const int* ctx_len, int block_size, int T, int n_q,
-                                  int n_kv, int dk, int dv, float scale, int window, float softcap, const float* sink, void* out,
+                                  int n_kv, int dk, int dv, float scale, int window, int chunk, float softcap, const float* sink, void* out,
                                   long long o_head, long long o_row, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (T == 0) return 0;
@@ -813,12 +821,12 @@ extern "C" int dmoe_any_attention(int is_f32, const void* q, long long q_head, l
   if (is_f32)
     any_attn_kernel<float><<<grid, kAnyKeys, smem, stream>>>(
         static_cast<const float*>(q), q_head, q_row, static_cast<const float*>(kcache), k_tok, static_cast<const float*>(vcache),
-        v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, softcap, sink,
+        v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, chunk, softcap, sink,
         static_cast<float*>(out), o_head, o_row);
   else
     any_attn_kernel<__nv_bfloat16><<<grid, kAnyKeys, smem, stream>>>(
         static_cast<const __nv_bfloat16*>(q), q_head, q_row, static_cast<const __nv_bfloat16*>(kcache), k_tok,
         static_cast<const __nv_bfloat16*>(vcache), v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv,
-        dk, dv, scale, window, softcap, sink, static_cast<__nv_bfloat16*>(out), o_head, o_row);
+        dk, dv, scale, window, chunk, softcap, sink, static_cast<__nv_bfloat16*>(out), o_head, o_row);
   return static_cast<int>(cudaGetLastError());
 }

@@ -6,6 +6,30 @@
 
 #ifdef __cplusplus
 extern "C" {
+
+// Router of dmoe_sum_norm (weight [E, W] in the activations' dtype): softmax scores or, sigmoid = 1, sigmoid scores with a
+// correction (NULL: none) that counts for the choice alone, inside the best `keep` of `groups` equal groups of neighbours.
+typedef struct DmoeRouter {
+  const void* weight;
+  const float* correction;  // [E]
+  int* ids;                 // [rows, K]
+  float* wts;               // [rows, K]: scores, with renorm divided by their sum, times wscale
+  int* counts;              // [E], may be NULL
+  int E, K, renorm, sigmoid, groups, keep;
+  float wscale;
+} DmoeRouter;
+// Token shift: n_mix outputs h + (before - h) mu per row, `before` = the row before in the sequence, kept per slot in `last`.
+// singles: int4 {row, 1, slot, position}; NULL: one-token segment i is row i, as in DmoeRecur.
+typedef struct DmoeShift {
+  const float* mu;          // [n_mix, W]
+  float* last;              // [n_slots, W]
+  const void* singles;
+  const int* positions;
+  const int* rows;
+  const long long* kv_slots;
+  long long mix_stride;     // elements from one output to the next
+  int n_mix, n_slots, n_single;
+} DmoeShift;
 #endif
 
 // ---- GEMM (gemm.cu) -------------------------------------------------------------------------------
@@ -73,7 +97,7 @@ typedef struct DmoeGemm {
   // != 0: W is stored tile by tile, [group][128-row tile][K / 64][128][64] (see ops/gemm.py: block_weight), so that
   // every 16 KB box the kernel fetches is one contiguous run of HBM; needs F % 128 == 0 and K % 64 == 0
   int w_blocked;
-  // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form)
+  // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form); plain epilogue: 2 = tanh of the output
   int act;
   // profiling aid, normally null: 16 x uint64 of device memory that CTA 0 fills with %globaltimer stamps (entry, set-up
   // done, first TMA issued, first stage landed, last MMA committed, accumulator seen by the epilogue, epilogue done,
@@ -115,11 +139,11 @@ int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, cons
 // of size vd. (hd, vd) = (64, 32), (64, 64), (128, 64), (128, 128), up to 64 query heads per kv head.
 int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
                              int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
-                             int hd, int vd, float scale, int window, float softcap, const float* sink, int splits, void* out,
+                             int hd, int vd, float scale, int window, int chunk, float softcap, const float* sink, int splits, void* out,
                              long long ld_out, float* workspace, void* stream);
 int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                const int* block_tables, int max_blocks, const void* tiles, int n_tiles, int block_size,
-                               int n_q, int n_kv, int hd, int vd, float scale, int window, float softcap, const float* sink,
+                               int n_q, int n_kv, int hd, int vd, float scale, int window, int chunk, float softcap, const float* sink,
                                void* out, long long ld_out, void* stream);
 // Any key / value size and query group, bf16 or fp32 cache, fp32 arithmetic on the CUDA cores. Query i of head h starts at
 // q + i * q_row + h * q_head (output likewise) and has the context of batch row rows[i] (NULL: i); the heads of a cached token
@@ -127,7 +151,7 @@ int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache
 int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_row, const void* kcache, long long k_tok,
                        const void* vcache, long long v_tok, const int* block_tables, int max_blocks, const int* bt_row,
                        const int* rows, const int* ctx_len, int block_size, int T, int n_q, int n_kv, int dk, int dv,
-                       float scale, int window, float softcap, const float* sink, void* out, long long o_head, long long o_row,
+                       float scale, int window, int chunk, float softcap, const float* sink, void* out, long long o_head, long long o_row,
                        void* stream);
 
 // ---- latent attention (latent_attention.cu): the cache has one row [latent rankp | rotated key part rotp] per token,
@@ -135,9 +159,10 @@ int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_
 // Projection rows y = [heads x (q dimp | rotp) | latent rankp | key part rotp] (every part padded to a multiple of 8): RMS norm
 // of the latent, rotation of the key part, both to cache rows at slots (< 0: skip); rotation of the queries in place, and for
 // rows with loose[t] = i >= 0 (NULL: i = t) to xq [heads, n_loose, dimp] and columns rankp.. of qa [heads, n_loose, row].
+// gate (NULL: none; row stride ld): sigmoid(gate[t, h]) becomes the weight of record h * n_loose + i of recs (see DmoeGemm).
 int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
                      int heads, int dim, int rot_dim, int rank, int row, int rot, int interleaved, const void* table, int max_pos,
-                     const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa, void* stream);
+                     const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa, const void* gate, void* recs, void* stream);
 // Queries qa [heads, n, row] over cache rows (keys: the first kd columns, values: the first rankp), out [heads, n, rankp];
 // rankp <= 512, kd <= 640, row an odd multiple of 8, block_size a multiple of 16. workspace: heads * n * splits * (rankp + 1) floats where splits > 1. status (may be NULL): non-zero
 // after a bounded wait gave up.
@@ -148,10 +173,11 @@ int dmoe_latent_attention(const void* qa, const void* cache, const int* block_ta
 int dmoe_latent_gather(const void* cache, const int* block_tables, int max_blocks, const void* keys, int n, int block_size,
                        int row, void* out, void* stream);
 // Prompt tiles over expanded keys and values: tile i's key at position p is row base[i] + p of kv [heads x (dimp | vdimp)] and
-// of lat (columns rankp ..: its rotated part).
+// of lat (columns rankp ..: its rotated part). gate (NULL: none): head h's output is scaled by sigmoid(gate[row, h]).
 int dmoe_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
                         const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp, int vdimp,
-                        float scale, int window, const float* sink, void* out, long long ld_out, void* stream);
+                        float scale, int window, const float* sink, const void* gate, long long ld_gate, void* out, long long ld_out,
+                        void* stream);
 
 // Tiled causal attention for prompt tokens: CTA column i handles tiles[i] = int4 {first row in q / out, tokens
 // (<= dmoe_prefill_tile_tokens), block-table row, position of the first token}; the tokens of a tile are consecutive
@@ -172,23 +198,28 @@ int dmoe_resid_norm(int is_f32, float* resid, const void* y, long long ld_y, con
 int dmoe_rope_freq_table(void* table, int max_pos, int half, const double* freq, float mscale, void* stream);
 // Per-head RMS norm of q and k (qw, kw; NULL: none), rotation of pairs (i, i + rot / 2), i < rot / 2, or (2i, 2i + 1) where
 // interleaved; q in place, k / v into the paged caches, v as (1 - v_lambda) v + v_lambda v_first where that is given
-// (row stride ld_first, head stride first_head).
+// (row stride ld_first, head stride first_head). tied: rows [q | k], the values are the first dv dimensions of the k heads before
+// their rotation.
 int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots, void* kcache,
                       void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved, const void* table,
                       int max_pos, const float* qw, const float* kw, float eps, const void* v_first, long long ld_first,
-                      int first_head, float v_lambda, void* stream);
-// x = resid[r] + y[r] + sum of n_parts rows of parts (both may be NULL); resid[r] = x unless a row table picks r = rows[i];
-// h[i] = norm(x) * w, RMS norm or with `centred` layer norm. With gate_w [E, W] also softmax router over h: the K largest
-// scores (renorm: divided by their sum) and, where counts is given, the histogram of the chosen experts. E <= 256, K <= 32.
+                      int first_head, float v_lambda, int tied, void* stream);
+// x = resid[r] + mult (y[r] + sum of n_parts rows of parts) (both may be NULL); resid[r] = x unless a row table picks
+// r = rows[i]; h[i] = norm(x) * w, RMS norm or with `centred` layer norm, as fp32 where h_f32. router: the K best experts of
+// every h and, where counts is given, the histogram of the chosen ones; E <= 256, K <= 32. shift (all rows one-token segments):
+// h gets the n_mix mixed rows instead.
 int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
-                  long long part_row, long long part_stride, const float* w, int centred, float eps, const int* rows, void* h,
-                  long long ld_h, int n, int W, const void* gate_w, int E, int K, int renorm, int* ids, float* wts, int* counts,
-                  void* stream);
+                  long long part_row, long long part_stride, float mult, const float* w, int centred, float eps, const int* rows,
+                  void* h, int h_f32, long long ld_h, int n, int W, const DmoeRouter* router, const DmoeShift* shift, void* stream);
+// The token shift of a batch with longer segments (tables as in DmoeRecur: segs of the longer ones, their chunks): fp32 rows h ->
+// n_mix outputs; the slots keep the last row of every segment.
+int dmoe_token_shift(int is_f32, const float* h, const DmoeShift* s, const void* multi, int n_multi, const void* chunks, int n_chunks,
+                     void* out, long long ld, int W, void* stream);
 // out[t, i] = act(gu[t, i]) * gu[t, I + i]; act 0: silu, 1: gelu (tanh form)
 int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I, void* stream);
 // Y = X W^T on the CUDA cores in fp32 arithmetic: fp32 operands, or bf16 operands of any alignment.
 int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y, long long ldy,
-                     int T, int F, int K, void* stream);
+                     int T, int F, int K, int act, void* stream);      // act 2: tanh of the output
 // The same over row groups: rows offs[g] .. offs[g + 1] of X with W[g] [F, K]; recs / bases (may be NULL): row t goes, scaled,
 // where recs[t] says (see DmoeGemm), in X's type.
 int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y, long long ldy,
@@ -211,23 +242,26 @@ typedef struct DmoeRecur {
   const int* rows;
   const long long* kv_slots;
   float* state;             // [n_slots, heads, dim, vdim]
-  const float* norm_w;      // [vdim]
+  const float* norm_w;      // [vdim], or [heads, vdim] with norm_ld = vdim (0: one for all heads)
   void* out;                // [rows, heads * vdim]
   float* raw;               // read-outs before norm and gate
   long long ldq, ldk, ldv, ldg, ldb, ldz, ldo, ldraw;
   int n_segs, n_slots, heads, kv_heads, dim, vdim, taps;
   int delta;                // 0: plain write, 1: delta rule (q and k are made unit vectors)
-  int decay_kind;           // 0: log a = log sigmoid(z + b) * inv_tau, 1: log a = -exp(a_log) softplus(z + b)
+  int decay_kind;           // 0: log a = log sigmoid(z + b) * inv_tau, 1: log a = -exp(a_log) softplus(z + b), 2: log a = -exp(z + b)
   int gate_kind;            // 0: silu, 1: sigmoid
   int is_f32;
   int one_token;            // dmoe_recur_step: every segment has one token
   float qscale, inv_tau, eps;
   int* status;              // optional device status word: non-zero after a bounded wait gave up
+  const float* bonus;       // plain write only: [heads, dim]; the read-out precedes decay and write, and the token's own write
+                            // enters it weighed by the bonus of the key channel
+  int norm_ld;
 } DmoeRecur;
 int dmoe_recur_value_tile(int dim, int vdim);
 int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream);
 int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw, const void* gate,
-                   long long ldg, const float* norm_w, float eps, int gate_kind, void* out, long long ldo, int heads, int V,
+                   long long ldg, const float* norm_w, int norm_ld, float eps, int gate_kind, void* out, long long ldo, int heads, int V,
                    void* stream);
 // The same recurrence chunk by chunk on the tensor cores (recurrent_chunk.cu), bf16 activations, for segments of any length.
 int dmoe_recur_chunk_ok(int dim, int vdim);

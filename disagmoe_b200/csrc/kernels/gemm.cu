@@ -96,7 +96,7 @@ struct GemmArgs {
   // w_blocked: the weights are stored tile by tile ([group][128-row tile][K block][128][64], every 16 KB TMA box one
   // contiguous run of HBM) instead of row-major [group][row][K]
   int w_blocked;
-  int act;      // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form)
+  int act;      // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form); plain epilogue: 2 = tanh of the output
   // optional [16] nanosecond stamps written by CTA 0 (a profiling aid, null in normal launches): 0 entry, 1 set-up done,
   // 2 first TMA issued, 3 first stage landed, 4 last MMA committed, 5 accumulator seen by the epilogue, 6 epilogue done,
   // 7 tear-down reached; 8-12 inside the first epilogue chunk: TMEM read done, staged to shared memory, barrier passed,
@@ -145,6 +145,9 @@ __device__ __forceinline__ float gate_act(float g, int act) {
   const float z = act == 0 ? g : 1.5957691216057308f * (g + 0.044715f * g * g * g);
   return g / (1.f + __expf(-z));
 }
+
+// tanh(x) = 1 - 2 / (exp(2x) + 1), good to about 1e-7 absolute
+__device__ __forceinline__ float out_tanh(float x) { return 1.f - __fdividef(2.f, __expf(fminf(2.f * x, 40.f)) + 1.f); }
 
 __device__ __forceinline__ int ld_acquire_sys(const int* p) {
   int v;
@@ -539,6 +542,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
             if (PAIR) mbar_arrive_cluster(mapa_rank(smem_u32(&tempty_bar[buf]), 0));
             else mbar_arrive(smem_u32(&tempty_bar[buf]));
           }
+        }
+        if (EPI == EPI_PLAIN && a.act == 2) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) acc[j] = out_tanh(acc[j]);
         }
         if ((EPI == EPI_PLAIN || EPI == EPI_SWIGLU) && vec) {
           if (jmax <= 0) continue;                   // uniform over the CTA: no barrier is skipped by some threads only

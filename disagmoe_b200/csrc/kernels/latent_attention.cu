@@ -17,13 +17,15 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr int pad8(int n) { return (n + 7) / 8 * 8; }
 
 // One CTA per row. A row of y is [heads x (dimp | rotp) | rankp | rotp], parts padded with zeros to multiples of 8.
-// VEC: the rotation is interleaved, covers all of rotp and moves in 16-byte units.
+// VEC: the rotation is interleaved, covers all of rotp and moves in 16-byte units. gate (NULL: none): a row has one gate per head;
+// the sigmoid of a loose row's gates becomes the weight of its heads' records.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
                    T* __restrict__ cache, int heads, int dimp, int rotp, int rank, int rankp, int row, int rot,
                    int interleaved, const float2* __restrict__ table, int max_pos, const float* __restrict__ norm_w, float eps,
-                   const int* __restrict__ loose, int n_loose, T* __restrict__ xq, T* __restrict__ qa) {
+                   const int* __restrict__ loose, int n_loose, T* __restrict__ xq, T* __restrict__ qa,
+                   const T* __restrict__ gate, int4* __restrict__ recs) {
   __shared__ float red[8];
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -34,6 +36,10 @@ latent_prep_kernel(T* __restrict__ y, long long ld, const int* __restrict__ posi
   const float2* tab = table + static_cast<long long>(pos) * half;
   T* yr = y + t * ld;
   const T* c = yr + static_cast<long long>(heads) * qd;
+
+  if (gate != nullptr && li >= 0)
+    for (int h = threadIdx.x; h < heads; h += blockDim.x)
+      recs[static_cast<long long>(h) * n_loose + li].z = __float_as_int(1.f / (1.f + expf(-static_cast<float>(gate[t * ld + h]))));
 
   // rotated part of a head (or of the key): pairs turn, what is not rotated passes
   auto turn = [&](const T* p, T* dst, int first, int step) {
@@ -416,7 +422,7 @@ __global__ void __launch_bounds__(128)
 latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __restrict__ kv, long long ld_kv,
                       const bf16* __restrict__ lat, long long ld_lat, const int4* __restrict__ tiles, const int* __restrict__ base,
                       int dimp, int rotp, int rankp, int vdimp, float scale_log2, int window, const float* __restrict__ sink,
-                      bf16* __restrict__ out, long long ld_out) {
+                      const bf16* __restrict__ gate, long long ld_gate, bf16* __restrict__ out, long long ld_out) {
   constexpr int KP = KD * 2 + 16, VP = VD * 2 + 16;       // row pitches: odd numbers of 16-byte units
   constexpr int STAGE = kLpKeys * (KP + VP);
   constexpr int KS = KD / 16, NT = VD / 8;
@@ -567,6 +573,10 @@ latent_prefill_kernel(const bf16* __restrict__ q, long long ld_q, const bf16* __
     inv0 = f0 / (l0 * f0 + exp2f(sk - M0));
     inv1 = f1 / (l1 * f1 + exp2f(sk - M1));
   }
+  if (gate != nullptr) {
+    if (v0) inv0 *= 1.f / (1.f + expf(-__bfloat162float(gate[(row0 + t0) * ld_gate + head])));
+    if (v1) inv1 *= 1.f / (1.f + expf(-__bfloat162float(gate[(row0 + t1) * ld_gate + head])));
+  }
   bf16* o0 = out + static_cast<long long>(row0 + t0) * ld_out + head * vdimp;
   bf16* o1 = out + static_cast<long long>(row0 + t1) * ld_out + head * vdimp;
 #pragma unroll
@@ -605,8 +615,8 @@ static int launch_latent(const void* q, const void* cache, const int* bt, int ma
 template <int KD, int VD>
 static int launch_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
                                  const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp,
-                                 int vdimp, float scale, int window, const float* sink, void* out, long long ld_out,
-                                 cudaStream_t stream) {
+                                 int vdimp, float scale, int window, const float* sink, const void* gate, long long ld_gate,
+                                 void* out, long long ld_out, cudaStream_t stream) {
   constexpr int smem = 2 * kLpKeys * (KD * 2 + VD * 2 + 32);
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
@@ -615,7 +625,8 @@ static int launch_latent_prefill(const void* q, long long ld_q, const void* kv, 
   if (rc != 0) return rc;
   latent_prefill_kernel<KD, VD><<<dim3(n_tiles, heads), 128, smem, stream>>>(
       static_cast<const bf16*>(q), ld_q, static_cast<const bf16*>(kv), ld_kv, static_cast<const bf16*>(lat), ld_lat,
-      static_cast<const int4*>(tiles), base, dimp, rotp, rankp, vdimp, scale * kLog2e, window, sink, static_cast<bf16*>(out), ld_out);
+      static_cast<const int4*>(tiles), base, dimp, rotp, rankp, vdimp, scale * kLog2e, window, sink,
+      static_cast<const bf16*>(gate), ld_gate, static_cast<bf16*>(out), ld_out);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -626,12 +637,13 @@ using namespace dmoe;
 extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* positions, const long long* slots, void* cache, int T,
                                 int heads, int dim, int rot_dim, int rank, int row, int rot, int interleaved, const void* table,
                                 int max_pos, const float* norm_w, float eps, const int* loose, int n_loose, void* xq, void* qa,
-                                void* stream_) {
+                                const void* gate, void* recs, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (heads < 1 || dim < 1 || rot_dim < 0 || rank < 1 || rot < 0 || rot % 2 != 0 || rot > rot_dim || (rot > 0 && table == nullptr)) return -10;
   const int align = is_f32 ? 4 : 8;
   if (row % align != 0 || row < pad8(rank) + pad8(rot_dim)) return -10;
   if (ld % align != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 || (loose == nullptr && n_loose < T)) return -10;
+  if (gate != nullptr && n_loose > 0 && recs == nullptr) return -10;
   if (T == 0) return 0;
   const int dimp = pad8(dim), rotp = pad8(rot_dim), rankp = pad8(rank);
   const bool vec = interleaved && rot == rotp && rot > 0;
@@ -639,7 +651,7 @@ extern "C" int dmoe_latent_prep(int is_f32, void* y, long long ld, const int* po
   latent_prep_kernel<T_, VEC_><<<T, 256, 0, stream>>>(                                                                       \
       static_cast<T_*>(y), ld, positions, slots, static_cast<T_*>(cache), heads, dimp, rotp, rank, rankp, row, rot,          \
       interleaved, static_cast<const float2*>(table), max_pos, norm_w, eps, loose, n_loose, static_cast<T_*>(xq),            \
-      static_cast<T_*>(qa))
+      static_cast<T_*>(qa), static_cast<const T_*>(gate), static_cast<int4*>(recs))
   if (is_f32 && vec) DMOE_PREP(float, true);
   else if (is_f32) DMOE_PREP(float, false);
   else if (vec) DMOE_PREP(bf16, true);
@@ -679,8 +691,8 @@ extern "C" int dmoe_latent_gather(const void* cache, const int* block_tables, in
 
 extern "C" int dmoe_latent_prefill(const void* q, long long ld_q, const void* kv, long long ld_kv, const void* lat, long long ld_lat,
                                    const void* tiles, const int* base, int n_tiles, int heads, int dimp, int rotp, int rankp,
-                                   int vdimp, float scale, int window, const float* sink, void* out, long long ld_out,
-                                   void* stream_) {
+                                   int vdimp, float scale, int window, const float* sink, const void* gate, long long ld_gate,
+                                   void* out, long long ld_out, void* stream_) {
   if (n_tiles == 0) return 0;
   if (n_tiles < 0 || heads < 1 || heads > 65535 || dimp % 8 != 0 || rotp % 8 != 0 || rankp % 8 != 0 || vdimp % 8 != 0) return -10;
   if (ld_q % 8 != 0 || ld_kv % 8 != 0 || ld_lat % 8 != 0 || ld_out % 8 != 0 || tiles == nullptr || base == nullptr) return -10;
@@ -689,7 +701,7 @@ extern "C" int dmoe_latent_prefill(const void* q, long long ld_q, const void* kv
 #define DMOE_LP(KD_, VD_)                                                                                               \
   if (kd <= KD_ && vdimp <= VD_)                                                                                        \
     return launch_latent_prefill<KD_, VD_>(q, ld_q, kv, ld_kv, lat, ld_lat, tiles, base, n_tiles, heads, dimp, rotp, rankp, \
-                                           vdimp, scale, window, sink, out, ld_out, stream)
+                                           vdimp, scale, window, sink, gate, ld_gate, out, ld_out, stream)
   DMOE_LP(96, 64);
   DMOE_LP(128, 128);
   DMOE_LP(192, 128);

@@ -1,6 +1,6 @@
 // Row kernels of decoders whose residual stream is kept in fp32, for bf16 and fp32 activations: scaled embedding,
-// post-norm + residual add + pre-norm in one pass, residual sum + norm + softmax router in one pass, per-head query / key
-// norm + partial rotary embedding + value mixing + paged KV append, rotary table from arbitrary frequencies, act(gate) * up,
+// post-norm + residual add + pre-norm in one pass, residual sum + norm + router (or token shift) in one pass, token shift of
+// whole segments, per-head query / key norm + partial rotary embedding + value mixing + paged KV append, rotary table from arbitrary frequencies, act(gate) * up,
 // and a CUDA-core GEMM, dense or over row groups, for fp32 operands (and for bf16 shapes the tcgen05 kernel's TMA cannot
 // address).
 #include "dmoe_kernels.h"
@@ -147,8 +147,12 @@ resid_norm_kernel(float* __restrict__ resid, const T* __restrict__ y, long long 
 }
 
 // Residual sum, norm and (optionally) router of blocks whose sublayers share a norm, TPC rows per CTA of 256 threads:
-//   x = resid[r] + y[r] + sum_p parts[r, p];  resid[r] = x (unless a row table picks the rows);  h = norm(x) * w
-//   router: logits = gate_w h, softmax, the K largest (lowest index first among equals).
+//   x = resid[r] + mult (y[r] + sum_p parts[r, p]);  resid[r] = x (unless a row table picks the rows);  h = norm(x) * w
+//   router: logits z = gate_w h; scores softmax(z), or sigmoid(z); the K largest (lowest index first among equals). Sigmoid
+//   scores are chosen by score + correction, among the `keep` of `groups` equal runs of neighbouring experts whose two best
+//   choice scores have the largest sum. Weights: scores, divided by their sum with renorm, times wscale.
+//   shift: instead of h, S rows h + (before - h) mu_s per row, `before` = the slot's last row (0 at position 0), which h replaces.
+// h_f32: h is stored as fp32.
 // The rows stay in shared memory (fp32) from the sum on; with several rows per CTA the router's weights are fetched once for
 // all of them.
 struct SumNormArgs {
@@ -170,7 +174,18 @@ struct SumNormArgs {
   int* ids;
   float* wts;
   int* counts;
+  float mult;
+  int h_f32;
+  int sigmoid, groups, keep;
+  const float* correction;
+  float wscale;
+  DmoeShift shift;            // n_mix = 0: none
 };
+// Segment of row i of a batch of one-token segments: {row, tokens (0: padding), slot, position}
+__device__ __forceinline__ int4 single_segment(const DmoeShift& s, long long i) {
+  if (s.singles != nullptr) return static_cast<const int4*>(s.singles)[i];
+  return make_int4(static_cast<int>(i), s.kv_slots[i] >= 0 ? 1 : 0, s.rows[i], s.positions[i]);
+}
 constexpr int kSumThreads = 256, kSumWarps = kSumThreads / 32;
 constexpr int kMaxExperts = 256, kMaxTop = 32;
 
@@ -179,7 +194,8 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
   constexpr int G = kSumThreads / TPC, GW = G / 32;       // threads / warps per row
   extern __shared__ __align__(16) float s_row[];          // [TPC][W]
   __shared__ float red[kSumWarps];
-  __shared__ float slog[TPC][kMaxExperts];
+  __shared__ float slog[TPC][kMaxExperts];                // logits, then choice scores
+  __shared__ float sscore[TPC][kMaxExperts], sgroup[TPC][kMaxExperts];      // sigmoid router: scores, sums of the groups
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int j = threadIdx.x / G, tid = threadIdx.x % G;
   const int W = a.W, nvec = W / VEC;
@@ -209,12 +225,12 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
       if (y != nullptr) {
         Pack<T, VEC>::load(y + r * a.ld_y + v * VEC, t);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x[e] += t[e];
+        for (int e = 0; e < VEC; ++e) x[e] += a.mult * t[e];
       }
       for (int p = 0; p < a.n_parts; ++p) {
         Pack<T, VEC>::load(parts + r * a.part_row + p * a.part_stride + v * VEC, t);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x[e] += t[e];
+        for (int e = 0; e < VEC; ++e) x[e] += a.mult * t[e];
       }
       if (a.rows == nullptr && (y != nullptr || a.n_parts > 0)) Pack<float, VEC>::store(a.resid + r * W + v * VEC, x);
       Pack<float, VEC>::store(row + v * VEC, x);
@@ -232,6 +248,28 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
         ss += d * d;
       }
   const float inv = 1.f / sqrtf(group_sum(ss) / static_cast<float>(W) + a.eps);
+  if (a.shift.n_mix > 0) {
+    if (!valid) return;
+    const int4 seg = single_segment(a.shift, i);
+    const bool live = seg.y > 0 && seg.z >= 0 && seg.z < a.shift.n_slots;
+    float* last = a.shift.last + (live ? static_cast<long long>(seg.z) * W : 0);
+    for (int v = tid; v < nvec; v += G) {
+      float x[VEC], w[VEC], b[VEC] = {};
+      Pack<float, VEC>::load(row + v * VEC, x);
+      Pack<float, VEC>::load(a.w + v * VEC, w);
+      if (live && seg.w > 0) Pack<float, VEC>::load(last + v * VEC, b);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = (x[e] - mean) * inv * w[e];
+      if (live) Pack<float, VEC>::store(last + v * VEC, x);
+      for (int s = 0; s < a.shift.n_mix; ++s) {
+        Pack<float, VEC>::load(a.shift.mu + s * W + v * VEC, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) w[e] = x[e] + (b[e] - x[e]) * w[e];
+        Pack<T, VEC>::store(static_cast<T*>(a.h) + s * a.shift.mix_stride + i * a.ld_h + v * VEC, w);
+      }
+    }
+    return;
+  }
   if (valid)
     for (int v = tid; v < nvec; v += G) {
       float x[VEC], w[VEC];
@@ -239,6 +277,10 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
       Pack<float, VEC>::load(a.w + v * VEC, w);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x[e] = (x[e] - mean) * inv * w[e];
+      if (a.h_f32) {
+        Pack<float, VEC>::store(static_cast<float*>(a.h) + i * a.ld_h + v * VEC, x);
+        continue;
+      }
       Pack<T, VEC>::store(static_cast<T*>(a.h) + i * a.ld_h + v * VEC, x);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x[e] = static_cast<float>(static_cast<T>(x[e]));
@@ -278,13 +320,42 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
   const long long tok = static_cast<long long>(blockIdx.x) * TPC + warp;
   if (warp >= TPC || tok >= a.n) return;
   float* lg = slog[warp];
-  float mx = -INFINITY;
-  for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, lg[e]);
+  float* score = sscore[warp];
+  float mx = -INFINITY, den = 0.f;
+  if (a.sigmoid) {
+    for (int e = lane; e < a.E; e += 32) {
+      score[e] = 1.f / (1.f + expf(-lg[e]));
+      lg[e] = score[e] + (a.correction != nullptr ? a.correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (a.keep < a.groups) {
+      const int per = a.E / a.groups;
+      float* sum = sgroup[warp];
+      for (int g = lane; g < a.groups; g += 32) {
+        float first = -INFINITY, second = -INFINITY;
+        for (int e = g * per; e < (g + 1) * per; ++e) {
+          const float c = lg[e];
+          if (c > first) { second = first; first = c; }
+          else if (c > second) second = c;
+        }
+        sum[g] = per > 1 ? first + second : first;
+      }
+      __syncwarp();
+      for (int g = lane; g < a.groups; g += 32) {
+        int ahead = 0;
+        for (int q = 0; q < a.groups; ++q) ahead += sum[q] > sum[g] || (sum[q] == sum[g] && q < g);
+        if (ahead >= a.keep)
+          for (int e = g * per; e < (g + 1) * per; ++e) lg[e] = -INFINITY;
+      }
+      __syncwarp();
+    }
+  } else {
+    for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, lg[e]);
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-  float den = 0.f;
-  for (int e = lane; e < a.E; e += 32) den += expf(lg[e] - mx);
-  den = warp_sum(den);
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    for (int e = lane; e < a.E; e += 32) den += expf(lg[e] - mx);
+    den = warp_sum(den);
+  }
   int my_id = -1;           // lane k keeps the k-th choice
   float my_w = 0.f, total = 0.f;
   for (int k = 0; k < a.K; ++k) {
@@ -298,7 +369,7 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
     }
-    float s = expf(best - mx) / den;
+    float s = a.sigmoid ? (bi < a.E ? score[bi] : 0.f) : expf(best - mx) / den;
     if (bi >= a.E) {        // no finite logit left: the lowest expert not chosen yet, so that the ids stay valid
       for (bi = 0; __any_sync(0xffffffffu, my_id == bi);) ++bi;
       s = 0.f;
@@ -311,8 +382,69 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
   }
   if (lane < a.K) {
     a.ids[tok * a.K + lane] = my_id;
-    a.wts[tok * a.K + lane] = a.renorm && total > 0.f ? my_w / total : my_w;
+    a.wts[tok * a.K + lane] = (a.renorm && total > 0.f ? my_w / total : my_w) * a.wscale;
     if (a.counts != nullptr) atomicAdd(&a.counts[my_id], 1);
+  }
+}
+
+// Token shift of a batch that holds longer segments: rows h (fp32) -> S mixed rows h + (before - h) mu_s, `before` = the row before
+// of the same segment or, for its first row, the slot's last row. grid.x: the one-token segments, then the chunks of the longer ones
+// (int4 {first row, tokens, segment, number in the segment}); grid.y: runs of kShiftRows rows of a chunk; grid.z: columns. The
+// thread that reads the slot's old row writes the new one, the segment's last.
+constexpr int kShiftRows = 16, kShiftThreads = 128, kMaxMix = 8;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kShiftThreads)
+token_shift_kernel(const float* __restrict__ h, const DmoeShift a, const int4* __restrict__ multi, const int4* __restrict__ chunks,
+                   T* __restrict__ out, long long ld, int W) {
+  int row0, n, slot, pos0, last_row = -1;       // rows [row0, row0 + n); last_row >= 0: row0 starts its segment, which ends there
+  bool first;
+  if (blockIdx.x < a.n_single) {
+    if (blockIdx.y > 0) return;
+    const int4 seg = single_segment(a, blockIdx.x);
+    if (seg.y <= 0) return;
+    row0 = last_row = seg.x; n = 1; slot = seg.z; pos0 = seg.w; first = true;
+  } else {
+    const int4 ck = chunks[blockIdx.x - a.n_single];
+    const int4 seg = multi[ck.z];
+    const int skip = blockIdx.y * kShiftRows;
+    if (skip >= ck.y) return;
+    row0 = ck.x + skip; n = min(kShiftRows, ck.y - skip); slot = seg.z; pos0 = seg.w;
+    first = row0 == seg.x;
+    last_row = seg.x + seg.y - 1;
+  }
+  if (slot < 0 || slot >= a.n_slots) return;
+  const int c = (blockIdx.z * kShiftThreads + threadIdx.x) * VEC;
+  if (c >= W) return;
+  float b[VEC] = {};
+  float* last = a.last + static_cast<long long>(slot) * W + c;
+  if (!first) Pack<float, VEC>::load(h + (row0 - 1ll) * W + c, b);
+  else {
+    if (pos0 > 0) Pack<float, VEC>::load(last, b);
+    float x[VEC];
+    Pack<float, VEC>::load(h + static_cast<long long>(last_row) * W + c, x);
+    Pack<float, VEC>::store(last, x);
+  }
+  for (int s0 = 0; s0 < a.n_mix; s0 += 3) {          // mixing factors of three outputs at a time in registers
+    float mu[3][VEC], p[VEC];
+#pragma unroll
+    for (int s = 0; s < 3; ++s)
+      if (s0 + s < a.n_mix) Pack<float, VEC>::load(a.mu + (s0 + s) * static_cast<long long>(W) + c, mu[s]);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) p[e] = b[e];
+    for (int t = 0; t < n; ++t) {
+      float x[VEC], y[VEC];
+      Pack<float, VEC>::load(h + static_cast<long long>(row0 + t) * W + c, x);
+#pragma unroll
+      for (int s = 0; s < 3; ++s) {
+        if (s0 + s >= a.n_mix) break;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = x[e] + (p[e] - x[e]) * mu[s][e];
+        Pack<T, VEC>::store(out + (s0 + s) * a.mix_stride + static_cast<long long>(row0 + t) * ld + c, y);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) p[e] = x[e];
+    }
   }
 }
 
@@ -329,14 +461,15 @@ __global__ void rope_freq_table_kernel(float2* __restrict__ table, int max_pos, 
 // rows [q heads | k heads | v heads] (the last two only where n_kv > 0): RMS norm over each q / k head with its weight (qw !=
 // NULL), rotation of the pairs (i, i + rot / 2) or, interleaved, (2i, 2i + 1), i < rot / 2, q written back in place, k and v
 // appended to the paged caches ([blocks, block_size, n_kv, dk] and [.., dv]) at slots[t] (< 0: skip). v_first != NULL: what is
-// appended is (1 - lambda) v + lambda v_first (head size first_head in memory). One warp per head.
+// appended is (1 - lambda) v + lambda v_first (head size first_head in memory). tied: rows end after the k heads, and the values
+// are the first dv dimensions of every k head as it stands there, not rotated. One warp per head.
 template <typename T>
 __global__ void __launch_bounds__(256)
 qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ positions,
                     const long long* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache, int n_q, int n_kv,
                     int dk, int dv, int rot, int interleaved, const float2* __restrict__ table, int max_pos,
                     const float* __restrict__ qw, const float* __restrict__ kw, float eps, const T* __restrict__ v_first,
-                    long long ld_first, int first_head, float v_lambda) {
+                    long long ld_first, int first_head, float v_lambda, int tied) {
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int half = rot / 2;
@@ -374,10 +507,10 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
     }
   }
   if (slot >= 0) {
-    const T* src = row + static_cast<long long>(n_q + n_kv) * dk;
+    const T* src = row + static_cast<long long>(tied ? n_q : n_q + n_kv) * dk;
     T* dst = vcache + slot * n_kv * dv;
     for (int i = threadIdx.x; i < n_kv * dv; i += blockDim.x) {
-      if (v_first == nullptr) { dst[i] = src[i]; continue; }
+      if (v_first == nullptr) { dst[i] = src[tied ? i / dv * dk + i % dv : i]; continue; }
       const int d = i % dv;
       const float first = d < first_head ? static_cast<float>(v_first[t * ld_first + i / dv * first_head + d]) : 0.f;
       dst[i] = static_cast<T>((1.f - v_lambda) * static_cast<float>(src[i]) + v_lambda * first);
@@ -385,13 +518,14 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
   }
 }
 
-// The same for interleaved rotation without norms where everything moves in 16-byte units (dk, dv and rot multiples of 8):
-// the units of a row's heads are dealt out to the threads.
+// The same without norms where everything moves in 16-byte units (dk, dv and rot multiples of 8; rot / 2 too where pairs are
+// half a rotation apart): the units of a row's heads are dealt out to the threads, a unit of first halves together with the unit
+// of its second halves.
 __global__ void __launch_bounds__(256)
 rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
                    bf16* __restrict__ kcache, bf16* __restrict__ vcache, int n_q, int n_kv, int dk, int dv, int rot,
-                   const float2* __restrict__ table, int max_pos, const bf16* __restrict__ v_first, long long ld_first,
-                   int first_head, float v_lambda) {
+                   int interleaved, const float2* __restrict__ table, int max_pos, const bf16* __restrict__ v_first,
+                   long long ld_first, int first_head, float v_lambda, int tied) {
   const long long t = blockIdx.x;
   const int pos = min(max(positions[t], 0), max_pos - 1);
   const long long slot = slots[t];
@@ -402,10 +536,22 @@ rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__
     const int d = u * 8 % dk;
     const bool is_q = u < uq;
     if (is_q && d >= rot) continue;           // in place already
+    if (!interleaved && d >= rot / 2 && d < rot) continue;      // goes with its first half
     bf16* dst = is_q ? row + u * 8 : kcache + slot * n_kv * dk + (u - uq) * 8;
     float x[8];
     Pack<bf16, 8>::load(row + u * 8, x);
-    if (d < rot) {
+    if (!interleaved && d < rot) {
+      float y[8];
+      Pack<bf16, 8>::load(row + u * 8 + rot / 2, y);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float2 cs = tab[d + e];
+        const float p = x[e], q = y[e];
+        x[e] = p * cs.x - q * cs.y;
+        y[e] = q * cs.x + p * cs.y;
+      }
+      Pack<bf16, 8>::store(dst + rot / 2, y);
+    } else if (d < rot) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 cs = tab[d / 2 + e];
@@ -417,11 +563,11 @@ rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__
     Pack<bf16, 8>::store(dst, x);
   }
   if (slot < 0) return;
-  const bf16* src = row + static_cast<long long>(n_q + n_kv) * dk;
+  const bf16* src = row + static_cast<long long>(tied ? n_q : n_q + n_kv) * dk;
   bf16* dst = vcache + slot * n_kv * dv;
   for (int u = threadIdx.x; u < n_kv * dv / 8; u += blockDim.x) {
     float x[8];
-    Pack<bf16, 8>::load(src + u * 8, x);
+    Pack<bf16, 8>::load(src + (tied ? u * 8 / dv * dk + u * 8 % dv : u * 8), x);
     if (v_first != nullptr) {
       const int h = u * 8 / dv, d = u * 8 % dv;
       float y[8] = {};
@@ -447,14 +593,14 @@ __global__ void gate_mul_kernel(const T* __restrict__ gu, long long ld, T* __res
 
 // Y[t, f] = sum_k X[t, k] W[f, k] with fp32 multiply-adds: 64 x 64 tiles, 4 x 4 outputs per thread. With offs, W is a stack of
 // G matrices [F, K] and group g has rows offs[g] .. offs[g + 1] (blockIdx.y counts row tiles group after group); with recs, row
-// t is scaled and stored where its record {buffer, row or < 0, weight bits, -} says.
+// t is scaled and stored where its record {buffer, row or < 0, weight bits, -} says. act 2: tanh of the output.
 constexpr int kSgTile = 64, kSgK = 16;
 
 template <typename T, typename TY>
 __global__ void __launch_bounds__(256)
 simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw, TY* __restrict__ Y,
                  long long ldy, int M, int F, int K, const int* __restrict__ offs, int G, const int4* __restrict__ recs,
-                 void* const* __restrict__ bases) {
+                 void* const* __restrict__ bases, int act) {
   __shared__ float sx[kSgK][kSgTile + 4], sw[kSgK][kSgTile + 4];
   int t0 = blockIdx.y * kSgTile, t1 = M;
   const int f0 = blockIdx.x * kSgTile;
@@ -507,7 +653,7 @@ simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int f = f0 + tx * 4 + j;
-      if (f < F) dst[f] = static_cast<TY>(acc[i][j] * scale);
+      if (f < F) dst[f] = static_cast<TY>(act == 2 ? tanhf(acc[i][j]) : acc[i][j] * scale);
     }
   }
 }
@@ -592,51 +738,85 @@ extern "C" int dmoe_rope_freq_table(void* table, int max_pos, int half, const do
 }
 
 extern "C" int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
-                             long long part_row, long long part_stride, const float* w, int centred, float eps, const int* rows,
-                             void* h, long long ld_h, int n, int W, const void* gate_w, int E, int K, int renorm, int* ids,
-                             float* wts, int* counts, void* stream_) {
+                             long long part_row, long long part_stride, float mult, const float* w, int centred, float eps,
+                             const int* rows, void* h, int h_f32, long long ld_h, int n, int W, const DmoeRouter* router,
+                             const DmoeShift* shift, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (W < 1 || resid == nullptr || h == nullptr || w == nullptr || n_parts < 0) return -10;
-  if (gate_w != nullptr && (E < 1 || E > kMaxExperts || K < 1 || K > kMaxTop || K > E || ids == nullptr || wts == nullptr)) return -10;
+  static const DmoeRouter no_router = {};
+  static const DmoeShift no_shift = {};
+  const DmoeRouter& r = router != nullptr ? *router : no_router;
+  const DmoeShift& s = shift != nullptr ? *shift : no_shift;
+  if (router != nullptr && (r.weight == nullptr || r.E < 1 || r.E > kMaxExperts || r.K < 1 || r.K > kMaxTop || r.K > r.E ||
+                            r.ids == nullptr || r.wts == nullptr || h_f32 || shift != nullptr)) return -10;
+  if (r.sigmoid && (r.groups < 1 || r.E % r.groups != 0 || r.keep < 1)) return -10;
+  if (shift != nullptr && (rows != nullptr || s.n_single != n || s.n_mix < 1 || s.mu == nullptr || s.last == nullptr ||
+                           (s.singles == nullptr && (s.positions == nullptr || s.rows == nullptr || s.kv_slots == nullptr)))) return -10;
   if (n == 0) return 0;
   if (parts == nullptr) n_parts = 0;
-  const SumNormArgs a{resid, y, ld_y, parts, n_parts, part_row, part_stride, w, centred, eps, rows, h, ld_h, n, W, gate_w, E, K,
-                      renorm, ids, wts, counts};
+  const SumNormArgs a{resid, y, ld_y, parts, n_parts, part_row, part_stride, w, centred, eps, rows, h, ld_h, n, W, r.weight, r.E,
+                      r.K, r.renorm, r.ids, r.wts, r.counts, mult, h_f32, r.sigmoid, r.groups, r.keep, r.correction, r.wscale, s};
   const bool vec = W % 8 == 0 && ld_y % 8 == 0 && ld_h % 8 == 0 && part_row % 8 == 0 && part_stride % 8 == 0 && aligned16(resid) &&
-                   aligned16(y) && aligned16(parts) && aligned16(w) && aligned16(h) && aligned16(gate_w);
+                   aligned16(y) && aligned16(parts) && aligned16(w) && aligned16(h) && aligned16(r.weight) && aligned16(s.mu) &&
+                   aligned16(s.last) && s.mix_stride % 8 == 0;
   if (is_f32) return vec ? launch_sum_norm<float, 8>(a, stream) : launch_sum_norm<float, 1>(a, stream);
   return vec ? launch_sum_norm<bf16, 8>(a, stream) : launch_sum_norm<bf16, 1>(a, stream);
+}
+
+extern "C" int dmoe_token_shift(int is_f32, const float* h, const DmoeShift* s, const void* multi, int n_multi, const void* chunks,
+                                int n_chunks, void* out, long long ld, int W, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (W < 1 || h == nullptr || out == nullptr || s->n_mix < 1 || s->n_mix > kMaxMix || s->mu == nullptr || s->last == nullptr) return -10;
+  if (s->n_single < 0 || n_chunks < 0 || (n_chunks > 0 && (multi == nullptr || chunks == nullptr || n_multi < 1))) return -10;
+  if (s->n_single > 0 && s->singles == nullptr && (s->positions == nullptr || s->rows == nullptr || s->kv_slots == nullptr)) return -10;
+  if (s->n_single + n_chunks == 0) return 0;
+  const bool vec = W % 8 == 0 && ld % 8 == 0 && s->mix_stride % 8 == 0 && aligned16(h) && aligned16(out) && aligned16(s->mu) &&
+                   aligned16(s->last);
+  const int per = kShiftThreads * (vec ? 8 : 1);
+  const dim3 grid(s->n_single + n_chunks, n_chunks > 0 ? 64 / kShiftRows : 1, (W + per - 1) / per);
+  const int4* mt = static_cast<const int4*>(multi);
+  const int4* ck = static_cast<const int4*>(chunks);
+#define DMOE_SHIFT(T_, VEC_) token_shift_kernel<T_, VEC_><<<grid, kShiftThreads, 0, stream>>>(h, *s, mt, ck, static_cast<T_*>(out), ld, W)
+  if (is_f32 && vec) DMOE_SHIFT(float, 8);
+  else if (is_f32) DMOE_SHIFT(float, 1);
+  else if (vec) DMOE_SHIFT(bf16, 8);
+  else DMOE_SHIFT(bf16, 1);
+#undef DMOE_SHIFT
+  return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots,
                                  void* kcache, void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved,
                                  const void* table, int max_pos, const float* qw, const float* kw, float eps,
-                                 const void* v_first, long long ld_first, int first_head, float v_lambda, void* stream_) {
+                                 const void* v_first, long long ld_first, int first_head, float v_lambda, int tied,
+                                 void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (n_q < 1 || n_kv < 0 || dk < 1 || rot < 0 || rot % 2 != 0 || rot > dk || (rot > 0 && table == nullptr)) return -10;
   if (n_kv > 0 && (kcache == nullptr || vcache == nullptr || (qw != nullptr && kw == nullptr))) return -10;
-  if (v_first != nullptr && first_head < 1) return -10;
+  if (v_first != nullptr && (first_head < 1 || tied)) return -10;
+  if (tied && dv > dk) return -10;
   if (T == 0) return 0;
   int threads = (n_q + n_kv) * 32;
   if (threads > 256) threads = 256;
-  if (!is_f32 && qw == nullptr && n_kv > 0 && (interleaved || rot == 0) && dk % 8 == 0 && dv % 8 == 0 && rot % 8 == 0 &&
+  if (!is_f32 && qw == nullptr && n_kv > 0 && dk % 8 == 0 && dv % 8 == 0 && rot % (interleaved ? 8 : 16) == 0 &&
       ld % 8 == 0 && first_head % 8 == 0 && ld_first % 8 == 0 && aligned16(qkv) && aligned16(kcache) && aligned16(vcache) &&
       aligned16(v_first)) {
     rope_append_kernel<<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk, dv,
-        rot, static_cast<const float2*>(table), max_pos, static_cast<const bf16*>(v_first), ld_first, first_head, v_lambda);
+        rot, interleaved, static_cast<const float2*>(table), max_pos, static_cast<const bf16*>(v_first), ld_first, first_head,
+        v_lambda, tied);
     return static_cast<int>(cudaGetLastError());
   }
   if (is_f32)
     qk_norm_rope_kernel<float><<<T, threads, 0, stream>>>(
         static_cast<float*>(qkv), ld, positions, slots, static_cast<float*>(kcache), static_cast<float*>(vcache), n_q, n_kv,
         dk, dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const float*>(v_first),
-        ld_first, first_head, v_lambda);
+        ld_first, first_head, v_lambda, tied);
   else
     qk_norm_rope_kernel<bf16><<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk,
         dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const bf16*>(v_first),
-        ld_first, first_head, v_lambda);
+        ld_first, first_head, v_lambda, tied);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -658,7 +838,7 @@ extern "C" int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, 
 }
 
 extern "C" int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y,
-                                long long ldy, int T, int F, int K, void* stream_) {
+                                long long ldy, int T, int F, int K, int act, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (F < 1 || K < 1 || (x_f32 && !y_f32)) return -10;
   if (T == 0) return 0;
@@ -667,13 +847,13 @@ extern "C" int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long l
   const dim3 grid((F + kSgTile - 1) / kSgTile, static_cast<unsigned>(ty));
   if (x_f32)
     simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W),
-                                                             ldw, static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
+                                                             ldw, static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
   else if (y_f32)
     simt_gemm_kernel<bf16, float><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                            static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
+                                                            static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
   else
     simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                           static_cast<bf16*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr);
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -689,9 +869,9 @@ extern "C" int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const
   void* const* b = static_cast<void* const*>(bases);
   if (is_f32)
     simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W), K,
-                                                             static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b);
+                                                             static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b, 0);
   else
     simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), K,
-                                                           static_cast<bf16*>(Y), ldy, T, F, K, offs, G, r, b);
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, offs, G, r, b, 0);
   return static_cast<int>(cudaGetLastError());
 }

@@ -1,9 +1,10 @@
 // Linear recurrences with a matrix-valued state per head, S [dim, vdim] in fp32, a decay per head and key channel and
-// one of two writes per token:
+// one of two writes per token (the plain one with two places of the read-out):
 //
 //   plain   S <- diag(a) S + k v^T                                 (gated linear attention)
 //   delta   S <- diag(a) S;  S <- S + k (beta (v - S^T k))^T       (gated delta rule)
 //   o = S^T q, read after the write
+//   bonus   o = (S + diag(u) k v^T)^T q, then the plain write      (RWKV-style time mixing)
 //
 // States live in slots: slot = block-table row of the sequence, so a sequence's state is found with the same index as
 // its KV pages, and a sequence whose first token is in the batch (position 0) starts from zero whatever the slot held.
@@ -23,9 +24,9 @@ constexpr int kStepThreads = 256;
 constexpr int kStepRows = 16;        // state rows a thread holds in registers
 
 // Decay factor, q and k of the token's key channels and its values -> shared memory (convolved and activated with CONV).
-template <typename T, bool DELTA, bool CONV>
+template <typename T, int MODE, bool CONV>
 __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, int pos, int slot, int h, int hk, int v0, int nv,
-                                             float decay_scale, float4* s_gqk, float* s_v) {
+                                             float scale, float4* s_gqk, float* s_v) {
   const int D = a.dim, V = a.vdim, group = a.heads / a.kv_heads;
   for (int i = threadIdx.x; i < D + nv; i += blockDim.x) {
     if (i < D) {
@@ -42,7 +43,7 @@ __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, 
         q = static_cast<float>(static_cast<const T*>(a.q)[row * a.ldq + hk * D + i]);
         k = static_cast<float>(static_cast<const T*>(a.k)[row * a.ldk + hk * D + i]);
       }
-      s_gqk[i] = make_float4(expf(log_decay(a.decay_kind, z, decay_scale)), q, k, 0.f);
+      s_gqk[i] = make_float4(expf(log_decay(a.decay_kind, z, scale)), q, k, MODE == kBonus ? a.bonus[h * D + i] : 0.f);
     } else {
       const int c = h * V + v0 + i - D;
       if (CONV) {
@@ -56,24 +57,25 @@ __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, 
   }
 }
 
-// Factors that turn the raw rows into q (scaled, unit) and k (unit), and q.k of the raw rows; every warp on its own.
+// Factors that turn the raw rows into q (scaled, unit) and k (unit), and the weight of the token's own write in its read-out:
+// q.k of the raw rows, with the bonus q.(u k); every warp on its own.
 struct RowFactors {
   float fq, fk, qk;
 };
-template <bool DELTA>
+template <int MODE>
 __device__ __forceinline__ RowFactors row_factors(const DmoeRecur& a, const float4* s_gqk) {
   float qq = 0.f, kk = 0.f, qk = 0.f;
   for (int d = threadIdx.x & 31; d < a.dim; d += 32) {
     const float4 x = s_gqk[d];
     qq += x.y * x.y;
     kk += x.z * x.z;
-    qk += x.y * x.z;
+    qk += MODE == kBonus ? x.y * (x.z * x.w) : x.y * x.z;
   }
   RowFactors f;
   f.qk = warp_sum(qk);
   f.fq = a.qscale;
   f.fk = 1.f;
-  if (DELTA) {
+  if (MODE == kDelta) {
     f.fq *= 1.f / sqrtf(warp_sum(qq) + 1e-6f);
     f.fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
   }
@@ -82,11 +84,12 @@ __device__ __forceinline__ RowFactors row_factors(const DmoeRecur& a, const floa
 
 // One CTA: one segment, one head, `vt` value columns. Threads form a grid of (vt / VEC) column groups x rpp row groups;
 // a thread keeps rows rg, rg + rpp, ... of its VEC columns in registers for the whole segment. Per token the read-outs
-// of the decayed state at k and at q are reduced together, and o = (a S)^T q + (k.q) u gives the read-out after the
-// write without a second pass.
-template <typename T, bool DELTA, bool CONV, int VEC>
+// of the decayed (with a bonus: undecayed) state at k and at q are reduced together, and o = (a S)^T q + (k.q) u gives the
+// read-out after the write without a second pass.
+template <typename T, int MODE, bool CONV, int VEC>
 __global__ void __launch_bounds__(kStepThreads, 2)
 step_kernel(const DmoeRecur a, int vt) {
+  constexpr bool DELTA = MODE == kDelta;
   extern __shared__ __align__(16) float s_mem[];
   const int tid = threadIdx.x, lane = tid & 31;
   const int4 seg = a.segs != nullptr ? static_cast<const int4*>(a.segs)[blockIdx.x] : row_segment(a, blockIdx.x);
@@ -113,7 +116,8 @@ step_kernel(const DmoeRecur a, int vt) {
     for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
     if (mine && d < D && pos0 > 0) load_vec<VEC>(sp + static_cast<long long>(d) * V, S[i]);
   }
-  const float decay_scale = a.decay_kind == 0 ? a.inv_tau : expf(a.a_log[h]);
+  const float dscale = decay_scale(a, h);
+  const float* norm_w = a.norm_w + h * a.norm_ld;
 
   for (int t = 0; t < ntok; ++t) {
     const long long row = row0 + t;
@@ -125,11 +129,11 @@ step_kernel(const DmoeRecur a, int vt) {
     if (DELTA) beta = static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h]);
     if (fused) {
       gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + oc]);
-      weight = a.norm_w[oc];
+      weight = norm_w[oc];
     }
-    token_inputs<T, DELTA, CONV>(a, row, pos, slot, h, hk, v0, nv, decay_scale, s_gqk, s_v);
+    token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, v0, nv, dscale, s_gqk, s_v);
     __syncthreads();
-    const RowFactors f = row_factors<DELTA>(a, s_gqk);
+    const RowFactors f = row_factors<MODE>(a, s_gqk);
     const float fq = f.fq, fk = f.fk, qk = f.qk;
     if (DELTA) beta = 1.f / (1.f + expf(-beta));
     float rq[VEC], rk[VEC];
@@ -143,8 +147,9 @@ step_kernel(const DmoeRecur a, int vt) {
           const float4 x = s_gqk[d];
 #pragma unroll
           for (int e = 0; e < VEC; ++e) {
+            if (MODE == kBonus) rq[e] += S[i][e] * x.y;
             S[i][e] *= x.x;
-            rq[e] += S[i][e] * x.y;
+            if (MODE != kBonus) rq[e] += S[i][e] * x.y;
             if (DELTA) rk[e] += S[i][e] * x.z;
           }
         }
@@ -191,7 +196,7 @@ step_kernel(const DmoeRecur a, int vt) {
       for (int c = tid; c < V; c += kStepThreads) {
         if (c != tid) {                // heads wider than the CTA
           gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
-          weight = a.norm_w[c];
+          weight = norm_w[c];
         }
         static_cast<T*>(a.out)[row * a.ldo + h * V + c] = static_cast<T>(s_o[c] * inv * weight * gate_value(a.gate_kind, gate));
       }
@@ -203,9 +208,10 @@ step_kernel(const DmoeRecur a, int vt) {
 // Decode steps at full bandwidth: one CTA per (sequence, head), the head's state fetched by one bulk copy into shared memory
 // while the token's inputs are prepared (three CTAs per SM keep copies in flight), updated from there straight back to
 // global memory. One-token segments, whole heads, vdim a multiple of 4.
-template <typename T, bool DELTA, bool CONV>
+template <typename T, int MODE, bool CONV>
 __global__ void __launch_bounds__(kStepThreads, 3)
 stream_step_kernel(const DmoeRecur a) {
+  constexpr bool DELTA = MODE == kDelta;
   extern __shared__ __align__(128) float s_stream[];
   __shared__ __align__(8) unsigned long long s_bar;
   __shared__ int s_abort;
@@ -236,15 +242,16 @@ stream_step_kernel(const DmoeRecur a) {
   }
   const int vq = V / 4, rpp = kStepThreads / vq, cg = tid % vq, rg = tid / vq;
   const bool mine = rg < rpp;
+  const float* norm_w = a.norm_w + h * a.norm_ld;
   float beta = 0.f, gate = 0.f, weight = 0.f;
   if (DELTA) beta = static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h]);
   if (tid < V) {
     gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + tid]);
-    weight = a.norm_w[tid];
+    weight = norm_w[tid];
   }
-  token_inputs<T, DELTA, CONV>(a, row, pos, slot, h, hk, 0, V, a.decay_kind == 0 ? a.inv_tau : expf(a.a_log[h]), s_gqk, s_v);
+  token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, 0, V, decay_scale(a, h), s_gqk, s_v);
   __syncthreads();                                               // the inputs, and the barrier's initialisation
-  const RowFactors f = row_factors<DELTA>(a, s_gqk);
+  const RowFactors f = row_factors<MODE>(a, s_gqk);
   if (DELTA) beta = 1.f / (1.f + expf(-beta));
   if (pos > 0 && !mbar_wait(bar, 0, &s_abort) && tid == 0 && a.status != nullptr) atomicExch(a.status, kStatusBarrierTimeout);
   float rq[4] = {0.f, 0.f, 0.f, 0.f}, rk[4] = {0.f, 0.f, 0.f, 0.f};
@@ -254,7 +261,8 @@ stream_step_kernel(const DmoeRecur a) {
       for (int d = rg; d < D; d += rpp) {
         const float4 x = s_gqk[d];
         const float4 s = *reinterpret_cast<const float4*>(s_S + d * V + cg * 4);
-        const float sv[4] = {s.x * x.x, s.y * x.x, s.z * x.x, s.w * x.x};
+        const float f0 = MODE == kBonus ? 1.f : x.x;
+        const float sv[4] = {s.x * f0, s.y * f0, s.z * f0, s.w * f0};
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           rq[e] += sv[e] * x.y;
@@ -300,7 +308,7 @@ stream_step_kernel(const DmoeRecur a) {
   for (int c = tid; c < V; c += kStepThreads) {
     if (c != tid) {                                              // heads wider than the CTA
       gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
-      weight = a.norm_w[c];
+      weight = norm_w[c];
     }
     static_cast<T*>(a.out)[row * a.ldo + h * V + c] = static_cast<T>(s_o[c] * inv * weight * gate_value(a.gate_kind, gate));
   }
@@ -311,22 +319,23 @@ stream_step_kernel(const DmoeRecur a) {
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, long long ldraw, const T* __restrict__ gate,
-                 long long ldg, const float* __restrict__ norm_w, float eps, int gate_kind, T* __restrict__ out,
+                 long long ldg, const float* __restrict__ norm_w, int norm_ld, float eps, int gate_kind, T* __restrict__ out,
                  long long ldo, int heads, int V) {
   const int4 e = table != nullptr ? table[blockIdx.x] : make_int4(blockIdx.x, 1, 0, 0);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  for (int i = blockIdx.y * nw + warp; i < e.y * heads; i += gridDim.y * nw) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  for (int i = blockIdx.y * warps + warp; i < e.y * heads; i += gridDim.y * warps) {
     const long long row = e.x + i / heads;
     const int h = i % heads;
     const float* r = raw + row * ldraw + h * V;
     const T* gp = gate + row * ldg + h * V;
+    const float* nw = norm_w + h * norm_ld;
     float x[VEC], gv[VEC], w[VEC];
     float ss = 0.f;
     const int c0 = lane * VEC;
     if (c0 < V) {                          // the first pass stays in registers (all of it where V <= 32 VEC)
       load_vec<VEC>(r + c0, x);
       load_any<VEC>(gp + c0, gv);
-      load_vec<VEC>(norm_w + c0, w);
+      load_vec<VEC>(nw + c0, w);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) ss += x[k] * x[k];
     }
@@ -341,7 +350,7 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
       if (c != c0) {
         load_vec<VEC>(r + c, x);
         load_any<VEC>(gp + c, gv);
-        load_vec<VEC>(norm_w + c, w);
+        load_vec<VEC>(nw + c, w);
       }
 #pragma unroll
       for (int k = 0; k < VEC; ++k) x[k] *= inv * w[k] * gate_value(gate_kind, gv[k]);
@@ -432,7 +441,7 @@ static int check_recur(const DmoeRecur* a) {
   if (a->heads < 1 || a->kv_heads < 1 || a->heads % a->kv_heads != 0 || a->dim < 1 || a->vdim < 1) return -10;
   if (a->heads > 65535 || a->state == nullptr || a->z_bias == nullptr || a->n_slots < 1) return -10;
   if (a->segs == nullptr && (a->positions == nullptr || a->rows == nullptr || a->kv_slots == nullptr)) return -10;
-  if (a->decay_kind != 0 && a->a_log == nullptr) return -10;
+  if ((a->decay_kind == 1 && a->a_log == nullptr) || (a->bonus != nullptr && (a->delta || a->taps > 0))) return -10;
   if (a->taps < 0 || a->taps > kMaxTaps || (a->taps > 0 && (a->conv_w == nullptr || a->ring == nullptr))) return -11;
   return 0;
 }
@@ -449,25 +458,25 @@ static size_t stream_smem(const DmoeRecur& a) {
   return b <= kStreamSmem ? b : 0;
 }
 
-template <typename T, bool DELTA, bool CONV>
+template <typename T, int MODE, bool CONV>
 static int launch_stream(const DmoeRecur& a, size_t smem, cudaStream_t stream) {
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(stream_step_kernel<T, DELTA, CONV>,
+    return static_cast<int>(cudaFuncSetAttribute(stream_step_kernel<T, MODE, CONV>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, kStreamSmem));
   });
   if (rc != 0) return rc;
-  return static_cast<int>(launch_kernel(stream_step_kernel<T, DELTA, CONV>, dim3(a.n_segs, a.heads), dim3(kStepThreads), smem,
+  return static_cast<int>(launch_kernel(stream_step_kernel<T, MODE, CONV>, dim3(a.n_segs, a.heads), dim3(kStepThreads), smem,
                                         stream, a));
 }
 
-template <typename T, bool DELTA, bool CONV, int VEC>
+template <typename T, int MODE, bool CONV, int VEC>
 static int launch_step(const DmoeRecur& a, int vt, cudaStream_t stream) {
   const int vq = vt / VEC, rpp = kStepThreads / vq;
-  const size_t smem = (4 * static_cast<size_t>(a.dim) + 3 * vt + static_cast<size_t>(DELTA ? 2 : 1) * rpp * vt) * sizeof(float);
+  const size_t smem = (4 * static_cast<size_t>(a.dim) + 3 * vt + static_cast<size_t>(MODE == kDelta ? 2 : 1) * rpp * vt) * sizeof(float);
   if (smem > 48 * 1024) return -13;
   const dim3 grid(a.n_segs, a.heads, (a.vdim + vt - 1) / vt);
-  return static_cast<int>(launch_kernel(step_kernel<T, DELTA, CONV, VEC>, grid, dim3(kStepThreads), smem, stream, a, vt));
+  return static_cast<int>(launch_kernel(step_kernel<T, MODE, CONV, VEC>, grid, dim3(kStepThreads), smem, stream, a, vt));
 }
 
 template <typename T>
@@ -475,15 +484,18 @@ static int step_dispatch(const DmoeRecur& a, int vt, bool vec, cudaStream_t stre
   const bool conv = a.taps > 0;
   const size_t smem = a.one_token ? stream_smem(a) : 0;
   if (smem > 0) {
-    if (!a.delta) return conv ? -12 : launch_stream<T, false, false>(a, smem, stream);
-    return conv ? launch_stream<T, true, true>(a, smem, stream) : launch_stream<T, true, false>(a, smem, stream);
+    if (a.bonus != nullptr) return launch_stream<T, kBonus, false>(a, smem, stream);
+    if (!a.delta) return conv ? -12 : launch_stream<T, kPlain, false>(a, smem, stream);
+    return conv ? launch_stream<T, kDelta, true>(a, smem, stream) : launch_stream<T, kDelta, false>(a, smem, stream);
   }
+  if (a.bonus != nullptr)
+    return vec ? launch_step<T, kBonus, false, 4>(a, vt, stream) : launch_step<T, kBonus, false, 1>(a, vt, stream);
   if (!a.delta) {
     if (conv) return -12;
-    return vec ? launch_step<T, false, false, 4>(a, vt, stream) : launch_step<T, false, false, 1>(a, vt, stream);
+    return vec ? launch_step<T, kPlain, false, 4>(a, vt, stream) : launch_step<T, kPlain, false, 1>(a, vt, stream);
   }
-  if (conv) return vec ? launch_step<T, true, true, 4>(a, vt, stream) : launch_step<T, true, true, 1>(a, vt, stream);
-  return vec ? launch_step<T, true, false, 4>(a, vt, stream) : launch_step<T, true, false, 1>(a, vt, stream);
+  if (conv) return vec ? launch_step<T, kDelta, true, 4>(a, vt, stream) : launch_step<T, kDelta, true, 1>(a, vt, stream);
+  return vec ? launch_step<T, kDelta, false, 4>(a, vt, stream) : launch_step<T, kDelta, false, 1>(a, vt, stream);
 }
 
 }  // namespace dmoe
@@ -518,7 +530,7 @@ extern "C" int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream_) {
 }
 
 extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw,
-                              const void* gate, long long ldg, const float* norm_w, float eps, int gate_kind, void* out,
+                              const void* gate, long long ldg, const float* norm_w, int norm_ld, float eps, int gate_kind, void* out,
                               long long ldo, int heads, int V, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (heads < 1 || V < 1 || max_tokens < 1) return -10;
@@ -527,10 +539,10 @@ extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_toke
   if (by > 1024) by = 1024;
   const dim3 grid(n, static_cast<unsigned>(by));
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool vec = V % 4 == 0 && ldraw % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(raw) && al(gate) && al(out) && al(norm_w);
+  const bool vec = V % 4 == 0 && norm_ld % 4 == 0 && ldraw % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(raw) && al(gate) && al(out) && al(norm_w);
 #define DMOE_GATE_NORM(T_, VEC_)                                                                                       \
   gate_norm_kernel<T_, VEC_><<<grid, 256, 0, stream>>>(static_cast<const int4*>(table), raw, ldraw,                    \
-                                                       static_cast<const T_*>(gate), ldg, norm_w, eps, gate_kind,      \
+                                                       static_cast<const T_*>(gate), ldg, norm_w, norm_ld, eps, gate_kind, \
                                                        static_cast<T_*>(out), ldo, heads, V)
   if (is_f32) {
     if (vec) DMOE_GATE_NORM(float, 4);

@@ -6,6 +6,7 @@
 namespace dmoe {
 
 constexpr int kMaxTaps = 8;
+enum { kPlain = 0, kDelta = 1, kBonus = 2 };      // MODE of the kernels: how a token writes and where it reads, see recurrent.cu
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -26,9 +27,13 @@ __device__ __forceinline__ float log1p_unit(float e) {
   return 2.f * (s + s * q * p);
 }
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1p_unit(expf(-fabsf(x))); }
-// log of the decay of one key channel: kind 0: log sigmoid(z) * scale, kind 1: -scale * softplus(z)
+// log of the decay of one key channel: kind 0: log sigmoid(z) * scale, kind 1: -scale * softplus(z), kind 2: -exp(z)
 __device__ __forceinline__ float log_decay(int kind, float z, float scale) {
+  if (kind == 2) return -expf(z);
   return kind == 0 ? -softplus(-z) * scale : -scale * softplus(z);
+}
+__device__ __forceinline__ float decay_scale(const DmoeRecur& a, int h) {
+  return a.decay_kind == 0 ? a.inv_tau : a.decay_kind == 1 ? expf(a.a_log[h]) : 1.f;
 }
 __device__ __forceinline__ float gate_value(int kind, float g) { return (kind == 0 ? g : 1.f) / (1.f + expf(-g)); }
 

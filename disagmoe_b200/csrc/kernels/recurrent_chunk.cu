@@ -7,6 +7,9 @@
 //   o_t = (q_t e^(b_t)) S_0 + sum_{j <= t} P_tj u_j,   P_tj = sum_d q_t k_j e^(b_t - b_j)
 //   S   = e^(b_end) S_0 + sum_j (k_j e^(b_end - b_j)) u_j^T
 //
+// With a bonus the read-out precedes the token's decay and write: b_(t-1) takes the place of b_t in o_t and P_tj, j < t, and
+// P_tt = sum_d q_t bonus k_t; the scan is that of the plain write.
+//
 // chunk_prep_kernel computes everything that does not depend on S_0, one CTA per (chunk, head): P, q e^b, k e^(b_end - b)
 // and for the delta rule T = (I + A)^-1, W = -T (beta k e^b), U0 = T (beta v), so that u = U0 + W S_0.
 // chunk_scan_kernel then walks the chunks of a segment in order, one CTA per (segment, head, value tile), with the state in
@@ -138,25 +141,27 @@ __device__ __forceinline__ void invert_unit_lower(const float* A, float* T, floa
   }
 }
 
-template <int DP, bool DELTA>
+template <int DP, int MODE>
 struct PrepSmem {
+  static constexpr bool DELTA = MODE == kDelta;
   static constexpr int kKs = DP + 8;
   static constexpr int kKn = 2 * kChunk * kKs * 2, kTX = DELTA ? 4 * kChunk * kPs * 2 : 0;
   static constexpr int kRegion = kKn > kTX ? kKn : kTX;
   static constexpr int kBytes = 4 * kChunk * DP + 3 * 4 * kChunk + kRegion + (DELTA ? 2 * 4 * kChunk * (kChunk + 1) : 0) + 16;
 };
 
-template <int DP, bool DELTA>
+template <int DP, int MODE>
 __global__ void __launch_bounds__(kChunkThreads, 2)
 chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* __restrict__ ws, long long ws_stride, int h0) {
   using L = ChunkWs<DP>;
-  using SM = PrepSmem<DP, DELTA>;
+  using SM = PrepSmem<DP, MODE>;
+  constexpr bool DELTA = MODE == kDelta, BONUS = MODE == kBonus;
   constexpr int PL = DP / 32, KS = DP / 16, MT = DP / 16, LDA = kChunk + 1, ROWS = kChunk / 8;
   extern __shared__ __align__(16) uint8_t s_raw[];
   float* s_b = reinterpret_cast<float*>(s_raw);                 // [64][DP] running log2 decay
   float* s_fq = s_b + kChunk * DP;                              // [64] factors of the raw q and k rows
   float* s_fk = s_fq + kChunk;
-  float* s_beta = s_fk + kChunk;
+  float* s_beta = s_fk + kChunk;                                // delta: write strengths; bonus: P_tt
   uint8_t* region = reinterpret_cast<uint8_t*>(s_beta + kChunk);
   __nv_bfloat16* s_kh = reinterpret_cast<__nv_bfloat16*>(region);          // scaled k rows, hi then lo plane
   __nv_bfloat16* s_kl = s_kh + kChunk * SM::kKs;
@@ -185,7 +190,7 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   // ---- log2 decays and their running sums; a thread keeps one channel
   {
     constexpr int NG = kChunkThreads / DP, LEN = kChunk / NG;
-    const float scale = a.decay_kind == 0 ? a.inv_tau : expf(a.a_log[h]);
+    const float scale = decay_scale(a, h);
     const int d = tid % DP, gi = tid / DP;
     const float bias = d < D ? a.z_bias[h * D + d] : 0.f;
     const float* zp = a.z + row0 * a.ldz + h * D + d;
@@ -218,9 +223,11 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
       for (int t = gi * LEN; t < (gi + 1) * LEN; ++t) s_b[t * DP + d] += before;
     }
   }
-  // ---- factors of the rows: scale and unit norms
-  if (DELTA) {
-    float q[ROWS][PL];
+  // ---- factors of the rows: scale and unit norms; with a bonus the diagonal of P
+  if (DELTA || BONUS) {
+    float q[ROWS][PL], bonus[PL];
+#pragma unroll
+    for (int e = 0; e < PL; ++e) bonus[e] = BONUS && d0 < D ? a.bonus[h * D + d0 + e] : 0.f;
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
 #pragma unroll
@@ -230,6 +237,13 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
       float qq = 0.f, kk = 0.f;
+      if (BONUS) {
+#pragma unroll
+        for (int e = 0; e < PL; ++e) qq += q[i][e] * (k[i][e] * bonus[e]);
+        qq = warp_sum(qq);
+        if (lane == 0) { s_fq[t0 + i] = a.qscale; s_fk[t0 + i] = 1.f; s_beta[t0 + i] = qq * a.qscale; }
+        continue;
+      }
 #pragma unroll
       for (int e = 0; e < PL; ++e) { qq += q[i][e] * q[i][e]; kk += k[i][e] * k[i][e]; }
       const float fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f), fq = a.qscale / sqrtf(warp_sum(qq) + 1e-6f);
@@ -245,7 +259,7 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   bool wide = false;
   if (tid < DP) {
     const float m = s_b[kMid * DP + tid];
-    wide = s_b[tid] - m > kMaxShift || m - s_b[(kChunk - 1) * DP + tid] > kMaxShift;
+    wide = (BONUS ? 0.f : s_b[tid]) - m > kMaxShift || m - s_b[(kChunk - 1) * DP + tid] > kMaxShift;
     reinterpret_cast<float*>(w + L::kDec)[tid] = exp2f(s_b[(kChunk - 1) * DP + tid]);
   }
   const bool slow = __syncthreads_or(wide);
@@ -319,7 +333,9 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
             float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[kk][j]));
             x.x *= f;
             x.y *= f;
-            const float2 b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
+            float2 b = make_float2(0.f, 0.f);
+            if (second || !BONUS) b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
+            else if (r > 0) b = *reinterpret_cast<const float2*>(s_b + (r - 1) * DP + c);
             const float2 m = *reinterpret_cast<const float2*>(s_b + kMid * DP + c);
             split2(x.x * exp2f(b.x - m.x), x.y * exp2f(b.y - m.y), ah[j], al[j]);
             if (!second) split2(x.x * exp2f(b.x), x.y * exp2f(b.y), zh[j], zl[j]);
@@ -345,11 +361,17 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
       if (!slow) {
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) {
-          const int c = nt * 8 + 2 * tq, edge = second ? -1 : 0;        // A is strictly below the diagonal
+          const int c = nt * 8 + 2 * tq, edge = second || BONUS ? -1 : 0;        // A is strictly below the diagonal
           if (c > r0 + edge) acc[nt][0] = 0.f;
           if (c + 1 > r0 + edge) acc[nt][1] = 0.f;
           if (c > r1 + edge) acc[nt][2] = 0.f;
           if (c + 1 > r1 + edge) acc[nt][3] = 0.f;
+          if (BONUS) {
+            if (c == r0) acc[nt][0] = s_beta[r0];
+            if (c + 1 == r0) acc[nt][1] = s_beta[r0];
+            if (c == r1) acc[nt][2] = s_beta[r1];
+            if (c + 1 == r1) acc[nt][3] = s_beta[r1];
+          }
           if (DELTA && second) {
             s_A[r0 * LDA + c] = acc[nt][0] * s_beta[r0];
             s_A[r0 * LDA + c + 1] = acc[nt][1] * s_beta[r0];
@@ -369,15 +391,16 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
     for (int i = tid; i < kChunk * kChunk; i += kChunkThreads) {
       const int t = i / kChunk, j = i % kChunk;
       float p = 0.f, kk = 0.f;
-      if (j <= t && t < n) {
+      if ((BONUS ? j < t : j <= t) && t < n) {
+        const int tr = BONUS ? t - 1 : t;              // place of the read-out
         for (int d = 0; d < D; ++d) {
-          const float e = __bfloat162float(kp[j * a.ldk + d]) * s_fk[j] * exp2f(s_b[t * DP + d] - s_b[j * DP + d]);
+          const float e = __bfloat162float(kp[j * a.ldk + d]) * s_fk[j] * exp2f(s_b[tr * DP + d] - s_b[j * DP + d]);
           p += __bfloat162float(qp[t * a.ldq + d]) * e;
           if (DELTA) kk += __bfloat162float(kp[t * a.ldk + d]) * e;
         }
       }
       // place of element (t, j) in the fragment tiles
-      const float pv = p * s_fq[t];
+      const float pv = BONUS && j == t ? s_beta[t] : p * s_fq[t];
       const int r = t % 16, c = j % 16;
       __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(w + L::kP + (t / 16 * 4 + j / 16) * 2 * kFrag) +
                          ((r % 8) * 4 + c % 8 / 2) * 8 + ((r >= 8) + 2 * (c >= 8)) * 2 + c % 2;
@@ -701,17 +724,17 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
   }
 }
 
-template <int DP, bool DELTA>
+template <int DP, int MODE>
 static int launch_prep(const DmoeRecur& a, const void* chunks, int n_chunks, uint8_t* ws, long long stride, int h0, int hn,
                        cudaStream_t stream) {
-  using SM = PrepSmem<DP, DELTA>;
+  using SM = PrepSmem<DP, MODE>;
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(chunk_prep_kernel<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return static_cast<int>(cudaFuncSetAttribute(chunk_prep_kernel<DP, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  SM::kBytes));
   });
   if (rc != 0) return rc;
-  chunk_prep_kernel<DP, DELTA><<<dim3(n_chunks, hn), kChunkThreads, SM::kBytes, stream>>>(
+  chunk_prep_kernel<DP, MODE><<<dim3(n_chunks, hn), kChunkThreads, SM::kBytes, stream>>>(
       a, static_cast<const int4*>(chunks), ws, stride, h0);
   return static_cast<int>(cudaGetLastError());
 }
@@ -723,8 +746,9 @@ static int launch_scan(const DmoeRecur& a, const uint8_t* ws, long long stride, 
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int DP, bool DELTA>
+template <int DP, int MODE>
 static int run_chunks(const DmoeRecur& a, const void* chunks, int n_chunks, uint8_t* ws, long long ws_bytes, cudaStream_t stream) {
+  constexpr bool DELTA = MODE == kDelta;
   const long long stride = (ChunkWs<DP>::bytes(DELTA, a.vdim) + 127) / 128 * 128;
   long long per = ws_bytes / (stride * n_chunks);               // heads whose chunks fit the workspace at a time
   if (per < 1) return -15;
@@ -734,7 +758,7 @@ static int run_chunks(const DmoeRecur& a, const void* chunks, int n_chunks, uint
   const bool narrow = a.vdim <= 16 || wide < device_num_sms();
   for (int h0 = 0; h0 < a.heads; h0 += static_cast<int>(per)) {
     const int hn = a.heads - h0 < per ? a.heads - h0 : static_cast<int>(per);
-    int rc = launch_prep<DP, DELTA>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
+    int rc = launch_prep<DP, MODE>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
     if (rc != 0) return rc;
     rc = narrow ? launch_scan<DP, 16, DELTA>(a, ws, stride, h0, hn, stream)
                 : launch_scan<DP, 32, DELTA>(a, ws, stride, h0, hn, stream);
@@ -772,17 +796,17 @@ extern "C" int dmoe_recur_chunks(const DmoeRecur* a, const void* chunks, int n_c
     return -10;
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   if (a->ldq % 8 != 0 || a->ldk % 8 != 0 || a->ldv % 8 != 0 || a->ldraw % 2 != 0 || !al(a->q) || !al(a->k) || !al(a->v) ||
-      !al(ws) || !al(a->state) || !al(a->raw) || (a->decay_kind != 0 && a->a_log == nullptr) || a->z_bias == nullptr)
+      !al(ws) || !al(a->state) || !al(a->raw) || (a->decay_kind == 1 && a->a_log == nullptr) || a->z_bias == nullptr || (a->bonus != nullptr && a->delta))
     return -11;
   if (n_chunks == 0 || a->n_segs == 0) return 0;
   uint8_t* w = static_cast<uint8_t*>(ws);
   const int dp = padded_dim(a->dim);
-  if (a->delta) {
-    if (dp == 32) return run_chunks<32, true>(*a, chunks, n_chunks, w, ws_bytes, stream);
-    if (dp == 64) return run_chunks<64, true>(*a, chunks, n_chunks, w, ws_bytes, stream);
-    return run_chunks<128, true>(*a, chunks, n_chunks, w, ws_bytes, stream);
-  }
-  if (dp == 32) return run_chunks<32, false>(*a, chunks, n_chunks, w, ws_bytes, stream);
-  if (dp == 64) return run_chunks<64, false>(*a, chunks, n_chunks, w, ws_bytes, stream);
-  return run_chunks<128, false>(*a, chunks, n_chunks, w, ws_bytes, stream);
+#define DMOE_CHUNKS(MODE_)                                                                     \
+  if (dp == 32) return run_chunks<32, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream);       \
+  if (dp == 64) return run_chunks<64, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream);       \
+  return run_chunks<128, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream)
+  if (a->bonus != nullptr) { DMOE_CHUNKS(kBonus); }
+  if (a->delta) { DMOE_CHUNKS(kDelta); }
+  DMOE_CHUNKS(kPlain);
+#undef DMOE_CHUNKS
 }

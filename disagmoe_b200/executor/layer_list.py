@@ -3,11 +3,13 @@
     sandwich  embed * scale -> per layer [ norm -> mixer -> norm + add (-> norm -> gated feed-forward -> norm + add) ]
     parallel  embed * scale -> per layer [ norm (+ router) -> mixer, feed-forward or experts on the same rows -> add both ]
               -> norm -> head -> argmax
+    prenorm   embed * scale -> per layer [ norm (+ token shift) -> mixer -> add (-> norm + router -> experts -> add) ]
+              -> norm -> head -> argmax
 
 The residual stream is fp32; what stands between two sublayers (norm after, residual add, norm before, and the router of a
 layer with experts) is one launch. Two kinds of per-sequence memory: pages for the attention layers that have keys and values
 of their own (layers that read another layer's have none; latent attention keeps one latent row per token), and for recurrent
-layers one state slot per sequence, numbered like its row of the block table, so the block manager's row allocation is the
+layers one state slot per sequence (layers that share weights have caches and states of their own), numbered like its row of the block table, so the block manager's row allocation is the
 slot allocation. As in the MoE executor, a decode iteration is one chain of launches captured per batch-size bucket, prompts
 run eagerly, and CPU tensors run the PyTorch restatements.
 """
@@ -18,7 +20,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec, LatentAttentionSpec
+from ..config import AttentionSpec, LatentAttentionSpec, WkvSpec
 from ..models import weights as W
 from ..models.mixers import (GatedFeedForward, LatentTables, RoutedBuffers, RoutedFeedForward, ScatterRows, StepMeta,
                              make_mixer)
@@ -38,6 +40,7 @@ class LayerListBuffers(TokenBuffers):
         for size in {m.lay.heads * m.lay.vdimp for m in mixers if hasattr(m, "lay")}:
             self.latent_out[size] = ScatterRows(cap, size, device, dtype)
         self.latent: Dict[Tuple, LatentTables] = {}          # of a prefill step
+        self.block_offs: Optional[torch.Tensor] = None       # likewise
         self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=device)
         self.segments: Optional[SegmentTables] = None        # None: decode step, every row its own segment
         self.prefill_tiles: Dict[int, Tuple[torch.Tensor, int]] = {}    # tokens per tile -> (table, tiles)
@@ -53,23 +56,27 @@ class LayerListExecutor(StepExecutor):
             raise ValueError(f"short convolutions longer than {MAX_TAPS} taps are not supported")
         # without a checkpoint: seeded random weights, created on the device tensor by tensor
         sd = state_dict if state_dict is not None else W.init_state_dict(cfg, dev, dt)
-        # sandwich norms are stored as offsets from one
+        # norms are stored as offsets from one, but for those of parallel blocks
         plus = 0.0 if cfg.block == "parallel" else 1.0
         norm = lambda n: (plus + sd[n].to(device=dev, dtype=torch.float32)).contiguous()
         self.embed_w = sd["embed"].to(device=dev, dtype=dt).contiguous()
         self.head_w = sd["head"].to(device=dev, dtype=dt).contiguous()
         self.final_norm = norm("final.norm")
-        self.mixers, self.ffs, self.norms = [], [], []
+        mixers, ffs, norms = {}, {}, {}
         for i, layer in enumerate(cfg.layers):
-            m = make_mixer(cfg, i, dev, dt)
-            m.load_weights(sd)
-            self.mixers.append(m)
+            if layer.weights_of is not None:
+                continue
+            mixers[i] = make_mixer(cfg, i, dev, dt)
+            mixers[i].load_weights(sd)
             p = f"l{i}.mlp."
-            self.ffs.append(RoutedFeedForward(sd, p, layer.routed, dev, dt) if layer.routed else
-                            GatedFeedForward(sd, p, layer.ff, layer.act, dev, dt) if layer.ff else None)
-            self.norms.append({n: norm(f"l{i}.{n}") for n in W.layer_norm_names(cfg, i)})
+            ffs[i] = RoutedFeedForward(sd, p, layer.routed, dev, dt) if layer.routed else \
+                GatedFeedForward(sd, p, layer.ff, layer.act, dev, dt) if layer.ff else None
+            norms[i] = {n: norm(f"l{i}.{n}") for n in W.layer_norm_names(cfg, i)}
+        owners = [cfg.weight_layer(i) for i in range(cfg.num_layers)]
+        self.mixers, self.ffs, self.norms = ([x[j] for j in owners] for x in (mixers, ffs, norms))
+        self.blocks_of_rows = 4 if any(isinstance(l.mixer, WkvSpec) for l in cfg.layers) else 0
         self.latent_specs = {LatentTables.key(l.mixer): l.mixer for l in cfg.layers if isinstance(l.mixer, LatentAttentionSpec)}
-        self.decode_tables: Dict[int, Dict[Tuple, LatentTables]] = {}
+        self.decode_tables: Dict[int, Tuple[Dict[Tuple, LatentTables], Optional[torch.Tensor]]] = {}
 
     # ---- cache and state ------------------------------------------------------------------------------------------
     def _owns_kv(self, i: int) -> bool:
@@ -120,6 +127,7 @@ class LayerListExecutor(StepExecutor):
         buf.prefill_tiles, buf.ctx_len_decode, buf.n_untiled = {}, None, T
         buf.latent = {k: LatentTables.prefill(m, bt_row, positions, self.device, self.dtype)
                       for k, m in self.latent_specs.items()}
+        buf.block_offs = self._block_offs(T)
         for mixer in self.mixers:
             m = mixer.spec
             if not isinstance(m, AttentionSpec) or not mixer.tiled():
@@ -135,12 +143,17 @@ class LayerListExecutor(StepExecutor):
                 buf.ctx_len_decode, buf.n_untiled = cd.to(self.device), int((~covered).sum())
 
     def _end_prefill(self, buf: LayerListBuffers) -> None:
-        buf.segments, buf.prefill_tiles, buf.ctx_len_decode, buf.latent = None, {}, None, {}
+        buf.segments, buf.prefill_tiles, buf.ctx_len_decode, buf.latent, buf.block_offs = None, {}, None, {}, None
 
-    def _decode_tables(self, T: int) -> Dict[Tuple, LatentTables]:
-        """Made once per batch size: graphs replay on them."""
+    def _block_offs(self, T: int) -> Optional[torch.Tensor]:
+        n = self.blocks_of_rows
+        return (torch.arange(n + 1, dtype=torch.int32) * T).to(self.device) if n else None
+
+    def _decode_tables(self, T: int) -> Tuple[Dict[Tuple, LatentTables], Optional[torch.Tensor]]:
+        """Latent tables and block offsets, made once per batch size: graphs replay on them."""
         if T not in self.decode_tables:
-            self.decode_tables[T] = {k: LatentTables.decode(m, T, self.device) for k, m in self.latent_specs.items()}
+            self.decode_tables[T] = ({k: LatentTables.decode(m, T, self.device) for k, m in self.latent_specs.items()},
+                                     self._block_offs(T))
         return self.decode_tables[T]
 
     def _forward(self, buf: LayerListBuffers, T: int, max_ctx: int, want_logits: bool):
@@ -148,14 +161,15 @@ class LayerListExecutor(StepExecutor):
         pos, slots, rows = buf.positions[:T], buf.slots[:T], buf.bt_row[:T]
         segs = buf.segments if buf.segments is not None else decode_segments(pos, rows, slots)
         prompts = buf.segments is not None
+        latent, block_offs = (buf.latent, buf.block_offs) if prompts else self._decode_tables(T)
         meta = StepMeta(pos, slots, self.block_tables, rows, buf.ctx_len[:T], max_ctx=max_ctx,
                         num_decode_tokens=buf.n_untiled if prompts else T,
                         prefill_tiles=buf.prefill_tiles if prompts else None,
                         ctx_len_decode=buf.ctx_len_decode, segments=segs,
-                        latent=buf.latent if prompts else self._decode_tables(T), latent_out=buf.latent_out)
+                        latent=latent, latent_out=buf.latent_out, block_offs=block_offs)
         resid = buf.resid[:T]
         F.embed_f32(buf.ids[:T], self.embed_w, cfg.embed_scale, resid)
-        h = (self._parallel_blocks if cfg.block == "parallel" else self._sandwich_blocks)(buf, resid, meta)
+        h = getattr(self, f"_{cfg.block}_blocks")(buf, resid, meta)
         n_out = h.shape[0]
         logits = gemm.linear(h, self.head_w, out=buf.logits[:n_out] if n_out <= buf.logits.shape[0] else None,
                              out_dtype=torch.float32)
@@ -189,3 +203,18 @@ class LayerListExecutor(StepExecutor):
             y = mixer(h, self._memory(i), meta)
             z = ff(h, ids, weights, rb) if r else ff(h) if ff is not None else None
         return F.sum_norm(resid, y, z, self.final_norm, eps, dt, True, rows=buf.out_rows)[0]
+
+    def _prenorm_blocks(self, buf: LayerListBuffers, resid: torch.Tensor, meta: StepMeta) -> torch.Tensor:
+        cfg, eps, dt = self.cfg, self.cfg.rms_norm_eps, self.dtype
+        y = z = None                    # what the last sublayer left to be added: rows, or rows per chosen expert
+        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
+            memory = self._memory(i)
+            h, _, _ = F.sum_norm(resid, y, z, n["norm1"], eps, dt, False, mult=cfg.residual_mult, shift=mixer.shift(memory, meta))
+            y, z = mixer(h, memory, meta), None
+            r = cfg.layers[i].routed
+            rb = buf.routed[r.experts, r.top] if r else None
+            if ff is not None:
+                h, ids, weights = F.sum_norm(resid, y, None, n["norm2"], eps, dt, False, mult=cfg.residual_mult,
+                                             router=ff.router(rb) if r else None)
+                y, z = (None, ff(h, ids, weights, rb)) if r else (ff(h), None)
+        return F.sum_norm(resid, y, z, self.final_norm, eps, dt, False, rows=buf.out_rows, mult=cfg.residual_mult)[0]

@@ -13,23 +13,25 @@ from typing import Dict, List, Optional, Tuple
 import numpy as np
 import torch
 
-from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig
+from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, WkvSpec
 from ..ops import functional as F
 from ..ops import gemm
 from ..ops.recurrent import Recurrence, RecurrentState, SegmentTables, recurrent_attention
 from .attention import AttnMeta
 from .experts import ExpertStack
-from .weights import StateDict
+from .weights import WKV_MIXES, StateDict
 
 
 @dataclass
 class StepMeta(AttnMeta):
     """Attention metadata of a step plus the segments the recurrent layers run over, the row tables of the latent attention
-    layers and the values that value-mixing layers mix in (set by the first of them)."""
+    layers, the values that value-mixing layers mix in (set by the first of them) and the row offsets of grouped GEMMs over
+    equal blocks of a step's rows."""
     segments: Optional[SegmentTables] = None
     latent: Dict[Tuple, "LatentTables"] = field(default_factory=dict)
     latent_out: Dict[int, "ScatterRows"] = field(default_factory=dict)      # by row size
     v_first: Optional[torch.Tensor] = None
+    block_offs: Optional[torch.Tensor] = None                                 # int32: 0, T, 2T, ...
 
 
 class ScatterRows:
@@ -57,7 +59,7 @@ class LatentTables:
 
     @staticmethod
     def key(m: LatentAttentionSpec) -> Tuple:
-        return m.heads, m.window, latent_layout(m).min_run()
+        return m.heads, m.window, latent_layout(m).min_run(), m.gate      # gated layers write the weights of the records
 
     @staticmethod
     def _per_head(rows: torch.Tensor, heads: int, device):
@@ -161,6 +163,10 @@ class Mixer(torch.nn.Module):
         self.device, self.dtype = torch.device(device), dtype
         self.eps = cfg.rms_norm_eps
 
+    def shift(self, memory, meta: StepMeta) -> Optional[F.TokenShift]:
+        """The token shift that the mixer's input goes through (forward then takes its mixes), if it has one."""
+        return None
+
     def _get(self, sd: StateDict, name: str, dtype=None) -> torch.Tensor:
         return sd[f"l{self.layer_id}.mix.{name}"].to(device=self.device, dtype=dtype or self.dtype).contiguous()
 
@@ -194,9 +200,36 @@ class RecurrentMixer(Mixer):
         return gemm.linear(o, self.o)
 
 
+class WkvMixer(Mixer):
+    """RWKV-style time mixing. The maps of the mixes to r, k, v and the gate run as one grouped GEMM, the map to the decays as
+    two small ones with tanh in the epilogue of the first."""
+
+    def load_weights(self, sd: StateDict) -> None:
+        m = self.spec
+        f32 = lambda n: self._get(sd, n, torch.float32)
+        self.mu = torch.stack([f32("mu." + n) for n in WKV_MIXES]).contiguous()
+        self.rkvg = torch.stack([self._get(sd, n) for n in WKV_MIXES[:4]]).contiguous()
+        rank = _pad8(m.rank)
+        self.w1 = _pad_rows(self._get(sd, "w1"), rank).contiguous()
+        self.w2 = _pad_cols(self._get(sd, "w2"), rank).contiguous()
+        self.o = self._get(sd, "o")
+        self.recur = Recurrence(m.heads, m.heads, m.dim, m.dim, False, f32("w0"), f32("norm"), self.eps, exp_decay=True,
+                                bonus=f32("u"), qscale=1.0, shift_width=self.cfg.hidden_size)
+
+    def shift(self, memory: RecurrentState, meta: StepMeta) -> F.TokenShift:
+        return F.TokenShift(self.mu, memory.last, meta.segments)
+
+    def forward(self, mixes: torch.Tensor, state: RecurrentState, meta: StepMeta) -> torch.Tensor:
+        T, n = mixes.shape[1], self.rkvg.shape[1]
+        bn = gemm.pick_even_bn(T, n, 4) if mixes.is_cuda else 0
+        r, k, v, gate = gemm.grouped_linear(mixes[:4].reshape(4 * T, -1), self.rkvg, meta.block_offs, bn=bn).view(4, T, n)
+        z = gemm.linear(gemm.linear(mixes[4], self.w1, tanh=True), self.w2, out_dtype=torch.float32)
+        return gemm.linear(recurrent_attention(self.recur, r, k, v, gate, None, z, state, meta.segments), self.o)
+
+
 class SoftmaxAttention(Mixer):
     """Softmax attention over the layer's own paged cache or, with ``kv_from``, an earlier layer's: optional per-head query /
-    key norm, rotation, window, score soft cap, sink and value mixing. Head sizes without a tensor-core kernel are kept
+    key norm, rotation, window or chunks, score soft cap, sink, value mixing, values tied to the keys. Head sizes without a tensor-core kernel are kept
     padded with zeros to those of the next one (not where heads are normed)."""
 
     def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
@@ -217,7 +250,8 @@ class SoftmaxAttention(Mixer):
         m = self.spec
         own = m.kv_from is None
         # contiguous head blocks [q | k | v]: the norm + rotation kernel walks them as one row of heads
-        parts = [("q", m.heads, m.dim, self.dk)] + ([("k", m.kv_heads, m.dim, self.dk), ("v", m.kv_heads, m.vdim, self.dv)] if own else [])
+        parts = [("q", m.heads, m.dim, self.dk)] + ([("k", m.kv_heads, m.dim, self.dk)] if own else []) + \
+            ([("v", m.kv_heads, m.vdim, self.dv)] if own and not m.tied_values else [])
         self.proj = FusedProjection([(n, _pad_heads(self._get(sd, n), h, [(d, p)])) for n, h, d, p in parts], pad=False)
         self.o = _pad_head_cols(self._get(sd, "o"), m.heads, m.vdim, self.dv).contiguous()
         self.q_norm = self._get(sd, "q.norm", torch.float32) if m.qk_norm else None
@@ -233,17 +267,18 @@ class SoftmaxAttention(Mixer):
         qkv = self.proj(h)
         first = meta.v_first if self.v_lambda is not None else None
         F.qk_norm_rope(qkv, meta.positions, meta.slots, kc, vc, m.heads, n_kv, self.dk, self.dv, self.rope, self.q_norm,
-                       self.k_norm, self.eps, m.rot is not None and m.rot.interleaved, first, self.v_lambda or 0.0)
+                       self.k_norm, self.eps, m.rot is not None and m.rot.interleaved, first, self.v_lambda or 0.0,
+                       m.tied_values)
         if m.v_mix and self.v_lambda is None:
             meta.v_first = qkv[:, (m.heads + n_kv) * self.dk:].view(-1, n_kv, self.dv)
         q = qkv[:, :m.heads * self.dk]
-        opt = dict(scale=m.scale, window=m.window, softcap=m.softcap, fp32_weights=True, sink=self.sink)
+        opt = dict(scale=m.scale, window=m.window, chunk=m.chunk, softcap=m.softcap, fp32_weights=True, sink=self.sink)
         cuda = self.tiled()
         tiles, n_tiles = meta.prefill_tiles.get(F.prefill_tile_tokens(m.heads, m.kv_heads), (None, 0)) \
             if cuda and meta.prefill_tiles else (None, 0)
         splits = 1
         if cuda:
-            reach = min(meta.max_ctx, m.window or meta.max_ctx)
+            reach = min(meta.max_ctx, m.window or meta.max_ctx, m.chunk or meta.max_ctx)
             splits = F.pick_attn_splits(q.shape[0], m.kv_heads, reach, kc.shape[1])
         attn = None
         if n_tiles == 0 or meta.num_decode_tokens > 0:
@@ -274,7 +309,7 @@ class LatentAttention(Mixer):
         H = m.heads
         q = _pad_heads(self._get(sd, "q"), H, [(m.dim, lay.dimp), (m.rot_dim, lay.rotp)])
         dkv = _pad_heads(self._get(sd, "dkv"), 1, [(m.kv_rank, lay.rankp), (m.rot_dim, lay.rotp)])
-        self.proj = FusedProjection([("q", q), ("dkv", dkv)])
+        self.proj = FusedProjection([("q", q), ("dkv", dkv)] + ([("g", self._get(sd, "g"))] if m.gate else []))
         uk = _pad_cols(_pad_heads(self._get(sd, "uk"), H, [(m.dim, lay.dimp)]), lay.rankp).view(H, lay.dimp, lay.rankp)
         uv = _pad_cols(_pad_heads(self._get(sd, "uv"), H, [(m.vdim, lay.vdimp)]), lay.rankp).view(H, lay.vdimp, lay.rankp)
         self.absorb, self.expand_v = uk.transpose(1, 2).contiguous(), uv.contiguous()
@@ -289,8 +324,9 @@ class LatentAttention(Mixer):
         m, lay, cache = self.spec, self.lay, kv[0]
         T, t = h.shape[0], meta.latent[LatentTables.key(m)]
         y = self.proj(h)
+        gate = self.proj.block(y, "g") if m.gate else None
         xq, qa = F.latent_prep(y, meta.positions, meta.slots, cache, lay, self.rope, self.norm, self.eps, t.loose, t.n_loose,
-                               m.rot is not None and m.rot.interleaved)
+                               m.rot is not None and m.rot.interleaved, gate, t.recs)
         out = meta.latent_out[m.heads * lay.vdimp]
         attn = out.rows[:T]
         if t.n_loose:
@@ -304,7 +340,7 @@ class LatentAttention(Mixer):
         if t.n_tiles:
             lat = F.latent_gather(cache, meta.block_tables, t.keys, t.n_keys)
             kvx = gemm.linear(lat[:, :lay.rankp], self.expand)
-            F.latent_prefill(y, kvx, lat, t.tiles, t.base, t.n_tiles, lay, m.scale, m.window, self.sink, attn)
+            F.latent_prefill(y, kvx, lat, t.tiles, t.base, t.n_tiles, lay, m.scale, m.window, self.sink, attn, gate)
         return gemm.linear(attn, self.o)
 
 
@@ -353,9 +389,12 @@ class RoutedFeedForward:
         self.stack = ExpertStack(spec.experts, w2.shape[1], w2.shape[2], device, dtype, spec.act)
         self.stack.set_weights(w13, w2)
         self.router_w = sd[prefix + "router"].to(device=device, dtype=dtype).contiguous()
+        self.correction = sd[prefix + "correction"].to(device=device, dtype=torch.float32).contiguous() if spec.correction else None
 
     def router(self, buf: RoutedBuffers) -> F.Router:
-        return F.Router(self.router_w, self.spec.top, self.spec.renormalize, buf.dispatch.counts)
+        s = self.spec
+        return F.Router(self.router_w, s.top, s.renormalize, buf.dispatch.counts, s.scoring == "sigmoid", self.correction,
+                        s.groups, s.keep, s.scale)
 
     def __call__(self, h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, buf: RoutedBuffers) -> torch.Tensor:
         """Output rows [T, top, width], to be summed over the choices."""
@@ -367,7 +406,7 @@ class RoutedFeedForward:
 
 
 MIXERS = {AttentionSpec: SoftmaxAttention, LatentAttentionSpec: LatentAttention, GatedLinearSpec: RecurrentMixer,
-          ChannelDeltaSpec: RecurrentMixer}
+          ChannelDeltaSpec: RecurrentMixer, WkvSpec: WkvMixer}
 
 
 def make_mixer(cfg: LayerListConfig, layer_id: int, device, dtype) -> Mixer:

@@ -14,7 +14,7 @@ from typing import Any, Callable, Dict, Optional, Tuple
 import torch
 
 from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, LayerSpec,
-                      ModelConfig, PRESETS, RotarySpec, RoutedSpec, get_preset)
+                      ModelConfig, PRESETS, RotarySpec, RoutedSpec, WkvSpec, get_preset)
 from . import weights as W
 
 
@@ -84,6 +84,45 @@ def supinex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, .
                                 architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
 
 
+# ---- Vufinex: RWKV-style time mixing, gated latent attention and chunked attention in any order, grouped sigmoid routers; layers
+# may use the weights of others ---------------------------------------------------------------------------------------------
+def _vufinex_layer(i: int, layer: dict, j: int, shapes: Dict[str, Tuple[int, ...]]) -> LayerSpec:
+    """``j``: the layer whose tensors layer i uses."""
+    m, kind, mlp = layer["mixer"], layer["type"], layer.get("mlp")
+    if kind == "wkv":
+        mixer = WkvSpec(m["heads"], m["dim"], shapes.get(f"l{j}.mix.w1", (16,))[0])
+    elif kind == "latent_attention":
+        mixer = LatentAttentionSpec(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], float(m["scale"]),
+                                    _rotary(m.get("rot"), interleaved=True), gate=True)
+    elif kind == "attention":
+        mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), _rotary(m.get("rot")),
+                              qk_norm=False, chunk=_window(m), tied_values=True)
+    else:
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    routed = None
+    if mlp is not None:
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        r = mlp["router"]
+        g = r.get("groups") or {"count": 1, "keep": 1}
+        routed = RoutedSpec(r["experts"], r["top"], mlp["expert"]["ff"], renormalize=True, scoring="sigmoid", correction=True,
+                            groups=g["count"], keep=g["keep"], scale=float(r["scale"]))
+    return LayerSpec(mixer, routed=routed, weights_of=layer.get("weights_of"))
+
+
+def vufinex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, ...]], **kw) -> LayerListConfig:
+    def owner(i: int) -> int:
+        for _ in raw["layers"]:
+            if raw["layers"][i].get("weights_of") is None:
+                break
+            i = raw["layers"][i]["weights_of"]
+        return i
+    layers = [_vufinex_layer(i, l, owner(i), shapes) for i, l in enumerate(raw["layers"])]
+    return LayerListConfig.make(raw["width"], raw["vocab"], layers, rms_norm_eps=float(raw["norm"]["eps"]), block="prenorm",
+                                embed_scale=float(raw["embedding"]["scale"]), residual_mult=float(raw["residual_mult"]),
+                                architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
+
+
 @dataclass(frozen=True)
 class Architecture:
     config_from_json: Callable[..., ModelConfig]
@@ -92,6 +131,7 @@ class Architecture:
 ARCHITECTURES: Dict[str, Architecture] = {
     "Rurunex": Architecture(rurunex_config_from_json),
     "Supinex": Architecture(supinex_config_from_json),
+    "Vufinex": Architecture(vufinex_config_from_json),
 }
 
 

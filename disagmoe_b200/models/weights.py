@@ -30,25 +30,31 @@ from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, ModelConfig
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, ModelConfig,
+                      WkvSpec)
 
 StateDict = Dict[str, torch.Tensor]
+WKV_MIXES = ("r", "k", "v", "g", "w")       # the mixed inputs of RWKV-style time mixing, in the order the mixer keeps them
 
 
 def layer_norm_names(cfg: LayerListConfig, i: int) -> Tuple[str, ...]:
     """The residual-stream norms of layer i."""
     if cfg.block == "parallel":
         return ("norm1",)
+    if cfg.block == "prenorm":
+        return ("norm1", "norm2") if cfg.layers[i].ff or cfg.layers[i].routed else ("norm1",)
     return ("norm1", "norm1b") + (("norm2", "norm2b") if cfg.layers[i].ff else ())
 
 
 def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
     """Names and shapes of a layer-list checkpoint: ``l<i>.norm1 / norm1b / norm2 / norm2b`` around the sublayers (parallel
-    blocks have ``norm1`` alone), ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward, with ``e<j>.`` in front of an
-    expert's tensors; linear weights [out, in]."""
+    blocks have ``norm1`` alone, pre-norm blocks ``norm1`` and ``norm2``), ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward, with ``e<j>.`` in front of an
+    expert's tensors; linear weights [out, in]. A layer that uses another one's weights has none."""
     H = cfg.hidden_size
     out: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab_size, H)}
     for i, layer in enumerate(cfg.layers):
+        if layer.weights_of is not None:
+            continue
         p, m = f"l{i}.", layer.mixer
         x = p + "mix."
         for n in layer_norm_names(cfg, i):
@@ -68,11 +74,19 @@ def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
         elif isinstance(m, LatentAttentionSpec):
             out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.kv_rank + m.rot_dim, H),
                         x + "dkv.norm": (m.kv_rank,), x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (vs, m.kv_rank)})
+            if m.gate:
+                out[x + "g"] = (m.heads, H)
+        elif isinstance(m, WkvSpec):
+            out.update({x + "mu." + n: (H,) for n in WKV_MIXES})
+            out.update({x + n: (vs, H) for n in ("r", "k", "v", "g")})
+            out.update({x + "w1": (m.rank, H), x + "w2": (vs, m.rank), x + "w0": (vs,), x + "u": (m.heads, m.dim), x + "norm": (vs,)})
         else:
             own = m.kv_from is None
             out[x + "q"] = (m.heads * m.dim, H)
             if own:
-                out.update({x + "k": (m.kv_heads * m.dim, H), x + "v": (m.kv_heads * m.vdim, H)})
+                out[x + "k"] = (m.kv_heads * m.dim, H)
+            if own and not m.tied_values:
+                out[x + "v"] = (m.kv_heads * m.vdim, H)
             if m.qk_norm:
                 out.update({x + n + ".norm": (m.dim,) for n in (("q", "k") if own else ("q",))})
             if m.v_mix:
@@ -87,6 +101,8 @@ def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
             for e in range(layer.routed.experts):
                 out.update(gated(f"{p}mlp.e{e}.", layer.routed.ff))
             out[p + "mlp.router"] = (layer.routed.experts, H)
+            if layer.routed.correction:
+                out[p + "mlp.correction"] = (layer.routed.experts,)
     out.update({"final.norm": (H,), "head": (cfg.vocab_size, H)})
     return out
 
@@ -95,6 +111,8 @@ def _init_layer_list_tensor(cfg: LayerListConfig, name: str, shape: Tuple[int, .
     """Random values of the order a trained model has: weights of unit gain, norms near one, slow decays."""
     r = torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
     leaf = name.split(".mix.")[-1]
+    if leaf == "u":
+        return r * 0.5
     if len(shape) == 2:
         return r * (0.02 if name == "embed" else shape[1] ** -0.5)
     if leaf == "A_log":
@@ -103,11 +121,17 @@ def _init_layer_list_tensor(cfg: LayerListConfig, name: str, shape: Tuple[int, .
         return r * 0.5 - 4.0
     if leaf == "a2.b":
         return r + 2.0
+    if leaf.startswith("mu."):
+        return torch.sigmoid(r)
+    if leaf == "w0":
+        return r - 3.0
+    if leaf.endswith(".correction"):
+        return r * 0.1
     if leaf == "vmix":
         return 0.5 + 0.1 * r
     if leaf == "sink":
         return r
-    # norms of the residual stream: the sandwich block stores offsets from one
+    # norms of the residual stream: all blocks but the parallel one store offsets from one
     return 1.0 + 0.05 * r if ".mix." in name or cfg.block == "parallel" else 0.05 * r
 
 

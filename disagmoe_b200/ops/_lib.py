@@ -70,7 +70,17 @@ class DmoeRecur(ctypes.Structure):
                [(n, _ll) for n in ("ldq", "ldk", "ldv", "ldg", "ldb", "ldz", "ldo", "ldraw")] + \
                [(n, _i) for n in ("n_segs", "n_slots", "heads", "kv_heads", "dim", "vdim", "taps", "delta", "decay_kind",
                                   "gate_kind", "is_f32", "one_token")] + \
-               [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp)]
+               [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp), ("bonus", _vp), ("norm_ld", _i)]
+
+
+class DmoeRouter(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("weight", "correction", "ids", "wts", "counts")] + \
+               [(n, _i) for n in ("E", "K", "renorm", "sigmoid", "groups", "keep")] + [("wscale", _f)]
+
+
+class DmoeShift(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("mu", "last", "singles", "positions", "rows", "kv_slots")] + [("mix_stride", _ll)] + \
+               [(n, _i) for n in ("n_mix", "n_slots", "n_single")]
 
 
 def lib_path() -> str:

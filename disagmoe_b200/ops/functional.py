@@ -134,15 +134,16 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
                     out: Optional[torch.Tensor] = None, splits: int = 1, scale: Optional[float] = None,
                     window: Optional[int] = None, softcap: Optional[float] = None, fp32_weights: bool = False,
-                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
     """out[t] = softmax(q[t] K^T * scale) V over the first ctx_len[t] cached tokens of block-table row bt_row[t], or the
-    last ``window`` of them; ``softcap``: scores are soft-capped, cap * tanh(score / cap); ``sink`` (fp32 [n_q]): the softmax
+    last ``window`` of them, or those from the start of the last one's ``chunk`` (of so many positions, counted from position
+    0) on; ``softcap``: scores are soft-capped, cap * tanh(score / cap); ``sink`` (fp32 [n_q]): the softmax
     denominator has exp(sink) of the head in addition. ``fp32_weights`` keeps the softmax weights at fp32 accuracy in the
     product with V (implied by the options before). Value heads may have another size than key heads
     (``vcache.shape[-1]``)."""
     if not q.is_cuda:
         o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale, window, softcap,
-                                      sink)
+                                      sink, chunk)
         if out is not None:
             out.copy_(o)
             return out
@@ -155,14 +156,14 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     _check_sink(sink, n_q)
     if not attention_on_tensor_cores(q.dtype, n_q, n_kv, hd, vd):
         return _any_attention(q, hd, q.stride(0), kcache, vcache, block_tables, bt_row, None, ctx_len, T, n_q, n_kv, hd, vd,
-                              scale, window, softcap, sink, out, vd, out.stride(0))
+                              scale, window, softcap, sink, out, vd, out.stride(0), chunk)
     assert block_tables.dtype == torch.int32 and ctx_len.dtype == torch.int32 and block_tables.stride(1) == 1
     ws = _attn_workspace(q.device, T * n_q * splits * (vd + 1)) if splits > 1 else None
-    if window or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
+    if window or chunk or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
         _lib.check(_lib.lib().dmoe_paged_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
             _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd),
-            c_float(scale), c_int(window or 0), c_float(softcap or 0.0), _vp(sink), c_int(splits), _vp(out),
+            c_float(scale), c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), c_int(splits), _vp(out),
             c_ll(out.stride(0)), _vp(ws), _st()), "dmoe_paged_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_paged_attention(
@@ -173,7 +174,7 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
 
 
 def _any_attention(q, q_head, q_row, kcache, vcache, block_tables, bt_row, rows, ctx_len, T, n_q, n_kv, hd, vd, scale, window,
-                   softcap, sink, out, o_head, o_row):
+                   softcap, sink, out, o_head, o_row, chunk=None):
     """CUDA-core attention with free strides: query t of head h at q + t * q_row + h * q_head, likewise the output; the
     cached heads of a token are contiguous, tokens ``stride(1)`` apart. Query t has the context of batch row rows[t]
     (None: t)."""
@@ -183,7 +184,7 @@ def _any_attention(q, q_head, q_row, kcache, vcache, block_tables, bt_row, rows,
         c_int(int(q.dtype == torch.float32)), _vp(q), c_ll(q_head), c_ll(q_row), _vp(kcache), c_ll(kcache.stride(1)),
         _vp(vcache), c_ll(vcache.stride(1)), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows),
         _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
-        c_int(window or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(o_head), c_ll(o_row), _st()),
+        c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(o_head), c_ll(o_row), _st()),
         "dmoe_any_attention")
     return out
 
@@ -440,7 +441,8 @@ def build_prefill_tiles(bt_row, positions, tile_tokens: int, min_len: int = 8):
 def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                       tiles: torch.Tensor, n_tiles: int, n_q: int, n_kv: int, hd: int, out: torch.Tensor,
                       scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
-                      fp32_weights: bool = False, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      fp32_weights: bool = False, sink: Optional[torch.Tensor] = None,
+                      chunk: Optional[int] = None) -> torch.Tensor:
     """Causal attention of the prompt tokens named by ``tiles`` (device int32 [>= n_tiles, 4], see
     :func:`build_prefill_tiles`) over the paged cache, which already holds their own K / V; writes their rows of
     ``out``. Every tile streams its sequence's K / V once (the per-token kernel streams it once per row)."""
@@ -450,11 +452,11 @@ def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     vd = vcache.shape[-1]
     _check_sink(sink, n_q)
-    if window or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
+    if window or chunk or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
         _lib.check(_lib.lib().dmoe_prefill_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
             _vp(tiles), c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
-            c_int(window or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()),
+            c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()),
             "dmoe_prefill_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_prefill_attention(
@@ -502,52 +504,107 @@ def resid_norm(resid: torch.Tensor, y: Optional[torch.Tensor], post: Optional[to
 
 @dataclass
 class Router:
-    """Softmax router over rows that are already normalised: ``weight`` [experts, width] in the activations' dtype, the
-    ``top`` largest scores as weights (``renormalize``: divided by their sum); ``counts`` (int32 [experts]) is the histogram
-    that :func:`dispatch_local` reads and clears."""
+    """Router over rows that are already normalised: ``weight`` [experts, width] in the activations' dtype. ``sigmoid``: scores
+    sigmoid(logit) instead of softmax; then ``correction`` (fp32 [experts]) is added for the choice alone, and of ``groups`` equal
+    groups of neighbouring experts only the ``keep`` whose two best choice scores have the largest sum are open. The ``top``
+    experts with the largest (choice) scores are chosen; their weights are the scores, with ``renormalize`` divided by their
+    sum, times ``scale``. ``counts`` (int32 [experts]) is the histogram that :func:`dispatch_local` reads and clears."""
     weight: torch.Tensor
     top: int
     renormalize: bool = False
     counts: Optional[torch.Tensor] = None
+    sigmoid: bool = False
+    correction: Optional[torch.Tensor] = None
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
 
     MAX_EXPERTS, MAX_TOP = 256, 32
 
 
+@dataclass
+class TokenShift:
+    """Mixes of every row with the row before it in its sequence: h + (before - h) mu_s. ``mu`` fp32 [n, W]; ``last`` fp32
+    [slots, W] keeps the last row of every sequence from step to step (not read at position 0); ``segs``: the segments of the
+    step (:class:`disagmoe_b200.ops.recurrent.SegmentTables`)."""
+    mu: torch.Tensor
+    last: torch.Tensor
+    segs: "SegmentTables"                        # noqa: F821
+
+    def descriptor(self, T: int) -> _lib.DmoeShift:
+        d, s = _lib.DmoeShift(), self.segs
+        n, W = self.mu.shape
+        assert self.mu.dtype == self.last.dtype == torch.float32 and self.mu.is_contiguous() and self.last.is_contiguous()
+        assert self.last.shape[1] == W
+        d.mu, d.last, d.singles = self.mu.data_ptr(), self.last.data_ptr(), _lib.ptr(s.singles) if s.n_single else 0
+        d.positions, d.rows, d.kv_slots = _lib.ptr(s.positions), _lib.ptr(s.rows), _lib.ptr(s.kv_slots)
+        d.mix_stride, d.n_mix, d.n_slots, d.n_single = T * W, n, self.last.shape[0], s.n_single
+        return d
+
+
+def token_shift(h: torch.Tensor, shift: TokenShift, dtype: torch.dtype) -> torch.Tensor:
+    """fp32 rows h [T, W] -> the mixes [n, T, W] in ``dtype``; ``shift.last`` takes the last row of every segment."""
+    if not h.is_cuda:
+        return reference.token_shift(h, shift.mu, shift.last, shift.segs).to(dtype)
+    T, W = h.shape
+    s, n = shift.segs, shift.mu.shape[0]
+    assert h.dtype == torch.float32 and h.is_contiguous()
+    out = torch.empty(n, T, W, dtype=dtype, device=h.device)
+    d = shift.descriptor(T)
+    _lib.check(_lib.lib().dmoe_token_shift(_f32(dtype), _vp(h), ctypes.byref(d), _vp(s.multi), c_int(s.n_multi), _vp(s.chunks),
+                                           c_int(s.n_chunks), _vp(out), c_ll(W), c_int(W), _st()), "dmoe_token_shift")
+    return out
+
+
 def sum_norm(resid: torch.Tensor, y: Optional[torch.Tensor], parts: Optional[torch.Tensor], w: torch.Tensor, eps: float,
-             dtype: torch.dtype, centred: bool, rows: Optional[torch.Tensor] = None, router: Optional[Router] = None):
-    """One step of a residual stream kept in fp32 whose sublayers share a norm: resid += y + parts.sum(1) (y [T, W], parts
-    [T, P, W] or [T, W], each may be None), then h = norm(resid) * w in ``dtype``; ``centred``: layer norm, otherwise RMS
-    norm. ``rows`` (int32) picks the rows to return; resid itself is then left as it is. Returns (h, expert ids [T, top],
-    weights [T, top]), the last two None without a ``router``, which sees h."""
+             dtype: torch.dtype, centred: bool, rows: Optional[torch.Tensor] = None, router: Optional[Router] = None,
+             mult: float = 1.0, shift: Optional[TokenShift] = None):
+    """One step of a residual stream kept in fp32: resid += mult * (y + parts.sum(1)) (y [T, W], parts [T, P, W] or [T, W],
+    each may be None), then h = norm(resid) * w in ``dtype``; ``centred``: layer norm, otherwise RMS norm. ``rows`` (int32)
+    picks the rows to return; resid itself is then left as it is. Returns (h, expert ids [T, top], weights [T, top]), the last
+    two None without a ``router``, which sees h. With a token ``shift``, h (kept in fp32 on the way) becomes its mixes
+    [n, T, W]; where every segment has one token (decoding) that is one launch."""
     if not resid.is_cuda:
-        h = reference.sum_norm(resid, y, parts, w, eps, dtype, centred, rows)
+        h = reference.sum_norm(resid, y, parts, w, eps, torch.float32 if shift else dtype, centred, rows, mult)
+        if shift is not None:
+            return token_shift(h, shift, dtype), None, None
         if router is None:
             return h, None, None
-        _, ids, wts, _ = reference.route(h, None, eps, router.weight, router.top, router.renormalize)
+        if router.sigmoid:
+            ids, wts = reference.sigmoid_route(h, router)
+        else:
+            _, ids, wts, _ = reference.route(h, None, eps, router.weight, router.top, router.renormalize)
+            wts = wts * router.scale
         if router.counts is not None:
             router.counts += torch.bincount(ids.reshape(-1).long(), minlength=router.weight.shape[0]).int()
         return h, ids, wts
     n, W = (resid.shape[0] if rows is None else rows.shape[0]), resid.shape[1]
     if parts is not None and parts.dim() == 2:
         parts = parts.unsqueeze(1)
-    h = torch.empty(n, W, dtype=dtype, device=resid.device)
+    two_steps = shift is not None and shift.segs.n_multi > 0
+    h = torch.empty((n, W) if shift is None or two_steps else (shift.mu.shape[0], n, W),
+                    dtype=torch.float32 if two_steps else dtype, device=resid.device)
     assert resid.dtype == torch.float32 and resid.is_contiguous() and w.dtype == torch.float32
     assert all(a is None or (a.dtype == dtype and a.stride(-1) == 1) for a in (y, parts)) and (rows is None or rows.dtype == torch.int32)
-    ids = wts = None
-    E = K = 0
+    ids = wts = rd = sd = None
     if router is not None:
         E, K = router.weight.shape[0], router.top
-        assert rows is None and router.weight.dtype == dtype and router.weight.is_contiguous()
+        assert rows is None and shift is None and router.weight.dtype == dtype and router.weight.is_contiguous()
+        c = router.correction
+        assert c is None or (router.sigmoid and c.dtype == torch.float32 and c.numel() == E and c.is_contiguous())
         ids = torch.empty(n, K, dtype=torch.int32, device=resid.device)
         wts = torch.empty(n, K, dtype=torch.float32, device=resid.device)
+        rd = _lib.DmoeRouter(router.weight.data_ptr(), _lib.ptr(c), ids.data_ptr(), wts.data_ptr(), _lib.ptr(router.counts), E, K,
+                             int(router.renormalize), int(router.sigmoid), router.groups, router.keep, router.scale)
+    if shift is not None and not two_steps:
+        sd = shift.descriptor(n)
     _lib.check(_lib.lib().dmoe_sum_norm(
         _f32(dtype), _vp(resid), _vp(y), c_ll(y.stride(0) if y is not None else 0), _vp(parts),
         c_int(parts.shape[1] if parts is not None else 0), c_ll(parts.stride(0) if parts is not None else 0),
-        c_ll(parts.stride(1) if parts is not None else 0), _vp(w), c_int(int(centred)), c_float(eps), _vp(rows), _vp(h), c_ll(W),
-        c_int(n), c_int(W), _vp(router.weight if router else None), c_int(E), c_int(K),
-        c_int(int(bool(router and router.renormalize))), _vp(ids), _vp(wts), _vp(router.counts if router else None), _st()),
-        "dmoe_sum_norm")
-    return h, ids, wts
+        c_ll(parts.stride(1) if parts is not None else 0), c_float(mult), _vp(w), c_int(int(centred)), c_float(eps), _vp(rows),
+        _vp(h), c_int(int(two_steps)), c_ll(W), c_int(n), c_int(W), ctypes.byref(rd) if rd else None,
+        ctypes.byref(sd) if sd else None, _st()), "dmoe_sum_norm")
+    return (token_shift(h, shift, dtype) if two_steps else h), ids, wts
 
 
 def rope_frequencies(dims: int, base: float, factor: Optional[float] = None, original: float = 0.0, fast: float = 32.0,
@@ -593,14 +650,15 @@ def rope_freq_table(spec, max_pos: int, device) -> Optional[torch.Tensor]:
 def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: Optional[torch.Tensor],
                  vcache: Optional[torch.Tensor], n_q: int, n_kv: int, dk: int, dv: int, table: Optional[torch.Tensor],
                  qw: Optional[torch.Tensor], kw: Optional[torch.Tensor], eps: float, interleaved: bool = False,
-                 v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0) -> None:
+                 v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, tied: bool = False) -> None:
     """RMS norm of every q / k head (weights fp32 [dk]; None: no norm) and rotation by ``table`` (:func:`rope_freq_table`,
     None: no rotation; ``interleaved``: of neighbouring dimensions) on rows [q | k | v]; q in place, k and v to the paged
     caches at ``slots``. n_kv = 0: q only (a layer that reads another layer's cache). ``v_first`` [T, n_kv, >= dv]: the
-    values become (1 - v_lambda) v + v_lambda v_first on their way to the cache."""
+    values become (1 - v_lambda) v + v_lambda v_first on their way to the cache. ``tied``: rows [q | k], the values are the first
+    dv dimensions of the keys before their norm and rotation."""
     if not qkv.is_cuda:
         return reference.qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps,
-                                      interleaved, v_first, v_lambda)
+                                      interleaved, v_first, v_lambda, tied)
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and qkv.stride(1) == 1
     assert n_kv == 0 or (kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == qkv.dtype)
     rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
@@ -608,7 +666,7 @@ def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor
         _f32(qkv.dtype), _vp(qkv), c_ll(qkv.stride(0)), _vp(positions), _vp(slots), _vp(kcache), _vp(vcache),
         c_int(qkv.shape[0]), c_int(n_q), c_int(n_kv), c_int(dk), c_int(dv), c_int(rot), c_int(int(interleaved)), _vp(table),
         c_int(max_pos), _vp(qw), _vp(kw), c_float(eps), _vp(v_first), c_ll(v_first.stride(0) if v_first is not None else 0),
-        c_int(v_first.stride(1) if v_first is not None else 0), c_float(v_lambda), _st()), "dmoe_qk_norm_rope")
+        c_int(v_first.stride(1) if v_first is not None else 0), c_float(v_lambda), c_int(int(tied)), _st()), "dmoe_qk_norm_rope")
 
 
 # ---- latent attention (csrc/kernels/latent_attention.cu) ---------------------------------------------------------------
@@ -620,7 +678,7 @@ def _pad8(n: int) -> int:
 class LatentLayout:
     """Sizes of a latent attention layer as its kernels see them: every part of a row is padded to a multiple of 8 (zeros).
 
-    projection row   [heads x (q unrotated | q rotated) | latent | rotated key part]
+    projection row   [heads x (q unrotated | q rotated) | latent | rotated key part (| one gate per head)]
     cache row        [latent | rotated key part], an odd multiple of 8 elements from one row to the next: tiles that are copied
                      to shared memory as they are read without bank conflicts
     """
@@ -675,23 +733,27 @@ LATENT_MAX_RANK, LATENT_MAX_KEY = 512, 640            # of the tensor-core kerne
 
 def latent_prep(y: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, lay: LatentLayout,
                 table: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float, loose: Optional[torch.Tensor], n_loose: int,
-                interleaved: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
+                interleaved: bool = True, gate: Optional[torch.Tensor] = None,
+                recs: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """From projection rows y (:class:`LatentLayout`): RMS norm of the latent (weight fp32 [rank]), rotation of the shared
     key part, both to the paged ``cache`` [blocks, block_size, row] at ``slots``; rotation of the queries, in place. Rows with
     loose[t] = i >= 0 (None: row t is i = t) are attended over the latents themselves, so their queries are also written
     head by head: returns (unrotated part [heads, n_loose, dimp], [heads, n_loose, row] with the rotated part in place and
-    the latent part still to be filled)."""
+    the latent part still to be filled). ``gate`` (columns of y, [T, heads]): sigmoid(gate) becomes the weight of the loose rows'
+    records ``recs`` [heads * n_loose, 4] (:func:`disagmoe_b200.ops.gemm.grouped_combine`)."""
     if not y.is_cuda:
-        return reference.latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved)
+        return reference.latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved, gate, recs)
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and y.stride(1) == 1 and cache.is_contiguous()
-    assert y.shape[1] == lay.heads * lay.qd + lay.kd and cache.dtype == y.dtype and norm_w.dtype == torch.float32
+    assert gate is None or (gate.dtype == y.dtype and gate.stride(1) == 1 and gate.stride(0) == y.stride(0))
+    assert gate is None or n_loose == 0 or (recs.is_contiguous() and recs.shape == (lay.heads * n_loose, 4))
+    assert y.shape[1] >= lay.heads * lay.qd + lay.kd and cache.dtype == y.dtype and norm_w.dtype == torch.float32
     xq = torch.empty(lay.heads, n_loose, lay.dimp, dtype=y.dtype, device=y.device)
     qa = torch.empty(lay.heads, n_loose, lay.row, dtype=y.dtype, device=y.device)
     rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
     _lib.check(_lib.lib().dmoe_latent_prep(
         _f32(y.dtype), _vp(y), c_ll(y.stride(0)), _vp(positions), _vp(slots), _vp(cache), c_int(y.shape[0]), c_int(lay.heads),
         c_int(lay.dim), c_int(lay.rot), c_int(lay.rank), c_int(lay.row), c_int(rot), c_int(int(interleaved)), _vp(table), c_int(max_pos),
-        _vp(norm_w), c_float(eps), _vp(loose), c_int(n_loose), _vp(xq), _vp(qa), _st()), "dmoe_latent_prep")
+        _vp(norm_w), c_float(eps), _vp(loose), c_int(n_loose), _vp(xq), _vp(qa), _vp(gate), _vp(recs), _st()), "dmoe_latent_prep")
     return xq, qa
 
 
@@ -744,14 +806,17 @@ def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, keys: torch.T
 
 def latent_prefill(q: torch.Tensor, kv: torch.Tensor, lat: torch.Tensor, tiles: torch.Tensor, base: torch.Tensor, n_tiles: int,
                    lay: LatentLayout, scale: float, window: Optional[int], sink: Optional[torch.Tensor],
-                   out: torch.Tensor) -> torch.Tensor:
+                   out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the prompt tokens named by ``tiles`` over expanded keys and values: kv [keys, heads x (key
     unrotated | value)], rotated key parts in the gathered cache rows ``lat`` [keys, row]; the key at position p of tile i's
-    sequence is row base[i] + p. q: projection rows with rotated queries. Writes the tokens' rows of out [T, heads x vdimp]."""
+    sequence is row base[i] + p. q: projection rows with rotated queries. Writes the tokens' rows of out [T, heads x vdimp], scaled by sigmoid(gate)
+    per head where ``gate`` [T, heads] is given."""
     _check_sink(sink, lay.heads)
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1)
     assert tiles.dtype == base.dtype == torch.int32 and kv.stride(1) == lat.stride(1) == 1
     _lib.check(_lib.lib().dmoe_latent_prefill(
         _vp(q), c_ll(q.stride(0)), _vp(kv), c_ll(kv.stride(0)), _vp(lat), c_ll(lat.stride(0)), _vp(tiles), _vp(base),
         c_int(n_tiles), c_int(lay.heads), c_int(lay.dimp), c_int(lay.rotp), c_int(lay.rankp), c_int(lay.vdimp), c_float(scale),
-        c_int(window or 0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()), "dmoe_latent_prefill")
+        c_int(window or 0), _vp(sink), _vp(gate), c_ll(gate.stride(0) if gate is not None else 0), _vp(out), c_ll(out.stride(0)),
+        _st()), "dmoe_latent_prefill")
     return out

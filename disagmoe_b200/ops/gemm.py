@@ -21,6 +21,7 @@ import torch
 from . import _lib, reference
 
 ACTS = {"silu": 0, "gelu_tanh": 1}
+ACT_TANH = 2         # of the output of a plain GEMM
 EPI_PLAIN, EPI_SWIGLU, EPI_COMBINE = 0, 1, 2
 STREAM_K = True      # default work distribution of every GEMM launched without an explicit split (tests may turn it off)
 TRACE = None         # profiling aid: an int64 [8] CUDA tensor that CTA 0 of every launch fills with nanosecond stamps
@@ -221,10 +222,10 @@ def rope_table(max_pos: int, hd: int, theta: float, device) -> torch.Tensor:
 
 
 def _launch(W, X, Y, R, offs, recs, bases, G, T, F, K, epi, bn, splitk, ldy, y_f32, comm: Optional[GemmComm] = None,
-            streamk: bool = False, pair: bool = False, w_blocked: bool = False, act: str = "silu"):
+            streamk: bool = False, pair: bool = False, w_blocked: bool = False, act: int = 0):
     s = scratch(X.device)
     d = _lib.DmoeGemm()
-    d.w_blocked, d.act = int(w_blocked), ACTS[act]
+    d.w_blocked, d.act = int(w_blocked), act
     d.trace = TRACE.data_ptr() if TRACE is not None else None
     d.streamk, d.n_counters = int(streamk and splitk <= 1 and not pair), s.counters.numel()
     d.pair = int(pair)
@@ -251,7 +252,7 @@ def _tma_ok(x, w) -> bool:
     return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
 
 
-def _simt_linear(x, w, out, out_dtype):
+def _simt_linear(x, w, out, out_dtype, tanh=False):
     """fp32 operands (true fp32 arithmetic), or bf16 operands that TMA cannot address: the CUDA-core GEMM."""
     T, K = x.shape
     F = w.shape[0]
@@ -263,7 +264,7 @@ def _simt_linear(x, w, out, out_dtype):
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
     _lib.check(_lib.lib().dmoe_simt_linear(
         i(int(f32)), i(int(out.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), ll(K),
-        v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), v(_lib.stream_ptr())), "dmoe_simt_linear")
+        v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), i(ACT_TANH if tanh else 0), v(_lib.stream_ptr())), "dmoe_simt_linear")
     return out
 
 
@@ -298,13 +299,15 @@ def _check_x(x):
 
 def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = None,
            out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, bn: int = 0,
-           splitk: int = 0, comm: Optional["GemmComm"] = None, pair: bool = False) -> torch.Tensor:
-    """y[T, F] = x[T, K] @ w[F, K].T (+ residual[T, F]). ``pair``: CTA pairs (tcgen05 cta_group::2) on tiles of 256
+           splitk: int = 0, comm: Optional["GemmComm"] = None, pair: bool = False, tanh: bool = False) -> torch.Tensor:
+    """y[T, F] = x[T, K] @ w[F, K].T (+ residual[T, F]); ``tanh``: of the product. ``pair``: CTA pairs (tcgen05 cta_group::2) on tiles of 256
     weight rows x ``bn`` (128 / 256) tokens, whole tiles."""
     T, K = x.shape
     F = w.shape[0]
     if not x.is_cuda:
         y = torch.nn.functional.linear(x.float(), w.float())
+        if tanh:
+            y = torch.tanh(y)
         if residual is not None:
             y = y + residual.float()
         y = y.to(out_dtype or x.dtype)
@@ -314,7 +317,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         return y
     if x.dtype == torch.float32 or (comm is None and residual is None and not _tma_ok(x, w)):
         assert comm is None and residual is None
-        return _simt_linear(x, w, out, out_dtype)
+        return _simt_linear(x, w, out, out_dtype, tanh)
     _check_x(x)
     assert w.is_contiguous() and w.dtype == torch.bfloat16 and w.shape[1] == K
     odt = out_dtype or torch.bfloat16
@@ -343,7 +346,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         splitk = splitk or auto_sk or pick_splitk(T, F, K, bn, sms)
     _launch(w, x, out, residual, None, None, None, 1, T, F, K, EPI_PLAIN, bn, splitk,
             F if scatter else out.stride(0), (not scatter) and out.dtype == torch.float32, comm, streamk=streamk,
-            pair=pair)
+            pair=pair, act=ACT_TANH if tanh else 0)
     return out
 
 
@@ -391,7 +394,7 @@ def grouped_swiglu(x: torch.Tensor, w13: torch.Tensor, offs: Optional[torch.Tens
         bn = max(bn, 128)
     sk = want_streamk(EPI_SWIGLU, I, G, T, bn, num_sms(x.device)) if streamk is None else streamk
     _launch(w13, x, out, None, offs, None, None, G, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False, comm,
-            streamk=sk, pair=pair, w_blocked=w_blocked, act=act)
+            streamk=sk, pair=pair, w_blocked=w_blocked, act=ACTS[act])
     return out
 
 
@@ -513,5 +516,5 @@ def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor
         return out
     bn = bn or pick_bn(T, EPI_SWIGLU)
     _launch(w13, x, out, None, None, None, None, 1, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False,
-            act=act)
+            act=ACTS[act])
     return out

@@ -1,5 +1,5 @@
-"""Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``, ``recurrent_chunk.cu``): gated linear attention and the gated
-delta rule, with one decay per head and key channel. CUDA tensors run the kernels, CPU tensors the PyTorch restatements.
+"""Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``, ``recurrent_chunk.cu``): gated linear
+attention, the gated delta rule and RWKV-style time mixing, with one decay per head and key channel. CUDA tensors run the kernels, CPU tensors the PyTorch restatements.
 
 A step's rows fall into segments (consecutive rows of one sequence). One-token segments (decoding) take one launch from
 the projections to the gated, normalised output; longer ones (prompts and portions of prompts) are convolved and then run
@@ -39,6 +39,12 @@ class SegmentTables:
     rows: Optional[torch.Tensor] = None
     kv_slots: Optional[torch.Tensor] = None
 
+    def table(self):
+        """(first row, tokens, slot, first position) of every segment that is not padding (reads the tables back)."""
+        if self.singles is None and self.n_single:
+            return [(i, 1, int(self.rows[i]), int(self.positions[i])) for i in range(self.n_single) if self.kv_slots[i] >= 0]
+        return self.singles.tolist() + self.multi.tolist()
+
 
 def build_segments(bt_row, positions, device) -> SegmentTables:
     """Tables of a batch given on the host (rows of one sequence are consecutive, as every scheduler emits them)."""
@@ -65,19 +71,23 @@ def decode_segments(positions: torch.Tensor, rows: torch.Tensor, kv_slots: torch
 
 @dataclass
 class RecurrentState:
-    """Per-layer state pool: S fp32 [slots, heads, dim, vdim] and, with a short convolution, the ring of its last inputs
-    [slots, taps, channels]. A slot needs no clearing: a segment at position 0 starts from zero."""
+    """Per-layer state pool: S fp32 [slots, heads, dim, vdim]; with a short convolution the ring of its last inputs [slots,
+    taps, channels]; with a token shift the last input row, fp32 [slots, width]. A slot needs no clearing: a segment at position 0 starts from zero."""
     S: torch.Tensor
     ring: Optional[torch.Tensor] = None
+    last: Optional[torch.Tensor] = None
 
     def tensors(self):
-        return [self.S] + ([self.ring] if self.ring is not None else [])
+        return [t for t in (self.S, self.ring, self.last) if t is not None]
 
 
 @dataclass
 class Recurrence:
     """Constants of one recurrent layer (weights fp32). ``delta``: the gated delta rule with unit-norm q / k and
-    log a = -exp(a_log) softplus(z + z_bias); otherwise the plain write with log a = log sigmoid(z + z_bias) / tau."""
+    log a = -exp(a_log) softplus(z + z_bias); otherwise the plain write with log a = log sigmoid(z + z_bias) / tau or,
+    ``exp_decay``, log a = -exp(z + z_bias). ``bonus`` [heads, dim]: the read-out precedes decay and write, and the token's own
+    write enters it weighed by the bonus. ``norm_w``: [vdim], or [heads * vdim] with a weight per head; ``qscale``: factor of q
+    (None: dim ** -0.5); ``shift_width``: width of the token shift whose last row belongs to the state (0: none)."""
     heads: int
     kv_heads: int
     dim: int
@@ -90,6 +100,22 @@ class Recurrence:
     tau: float = 1.0
     conv_w: Optional[torch.Tensor] = None            # [2 kv_heads dim + heads vdim, taps]
     sigmoid_gate: bool = False
+    exp_decay: bool = False
+    bonus: Optional[torch.Tensor] = None
+    qscale: Optional[float] = None
+    shift_width: int = 0
+
+    @property
+    def decay_kind(self) -> int:
+        return 2 if self.exp_decay else int(self.delta)
+
+    @property
+    def norm_ld(self) -> int:
+        return 0 if self.norm_w.numel() == self.vdim else self.vdim
+
+    @property
+    def q_factor(self) -> float:
+        return self.dim ** -0.5 if self.qscale is None else self.qscale
 
     @property
     def taps(self) -> int:
@@ -102,7 +128,8 @@ class Recurrence:
     def new_state(self, slots: int, dtype, device) -> RecurrentState:
         S = torch.zeros(slots, self.heads, self.dim, self.vdim, dtype=torch.float32, device=device)
         ring = torch.zeros(slots, self.taps, self.channels, dtype=dtype, device=device) if self.taps else None
-        return RecurrentState(S, ring)
+        last = torch.zeros(slots, self.shift_width, dtype=torch.float32, device=device) if self.shift_width else None
+        return RecurrentState(S, ring, last)
 
 
 def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) -> _lib.DmoeRecur:
@@ -115,9 +142,10 @@ def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) ->
     d.z_bias, d.a_log, d.norm_w = _lib.ptr(r.z_bias), _lib.ptr(r.a_log), _lib.ptr(r.norm_w)
     d.state, d.n_slots = _lib.ptr(state.S), state.S.shape[0]
     d.heads, d.kv_heads, d.dim, d.vdim = r.heads, r.kv_heads, r.dim, r.vdim
-    d.delta, d.decay_kind, d.gate_kind = int(r.delta), int(r.delta), int(r.sigmoid_gate)
+    d.delta, d.decay_kind, d.gate_kind = int(r.delta), r.decay_kind, int(r.sigmoid_gate)
+    d.bonus, d.norm_ld = _lib.ptr(r.bonus), r.norm_ld
     d.is_f32 = int(q.dtype == torch.float32)
-    d.qscale, d.inv_tau, d.eps = r.dim ** -0.5, 1.0 / r.tau, r.eps
+    d.qscale, d.inv_tau, d.eps = r.q_factor, 1.0 / r.tau, r.eps
     d.status = scratch(q.device).status.data_ptr()
     return d
 
@@ -126,7 +154,7 @@ def _gate_norm(r: Recurrence, table, n, max_tokens, raw, gate, out) -> None:
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
     _lib.check(_lib.lib().dmoe_gate_norm(
         i(int(out.dtype == torch.float32)), v(_lib.ptr(table)), i(n), i(max_tokens), v(raw.data_ptr()), ll(raw.stride(0)),
-        v(gate.data_ptr()), ll(gate.stride(0)), v(r.norm_w.data_ptr()), ctypes.c_float(r.eps), i(int(r.sigmoid_gate)),
+        v(gate.data_ptr()), ll(gate.stride(0)), v(r.norm_w.data_ptr()), i(r.norm_ld), ctypes.c_float(r.eps), i(int(r.sigmoid_gate)),
         v(out.data_ptr()), ll(out.stride(0)), i(r.heads), i(r.vdim), v(_lib.stream_ptr())), "dmoe_gate_norm")
 
 
@@ -190,21 +218,17 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
 
 def _reference(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, segs: SegmentTables) -> torch.Tensor:
     T, H, G, D, V = q.shape[0], r.heads, r.kv_heads, r.dim, r.vdim
-    if segs.singles is None and segs.n_single:
-        table = [(i, 1, int(segs.rows[i]), int(segs.positions[i])) for i in range(segs.n_single) if segs.kv_slots[i] >= 0]
-    else:
-        table = segs.singles.tolist() + segs.multi.tolist()
     zb = z.float() + r.z_bias
-    logd = (-torch.exp(r.a_log)[:, None] * torch.nn.functional.softplus(zb).view(T, H, D)) if r.delta else \
+    logd = -torch.exp(zb).view(T, H, D) if r.exp_decay else (-torch.exp(r.a_log)[:, None] * torch.nn.functional.softplus(zb).view(T, H, D)) if r.delta else \
         torch.nn.functional.logsigmoid(zb).view(T, H, D) / r.tau
     out = torch.zeros(T, H * V, dtype=q.dtype)
-    for a, n, slot, pos0 in table:
+    for a, n, slot, pos0 in segs.table():
         x = torch.cat([q[a:a + n], k[a:a + n], v[a:a + n]], 1)
         if r.taps:
             x = reference.conv_segment(x, r.conv_w, state.ring[slot], pos0)
         qq, kk = (x[:, j * G * D:(j + 1) * G * D].view(n, G, D).repeat_interleave(H // G, 1) for j in (0, 1))
         o = reference.recur_segment(qq, kk, x[:, 2 * G * D:].view(n, H, V), None if beta is None else beta[a:a + n],
-                                    logd[a:a + n], state.S[slot], pos0, r.delta, D ** -0.5)
-        o = reference.gate_norm(o, gate[a:a + n].view(n, H, V), r.norm_w, r.eps, r.sigmoid_gate)
+                                    logd[a:a + n], state.S[slot], pos0, r.delta, r.q_factor, r.bonus)
+        o = reference.gate_norm(o, gate[a:a + n].view(n, H, V), r.norm_w.view(-1, V), r.eps, r.sigmoid_gate)
         out[a:a + n] = o.reshape(n, H * V).to(q.dtype)
     return out

@@ -59,9 +59,9 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slots: Optional[t
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
                     scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
-                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
     """Token t attends to the first ctx_len[t] cached tokens of block-table row bt_row[t] (default t), or to the last
-    ``window`` of them; ``softcap``: scores become cap * tanh(score / cap); ``sink`` [n_q]: the softmax denominator has
+    ``window`` of them, or to those in the same ``chunk`` of positions as the last one; ``softcap``: scores become cap * tanh(score / cap); ``sink`` [n_q]: the softmax denominator has
     exp(sink) in addition."""
     T = q.shape[0]
     block_size = kcache.shape[1]
@@ -80,6 +80,9 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         v = vcache[blocks].reshape(nb * block_size, n_kv, vd)[:L].float()
         if window:
             k, v = k[-window:], v[-window:]
+        if chunk:
+            n = (L - 1) % chunk + 1
+            k, v = k[-n:], v[-n:]
         qt = q[t].float().view(n_kv, gq, hd)
         s = torch.einsum("kgd,lkd->kgl", qt, k) * scale
         if softcap:
@@ -105,6 +108,23 @@ def route(x: torch.Tensor, norm_w: Optional[torch.Tensor], eps: float, gate_w: t
     if renormalize:
         w = w / w.sum(-1, keepdim=True)
     return y, ids.int(), w.float(), logits
+
+
+def sigmoid_route(h: torch.Tensor, r) -> Tuple[torch.Tensor, torch.Tensor]:
+    """(ids int32 [T, top], weights fp32 [T, top]) of a sigmoid :class:`disagmoe_b200.ops.functional.Router`."""
+    s = torch.sigmoid(h.float() @ r.weight.float().T)
+    choice = s if r.correction is None else s + r.correction
+    T, E = s.shape
+    if r.keep < r.groups:
+        grouped = choice.view(T, r.groups, E // r.groups)
+        rank = grouped.topk(min(2, E // r.groups), dim=-1).values.sum(-1)
+        open_ = torch.zeros_like(rank, dtype=torch.bool).scatter_(1, rank.topk(r.keep, dim=-1).indices, True)
+        choice = grouped.masked_fill(~open_[..., None], float("-inf")).reshape(T, E)
+    ids = choice.topk(r.top, dim=-1).indices
+    w = s.gather(1, ids)
+    if r.renormalize:
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return ids.int(), w * r.scale
 
 
 def expert_offsets(topk_ids: torch.Tensor, num_experts: int) -> torch.Tensor:
@@ -180,14 +200,14 @@ def resid_norm(resid, y, post, pre, eps, dtype, out_scale=1.0, rows=None):
     return None if pre is None else (_rms_scale(x, eps) * pre * out_scale).to(dtype)
 
 
-def sum_norm(resid, y, parts, w, eps, dtype, centred, rows=None):
-    """resid += y + parts.sum(1) (either may be None; ``rows``: only these rows are returned, resid untouched); returns the
+def sum_norm(resid, y, parts, w, eps, dtype, centred, rows=None, mult=1.0):
+    """resid += mult * (y + parts.sum(1)) (either may be None; ``rows``: only these rows are returned, resid untouched); returns the
     RMS norm of resid times w, or with ``centred`` its layer norm (mean taken off) times w."""
     x = resid if rows is None else resid[rows.long()]
     for a in (y, parts):
         if a is not None:
             a = a if rows is None else a[rows.long()]
-            x = x + (a.float() if a.dim() == 2 else a.float().sum(1))
+            x = x + mult * (a.float() if a.dim() == 2 else a.float().sum(1))
     if rows is None:
         resid.copy_(x)
     if centred:
@@ -209,9 +229,9 @@ def _turn(x, table, positions, interleaved):
 
 
 def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps, interleaved=False,
-                 v_first=None, v_lambda=0.0) -> None:
+                 v_first=None, v_lambda=0.0, tied=False) -> None:
     """Per-head norm (where weights are given) + partial rotation of q (in place) and k, K / V append at slots >= 0; with
-    ``v_first`` [T, n_kv, >= dv] the values appended are (1 - v_lambda) v + v_lambda v_first."""
+    ``v_first`` [T, n_kv, >= dv] the values appended are (1 - v_lambda) v + v_lambda v_first, ``tied`` those of the raw keys."""
     T = qkv.shape[0]
 
     def turn(x, w):
@@ -224,18 +244,19 @@ def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table
         k = turn(qkv[:, qs:qs + ks].reshape(T, n_kv, dk), kw).to(qkv.dtype)
         ok = slots >= 0
         kcache.view(-1, n_kv, dk)[slots[ok]] = k[ok]
-        v = qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
+        v = qkv[ok][:, qs:qs + ks].reshape(-1, n_kv, dk)[..., :dv] if tied else \
+            qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
         if v_first is not None:
             v = ((1.0 - v_lambda) * v.float() + v_lambda * v_first[ok][..., :dv].float()).to(v.dtype)
         vcache.view(-1, n_kv, dv)[slots[ok]] = v
     qkv[:, :qs] = q.reshape(T, qs).clone()
 
 
-def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved):
+def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_loose, interleaved, gate=None, recs=None):
     """See :func:`disagmoe_b200.ops.functional.latent_prep`."""
     T, H = y.shape[0], lay.heads
     q = y[:, :H * lay.qd].reshape(T, H, lay.qd)
-    d = y[:, H * lay.qd:]
+    d = y[:, H * lay.qd:H * lay.qd + lay.kd]
     c = (_rms_scale(d[:, :lay.rank].float(), eps) * norm_w).to(y.dtype)
     kr = _turn(d[:, None, lay.rankp:lay.rankp + lay.rot].float(), table, positions, interleaved)[:, 0].to(y.dtype)
     ok = slots >= 0
@@ -248,6 +269,10 @@ def latent_prep(y, positions, slots, cache, lay, table, norm_w, eps, loose, n_lo
     on = idx >= 0
     xq[:, idx[on]] = q[on][..., :lay.dimp].transpose(0, 1)
     qa[:, idx[on], lay.rankp:lay.rankp + lay.rot] = qr[on].transpose(0, 1)
+    if gate is not None and n_loose:
+        g = torch.zeros(H, n_loose)
+        g[:, idx[on]] = torch.sigmoid(gate[on].float()).T
+        recs[:, 2] = g.reshape(-1).view(torch.int32)
     y[:, :H * lay.qd] = torch.cat([q[..., :lay.dimp], qr, q[..., lay.dimp + lay.rot:]], -1).reshape(T, -1)
     return xq, qa
 
@@ -265,9 +290,21 @@ def conv_segment(x: torch.Tensor, w: torch.Tensor, ring: Optional[torch.Tensor],
     return torch.nn.functional.silu(acc).to(x.dtype)
 
 
-def recur_segment(q, k, v, beta, logd, state: torch.Tensor, pos0: int, delta: bool, qscale: float) -> torch.Tensor:
+def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, segs) -> torch.Tensor:
+    """See :func:`disagmoe_b200.ops.functional.token_shift`: fp32 [n, T, W]."""
+    before = torch.zeros_like(h)
+    for a, n, slot, pos0 in segs.table():
+        before[a + 1:a + n] = h[a:a + n - 1]
+        if pos0 > 0:
+            before[a] = last[slot]
+        last[slot] = h[a + n - 1]
+    return h + (before - h) * mu[:, None]
+
+
+def recur_segment(q, k, v, beta, logd, state: torch.Tensor, pos0: int, delta: bool, qscale: float, bonus=None) -> torch.Tensor:
     """Token-by-token recurrence of one segment: q, k, logd [n, H, D], v [n, H, V], beta [n, H] (delta); ``state``
-    [H, D, V] is read (zero where pos0 = 0) and updated. Returns fp32 read-outs [n, H, V]."""
+    [H, D, V] is read (zero where pos0 = 0) and updated. ``bonus`` [H, D]: the read-out precedes decay and write, and the
+    token's own write enters it with that weight. Returns fp32 read-outs [n, H, V]."""
     q, k, v = q.float(), k.float(), v.float()
     if delta:
         q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6)
@@ -276,6 +313,11 @@ def recur_segment(q, k, v, beta, logd, state: torch.Tensor, pos0: int, delta: bo
     S = state.clone() if pos0 > 0 else torch.zeros_like(state)
     out = []
     for t in range(q.shape[0]):
+        if bonus is not None:
+            kv = k[t][..., None] * v[t][:, None, :]
+            out.append(torch.einsum("hdv,hd->hv", S + bonus[..., None] * kv, q[t]))
+            S = S * torch.exp(logd[t])[..., None] + kv
+            continue
         S = S * torch.exp(logd[t])[..., None]
         u = v[t]
         if delta:
