@@ -1,12 +1,14 @@
 """Prefill and decode throughput of layer-list decoders beside the closest decoder of the package at equal size.
 
-    python bench.py --layer-list [rurunex | supinex] [--steps K --warmup W]
+    python bench.py --layer-list [rurunex | supinex | vufinex] [--steps K --warmup W]
 
 Both run through the same engine classes with random weights.
   rurunex  repeats (gated linear attention, channel-wise delta rule, windowed attention), every layer with a gated
            feed-forward; beside the MoE decoder with a dense feed-forward in every layer and full attention: same width, heads,
            feed-forward and number of layers
   supinex  repeats (attention over everything, windowed latent attention), experts in every layer but the first; beside the MoE
+           decoder with the same width, heads, experts and number of layers
+  vufinex  repeats (RWKV-style time mixing, gated latent attention, chunked attention), experts in every layer; beside the MoE
            decoder with the same width, heads, experts and number of layers
 Prints one JSON line per (size, phase, model): tokens/s from device-timed steps (CUDA events, L2 flushed between steps), and
 one per (size, phase) with the device time per kernel.
@@ -20,7 +22,7 @@ from typing import Dict, List
 import torch
 
 from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec,
-                                  LayerListConfig, LayerSpec, ModelConfig, RotarySpec, RoutedSpec)
+                                  LayerListConfig, LayerSpec, ModelConfig, RotarySpec, RoutedSpec, WkvSpec)
 from disagmoe_b200.frontend.colocated import ColocatedEngine
 from disagmoe_b200.ops import _lib, gemm
 
@@ -59,11 +61,21 @@ def parallel_config(size: str, window: int = 1024, max_seq_len: int = 8192) -> L
     return LayerListConfig.make(W, VOCAB, layers, max_seq_len=max_seq_len, block="parallel", name="supinex-" + size)
 
 
-def moe_config(size: str, max_seq_len: int = 8192) -> ModelConfig:
+def prenorm_config(size: str, chunk: int = 1024, max_seq_len: int = 8192) -> LayerListConfig:
+    W, H, G, D, ff, n, rank, E, K = MOE_SIZES[size]
+    moe = RoutedSpec(E, K, ff, renormalize=True, scoring="sigmoid", correction=True, groups=8, keep=4, scale=2.0)
+    mixers = (WkvSpec(2 * H, D // 2, D // 2),
+              LatentAttentionSpec(H, D, D // 2, D, rank, (D + D // 2) ** -0.5, RotarySpec(D // 2, 1e6, interleaved=True), gate=True),
+              AttentionSpec(H, G, D, D, D ** -0.5, RotarySpec(D // 2, 5e5), qk_norm=False, chunk=chunk, tied_values=True))
+    return LayerListConfig.make(W, VOCAB, [LayerSpec(mixers[i % 3], routed=moe) for i in range(n)], max_seq_len=max_seq_len,
+                                block="prenorm", embed_scale=32.0, residual_mult=0.5, name="vufinex-" + size)
+
+
+def moe_config(size: str, max_seq_len: int = 8192, dense_layers: int = 1) -> ModelConfig:
     W, H, G, D, ff, n, _, E, K = MOE_SIZES[size]
     return ModelConfig(hidden_size=W, num_layers=n, num_heads=H, num_kv_heads=G, num_experts=E, intermediate_size=ff,
                        dtype=torch.bfloat16, ep_size=1, top_k=K, vocab_size=VOCAB, head_dim=D, rope_theta=5e5,
-                       norm_topk_prob=False, first_k_dense=1, dense_intermediate_size=4 * ff, max_seq_len=max_seq_len,
+                       norm_topk_prob=False, first_k_dense=dense_layers, dense_intermediate_size=4 * ff, max_seq_len=max_seq_len,
                        name="moe-" + size)
 
 
@@ -130,8 +142,9 @@ def main(args) -> int:
     flush = Flush()
     for size in (args.layer_list_sizes or "1024,2048,4096").split(","):
         for phase, n, length in (("prefill", 1, 4096), ("prefill", 4, 2048), ("decode", 16, 2048), ("decode", 256, 1024)):
-            for cfg in (hybrid_config(size), dense_config(size)) if args.layer_list == "rurunex" else \
-                    (parallel_config(size), moe_config(size)):
+            for cfg in {"rurunex": lambda: (hybrid_config(size), dense_config(size)),
+                        "supinex": lambda: (parallel_config(size), moe_config(size)),
+                        "vufinex": lambda: (prenorm_config(size), moe_config(size, dense_layers=0))}[args.layer_list]():
                 B = n if phase == "decode" else 8
                 eng = make_engine(cfg, B, n * length if phase == "prefill" else B, length if phase == "decode" else 16, 8)
                 ex = eng.executor

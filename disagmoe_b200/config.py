@@ -380,7 +380,29 @@ supinex_config = LayerListConfig.make(
     2048, 32000, _supinex_layers(8, 16, 128, 512, 5632, RoutedSpec(64, 6, 1408), 1024), max_seq_len=8192, block="parallel",
     architecture="Supinex", name="supinex-16l")
 
+# Vufinex design at the size of a small production model (random weights): RWKV-style time mixing, gated latent attention and
+# chunked attention in turn, every second attention layer on the weights of the one before it; grouped sigmoid routers.
+def _vufinex_layers(groups: int, heads: int, dim: int, rank: int, experts: RoutedSpec, chunk: int) -> List[LayerSpec]:
+    half = dim // 2
+    wkv = WkvSpec(2 * heads, half, half)
+    latent = LatentAttentionSpec(heads, dim, half, dim, rank, scale=(dim + half) ** -0.5, gate=True,
+                                 rot=RotarySpec(half, 1e6, interleaved=True))
+    attn = AttentionSpec(heads, max(1, heads // 4), dim, dim, scale=dim ** -0.5, rot=RotarySpec(half, 5e5), qk_norm=False,
+                         chunk=chunk, tied_values=True)
+    out: List[LayerSpec] = []
+    for g in range(groups):
+        out += [LayerSpec(m, routed=experts, weights_of=4 * (g - 1) + i if g % 2 and i == 3 else None)
+                for i, m in enumerate((wkv, latent, wkv, attn))]
+    return out
+
+
+vufinex_config = LayerListConfig.make(
+    2048, 32000, _vufinex_layers(4, 16, 128, 512, RoutedSpec(64, 6, 1408, renormalize=True, scoring="sigmoid", correction=True,
+                                                             groups=8, keep=3, scale=2.5), 1024),
+    max_seq_len=8192, block="prenorm", embed_scale=45.25, residual_mult=0.5, architecture="Vufinex", name="vufinex-16l")
+
 PRESETS = {
+    "vufinex": vufinex_config,
     "supinex": supinex_config,
     "rurunex": rurunex_config,
     "mixtral": mixtral_config, "mixtral-8x7b": mixtral_config, "duo": duo_expert_mixtral,
