@@ -1,6 +1,7 @@
-"""Recurrent layers alone: prompts (chunked kernels) and decode steps, gated linear attention and the channel-wise delta rule.
+"""Recurrent layers alone: prompts (chunked kernels) and decode steps; gated linear attention, the channel-wise delta rule and
+RWKV-style time mixing (wkv), the last with its token shift on its own.
 
-    python -m benchmark.ops.recurrence [--heads 16] [--dim 128] [--tokens 4096] [--batch 256]
+    python -m benchmark.ops.recurrence [--kinds gla,delta,wkv] [--heads 16] [--dim 128] [--tokens 4096] [--batch 256]
 
 Device time (CUDA events, L2 flushed in between) beside the bytes the operation has to move: projections in, output out and,
 for a decode step, every state read and written once.
@@ -15,6 +16,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))))
 
+from disagmoe_b200.ops import functional as F
 from disagmoe_b200.ops.recurrent import Recurrence, build_segments, decode_segments, recurrent_attention
 
 
@@ -22,6 +24,9 @@ def layer(kind, H, D, V, dev="cuda"):
     r = lambda *s: torch.randn(*s, device=dev)
     if kind == "gla":
         return Recurrence(H, H, D, V, False, r(H * D) + 2.0, 1 + 0.1 * r(V), 1e-6, tau=16.0)
+    if kind == "wkv":
+        return Recurrence(H, H, D, V, False, r(H * D) - 3.0, 1 + 0.1 * r(H * D), 1e-6, exp_decay=True, bonus=0.5 * r(H, D), qscale=1.0,
+                          shift_width=H * D)
     return Recurrence(H, H, D, V, True, 0.5 * r(H * D) - 4.0, 1 + 0.1 * r(V), 1e-6, a_log=0.3 * r(H),
                       conv_w=0.5 * r(2 * H * D + H * V, 4), sigmoid_gate=True)
 
@@ -35,11 +40,12 @@ def main():
     p.add_argument("--batch", type=int, default=256, help="decoding sequences")
     p.add_argument("--iters", type=int, default=10)
     p.add_argument("--only", default="", help="prompt | decode")
+    p.add_argument("--kinds", default="gla,delta,wkv")
     a = p.parse_args()
     H, D = a.heads, a.dim
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
     peak = json.load(open("MEASURED_PEAKS.json"))["hbm_gbs"] if os.path.exists("MEASURED_PEAKS.json") else 6650.0
-    for kind in ("gla", "delta"):
+    for kind in a.kinds.split(","):
         r = layer(kind, H, D, D)
         for phase in ("prompt", "decode"):
             if a.only not in ("", phase):
@@ -57,21 +63,31 @@ def main():
             else:
                 i = torch.arange(T, device="cuda")
                 segs = decode_segments(torch.full((T,), 100, dtype=torch.int32, device="cuda"), i.int(), i)
-            fn = lambda: recurrent_attention(r, q, k, v, gate, beta if kind == "delta" else None, z, state, segs)
-            ms = []
-            for it in range(a.iters + 3):
-                flush.zero_()
-                e = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
-                e[0].record()
-                fn()
-                e[1].record()
-                torch.cuda.synchronize()
-                ms.append(e[0].elapsed_time(e[1]))
-            t = statistics.median(ms[3:])
-            moved = T * H * D * (2 * 5 + 4) + (2 * state.S.numel() * 4 if phase == "decode" else 0)
-            print(json.dumps({"kind": kind, "phase": phase, "tokens": T, "heads": H, "dim": D, "us": round(t * 1e3, 1),
-                              "MB": round(moved / 1e6, 1), "GB_s": round(moved / t / 1e6), "of_measured_copy": round(moved / t / 1e6 / peak, 3)}),
-                  flush=True)
+            cases = [(kind, T * H * D * (2 * 5 + 4) + (2 * state.S.numel() * 4 if phase == "decode" else 0),
+                      lambda: recurrent_attention(r, q, k, v, gate, beta if kind == "delta" else None, z, state, segs))]
+            if kind == "wkv":
+                W = H * D
+                mu, w, resid = torch.rand(5, W, device="cuda"), torch.ones(W, device="cuda"), torch.randn(T, W, device="cuda")
+                shift = F.TokenShift(mu, state.last, segs)
+                if phase == "prompt":
+                    cases.append(("token shift", T * W * (4 + 5 * 2), lambda: F.token_shift(resid, shift, torch.bfloat16)))
+                else:
+                    cases.append(("norm + token shift", T * W * (4 + 5 * 2 + 8),
+                                  lambda: F.sum_norm(resid, None, None, w, 1e-6, torch.bfloat16, False, shift=shift)))
+            for name, moved, fn in cases:
+                ms = []
+                for it in range(a.iters + 3):
+                    flush.zero_()
+                    e = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+                    e[0].record()
+                    fn()
+                    e[1].record()
+                    torch.cuda.synchronize()
+                    ms.append(e[0].elapsed_time(e[1]))
+                t = statistics.median(ms[3:])
+                print(json.dumps({"kind": name, "phase": phase, "tokens": T, "heads": H, "dim": D, "us": round(t * 1e3, 1),
+                                  "MB": round(moved / 1e6, 1), "GB_s": round(moved / t / 1e6),
+                                  "of_measured_copy": round(moved / t / 1e6 / peak, 3)}), flush=True)
 
 
 if __name__ == "__main__":

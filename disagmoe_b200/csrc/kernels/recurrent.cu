@@ -206,10 +206,10 @@ step_kernel(const DmoeRecur a, int vt) {
 }
 
 // Decode steps at full bandwidth: one CTA per (sequence, head), the head's state fetched by one bulk copy into shared memory
-// while the token's inputs are prepared (three CTAs per SM keep copies in flight), updated from there straight back to
-// global memory. One-token segments, whole heads, vdim a multiple of 4.
-template <typename T, int MODE, bool CONV>
-__global__ void __launch_bounds__(kStepThreads, 3)
+// while the token's inputs are prepared (three CTAs per SM, six of half the threads for small states, keep copies in flight),
+// updated from there straight back to global memory. One-token segments, whole heads, vdim a multiple of 4.
+template <typename T, int MODE, bool CONV, int NT>
+__global__ void __launch_bounds__(NT, 3 * kStepThreads / NT)
 stream_step_kernel(const DmoeRecur a) {
   constexpr bool DELTA = MODE == kDelta;
   extern __shared__ __align__(128) float s_stream[];
@@ -240,7 +240,7 @@ stream_step_kernel(const DmoeRecur a) {
                    "l"(sp), "r"(bytes), "r"(bar) : "memory");
     }
   }
-  const int vq = V / 4, rpp = kStepThreads / vq, cg = tid % vq, rg = tid / vq;
+  const int vq = V / 4, rpp = NT / vq, cg = tid % vq, rg = tid / vq;
   const bool mine = rg < rpp;
   const float* norm_w = a.norm_w + h * a.norm_ld;
   float beta = 0.f, gate = 0.f, weight = 0.f;
@@ -278,7 +278,7 @@ stream_step_kernel(const DmoeRecur a) {
     for (int i = 0; i < (1 << 20) && !mbar_try_wait(bar, 0); ++i) {}
     return;
   }
-  for (int c = tid; c < V; c += kStepThreads) {
+  for (int c = tid; c < V; c += NT) {
     float oq = 0.f, ok = 0.f;
 #pragma unroll 4
     for (int r = 0; r < rpp; ++r) {
@@ -305,7 +305,7 @@ stream_step_kernel(const DmoeRecur a) {
   float ss = 0.f;
   for (int c = lane; c < V; c += 32) ss += s_o[c] * s_o[c];
   const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + a.eps);
-  for (int c = tid; c < V; c += kStepThreads) {
+  for (int c = tid; c < V; c += NT) {
     if (c != tid) {                                              // heads wider than the CTA
       gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + c]);
       weight = norm_w[c];
@@ -315,15 +315,22 @@ stream_step_kernel(const DmoeRecur a) {
 }
 
 // out[row, h, :] = raw / sqrt(mean(raw^2) + eps) * norm_w * gate for the rows of a table (segs or chunks; NULL: entry i is
-// row i); one warp per (row, head), VEC consecutive columns per lane and pass
+// row i); `lanes` (a power of two) threads per (row, head), VEC consecutive columns per lane and pass
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, long long ldraw, const T* __restrict__ gate,
                  long long ldg, const float* __restrict__ norm_w, int norm_ld, float eps, int gate_kind, T* __restrict__ out,
-                 long long ldo, int heads, int V) {
+                 long long ldo, int heads, int V, int lanes) {
   const int4 e = table != nullptr ? table[blockIdx.x] : make_int4(blockIdx.x, 1, 0, 0);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-  for (int i = blockIdx.y * warps + warp; i < e.y * heads; i += gridDim.y * warps) {
+  const int lane = threadIdx.x & (lanes - 1), per = blockDim.x / lanes;       // (row, head) pairs of the CTA at a time
+  const auto sum = [&](float v) {                // over the lanes of a pair; the whole warp takes part
+    for (int o = lanes / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+  };
+  const int pairs = e.y * heads;
+  for (int i0 = blockIdx.y * per; i0 < pairs; i0 += gridDim.y * per) {
+    const bool on = i0 + static_cast<int>(threadIdx.x) / lanes < pairs;
+    const int i = on ? i0 + threadIdx.x / lanes : pairs - 1;
     const long long row = e.x + i / heads;
     const int h = i % heads;
     const float* r = raw + row * ldraw + h * V;
@@ -339,14 +346,14 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
 #pragma unroll
       for (int k = 0; k < VEC; ++k) ss += x[k] * x[k];
     }
-    for (int c = c0 + 32 * VEC; c < V; c += 32 * VEC) {
+    for (int c = c0 + lanes * VEC; c < V; c += lanes * VEC) {
       float y[VEC];
       load_vec<VEC>(r + c, y);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) ss += y[k] * y[k];
     }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
-    for (int c = c0; c < V; c += 32 * VEC) {
+    const float inv = 1.f / sqrtf(sum(ss) / static_cast<float>(V) + eps);
+    for (int c = on ? c0 : V; c < V; c += lanes * VEC) {
       if (c != c0) {
         load_vec<VEC>(r + c, x);
         load_any<VEC>(gp + c, gv);
@@ -447,27 +454,36 @@ static int check_recur(const DmoeRecur* a) {
 }
 
 constexpr int kStreamSmem = 76400;       // three CTAs per SM
+constexpr int kSmallState = 32 * 1024;   // states up to here take half the threads, six CTAs per SM
 
 // Shared memory of stream_step_kernel, or 0 where it does not apply: whole heads of a multiple of 4 value columns whose
 // state leaves room for three CTAs per SM.
+static int stream_threads(const DmoeRecur& a) {
+  return a.dim * a.vdim * 4 <= kSmallState && a.vdim <= 2 * kStepThreads ? kStepThreads / 2 : kStepThreads;
+}
 static size_t stream_smem(const DmoeRecur& a) {
   if (a.raw != nullptr || a.vdim % 4 != 0 || a.vdim > 4 * kStepThreads || (reinterpret_cast<uintptr_t>(a.state) & 15) != 0)
     return 0;
-  const int rpp = kStepThreads / (a.vdim / 4);
+  const int rpp = stream_threads(a) / (a.vdim / 4);
   const size_t b = (static_cast<size_t>(a.dim) * a.vdim + 4 * a.dim + a.vdim + static_cast<size_t>(a.delta ? 2 : 1) * rpp * a.vdim) * 4;
   return b <= kStreamSmem ? b : 0;
 }
 
-template <typename T, int MODE, bool CONV>
-static int launch_stream(const DmoeRecur& a, size_t smem, cudaStream_t stream) {
+template <typename T, int MODE, bool CONV, int NT>
+static int launch_stream_nt(const DmoeRecur& a, size_t smem, cudaStream_t stream) {
   static PerDeviceOnce configured;
   const int rc = configured.run([] {
-    return static_cast<int>(cudaFuncSetAttribute(stream_step_kernel<T, MODE, CONV>,
+    return static_cast<int>(cudaFuncSetAttribute(stream_step_kernel<T, MODE, CONV, NT>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, kStreamSmem));
   });
   if (rc != 0) return rc;
-  return static_cast<int>(launch_kernel(stream_step_kernel<T, MODE, CONV>, dim3(a.n_segs, a.heads), dim3(kStepThreads), smem,
+  return static_cast<int>(launch_kernel(stream_step_kernel<T, MODE, CONV, NT>, dim3(a.n_segs, a.heads), dim3(NT), smem,
                                         stream, a));
+}
+template <typename T, int MODE, bool CONV>
+static int launch_stream(const DmoeRecur& a, size_t smem, cudaStream_t stream) {
+  return stream_threads(a) == kStepThreads ? launch_stream_nt<T, MODE, CONV, kStepThreads>(a, smem, stream)
+                                           : launch_stream_nt<T, MODE, CONV, kStepThreads / 2>(a, smem, stream);
 }
 
 template <typename T, int MODE, bool CONV, int VEC>
@@ -540,10 +556,12 @@ extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_toke
   const dim3 grid(n, static_cast<unsigned>(by));
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec = V % 4 == 0 && norm_ld % 4 == 0 && ldraw % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(raw) && al(gate) && al(out) && al(norm_w);
+  int lanes = 32;
+  while (lanes > 4 && (lanes / 2) * (vec ? 4 : 1) >= V) lanes /= 2;
 #define DMOE_GATE_NORM(T_, VEC_)                                                                                       \
   gate_norm_kernel<T_, VEC_><<<grid, 256, 0, stream>>>(static_cast<const int4*>(table), raw, ldraw,                    \
                                                        static_cast<const T_*>(gate), ldg, norm_w, norm_ld, eps, gate_kind, \
-                                                       static_cast<T_*>(out), ldo, heads, V)
+                                                       static_cast<T_*>(out), ldo, heads, V, lanes)
   if (is_f32) {
     if (vec) DMOE_GATE_NORM(float, 4);
     else DMOE_GATE_NORM(float, 1);

@@ -18,7 +18,9 @@
 // Precision: decays, their sums and exponentials, unit norms, T and the state are fp32; matrix products split both
 // operands into bf16 hi + lo parts and accumulate in fp32 (see mma_sync.cuh). P and A are products of rows scaled by
 // e^(b_t - m) and e^(m - b_j), m = b in the middle of the chunk; where a channel decays so fast that these could
-// overflow (more than 2^60 either way), the pairwise exponentials are evaluated one by one.
+// overflow (more than 2^60 either way), the pairwise exponentials are evaluated one by one. With a bonus (decays are free there
+// and often fast) the scale is that of the key's tile of 16 tokens: q e^(b_(t-1) - m) and k e^(m - b_j), m = b at the tile's end,
+// are at most 1 but inside the tile itself, so that only 2^100 within 16 tokens is too fast, and then for the tiles on the diagonal.
 #include "mma_sync.cuh"
 #include "recurrent.cuh"
 
@@ -28,6 +30,7 @@ constexpr int kChunk = 64;
 constexpr int kChunkThreads = 256;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kMaxShift = 60.f;          // log2 units
+constexpr float kMaxTileShift = 100.f;
 constexpr int kMid = 31;
 constexpr int kPs = kChunk + 8;            // row stride (elements) of 64-column bf16 tiles in shared memory
 
@@ -147,11 +150,12 @@ struct PrepSmem {
   static constexpr int kKs = DP + 8;
   static constexpr int kKn = 2 * kChunk * kKs * 2, kTX = DELTA ? 4 * kChunk * kPs * 2 : 0;
   static constexpr int kRegion = kKn > kTX ? kKn : kTX;
-  static constexpr int kBytes = 4 * kChunk * DP + 3 * 4 * kChunk + kRegion + (DELTA ? 2 * 4 * kChunk * (kChunk + 1) : 0) + 16;
+  static constexpr int kBytes = 4 * kChunk * DP + 3 * 4 * kChunk + kRegion + (DELTA ? 2 * 4 * kChunk * (kChunk + 1) : 0) +
+                                (MODE == kBonus ? 4 * 4 * DP : 0) + 16;
 };
 
 template <int DP, int MODE>
-__global__ void __launch_bounds__(kChunkThreads, 2)
+__global__ void __launch_bounds__(kChunkThreads, MODE == kBonus && DP <= 64 ? 3 : 2)
 chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* __restrict__ ws, long long ws_stride, int h0) {
   using L = ChunkWs<DP>;
   using SM = PrepSmem<DP, MODE>;
@@ -167,6 +171,7 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   __nv_bfloat16* s_kl = s_kh + kChunk * SM::kKs;
   float* s_A = reinterpret_cast<float*>(region + SM::kRegion);
   float* s_T = s_A + kChunk * LDA;
+  float* s_step = s_A;                                          // bonus: [4][DP] decay over tile i of 16 tokens
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int lm_mi = lane >> 3, lm_r = lane & 7;
@@ -259,7 +264,18 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   bool wide = false;
   if (tid < DP) {
     const float m = s_b[kMid * DP + tid];
-    wide = (BONUS ? 0.f : s_b[tid]) - m > kMaxShift || m - s_b[(kChunk - 1) * DP + tid] > kMaxShift;
+    if (BONUS) {
+      float from = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float end = s_b[(16 * i + 15) * DP + tid];
+        wide = wide || from - end > kMaxTileShift;
+        s_step[i * DP + tid] = exp2f(end - from);
+        from = end;
+      }
+    } else {
+      wide = s_b[tid] - m > kMaxShift || m - s_b[(kChunk - 1) * DP + tid] > kMaxShift;
+    }
     reinterpret_cast<float*>(w + L::kDec)[tid] = exp2f(s_b[(kChunk - 1) * DP + tid]);
   }
   const bool slow = __syncthreads_or(wide);
@@ -271,9 +287,19 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
       store_split<PL>(s_kh + (t0 + i) * SM::kKs + d0, s_kl + (t0 + i) * SM::kKs + d0, k[i]);
   };
   float to_mid[PL];                                  // e^(m - b_end)
+  float k_tile[BONUS ? ROWS : 1][PL];                // k e^(b at the end of its tile - b)
 #pragma unroll
   for (int e = 0; e < PL; ++e) {
     const float end = s_b[(kChunk - 1) * DP + d0 + e];
+    if (BONUS) {
+      const float tile = s_b[(warp / 2 * 16 + 15) * DP + d0 + e], rest = exp2f(end - tile);
+#pragma unroll
+      for (int i = 0; i < ROWS; ++i) {
+        k_tile[BONUS ? i : 0][e] = k[i][e] * exp2f(tile - s_b[(t0 + i) * DP + d0 + e]);
+        k[i][e] = k_tile[BONUS ? i : 0][e] * rest;
+      }
+      continue;
+    }
     to_mid[e] = slow ? 0.f : exp2f(s_b[kMid * DP + d0 + e] - end);
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) k[i][e] *= exp2f(end - s_b[(t0 + i) * DP + d0 + e]);
@@ -290,17 +316,104 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
     store_frag(w + L::kK + (i * 2 + 1) * kFrag, lane, f);
   }
   __syncthreads();
-  if (!slow) {                                       // now k e^(m - b): right operand of P and A
+  if (BONUS || !slow) {                              // now k e^(m - b): right operand of P and A
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
 #pragma unroll
-      for (int e = 0; e < PL; ++e) k[i][e] *= to_mid[e];
+      for (int e = 0; e < PL; ++e) k[i][e] = BONUS ? k_tile[BONUS ? i : 0][e] : k[i][e] * to_mid[e];
     stage_k();
   }
   __syncthreads();
 
-  // ---- P and the fragments of q e^b (warps 0-3), A (warps 4-7)
-  {
+  // ---- P and the fragments of q e^b. With a bonus warp w and w + 4 share the row tile mi: the upper and the lower half of its key
+  // tiles. q's scale starts at the end of the warp's first tile and steps down to the others', at last to the chunk's start.
+  if (BONUS) {
+    const int mi = warp & 3, r0 = mi * 16 + g, r1 = r0 + 8;
+    const int top = warp < 4 ? mi : (mi - 1) / 2, low = warp < 4 ? (mi + 1) / 2 : 0;      // key tiles top .. low
+    const bool to_start = low == 0;
+    const int skip = slow && warp < 4 ? 1 : 0;       // too fast: the diagonal tile is left to the pairwise path below
+    const int from = top - skip;                     // tile whose end is the first scale, -1: the chunk's start
+    if (warp < 4 || mi > 0) {
+      float acc[2][2][4];                            // [top - kg][8-column half]
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][0][e] = acc[i][1][e] = 0.f;
+      const uint32_t bh = smem_u32(s_kh), bl = smem_u32(s_kl);
+#pragma unroll
+      for (int kb = 0; kb < KS; kb += 4) {           // raw values of up to four k tiles in flight
+        uint32_t raw[4][4];
+#pragma unroll
+        for (int kk = 0; kk < 4 && kb + kk < KS; ++kk)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int r = j & 1 ? r1 : r0, c = (kb + kk) * 16 + 2 * tq + (j >> 1) * 8;
+            raw[kk][j] = r < n && c < D ? *reinterpret_cast<const uint32_t*>(qp + r * a.ldq + c) : 0u;
+          }
+#pragma unroll
+        for (int kk = 0; kk < 4 && kb + kk < KS; ++kk) {
+          const int ks = kb + kk;
+          float2 x[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int r = j & 1 ? r1 : r0, c = ks * 16 + 2 * tq + (j >> 1) * 8;
+            x[j] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[kk][j]));
+            float2 b = make_float2(0.f, 0.f);
+            if (r > 0) b = *reinterpret_cast<const float2*>(s_b + (r - 1) * DP + c);
+            float2 m = make_float2(0.f, 0.f);
+            if (from >= 0) m = *reinterpret_cast<const float2*>(s_b + (16 * from + 15) * DP + c);
+            x[j].x *= a.qscale * exp2f(b.x - m.x);
+            x[j].y *= a.qscale * exp2f(b.y - m.y);
+          }
+          uint32_t ah[4], al[4];
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int kg = top - i;
+            if (kg < low) break;
+            if (i < skip) continue;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) split2(x[j].x, x[j].y, ah[j], al[j]);
+            const uint32_t off = ((kg * 16 + (lm_mi >> 1) * 8 + lm_r) * SM::kKs + ks * 16 + (lm_mi & 1) * 8) * 2;
+            uint32_t h0_, h1_, h2_, h3_, l0_, l1_, l2_, l3_;
+            ldmatrix_x4(bh + off, h0_, h1_, h2_, h3_);
+            ldmatrix_x4(bl + off, l0_, l1_, l2_, l3_);
+            mma_split(acc[i][0], ah, al, h0_, h1_, l0_, l1_);
+            mma_split(acc[i][1], ah, al, h2_, h3_, l2_, l3_);
+            if (kg > low || to_start) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const float2 st = *reinterpret_cast<const float2*>(s_step + kg * DP + ks * 16 + 2 * tq + (j >> 1) * 8);
+                x[j].x *= st.x;
+                x[j].y *= st.y;
+              }
+            }
+          }
+          if (to_start) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) split2(x[j].x, x[j].y, ah[j], al[j]);
+            store_frag(w + L::kQ + (mi * KS + ks) * 2 * kFrag, lane, ah);
+            store_frag(w + L::kQ + ((mi * KS + ks) * 2 + 1) * kFrag, lane, al);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int kg = top - i;
+        if (kg < low) break;
+        if (i < skip) continue;
+        if (kg == mi) {
+#pragma unroll
+          for (int h8 = 0; h8 < 2; ++h8)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {            // strictly below the diagonal, and the bonus on it
+              const int r = e < 2 ? r0 : r1, c = kg * 16 + h8 * 8 + 2 * tq + (e & 1);
+              acc[i][h8][e] = c < r ? acc[i][h8][e] : c == r ? s_beta[r] : 0.f;
+            }
+        }
+        store_acc_frag(w + L::kP + (mi * 4 + kg) * 2 * kFrag, lane, acc[i][0], acc[i][1]);
+      }
+    }
+  } else {                                           // warps 0-3; A (warps 4-7)
     const int mi = warp & 3;
     const bool second = warp >= 4;
     if (!second || (DELTA && !slow)) {
@@ -333,9 +446,7 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
             float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[kk][j]));
             x.x *= f;
             x.y *= f;
-            float2 b = make_float2(0.f, 0.f);
-            if (second || !BONUS) b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
-            else if (r > 0) b = *reinterpret_cast<const float2*>(s_b + (r - 1) * DP + c);
+            const float2 b = *reinterpret_cast<const float2*>(s_b + r * DP + c);
             const float2 m = *reinterpret_cast<const float2*>(s_b + kMid * DP + c);
             split2(x.x * exp2f(b.x - m.x), x.y * exp2f(b.y - m.y), ah[j], al[j]);
             if (!second) split2(x.x * exp2f(b.x), x.y * exp2f(b.y), zh[j], zl[j]);
@@ -361,17 +472,11 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
       if (!slow) {
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) {
-          const int c = nt * 8 + 2 * tq, edge = second || BONUS ? -1 : 0;        // A is strictly below the diagonal
+          const int c = nt * 8 + 2 * tq, edge = second ? -1 : 0;        // A is strictly below the diagonal
           if (c > r0 + edge) acc[nt][0] = 0.f;
           if (c + 1 > r0 + edge) acc[nt][1] = 0.f;
           if (c > r1 + edge) acc[nt][2] = 0.f;
           if (c + 1 > r1 + edge) acc[nt][3] = 0.f;
-          if (BONUS) {
-            if (c == r0) acc[nt][0] = s_beta[r0];
-            if (c + 1 == r0) acc[nt][1] = s_beta[r0];
-            if (c == r1) acc[nt][2] = s_beta[r1];
-            if (c + 1 == r1) acc[nt][3] = s_beta[r1];
-          }
           if (DELTA && second) {
             s_A[r0 * LDA + c] = acc[nt][0] * s_beta[r0];
             s_A[r0 * LDA + c + 1] = acc[nt][1] * s_beta[r0];
@@ -388,8 +493,8 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
     }
   }
   if (slow) {
-    for (int i = tid; i < kChunk * kChunk; i += kChunkThreads) {
-      const int t = i / kChunk, j = i % kChunk;
+    for (int i = tid; i < (BONUS ? kChunk * 16 : kChunk * kChunk); i += kChunkThreads) {
+      const int t = BONUS ? i / 16 : i / kChunk, j = BONUS ? i / 256 * 16 + i % 16 : i % kChunk;
       float p = 0.f, kk = 0.f;
       if ((BONUS ? j < t : j <= t) && t < n) {
         const int tr = BONUS ? t - 1 : t;              // place of the read-out

@@ -106,7 +106,7 @@ def _vufinex_layer(i: int, layer: dict, j: int, shapes: Dict[str, Tuple[int, ...
         r = mlp["router"]
         g = r.get("groups") or {"count": 1, "keep": 1}
         routed = RoutedSpec(r["experts"], r["top"], mlp["expert"]["ff"], renormalize=True, scoring="sigmoid", correction=True,
-                            groups=g["count"], keep=g["keep"], scale=float(r["scale"]))
+                            groups=g["count"], keep=g["keep"], scale=float(r.get("scale", 1.0)))
     return LayerSpec(mixer, routed=routed, weights_of=layer.get("weights_of"))
 
 
