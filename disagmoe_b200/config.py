@@ -185,9 +185,9 @@ class WkvSpec:
 class RoutedSpec:
     """Feed-forward of ``experts`` gated feed-forwards of width ``ff``; a token uses the ``top`` ones with the largest
     scores, weighted by these scores (``renormalize``: divided by their sum) times ``scale``. ``scoring``: "softmax", or
-    "sigmoid" of every logit; ``correction``: a stored number per expert is added for the choice alone (sigmoid scores);
-    ``groups`` / ``keep``: experts form equal groups of neighbours and only those of the ``keep`` groups whose two best choice
-    scores have the largest sum can be chosen (sigmoid scores)."""
+    "sigmoid" of every logit. With sigmoid scores, ``correction``: a stored number per expert enters the choice, not the weight;
+    ``groups`` / ``keep``: the list of experts is cut into ``groups`` runs of one length, ranked by the sum of their two best
+    corrected scores, and a token chooses within the first ``keep`` of them."""
     experts: int
     top: int
     ff: int
@@ -206,7 +206,7 @@ class LayerSpec:
     ff: Optional[int] = None                    # width of the dense gated feed-forward, None = the layer has none
     act: str = "silu"                           # of the dense feed-forward: silu or gelu_tanh
     routed: Optional[RoutedSpec] = None         # experts instead of a dense feed-forward
-    weights_of: Optional[int] = None            # the layer whose tensors this one uses, with a cache or state of its own
+    weights_of: Optional[int] = None            # the layer that lends this one its tensors (caches and states stay per layer)
 
 
 @dataclass

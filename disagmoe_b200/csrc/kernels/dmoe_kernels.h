@@ -8,7 +8,7 @@
 extern "C" {
 
 // Router of dmoe_sum_norm (weight [E, W] in the activations' dtype): softmax scores or, sigmoid = 1, sigmoid scores with a
-// correction (NULL: none) that counts for the choice alone, inside the best `keep` of `groups` equal groups of neighbours.
+// correction (NULL: none) that enters the choice, not the weight, within the best `keep` of `groups` runs of E / groups experts.
 typedef struct DmoeRouter {
   const void* weight;
   const float* correction;  // [E]

@@ -9,7 +9,7 @@ from disagmoe_b200.models import weights as W
 from disagmoe_b200.models.registry import load_model, vufinex_config_from_json
 from layer_list_util import error, feed, tokens
 from oracles import prenorm_stack as oracle
-from prenorm_util import MODELS, again, attn, latent, make_engine, model, moe, wkv
+from prenorm_util import MODELS, attn, make_engine, model, wkv
 
 TOL = 2e-5
 
