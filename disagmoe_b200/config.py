@@ -7,7 +7,7 @@ layers) and what the Blackwell kernels need to know.
 from __future__ import annotations
 
 from dataclasses import dataclass, field, replace
-from typing import List, Optional, Union
+from typing import List, Optional, Tuple, Union
 
 import torch
 
@@ -80,6 +80,7 @@ class ModelConfig:
 
 
 ACTIVATIONS = ("silu", "gelu_tanh")             # of gated feed-forwards
+EXPERT_ACTIVATIONS = ACTIVATIONS + ("clamped",)     # of experts: also min(g, limit) sigmoid(1.702 g) (clamp(u, limit) + 1)
 
 
 # ---- decoders described layer by layer --------------------------------------------------------------------------------
@@ -100,13 +101,22 @@ class RotarySpec:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """Scores of the query at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: int
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
     """Softmax attention. ``window``: how many of the latest tokens, its own included, a query attends to (None: all).
     ``chunk``: positions fall into chunks of that size, counted from 0, and a query attends to its own chunk only.
     ``kv_from``: the earlier layer whose cached keys and values this layer reads (it then has none). ``qk_norm``: RMS norm
     of every query and key head. ``sink``: a learned number per head enters the softmax denominator. ``v_mix``: the values
     are mixed with those that the first such layer computed for the same token. ``tied_values``: the values are the keys before
-    their rotation (vdim = dim, no map of their own)."""
+    their rotation (vdim = dim, no map of their own). ``value_norm``: every value head is divided by its root mean square before it
+    is cached. ``gate``: every head's output is scaled by the sigmoid of a linear map of the layer's input. ``q_temp``: query
+    temperature by position."""
     heads: int
     kv_heads: int
     dim: int
@@ -121,6 +131,9 @@ class AttentionSpec:
     v_mix: bool = False
     chunk: Optional[int] = None
     tied_values: bool = False
+    value_norm: bool = False
+    gate: bool = False
+    q_temp: Optional[QueryTemperature] = None
 
 
 @dataclass(frozen=True)
@@ -182,12 +195,81 @@ class WkvSpec:
 
 
 @dataclass(frozen=True)
+class HeadDecaySpec:
+    """Lightning attention: linear attention with silu on queries, keys and values and one constant decay per head; all heads'
+    read-outs are normed together and gated."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory of xLSTM: exponential input gate and sigmoid forget gate per head and token, logits soft-capped at
+    ``gate_cap``; beside the state a normaliser and a running maximum per head."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+
+@dataclass(frozen=True)
+class GatedUnitSpec:
+    """Griffin's recurrent block: a branch through a short convolution of ``conv`` taps and a real-gated diagonal recurrence of
+    ``width`` channels, multiplied by a gelu branch. The two gates are linear within each of the ``blocks`` equal parts."""
+    width: int
+    blocks: int
+    conv: int
+
+    @property
+    def heads(self) -> int:
+        return self.blocks
+
+    @property
+    def kv_heads(self) -> int:
+        return self.blocks
+
+    @property
+    def dim(self) -> int:
+        return self.width // self.blocks
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    """Two mixers on the same rows; the result is half the sum of their outputs, each normed over the model width first."""
+    left: AttentionSpec
+    right: MatrixMemorySpec
+
+    @property
+    def heads(self) -> int:
+        return max(self.left.heads, self.right.heads)
+
+    @property
+    def dim(self) -> int:
+        return max(self.left.dim, self.right.dim)
+
+
+@dataclass(frozen=True)
 class RoutedSpec:
     """Feed-forward of ``experts`` gated feed-forwards of width ``ff``; a token uses the ``top`` ones with the largest
     scores, weighted by these scores (``renormalize``: divided by their sum) times ``scale``. ``scoring``: "softmax", or
     "sigmoid" of every logit. With sigmoid scores, ``correction``: a stored number per expert enters the choice, not the weight;
     ``groups`` / ``keep``: the list of experts is cut into ``groups`` runs of one length, ranked by the sum of their two best
-    corrected scores, and a token chooses within the first ``keep`` of them."""
+    corrected scores, and a token chooses within the first ``keep`` of them. ``limit``: of the "clamped" activation.
+    ``weigh_input``: the weight scales what an expert reads, not what it returns."""
     experts: int
     top: int
     ff: int
@@ -198,11 +280,14 @@ class RoutedSpec:
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
+    limit: float = 0.0
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, ChannelDeltaSpec, WkvSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, ChannelDeltaSpec, WkvSpec, HeadDecaySpec, GatedUnitSpec,
+                 SideBySideSpec]
     ff: Optional[int] = None                    # width of the dense gated feed-forward, None = the layer has none
     act: str = "silu"                           # of the dense feed-forward: silu or gelu_tanh
     routed: Optional[RoutedSpec] = None         # experts instead of a dense feed-forward
@@ -218,6 +303,10 @@ class LayerListConfig(ModelConfig):
       "sandwich"  x += post(mixer(pre(x))), then x += post(ff(pre(x))); RMS norms whose stored weight is an offset from one
       "parallel"  h = norm(x); x += mixer(h) + ff(h); layer norms (mean taken off) with a plain weight
       "prenorm"   x += m mixer(pre(x)), then x += m ff(pre(x)), m = ``residual_mult``; RMS norms as in "sandwich"
+    Options of pre-norm blocks: ``layer_norm`` (norms take the mean off and have a plain weight and a bias), ``residual_gate`` (every
+    sublayer's result is multiplied by sigmoid(W h + b), h = its normed input), ``input_conv`` taps > 0 (the mixer reads h + a
+    causal convolution of h per channel). Of the whole model: ``positions`` > 0 learned position vectors, ``tied_head`` (the
+    head is the embedding table).
     """
     layers: List[LayerSpec] = field(default_factory=list)
     embed_scale: float = 1.0
@@ -225,6 +314,11 @@ class LayerListConfig(ModelConfig):
     architecture: str = ""
     block: str = "sandwich"
     residual_mult: float = 1.0
+    layer_norm: bool = False
+    residual_gate: bool = False
+    input_conv: int = 0
+    positions: int = 0
+    tied_head: bool = False
 
     def is_dense_layer(self, layer_id: int) -> bool:
         return True
@@ -232,9 +326,25 @@ class LayerListConfig(ModelConfig):
     def __post_init__(self):
         super().__post_init__()
         assert self.num_layers == len(self.layers) and self.block in ("sandwich", "parallel", "prenorm")
+        if self.block != "prenorm" and (self.layer_norm or self.residual_gate or self.input_conv):
+            raise ValueError("layer norms with a bias, gated residuals and input convolutions need pre-norm blocks")
+        if self.positions:
+            self.max_seq_len = min(self.max_seq_len, self.positions)
         for i, layer in enumerate(self.layers):
             m, r = layer.mixer, layer.routed
-            if layer.act not in ACTIVATIONS or (r is not None and r.act not in ACTIVATIONS):
+            if isinstance(m, HeadDecaySpec) and (len(m.decay) != m.heads or not all(0.0 <= d <= 1.0 for d in m.decay)):
+                raise ValueError(f"layer {i}: {m.heads} heads need one decay in 0 .. 1 each")
+            if isinstance(m, GatedUnitSpec) and m.width % m.blocks:
+                raise ValueError(f"layer {i}: {m.width} channels do not make {m.blocks} equal blocks")
+            if r is not None and r.act == "clamped" and r.limit <= 0.0:
+                raise ValueError(f"layer {i}: clamped experts need a limit")
+            if isinstance(m, SideBySideSpec):
+                m = m.left
+                if m.kv_from is not None or m.v_mix:
+                    raise ValueError(f"layer {i}: attention beside another mixer shares no keys or values")
+            if getattr(m, "q_temp", None) is not None and m.q_temp.every < 1:
+                raise ValueError(f"layer {i}: the query temperature changes every {m.q_temp.every} tokens")
+            if layer.act not in ACTIVATIONS or (r is not None and r.act not in EXPERT_ACTIVATIONS):
                 raise ValueError(f"layer {i}: unknown activation (known: {', '.join(ACTIVATIONS)})")
             if r is not None and (layer.ff or self.block == "sandwich" or not 1 <= r.top <= r.experts):
                 raise ValueError(f"layer {i}: experts need a parallel or pre-norm block, no dense feed-forward beside them and "
@@ -251,10 +361,12 @@ class LayerListConfig(ModelConfig):
             rot = getattr(m, "rot", None)
             if rot is not None and (rot.dims % 2 or rot.dims > (m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim)):
                 raise ValueError(f"layer {i}: {rot.dims} rotated dimensions do not fit the head")
-            if isinstance(m, (GatedLinearSpec, LatentAttentionSpec, WkvSpec)):
+            if isinstance(m, (GatedLinearSpec, LatentAttentionSpec, WkvSpec, HeadDecaySpec, GatedUnitSpec)):
                 continue
-            if getattr(m, "tied_values", False) and (m.vdim != m.dim or m.v_mix or m.kv_from is not None or m.qk_norm):
+            if getattr(m, "tied_values", False) and (m.vdim != m.dim or m.v_mix or m.kv_from is not None or m.qk_norm or m.value_norm):
                 raise ValueError(f"layer {i}: values tied to the keys have their size and no norm, mixing or sharing")
+            if getattr(m, "value_norm", False) and (m.v_mix or m.kv_from is not None):
+                raise ValueError(f"layer {i}: normed values are neither mixed nor read from another layer")
             if m.heads % m.kv_heads:
                 raise ValueError(f"layer {i}: {m.heads} heads do not share {m.kv_heads} key / value heads evenly")
             src = getattr(m, "kv_from", None)
@@ -401,7 +513,23 @@ vufinex_config = LayerListConfig.make(
                                                              groups=8, keep=3, scale=2.5), 1024),
     max_seq_len=8192, block="prenorm", embed_scale=45.25, residual_mult=0.5, architecture="Vufinex", name="vufinex-16l")
 
+# Panarax design at the size of a small production model (random weights): attention beside a matrix memory, a gated diagonal
+# recurrence and lightning attention in turn; the first of the three has a dense feed-forward, the others experts.
+def _panarax_layers(groups: int, heads: int, dim: int, ff: int, experts: RoutedSpec) -> List[LayerSpec]:
+    both = SideBySideSpec(AttentionSpec(heads, max(1, heads // 4), dim, dim, scale=dim ** -0.5, qk_norm=False, value_norm=True, gate=True,
+                                        q_temp=QueryTemperature(0.1, 1024)), MatrixMemorySpec(heads // 2, dim, dim, 15.0))
+    unit = GatedUnitSpec(heads * dim, heads, 4)
+    decays = HeadDecaySpec(heads, dim, dim, tuple(2.718281828459045 ** -(2.0 ** (-8.0 * (i + 1) / heads)) for i in range(heads)))
+    return [LayerSpec(both, ff), LayerSpec(unit, routed=experts), LayerSpec(decays, routed=experts)] * groups
+
+
+panarax_config = LayerListConfig.make(
+    2048, 32000, _panarax_layers(5, 16, 128, 5632, RoutedSpec(32, 2, 1408, act="clamped", scoring="sigmoid", limit=7.0, weigh_input=True)),
+    max_seq_len=8192, block="prenorm", layer_norm=True, residual_gate=True, input_conv=4, positions=8192, tied_head=True,
+    architecture="Panarax", name="panarax-15l")
+
 PRESETS = {
+    "panarax": panarax_config,
     "vufinex": vufinex_config,
     "supinex": supinex_config,
     "rurunex": rurunex_config,

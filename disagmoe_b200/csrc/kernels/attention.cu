@@ -54,6 +54,8 @@ __device__ __forceinline__ void cp_async16_stream(uint32_t dst, const void* src,
 //   chunk > 0: it sees only keys of its own chunk of `chunk` positions, counted from position 0;
 //   cap_log2 > 0: score <- cap * tanh(score / cap) before the softmax (cap_log2 = cap * log2 e, cap_in = 2 scale log2 e / cap);
 //   sink != NULL: exp(sink[head]) enters the softmax denominator (no key, no value);
+//   temp_every > 0: scores are multiplied by the query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1);
+//   gate != NULL: head outputs are multiplied by sigmoid(gate[row, head]) (row stride ld_gate);
 //   gq: query heads per kv head where the instantiation leaves it open (GQ = 0).
 // The EXT kernels also keep the softmax weights at fp32 accuracy in the P V product: P = hi + lo, both bf16, two MMAs.
 struct AttnExt {
@@ -61,7 +63,18 @@ struct AttnExt {
   float cap_in, cap_log2;
   const float* sink;
   int gq;
+  const void* gate;
+  long long ld_gate;
+  float temp_coef;
+  int temp_every;
 };
+__device__ __forceinline__ float query_temperature(const AttnExt& x, int p) {
+  return x.temp_every > 0 ? 1.f + x.temp_coef * logf(static_cast<float>((p + 1) / x.temp_every + 1)) : 1.f;
+}
+template <typename T>
+__device__ __forceinline__ float head_gate(const AttnExt& x, long long row, int head) {
+  return x.gate != nullptr ? 1.f / (1.f + expf(-static_cast<float>(static_cast<const T*>(x.gate)[row * x.ld_gate + head]))) : 1.f;
+}
 constexpr float kLog2e = 1.4426950408889634f;
 // first key that a query at position p sees
 __device__ __forceinline__ int first_key(int p, int window, int chunk) {
@@ -185,6 +198,7 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
 #pragma unroll
   for (int i = 0; i < NT; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m = -INFINITY, l = 0.f;
+  const float temp = EXT ? query_temperature(ext, len - 1) : 1.f;
 
   // ldmatrix lane roles
   const int lm_mi = lane >> 3, lm_r = lane & 7;
@@ -210,10 +224,10 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
     // row g: tokens tok0 + 2 tq + {0, 1} (s0) and tok0 + 8 + 2 tq + {0, 1} (s1)
     const int tk = tok0 + 2 * tq;
     auto seen = [&](int j) { return j < c1 && (!EXT || j >= vis0); };
-    float p00 = seen(tk) ? attn_score<EXT>(s0[0], scale_log2, ext) : -INFINITY;
-    float p01 = seen(tk + 1) ? attn_score<EXT>(s0[1], scale_log2, ext) : -INFINITY;
-    float p10 = seen(tk + 8) ? attn_score<EXT>(s1[0], scale_log2, ext) : -INFINITY;
-    float p11 = seen(tk + 9) ? attn_score<EXT>(s1[1], scale_log2, ext) : -INFINITY;
+    float p00 = seen(tk) ? attn_score<EXT>(s0[0] * temp, scale_log2, ext) : -INFINITY;
+    float p01 = seen(tk + 1) ? attn_score<EXT>(s0[1] * temp, scale_log2, ext) : -INFINITY;
+    float p10 = seen(tk + 8) ? attn_score<EXT>(s1[0] * temp, scale_log2, ext) : -INFINITY;
+    float p11 = seen(tk + 9) ? attn_score<EXT>(s1[1] * temp, scale_log2, ext) : -INFINITY;
     float mx = fmaxf(fmaxf(p00, p01), fmaxf(p10, p11));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -280,7 +294,8 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
     }
     const float val = L > 0.f ? O / L : 0.f;
     if (splits == 1) {
-      out[static_cast<long long>(t) * ld_out + head * VD + d] = __float2bfloat16(val);
+      const float gated = EXT ? val * head_gate<__nv_bfloat16>(ext, t, head) : val;
+      out[static_cast<long long>(t) * ld_out + head * VD + d] = __float2bfloat16(gated);
     } else {
       const long long pi = (static_cast<long long>(t) * n_q + head) * splits + split;
       part_o[pi * VD + d] = val;
@@ -289,10 +304,10 @@ paged_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __n
   }
 }
 
-// out[t, head] = sum_s softmax_s(lse) * part_o[t, head, s]
+// out[t, head] = sum_s softmax_s(lse) * part_o[t, head, s], gated
 template <int VD>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, int splits,
-                                  int n_q, __nv_bfloat16* __restrict__ out, long long ld_out) {
+                                  int n_q, __nv_bfloat16* __restrict__ out, long long ld_out, AttnExt ext) {
   const int t = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
   const long long pi = (static_cast<long long>(t) * n_q + head) * splits;
   float M = -INFINITY;
@@ -305,7 +320,8 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
       O += w * part_o[(pi + s) * VD + d];
     }
   }
-  out[static_cast<long long>(t) * ld_out + head * VD + d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
+  out[static_cast<long long>(t) * ld_out + head * VD + d] =
+      __float2bfloat16(L > 0.f ? O / L * head_gate<__nv_bfloat16>(ext, t, head) : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -420,6 +436,7 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
   const int wlast = pos0 + min(ntok - 1, (warp * 16 + 15) / gq);
   // and, with a window or chunks, those entirely before the reach of its first query; a row's first visible key
   const int wfirst = EXT ? first_key(pos0 + warp * 16 / gq, ext.window, ext.chunk) : 0;
+  const float temp0 = EXT ? query_temperature(ext, qpos0) : 1.f, temp1 = EXT ? query_temperature(ext, qpos1) : 1.f;
   const int lo0 = EXT ? first_key(qpos0, ext.window, ext.chunk) : 0;
   const int lo1 = EXT ? first_key(qpos1, ext.window, ext.chunk) : 0;
 
@@ -453,10 +470,10 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
         const int k0 = key0 + nt * 8 + 2 * tq;
         const bool a0 = v0 && k0 <= qpos0 && (!EXT || k0 >= lo0), a1 = v0 && k0 + 1 <= qpos0 && (!EXT || k0 + 1 >= lo0);
         const bool b0 = v1 && k0 <= qpos1 && (!EXT || k0 >= lo1), b1 = v1 && k0 + 1 <= qpos1 && (!EXT || k0 + 1 >= lo1);
-        s[nt][0] = a0 ? attn_score<EXT>(s[nt][0], scale_log2, ext) : -INFINITY;
-        s[nt][1] = a1 ? attn_score<EXT>(s[nt][1], scale_log2, ext) : -INFINITY;
-        s[nt][2] = b0 ? attn_score<EXT>(s[nt][2], scale_log2, ext) : -INFINITY;
-        s[nt][3] = b1 ? attn_score<EXT>(s[nt][3], scale_log2, ext) : -INFINITY;
+        s[nt][0] = a0 ? attn_score<EXT>(s[nt][0] * temp0, scale_log2, ext) : -INFINITY;
+        s[nt][1] = a1 ? attn_score<EXT>(s[nt][1] * temp0, scale_log2, ext) : -INFINITY;
+        s[nt][2] = b0 ? attn_score<EXT>(s[nt][2] * temp1, scale_log2, ext) : -INFINITY;
+        s[nt][3] = b1 ? attn_score<EXT>(s[nt][3] * temp1, scale_log2, ext) : -INFINITY;
         mx0 = fmaxf(mx0, fmaxf(s[nt][0], s[nt][1]));
         mx1 = fmaxf(mx1, fmaxf(s[nt][2], s[nt][3]));
       }
@@ -522,6 +539,10 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
     inv0 = sink_inverse(m0, l0, ext.sink[head0]);
     inv1 = sink_inverse(m1, l1, ext.sink[head1]);
   }
+  if (EXT && ext.gate != nullptr) {
+    if (v0) inv0 *= head_gate<__nv_bfloat16>(ext, row0 + t0, head0);
+    if (v1) inv1 *= head_gate<__nv_bfloat16>(ext, row0 + t1, head1);
+  }
   if (v0) {
     __nv_bfloat16* op = out + static_cast<long long>(row0 + t0) * ld_out + head0 * VD;
 #pragma unroll
@@ -537,8 +558,12 @@ prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const _
 }
 
 // Options of a launch as the kernels take them (softcap <= 0: none; window, chunk <= 0: every key).
-static AttnExt make_ext(float scale, int window, int chunk, float softcap, const float* sink, int gq) {
+static AttnExt make_ext(float scale, int window, int chunk, float softcap, const float* sink, int gq, const DmoeAttnExtra* extra) {
   AttnExt x;
+  x.gate = extra != nullptr ? extra->gate : nullptr;
+  x.ld_gate = extra != nullptr ? extra->ld_gate : 0;
+  x.temp_coef = extra != nullptr ? extra->temp_coef : 0.f;
+  x.temp_every = extra != nullptr ? extra->temp_every : 0;
   x.sink = sink;
   x.gq = gq;
   x.window = window > 0 ? window : 0;
@@ -590,7 +615,7 @@ static int launch_attn(const void* q, long long ld_q, const void* kc, const void
   if (splits > 1) {
     dim3 g2(T, n_kv * gq);
     attn_merge_kernel<VD><<<g2, VD, 0, stream>>>(part_o, part_lse, splits, n_kv * gq,
-                                                  static_cast<__nv_bfloat16*>(out), ld_out);
+                                                  static_cast<__nv_bfloat16*>(out), ld_out, ext);
     e = cudaGetLastError();
   }
   return static_cast<int>(e);
@@ -625,6 +650,7 @@ static int attn_dispatch(const void* q, long long ld_q, const void* kcache, cons
     if (gq > 64) return -11;
     if (hd == 128 && vd == 128) DMOE_ATTN(128, 128, 0);
     if (hd == 128 && vd == 64) DMOE_ATTN(128, 64, 0);
+    if (hd == 64 && vd == 128) DMOE_ATTN(64, 128, 0);
     if (hd == 64 && vd == 64) DMOE_ATTN(64, 64, 0);
     if (hd == 64 && vd == 32) DMOE_ATTN(64, 32, 0);
   } else if (hd == 128) {
@@ -651,7 +677,7 @@ extern "C" int dmoe_paged_attention(const void* q, long long ld_q, const void* k
                                     int block_size, int T, int n_q, int n_kv, int hd, float scale, int splits, void* out,
                                     long long ld_out, float* workspace, void* stream_) {
   return attn_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                              hd, hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0, 0.f, nullptr, 0),
+                              hd, hd, scale, splits, out, ld_out, workspace, make_ext(scale, 0, 0, 0.f, nullptr, 0, nullptr),
                               static_cast<cudaStream_t>(stream_));
 }
 
@@ -661,10 +687,10 @@ extern "C" int dmoe_paged_attention_ext(const void* q, long long ld_q, const voi
                                         const int* block_tables, int max_blocks, const int* bt_row, const int* ctx_len,
                                         int block_size, int T, int n_q, int n_kv, int hd, int vd, float scale, int window,
                                         int chunk, float softcap, const float* sink, int splits, void* out, long long ld_out,
-                                        float* workspace, void* stream_) {
+                                        float* workspace, const DmoeAttnExtra* extra, void* stream_) {
   if (n_kv < 1) return -10;
   return attn_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, bt_row, ctx_len, block_size, T, n_q, n_kv,
-                             hd, vd, scale, splits, out, ld_out, workspace, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv),
+                             hd, vd, scale, splits, out, ld_out, workspace, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv, extra),
                              static_cast<cudaStream_t>(stream_));
 }
 
@@ -688,6 +714,7 @@ static int prefill_dispatch(const void* q, long long ld_q, const void* kcache, c
     if (gq > kPreRows) return -11;
     if (hd == 128 && vd == 128) DMOE_PRE(128, 128, 0);
     if (hd == 128 && vd == 64) DMOE_PRE(128, 64, 0);
+    if (hd == 64 && vd == 128) DMOE_PRE(64, 128, 0);
     if (hd == 64 && vd == 64) DMOE_PRE(64, 64, 0);
     if (hd == 64 && vd == 32) DMOE_PRE(64, 32, 0);
   } else if (hd == 128) {
@@ -714,17 +741,18 @@ extern "C" int dmoe_prefill_attention(const void* q, long long ld_q, const void*
                                       int block_size, int n_q, int n_kv, int hd, float scale, void* out, long long ld_out,
                                       void* stream_) {
   return prefill_dispatch<false>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                 hd, hd, scale, out, ld_out, make_ext(scale, 0, 0, 0.f, nullptr, 0),
+                                 hd, hd, scale, out, ld_out, make_ext(scale, 0, 0, 0.f, nullptr, 0, nullptr),
                                  static_cast<cudaStream_t>(stream_));
 }
 
 extern "C" int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                           const int* block_tables, int max_blocks, const void* tiles, int n_tiles,
                                           int block_size, int n_q, int n_kv, int hd, int vd, float scale, int window,
-                                          int chunk, float softcap, const float* sink, void* out, long long ld_out, void* stream_) {
+                                          int chunk, float softcap, const float* sink, void* out, long long ld_out,
+                                          const DmoeAttnExtra* extra, void* stream_) {
   if (n_kv < 1) return -10;
   return prefill_dispatch<true>(q, ld_q, kcache, vcache, block_tables, max_blocks, tiles, n_tiles, block_size, n_q, n_kv,
-                                hd, vd, scale, out, ld_out, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv),
+                                hd, vd, scale, out, ld_out, make_ext(scale, window, chunk, softcap, sink, n_q / n_kv, extra),
                                 static_cast<cudaStream_t>(stream_));
 }
 
@@ -742,7 +770,7 @@ any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, cons
                 const T* __restrict__ vcache, long long v_tok, const int* __restrict__ block_tables, int max_blocks,
                 const int* __restrict__ bt_row, const int* __restrict__ rows, const int* __restrict__ ctx_len, int block_size,
                 int n_q, int n_kv, int dk, int dv, float scale, int window, int chunk, float softcap, const float* __restrict__ sink,
-                T* __restrict__ out, long long o_head, long long o_row) {
+                T* __restrict__ out, long long o_head, long long o_row, AttnExt ext) {
   extern __shared__ float s_any[];          // q [dk] | acc [dv]
   __shared__ float s_p[kAnyKeys];
   __shared__ long long s_slot[kAnyKeys];
@@ -759,6 +787,7 @@ any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, cons
   for (int d = tid; d < dv; d += kAnyKeys) s_acc[d] = 0.f;
   __syncthreads();
   float m = -INFINITY, l = 0.f;
+  scale *= query_temperature(ext, len - 1);
   for (int j0 = len > 0 ? first_key(len - 1, window, chunk) : 0; j0 < len; j0 += kAnyKeys) {
     const int n = min(kAnyKeys, len - j0);
     float s = -INFINITY;
@@ -796,11 +825,12 @@ any_attn_kernel(const T* __restrict__ q, long long q_head, long long q_row, cons
     }
     __syncthreads();
   }
-  float f = 1.f;
+  float f = head_gate<T>(ext, t, head);
   if (sink != nullptr && len > 0) {
     const float mn = fmaxf(m, sink[head]);
-    f = expf(m - mn);
-    l = l * f + expf(sink[head] - mn);
+    const float shrink = expf(m - mn);
+    f *= shrink;
+    l = l * shrink + expf(sink[head] - mn);
   }
   for (int d = tid; d < dv; d += kAnyKeys)
     out[blockIdx.x * o_row + head * o_head + d] = static_cast<T>(l > 0.f ? s_acc[d] * f / l : 0.f);
@@ -812,21 +842,22 @@ extern "C" int dmoe_any_attention(int is_f32, const void* q, long long q_head, l
                                   long long k_tok, const void* vcache, long long v_tok, const int* block_tables, int max_blocks,
                                   const int* bt_row, const int* rows, const int* ctx_len, int block_size, int T, int n_q,
                                   int n_kv, int dk, int dv, float scale, int window, int chunk, float softcap, const float* sink, void* out,
-                                  long long o_head, long long o_row, void* stream_) {
+                                  long long o_head, long long o_row, const DmoeAttnExtra* extra, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (T == 0) return 0;
   if (n_kv < 1 || n_q % n_kv != 0 || n_q > 65535 || block_size < 1 || dk < 1 || dv < 1 || dk + dv > 8192) return -10;
   const dim3 grid(T, n_q);
+  const AttnExt ext = make_ext(scale, window, chunk, softcap, sink, n_q / n_kv, extra);
   const size_t smem = static_cast<size_t>(dk + dv) * sizeof(float);
   if (is_f32)
     any_attn_kernel<float><<<grid, kAnyKeys, smem, stream>>>(
         static_cast<const float*>(q), q_head, q_row, static_cast<const float*>(kcache), k_tok, static_cast<const float*>(vcache),
         v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv, dk, dv, scale, window, chunk, softcap, sink,
-        static_cast<float*>(out), o_head, o_row);
+        static_cast<float*>(out), o_head, o_row, ext);
   else
     any_attn_kernel<__nv_bfloat16><<<grid, kAnyKeys, smem, stream>>>(
         static_cast<const __nv_bfloat16*>(q), q_head, q_row, static_cast<const __nv_bfloat16*>(kcache), k_tok,
         static_cast<const __nv_bfloat16*>(vcache), v_tok, block_tables, max_blocks, bt_row, rows, ctx_len, block_size, n_q, n_kv,
-        dk, dv, scale, window, chunk, softcap, sink, static_cast<__nv_bfloat16*>(out), o_head, o_row);
+        dk, dv, scale, window, chunk, softcap, sink, static_cast<__nv_bfloat16*>(out), o_head, o_row, ext);
   return static_cast<int>(cudaGetLastError());
 }

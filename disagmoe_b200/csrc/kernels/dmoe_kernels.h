@@ -30,6 +30,60 @@ typedef struct DmoeShift {
   long long mix_stride;     // elements from one output to the next
   int n_mix, n_slots, n_single;
 } DmoeShift;
+// Causal convolution over time per channel: sum_j w[j] x_(t - taps + 1 + j) + out_bias of the inputs x + in_bias, with `residual` plus
+// the input itself. The last inputs (without their bias) of a sequence sit in its slot's ring by position modulo taps. blocks: the
+// output columns are cut into equal blocks, stored one after the other in rows of `padded` numbers. Singles as in DmoeShift.
+typedef struct DmoeConv {
+  const float* w;           // [taps, C]
+  const float* in_bias;     // [C], may be NULL
+  const float* out_bias;
+  void* ring;               // [n_slots, taps, C]
+  const void* singles;
+  const int* positions;
+  const int* rows;
+  const long long* kv_slots;
+  int n_single, n_slots, taps, residual, blocks, padded;
+} DmoeConv;
+// Further steps of dmoe_sum_norm (all optional): a bias of the norm [W]; what is added to the residual is multiplied by
+// sigmoid(gate_z[row] + gate_bias); `side`: two rows per row instead of y, added up as side_scale * their RMS norms times side_w [2, W];
+// conv (all rows one-token segments): the second output, one matrix of n rows after h, is the convolution of h.
+typedef struct DmoeSumExtra {
+  const float* bias;
+  const void* gate_z;
+  const float* gate_bias;
+  const void* side;
+  const float* side_w;
+  const DmoeConv* conv;
+  long long ld_gate, ld_side, side_stride;
+  float side_scale;
+} DmoeSumExtra;
+// Options of the attention kernels: head outputs times sigmoid(gate[row, head]) (NULL: none), scores times the query temperature
+// 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) of the query's position p (temp_every 0: none).
+typedef struct DmoeAttnExtra {
+  const void* gate;
+  long long ld_gate;
+  float temp_coef;
+  int temp_every;
+} DmoeAttnExtra;
+// Real-gated diagonal recurrence (diag_recurrent.cu): u [blocks, block_rows, padded], gate logits [blocks, block_rows, 2, padded] with
+// biases [blocks, 2, padded], y and out [rows, width]; state [n_slots, width]; segment tables as in DmoeRecur.
+typedef struct DmoeUnit {
+  const void* u;
+  const float* gates;
+  const float* gate_bias;
+  const float* decay;       // [width] log decay of an open gate
+  const void* y;
+  const float* y_bias;
+  float* state;
+  void* out;
+  const void* singles;
+  const int* positions;
+  const int* rows;
+  const long long* kv_slots;
+  const void* multi;
+  long long ldy, ldo, block_rows;
+  int n_single, n_multi, n_slots, width, blocks, padded;
+} DmoeUnit;
 #endif
 
 // ---- GEMM (gemm.cu) -------------------------------------------------------------------------------
@@ -97,12 +151,17 @@ typedef struct DmoeGemm {
   // != 0: W is stored tile by tile, [group][128-row tile][K / 64][128][64] (see ops/gemm.py: block_weight), so that
   // every 16 KB box the kernel fetches is one contiguous run of HBM; needs F % 128 == 0 and K % 64 == 0
   int w_blocked;
-  // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form); plain epilogue: 2 = tanh of the output
+  // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form), 3 clamped: min(g, act_limit) sigmoid(1.702 g)
+  // (clamp(u, act_limit) + 1); plain epilogue: 2 = tanh of the output, 4 = silu of its first act_cols columns. SwiGLU with
+  // recs: gate and up of row t are multiplied by the weight of record t first.
   int act;
   // profiling aid, normally null: 16 x uint64 of device memory that CTA 0 fills with %globaltimer stamps (entry, set-up
   // done, first TMA issued, first stage landed, last MMA committed, accumulator seen by the epilogue, epilogue done,
   // tear-down reached, then five points inside the first epilogue chunk and three inside the producer's start)
   void* trace;
+  float act_limit;
+  int act_cols;
+  int unit_weights;   // combine: the records' weights are left out
 } DmoeGemm;
 
 int dmoe_gemm(const DmoeGemm* desc, void* stream);
@@ -136,15 +195,15 @@ int dmoe_paged_attention(const void* q, long long ld_q, const void* kcache, cons
 
 // With a sliding window (a query sees the last `window` tokens, itself included; 0 = all), a score soft cap
 // (cap * tanh(score / cap); 0 = none) and a sink (exp(sink[head]) enters the softmax denominator; NULL = none); value heads
-// of size vd. (hd, vd) = (64, 32), (64, 64), (128, 64), (128, 128), up to 64 query heads per kv head.
+// of size vd. (hd, vd) = (64, 32), (64, 64), (64, 128), (128, 64), (128, 128), up to 64 query heads per kv head.
 int dmoe_paged_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache, const int* block_tables,
                              int max_blocks, const int* bt_row, const int* ctx_len, int block_size, int T, int n_q, int n_kv,
                              int hd, int vd, float scale, int window, int chunk, float softcap, const float* sink, int splits, void* out,
-                             long long ld_out, float* workspace, void* stream);
+                             long long ld_out, float* workspace, const DmoeAttnExtra* extra, void* stream);
 int dmoe_prefill_attention_ext(const void* q, long long ld_q, const void* kcache, const void* vcache,
                                const int* block_tables, int max_blocks, const void* tiles, int n_tiles, int block_size,
                                int n_q, int n_kv, int hd, int vd, float scale, int window, int chunk, float softcap, const float* sink,
-                               void* out, long long ld_out, void* stream);
+                               void* out, long long ld_out, const DmoeAttnExtra* extra, void* stream);
 // Any key / value size and query group, bf16 or fp32 cache, fp32 arithmetic on the CUDA cores. Query i of head h starts at
 // q + i * q_row + h * q_head (output likewise) and has the context of batch row rows[i] (NULL: i); the heads of a cached token
 // are contiguous, tokens k_tok / v_tok elements apart.
@@ -152,7 +211,7 @@ int dmoe_any_attention(int is_f32, const void* q, long long q_head, long long q_
                        const void* vcache, long long v_tok, const int* block_tables, int max_blocks, const int* bt_row,
                        const int* rows, const int* ctx_len, int block_size, int T, int n_q, int n_kv, int dk, int dv,
                        float scale, int window, int chunk, float softcap, const float* sink, void* out, long long o_head, long long o_row,
-                       void* stream);
+                       const DmoeAttnExtra* extra, void* stream);
 
 // ---- latent attention (latent_attention.cu): the cache has one row [latent rankp | rotated key part rotp] per token,
 // `row` elements apart ------
@@ -188,8 +247,9 @@ int dmoe_prefill_attention(const void* q, long long ld_q, const void* kcache, co
                            int n_q, int n_kv, int hd, float scale, void* out, long long ld_out, void* stream);
 
 // ---- fp32-residual decoders (layer_ops.cu); is_f32: fp32 activations instead of bf16 -----------------------
-// out[t] = table[ids[t]] * scale (fp32)
-int dmoe_embed_f32(const int* ids, const void* table, int is_f32, float scale, float* out, int T, int W, int vocab, void* stream);
+// out[t] = table[ids[t]] * scale (+ pos_table[positions[t]] where given, n_pos rows) (fp32)
+int dmoe_embed_f32(const int* ids, const void* table, int is_f32, float scale, float* out, int T, int W, int vocab,
+                   const int* positions, const void* pos_table, int n_pos, void* stream);
 // x = resid[r] + norm(y[r]) * post (y may be NULL: x = resid[r]); resid[r] = x unless a row table picks r = rows[i];
 // h[i] = norm(x) * pre * out_scale (h may be NULL); norm(v) = v / sqrt(mean(v^2) + eps). resid fp32 [.., W].
 int dmoe_resid_norm(int is_f32, float* resid, const void* y, long long ld_y, const float* post, const float* pre,
@@ -199,31 +259,36 @@ int dmoe_rope_freq_table(void* table, int max_pos, int half, const double* freq,
 // Per-head RMS norm of q and k (qw, kw; NULL: none), rotation of pairs (i, i + rot / 2), i < rot / 2, or (2i, 2i + 1) where
 // interleaved; q in place, k / v into the paged caches, v as (1 - v_lambda) v + v_lambda v_first where that is given
 // (row stride ld_first, head stride first_head). tied: rows [q | k], the values are the first dv dimensions of the k heads before
-// their rotation.
+// their rotation. v_norm > 0: every value head is divided by its root mean square over v_norm dimensions (the rest is zeros).
 int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots, void* kcache,
                       void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved, const void* table,
                       int max_pos, const float* qw, const float* kw, float eps, const void* v_first, long long ld_first,
-                      int first_head, float v_lambda, int tied, void* stream);
+                      int first_head, float v_lambda, int tied, int v_norm, void* stream);
 // x = resid[r] + mult (y[r] + sum of n_parts rows of parts) (both may be NULL); resid[r] = x unless a row table picks
 // r = rows[i]; h[i] = norm(x) * w, RMS norm or with `centred` layer norm, as fp32 where h_f32. router: the K best experts of
 // every h and, where counts is given, the histogram of the chosen ones; E <= 256, K <= 32. shift (all rows one-token segments):
 // h gets the n_mix mixed rows instead.
 int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
                   long long part_row, long long part_stride, float mult, const float* w, int centred, float eps, const int* rows,
-                  void* h, int h_f32, long long ld_h, int n, int W, const DmoeRouter* router, const DmoeShift* shift, void* stream);
+                  void* h, int h_f32, long long ld_h, int n, int W, const DmoeRouter* router, const DmoeShift* shift, const DmoeSumExtra* extra,
+                  void* stream);
 // The token shift of a batch with longer segments (tables as in DmoeRecur: segs of the longer ones, their chunks): fp32 rows h ->
 // n_mix outputs; the slots keep the last row of every segment.
 int dmoe_token_shift(int is_f32, const float* h, const DmoeShift* s, const void* multi, int n_multi, const void* chunks, int n_chunks,
                      void* out, long long ld, int W, void* stream);
-// out[t, i] = act(gu[t, i]) * gu[t, I + i]; act 0: silu, 1: gelu (tanh form)
-int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I, void* stream);
+int dmoe_seq_conv(int is_f32, const void* x, long long ldx, const DmoeConv* a, const void* multi, int n_multi, const void* chunks,
+                  int n_chunks, void* out, long long ldo, long long block_stride, int C, void* stream);
+int dmoe_unit_recurrence(int is_f32, const DmoeUnit* d, void* stream);
+// out[t, i] = act(gu[t, i]) * gu[t, I + i]; act, limit and recs as in DmoeGemm
+int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I, float limit,
+                  const void* recs, void* stream);
 // Y = X W^T on the CUDA cores in fp32 arithmetic: fp32 operands, or bf16 operands of any alignment.
 int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y, long long ldy,
-                     int T, int F, int K, int act, void* stream);      // act 2: tanh of the output
+                     int T, int F, int K, int act, int act_cols, void* stream);      // act 2: tanh of the output, 4: silu of its first columns
 // The same over row groups: rows offs[g] .. offs[g + 1] of X with W[g] [F, K]; recs / bases (may be NULL): row t goes, scaled,
 // where recs[t] says (see DmoeGemm), in X's type.
-int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y, long long ldy,
-                      const void* recs, const void* bases, int T, int F, int K, void* stream);
+int dmoe_simt_grouped(int is_f32, int y_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y, long long ldy,
+                      const void* recs, const void* bases, int unit_weights, int T, int F, int K, void* stream);
 
 // ---- linear recurrences with a matrix state per head (recurrent.cu) ---------------------------------------
 typedef struct DmoeRecur {
@@ -232,7 +297,7 @@ typedef struct DmoeRecur {
   const void* v;            // [rows, heads * vdim]
   const void* gate;         // [rows, heads * vdim] output gate before its activation
   const void* beta;         // delta: [rows, heads] write strength before its sigmoid
-  const float* z;           // [rows, heads * dim] decay logits without their bias
+  const float* z;           // [rows, heads * dim] decay logits without their bias (kinds 0 to 2)
   const float* z_bias;      // [heads * dim]
   const float* a_log;       // [heads], decay_kind 1
   const float* conv_w;      // [2 kv_heads dim + heads vdim, taps], last column = current token
@@ -249,6 +314,7 @@ typedef struct DmoeRecur {
   int n_segs, n_slots, heads, kv_heads, dim, vdim, taps;
   int delta;                // 0: plain write, 1: delta rule (q and k are made unit vectors)
   int decay_kind;           // 0: log a = log sigmoid(z + b) * inv_tau, 1: log a = -exp(a_log) softplus(z + b), 2: log a = -exp(z + b)
+                            // 3: log a = head_decay[h]; 4: matrix memory (below)
   int gate_kind;            // 0: silu, 1: sigmoid
   int is_f32;
   int one_token;            // dmoe_recur_step: every segment has one token
@@ -257,12 +323,28 @@ typedef struct DmoeRecur {
   const float* bonus;       // plain write only: [heads, dim]; the read-out precedes decay and write, and the token's own write
                             // enters it weighed by the bonus of the key channel
   int norm_ld;
+  const float* head_decay;  // [heads]
+  // matrix memory: logs i = cap(gates[row, h] + gate_bias[h]), f = log sigmoid(cap(gates[row, heads + h] + ..)), cap(z) = gate_cap
+  // tanh(z / gate_cap); running maximum m <- max(f + m, i), decay exp(f + m - m'), k scaled by exp(i - m'); read-outs are divided by
+  // max(|n . q|, exp(-m)) + 1e-6, n decayed and written like a state of one value column of ones
+  const float* gates;       // [rows, 2 heads], row stride ldgates
+  const float* gate_bias;   // [2 heads]
+  float* norm_state;        // [n_slots, heads, dim]
+  float* max_state;         // [n_slots, 2, heads]: m at the parity of its position
+  float* keep;              // [rows, heads] log decays, factors of k and running maxima of longer segments (dmoe_memory_gates)
+  float* put;
+  float* run_max;
+  float* scale;             // with raw: [rows, heads] factors of the read-outs (the divisions above)
+  long long ldgates;
+  float gate_cap;
 } DmoeRecur;
+// keep, put and run_max of the rows of a->segs; the running maxima in the slots move on.
+int dmoe_memory_gates(const DmoeRecur* a, void* stream);
 int dmoe_recur_value_tile(int dim, int vdim);
 int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream);
 int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw, const void* gate,
                    long long ldg, const float* norm_w, int norm_ld, float eps, int gate_kind, void* out, long long ldo, int heads, int V,
-                   void* stream);
+                   const float* scale, void* stream);      // scale [rows, heads]: factors of the raw rows, may be NULL
 // The same recurrence chunk by chunk on the tensor cores (recurrent_chunk.cu), bf16 activations, for segments of any length.
 int dmoe_recur_chunk_ok(int dim, int vdim);
 long long dmoe_recur_chunk_bytes(int dim, int vdim, int delta, int n_chunks);

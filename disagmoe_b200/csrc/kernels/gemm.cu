@@ -96,7 +96,11 @@ struct GemmArgs {
   // w_blocked: the weights are stored tile by tile ([group][128-row tile][K block][128][64], every 16 KB TMA box one
   // contiguous run of HBM) instead of row-major [group][row][K]
   int w_blocked;
-  int act;      // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form); plain epilogue: 2 = tanh of the output
+  int act;      // gate activation of the SwiGLU epilogue: 0 silu, 1 gelu (tanh form), 3 clamped; plain epilogue: 2 = tanh of the
+                // output, 4 = silu of the first act_cols columns
+  float act_limit;
+  int act_cols;
+  int unit_weights;   // combine: rows are not scaled
   // optional [16] nanosecond stamps written by CTA 0 (a profiling aid, null in normal launches): 0 entry, 1 set-up done,
   // 2 first TMA issued, 3 first stage landed, 4 last MMA committed, 5 accumulator seen by the epilogue, 6 epilogue done,
   // 7 tear-down reached; 8-12 inside the first epilogue chunk: TMEM read done, staged to shared memory, barrier passed,
@@ -144,6 +148,13 @@ __device__ __forceinline__ void trace_stamp(const GemmArgs& a, int i) {
 __device__ __forceinline__ float gate_act(float g, int act) {
   const float z = act == 0 ? g : 1.5957691216057308f * (g + 0.044715f * g * g * g);
   return g / (1.f + __expf(-z));
+}
+
+// act(g) * u; clamped: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1)
+__device__ __forceinline__ float gated(float g, float u, int act, float limit) {
+  if (act != 3) return gate_act(g, act) * u;
+  const float m = fminf(g, limit);
+  return __fdividef(m, 1.f + __expf(-1.702f * m)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }
 
 // tanh(x) = 1 - 2 / (exp(2x) + 1), good to about 1e-7 absolute
@@ -514,7 +525,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
           }
           if (EPI == EPI_SWIGLU) {
 #pragma unroll
-            for (int j = 0; j < 32; ++j) acc[j] = gate_act(acc[j], a.act) * up[j];
+            for (int j = 0; j < 32; ++j) {
+              const float s = a.recs != nullptr && j < jmax ? __int_as_float(__ldg(&a.recs[tok_base + c * 32 + j].z)) : 1.f;
+              acc[j] = gated(acc[j] * s, up[j] * s, a.act, a.act_limit);
+            }
           }
         } else {
           uint32_t v[32];
@@ -526,9 +540,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
             if (et == 0 && c == 0) trace_stamp(a, 8);
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
-              const float g = __uint_as_float(v[j]);
-              const float up = __uint_as_float(uu[j]);
-              acc[j] = gate_act(g, a.act) * up;
+              const float s = a.recs != nullptr && j < jmax ? __int_as_float(__ldg(&a.recs[tok_base + c * 32 + j].z)) : 1.f;
+              const float g = __uint_as_float(v[j]) * s;
+              const float up = __uint_as_float(uu[j]) * s;
+              acc[j] = gated(g, up, a.act, a.act_limit);
             }
           } else {
             tmem_ld_wait();
@@ -546,6 +561,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
         if (EPI == EPI_PLAIN && a.act == 2) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) acc[j] = out_tanh(acc[j]);
+        }
+        if (EPI == EPI_PLAIN && a.act == 4 && f < a.act_cols) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) acc[j] = gate_act(acc[j], 0);
         }
         if ((EPI == EPI_PLAIN || EPI == EPI_SWIGLU) && vec) {
           if (jmax <= 0) continue;                   // uniform over the CTA: no barrier is skipped by some threads only
@@ -742,7 +761,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               const int j = tk0 + q * 8;
-              const float w = __int_as_float(rec4[q].z);
+              const float w = a.unit_weights ? 1.f : __int_as_float(rec4[q].z);
               const float4 x0 = *reinterpret_cast<const float4*>(&epi_stage[j * kBM + fg * 8]);
               const float4 x1 = *reinterpret_cast<const float4*>(&epi_stage[j * kBM + fg * 8 + 4]);
               __nv_bfloat162* pp = reinterpret_cast<__nv_bfloat162*>(&pk[q]);
@@ -774,7 +793,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
             if (j >= jmax) break;
             const int4 rec = __ldg(&a.recs[tok_base + c * 32 + j]);
             if (rec.y < 0) continue;
-            const __nv_bfloat16 val = __float2bfloat16(acc[j] * __int_as_float(rec.z));
+            const __nv_bfloat16 val = __float2bfloat16(a.unit_weights ? acc[j] : acc[j] * __int_as_float(rec.z));
             if (a.fanout <= 1) {
               (reinterpret_cast<__nv_bfloat16*>(a.bases[rec.x]) + static_cast<long long>(rec.y) * a.ldy)[f] = val;
             } else {
@@ -1015,7 +1034,7 @@ extern "C" int dmoe_gemm(const DmoeGemm* d, void* stream_) {
   const long long ldx = d->ldx > 0 ? d->ldx : d->K;
   a.trace = static_cast<unsigned long long*>(d->trace);
   a.w_blocked = d->w_blocked != 0;
-  a.act = d->act;
+  a.act = d->act; a.act_limit = d->act_limit; a.act_cols = d->act_cols; a.unit_weights = d->unit_weights;
   if (a.w_blocked) {
     // whole 128-row tiles and whole 64-element K blocks only; row coordinates must stay below 2^31
     const long long rows = static_cast<long long>(d->G) * a.w_rows * (d->K / kBK);

@@ -4,52 +4,9 @@
 // and a CUDA-core GEMM, dense or over row groups, for fp32 operands (and for bf16 shapes the tcgen05 kernel's TMA cannot
 // address).
 #include "dmoe_kernels.h"
-#include "sm100.cuh"
+#include "row_pack.cuh"
 
 namespace dmoe {
-
-typedef __nv_bfloat16 bf16;
-
-template <typename T, int VEC>
-struct Pack;   // VEC elements of T <-> floats, one aligned access where VEC > 1
-template <typename T>
-struct Pack<T, 1> {
-  static __device__ __forceinline__ void load(const T* p, float* f) { f[0] = static_cast<float>(p[0]); }
-  static __device__ __forceinline__ void store(T* p, const float* f) { p[0] = static_cast<T>(f[0]); }
-};
-template <>
-struct Pack<float, 8> {
-  static __device__ __forceinline__ void load(const float* p, float* f) {
-    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-  }
-  static __device__ __forceinline__ void store(float* p, const float* f) {
-    reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
-    reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
-  }
-};
-template <>
-struct Pack<bf16, 8> {
-  static __device__ __forceinline__ void load(const bf16* p, float* f) {
-    const uint4 r = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 t = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
-      f[2 * i] = t.x;
-      f[2 * i + 1] = t.y;
-    }
-  }
-  static __device__ __forceinline__ void store(bf16* p, const float* f) {
-    uint32_t w[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
-      w[i] = *reinterpret_cast<const uint32_t*>(&t);
-    }
-    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-  }
-};
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -66,15 +23,18 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
   return t;
 }
 
-// out[t] = table[ids[t]] * scale, fp32
+// out[t] = table[ids[t]] * scale (+ ptab[positions[t]]), fp32
 template <typename T>
 __global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float scale,
-                                 float* __restrict__ out, int W, int vocab) {
+                                 float* __restrict__ out, int W, int vocab, const int* __restrict__ positions,
+                                 const T* __restrict__ ptab, int n_pos) {
   const long long t = blockIdx.x;
   int id = ids[t];
   if (id < 0 || id >= vocab) id = 0;
   const T* src = table + static_cast<long long>(id) * W;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) out[t * W + i] = static_cast<float>(src[i]) * scale;
+  const T* ps = ptab != nullptr ? ptab + static_cast<long long>(min(max(positions[t], 0), n_pos - 1)) * W : nullptr;
+  for (int i = threadIdx.x; i < W; i += blockDim.x)
+    out[t * W + i] = static_cast<float>(src[i]) * scale + (ps != nullptr ? static_cast<float>(ps[i]) : 0.f);
 }
 
 // r = rows != NULL ? rows[i] : i;  x = resid[r] + (y != NULL ? norm(y[r]) * post : 0);  resid[r] = x where y is given and
@@ -152,6 +112,9 @@ resid_norm_kernel(float* __restrict__ resid, const T* __restrict__ y, long long 
 //   scores are chosen by score + correction, among the `keep` of `groups` equal runs of neighbouring experts whose two best
 //   choice scores have the largest sum. Weights: scores, divided by their sum with renorm, times wscale.
 //   shift: instead of h, S rows h + (before - h) mu_s per row, `before` = the slot's last row (0 at position 0), which h replaces.
+//   gate: what is added is multiplied by sigmoid(gate_z + gate_bias) first; side: y is side_scale times the sum of two rows, each
+//   divided by its root mean square and multiplied by its weights; bias: of the norm; conv: h and, n rows further, h + the causal
+//   convolution of h with the rows in the slot's ring, which takes h.
 // h_f32: h is stored as fp32.
 // The rows stay in shared memory (fp32) from the sum on; with several rows per CTA the router's weights are fetched once for
 // all of them.
@@ -180,14 +143,60 @@ struct SumNormArgs {
   const float* correction;
   float wscale;
   DmoeShift shift;            // n_mix = 0: none
+  const float* bias;
+  const void* gate_z;
+  long long ld_gate;
+  const float* gate_bias;
+  const void* side;
+  long long ld_side, side_stride;
+  const float* side_w;
+  float side_scale;
+  DmoeConv conv;              // taps = 0: none
 };
 // Segment of row i of a batch of one-token segments: {row, tokens (0: padding), slot, position}
-__device__ __forceinline__ int4 single_segment(const DmoeShift& s, long long i) {
+template <typename A>
+__device__ __forceinline__ int4 single_segment(const A& s, long long i) {
   if (s.singles != nullptr) return static_cast<const int4*>(s.singles)[i];
   return make_int4(static_cast<int>(i), s.kv_slots[i] >= 0 ? 1 : 0, s.rows[i], s.positions[i]);
 }
 constexpr int kSumThreads = 256, kSumWarps = kSumThreads / 32;
 constexpr int kMaxExperts = 256, kMaxTop = 32;
+
+// add += sum over the two sides of row / root mean square (with the scale: inv) * weights, columns v * VEC ..
+template <typename T, int VEC>
+__device__ __forceinline__ void add_sides(const T* side, long long stride, const float* w, int W, const float (&inv)[2], int v,
+                                          float* add) {
+#pragma unroll
+  for (int s = 0; s < 2; ++s) {
+    float t[VEC], f[VEC];
+    Pack<T, VEC>::load(side + s * stride + v * VEC, t);
+    Pack<float, VEC>::load(w + static_cast<long long>(s) * W + v * VEC, f);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) add[e] += t[e] * inv[s] * f[e];
+  }
+}
+
+// Row i of h (columns v * VEC .., as stored) -> its convolved row; the ring of the row's slot takes x.
+template <typename T, int VEC>
+__device__ __forceinline__ void convolve_single(const SumNormArgs& a, long long i, int v, const float* x) {
+  const int4 seg = single_segment(a.conv, i);
+  const int R = a.conv.taps, W = a.W, pos = seg.w;
+  const bool live = seg.y > 0 && seg.z >= 0 && seg.z < a.conv.n_slots;
+  T* ring = static_cast<T*>(a.conv.ring) + (live ? static_cast<long long>(seg.z) * R * W : 0) + v * VEC;
+  float y[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) y[e] = x[e];
+  for (int j = R - 1; j >= 0; --j) {
+    float t[VEC], w[VEC];
+    if (j > 0 && !(live && pos - j >= 0)) continue;
+    if (j > 0) Pack<T, VEC>::load(ring + static_cast<long long>((pos - j) % R) * W, t);
+    Pack<float, VEC>::load(a.conv.w + static_cast<long long>(R - 1 - j) * W + v * VEC, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y[e] += w[e] * (j > 0 ? t[e] : x[e]);
+  }
+  if (live && R > 1) Pack<T, VEC>::store(ring + static_cast<long long>(pos % R) * W, x);
+  Pack<T, VEC>::store(static_cast<T*>(a.h) + (a.n + i) * a.ld_h + v * VEC, y);
+}
 
 template <typename T, int VEC, int TPC>
 __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs a) {
@@ -217,11 +226,54 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
     return t;
   };
 
+  float sinv[2] = {0.f, 0.f};           // side_scale / root mean square of the two rows
+  const T* side = static_cast<const T*>(a.side) + (a.side != nullptr ? r * a.ld_side : 0);
+  if (a.side != nullptr) {
+#pragma unroll
+    for (int s = 0; s < 2; ++s) {
+      float ss = 0.f;
+      if (valid)
+        for (int v = tid; v < nvec; v += G) {
+          float t[VEC];
+          Pack<T, VEC>::load(side + s * a.side_stride + v * VEC, t);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) ss += t[e] * t[e];
+        }
+      sinv[s] = a.side_scale / sqrtf(group_sum(ss) / static_cast<float>(W) + a.eps);
+    }
+  }
   float sum = 0.f;
   if (valid) {
     for (int v = tid; v < nvec; v += G) {
       float x[VEC], t[VEC];
       Pack<float, VEC>::load(a.resid + r * W + v * VEC, x);
+      if (a.gate_z != nullptr) {
+        // the sublayer's result first, then its gate
+        float add[VEC] = {};
+        if (y != nullptr) Pack<T, VEC>::load(y + r * a.ld_y + v * VEC, add);
+        for (int p = 0; p < a.n_parts; ++p) {
+          Pack<T, VEC>::load(parts + r * a.part_row + p * a.part_stride + v * VEC, t);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) add[e] += t[e];
+        }
+        if (a.side != nullptr) add_sides<T, VEC>(side, a.side_stride, a.side_w, W, sinv, v, add);
+        float z[VEC];
+        Pack<T, VEC>::load(static_cast<const T*>(a.gate_z) + r * a.ld_gate + v * VEC, z);
+        Pack<float, VEC>::load(a.gate_bias + v * VEC, t);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += a.mult * add[e] / (1.f + expf(-(z[e] + t[e])));
+        if (a.rows == nullptr) Pack<float, VEC>::store(a.resid + r * W + v * VEC, x);
+        Pack<float, VEC>::store(row + v * VEC, x);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sum += x[e];
+        continue;
+      }
+      if (a.side != nullptr) {
+        float add[VEC] = {};
+        add_sides<T, VEC>(side, a.side_stride, a.side_w, W, sinv, v, add);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += a.mult * add[e];
+      }
       if (y != nullptr) {
         Pack<T, VEC>::load(y + r * a.ld_y + v * VEC, t);
 #pragma unroll
@@ -232,7 +284,7 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
 #pragma unroll
         for (int e = 0; e < VEC; ++e) x[e] += a.mult * t[e];
       }
-      if (a.rows == nullptr && (y != nullptr || a.n_parts > 0)) Pack<float, VEC>::store(a.resid + r * W + v * VEC, x);
+      if (a.rows == nullptr && (y != nullptr || a.n_parts > 0 || a.side != nullptr)) Pack<float, VEC>::store(a.resid + r * W + v * VEC, x);
       Pack<float, VEC>::store(row + v * VEC, x);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) sum += x[e];
@@ -277,6 +329,11 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
       Pack<float, VEC>::load(a.w + v * VEC, w);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x[e] = (x[e] - mean) * inv * w[e];
+      if (a.bias != nullptr) {
+        Pack<float, VEC>::load(a.bias + v * VEC, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += w[e];
+      }
       if (a.h_f32) {
         Pack<float, VEC>::store(static_cast<float*>(a.h) + i * a.ld_h + v * VEC, x);
         continue;
@@ -284,7 +341,8 @@ __global__ void __launch_bounds__(kSumThreads) sum_norm_kernel(const SumNormArgs
       Pack<T, VEC>::store(static_cast<T*>(a.h) + i * a.ld_h + v * VEC, x);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x[e] = static_cast<float>(static_cast<T>(x[e]));
-      Pack<float, VEC>::store(row + v * VEC, x);
+      if (a.conv.taps > 0) convolve_single<T, VEC>(a, i, v, x);
+      else Pack<float, VEC>::store(row + v * VEC, x);
     }
   if (a.gate_w == nullptr) return;
   __syncthreads();
@@ -469,7 +527,7 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
                     const long long* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache, int n_q, int n_kv,
                     int dk, int dv, int rot, int interleaved, const float2* __restrict__ table, int max_pos,
                     const float* __restrict__ qw, const float* __restrict__ kw, float eps, const T* __restrict__ v_first,
-                    long long ld_first, int first_head, float v_lambda, int tied) {
+                    long long ld_first, int first_head, float v_lambda, int tied, int v_norm) {
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int half = rot / 2;
@@ -509,7 +567,16 @@ qk_norm_rope_kernel(T* __restrict__ qkv, long long ld, const int* __restrict__ p
   if (slot >= 0) {
     const T* src = row + static_cast<long long>(tied ? n_q : n_q + n_kv) * dk;
     T* dst = vcache + slot * n_kv * dv;
-    for (int i = threadIdx.x; i < n_kv * dv; i += blockDim.x) {
+    for (int head = warp; v_norm > 0 && head < n_kv; head += nw) {
+      float ss = 0.f;
+      for (int d = lane; d < dv; d += 32) {
+        const float x = static_cast<float>(src[head * dv + d]);
+        ss += x * x;
+      }
+      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(v_norm) + eps);
+      for (int d = lane; d < dv; d += 32) dst[head * dv + d] = static_cast<T>(static_cast<float>(src[head * dv + d]) * inv);
+    }
+    for (int i = threadIdx.x; v_norm == 0 && i < n_kv * dv; i += blockDim.x) {
       if (v_first == nullptr) { dst[i] = src[tied ? i / dv * dk + i % dv : i]; continue; }
       const int d = i % dv;
       const float first = d < first_head ? static_cast<float>(v_first[t * ld_first + i / dv * first_head + d]) : 0.f;
@@ -525,7 +592,7 @@ __global__ void __launch_bounds__(256)
 rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__ positions, const long long* __restrict__ slots,
                    bf16* __restrict__ kcache, bf16* __restrict__ vcache, int n_q, int n_kv, int dk, int dv, int rot,
                    int interleaved, const float2* __restrict__ table, int max_pos, const bf16* __restrict__ v_first,
-                   long long ld_first, int first_head, float v_lambda, int tied) {
+                   long long ld_first, int first_head, float v_lambda, int tied, int v_norm, float eps) {
   const long long t = blockIdx.x;
   const int pos = min(max(positions[t], 0), max_pos - 1);
   const long long slot = slots[t];
@@ -565,6 +632,25 @@ rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__
   if (slot < 0) return;
   const bf16* src = row + static_cast<long long>(tied ? n_q : n_q + n_kv) * dk;
   bf16* dst = vcache + slot * n_kv * dv;
+  if (v_norm > 0) {                               // `lanes` threads of a warp per head
+    int lanes = 1;
+    while (lanes < dv / 8) lanes *= 2;
+    const int l = threadIdx.x & (lanes - 1);
+    for (int h0 = 0; h0 < n_kv; h0 += blockDim.x / lanes) {
+      const int head = h0 + threadIdx.x / lanes;
+      const bool on = head < n_kv && l < dv / 8;
+      float x[8] = {}, ss = 0.f;
+      if (on) Pack<bf16, 8>::load(src + head * dv + l * 8, x);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+      for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.f / sqrtf(ss / static_cast<float>(v_norm) + eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= inv;
+      if (on) Pack<bf16, 8>::store(dst + head * dv + l * 8, x);
+    }
+    return;
+  }
   for (int u = threadIdx.x; u < n_kv * dv / 8; u += blockDim.x) {
     float x[8];
     Pack<bf16, 8>::load(src + (tied ? u * 8 / dv * dk + u * 8 % dv : u * 8), x);
@@ -579,13 +665,20 @@ rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__
   }
 }
 
-// out[t, i] = act(gu[t, i]) * gu[t, I + i]
+// out[t, i] = act(gu[t, i]) * gu[t, I + i] (act, limit, recs: see DmoeGemm)
 template <typename T>
-__global__ void gate_mul_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ld_out, int I, int act) {
+__global__ void gate_mul_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ld_out, int I, int act,
+                                float limit, const int4* __restrict__ recs) {
   const long long t = blockIdx.y;
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= I) return;
-  const float g = static_cast<float>(gu[t * ld + i]), u = static_cast<float>(gu[t * ld + I + i]);
+  const float s = recs != nullptr ? __int_as_float(recs[t].z) : 1.f;
+  const float g = static_cast<float>(gu[t * ld + i]) * s, u = static_cast<float>(gu[t * ld + I + i]) * s;
+  if (act == 3) {
+    const float m = fminf(g, limit);
+    out[t * ld_out + i] = static_cast<T>(m / (1.f + expf(-1.702f * m)) * (fminf(fmaxf(u, -limit), limit) + 1.f));
+    return;
+  }
   const float v = act == 0 ? g / (1.f + expf(-g))
                            : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
   out[t * ld_out + i] = static_cast<T>(v * u);
@@ -593,14 +686,15 @@ __global__ void gate_mul_kernel(const T* __restrict__ gu, long long ld, T* __res
 
 // Y[t, f] = sum_k X[t, k] W[f, k] with fp32 multiply-adds: 64 x 64 tiles, 4 x 4 outputs per thread. With offs, W is a stack of
 // G matrices [F, K] and group g has rows offs[g] .. offs[g + 1] (blockIdx.y counts row tiles group after group); with recs, row
-// t is scaled and stored where its record {buffer, row or < 0, weight bits, -} says. act 2: tanh of the output.
+// t is scaled (not with `unit`) and stored where its record {buffer, row or < 0, weight bits, -} says. act 2: tanh of the output, 4:
+// silu of its first act_cols columns.
 constexpr int kSgTile = 64, kSgK = 16;
 
 template <typename T, typename TY>
 __global__ void __launch_bounds__(256)
 simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W, long long ldw, TY* __restrict__ Y,
                  long long ldy, int M, int F, int K, const int* __restrict__ offs, int G, const int4* __restrict__ recs,
-                 void* const* __restrict__ bases, int act) {
+                 void* const* __restrict__ bases, int act, int act_cols, int unit) {
   __shared__ float sx[kSgK][kSgTile + 4], sw[kSgK][kSgTile + 4];
   int t0 = blockIdx.y * kSgTile, t1 = M;
   const int f0 = blockIdx.x * kSgTile;
@@ -648,12 +742,13 @@ simt_gemm_kernel(const T* __restrict__ X, long long ldx, const T* __restrict__ W
       const int4 rec = recs[t];
       if (rec.y < 0) continue;
       dst = static_cast<TY*>(bases[rec.x]) + rec.y * ldy;
-      scale = __int_as_float(rec.z);
+      scale = unit ? 1.f : __int_as_float(rec.z);
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int f = f0 + tx * 4 + j;
-      if (f < F) dst[f] = static_cast<TY>(act == 2 ? tanhf(acc[i][j]) : acc[i][j] * scale);
+      const float v = acc[i][j];
+      if (f < F) dst[f] = static_cast<TY>(act == 2 ? tanhf(v) : act == 4 && f < act_cols ? v / (1.f + expf(-v)) : v * scale);
     }
   }
 }
@@ -707,15 +802,17 @@ static int launch_sum_norm(const SumNormArgs& a, cudaStream_t stream) {
 using namespace dmoe;
 
 extern "C" int dmoe_embed_f32(const int* ids, const void* table, int is_f32, float scale, float* out, int T, int W, int vocab,
-                              void* stream_) {
+                              const int* positions, const void* pos_table, int n_pos, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (W < 1 || vocab < 1) return -10;
+  if (W < 1 || vocab < 1 || (pos_table != nullptr && (positions == nullptr || n_pos < 1))) return -10;
   if (T == 0) return 0;
   const int threads = W >= 256 ? 256 : 64;
   if (is_f32)
-    embed_f32_kernel<float><<<T, threads, 0, stream>>>(ids, static_cast<const float*>(table), scale, out, W, vocab);
+    embed_f32_kernel<float><<<T, threads, 0, stream>>>(ids, static_cast<const float*>(table), scale, out, W, vocab, positions,
+                                                       static_cast<const float*>(pos_table), n_pos);
   else
-    embed_f32_kernel<bf16><<<T, threads, 0, stream>>>(ids, static_cast<const bf16*>(table), scale, out, W, vocab);
+    embed_f32_kernel<bf16><<<T, threads, 0, stream>>>(ids, static_cast<const bf16*>(table), scale, out, W, vocab, positions,
+                                                      static_cast<const bf16*>(pos_table), n_pos);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -740,7 +837,7 @@ extern "C" int dmoe_rope_freq_table(void* table, int max_pos, int half, const do
 extern "C" int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long ld_y, const void* parts, int n_parts,
                              long long part_row, long long part_stride, float mult, const float* w, int centred, float eps,
                              const int* rows, void* h, int h_f32, long long ld_h, int n, int W, const DmoeRouter* router,
-                             const DmoeShift* shift, void* stream_) {
+                             const DmoeShift* shift, const DmoeSumExtra* extra, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (W < 1 || resid == nullptr || h == nullptr || w == nullptr || n_parts < 0) return -10;
   static const DmoeRouter no_router = {};
@@ -752,13 +849,25 @@ extern "C" int dmoe_sum_norm(int is_f32, float* resid, const void* y, long long 
   if (r.sigmoid && (r.groups < 1 || r.E % r.groups != 0 || r.keep < 1)) return -10;
   if (shift != nullptr && (rows != nullptr || s.n_single != n || s.n_mix < 1 || s.mu == nullptr || s.last == nullptr ||
                            (s.singles == nullptr && (s.positions == nullptr || s.rows == nullptr || s.kv_slots == nullptr)))) return -10;
+  static const DmoeSumExtra no_extra = {};
+  static const DmoeConv no_conv = {};
+  const DmoeSumExtra& x = extra != nullptr ? *extra : no_extra;
+  const DmoeConv& c = x.conv != nullptr ? *x.conv : no_conv;
+  if ((x.gate_z != nullptr && x.gate_bias == nullptr) || (x.side != nullptr && (x.side_w == nullptr || y != nullptr))) return -10;
+  if (shift != nullptr && x.bias != nullptr) return -10;
+  if (x.conv != nullptr && (rows != nullptr || router != nullptr || shift != nullptr || h_f32 || c.n_single != n || c.taps < 1 ||
+                            c.w == nullptr || c.ring == nullptr || c.n_slots < 1 ||
+                            (c.singles == nullptr && (c.positions == nullptr || c.rows == nullptr || c.kv_slots == nullptr)))) return -10;
   if (n == 0) return 0;
   if (parts == nullptr) n_parts = 0;
   const SumNormArgs a{resid, y, ld_y, parts, n_parts, part_row, part_stride, w, centred, eps, rows, h, ld_h, n, W, r.weight, r.E,
-                      r.K, r.renorm, r.ids, r.wts, r.counts, mult, h_f32, r.sigmoid, r.groups, r.keep, r.correction, r.wscale, s};
+                      r.K, r.renorm, r.ids, r.wts, r.counts, mult, h_f32, r.sigmoid, r.groups, r.keep, r.correction, r.wscale, s,
+                      x.bias, x.gate_z, x.ld_gate, x.gate_bias, x.side, x.ld_side, x.side_stride, x.side_w, x.side_scale, c};
   const bool vec = W % 8 == 0 && ld_y % 8 == 0 && ld_h % 8 == 0 && part_row % 8 == 0 && part_stride % 8 == 0 && aligned16(resid) &&
                    aligned16(y) && aligned16(parts) && aligned16(w) && aligned16(h) && aligned16(r.weight) && aligned16(s.mu) &&
-                   aligned16(s.last) && s.mix_stride % 8 == 0;
+                   aligned16(s.last) && s.mix_stride % 8 == 0 && aligned16(x.bias) && aligned16(x.gate_z) && aligned16(x.gate_bias) &&
+                   aligned16(x.side) && aligned16(x.side_w) && x.ld_gate % 8 == 0 && x.ld_side % 8 == 0 && x.side_stride % 8 == 0 &&
+                   aligned16(c.w) && aligned16(c.ring);
   if (is_f32) return vec ? launch_sum_norm<float, 8>(a, stream) : launch_sum_norm<float, 1>(a, stream);
   return vec ? launch_sum_norm<bf16, 8>(a, stream) : launch_sum_norm<bf16, 1>(a, stream);
 }
@@ -788,57 +897,59 @@ extern "C" int dmoe_token_shift(int is_f32, const float* h, const DmoeShift* s, 
 extern "C" int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int* positions, const long long* slots,
                                  void* kcache, void* vcache, int T, int n_q, int n_kv, int dk, int dv, int rot, int interleaved,
                                  const void* table, int max_pos, const float* qw, const float* kw, float eps,
-                                 const void* v_first, long long ld_first, int first_head, float v_lambda, int tied,
+                                 const void* v_first, long long ld_first, int first_head, float v_lambda, int tied, int v_norm,
                                  void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (n_q < 1 || n_kv < 0 || dk < 1 || rot < 0 || rot % 2 != 0 || rot > dk || (rot > 0 && table == nullptr)) return -10;
   if (n_kv > 0 && (kcache == nullptr || vcache == nullptr || (qw != nullptr && kw == nullptr))) return -10;
   if (v_first != nullptr && (first_head < 1 || tied)) return -10;
   if (tied && dv > dk) return -10;
+  if (v_norm < 0 || (v_norm > 0 && (tied || v_first != nullptr || v_norm > dv))) return -10;
   if (T == 0) return 0;
   int threads = (n_q + n_kv) * 32;
   if (threads > 256) threads = 256;
-  if (!is_f32 && qw == nullptr && n_kv > 0 && dk % 8 == 0 && dv % 8 == 0 && rot % (interleaved ? 8 : 16) == 0 &&
+  if (!is_f32 && qw == nullptr && n_kv > 0 && (v_norm == 0 || dv <= 256) && dk % 8 == 0 && dv % 8 == 0 && rot % (interleaved ? 8 : 16) == 0 &&
       ld % 8 == 0 && first_head % 8 == 0 && ld_first % 8 == 0 && aligned16(qkv) && aligned16(kcache) && aligned16(vcache) &&
       aligned16(v_first)) {
     rope_append_kernel<<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk, dv,
         rot, interleaved, static_cast<const float2*>(table), max_pos, static_cast<const bf16*>(v_first), ld_first, first_head,
-        v_lambda, tied);
+        v_lambda, tied, v_norm, eps);
     return static_cast<int>(cudaGetLastError());
   }
   if (is_f32)
     qk_norm_rope_kernel<float><<<T, threads, 0, stream>>>(
         static_cast<float*>(qkv), ld, positions, slots, static_cast<float*>(kcache), static_cast<float*>(vcache), n_q, n_kv,
         dk, dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const float*>(v_first),
-        ld_first, first_head, v_lambda, tied);
+        ld_first, first_head, v_lambda, tied, v_norm);
   else
     qk_norm_rope_kernel<bf16><<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk,
         dv, rot, interleaved, static_cast<const float2*>(table), max_pos, qw, kw, eps, static_cast<const bf16*>(v_first),
-        ld_first, first_head, v_lambda, tied);
+        ld_first, first_head, v_lambda, tied, v_norm);
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int dmoe_gate_mul(int is_f32, int act, const void* gu, long long ld, void* out, long long ld_out, int T, int I,
-                             void* stream_) {
+                             float limit, const void* recs, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (I < 1 || act < 0 || act > 1) return -10;
+  if (I < 1 || (act != 0 && act != 1 && act != 3)) return -10;
   for (int t0 = 0; t0 < T; t0 += 65535) {      // grid.y limit
     const int n = T - t0 < 65535 ? T - t0 : 65535;
     const dim3 grid((I + 255) / 256, n);
+    const int4* rc = recs != nullptr ? static_cast<const int4*>(recs) + t0 : nullptr;
     if (is_f32)
       gate_mul_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(gu) + t0 * ld, ld,
-                                                       static_cast<float*>(out) + t0 * ld_out, ld_out, I, act);
+                                                       static_cast<float*>(out) + t0 * ld_out, ld_out, I, act, limit, rc);
     else
       gate_mul_kernel<bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(gu) + t0 * ld, ld,
-                                                      static_cast<bf16*>(out) + t0 * ld_out, ld_out, I, act);
+                                                      static_cast<bf16*>(out) + t0 * ld_out, ld_out, I, act, limit, rc);
   }
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long ldx, const void* W, long long ldw, void* Y,
-                                long long ldy, int T, int F, int K, int act, void* stream_) {
+                                long long ldy, int T, int F, int K, int act, int act_cols, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (F < 1 || K < 1 || (x_f32 && !y_f32)) return -10;
   if (T == 0) return 0;
@@ -847,18 +958,19 @@ extern "C" int dmoe_simt_linear(int x_f32, int y_f32, const void* X, long long l
   const dim3 grid((F + kSgTile - 1) / kSgTile, static_cast<unsigned>(ty));
   if (x_f32)
     simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W),
-                                                             ldw, static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
+                                                             ldw, static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act, act_cols, 0);
   else if (y_f32)
     simt_gemm_kernel<bf16, float><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                            static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
+                                                            static_cast<float*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act, act_cols, 0);
   else
     simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), ldw,
-                                                           static_cast<bf16*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act);
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, nullptr, 0, nullptr, nullptr, act, act_cols, 0);
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y,
-                                 long long ldy, const void* recs, const void* bases, int T, int F, int K, void* stream_) {
+extern "C" int dmoe_simt_grouped(int is_f32, int y_f32, const void* X, long long ldx, const void* W, const int* offs, int G, void* Y,
+                                 long long ldy, const void* recs, const void* bases, int unit_weights, int T, int F, int K,
+                                 void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (F < 1 || K < 1 || G < 1 || offs == nullptr || (recs == nullptr && Y == nullptr) || (recs != nullptr && bases == nullptr)) return -10;
   if (T == 0) return 0;
@@ -869,9 +981,12 @@ extern "C" int dmoe_simt_grouped(int is_f32, const void* X, long long ldx, const
   void* const* b = static_cast<void* const*>(bases);
   if (is_f32)
     simt_gemm_kernel<float, float><<<grid, 256, 0, stream>>>(static_cast<const float*>(X), ldx, static_cast<const float*>(W), K,
-                                                             static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b, 0);
+                                                             static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b, 0, 0, unit_weights);
+  else if (y_f32)
+    simt_gemm_kernel<bf16, float><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), K,
+                                                            static_cast<float*>(Y), ldy, T, F, K, offs, G, r, b, 0, 0, unit_weights);
   else
     simt_gemm_kernel<bf16, bf16><<<grid, 256, 0, stream>>>(static_cast<const bf16*>(X), ldx, static_cast<const bf16*>(W), K,
-                                                           static_cast<bf16*>(Y), ldy, T, F, K, offs, G, r, b, 0);
+                                                           static_cast<bf16*>(Y), ldy, T, F, K, offs, G, r, b, 0, 0, unit_weights);
   return static_cast<int>(cudaGetLastError());
 }

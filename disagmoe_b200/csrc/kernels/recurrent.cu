@@ -5,6 +5,10 @@
 //   delta   S <- diag(a) S;  S <- S + k (beta (v - S^T k))^T       (gated delta rule)
 //   o = S^T q, read after the write
 //   bonus   o = (S + diag(u) k v^T)^T q, then the plain write      (RWKV-style time mixing)
+//   memory  the plain write with k scaled and one decay per head and token, both relative to a running maximum m of the logs of
+//           the gates; o = S^T q / (max(|n.q|, e^-m) + 1e-6) with n <- a n + k            (matrix memory of xLSTM)
+//
+// Plain writes also come with one constant decay per head (lightning attention).
 //
 // States live in slots: slot = block-table row of the sequence, so a sequence's state is found with the same index as
 // its KV pages, and a sequence whose first token is in the batch (position 0) starts from zero whatever the slot held.
@@ -23,14 +27,38 @@ namespace dmoe {
 constexpr int kStepThreads = 256;
 constexpr int kStepRows = 16;        // state rows a thread holds in registers
 
-// Decay factor, q and k of the token's key channels and its values -> shared memory (convolved and activated with CONV).
+// Matrix memory: decay factor, factor of k and running maximum of a token, from the arrays of dmoe_memory_gates or, for a token on
+// its own, from its gates and the slot's maximum.
+struct TokenGates {
+  float keep, put, top;
+};
+__device__ __forceinline__ TokenGates token_gates(const DmoeRecur& a, long long row, int pos, int slot, int h) {
+  TokenGates g;
+  if (a.keep != nullptr) {
+    const long long at = row * a.heads + h;
+    g.keep = expf(a.keep[at]);
+    g.put = a.put[at];
+    g.top = a.run_max[at];
+    return g;
+  }
+  float i, f;
+  memory_logs(a, row, h, i, f);
+  if (pos > 0) f += *max_state(a, slot, pos - 1, h);
+  g.top = fmaxf(f, i);
+  g.keep = expf(f - g.top);
+  g.put = expf(i - g.top);
+  return g;
+}
+
+// Decay factor, q and k of the token's key channels and its values -> shared memory (convolved and activated with CONV). Matrix
+// memory: with them the normaliser, which moves on in its slot (the CTA of the first value columns has it).
 template <typename T, int MODE, bool CONV>
 __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, int pos, int slot, int h, int hk, int v0, int nv,
-                                             float scale, float4* s_gqk, float* s_v) {
+                                             float scale, const TokenGates& tg, float4* s_gqk, float* s_v) {
   const int D = a.dim, V = a.vdim, group = a.heads / a.kv_heads;
   for (int i = threadIdx.x; i < D + nv; i += blockDim.x) {
     if (i < D) {
-      const float z = a.z[row * a.ldz + h * D + i] + a.z_bias[h * D + i];
+      const float z = MODE != kMemory && a.z != nullptr ? a.z[row * a.ldz + h * D + i] + a.z_bias[h * D + i] : 0.f;
       float q, k;
       if (CONV) {
         ConvInputs<T> xq, xk;
@@ -42,6 +70,16 @@ __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, 
       } else {
         q = static_cast<float>(static_cast<const T*>(a.q)[row * a.ldq + hk * D + i]);
         k = static_cast<float>(static_cast<const T*>(a.k)[row * a.ldk + hk * D + i]);
+      }
+      if (MODE == kMemory) {
+        float n = 0.f;
+        if (v0 == 0) {
+          float* np = a.norm_state + (static_cast<long long>(slot) * a.heads + h) * D + i;
+          if (pos > 0) n = *np;
+          *np = tg.keep * n + tg.put * k;
+        }
+        s_gqk[i] = make_float4(tg.keep, q, k, n);
+        continue;
       }
       s_gqk[i] = make_float4(expf(log_decay(a.decay_kind, z, scale)), q, k, MODE == kBonus ? a.bonus[h * D + i] : 0.f);
     } else {
@@ -58,23 +96,29 @@ __device__ __forceinline__ void token_inputs(const DmoeRecur& a, long long row, 
 }
 
 // Factors that turn the raw rows into q (scaled, unit) and k (unit), and the weight of the token's own write in its read-out:
-// q.k of the raw rows, with the bonus q.(u k); every warp on its own.
+// q.k of the raw rows, with the bonus q.(u k); every warp on its own. Matrix memory: the factor of the read-out.
 struct RowFactors {
-  float fq, fk, qk;
+  float fq, fk, qk, scale;
 };
 template <int MODE>
-__device__ __forceinline__ RowFactors row_factors(const DmoeRecur& a, const float4* s_gqk) {
-  float qq = 0.f, kk = 0.f, qk = 0.f;
+__device__ __forceinline__ RowFactors row_factors(const DmoeRecur& a, const float4* s_gqk, const TokenGates& tg) {
+  float qq = 0.f, kk = 0.f, qk = 0.f, nq = 0.f;
   for (int d = threadIdx.x & 31; d < a.dim; d += 32) {
     const float4 x = s_gqk[d];
     qq += x.y * x.y;
     kk += x.z * x.z;
     qk += MODE == kBonus ? x.y * (x.z * x.w) : x.y * x.z;
+    if (MODE == kMemory) nq += x.y * x.w;
   }
   RowFactors f;
   f.qk = warp_sum(qk);
   f.fq = a.qscale;
   f.fk = 1.f;
+  f.scale = 1.f;
+  if (MODE == kMemory) {
+    f.fk = tg.put;
+    f.scale = memory_scale((tg.keep * warp_sum(nq) + tg.put * f.qk) * f.fq, tg.top);
+  }
   if (MODE == kDelta) {
     f.fq *= 1.f / sqrtf(warp_sum(qq) + 1e-6f);
     f.fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
@@ -131,9 +175,15 @@ step_kernel(const DmoeRecur a, int vt) {
       gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + oc]);
       weight = norm_w[oc];
     }
-    token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, v0, nv, dscale, s_gqk, s_v);
+    TokenGates tg = {};
+    if (MODE == kMemory) {
+      tg = token_gates(a, row, pos, slot, h);
+      if (a.keep == nullptr && v0 == 0 && tid == 0) *max_state(a, slot, pos, h) = tg.top;
+    }
+    token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, v0, nv, dscale, tg, s_gqk, s_v);
     __syncthreads();
-    const RowFactors f = row_factors<MODE>(a, s_gqk);
+    const RowFactors f = row_factors<MODE>(a, s_gqk, tg);
+    if (MODE == kMemory && !fused && v0 == 0 && tid == 0) a.scale[row * a.heads + h] = f.scale;
     const float fq = f.fq, fk = f.fk, qk = f.qk;
     if (DELTA) beta = 1.f / (1.f + expf(-beta));
     float rq[VEC], rk[VEC];
@@ -169,7 +219,7 @@ step_kernel(const DmoeRecur a, int vt) {
       if (DELTA) u = beta * (u - ok * fk);
       s_u[c] = u * fk;
       const float o = oq * fq + qk * fq * fk * u;
-      if (fused) s_o[c] = o;
+      if (fused) s_o[c] = o * f.scale;
       else a.raw[row * a.ldraw + h * V + v0 + c] = o;
     }
     __syncthreads();
@@ -245,13 +295,20 @@ stream_step_kernel(const DmoeRecur a) {
   const float* norm_w = a.norm_w + h * a.norm_ld;
   float beta = 0.f, gate = 0.f, weight = 0.f;
   if (DELTA) beta = static_cast<float>(static_cast<const T*>(a.beta)[row * a.ldb + h]);
-  if (tid < V) {
+  const bool fused = a.raw == nullptr;
+  if (fused && tid < V) {
     gate = static_cast<float>(static_cast<const T*>(a.gate)[row * a.ldg + h * V + tid]);
     weight = norm_w[tid];
   }
-  token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, 0, V, decay_scale(a, h), s_gqk, s_v);
+  TokenGates tg = {};
+  if (MODE == kMemory) {
+    tg = token_gates(a, row, pos, slot, h);
+    if (tid == 0) *max_state(a, slot, pos, h) = tg.top;
+  }
+  token_inputs<T, MODE, CONV>(a, row, pos, slot, h, hk, 0, V, decay_scale(a, h), tg, s_gqk, s_v);
   __syncthreads();                                               // the inputs, and the barrier's initialisation
-  const RowFactors f = row_factors<MODE>(a, s_gqk);
+  const RowFactors f = row_factors<MODE>(a, s_gqk, tg);
+  if (MODE == kMemory && !fused && tid == 0) a.scale[row * a.heads + h] = f.scale;
   if (DELTA) beta = 1.f / (1.f + expf(-beta));
   if (pos > 0 && !mbar_wait(bar, 0, &s_abort) && tid == 0 && a.status != nullptr) atomicExch(a.status, kStatusBarrierTimeout);
   float rq[4] = {0.f, 0.f, 0.f, 0.f}, rk[4] = {0.f, 0.f, 0.f, 0.f};
@@ -288,7 +345,9 @@ stream_step_kernel(const DmoeRecur a) {
     float u = s_v[c];
     if (DELTA) u = beta * (u - ok * f.fk);
     s_u[c] = u * f.fk;
-    s_o[c] = oq * f.fq + f.qk * f.fq * f.fk * u;
+    const float o = oq * f.fq + f.qk * f.fq * f.fk * u;
+    if (fused) s_o[c] = o * f.scale;
+    else a.raw[row * a.ldraw + h * V + c] = o;
   }
   __syncthreads();
   if (mine) {
@@ -302,6 +361,7 @@ stream_step_kernel(const DmoeRecur a) {
           make_float4(s.x * x.x + x.z * u.x, s.y * x.x + x.z * u.y, s.z * x.x + x.z * u.z, s.w * x.x + x.z * u.w);
     }
   }
+  if (!fused) return;
   float ss = 0.f;
   for (int c = lane; c < V; c += 32) ss += s_o[c] * s_o[c];
   const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(V) + a.eps);
@@ -320,7 +380,7 @@ template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, long long ldraw, const T* __restrict__ gate,
                  long long ldg, const float* __restrict__ norm_w, int norm_ld, float eps, int gate_kind, T* __restrict__ out,
-                 long long ldo, int heads, int V, int lanes) {
+                 long long ldo, int heads, int V, int lanes, const float* __restrict__ scale) {
   const int4 e = table != nullptr ? table[blockIdx.x] : make_int4(blockIdx.x, 1, 0, 0);
   const int lane = threadIdx.x & (lanes - 1), per = blockDim.x / lanes;       // (row, head) pairs of the CTA at a time
   const auto sum = [&](float v) {                // over the lanes of a pair; the whole warp takes part
@@ -336,6 +396,7 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
     const float* r = raw + row * ldraw + h * V;
     const T* gp = gate + row * ldg + h * V;
     const float* nw = norm_w + h * norm_ld;
+    const float f = scale != nullptr ? scale[row * heads + h] : 1.f;
     float x[VEC], gv[VEC], w[VEC];
     float ss = 0.f;
     const int c0 = lane * VEC;
@@ -352,7 +413,7 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
 #pragma unroll
       for (int k = 0; k < VEC; ++k) ss += y[k] * y[k];
     }
-    const float inv = 1.f / sqrtf(sum(ss) / static_cast<float>(V) + eps);
+    const float inv = f / sqrtf(sum(ss) * f * f / static_cast<float>(V) + eps);
     for (int c = on ? c0 : V; c < V; c += lanes * VEC) {
       if (c != c0) {
         load_vec<VEC>(r + c, x);
@@ -363,6 +424,119 @@ gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, 
       for (int k = 0; k < VEC; ++k) x[k] *= inv * w[k] * gate_value(gate_kind, gv[k]);
       store_any<VEC>(out + row * ldo + h * V + c, x);
     }
+  }
+}
+
+// The same where all heads are normed together: one CTA per row, its first NV * 256 * VEC columns in registers.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+wide_gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ raw, long long ldraw, const T* __restrict__ gate,
+                      long long ldg, const float* __restrict__ norm_w, float eps, int gate_kind, T* __restrict__ out,
+                      long long ldo, int V) {
+  constexpr int NV = 2;
+  __shared__ float s_part[2][8];
+  const int4 e = table != nullptr ? table[blockIdx.x] : make_int4(blockIdx.x, 1, 0, 0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int buf = 0;
+  for (int t = blockIdx.y; t < e.y; t += gridDim.y, buf ^= 1) {
+    const long long row = e.x + t;
+    const float* r = raw + row * ldraw;
+    float x[NV][VEC], gv[NV][VEC], w[VEC], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * 256 + threadIdx.x) * VEC;
+      if (c < V) {
+        load_vec<VEC>(r + c, x[k]);
+        load_any<VEC>(gate + row * ldg + c, gv[k]);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss += x[k][i] * x[k][i];
+      }
+    }
+    for (int c = (NV * 256 + threadIdx.x) * VEC; c < V; c += 256 * VEC) {
+      float y[VEC];
+      load_vec<VEC>(r + c, y);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss += y[i] * y[i];
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) s_part[buf][warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) ss += s_part[buf][k];
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(V) + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * 256 + threadIdx.x) * VEC;
+      if (c < V) {
+        load_vec<VEC>(norm_w + c, w);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[k][i] *= inv * w[i] * gate_value(gate_kind, gv[k][i]);
+        store_any<VEC>(out + row * ldo + c, x[k]);
+      }
+    }
+    for (int c = (NV * 256 + threadIdx.x) * VEC; c < V; c += 256 * VEC) {
+      float y[VEC], g[VEC];
+      load_vec<VEC>(r + c, y);
+      load_any<VEC>(gate + row * ldg + c, g);
+      load_vec<VEC>(norm_w + c, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) y[i] *= inv * w[i] * gate_value(gate_kind, g[i]);
+      store_any<VEC>(out + row * ldo + c, y);
+    }
+  }
+}
+
+// Matrix memory, longer segments: log decay, factor of k and running maximum of every token, one CTA per (segment, head), 256 tokens
+// at a time. With F the running sum of the logs f, m_t = F_t + max(m_0, max_{j <= t} (i_j - F_j)).
+constexpr int kGateThreads = 256;
+__global__ void __launch_bounds__(kGateThreads) memory_gates_kernel(const DmoeRecur a) {
+  __shared__ float s_sum[kGateThreads / 32], s_max[kGateThreads / 32], s_top[kGateThreads];
+  const int4 seg = static_cast<const int4*>(a.segs)[blockIdx.x];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, slot = seg.z;
+  if (seg.y <= 0 || slot < 0 || slot >= a.n_slots) return;
+  float top = seg.w > 0 ? *max_state(a, slot, seg.w - 1, h) : 0.f;       // before the pass
+  float i = 0.f, f = 0.f;
+  if (tid < seg.y) memory_logs(a, seg.x + tid, h, i, f);
+  for (int t0 = 0; t0 < seg.y; t0 += kGateThreads) {
+    const int t = t0 + tid;
+    const bool on = t < seg.y;
+    float ni = 0.f, nf = 0.f;
+    if (t + kGateThreads < seg.y) memory_logs(a, seg.x + t + kGateThreads, h, ni, nf);
+    float F = on ? f : 0.f;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, F, o);
+      if (lane >= o) F += v;
+    }
+    if (lane == 31) s_sum[warp] = F;
+    __syncthreads();
+    for (int w = 0; w < warp; ++w) F += s_sum[w];
+    float best = on ? i - F : -INFINITY;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, best, o);
+      if (lane >= o) best = fmaxf(best, v);
+    }
+    if (lane == 31) s_max[warp] = best;
+    __syncthreads();
+    for (int w = 0; w < warp; ++w) best = fmaxf(best, s_max[w]);
+    const float m = F + fmaxf(top, best);
+    s_top[tid] = m;
+    __syncthreads();
+    if (on) {
+      const float before = tid > 0 ? s_top[tid - 1] : top;
+      const long long at = static_cast<long long>(seg.x + t) * a.heads + h;
+      // the maximum is only a scale: whatever its rounding, the steps below are exactly those between the stored values
+      a.keep[at] = f + before - m;
+      a.put[at] = expf(i - m);
+      a.run_max[at] = m;
+      if (t + 1 == seg.y) *max_state(a, slot, seg.w + t, h) = m;
+    }
+    top = s_top[kGateThreads - 1];
+    i = ni;
+    f = nf;
+    __syncthreads();                                     // s_top and the partial sums are rewritten
   }
 }
 
@@ -446,7 +620,11 @@ __global__ void __launch_bounds__(256) ring_update_kernel(const DmoeRecur a) {
 
 static int check_recur(const DmoeRecur* a) {
   if (a->heads < 1 || a->kv_heads < 1 || a->heads % a->kv_heads != 0 || a->dim < 1 || a->vdim < 1) return -10;
-  if (a->heads > 65535 || a->state == nullptr || a->z_bias == nullptr || a->n_slots < 1) return -10;
+  if (a->heads > 65535 || a->state == nullptr || a->n_slots < 1) return -10;
+  if (a->decay_kind < 3 ? a->z_bias == nullptr : a->decay_kind == 3 ? a->head_decay == nullptr
+                        : a->gates == nullptr || a->gate_bias == nullptr || a->norm_state == nullptr || a->max_state == nullptr) return -10;
+  if (a->decay_kind >= 3 && (a->delta || a->bonus != nullptr || a->taps > 0)) return -10;
+  if (a->decay_kind == 4 && a->raw != nullptr && a->scale == nullptr) return -10;
   if (a->segs == nullptr && (a->positions == nullptr || a->rows == nullptr || a->kv_slots == nullptr)) return -10;
   if ((a->decay_kind == 1 && a->a_log == nullptr) || (a->bonus != nullptr && (a->delta || a->taps > 0))) return -10;
   if (a->taps < 0 || a->taps > kMaxTaps || (a->taps > 0 && (a->conv_w == nullptr || a->ring == nullptr))) return -11;
@@ -462,7 +640,7 @@ static int stream_threads(const DmoeRecur& a) {
   return a.dim * a.vdim * 4 <= kSmallState && a.vdim <= 2 * kStepThreads ? kStepThreads / 2 : kStepThreads;
 }
 static size_t stream_smem(const DmoeRecur& a) {
-  if (a.raw != nullptr || a.vdim % 4 != 0 || a.vdim > 4 * kStepThreads || (reinterpret_cast<uintptr_t>(a.state) & 15) != 0)
+  if (a.vdim % 4 != 0 || a.vdim > 4 * kStepThreads || (reinterpret_cast<uintptr_t>(a.state) & 15) != 0)
     return 0;
   const int rpp = stream_threads(a) / (a.vdim / 4);
   const size_t b = (static_cast<size_t>(a.dim) * a.vdim + 4 * a.dim + a.vdim + static_cast<size_t>(a.delta ? 2 : 1) * rpp * a.vdim) * 4;
@@ -498,12 +676,15 @@ static int launch_step(const DmoeRecur& a, int vt, cudaStream_t stream) {
 template <typename T>
 static int step_dispatch(const DmoeRecur& a, int vt, bool vec, cudaStream_t stream) {
   const bool conv = a.taps > 0;
-  const size_t smem = a.one_token ? stream_smem(a) : 0;
+  const size_t smem = a.one_token && vt >= a.vdim ? stream_smem(a) : 0;
   if (smem > 0) {
+    if (a.decay_kind == 4) return launch_stream<T, kMemory, false>(a, smem, stream);
     if (a.bonus != nullptr) return launch_stream<T, kBonus, false>(a, smem, stream);
     if (!a.delta) return conv ? -12 : launch_stream<T, kPlain, false>(a, smem, stream);
     return conv ? launch_stream<T, kDelta, true>(a, smem, stream) : launch_stream<T, kDelta, false>(a, smem, stream);
   }
+  if (a.decay_kind == 4)
+    return vec ? launch_step<T, kMemory, false, 4>(a, vt, stream) : launch_step<T, kMemory, false, 1>(a, vt, stream);
   if (a.bonus != nullptr)
     return vec ? launch_step<T, kBonus, false, 4>(a, vt, stream) : launch_step<T, kBonus, false, 1>(a, vt, stream);
   if (!a.delta) {
@@ -539,6 +720,7 @@ extern "C" int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream_) {
   if (a->n_segs == 0) return 0;
   const bool vec = a->vdim % 4 == 0 && vt % 4 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 15) == 0;
   const int per = vec ? 4 : 1;
+  if (a->decay_kind == 4 && !a->one_token && (a->keep == nullptr || a->put == nullptr || a->run_max == nullptr)) return -15;
   if (vt < 1 || vt / per > kStepThreads || static_cast<long long>(kStepThreads / (vt / per)) * kStepRows < a->dim) return -13;
   if (a->raw == nullptr && (vt < a->vdim || a->out == nullptr || a->gate == nullptr || a->norm_w == nullptr)) return -14;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
@@ -547,10 +729,25 @@ extern "C" int dmoe_recur_step(const DmoeRecur* a, int vt, void* stream_) {
 
 extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_tokens, const float* raw, long long ldraw,
                               const void* gate, long long ldg, const float* norm_w, int norm_ld, float eps, int gate_kind, void* out,
-                              long long ldo, int heads, int V, void* stream_) {
+                              long long ldo, int heads, int V, const float* scale, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (heads < 1 || V < 1 || max_tokens < 1) return -10;
   if (n == 0) return 0;
+  if (heads == 1 && V > 512 && scale == nullptr) {
+    const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool v4 = V % 4 == 0 && ldraw % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al16(raw) && al16(gate) && al16(out) && al16(norm_w);
+    const dim3 g(n, max_tokens < 64 ? max_tokens : 64);
+    const int4* tb = static_cast<const int4*>(table);
+#define DMOE_WIDE(T_, VEC_)                                                                                                    \
+  wide_gate_norm_kernel<T_, VEC_><<<g, 256, 0, stream>>>(tb, raw, ldraw, static_cast<const T_*>(gate), ldg, norm_w, eps, gate_kind, \
+                                                         static_cast<T_*>(out), ldo, V)
+    if (is_f32 && v4) DMOE_WIDE(float, 4);
+    else if (is_f32) DMOE_WIDE(float, 1);
+    else if (v4) DMOE_WIDE(__nv_bfloat16, 4);
+    else DMOE_WIDE(__nv_bfloat16, 1);
+#undef DMOE_WIDE
+    return static_cast<int>(cudaGetLastError());
+  }
   long long by = (static_cast<long long>(max_tokens) * heads + 31) / 32;     // about four (row, head) pairs per warp
   if (by > 1024) by = 1024;
   const dim3 grid(n, static_cast<unsigned>(by));
@@ -561,7 +758,7 @@ extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_toke
 #define DMOE_GATE_NORM(T_, VEC_)                                                                                       \
   gate_norm_kernel<T_, VEC_><<<grid, 256, 0, stream>>>(static_cast<const int4*>(table), raw, ldraw,                    \
                                                        static_cast<const T_*>(gate), ldg, norm_w, norm_ld, eps, gate_kind, \
-                                                       static_cast<T_*>(out), ldo, heads, V, lanes)
+                                                       static_cast<T_*>(out), ldo, heads, V, lanes, scale)
   if (is_f32) {
     if (vec) DMOE_GATE_NORM(float, 4);
     else DMOE_GATE_NORM(float, 1);
@@ -570,6 +767,15 @@ extern "C" int dmoe_gate_norm(int is_f32, const void* table, int n, int max_toke
     else DMOE_GATE_NORM(__nv_bfloat16, 1);
   }
 #undef DMOE_GATE_NORM
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dmoe_memory_gates(const DmoeRecur* a, void* stream) {
+  const int rc = check_recur(a);
+  if (rc != 0) return rc;
+  if (a->decay_kind != 4 || a->segs == nullptr || a->keep == nullptr || a->put == nullptr || a->run_max == nullptr) return -15;
+  if (a->n_segs == 0) return 0;
+  memory_gates_kernel<<<dim3(a->n_segs, a->heads), kGateThreads, 0, static_cast<cudaStream_t>(stream)>>>(*a);
   return static_cast<int>(cudaGetLastError());
 }
 

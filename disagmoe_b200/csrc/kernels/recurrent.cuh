@@ -6,7 +6,7 @@
 namespace dmoe {
 
 constexpr int kMaxTaps = 8;
-enum { kPlain = 0, kDelta = 1, kBonus = 2 };      // MODE of the kernels: how a token writes and where it reads, see recurrent.cu
+enum { kPlain = 0, kDelta = 1, kBonus = 2, kMemory = 3 };      // MODE of the kernels: how a token writes and where it reads, see recurrent.cu
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -27,14 +27,27 @@ __device__ __forceinline__ float log1p_unit(float e) {
   return 2.f * (s + s * q * p);
 }
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1p_unit(expf(-fabsf(x))); }
-// log of the decay of one key channel: kind 0: log sigmoid(z) * scale, kind 1: -scale * softplus(z), kind 2: -exp(z)
+// log of the decay of one key channel: kind 0: log sigmoid(z) * scale, kind 1: -scale * softplus(z), kind 2: -exp(z), kind 3: scale
 __device__ __forceinline__ float log_decay(int kind, float z, float scale) {
   if (kind == 2) return -expf(z);
+  if (kind == 3) return scale;
   return kind == 0 ? -softplus(-z) * scale : -scale * softplus(z);
 }
 __device__ __forceinline__ float decay_scale(const DmoeRecur& a, int h) {
-  return a.decay_kind == 0 ? a.inv_tau : a.decay_kind == 1 ? expf(a.a_log[h]) : 1.f;
+  return a.decay_kind == 0 ? a.inv_tau : a.decay_kind == 1 ? expf(a.a_log[h]) : a.decay_kind == 3 ? a.head_decay[h] : 1.f;
 }
+// Matrix memory: logs of the input and the forget gate of a token
+__device__ __forceinline__ void memory_logs(const DmoeRecur& a, long long row, int h, float& i, float& f) {
+  const float* z = a.gates + row * a.ldgates;
+  i = a.gate_cap * tanhf((z[h] + a.gate_bias[h]) / a.gate_cap);
+  f = -softplus(-a.gate_cap * tanhf((z[a.heads + h] + a.gate_bias[a.heads + h]) / a.gate_cap));
+}
+// the running maximum in the slot is kept at the parity of its position: what one CTA writes no other one of the step reads
+__device__ __forceinline__ float* max_state(const DmoeRecur& a, int slot, int pos, int h) {
+  return a.max_state + (static_cast<long long>(slot) * 2 + (pos & 1)) * a.heads + h;
+}
+// factor of a read-out: 1 / (max(|n . q|, exp(-m)) + 1e-6)
+__device__ __forceinline__ float memory_scale(float nq, float m) { return 1.f / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f); }
 __device__ __forceinline__ float gate_value(int kind, float g) { return (kind == 0 ? g : 1.f) / (1.f + expf(-g)); }
 
 // Segment i of a decode step: row i alone.

@@ -15,6 +15,11 @@
 // chunk_scan_kernel then walks the chunks of a segment in order, one CTA per (segment, head, value tile), with the state in
 // its accumulators.
 //
+// Where a head has one decay (constant, or a matrix memory's), b_t is a number: P = (q k^T) e^(b_t - b_j) with the exponent applied to
+// the products of the rows as they are, and the factors of q and k are those of their rows (chunk_prep_head_kernel). The normaliser of a
+// matrix memory is one more value tile of the scan, whose only column is ones and whose state lies in n; the CTA that has it
+// turns n.q into the factor of the read-outs.
+//
 // Precision: decays, their sums and exponentials, unit norms, T and the state are fp32; matrix products split both
 // operands into bf16 hi + lo parts and accumulate in fp32 (see mma_sync.cuh). P and A are products of rows scaled by
 // e^(b_t - m) and e^(m - b_j), m = b in the middle of the chunk; where a channel decays so fast that these could
@@ -601,14 +606,132 @@ chunk_prep_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* _
   }
 }
 
+// Preparation where a head has one decay. Warps 0-3: P; warps 4-7: the fragments of q e^b and (k e^(b_end - b))^T.
+template <int DP, bool MEM>
+__global__ void __launch_bounds__(kChunkThreads, 3)
+chunk_prep_head_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8_t* __restrict__ ws, long long ws_stride, int h0) {
+  using L = ChunkWs<DP>;
+  constexpr int KS = DP / 16, MT = DP / 16, LD = DP + 8;
+  __shared__ __align__(16) __nv_bfloat16 s_q[kChunk * LD], s_k[kChunk * LD];
+  __shared__ float s_b[kChunk], s_put[kChunk];                  // running log2 decay; factor of k
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int lm_mi = lane >> 3, lm_r = lane & 7;
+  const int4 ck = chunks[blockIdx.x];
+  const long long row0 = ck.x;
+  const int n = ck.y, h = h0 + blockIdx.y, D = a.dim;
+  const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + row0 * a.ldq + h * D;
+  const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k) + row0 * a.ldk + h * D;
+  uint8_t* w = ws + (static_cast<long long>(blockIdx.x) * gridDim.y + blockIdx.y) * ws_stride;
+#pragma unroll
+  for (int i = tid; i < kChunk * DP / 8; i += kChunkThreads) {
+    const int t = i / (DP / 8), c = i % (DP / 8) * 8;
+    const bool in = t < n && c < D;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    *reinterpret_cast<uint4*>(s_q + t * LD + c) = in ? *reinterpret_cast<const uint4*>(qp + t * a.ldq + c) : zero;
+    *reinterpret_cast<uint4*>(s_k + t * LD + c) = in ? *reinterpret_cast<const uint4*>(kp + t * a.ldk + c) : zero;
+  }
+  if (warp == 0) {                                               // two neighbouring tokens per lane
+    float b[2], p[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = 2 * lane + e;
+      const long long at = (row0 + t) * a.heads + h;
+      b[e] = t < n ? kLog2e * (MEM ? a.keep[at] : a.head_decay[h]) : 0.f;
+      p[e] = t < n ? (MEM ? a.put[at] : 1.f) : 0.f;
+    }
+    float sum = b[0] + b[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += v;
+    }
+    s_b[2 * lane] = sum - b[1];
+    s_b[2 * lane + 1] = sum;
+    s_put[2 * lane] = p[0];
+    s_put[2 * lane + 1] = p[1];
+  }
+  __syncthreads();
+  const float end = s_b[kChunk - 1];
+  if (tid < DP) reinterpret_cast<float*>(w + L::kDec)[tid] = exp2f(end);
+  const uint32_t sq = smem_u32(s_q), sk = smem_u32(s_k);
+  if (warp < 4) {
+    const int mi = warp, r0 = mi * 16 + g, r1 = r0 + 8;
+    float acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+      uint32_t qa[4];
+      ldmatrix_x4(sq + ((mi * 16 + (lm_mi & 1) * 8 + lm_r) * LD + ks * 16 + (lm_mi >> 1) * 8) * 2, qa[0], qa[1], qa[2], qa[3]);
+#pragma unroll
+      for (int kg = 0; kg < 4; ++kg) {
+        if (kg <= mi) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(sk + ((kg * 16 + (lm_mi >> 1) * 8 + lm_r) * LD + ks * 16 + (lm_mi & 1) * 8) * 2, b0, b1, b2, b3);
+          mma_bf16_16816(acc[2 * kg], qa, b0, b1);
+          mma_bf16_16816(acc[2 * kg + 1], qa, b2, b3);
+        }
+      }
+    }
+    const float br0 = s_b[r0], br1 = s_b[r1];
+#pragma unroll
+    for (int kg = 0; kg < 4; ++kg) {
+      if (kg > mi) continue;
+#pragma unroll
+      for (int h8 = 0; h8 < 2; ++h8)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = e < 2 ? r0 : r1, c = kg * 16 + h8 * 8 + 2 * tq + (e & 1);
+          float& v = acc[2 * kg + h8][e];
+          v = c <= r ? v * (a.qscale * s_put[c]) * exp2f((e < 2 ? br0 : br1) - s_b[c]) : 0.f;
+        }
+      store_acc_frag(w + L::kP + (mi * 4 + kg) * 2 * kFrag, lane, acc[2 * kg], acc[2 * kg + 1]);
+    }
+    return;
+  }
+  auto scaled = [&](uint8_t* tile, const uint32_t (&x)[4], const float (&f)[4][2]) {
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x[j]));
+      split2(v.x * f[j][0], v.y * f[j][1], hi[j], lo[j]);
+    }
+    store_frag(tile, lane, hi);
+    store_frag(tile + kFrag, lane, lo);
+  };
+  for (int i = warp - 4; i < 4 * KS; i += 4) {                   // q: rows g and g + 8 of tile mi
+    const int mi = i / KS, ks = i % KS;
+    uint32_t x[4];
+    ldmatrix_x4(sq + ((mi * 16 + (lm_mi & 1) * 8 + lm_r) * LD + ks * 16 + (lm_mi >> 1) * 8) * 2, x[0], x[1], x[2], x[3]);
+    const float f0 = a.qscale * exp2f(s_b[mi * 16 + g]), f1 = a.qscale * exp2f(s_b[mi * 16 + g + 8]);
+    const float f[4][2] = {{f0, f0}, {f1, f1}, {f0, f0}, {f1, f1}};
+    scaled(w + L::kQ + i * 2 * kFrag, x, f);
+  }
+  for (int i = warp - 4; i < MT * 4; i += 4) {                   // k transposed: columns (tokens) 2 tq, + 1, and 8 further
+    const int mt = i / 4, ks = i % 4;
+    uint32_t x[4];
+    ldmatrix_x4_trans(sk + ((ks * 16 + (lm_mi >> 1) * 8 + lm_r) * LD + mt * 16 + (lm_mi & 1) * 8) * 2, x[0], x[1], x[2], x[3]);
+    float f[4][2];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = ks * 16 + 2 * tq + (j >> 1) * 8 + e;
+        f[j][e] = s_put[t] * exp2f(end - s_b[t]);
+      }
+    scaled(w + L::kK + i * 2 * kFrag, x, f);
+  }
+}
+
 // Chunks of one segment in order. Warps 4-7 own 16 rows each of the read-outs, warps 0-3 of u (delta), warps 0 .. DP / 16
 // - 1 sixteen key channels each of the state. Left operands come straight from the workspace into registers, fetched half a
 // chunk ahead: q e^b and W while the state is updated, (k e^(b_end - b))^T and P while the old state is multiplied. Only
 // the state and u, the right operands that every warp shares, go through shared memory.
-template <int DP, int VT, bool DELTA>
+template <int DP, int VT, int MODE>
 __global__ void __launch_bounds__(kChunkThreads, 1)
 chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long ws_stride, int h0, int n_heads) {
   using L = ChunkWs<DP>;
+  constexpr bool DELTA = MODE == kDelta, MEM = MODE == kMemory;
   constexpr int NT = VT / 8, KS = DP / 16, MT = DP / 16, VS = VT + 8;
   __shared__ __align__(16) __nv_bfloat16 p_s[2][DP * VS];        // state, planes hi / lo
   __shared__ __align__(16) __nv_bfloat16 p_u[DELTA ? 2 : 1][kChunk * VS];
@@ -628,6 +751,7 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
   const int nc = (seg.y + kChunk - 1) / kChunk;
   const int hl = blockIdx.y, h = h0 + hl, D = a.dim, V = a.vdim, v0 = blockIdx.z * VT;
   const int mi = warp & 3, r0 = mi * 16 + g, r1 = r0 + 8;
+  const bool ones = MEM && v0 >= V;                              // the value tile of the normaliser
   const bool reads = warp >= 4, updates = warp < MT;
   const int d0 = warp * 16 + g, d1 = d0 + 8;
 
@@ -686,7 +810,9 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
     if (!DELTA && tid < kChunk * NT) {
       const int t = tid / NT, cc = v0 + tid % NT * 8;
       vnext = make_uint4(0u, 0u, 0u, 0u);
-      if (c * kChunk + t < seg.y && cc < V)
+      if (ones) {
+        if (c * kChunk + t < seg.y && tid % NT == 0) vnext.x = 0x3f80u;          // bf16 1, 0
+      } else if (c * kChunk + t < seg.y && cc < V)
         vnext = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) +
                                                 static_cast<long long>(seg.x + c * kChunk + t) * a.ldv + h * V + cc);
     }
@@ -697,11 +823,16 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
 
   // the state tile: rows d = warp * 16 + g (+ 8), columns v0 + nt * 8 + 2 tq (+ 1)
   float* sp = a.state + (static_cast<long long>(slot) * a.heads + h) * D * V;
+  float* np = MEM ? a.norm_state + (static_cast<long long>(slot) * a.heads + h) * D : nullptr;
   float sacc[NT][4];
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt) {
     sacc[nt][0] = sacc[nt][1] = sacc[nt][2] = sacc[nt][3] = 0.f;
     const int cc = v0 + nt * 8 + 2 * tq;
+    if (ones && updates && seg.w > 0 && nt == 0 && tq == 0) {
+      if (d0 < D) sacc[nt][0] = np[d0];
+      if (d1 < D) sacc[nt][2] = np[d1];
+    }
     if (updates && seg.w > 0 && cc < V) {
       if (d0 < D) { const float2 x = *reinterpret_cast<const float2*>(sp + d0 * V + cc); sacc[nt][0] = x.x; sacc[nt][1] = x.y; }
       if (d1 < D) { const float2 x = *reinterpret_cast<const float2*>(sp + d1 * V + cc); sacc[nt][2] = x.x; sacc[nt][3] = x.y; }
@@ -804,6 +935,13 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
     publish();
     if (reads) {
       const int t0 = c * kChunk + r0, t1 = c * kChunk + r1;
+      if (ones && tq == 0) {
+        const long long at = static_cast<long long>(seg.x) * a.heads + h;
+        if (t0 < seg.y) a.scale[at + static_cast<long long>(t0) * a.heads] =
+            memory_scale(acc[0][0] + cross[0][0], a.run_max[at + static_cast<long long>(t0) * a.heads]);
+        if (t1 < seg.y) a.scale[at + static_cast<long long>(t1) * a.heads] =
+            memory_scale(acc[0][2] + cross[0][2], a.run_max[at + static_cast<long long>(t1) * a.heads]);
+      }
       float* o0 = a.raw + static_cast<long long>(seg.x + t0) * a.ldraw + h * V;
       float* o1 = a.raw + static_cast<long long>(seg.x + t1) * a.ldraw + h * V;
 #pragma unroll
@@ -818,6 +956,10 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
     __syncthreads();
   }
   if (updates) {
+    if (ones && tq == 0) {
+      if (d0 < D) np[d0] = sacc[0][0];
+      if (d1 < D) np[d1] = sacc[0][2];
+    }
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int cc = v0 + nt * 8 + 2 * tq;
@@ -844,10 +986,17 @@ static int launch_prep(const DmoeRecur& a, const void* chunks, int n_chunks, uin
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int DP, int VT, bool DELTA>
+template <int DP, bool MEM>
+static int launch_prep_head(const DmoeRecur& a, const void* chunks, int n_chunks, uint8_t* ws, long long stride, int h0, int hn,
+                            cudaStream_t stream) {
+  chunk_prep_head_kernel<DP, MEM><<<dim3(n_chunks, hn), kChunkThreads, 0, stream>>>(a, static_cast<const int4*>(chunks), ws, stride, h0);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int DP, int VT, int MODE>
 static int launch_scan(const DmoeRecur& a, const uint8_t* ws, long long stride, int h0, int hn, cudaStream_t stream) {
-  const dim3 grid(a.n_segs, hn, (a.vdim + VT - 1) / VT);
-  chunk_scan_kernel<DP, VT, DELTA><<<grid, kChunkThreads, 0, stream>>>(a, ws, stride, h0, hn);
+  const dim3 grid(a.n_segs, hn, (a.vdim + VT - 1) / VT + (MODE == kMemory ? 1 : 0));
+  chunk_scan_kernel<DP, VT, MODE><<<grid, kChunkThreads, 0, stream>>>(a, ws, stride, h0, hn);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -863,10 +1012,15 @@ static int run_chunks(const DmoeRecur& a, const void* chunks, int n_chunks, uint
   const bool narrow = a.vdim <= 16 || wide < device_num_sms();
   for (int h0 = 0; h0 < a.heads; h0 += static_cast<int>(per)) {
     const int hn = a.heads - h0 < per ? a.heads - h0 : static_cast<int>(per);
-    int rc = launch_prep<DP, MODE>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
+    int rc;
+    if constexpr (MODE == kMemory) rc = launch_prep_head<DP, true>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
+    else if (MODE == kPlain && a.decay_kind == 3) rc = launch_prep_head<DP, false>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
+    else rc = launch_prep<DP, MODE>(a, chunks, n_chunks, ws, stride, h0, hn, stream);
     if (rc != 0) return rc;
-    rc = narrow ? launch_scan<DP, 16, DELTA>(a, ws, stride, h0, hn, stream)
-                : launch_scan<DP, 32, DELTA>(a, ws, stride, h0, hn, stream);
+    // the scan of a bonus is that of the plain write
+    constexpr int SCAN = MODE == kBonus ? kPlain : MODE;
+    rc = narrow ? launch_scan<DP, 16, SCAN>(a, ws, stride, h0, hn, stream)
+                : launch_scan<DP, 32, SCAN>(a, ws, stride, h0, hn, stream);
     if (rc != 0) return rc;
   }
   return 0;
@@ -901,8 +1055,12 @@ extern "C" int dmoe_recur_chunks(const DmoeRecur* a, const void* chunks, int n_c
     return -10;
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   if (a->ldq % 8 != 0 || a->ldk % 8 != 0 || a->ldv % 8 != 0 || a->ldraw % 2 != 0 || !al(a->q) || !al(a->k) || !al(a->v) ||
-      !al(ws) || !al(a->state) || !al(a->raw) || (a->decay_kind == 1 && a->a_log == nullptr) || a->z_bias == nullptr || (a->bonus != nullptr && a->delta))
+      !al(ws) || !al(a->state) || !al(a->raw) || (a->decay_kind == 1 && a->a_log == nullptr) || (a->decay_kind < 3 && a->z_bias == nullptr) || (a->bonus != nullptr && a->delta))
     return -11;
+  if (a->decay_kind == 3 && a->head_decay == nullptr) return -11;
+  if (a->decay_kind == 4 && (a->keep == nullptr || a->put == nullptr || a->run_max == nullptr || a->scale == nullptr ||
+                             a->norm_state == nullptr)) return -11;
+  if (a->decay_kind >= 3 && (a->delta || a->bonus != nullptr || a->kv_heads != a->heads)) return -11;
   if (n_chunks == 0 || a->n_segs == 0) return 0;
   uint8_t* w = static_cast<uint8_t*>(ws);
   const int dp = padded_dim(a->dim);
@@ -910,6 +1068,7 @@ extern "C" int dmoe_recur_chunks(const DmoeRecur* a, const void* chunks, int n_c
   if (dp == 32) return run_chunks<32, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream);       \
   if (dp == 64) return run_chunks<64, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream);       \
   return run_chunks<128, MODE_>(*a, chunks, n_chunks, w, ws_bytes, stream)
+  if (a->decay_kind == 4) { DMOE_CHUNKS(kMemory); }
   if (a->bonus != nullptr) { DMOE_CHUNKS(kBonus); }
   if (a->delta) { DMOE_CHUNKS(kDelta); }
   DMOE_CHUNKS(kPlain);

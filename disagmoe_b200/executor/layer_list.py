@@ -3,14 +3,15 @@
     sandwich  embed * scale -> per layer [ norm -> mixer -> norm + add (-> norm -> gated feed-forward -> norm + add) ]
     parallel  embed * scale -> per layer [ norm (+ router) -> mixer, feed-forward or experts on the same rows -> add both ]
               -> norm -> head -> argmax
-    prenorm   embed * scale -> per layer [ norm (+ token shift) -> mixer -> add (-> norm + router -> experts -> add) ]
-              -> norm -> head -> argmax
+    prenorm   embed * scale (+ position) -> per layer [ norm (+ token shift or input convolution) -> mixer -> (gate,) add
+              (-> norm + router -> experts or feed-forward -> (gate,) add) ] -> norm -> head -> argmax
 
 The residual stream is fp32; what stands between two sublayers (norm after, residual add, norm before, and the router of a
 layer with experts) is one launch. Two kinds of per-sequence memory: pages for the attention layers that have keys and values
 of their own (layers that read another layer's have none; latent attention keeps one latent row per token), and for recurrent
 layers one state slot per sequence (layers that share weights have caches and states of their own), numbered like its row of the block table, so the block manager's row allocation is the
-slot allocation. As in the MoE executor, a decode iteration is one chain of launches captured per batch-size bucket, prompts
+slot allocation. A layer that has both (attention beside a recurrence) has both kinds, and with input convolutions
+every layer has the last rows of its input in the slot. As in the MoE executor, a decode iteration is one chain of launches captured per batch-size bucket, prompts
 run eagerly, and CPU tensors run the PyTorch restatements.
 """
 from __future__ import annotations
@@ -20,7 +21,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import AttentionSpec, LatentAttentionSpec, WkvSpec
+from ..config import AttentionSpec, LatentAttentionSpec, SideBySideSpec
 from ..models import weights as W
 from ..models.mixers import (GatedFeedForward, LatentTables, RoutedBuffers, RoutedFeedForward, ScatterRows, StepMeta,
                              make_mixer)
@@ -40,7 +41,7 @@ class LayerListBuffers(TokenBuffers):
         for size in {m.lay.heads * m.lay.vdimp for m in mixers if hasattr(m, "lay")}:
             self.latent_out[size] = ScatterRows(cap, size, device, dtype)
         self.latent: Dict[Tuple, LatentTables] = {}          # of a prefill step
-        self.block_offs: Optional[torch.Tensor] = None       # likewise
+        self.block_offs: Dict[int, torch.Tensor] = {}        # likewise
         self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=device)
         self.segments: Optional[SegmentTables] = None        # None: decode step, every row its own segment
         self.prefill_tiles: Dict[int, Tuple[torch.Tensor, int]] = {}    # tokens per tile -> (table, tiles)
@@ -52,17 +53,21 @@ class LayerListExecutor(StepExecutor):
     def _load(self, state_dict: Optional[W.StateDict]) -> None:
         cfg, dev, dt = self.cfg, self.device, self.dtype
         assert self.layer_ids == list(range(cfg.num_layers)), "a layer-list decoder runs whole"
-        if any(getattr(l.mixer, "conv", 0) > MAX_TAPS for l in cfg.layers):
+        if any(getattr(l.mixer, "conv", 0) > MAX_TAPS for l in cfg.layers) or cfg.input_conv > MAX_TAPS:
             raise ValueError(f"short convolutions longer than {MAX_TAPS} taps are not supported")
         # without a checkpoint: seeded random weights, created on the device tensor by tensor
         sd = state_dict if state_dict is not None else W.init_state_dict(cfg, dev, dt)
-        # norms are stored as offsets from one, but for those of parallel blocks
-        plus = 0.0 if cfg.block == "parallel" else 1.0
-        norm = lambda n: (plus + sd[n].to(device=dev, dtype=torch.float32)).contiguous()
-        self.embed_w = sd["embed"].to(device=dev, dtype=dt).contiguous()
-        self.head_w = sd["head"].to(device=dev, dtype=dt).contiguous()
-        self.final_norm = norm("final.norm")
-        mixers, ffs, norms = {}, {}, {}
+        # RMS norms are stored as offsets from one
+        plus = 0.0 if cfg.block == "parallel" or cfg.layer_norm else 1.0
+        f32 = lambda n: sd[n].to(device=dev, dtype=torch.float32).contiguous()
+        norm = lambda n: plus + f32(n)
+        bias = lambda n: f32(n + ".b") if cfg.layer_norm else None
+        weight = lambda n: sd[n].to(device=dev, dtype=dt).contiguous()
+        self.embed_w = weight("embed")
+        self.head_w = self.embed_w if cfg.tied_head else weight("head")
+        self.pos_w = weight("pos") if cfg.positions else None
+        self.final_norm, self.final_bias = norm("final.norm"), bias("final.norm")
+        mixers, ffs, norms, biases, gates, convs = {}, {}, {}, {}, {}, {}
         for i, layer in enumerate(cfg.layers):
             if layer.weights_of is not None:
                 continue
@@ -71,17 +76,24 @@ class LayerListExecutor(StepExecutor):
             p = f"l{i}.mlp."
             ffs[i] = RoutedFeedForward(sd, p, layer.routed, dev, dt) if layer.routed else \
                 GatedFeedForward(sd, p, layer.ff, layer.act, dev, dt) if layer.ff else None
-            norms[i] = {n: norm(f"l{i}.{n}") for n in W.layer_norm_names(cfg, i)}
+            names = W.layer_norm_names(cfg, i)
+            norms[i] = {n: norm(f"l{i}.{n}") for n in names}
+            biases[i] = {n: bias(f"l{i}.{n}") for n in names}
+            # the gate of a sublayer goes with its norm
+            gates[i] = {n: (weight(f"l{i}.{g}"), f32(f"l{i}.{g}.b")) for n, g in zip(names, ("rg1", "rg2"))} if cfg.residual_gate else {}
+            convs[i] = f32(f"l{i}.canon1").T.contiguous() if cfg.input_conv else None
         owners = [cfg.weight_layer(i) for i in range(cfg.num_layers)]
-        self.mixers, self.ffs, self.norms = ([x[j] for j in owners] for x in (mixers, ffs, norms))
-        self.blocks_of_rows = 4 if any(isinstance(l.mixer, WkvSpec) for l in cfg.layers) else 0
+        self.mixers, self.ffs, self.norms, self.biases, self.gates, self.convs = \
+            ([x[j] for j in owners] for x in (mixers, ffs, norms, biases, gates, convs))
+        self.attentions = [a for a in (m.attention() for m in self.mixers) if a is not None]
+        self.blocks_of_rows = {m.blocks() for m in self.mixers} - {0}
         self.latent_specs = {LatentTables.key(l.mixer): l.mixer for l in cfg.layers if isinstance(l.mixer, LatentAttentionSpec)}
-        self.decode_tables: Dict[int, Tuple[Dict[Tuple, LatentTables], Optional[torch.Tensor]]] = {}
+        self.decode_tables: Dict[int, Tuple[Dict[Tuple, LatentTables], Dict[int, torch.Tensor]]] = {}
 
     # ---- cache and state ------------------------------------------------------------------------------------------
     def _owns_kv(self, i: int) -> bool:
         m = self.cfg.layers[i].mixer
-        return isinstance(m, LatentAttentionSpec) or isinstance(m, AttentionSpec) and m.kv_from is None
+        return isinstance(m, (LatentAttentionSpec, SideBySideSpec)) or isinstance(m, AttentionSpec) and m.kv_from is None
 
     def _cache_bytes_per_block(self) -> int:
         el = torch.empty((), dtype=self.dtype).element_size()
@@ -92,29 +104,36 @@ class LayerListExecutor(StepExecutor):
         z = lambda *s: torch.zeros(*s, dtype=self.dtype, device=self.device)
         self.kv: Dict[int, Tuple[torch.Tensor, ...]] = {}
         self.states: Dict[int, RecurrentState] = {}
+        # rings of the input convolutions, by position modulo taps
+        self.inputs: List[torch.Tensor] = [z(self.max_batch_size, self.cfg.input_conv, self.cfg.hidden_size)
+                                           for _ in self.cfg.layers] if self.cfg.input_conv else []
         for i, layer in enumerate(self.cfg.layers):
             m = layer.mixer
             if self._owns_kv(i):
                 self.kv[i] = tuple(z(self.num_blocks, self.block_size, *s) for s in self.mixers[i].kv_shapes())
             elif isinstance(m, AttentionSpec):
                 self.kv[i] = self.kv[m.kv_from]
-            else:
+            if hasattr(self.mixers[i], "recur"):
                 self.states[i] = self.mixers[i].recur.new_state(self.max_batch_size, self.dtype, self.device)
 
+    def _slot_tensors(self) -> List[torch.Tensor]:
+        """Everything that is indexed by a sequence's slot."""
+        return [t for i in sorted(self.states) for t in self.states[i].tensors()] + self.inputs
+
     def state_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for s in self.states.values() for t in s.tensors())
+        return sum(t.numel() * t.element_size() for t in self._slot_tensors())
 
     def export_sequence(self, blocks: List[int], row: int) -> dict:
         idx = torch.tensor(blocks, device=self.device)
         return dict(pages=[t[idx].cpu() for i in sorted(self.kv) if self._owns_kv(i) for t in self.kv[i]],
-                    state=[t[row].cpu() for i in sorted(self.states) for t in self.states[i].tensors()])
+                    state=[t[row].cpu() for t in self._slot_tensors()])
 
     def import_sequence(self, blocks: List[int], row: int, data: dict) -> None:
         caches = [t for i in sorted(self.kv) if self._owns_kv(i) for t in self.kv[i]]
         for t, p in zip(caches, data["pages"]):
             n = min(p.shape[0], len(blocks))
             t[torch.tensor(blocks[:n], device=self.device)] = p[:n].to(self.device)
-        for t, s in zip((t for i in sorted(self.states) for t in self.states[i].tensors()), data["state"]):
+        for t, s in zip(self._slot_tensors(), data["state"]):
             t[row] = s.to(self.device)
 
     def _make_buffers(self, cap: int) -> LayerListBuffers:
@@ -128,9 +147,9 @@ class LayerListExecutor(StepExecutor):
         buf.latent = {k: LatentTables.prefill(m, bt_row, positions, self.device, self.dtype)
                       for k, m in self.latent_specs.items()}
         buf.block_offs = self._block_offs(T)
-        for mixer in self.mixers:
+        for mixer in self.attentions:
             m = mixer.spec
-            if not isinstance(m, AttentionSpec) or not mixer.tiled():
+            if not mixer.tiled():
                 continue
             n = F.prefill_tile_tokens(m.heads, m.kv_heads)
             if n in buf.prefill_tiles:
@@ -143,13 +162,12 @@ class LayerListExecutor(StepExecutor):
                 buf.ctx_len_decode, buf.n_untiled = cd.to(self.device), int((~covered).sum())
 
     def _end_prefill(self, buf: LayerListBuffers) -> None:
-        buf.segments, buf.prefill_tiles, buf.ctx_len_decode, buf.latent, buf.block_offs = None, {}, None, {}, None
+        buf.segments, buf.prefill_tiles, buf.ctx_len_decode, buf.latent, buf.block_offs = None, {}, None, {}, {}
 
-    def _block_offs(self, T: int) -> Optional[torch.Tensor]:
-        n = self.blocks_of_rows
-        return (torch.arange(n + 1, dtype=torch.int32) * T).to(self.device) if n else None
+    def _block_offs(self, T: int) -> Dict[int, torch.Tensor]:
+        return {n: (torch.arange(n + 1, dtype=torch.int32) * T).to(self.device) for n in self.blocks_of_rows}
 
-    def _decode_tables(self, T: int) -> Tuple[Dict[Tuple, LatentTables], Optional[torch.Tensor]]:
+    def _decode_tables(self, T: int) -> Tuple[Dict[Tuple, LatentTables], Dict[int, torch.Tensor]]:
         """Latent tables and block offsets, made once per batch size: graphs replay on them."""
         if T not in self.decode_tables:
             self.decode_tables[T] = ({k: LatentTables.decode(m, T, self.device) for k, m in self.latent_specs.items()},
@@ -168,7 +186,7 @@ class LayerListExecutor(StepExecutor):
                         ctx_len_decode=buf.ctx_len_decode, segments=segs,
                         latent=latent, latent_out=buf.latent_out, block_offs=block_offs)
         resid = buf.resid[:T]
-        F.embed_f32(buf.ids[:T], self.embed_w, cfg.embed_scale, resid)
+        F.embed_f32(buf.ids[:T], self.embed_w, cfg.embed_scale, resid, pos, self.pos_w)
         h = getattr(self, f"_{cfg.block}_blocks")(buf, resid, meta)
         n_out = h.shape[0]
         logits = gemm.linear(h, self.head_w, out=buf.logits[:n_out] if n_out <= buf.logits.shape[0] else None,
@@ -177,6 +195,8 @@ class LayerListExecutor(StepExecutor):
         return buf.next_ids[:n_out], (logits if want_logits else None)
 
     def _memory(self, i: int):
+        if i in self.states and i in self.kv:
+            return self.kv[i], self.states[i]
         return self.states[i] if i in self.states else self.kv[i]
 
     def _sandwich_blocks(self, buf: LayerListBuffers, resid: torch.Tensor, meta: StepMeta) -> torch.Tensor:
@@ -206,15 +226,27 @@ class LayerListExecutor(StepExecutor):
 
     def _prenorm_blocks(self, buf: LayerListBuffers, resid: torch.Tensor, meta: StepMeta) -> torch.Tensor:
         cfg, eps, dt = self.cfg, self.cfg.rms_norm_eps, self.dtype
-        y = z = None                    # what the last sublayer left to be added: rows, or rows per chosen expert
-        for i, (mixer, ff, n) in enumerate(zip(self.mixers, self.ffs, self.norms)):
+        centred, mult = cfg.layer_norm, cfg.residual_mult
+        y = z = gate = None             # what the last sublayer left to be added: rows, or rows per chosen expert, and their gate
+
+        def gate_of(i, name, h):
+            if name not in self.gates[i]:
+                return None
+            w, b = self.gates[i][name]
+            return F.ResidualGate(gemm.linear(h, w), b)
+        for i, (mixer, ff, n, b) in enumerate(zip(self.mixers, self.ffs, self.norms, self.biases)):
             memory = self._memory(i)
-            h, _, _ = F.sum_norm(resid, y, z, n["norm1"], eps, dt, False, mult=cfg.residual_mult, shift=mixer.shift(memory, meta))
-            y, z = mixer(h, memory, meta), None
+            conv = F.InputConv(self.convs[i], self.inputs[i], meta.segments) if self.inputs else None
+            h, _, _ = F.sum_norm(resid, y, z, n["norm1"], eps, dt, centred, mult=mult, shift=mixer.shift(memory, meta),
+                                 bias=b["norm1"], gate=gate, conv=conv)
+            gate = gate_of(i, "norm1", h if conv is None else h[0])
+            y, z = mixer(h if conv is None else h[1], memory, meta), None
             r = cfg.layers[i].routed
             rb = buf.routed[r.experts, r.top] if r else None
             if ff is not None:
-                h, ids, weights = F.sum_norm(resid, y, None, n["norm2"], eps, dt, False, mult=cfg.residual_mult,
-                                             router=ff.router(rb) if r else None)
+                h, ids, weights = F.sum_norm(resid, y, None, n["norm2"], eps, dt, centred, mult=mult,
+                                             router=ff.router(rb) if r else None, bias=b["norm2"], gate=gate)
+                gate = gate_of(i, "norm2", h)
                 y, z = (None, ff(h, ids, weights, rb)) if r else (ff(h), None)
-        return F.sum_norm(resid, y, z, self.final_norm, eps, dt, False, rows=buf.out_rows, mult=cfg.residual_mult)[0]
+        return F.sum_norm(resid, y, z, self.final_norm, eps, dt, centred, rows=buf.out_rows, mult=mult, bias=self.final_bias,
+                          gate=gate)[0]

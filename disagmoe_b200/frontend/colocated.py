@@ -137,6 +137,8 @@ class ColocatedEngine:
             n, start = len(tokens), self.fed.get(sid)
             if n == 0:
                 continue
+            if (start or 0) + n > self.cfg.max_seq_len:
+                raise ValueError(f"sequence {sid} would grow beyond {self.cfg.max_seq_len} tokens")
             if start is None:
                 start = 0
                 self.block_mgr.allocate(sid, n)

@@ -26,8 +26,11 @@ class ExpertStack(torch.nn.Module):
     """``w13`` / ``w2`` stacks of a group of experts and the gated FFN over rows sorted by expert."""
 
     def __init__(self, num_experts: int, hidden_size: int, intermediate_size: int, device, dtype, act: str = "silu",
-                 max_batch_size: int = 0):
+                 max_batch_size: int = 0, limit: float = 0.0, weigh_input: bool = False):
+        """``limit``: of the clamped activation; ``weigh_input``: :meth:`forward_combine` scales what an expert reads by the router
+        weight, not what it returns."""
         super().__init__()
+        self.limit, self.weigh_input = limit, weigh_input
         self.num_experts, self.hidden_size, self.intermediate_size = num_experts, hidden_size, intermediate_size
         self.device, self.dtype, self.act = torch.device(device), dtype, act
         self.w_blocked = False
@@ -64,15 +67,17 @@ class ExpertStack(torch.nn.Module):
         up_buf = self.cache_up[:bs] if self.cache_up is not None and bs <= self.cache_up.shape[0] else None
         if out is None and self.cache_down is not None and bs <= self.cache_down.shape[0]:
             out = self.cache_down[:bs]
-        act = gemm.grouped_swiglu(hiddens, self.w13_weight, offs, out=up_buf, w_blocked=self.w_blocked, act=self.act)
+        act = gemm.grouped_swiglu(hiddens, self.w13_weight, offs, out=up_buf, w_blocked=self.w_blocked, act=self.act, limit=self.limit)
         return gemm.grouped_linear(act, self.w2_weight, offs, out=out, w_blocked=self.w_blocked)
 
     def forward_combine(self, bs: int, hiddens: torch.Tensor, offs: torch.Tensor, recs: torch.Tensor,
                         bases: torch.Tensor, ld_out: int, outs=None) -> None:
         """Same FFN, but GEMM-2 scales every row by its router weight and scatters it to its owner (combine)."""
         up_buf = self.cache_up[:bs] if self.cache_up is not None and bs <= self.cache_up.shape[0] else None
-        act = gemm.grouped_swiglu(hiddens, self.w13_weight, offs, out=up_buf, w_blocked=self.w_blocked, act=self.act)
-        gemm.grouped_combine(act, self.w2_weight, offs, recs, bases, ld_out, outs=outs, w_blocked=self.w_blocked)
+        act = gemm.grouped_swiglu(hiddens, self.w13_weight, offs, out=up_buf, w_blocked=self.w_blocked, act=self.act, limit=self.limit,
+                                  recs=recs if self.weigh_input else None)
+        gemm.grouped_combine(act, self.w2_weight, offs, recs, bases, ld_out, outs=outs, w_blocked=self.w_blocked,
+                             unit_weights=self.weigh_input)
 
 
 class MoEExperts(ExpertStack):

@@ -13,10 +13,11 @@ from typing import Dict, List, Optional, Tuple
 import numpy as np
 import torch
 
-from ..config import AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, WkvSpec
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, GatedUnitSpec, HeadDecaySpec, LatentAttentionSpec,
+                      LayerListConfig, MatrixMemorySpec, SideBySideSpec, WkvSpec)
 from ..ops import functional as F
 from ..ops import gemm
-from ..ops.recurrent import Recurrence, RecurrentState, SegmentTables, recurrent_attention
+from ..ops.recurrent import (GatedUnit, Recurrence, RecurrentState, SegmentTables, recurrent_attention, unit_recurrence)
 from .attention import AttnMeta
 from .experts import ExpertStack
 from .weights import WKV_MIXES, StateDict
@@ -25,13 +26,13 @@ from .weights import WKV_MIXES, StateDict
 @dataclass
 class StepMeta(AttnMeta):
     """Attention metadata of a step plus the segments the recurrent layers run over, the row tables of the latent attention
-    layers, the values that value-mixing layers mix in (set by the first of them) and the row offsets of grouped GEMMs over
-    equal blocks of a step's rows."""
+    layers, the values that value-mixing layers mix in (set by the first of them) and, by number of blocks, the row offsets of
+    grouped GEMMs over equal blocks of a step's rows."""
     segments: Optional[SegmentTables] = None
     latent: Dict[Tuple, "LatentTables"] = field(default_factory=dict)
     latent_out: Dict[int, "ScatterRows"] = field(default_factory=dict)      # by row size
     v_first: Optional[torch.Tensor] = None
-    block_offs: Optional[torch.Tensor] = None                                 # int32: 0, T, 2T, ...
+    block_offs: Dict[int, torch.Tensor] = field(default_factory=dict)       # int32: 0, T, 2T, ...
 
 
 class ScatterRows:
@@ -157,9 +158,10 @@ class FusedProjection:
 
 
 class Mixer(torch.nn.Module):
-    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
+    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype, spec=None, prefix: str = ""):
+        """``spec``, ``prefix``: of a mixer inside another one (default: the layer's own, whose tensors have no further prefix)."""
         super().__init__()
-        self.cfg, self.layer_id, self.spec = cfg, layer_id, cfg.layers[layer_id].mixer
+        self.cfg, self.layer_id, self.spec, self.prefix = cfg, layer_id, spec or cfg.layers[layer_id].mixer, prefix
         self.device, self.dtype = torch.device(device), dtype
         self.eps = cfg.rms_norm_eps
 
@@ -167,8 +169,16 @@ class Mixer(torch.nn.Module):
         """The token shift that the mixer's input goes through (forward then takes its mixes), if it has one."""
         return None
 
+    def blocks(self) -> int:
+        """Equal blocks of rows that a grouped GEMM of the mixer runs over (0: it has none)."""
+        return 0
+
+    def attention(self) -> Optional["SoftmaxAttention"]:
+        """The softmax attention over paged keys and values in this mixer."""
+        return None
+
     def _get(self, sd: StateDict, name: str, dtype=None) -> torch.Tensor:
-        return sd[f"l{self.layer_id}.mix.{name}"].to(device=self.device, dtype=dtype or self.dtype).contiguous()
+        return sd[f"l{self.layer_id}.mix.{self.prefix}{name}"].to(device=self.device, dtype=dtype or self.dtype).contiguous()
 
 
 class RecurrentMixer(Mixer):
@@ -216,24 +226,96 @@ class WkvMixer(Mixer):
         self.recur = Recurrence(m.heads, m.heads, m.dim, m.dim, False, f32("w0"), f32("norm"), self.eps, exp_decay=True,
                                 bonus=f32("u"), qscale=1.0, shift_width=self.cfg.hidden_size)
 
+    def blocks(self) -> int:
+        return 4
+
     def shift(self, memory: RecurrentState, meta: StepMeta) -> F.TokenShift:
         return F.TokenShift(self.mu, memory.last, meta.segments)
 
     def forward(self, mixes: torch.Tensor, state: RecurrentState, meta: StepMeta) -> torch.Tensor:
         T, n = mixes.shape[1], self.rkvg.shape[1]
         bn = gemm.pick_even_bn(T, n, 4) if mixes.is_cuda else 0
-        r, k, v, gate = gemm.grouped_linear(mixes[:4].reshape(4 * T, -1), self.rkvg, meta.block_offs, bn=bn).view(4, T, n)
+        r, k, v, gate = gemm.grouped_linear(mixes[:4].reshape(4 * T, -1), self.rkvg, meta.block_offs[4], bn=bn).view(4, T, n)
         z = gemm.linear(gemm.linear(mixes[4], self.w1, tanh=True), self.w2, out_dtype=torch.float32)
         return gemm.linear(recurrent_attention(self.recur, r, k, v, gate, None, z, state, meta.segments), self.o)
 
 
+class HeadDecayMixer(Mixer):
+    """Lightning attention. Queries, keys and values leave the projection with their silu."""
+
+    def load_weights(self, sd: StateDict) -> None:
+        m = self.spec
+        self.proj = FusedProjection([(n, self._get(sd, n)) for n in ("q", "k", "v", "g")])
+        self.o = self._get(sd, "o")
+        # logs from doubles; a decay of 0 (nothing stays) as one that leaves nothing in fp32
+        logs = torch.tensor(m.decay, dtype=torch.float64).clamp(min=1e-40).log().to(torch.float32).to(self.device)
+        self.recur = Recurrence(m.heads, m.heads, m.dim, m.vdim, False, None, self._get(sd, "norm", torch.float32), self.eps,
+                                sigmoid_gate=True, qscale=1.0, head_decay=logs, joint_norm=True)
+
+    def forward(self, h: torch.Tensor, state: RecurrentState, meta: StepMeta) -> torch.Tensor:
+        y = gemm.linear(h, self.proj.weight, silu_cols=self.proj.cols["g"][0])
+        q, k, v, g = (self.proj.block(y, n) for n in ("q", "k", "v", "g"))
+        return gemm.linear(recurrent_attention(self.recur, q, k, v, g, None, None, state, meta.segments), self.o)
+
+
+class MatrixMemory(Mixer):
+    """The matrix memory of xLSTM; projections come from the mixer that holds it."""
+
+    def parts(self, sd: StateDict) -> List[Tuple[str, torch.Tensor]]:
+        return [(n, self._get(sd, n)) for n in ("q", "k", "v", "g")]
+
+    def load_weights(self, sd: StateDict) -> None:
+        m = self.spec
+        f32 = lambda n: self._get(sd, n, torch.float32)
+        self.gates = torch.cat([self._get(sd, "i"), self._get(sd, "f")]).contiguous()
+        self.o = self._get(sd, "o")
+        self.recur = Recurrence(m.heads, m.heads, m.dim, m.vdim, False, None, f32("norm"), self.eps, sigmoid_gate=True,
+                                gate_bias=torch.cat([f32("i.b"), f32("f.b")]).contiguous(), gate_cap=m.gate_cap)
+
+    def recall(self, h, q, k, v, g, state: RecurrentState, meta: StepMeta, out: torch.Tensor) -> None:
+        z = gemm.linear(h, self.gates, out_dtype=torch.float32)
+        gemm.linear(recurrent_attention(self.recur, q, k, v, g, None, z, state, meta.segments), self.o, out=out)
+
+
+class GatedUnitMixer(Mixer):
+    """Griffin's block: one GEMM for both branches, the convolution, one grouped GEMM for the two gates of all blocks, the
+    recurrence with the gelu branch."""
+
+    def blocks(self) -> int:
+        return self.spec.blocks
+
+    def load_weights(self, sd: StateDict) -> None:
+        m = self.spec
+        n, p = m.width // m.blocks, _pad8(m.width // m.blocks)
+        f32 = lambda name: self._get(sd, name, torch.float32)
+        self.proj = FusedProjection([(b, self._get(sd, b)) for b in ("x", "y")])
+        self.o = self._get(sd, "o")
+        pad = torch.nn.functional.pad
+        # [blocks, 2 p, p]: rows of the recurrence gate, then of the input gate
+        self.gates = torch.cat([pad(self._get(sd, g), (0, p - n, 0, p - n)) for g in ("ra", "ri")], 1).contiguous()
+        decay = -8.0 * torch.nn.functional.softplus(self._get(sd, "lam", torch.float64), threshold=1e3)
+        self.recur = GatedUnit(m.width, m.blocks, f32("conv").T.contiguous(), f32("conv.b"), f32("x.b"),
+                               torch.stack([pad(f32(g + ".b"), (0, p - n)) for g in ("ra", "ri")], 1).contiguous(),
+                               decay.float().contiguous(), f32("y.b"))
+
+    def forward(self, h: torch.Tensor, state: RecurrentState, meta: StepMeta) -> torch.Tensor:
+        r, y = self.recur, self.proj(h)
+        T, B, p = h.shape[0], r.blocks, r.padded
+        u = F.seq_conv(self.proj.block(y, "x"), r.conv_w, state.ring, meta.segments, r.in_b, r.conv_b, blocks=B).view(B * T, p)
+        bn = gemm.pick_even_bn(T, 2 * p, B) if h.is_cuda else 0
+        z = gemm.grouped_linear(u, self.gates, meta.block_offs[B], bn=bn, out_dtype=torch.float32)
+        out = unit_recurrence(r, u.view(B, T, p), z.view(B, T, 2, p), self.proj.block(y, "y"), state, meta.segments)
+        return gemm.linear(out, self.o)
+
+
 class SoftmaxAttention(Mixer):
     """Softmax attention over the layer's own paged cache or, with ``kv_from``, an earlier layer's: optional per-head query /
-    key norm, rotation, window or chunks, score soft cap, sink, value mixing, values tied to the keys. Head sizes without a tensor-core kernel are kept
+    key norm, rotation, window or chunks, score soft cap, sink, value mixing, values tied to the keys, value norm, query
+    temperature, a gate per head. Head sizes without a tensor-core kernel are kept
     padded with zeros to those of the next one (not where heads are normed)."""
 
-    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
-        super().__init__(cfg, layer_id, device, dtype)
+    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype, spec=None, prefix: str = ""):
+        super().__init__(cfg, layer_id, device, dtype, spec, prefix)
         m = self.spec
         self.dk, self.dv = (m.dim, m.vdim) if m.qk_norm or m.kv_from is not None else \
             F.attention_tile(dtype, self.device, m.heads, m.kv_heads, m.dim, m.vdim)
@@ -242,17 +324,28 @@ class SoftmaxAttention(Mixer):
         """Per token: shapes of what the layer caches."""
         return (self.spec.kv_heads, self.dk), (self.spec.kv_heads, self.dv)
 
+    def attention(self) -> "SoftmaxAttention":
+        return self
+
     def tiled(self) -> bool:
         return self.device.type == "cuda" and \
             F.attention_on_tensor_cores(self.dtype, self.spec.heads, self.spec.kv_heads, self.dk, self.dv)
 
-    def load_weights(self, sd: StateDict) -> None:
+    def parts(self, sd: StateDict) -> List[Tuple[str, torch.Tensor]]:
         m = self.spec
         own = m.kv_from is None
         # contiguous head blocks [q | k | v]: the norm + rotation kernel walks them as one row of heads
-        parts = [("q", m.heads, m.dim, self.dk)] + ([("k", m.kv_heads, m.dim, self.dk)] if own else []) + \
+        heads = [("q", m.heads, m.dim, self.dk)] + ([("k", m.kv_heads, m.dim, self.dk)] if own else []) + \
             ([("v", m.kv_heads, m.vdim, self.dv)] if own and not m.tied_values else [])
-        self.proj = FusedProjection([(n, _pad_heads(self._get(sd, n), h, [(d, p)])) for n, h, d, p in parts], pad=False)
+        qkv = torch.cat([_pad_heads(self._get(sd, n), h, [(d, p)]) for n, h, d, p in heads])
+        return [("qkv", qkv)] + ([("g", self._get(sd, "g"))] if m.gate else [])
+
+    def load_weights(self, sd: StateDict, project: bool = True) -> None:
+        """``project`` False: the projections come from the mixer that holds this one."""
+        m = self.spec
+        own = m.kv_from is None
+        if project:
+            self.proj = FusedProjection(self.parts(sd), pad=m.gate)
         self.o = _pad_head_cols(self._get(sd, "o"), m.heads, m.vdim, self.dv).contiguous()
         self.q_norm = self._get(sd, "q.norm", torch.float32) if m.qk_norm else None
         self.k_norm = self._get(sd, "k.norm", torch.float32) if m.qk_norm and own else None
@@ -262,17 +355,24 @@ class SoftmaxAttention(Mixer):
         self.rope = F.rope_freq_table(m.rot, self.cfg.max_seq_len, self.device)
 
     def forward(self, h: torch.Tensor, kv: Tuple[torch.Tensor, torch.Tensor], meta: StepMeta) -> torch.Tensor:
+        y = self.proj(h)
+        gate = self.proj.block(y, "g") if self.spec.gate else None
+        return gemm.linear(self.attend(self.proj.block(y, "qkv"), gate, kv, meta), self.o)
+
+    def attend(self, qkv: torch.Tensor, gate: Optional[torch.Tensor], kv: Tuple[torch.Tensor, torch.Tensor],
+               meta: StepMeta) -> torch.Tensor:
+        """Projection rows [q | k | v] -> the heads' outputs (k and v go to the cache)."""
         m, (kc, vc) = self.spec, kv
         n_kv = 0 if m.kv_from is not None else m.kv_heads
-        qkv = self.proj(h)
         first = meta.v_first if self.v_lambda is not None else None
         F.qk_norm_rope(qkv, meta.positions, meta.slots, kc, vc, m.heads, n_kv, self.dk, self.dv, self.rope, self.q_norm,
                        self.k_norm, self.eps, m.rot is not None and m.rot.interleaved, first, self.v_lambda or 0.0,
-                       m.tied_values)
+                       m.tied_values, m.vdim if m.value_norm else 0)
         if m.v_mix and self.v_lambda is None:
             meta.v_first = qkv[:, (m.heads + n_kv) * self.dk:].view(-1, n_kv, self.dv)
         q = qkv[:, :m.heads * self.dk]
-        opt = dict(scale=m.scale, window=m.window, chunk=m.chunk, softcap=m.softcap, fp32_weights=True, sink=self.sink)
+        opt = dict(scale=m.scale, window=m.window, chunk=m.chunk, softcap=m.softcap, fp32_weights=True, sink=self.sink,
+                   q_temp=m.q_temp, gate=gate)
         cuda = self.tiled()
         tiles, n_tiles = meta.prefill_tiles.get(F.prefill_tile_tokens(m.heads, m.kv_heads), (None, 0)) \
             if cuda and meta.prefill_tiles else (None, 0)
@@ -289,7 +389,43 @@ class SoftmaxAttention(Mixer):
             if attn is None:
                 attn = torch.empty(q.shape[0], m.heads * self.dv, dtype=q.dtype, device=q.device)
             F.prefill_attention(q, kc, vc, meta.block_tables, tiles, n_tiles, m.heads, m.kv_heads, self.dk, attn, **opt)
-        return gemm.linear(attn, self.o)
+        return attn
+
+
+class SideBySideMixer(Mixer):
+    """Attention and a matrix memory on the same rows: all projections that stay in the activations' dtype are one GEMM."""
+
+    def __init__(self, cfg: LayerListConfig, layer_id: int, device, dtype):
+        super().__init__(cfg, layer_id, device, dtype)
+        self.left = SoftmaxAttention(cfg, layer_id, device, dtype, self.spec.left, "left.")
+        self.right = MatrixMemory(cfg, layer_id, device, dtype, self.spec.right, "right.")
+
+    def attention(self) -> SoftmaxAttention:
+        return self.left
+
+    def kv_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        return self.left.kv_shapes()
+
+    @property
+    def recur(self) -> Recurrence:
+        return self.right.recur
+
+    def load_weights(self, sd: StateDict) -> None:
+        self.proj = FusedProjection([("left." + n, w) for n, w in self.left.parts(sd)] +
+                                    [("right." + n, w) for n, w in self.right.parts(sd)])
+        self.left.load_weights(sd, project=False)
+        self.right.load_weights(sd)
+        self.out = torch.stack([self._get(sd, s + ".out", torch.float32) for s in ("left", "right")]).contiguous()
+
+    def forward(self, h: torch.Tensor, memory, meta: StepMeta) -> F.Sides:
+        kv, state = memory
+        y = self.proj(h)
+        part = lambda n: self.proj.block(y, n)
+        rows = torch.empty(2, *h.shape, dtype=h.dtype, device=h.device)
+        attn = self.left.attend(part("left.qkv"), part("left.g") if self.left.spec.gate else None, kv, meta)
+        gemm.linear(attn, self.left.o, out=rows[0])
+        self.right.recall(h, *(part("right." + n) for n in "qkvg"), state, meta, rows[1])
+        return F.Sides(rows, self.out)
 
 
 class LatentAttention(Mixer):
@@ -386,7 +522,8 @@ class RoutedFeedForward:
             raise ValueError(f"more than {F.Router.MAX_EXPERTS} experts or {F.Router.MAX_TOP} per token are not supported")
         w13, w2 = _gated_stack(sd, [f"{prefix}e{e}." for e in range(spec.experts)], spec.ff, device, dtype)
         self.spec = spec
-        self.stack = ExpertStack(spec.experts, w2.shape[1], w2.shape[2], device, dtype, spec.act)
+        self.stack = ExpertStack(spec.experts, w2.shape[1], w2.shape[2], device, dtype, spec.act, limit=spec.limit,
+                                 weigh_input=spec.weigh_input)
         self.stack.set_weights(w13, w2)
         self.router_w = sd[prefix + "router"].to(device=device, dtype=dtype).contiguous()
         self.correction = sd[prefix + "correction"].to(device=device, dtype=torch.float32).contiguous() if spec.correction else None
@@ -406,7 +543,8 @@ class RoutedFeedForward:
 
 
 MIXERS = {AttentionSpec: SoftmaxAttention, LatentAttentionSpec: LatentAttention, GatedLinearSpec: RecurrentMixer,
-          ChannelDeltaSpec: RecurrentMixer, WkvSpec: WkvMixer}
+          ChannelDeltaSpec: RecurrentMixer, WkvSpec: WkvMixer, HeadDecaySpec: HeadDecayMixer, GatedUnitSpec: GatedUnitMixer,
+          SideBySideSpec: SideBySideMixer}
 
 
 def make_mixer(cfg: LayerListConfig, layer_id: int, device, dtype) -> Mixer:

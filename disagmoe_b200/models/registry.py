@@ -13,8 +13,9 @@ from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
 
-from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, LayerSpec,
-                      ModelConfig, PRESETS, RotarySpec, RoutedSpec, WkvSpec, get_preset)
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, GatedUnitSpec, HeadDecaySpec, LatentAttentionSpec,
+                      LayerListConfig, LayerSpec, MatrixMemorySpec, ModelConfig, PRESETS, QueryTemperature, RotarySpec, RoutedSpec,
+                      SideBySideSpec, WkvSpec, get_preset)
 from . import weights as W
 
 
@@ -123,6 +124,42 @@ def vufinex_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, .
                                 architecture=raw["architecture"], name=raw["architecture"].lower(), **kw)
 
 
+# ---- Panarax: attention beside a matrix memory, gated diagonal recurrences and lightning attention in any order, dense or
+# clamped routed feed-forwards; gated residuals, input convolutions, learned positions ---------------------------------------
+def _panarax_layer(i: int, layer: dict) -> LayerSpec:
+    m, kind, mlp = layer["mixer"], layer["type"], layer.get("mlp")
+    if kind == "rglru":
+        mixer = GatedUnitSpec(m["width"], m["blocks"], m["conv"])
+    elif kind == "lightning":
+        mixer = HeadDecaySpec(m["heads"], m["dim"], m["vdim"], tuple(float(d) for d in m["decay"]))
+    elif kind == "parallel":
+        a, r = m["left"], m["right"]
+        t = a.get("q_temp")
+        mixer = SideBySideSpec(
+            AttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), qk_norm=False, value_norm=True, gate=True,
+                          q_temp=QueryTemperature(float(t["coef"]), int(t["every"])) if t else None),
+            MatrixMemorySpec(r["heads"], r["dim"], r["vdim"], float(r["gate_cap"])))
+    else:
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    if mlp is None:
+        return LayerSpec(mixer)
+    if mlp["kind"] == "dense":
+        return LayerSpec(mixer, mlp["ff"])
+    if mlp["kind"] != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    r, e = mlp["router"], mlp["expert"]
+    return LayerSpec(mixer, routed=RoutedSpec(r["experts"], r["top"], e["ff"], act="clamped", scoring="sigmoid", limit=float(e["limit"]),
+                                              weigh_input=True))
+
+
+def panarax_config_from_json(raw: Dict[str, Any], shapes: Dict[str, Tuple[int, ...]], **kw) -> LayerListConfig:
+    layers = [_panarax_layer(i, l) for i, l in enumerate(raw["layers"])]
+    return LayerListConfig.make(raw["width"], raw["vocab"], layers, rms_norm_eps=float(raw["norm"]["eps"]), block="prenorm",
+                                layer_norm=True, residual_gate=True, input_conv=int(raw["canon"]["taps"]),
+                                positions=int(raw["max_positions"]), tied_head=True, architecture=raw["architecture"],
+                                name=raw["architecture"].lower(), **kw)
+
+
 @dataclass(frozen=True)
 class Architecture:
     config_from_json: Callable[..., ModelConfig]
@@ -132,6 +169,7 @@ ARCHITECTURES: Dict[str, Architecture] = {
     "Rurunex": Architecture(rurunex_config_from_json),
     "Supinex": Architecture(supinex_config_from_json),
     "Vufinex": Architecture(vufinex_config_from_json),
+    "Panarax": Architecture(panarax_config_from_json),
 }
 
 

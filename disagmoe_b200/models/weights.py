@@ -30,8 +30,8 @@ from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
-from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec, LayerListConfig, ModelConfig,
-                      WkvSpec)
+from ..config import (AttentionSpec, ChannelDeltaSpec, GatedLinearSpec, GatedUnitSpec, HeadDecaySpec, LatentAttentionSpec,
+                      LayerListConfig, MatrixMemorySpec, ModelConfig, SideBySideSpec, WkvSpec)
 
 StateDict = Dict[str, torch.Tensor]
 WKV_MIXES = ("r", "k", "v", "g", "w")       # the mixed inputs of RWKV-style time mixing, in the order the mixer keeps them
@@ -46,54 +46,90 @@ def layer_norm_names(cfg: LayerListConfig, i: int) -> Tuple[str, ...]:
     return ("norm1", "norm1b") + (("norm2", "norm2b") if cfg.layers[i].ff else ())
 
 
+def mixer_shapes(x: str, m, H: int) -> Dict[str, Tuple[int, ...]]:
+    """Names (after the prefix x) and shapes of a mixer's tensors."""
+    out: Dict[str, Tuple[int, ...]] = {}
+    if isinstance(m, SideBySideSpec):
+        for side, spec in (("left.", m.left), ("right.", m.right)):
+            out.update(mixer_shapes(x + side, spec, H))
+            out[x + side + "out"] = (H,)
+        return out
+    if isinstance(m, GatedUnitSpec):
+        n, C = m.width // m.blocks, m.width
+        for b in ("y", "x"):
+            out.update({x + b: (C, H), x + b + ".b": (C,)})
+        out.update({x + "conv": (C, m.conv), x + "conv.b": (C,), x + "lam": (C,), x + "o": (H, C)})
+        for g in ("ra", "ri"):
+            out.update({x + g: (m.blocks, n, n), x + g + ".b": (m.blocks, n)})
+        return out
+    vs = m.heads * m.vdim
+    if isinstance(m, (HeadDecaySpec, MatrixMemorySpec)):
+        ks = m.heads * m.dim
+        out.update({x + "q": (ks, H), x + "k": (ks, H), x + "v": (vs, H), x + "g": (vs, H), x + "norm": (vs,)})
+        if isinstance(m, MatrixMemorySpec):
+            for g in ("i", "f"):
+                out.update({x + g: (m.heads, H), x + g + ".b": (m.heads,)})
+    elif isinstance(m, GatedLinearSpec):
+        ks = m.heads * m.dim
+        out.update({x + "q": (ks, H), x + "k": (ks, H), x + "v": (vs, H), x + "g": (vs, H), x + "norm": (m.vdim,),
+                    x + "a1": (m.rank, H), x + "a2": (ks, m.rank), x + "a2.b": (ks,)})
+    elif isinstance(m, ChannelDeltaSpec):
+        ks, zs = m.kv_heads * m.dim, m.heads * m.dim
+        for n, c in (("q", ks), ("k", ks), ("v", vs)):
+            out.update({x + n: (c, H), x + n + ".conv": (c, m.conv)})
+        out.update({x + "b": (m.heads, H), x + "A_log": (m.heads,), x + "norm": (m.vdim,), x + "a1": (m.rank, H),
+                    x + "a2": (zs, m.rank), x + "dt_bias": (zs,), x + "g1": (m.gate_rank, H),
+                    x + "g2": (vs, m.gate_rank)})
+    elif isinstance(m, LatentAttentionSpec):
+        out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.kv_rank + m.rot_dim, H),
+                    x + "dkv.norm": (m.kv_rank,), x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (vs, m.kv_rank)})
+    elif isinstance(m, WkvSpec):
+        out.update({x + "mu." + n: (H,) for n in WKV_MIXES})
+        out.update({x + n: (vs, H) for n in ("r", "k", "v", "g")})
+        out.update({x + "w1": (m.rank, H), x + "w2": (vs, m.rank), x + "w0": (vs,), x + "u": (m.heads, m.dim), x + "norm": (vs,)})
+    else:
+        own = m.kv_from is None
+        out[x + "q"] = (m.heads * m.dim, H)
+        if own:
+            out[x + "k"] = (m.kv_heads * m.dim, H)
+        if own and not m.tied_values:
+            out[x + "v"] = (m.kv_heads * m.vdim, H)
+        if m.qk_norm:
+            out.update({x + n + ".norm": (m.dim,) for n in (("q", "k") if own else ("q",))})
+        if m.v_mix:
+            out[x + "vmix"] = ()
+    if isinstance(m, (AttentionSpec, LatentAttentionSpec)) and m.gate:
+        out[x + "g"] = (m.heads, H)
+    if getattr(m, "sink", False):
+        out[x + "sink"] = (m.heads,)
+    out[x + "o"] = (H, vs)
+    return out
+
+
 def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
     """Names and shapes of a layer-list checkpoint: ``l<i>.norm1 / norm1b / norm2 / norm2b`` around the sublayers (parallel
     blocks have ``norm1`` alone, pre-norm blocks ``norm1`` and ``norm2``), ``l<i>.mix.*`` the mixer, ``l<i>.mlp.*`` the feed-forward, with ``e<j>.`` in front of an
-    expert's tensors; linear weights [out, in]. A layer that uses another one's weights has none."""
+    expert's tensors, ``l<i>.canon1`` the input convolution, ``l<i>.rg1 / rg2`` the residual gates; a bias has ``.b`` after the name of
+    its weight; linear weights [out, in]. A layer that uses another one's weights has none."""
     H = cfg.hidden_size
     out: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab_size, H)}
+    if cfg.positions:
+        out["pos"] = (cfg.positions, H)
+
+    def norm(n: str) -> None:
+        out.update({n: (H,), n + ".b": (H,)} if cfg.layer_norm else {n: (H,)})
     for i, layer in enumerate(cfg.layers):
         if layer.weights_of is not None:
             continue
-        p, m = f"l{i}.", layer.mixer
-        x = p + "mix."
+        p = f"l{i}."
         for n in layer_norm_names(cfg, i):
-            out[p + n] = (H,)
-        vs = m.heads * m.vdim
-        if isinstance(m, GatedLinearSpec):
-            ks = m.heads * m.dim
-            out.update({x + "q": (ks, H), x + "k": (ks, H), x + "v": (vs, H), x + "g": (vs, H), x + "norm": (m.vdim,),
-                        x + "a1": (m.rank, H), x + "a2": (ks, m.rank), x + "a2.b": (ks,)})
-        elif isinstance(m, ChannelDeltaSpec):
-            ks, zs = m.kv_heads * m.dim, m.heads * m.dim
-            for n, c in (("q", ks), ("k", ks), ("v", vs)):
-                out.update({x + n: (c, H), x + n + ".conv": (c, m.conv)})
-            out.update({x + "b": (m.heads, H), x + "A_log": (m.heads,), x + "norm": (m.vdim,), x + "a1": (m.rank, H),
-                        x + "a2": (zs, m.rank), x + "dt_bias": (zs,), x + "g1": (m.gate_rank, H),
-                        x + "g2": (vs, m.gate_rank)})
-        elif isinstance(m, LatentAttentionSpec):
-            out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.kv_rank + m.rot_dim, H),
-                        x + "dkv.norm": (m.kv_rank,), x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (vs, m.kv_rank)})
-            if m.gate:
-                out[x + "g"] = (m.heads, H)
-        elif isinstance(m, WkvSpec):
-            out.update({x + "mu." + n: (H,) for n in WKV_MIXES})
-            out.update({x + n: (vs, H) for n in ("r", "k", "v", "g")})
-            out.update({x + "w1": (m.rank, H), x + "w2": (vs, m.rank), x + "w0": (vs,), x + "u": (m.heads, m.dim), x + "norm": (vs,)})
-        else:
-            own = m.kv_from is None
-            out[x + "q"] = (m.heads * m.dim, H)
-            if own:
-                out[x + "k"] = (m.kv_heads * m.dim, H)
-            if own and not m.tied_values:
-                out[x + "v"] = (m.kv_heads * m.vdim, H)
-            if m.qk_norm:
-                out.update({x + n + ".norm": (m.dim,) for n in (("q", "k") if own else ("q",))})
-            if m.v_mix:
-                out[x + "vmix"] = ()
-        if getattr(m, "sink", False):
-            out[x + "sink"] = (m.heads,)
-        out[x + "o"] = (H, vs)
+            norm(p + n)
+        out.update(mixer_shapes(p + "mix.", layer.mixer, H))
+        if cfg.input_conv:
+            out[p + "canon1"] = (H, cfg.input_conv)
+        if cfg.residual_gate:
+            for g in ("rg1", "rg2") if layer.ff or layer.routed else ("rg1",):
+                out.update({p + g: (H, H), p + g + ".b": (H,)})
         gated = lambda q, ff: {q + "gate": (ff, H), q + "up": (ff, H), q + "down": (H, ff)}
         if layer.ff:
             out.update(gated(p + "mlp.", layer.ff))
@@ -103,7 +139,9 @@ def layer_list_shapes(cfg: LayerListConfig) -> Dict[str, Tuple[int, ...]]:
             out[p + "mlp.router"] = (layer.routed.experts, H)
             if layer.routed.correction:
                 out[p + "mlp.correction"] = (layer.routed.experts,)
-    out.update({"final.norm": (H,), "head": (cfg.vocab_size, H)})
+    norm("final.norm")
+    if not cfg.tied_head:
+        out["head"] = (cfg.vocab_size, H)
     return out
 
 
@@ -113,8 +151,16 @@ def _init_layer_list_tensor(cfg: LayerListConfig, name: str, shape: Tuple[int, .
     leaf = name.split(".mix.")[-1]
     if leaf == "u":
         return r * 0.5
-    if len(shape) == 2:
-        return r * (0.02 if name == "embed" else shape[1] ** -0.5)
+    if name.endswith(".canon1") or leaf == "conv":
+        return 0.3 * r
+    if leaf == "lam":
+        return r - 4.0
+    if leaf == "right.f.b":
+        return 0.5 * r + 4.0
+    if leaf.endswith(".b") and leaf != "a2.b":
+        return 0.1 * r
+    if len(shape) >= 2:
+        return r * (0.02 if name in ("embed", "pos") else shape[-1] ** -0.5)
     if leaf == "A_log":
         return r * 0.3
     if leaf == "dt_bias":
@@ -131,8 +177,8 @@ def _init_layer_list_tensor(cfg: LayerListConfig, name: str, shape: Tuple[int, .
         return 0.5 + 0.1 * r
     if leaf == "sink":
         return r
-    # norms of the residual stream: all blocks but the parallel one store offsets from one
-    return 1.0 + 0.05 * r if ".mix." in name or cfg.block == "parallel" else 0.05 * r
+    # norms of the residual stream: RMS norms store offsets from one
+    return 1.0 + 0.05 * r if ".mix." in name or cfg.block == "parallel" or cfg.layer_norm else 0.05 * r
 
 
 def param_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:

@@ -40,6 +40,7 @@ class DmoeGemm(ctypes.Structure):
         ("streamk", ctypes.c_int), ("n_counters", ctypes.c_int), ("pair", ctypes.c_int),
         ("combine_vec", ctypes.c_int), ("w_blocked", ctypes.c_int), ("act", ctypes.c_int),
         ("trace", ctypes.c_void_p),
+        ("act_limit", ctypes.c_float), ("act_cols", ctypes.c_int), ("unit_weights", ctypes.c_int),
     ]
 
 
@@ -70,12 +71,35 @@ class DmoeRecur(ctypes.Structure):
                [(n, _ll) for n in ("ldq", "ldk", "ldv", "ldg", "ldb", "ldz", "ldo", "ldraw")] + \
                [(n, _i) for n in ("n_segs", "n_slots", "heads", "kv_heads", "dim", "vdim", "taps", "delta", "decay_kind",
                                   "gate_kind", "is_f32", "one_token")] + \
-               [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp), ("bonus", _vp), ("norm_ld", _i)]
+               [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp), ("bonus", _vp), ("norm_ld", _i)] + \
+               [(n, _vp) for n in ("head_decay", "gates", "gate_bias", "norm_state", "max_state", "keep", "put", "run_max", "scale")] + \
+               [("ldgates", _ll), ("gate_cap", _f)]
 
 
 class DmoeRouter(ctypes.Structure):
     _fields_ = [(n, _vp) for n in ("weight", "correction", "ids", "wts", "counts")] + \
                [(n, _i) for n in ("E", "K", "renorm", "sigmoid", "groups", "keep")] + [("wscale", _f)]
+
+
+class DmoeConv(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("w", "in_bias", "out_bias", "ring", "singles", "positions", "rows", "kv_slots")] + \
+               [(n, _i) for n in ("n_single", "n_slots", "taps", "residual", "blocks", "padded")]
+
+
+class DmoeSumExtra(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("bias", "gate_z", "gate_bias", "side", "side_w", "conv")] + \
+               [(n, _ll) for n in ("ld_gate", "ld_side", "side_stride")] + [("side_scale", _f)]
+
+
+class DmoeAttnExtra(ctypes.Structure):
+    _fields_ = [("gate", _vp), ("ld_gate", _ll), ("temp_coef", _f), ("temp_every", _i)]
+
+
+class DmoeUnit(ctypes.Structure):
+    _fields_ = [(n, _vp) for n in ("u", "gates", "gate_bias", "decay", "y", "y_bias", "state", "out", "singles", "positions", "rows",
+                                   "kv_slots", "multi")] + \
+               [(n, _ll) for n in ("ldy", "ldo", "block_rows")] + \
+               [(n, _i) for n in ("n_single", "n_multi", "n_slots", "width", "blocks", "padded")]
 
 
 class DmoeShift(ctypes.Structure):

@@ -99,7 +99,7 @@ _attn_ws = {}
 
 # (key size, value size) of the tensor-core kernels over the paged cache: with options (window, soft cap, sink, fp32 softmax
 # weights) for query groups of any size up to 64 heads, without for equal sizes and groups of 1, 2, 4 or 8.
-ATTN_TILES = ((64, 32), (64, 64), (128, 64), (128, 128))
+ATTN_TILES = ((64, 32), (64, 64), (64, 128), (128, 64), (128, 128))
 
 
 def attention_on_tensor_cores(dtype, n_q: int, n_kv: int, hd: int, vd: int) -> bool:
@@ -134,16 +134,19 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
                     out: Optional[torch.Tensor] = None, splits: int = 1, scale: Optional[float] = None,
                     window: Optional[int] = None, softcap: Optional[float] = None, fp32_weights: bool = False,
-                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None, q_temp=None,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = softmax(q[t] K^T * scale) V over the first ctx_len[t] cached tokens of block-table row bt_row[t], or the
     last ``window`` of them, or those from the start of the last one's ``chunk`` (of so many positions, counted from position
     0) on; ``softcap``: scores are soft-capped, cap * tanh(score / cap); ``sink`` (fp32 [n_q]): the softmax
     denominator has exp(sink) of the head in addition. ``fp32_weights`` keeps the softmax weights at fp32 accuracy in the
-    product with V (implied by the options before). Value heads may have another size than key heads
+    product with V (implied by the options before). ``q_temp`` (:class:`disagmoe_b200.config.QueryTemperature`): scores are multiplied by the query's
+    temperature at its position; ``gate`` ([T, n_q], columns of a wider matrix are fine): every head's output is multiplied by
+    sigmoid(gate). Value heads may have another size than key heads
     (``vcache.shape[-1]``)."""
     if not q.is_cuda:
         o = reference.paged_attention(q, kcache, vcache, block_tables, bt_row, ctx_len, n_q, n_kv, hd, scale, window, softcap,
-                                      sink, chunk)
+                                      sink, chunk, q_temp, gate)
         if out is not None:
             out.copy_(o)
             return out
@@ -156,15 +159,17 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     _check_sink(sink, n_q)
     if not attention_on_tensor_cores(q.dtype, n_q, n_kv, hd, vd):
         return _any_attention(q, hd, q.stride(0), kcache, vcache, block_tables, bt_row, None, ctx_len, T, n_q, n_kv, hd, vd,
-                              scale, window, softcap, sink, out, vd, out.stride(0), chunk)
+                              scale, window, softcap, sink, out, vd, out.stride(0), chunk, q_temp, gate)
     assert block_tables.dtype == torch.int32 and ctx_len.dtype == torch.int32 and block_tables.stride(1) == 1
     ws = _attn_workspace(q.device, T * n_q * splits * (vd + 1)) if splits > 1 else None
-    if window or chunk or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
+    if window or chunk or softcap or fp32_weights or sink is not None or q_temp is not None or gate is not None or hd != vd or \
+            n_q // n_kv not in (1, 2, 4, 8):
+        x = _attn_extra(q_temp, gate, q.dtype)
         _lib.check(_lib.lib().dmoe_paged_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
             _vp(bt_row), _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd),
             c_float(scale), c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), c_int(splits), _vp(out),
-            c_ll(out.stride(0)), _vp(ws), _st()), "dmoe_paged_attention_ext")
+            c_ll(out.stride(0)), _vp(ws), ctypes.byref(x) if x else None, _st()), "dmoe_paged_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_paged_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
@@ -173,19 +178,28 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     return out
 
 
+def _attn_extra(q_temp, gate, dtype) -> Optional[_lib.DmoeAttnExtra]:
+    if q_temp is None and gate is None:
+        return None
+    assert gate is None or (gate.dtype == dtype and gate.stride(1) == 1)
+    return _lib.DmoeAttnExtra(_lib.ptr(gate), gate.stride(0) if gate is not None else 0, q_temp.coef if q_temp else 0.0,
+                              q_temp.every if q_temp else 0)
+
+
 def _any_attention(q, q_head, q_row, kcache, vcache, block_tables, bt_row, rows, ctx_len, T, n_q, n_kv, hd, vd, scale, window,
-                   softcap, sink, out, o_head, o_row, chunk=None):
+                   softcap, sink, out, o_head, o_row, chunk=None, q_temp=None, gate=None):
     """CUDA-core attention with free strides: query t of head h at q + t * q_row + h * q_head, likewise the output; the
     cached heads of a token are contiguous, tokens ``stride(1)`` apart. Query t has the context of batch row rows[t]
     (None: t)."""
     assert q.dtype == kcache.dtype == vcache.dtype == out.dtype
+    x = _attn_extra(q_temp, gate, q.dtype)
     assert kcache.stride(0) == kcache.shape[1] * kcache.stride(1) and vcache.stride(0) == vcache.shape[1] * vcache.stride(1)
     _lib.check(_lib.lib().dmoe_any_attention(
         c_int(int(q.dtype == torch.float32)), _vp(q), c_ll(q_head), c_ll(q_row), _vp(kcache), c_ll(kcache.stride(1)),
         _vp(vcache), c_ll(vcache.stride(1)), _vp(block_tables), c_int(block_tables.stride(0)), _vp(bt_row), _vp(rows),
         _vp(ctx_len), c_int(kcache.shape[1]), c_int(T), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
-        c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(o_head), c_ll(o_row), _st()),
-        "dmoe_any_attention")
+        c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(o_head), c_ll(o_row),
+        ctypes.byref(x) if x else None, _st()), "dmoe_any_attention")
     return out
 
 
@@ -442,7 +456,7 @@ def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
                       tiles: torch.Tensor, n_tiles: int, n_q: int, n_kv: int, hd: int, out: torch.Tensor,
                       scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
                       fp32_weights: bool = False, sink: Optional[torch.Tensor] = None,
-                      chunk: Optional[int] = None) -> torch.Tensor:
+                      chunk: Optional[int] = None, q_temp=None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the prompt tokens named by ``tiles`` (device int32 [>= n_tiles, 4], see
     :func:`build_prefill_tiles`) over the paged cache, which already holds their own K / V; writes their rows of
     ``out``. Every tile streams its sequence's K / V once (the per-token kernel streams it once per row)."""
@@ -452,12 +466,14 @@ def prefill_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     vd = vcache.shape[-1]
     _check_sink(sink, n_q)
-    if window or chunk or softcap or fp32_weights or sink is not None or hd != vd or n_q // n_kv not in (1, 2, 4, 8):
+    if window or chunk or softcap or fp32_weights or sink is not None or q_temp is not None or gate is not None or hd != vd or \
+            n_q // n_kv not in (1, 2, 4, 8):
+        x = _attn_extra(q_temp, gate, q.dtype)
         _lib.check(_lib.lib().dmoe_prefill_attention_ext(
             _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)),
             _vp(tiles), c_int(n_tiles), c_int(kcache.shape[1]), c_int(n_q), c_int(n_kv), c_int(hd), c_int(vd), c_float(scale),
-            c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(out.stride(0)), _st()),
-            "dmoe_prefill_attention_ext")
+            c_int(window or 0), c_int(chunk or 0), c_float(softcap or 0.0), _vp(sink), _vp(out), c_ll(out.stride(0)),
+            ctypes.byref(x) if x else None, _st()), "dmoe_prefill_attention_ext")
         return out
     _lib.check(_lib.lib().dmoe_prefill_attention(
         _vp(q), c_ll(q.stride(0)), _vp(kcache), _vp(vcache), _vp(block_tables), c_int(block_tables.stride(0)), _vp(tiles),
@@ -472,15 +488,21 @@ def _f32(dtype) -> c_int:
     return c_int(int(dtype == torch.float32))
 
 
-def embed_f32(ids: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor) -> torch.Tensor:
-    """out (fp32) = table[ids] * scale."""
+def embed_f32(ids: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor, positions: Optional[torch.Tensor] = None,
+              pos_table: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out (fp32) = table[ids] * scale (+ pos_table[positions])."""
     if not table.is_cuda:
         out.copy_(table[ids.long()].float() * scale)
+        if pos_table is not None:
+            out += pos_table[positions.long()].float()
         return out
+    assert pos_table is None or (pos_table.dtype == table.dtype and pos_table.is_contiguous() and positions.dtype == torch.int32 and
+                                 pos_table.shape[1] == table.shape[1])
     assert ids.dtype == torch.int32 and table.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32
     _lib.check(_lib.lib().dmoe_embed_f32(_vp(ids), _vp(table), _f32(table.dtype), c_float(scale), _vp(out),
-                                         c_int(ids.shape[0]), c_int(table.shape[1]), c_int(table.shape[0]), _st()),
-               "dmoe_embed_f32")
+                                         c_int(ids.shape[0]), c_int(table.shape[1]), c_int(table.shape[0]),
+                                         _vp(positions if pos_table is not None else None), _vp(pos_table),
+                                         c_int(0 if pos_table is None else pos_table.shape[0]), _st()), "dmoe_embed_f32")
     return out
 
 
@@ -556,16 +578,88 @@ def token_shift(h: torch.Tensor, shift: TokenShift, dtype: torch.dtype) -> torch
     return out
 
 
-def sum_norm(resid: torch.Tensor, y: Optional[torch.Tensor], parts: Optional[torch.Tensor], w: torch.Tensor, eps: float,
+@dataclass
+class ResidualGate:
+    """What joins the residual stream is multiplied, number by number, by sigmoid(z + bias): z [T, W], bias fp32 [W]."""
+    z: torch.Tensor
+    bias: torch.Tensor
+
+
+@dataclass
+class Sides:
+    """Outputs of two mixers on the same rows, ``rows`` [2, T, W]; together they are scale * the sum of their RMS norms over the
+    width, each times its weights (fp32 [2, W])."""
+    rows: torch.Tensor
+    weights: torch.Tensor
+    scale: float = 0.5
+
+
+@dataclass
+class InputConv:
+    """h + causal convolution of h per channel: ``w`` fp32 [taps, W] (the last row belongs to the token itself); ``ring`` [slots,
+    taps, W] keeps a sequence's last rows by position modulo taps (not read before position 0); ``segs``: the step's segments."""
+    w: torch.Tensor
+    ring: torch.Tensor
+    segs: "SegmentTables"                        # noqa: F821
+
+    def descriptor(self) -> _lib.DmoeConv:
+        return _conv_descriptor(self.w, self.ring, self.segs)
+
+
+def _conv_descriptor(w, ring, segs, in_bias=None, out_bias=None, residual=True, blocks=1, padded=0) -> _lib.DmoeConv:
+    d, (taps, C) = _lib.DmoeConv(), w.shape
+    assert w.dtype == torch.float32 and w.is_contiguous() and ring.is_contiguous() and ring.shape[1:] == (taps, C)
+    assert all(b is None or (b.dtype == torch.float32 and b.numel() == C) for b in (in_bias, out_bias))
+    d.w, d.in_bias, d.out_bias, d.ring = w.data_ptr(), _lib.ptr(in_bias), _lib.ptr(out_bias), ring.data_ptr()
+    d.singles = _lib.ptr(segs.singles) if segs.n_single else 0
+    d.positions, d.rows, d.kv_slots = _lib.ptr(segs.positions), _lib.ptr(segs.rows), _lib.ptr(segs.kv_slots)
+    d.n_single, d.n_slots, d.taps, d.residual, d.blocks, d.padded = segs.n_single, ring.shape[0], taps, int(residual), blocks, padded
+    return d
+
+
+def seq_conv(x: torch.Tensor, w: torch.Tensor, ring: torch.Tensor, segs, in_bias: Optional[torch.Tensor] = None,
+             out_bias: Optional[torch.Tensor] = None, residual: bool = False, blocks: int = 1,
+             out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal convolution over time of every column of x [T, C] + in_bias within its segment: sum_j w[j] x_(t - taps + 1 + j) +
+    out_bias, with ``residual`` plus x itself. ``ring`` [slots, taps, C] keeps the last rows of x of every sequence by position modulo
+    taps. blocks > 1: returns the equal blocks of columns one after the other, [blocks, T, n] with n = C / blocks padded with
+    zeros to a multiple of 8."""
+    T, C = x.shape
+    n = C // blocks
+    padded = (n + 7) // 8 * 8 if blocks > 1 else n
+    if not x.is_cuda:
+        y = reference.seq_conv(x, w, ring, segs, in_bias, out_bias, residual).to(x.dtype)
+        if blocks > 1:
+            y = torch.nn.functional.pad(y.view(T, blocks, n).transpose(0, 1), (0, padded - n)).contiguous()
+        if out is not None:
+            return out.copy_(y)
+        return y
+    if out is None:
+        shape = (blocks, T, padded) if blocks > 1 else (T, C)
+        out = (torch.empty if padded == n else torch.zeros)(shape, dtype=x.dtype, device=x.device)
+    assert x.stride(1) == 1 and ring.dtype == x.dtype == out.dtype and out.stride(-1) == 1 and C == w.shape[1]
+    d = _conv_descriptor(w, ring, segs, in_bias, out_bias, residual, blocks, padded)
+    _lib.check(_lib.lib().dmoe_seq_conv(_f32(x.dtype), _vp(x), c_ll(x.stride(0)), ctypes.byref(d), _vp(segs.multi), c_int(segs.n_multi),
+                                        _vp(segs.chunks), c_int(segs.n_chunks), _vp(out), c_ll(out.stride(-2)),
+                                        c_ll(out.stride(0) if blocks > 1 else 0), c_int(C), _st()), "dmoe_seq_conv")
+    return out
+
+
+def sum_norm(resid: torch.Tensor, y, parts: Optional[torch.Tensor], w: torch.Tensor, eps: float,
              dtype: torch.dtype, centred: bool, rows: Optional[torch.Tensor] = None, router: Optional[Router] = None,
-             mult: float = 1.0, shift: Optional[TokenShift] = None):
-    """One step of a residual stream kept in fp32: resid += mult * (y + parts.sum(1)) (y [T, W], parts [T, P, W] or [T, W],
-    each may be None), then h = norm(resid) * w in ``dtype``; ``centred``: layer norm, otherwise RMS norm. ``rows`` (int32)
+             mult: float = 1.0, shift: Optional[TokenShift] = None, bias: Optional[torch.Tensor] = None,
+             gate: Optional[ResidualGate] = None, conv: Optional[InputConv] = None):
+    """One step of a residual stream kept in fp32: resid += mult * (y + parts.sum(1)) (y [T, W] or :class:`Sides`, parts [T, P, W] or
+    [T, W], each may be None; with a ``gate`` multiplied by its sigmoid), then h = norm(resid) * w (+ bias, fp32 [W]) in ``dtype``; ``centred``: layer norm, otherwise RMS norm. ``rows`` (int32)
     picks the rows to return; resid itself is then left as it is. Returns (h, expert ids [T, top], weights [T, top]), the last
     two None without a ``router``, which sees h. With a token ``shift``, h (kept in fp32 on the way) becomes its mixes
-    [n, T, W]; where every segment has one token (decoding) that is one launch."""
+    [n, T, W]; where every segment has one token (decoding) that is one launch. With an input ``conv``, h becomes [2, T, W]: h and
+    its convolved rows, likewise in one launch where every segment has one token."""
+    y, sides = (None, y) if isinstance(y, Sides) else (y, None)
     if not resid.is_cuda:
-        h = reference.sum_norm(resid, y, parts, w, eps, torch.float32 if shift else dtype, centred, rows, mult)
+        h = reference.sum_norm(resid, y, parts, w, eps, torch.float32 if shift else dtype, centred, rows, mult, bias, gate, sides)
+        if conv is not None:
+            return torch.stack([h, seq_conv(h, conv.w, conv.ring, conv.segs, residual=True)]), None, None
         if shift is not None:
             return token_shift(h, shift, dtype), None, None
         if router is None:
@@ -582,8 +676,8 @@ def sum_norm(resid: torch.Tensor, y: Optional[torch.Tensor], parts: Optional[tor
     if parts is not None and parts.dim() == 2:
         parts = parts.unsqueeze(1)
     two_steps = shift is not None and shift.segs.n_multi > 0
-    h = torch.empty((n, W) if shift is None or two_steps else (shift.mu.shape[0], n, W),
-                    dtype=torch.float32 if two_steps else dtype, device=resid.device)
+    shape = (2, n, W) if conv is not None else (n, W) if shift is None or two_steps else (shift.mu.shape[0], n, W)
+    h = torch.empty(shape, dtype=torch.float32 if two_steps else dtype, device=resid.device)
     assert resid.dtype == torch.float32 and resid.is_contiguous() and w.dtype == torch.float32
     assert all(a is None or (a.dtype == dtype and a.stride(-1) == 1) for a in (y, parts)) and (rows is None or rows.dtype == torch.int32)
     ids = wts = rd = sd = None
@@ -598,12 +692,33 @@ def sum_norm(resid: torch.Tensor, y: Optional[torch.Tensor], parts: Optional[tor
                              int(router.renormalize), int(router.sigmoid), router.groups, router.keep, router.scale)
     if shift is not None and not two_steps:
         sd = shift.descriptor(n)
+    x = cd = None
+    if bias is not None or gate is not None or sides is not None or conv is not None:
+        x = _lib.DmoeSumExtra()
+        assert bias is None or (bias.dtype == torch.float32 and bias.numel() == W)
+        x.bias = _lib.ptr(bias)
+        if gate is not None:
+            assert gate.z.dtype == dtype and gate.z.stride(1) == 1 and gate.bias.dtype == torch.float32 and gate.z.shape[1] == W
+            x.gate_z, x.gate_bias, x.ld_gate = gate.z.data_ptr(), gate.bias.data_ptr(), gate.z.stride(0)
+        if sides is not None:
+            s = sides.rows
+            assert s.dtype == dtype and s.stride(2) == 1 and s.shape[2] == W and sides.weights.dtype == torch.float32 and \
+                sides.weights.is_contiguous()
+            x.side, x.side_w, x.ld_side, x.side_stride, x.side_scale = s.data_ptr(), sides.weights.data_ptr(), s.stride(1), \
+                s.stride(0), sides.scale
+        if conv is not None:
+            assert rows is None and router is None and shift is None and conv.w.shape[1] == W and conv.ring.dtype == dtype
+            if conv.segs.n_multi == 0:
+                cd = conv.descriptor()
+                x.conv = ctypes.addressof(cd)
     _lib.check(_lib.lib().dmoe_sum_norm(
         _f32(dtype), _vp(resid), _vp(y), c_ll(y.stride(0) if y is not None else 0), _vp(parts),
         c_int(parts.shape[1] if parts is not None else 0), c_ll(parts.stride(0) if parts is not None else 0),
         c_ll(parts.stride(1) if parts is not None else 0), c_float(mult), _vp(w), c_int(int(centred)), c_float(eps), _vp(rows),
         _vp(h), c_int(int(two_steps)), c_ll(W), c_int(n), c_int(W), ctypes.byref(rd) if rd else None,
-        ctypes.byref(sd) if sd else None, _st()), "dmoe_sum_norm")
+        ctypes.byref(sd) if sd else None, ctypes.byref(x) if x else None, _st()), "dmoe_sum_norm")
+    if conv is not None and cd is None:
+        seq_conv(h[0], conv.w, conv.ring, conv.segs, residual=True, out=h[1])
     return (token_shift(h, shift, dtype) if two_steps else h), ids, wts
 
 
@@ -650,15 +765,16 @@ def rope_freq_table(spec, max_pos: int, device) -> Optional[torch.Tensor]:
 def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: Optional[torch.Tensor],
                  vcache: Optional[torch.Tensor], n_q: int, n_kv: int, dk: int, dv: int, table: Optional[torch.Tensor],
                  qw: Optional[torch.Tensor], kw: Optional[torch.Tensor], eps: float, interleaved: bool = False,
-                 v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, tied: bool = False) -> None:
+                 v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, tied: bool = False, v_norm: int = 0) -> None:
     """RMS norm of every q / k head (weights fp32 [dk]; None: no norm) and rotation by ``table`` (:func:`rope_freq_table`,
     None: no rotation; ``interleaved``: of neighbouring dimensions) on rows [q | k | v]; q in place, k and v to the paged
     caches at ``slots``. n_kv = 0: q only (a layer that reads another layer's cache). ``v_first`` [T, n_kv, >= dv]: the
     values become (1 - v_lambda) v + v_lambda v_first on their way to the cache. ``tied``: rows [q | k], the values are the first
-    dv dimensions of the keys before their norm and rotation."""
+    dv dimensions of the keys before their norm and rotation. ``v_norm`` > 0: every value head is divided by its root mean square over that
+    many dimensions (the rest of it is padding)."""
     if not qkv.is_cuda:
         return reference.qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps,
-                                      interleaved, v_first, v_lambda, tied)
+                                      interleaved, v_first, v_lambda, tied, v_norm)
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and qkv.stride(1) == 1
     assert n_kv == 0 or (kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == qkv.dtype)
     rot, max_pos = (2 * table.shape[1], table.shape[0]) if table is not None else (0, 1 << 30)
@@ -666,7 +782,8 @@ def qk_norm_rope(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor
         _f32(qkv.dtype), _vp(qkv), c_ll(qkv.stride(0)), _vp(positions), _vp(slots), _vp(kcache), _vp(vcache),
         c_int(qkv.shape[0]), c_int(n_q), c_int(n_kv), c_int(dk), c_int(dv), c_int(rot), c_int(int(interleaved)), _vp(table),
         c_int(max_pos), _vp(qw), _vp(kw), c_float(eps), _vp(v_first), c_ll(v_first.stride(0) if v_first is not None else 0),
-        c_int(v_first.stride(1) if v_first is not None else 0), c_float(v_lambda), c_int(int(tied)), _st()), "dmoe_qk_norm_rope")
+        c_int(v_first.stride(1) if v_first is not None else 0), c_float(v_lambda), c_int(int(tied)), c_int(v_norm),
+        _st()), "dmoe_qk_norm_rope")
 
 
 # ---- latent attention (csrc/kernels/latent_attention.cu) ---------------------------------------------------------------

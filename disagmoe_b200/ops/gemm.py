@@ -20,8 +20,8 @@ import torch
 
 from . import _lib, reference
 
-ACTS = {"silu": 0, "gelu_tanh": 1}
-ACT_TANH = 2         # of the output of a plain GEMM
+ACTS = {"silu": 0, "gelu_tanh": 1, "clamped": 3}      # of gated feed-forwards; clamped: min(g, limit) sigmoid(1.702 g) (clamp(u) + 1)
+ACT_TANH, ACT_SILU = 2, 4      # of the output of a plain GEMM (silu: of its first columns)
 EPI_PLAIN, EPI_SWIGLU, EPI_COMBINE = 0, 1, 2
 STREAM_K = True      # default work distribution of every GEMM launched without an explicit split (tests may turn it off)
 TRACE = None         # profiling aid: an int64 [8] CUDA tensor that CTA 0 of every launch fills with nanosecond stamps
@@ -222,9 +222,11 @@ def rope_table(max_pos: int, hd: int, theta: float, device) -> torch.Tensor:
 
 
 def _launch(W, X, Y, R, offs, recs, bases, G, T, F, K, epi, bn, splitk, ldy, y_f32, comm: Optional[GemmComm] = None,
-            streamk: bool = False, pair: bool = False, w_blocked: bool = False, act: int = 0):
+            streamk: bool = False, pair: bool = False, w_blocked: bool = False, act: int = 0, act_limit: float = 0.0,
+            act_cols: int = 0, unit_weights: bool = False):
     s = scratch(X.device)
     d = _lib.DmoeGemm()
+    d.act_limit, d.act_cols, d.unit_weights = act_limit, act_cols, int(unit_weights)
     d.w_blocked, d.act = int(w_blocked), act
     d.trace = TRACE.data_ptr() if TRACE is not None else None
     d.streamk, d.n_counters = int(streamk and splitk <= 1 and not pair), s.counters.numel()
@@ -252,7 +254,7 @@ def _tma_ok(x, w) -> bool:
     return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
 
 
-def _simt_linear(x, w, out, out_dtype, tanh=False):
+def _simt_linear(x, w, out, out_dtype, tanh=False, silu_cols=0):
     """fp32 operands (true fp32 arithmetic), or bf16 operands that TMA cannot address: the CUDA-core GEMM."""
     T, K = x.shape
     F = w.shape[0]
@@ -264,31 +266,32 @@ def _simt_linear(x, w, out, out_dtype, tanh=False):
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
     _lib.check(_lib.lib().dmoe_simt_linear(
         i(int(f32)), i(int(out.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), ll(K),
-        v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), i(ACT_TANH if tanh else 0), v(_lib.stream_ptr())), "dmoe_simt_linear")
+        v(out.data_ptr()), ll(out.stride(0)), i(T), i(F), i(K), i(ACT_TANH if tanh else ACT_SILU if silu_cols else 0), i(silu_cols),
+        v(_lib.stream_ptr())), "dmoe_simt_linear")
     return out
 
 
-def _simt_grouped(x, w, offs, out, recs=None, base=None, ld_out=0):
+def _simt_grouped(x, w, offs, out, recs=None, base=None, ld_out=0, unit_weights=False):
     """The CUDA-core GEMM over row groups: rows offs[g] .. offs[g + 1] of x times w[g].T, into ``out`` or, with ``recs``
     (combine), scaled and scattered to rows of the buffer at ``base[0]`` in x's dtype."""
     T, K = x.shape
     G, F, _ = w.shape
     assert w.is_contiguous() and w.dtype == x.dtype and w.shape[2] == K and x.stride(1) == 1
-    assert offs.dtype == torch.int32 and (out is None or out.dtype == x.dtype)
+    assert offs.dtype == torch.int32 and (out is None or out.dtype in (x.dtype, torch.float32))
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
     _lib.check(_lib.lib().dmoe_simt_grouped(
-        i(int(x.dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)), v(w.data_ptr()), v(offs.data_ptr()), i(G),
-        v(_lib.ptr(out)), ll(out.stride(0) if out is not None else ld_out), v(_lib.ptr(recs)), v(_lib.ptr(base)), i(T), i(F),
-        i(K), v(_lib.stream_ptr())), "dmoe_simt_grouped")
+        i(int(x.dtype == torch.float32)), i(int((x if out is None else out).dtype == torch.float32)), v(x.data_ptr()), ll(x.stride(0)),
+        v(w.data_ptr()), v(offs.data_ptr()), i(G), v(_lib.ptr(out)), ll(out.stride(0) if out is not None else ld_out),
+        v(_lib.ptr(recs)), v(_lib.ptr(base)), i(int(unit_weights)), i(T), i(F), i(K), v(_lib.stream_ptr())), "dmoe_simt_grouped")
     return out
 
 
-def _gate_mul(gu, out, I: int, act: str):
-    """out = act(gu[:, :I]) * gu[:, I:]"""
+def _gate_mul(gu, out, I: int, act: str, limit: float = 0.0, recs=None):
+    """out = act(gu[:, :I]) * gu[:, I:], gu scaled by the weights of ``recs`` first where these are given."""
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
     _lib.check(_lib.lib().dmoe_gate_mul(i(int(gu.dtype == torch.float32)), i(ACTS[act]), v(gu.data_ptr()), ll(gu.stride(0)),
-                                        v(out.data_ptr()), ll(out.stride(0)), i(gu.shape[0]), i(I), v(_lib.stream_ptr())),
-               "dmoe_gate_mul")
+                                        v(out.data_ptr()), ll(out.stride(0)), i(gu.shape[0]), i(I), ctypes.c_float(limit), v(_lib.ptr(recs)),
+                                        v(_lib.stream_ptr())), "dmoe_gate_mul")
     return out
 
 
@@ -299,8 +302,9 @@ def _check_x(x):
 
 def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = None,
            out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, bn: int = 0,
-           splitk: int = 0, comm: Optional["GemmComm"] = None, pair: bool = False, tanh: bool = False) -> torch.Tensor:
-    """y[T, F] = x[T, K] @ w[F, K].T (+ residual[T, F]); ``tanh``: of the product. ``pair``: CTA pairs (tcgen05 cta_group::2) on tiles of 256
+           splitk: int = 0, comm: Optional["GemmComm"] = None, pair: bool = False, tanh: bool = False,
+           silu_cols: int = 0) -> torch.Tensor:
+    """y[T, F] = x[T, K] @ w[F, K].T (+ residual[T, F]); ``tanh``: of the product; ``silu_cols``: silu of the first so many columns. ``pair``: CTA pairs (tcgen05 cta_group::2) on tiles of 256
     weight rows x ``bn`` (128 / 256) tokens, whole tiles."""
     T, K = x.shape
     F = w.shape[0]
@@ -308,6 +312,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         y = torch.nn.functional.linear(x.float(), w.float())
         if tanh:
             y = torch.tanh(y)
+        if silu_cols:
+            y[:, :silu_cols] = torch.nn.functional.silu(y[:, :silu_cols])
         if residual is not None:
             y = y + residual.float()
         y = y.to(out_dtype or x.dtype)
@@ -317,7 +323,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         return y
     if x.dtype == torch.float32 or (comm is None and residual is None and not _tma_ok(x, w)):
         assert comm is None and residual is None
-        return _simt_linear(x, w, out, out_dtype, tanh)
+        return _simt_linear(x, w, out, out_dtype, tanh, silu_cols)
     _check_x(x)
     assert w.is_contiguous() and w.dtype == torch.bfloat16 and w.shape[1] == K
     odt = out_dtype or torch.bfloat16
@@ -346,11 +352,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         splitk = splitk or auto_sk or pick_splitk(T, F, K, bn, sms)
     _launch(w, x, out, residual, None, None, None, 1, T, F, K, EPI_PLAIN, bn, splitk,
             F if scatter else out.stride(0), (not scatter) and out.dtype == torch.float32, comm, streamk=streamk,
-            pair=pair, act=ACT_TANH if tanh else 0)
+            pair=pair, act=ACT_TANH if tanh else ACT_SILU if silu_cols else 0, act_cols=silu_cols)
     return out
 
 
-def _grouped_ref(x, w, offs, swiglu, act="silu"):
+def _grouped_ref(x, w, offs, swiglu, act="silu", limit=0.0, recs=None):
     offs = offs.tolist()
     G = w.shape[0]
     F = w.shape[1] // 2 if swiglu else w.shape[1]
@@ -360,30 +366,35 @@ def _grouped_ref(x, w, offs, swiglu, act="silu"):
         if b <= a:
             continue
         h = x[a:b].float() @ w[g].float().T
+        if recs is not None:
+            h = h * recs[a:b, 2].contiguous().view(torch.float32)[:, None]
         if swiglu:
-            h = reference.swiglu(h, act)
+            h = reference.swiglu(h, act, limit)
         y[a:b] = h
     return y
 
 
 def grouped_swiglu(x: torch.Tensor, w13: torch.Tensor, offs: Optional[torch.Tensor], out: Optional[torch.Tensor] = None,
                    bn: int = 0, comm: Optional[GemmComm] = None, streamk: Optional[bool] = None,
-                   pair: bool = False, w_blocked: bool = False, act: str = "silu") -> torch.Tensor:
-    """y[T, I] = act(x @ w13[g, :I].T) * (x @ w13[g, I:].T) for the rows of group g; w13 is [G, 2I, K]."""
+                   pair: bool = False, w_blocked: bool = False, act: str = "silu", limit: float = 0.0,
+                   recs: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[T, I] = act(x @ w13[g, :I].T) * (x @ w13[g, I:].T) for the rows of group g; w13 is [G, 2I, K]. ``recs``: row t of x counts
+    with the weight of its record (see :func:`grouped_combine`)."""
     T, K = x.shape
     G, F2, _ = w13.shape
     I = F2 // 2
     if not x.is_cuda:
-        y = _grouped_ref(x, w13, offs, True, act).to(x.dtype)
+        y = _grouped_ref(x, w13, offs, True, act, limit, recs).to(x.dtype)
         if out is not None:
             out.copy_(y)
             return out
         return y
     if x.dtype == torch.float32 or (comm is None and not w_blocked and not _tma_ok(x, w13)):
         gu = _simt_grouped(x, w13, offs, torch.empty(T, F2, dtype=x.dtype, device=x.device))
-        return _gate_mul(gu, torch.empty(T, I, dtype=x.dtype, device=x.device) if out is None else out, I, act)
+        return _gate_mul(gu, torch.empty(T, I, dtype=x.dtype, device=x.device) if out is None else out, I, act, limit, recs)
     _check_x(x)
     assert w13.is_contiguous() and w13.dtype == torch.bfloat16
+    assert recs is None or (recs.dtype == torch.int32 and recs.is_contiguous() and recs.shape[1] == 4)
     assert comm is not None or (offs.dtype == torch.int32 and offs.is_cuda)
     if out is None:
         out = torch.empty(T, I, dtype=torch.bfloat16, device=x.device)
@@ -393,37 +404,38 @@ def grouped_swiglu(x: torch.Tensor, w13: torch.Tensor, offs: Optional[torch.Tens
     if pair:
         bn = max(bn, 128)
     sk = want_streamk(EPI_SWIGLU, I, G, T, bn, num_sms(x.device)) if streamk is None else streamk
-    _launch(w13, x, out, None, offs, None, None, G, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False, comm,
-            streamk=sk, pair=pair, w_blocked=w_blocked, act=ACTS[act])
+    _launch(w13, x, out, None, offs, recs, None, G, T, I, K, EPI_SWIGLU, bn, 1, out.stride(0), False, comm,
+            streamk=sk, pair=pair, w_blocked=w_blocked, act=ACTS[act], act_limit=limit)
     return out
 
 
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, out: Optional[torch.Tensor] = None,
                    bn: int = 0, streamk: Optional[bool] = None, pair: bool = False,
-                   w_blocked: bool = False) -> torch.Tensor:
-    """y[T, F] = x @ w[g].T for the rows of group g; w is [G, F, K]."""
+                   w_blocked: bool = False, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """y[T, F] = x @ w[g].T for the rows of group g; w is [G, F, K]. ``out_dtype``: that of x, or fp32."""
     T, K = x.shape
     G, F, _ = w.shape
+    dt = out.dtype if out is not None else out_dtype or x.dtype
     if not x.is_cuda:
-        y = _grouped_ref(x, w, offs, False).to(x.dtype)
+        y = _grouped_ref(x, w, offs, False).to(dt)
         if out is not None:
             out.copy_(y)
             return out
         return y
     if x.dtype == torch.float32 or (not w_blocked and not _tma_ok(x, w)):
-        return _simt_grouped(x, w, offs, torch.empty(T, F, dtype=x.dtype, device=x.device) if out is None else out)
+        return _simt_grouped(x, w, offs, torch.empty(T, F, dtype=dt, device=x.device) if out is None else out)
     _check_x(x)
     assert w.is_contiguous() and w.dtype == torch.bfloat16 and offs.dtype == torch.int32 and offs.is_cuda
     if out is None:
-        out = torch.empty(T, F, dtype=torch.bfloat16, device=x.device)
+        out = torch.empty(T, F, dtype=dt, device=x.device)
     if T == 0:
         return out
     bn = bn or pick_bn(_group_hint(T, G), EPI_PLAIN)
     if pair:
         bn = max(bn, 128)
     sk = want_streamk(EPI_PLAIN, F, G, T, bn, num_sms(x.device)) if streamk is None else streamk
-    _launch(w, x, out, None, offs, None, None, G, T, F, K, EPI_PLAIN, bn, 1, out.stride(0), False, streamk=sk, pair=pair,
-            w_blocked=w_blocked)
+    _launch(w, x, out, None, offs, None, None, G, T, F, K, EPI_PLAIN, bn, 1, out.stride(0), out.dtype == torch.float32,
+            streamk=sk, pair=pair, w_blocked=w_blocked)
     return out
 
 
@@ -464,23 +476,27 @@ def _bases_aligned(bases: torch.Tensor) -> bool:
 
 def grouped_combine(x: torch.Tensor, w: torch.Tensor, offs: Optional[torch.Tensor], recs: torch.Tensor,
                     bases: torch.Tensor, ld_out: int, bn: int = 0, outs=None, comm: Optional[GemmComm] = None,
-                    streamk: Optional[bool] = None, pair: bool = False, w_blocked: bool = False) -> None:
+                    streamk: Optional[bool] = None, pair: bool = False, w_blocked: bool = False,
+                    unit_weights: bool = False) -> None:
     """GEMM-2 with the combine epilogue: row t of group g becomes ``weight[t] * (x[t] @ w[g].T)`` written to row
     ``recs[t, 1]`` of the buffer ``bases[recs[t, 0]]`` (row stride ``ld_out`` elements).
 
     recs: int32 [T, 4] = (dst_rank, dst_row or -1, weight as fp32 bits, 0). bases: int64 [n_ranks] device
     tensor of raw pointers (peer buffers included). ``outs`` (CPU path only) is the list of destination tensors.
+    ``unit_weights``: the records' weights are left out.
     """
     T, K = x.shape
     G, F, _ = w.shape
     if not x.is_cuda:
-        y = _grouped_ref(x, w, offs, False) * recs[:, 2].contiguous().view(torch.float32)[:, None]
+        y = _grouped_ref(x, w, offs, False)
+        if not unit_weights:
+            y = y * recs[:, 2].contiguous().view(torch.float32)[:, None]
         for r, o in enumerate(outs):
             mine = (recs[:, 0] == r) & (recs[:, 1] >= 0)
             o[recs[mine, 1].long()] = y[mine].to(o.dtype)
         return
     if x.dtype == torch.float32 or (comm is None and not w_blocked and not _tma_ok(x, w)):
-        _simt_grouped(x, w, offs, None, recs, bases, ld_out)
+        _simt_grouped(x, w, offs, None, recs, bases, ld_out, unit_weights)
         return
     _check_x(x)
     assert recs.dtype == torch.int32 and recs.is_contiguous() and recs.shape[1] == 4 and bases.dtype == torch.int64
@@ -491,7 +507,7 @@ def grouped_combine(x: torch.Tensor, w: torch.Tensor, offs: Optional[torch.Tenso
         bn = max(bn, 128)
     sk = want_streamk(EPI_COMBINE, F, G, T, bn, num_sms(x.device)) if streamk is None else streamk
     _launch(w, x, None, None, offs, recs, bases, G, T, F, K, EPI_COMBINE, bn, 1, ld_out, False, comm, streamk=sk,
-            pair=pair, w_blocked=w_blocked)
+            pair=pair, w_blocked=w_blocked, unit_weights=unit_weights)
 
 
 def swiglu_linear(x: torch.Tensor, w13: torch.Tensor, out: Optional[torch.Tensor] = None, bn: int = 0,

@@ -1,5 +1,8 @@
 """Linear recurrences with a matrix state per head (``csrc/kernels/recurrent.cu``, ``recurrent_chunk.cu``): gated linear
-attention, the gated delta rule and RWKV-style time mixing, with one decay per head and key channel. CUDA tensors run the kernels, CPU tensors the PyTorch restatements.
+attention, the gated delta rule and RWKV-style time mixing, with one decay per head and key channel; lightning attention, with a
+constant decay per head; the matrix memory of xLSTM, with a decay per head and token and a normaliser beside the state. And the
+real-gated diagonal recurrence of Griffin's block (``diag_recurrent.cu``). CUDA tensors run the kernels, CPU tensors the PyTorch
+restatements.
 
 A step's rows fall into segments (consecutive rows of one sequence). One-token segments (decoding) take one launch from
 the projections to the gated, normalised output; longer ones (prompts and portions of prompts) are convolved and then run
@@ -72,13 +75,17 @@ def decode_segments(positions: torch.Tensor, rows: torch.Tensor, kv_slots: torch
 @dataclass
 class RecurrentState:
     """Per-layer state pool: S fp32 [slots, heads, dim, vdim]; with a short convolution the ring of its last inputs [slots,
-    taps, channels]; with a token shift the last input row, fp32 [slots, width]. A slot needs no clearing: a segment at position 0 starts from zero."""
+    taps, channels]; with a token shift the last input row, fp32 [slots, width]; of a matrix memory the normaliser ``n`` fp32 [slots,
+    heads, dim] and the running maximum ``m`` fp32 [slots, 2, heads], kept at the parity of its position. A diagonal recurrence has S
+    [slots, width]. A slot needs no clearing: a segment at position 0 starts from zero."""
     S: torch.Tensor
     ring: Optional[torch.Tensor] = None
     last: Optional[torch.Tensor] = None
+    n: Optional[torch.Tensor] = None
+    m: Optional[torch.Tensor] = None
 
     def tensors(self):
-        return [t for t in (self.S, self.ring, self.last) if t is not None]
+        return [t for t in (self.S, self.ring, self.last, self.n, self.m) if t is not None]
 
 
 @dataclass
@@ -87,13 +94,16 @@ class Recurrence:
     log a = -exp(a_log) softplus(z + z_bias); otherwise the plain write with log a = log sigmoid(z + z_bias) / tau or,
     ``exp_decay``, log a = -exp(z + z_bias). ``bonus`` [heads, dim]: the read-out precedes decay and write, and the token's own
     write enters it weighed by the bonus. ``norm_w``: [vdim], or [heads * vdim] with a weight per head; ``qscale``: factor of q
-    (None: dim ** -0.5); ``shift_width``: width of the token shift whose last row belongs to the state (0: none)."""
+    (None: dim ** -0.5); ``shift_width``: width of the token shift whose last row belongs to the state (0: none).
+    ``head_decay`` [heads]: constant logs of the decays (no z). ``gate_bias`` [2 heads]: matrix memory; z is then the logits
+    [T, 2 heads] of the input and the forget gates, soft-capped at ``gate_cap`` after the bias. ``joint_norm``: all heads' read-outs
+    are normed together (norm_w [heads * vdim])."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     delta: bool
-    z_bias: torch.Tensor
+    z_bias: Optional[torch.Tensor]
     norm_w: torch.Tensor
     eps: float
     a_log: Optional[torch.Tensor] = None
@@ -104,10 +114,14 @@ class Recurrence:
     bonus: Optional[torch.Tensor] = None
     qscale: Optional[float] = None
     shift_width: int = 0
+    head_decay: Optional[torch.Tensor] = None
+    gate_bias: Optional[torch.Tensor] = None
+    gate_cap: float = 1.0
+    joint_norm: bool = False
 
     @property
     def decay_kind(self) -> int:
-        return 2 if self.exp_decay else int(self.delta)
+        return 4 if self.gate_bias is not None else 3 if self.head_decay is not None else 2 if self.exp_decay else int(self.delta)
 
     @property
     def norm_ld(self) -> int:
@@ -129,11 +143,21 @@ class Recurrence:
         S = torch.zeros(slots, self.heads, self.dim, self.vdim, dtype=torch.float32, device=device)
         ring = torch.zeros(slots, self.taps, self.channels, dtype=dtype, device=device) if self.taps else None
         last = torch.zeros(slots, self.shift_width, dtype=torch.float32, device=device) if self.shift_width else None
-        return RecurrentState(S, ring, last)
+        n = m = None
+        if self.gate_bias is not None:
+            n = torch.zeros(slots, self.heads, self.dim, dtype=torch.float32, device=device)
+            m = torch.zeros(slots, 2, self.heads, dtype=torch.float32, device=device)
+        return RecurrentState(S, ring, last, n, m)
 
 
 def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) -> _lib.DmoeRecur:
     d = _lib.DmoeRecur()
+    if r.gate_bias is not None:
+        assert z is None or (z.stride(1) == 1 and z.dtype == torch.float32 and z.shape[1] == 2 * r.heads)
+        d.gates, d.ldgates, d.gate_bias, d.gate_cap = _lib.ptr(z), 0 if z is None else z.stride(0), r.gate_bias.data_ptr(), r.gate_cap
+        d.norm_state, d.max_state = state.n.data_ptr(), state.m.data_ptr()
+        z = None
+    d.head_decay = _lib.ptr(r.head_decay)
     for name, t in (("q", q), ("k", k), ("v", v), ("gate", gate), ("beta", beta), ("z", z)):
         assert t is None or (t.stride(1) == 1 and t.dtype == (torch.float32 if name == "z" else q.dtype))
         setattr(d, name, _lib.ptr(t))
@@ -150,18 +174,19 @@ def _descriptor(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState) ->
     return d
 
 
-def _gate_norm(r: Recurrence, table, n, max_tokens, raw, gate, out) -> None:
+def _gate_norm(r: Recurrence, table, n, max_tokens, raw, gate, out, scale=None) -> None:
     v, ll, i = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+    heads, vdim, norm_ld = (1, r.heads * r.vdim, 0) if r.joint_norm else (r.heads, r.vdim, r.norm_ld)
     _lib.check(_lib.lib().dmoe_gate_norm(
         i(int(out.dtype == torch.float32)), v(_lib.ptr(table)), i(n), i(max_tokens), v(raw.data_ptr()), ll(raw.stride(0)),
-        v(gate.data_ptr()), ll(gate.stride(0)), v(r.norm_w.data_ptr()), i(r.norm_ld), ctypes.c_float(r.eps), i(int(r.sigmoid_gate)),
-        v(out.data_ptr()), ll(out.stride(0)), i(r.heads), i(r.vdim), v(_lib.stream_ptr())), "dmoe_gate_norm")
+        v(gate.data_ptr()), ll(gate.stride(0)), v(r.norm_w.data_ptr()), i(norm_ld), ctypes.c_float(r.eps), i(int(r.sigmoid_gate)),
+        v(out.data_ptr()), ll(out.stride(0)), i(heads), i(vdim), v(_lib.ptr(scale)), v(_lib.stream_ptr())), "dmoe_gate_norm")
 
 
 def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, segs: SegmentTables) -> torch.Tensor:
     """q, k [T, kv_heads dim], v, gate [T, heads vdim], beta [T, heads] (delta) straight from the projections (columns of
-    one wider matrix are fine), z fp32 [T, heads dim]. Returns [T, heads vdim]: the recurrence's read-outs, normalised per
-    head, weighed and gated. Convolution inputs and states of the segments' slots are updated."""
+    one wider matrix are fine), z fp32 [T, heads dim] (constant decays: None; matrix memory: gate logits [T, 2 heads]). Returns [T,
+    heads vdim]: the recurrence's read-outs, normalised per head (or together), weighed and gated. Convolution inputs and states of the segments' slots are updated."""
     if not q.is_cuda:
         return _reference(r, q, k, v, gate, beta, z, state, segs)
     T = q.shape[0]
@@ -169,7 +194,16 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
     out = torch.empty(T, r.heads * r.vdim, dtype=q.dtype, device=q.device)
     vt = lib.dmoe_recur_value_tile(r.dim, r.vdim)
     assert vt > 0, "head too large for the recurrence kernels"
-    raw = None
+    raw = scale = None
+    memory = r.gate_bias is not None
+
+    def raw_rows(d):
+        """Read-outs go to fp32 rows, a matrix memory's with the factor of every row and head beside them."""
+        nonlocal raw, scale
+        if raw is None:
+            raw = torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=q.device)
+            scale = torch.empty(T, r.heads, dtype=torch.float32, device=q.device) if memory else None
+        d.raw, d.ldraw, d.scale = raw.data_ptr(), raw.stride(0), _lib.ptr(scale)
     if segs.n_single:
         d = _descriptor(r, q, k, v, gate, beta, z, state)
         if r.taps:
@@ -180,17 +214,15 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
         # few heads in flight: deal the value columns to more CTAs, at the price of a second (norm) launch
         while svt >= 32 and svt % 8 == 0 and segs.n_single * r.heads * ((r.vdim + svt - 1) // svt) < num_sms(q.device):
             svt //= 2
-        if svt >= r.vdim:
+        fused = svt >= r.vdim and not r.joint_norm
+        if fused:
             d.out, d.ldo = out.data_ptr(), out.stride(0)
         else:
-            raw = torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=q.device)
-            d.raw, d.ldraw = raw.data_ptr(), raw.stride(0)
+            raw_rows(d)
         _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(svt), st), "dmoe_recur_step")
-        if svt < r.vdim:
-            _gate_norm(r, segs.singles, segs.n_single, 1, raw, gate, out)
+        if not fused:
+            _gate_norm(r, segs.singles, segs.n_single, 1, raw, gate, out, scale)
     if segs.n_multi:
-        if raw is None:
-            raw = torch.empty(T, r.heads * r.vdim, dtype=torch.float32, device=q.device)
         qs, vs = r.kv_heads * r.dim, r.heads * r.vdim
         if r.taps:
             act = torch.empty(T, r.channels, dtype=q.dtype, device=q.device)
@@ -203,7 +235,11 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
             q, k, v = act[:, :qs], act[:, qs:2 * qs], act[:, 2 * qs:]
         d = _descriptor(r, q, k, v, gate, beta, z, state)
         d.segs, d.n_segs = segs.multi.data_ptr(), segs.n_multi
-        d.raw, d.ldraw = raw.data_ptr(), raw.stride(0)
+        raw_rows(d)
+        if memory:
+            steps = torch.empty(3, T, r.heads, dtype=torch.float32, device=q.device)
+            d.keep, d.put, d.run_max = (t.data_ptr() for t in steps)
+            _lib.check(lib.dmoe_memory_gates(ctypes.byref(d), st), "dmoe_memory_gates")
         if q.dtype == torch.bfloat16 and lib.dmoe_recur_chunk_ok(r.dim, r.vdim):
             per_head = lib.dmoe_recur_chunk_bytes(r.dim, r.vdim, int(r.delta), segs.n_chunks)
             ws = torch.empty(max(per_head, min(per_head * r.heads, WORKSPACE)), dtype=torch.uint8, device=q.device)
@@ -212,14 +248,17 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
                                              ctypes.c_longlong(ws.numel()), st), "dmoe_recur_chunks")
         else:
             _lib.check(lib.dmoe_recur_step(ctypes.byref(d), ctypes.c_int(vt), st), "dmoe_recur_step")
-        _gate_norm(r, segs.chunks, segs.n_chunks, CHUNK, raw, gate, out)
+        _gate_norm(r, segs.chunks, segs.n_chunks, CHUNK, raw, gate, out, scale)
     return out
 
 
 def _reference(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, segs: SegmentTables) -> torch.Tensor:
     T, H, G, D, V = q.shape[0], r.heads, r.kv_heads, r.dim, r.vdim
-    zb = z.float() + r.z_bias
-    logd = -torch.exp(zb).view(T, H, D) if r.exp_decay else (-torch.exp(r.a_log)[:, None] * torch.nn.functional.softplus(zb).view(T, H, D)) if r.delta else \
+    zb = None if z is None or r.gate_bias is not None else z.float() + r.z_bias
+    if r.gate_bias is not None:
+        i, f = (r.gate_cap * torch.tanh((z + r.gate_bias) / r.gate_cap)).split(H, 1)
+        f = torch.nn.functional.logsigmoid(f)
+    logd = None if r.gate_bias is not None else r.head_decay[:, None].expand(T, H, D) if zb is None else -torch.exp(zb).view(T, H, D) if r.exp_decay else (-torch.exp(r.a_log)[:, None] * torch.nn.functional.softplus(zb).view(T, H, D)) if r.delta else \
         torch.nn.functional.logsigmoid(zb).view(T, H, D) / r.tau
     out = torch.zeros(T, H * V, dtype=q.dtype)
     for a, n, slot, pos0 in segs.table():
@@ -227,8 +266,70 @@ def _reference(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentState, seg
         if r.taps:
             x = reference.conv_segment(x, r.conv_w, state.ring[slot], pos0)
         qq, kk = (x[:, j * G * D:(j + 1) * G * D].view(n, G, D).repeat_interleave(H // G, 1) for j in (0, 1))
-        o = reference.recur_segment(qq, kk, x[:, 2 * G * D:].view(n, H, V), None if beta is None else beta[a:a + n],
-                                    logd[a:a + n], state.S[slot], pos0, r.delta, r.q_factor, r.bonus)
-        o = reference.gate_norm(o, gate[a:a + n].view(n, H, V), r.norm_w.view(-1, V), r.eps, r.sigmoid_gate)
+        if r.gate_bias is not None:
+            o = reference.memory_segment(qq, kk, x[:, 2 * G * D:].view(n, H, V), i[a:a + n], f[a:a + n], state.S[slot], state.n[slot],
+                                         state.m[slot], pos0, r.q_factor)
+        else:
+            o = reference.recur_segment(qq, kk, x[:, 2 * G * D:].view(n, H, V), None if beta is None else beta[a:a + n],
+                                        logd[a:a + n], state.S[slot], pos0, r.delta, r.q_factor, r.bonus)
+        if r.joint_norm:
+            o = reference.gate_norm(o.reshape(n, H * V), gate[a:a + n], r.norm_w, r.eps, r.sigmoid_gate)
+        else:
+            o = reference.gate_norm(o, gate[a:a + n].view(n, H, V), r.norm_w.view(-1, V), r.eps, r.sigmoid_gate)
         out[a:a + n] = o.reshape(n, H * V).to(q.dtype)
+    return out
+
+
+# ---- real-gated diagonal recurrence ------------------------------------------------------------------------------------
+@dataclass
+class GatedUnit:
+    """Constants of Griffin's block (fp32): convolution ``conv_w`` [taps, width], ``conv_b``, bias ``in_b`` of its input; ``gate_b`` [blocks,
+    2, padded] biases of the two gates (padded = width / blocks rounded up to a multiple of 8); ``decay`` [width] log decay where the
+    recurrence gate is open; ``y_b`` bias of the gelu branch."""
+    width: int
+    blocks: int
+    conv_w: torch.Tensor
+    conv_b: torch.Tensor
+    in_b: torch.Tensor
+    gate_b: torch.Tensor
+    decay: torch.Tensor
+    y_b: torch.Tensor
+
+    @property
+    def padded(self) -> int:
+        return self.gate_b.shape[2]
+
+    def new_state(self, slots: int, dtype, device) -> RecurrentState:
+        ring = torch.zeros(slots, self.conv_w.shape[0], self.width, dtype=dtype, device=device)
+        return RecurrentState(torch.zeros(slots, self.width, dtype=torch.float32, device=device), ring)
+
+
+def unit_recurrence(g: GatedUnit, u: torch.Tensor, gates: torch.Tensor, y: torch.Tensor, state: RecurrentState,
+                    segs: SegmentTables) -> torch.Tensor:
+    """u [blocks, T, padded], gate logits fp32 [blocks, T, 2, padded] without their bias, y [T, width] (columns of a wider matrix are
+    fine) before bias and gelu -> [T, width]: S gelu(y), with log a = decay sigmoid(r), S <- a S + sqrt(1 - a^2) sigmoid(i) u per
+    channel. ``state.S`` of the segments' slots is updated."""
+    T, C = y.shape
+    if not u.is_cuda:
+        n = C // g.blocks
+        flat = lambda t: t[..., :n].transpose(0, 1).reshape(T, C).float()
+        r, i = (torch.sigmoid(flat(gates[:, :, j] + g.gate_b[:, None, j])) for j in (0, 1))
+        out, uu = torch.zeros(T, C, dtype=y.dtype), flat(u)
+        gel = torch.nn.functional.gelu(y.float() + g.y_b, approximate="tanh")
+        for a, k, slot, pos0 in segs.table():
+            S = reference.diagonal_segment(uu[a:a + k], r[a:a + k], i[a:a + k], g.decay, state.S[slot], pos0)
+            out[a:a + k] = (S * gel[a:a + k]).to(y.dtype)
+        return out
+    out = torch.empty(T, C, dtype=y.dtype, device=y.device)
+    assert u.is_contiguous() and gates.is_contiguous() and gates.dtype == torch.float32 and y.stride(1) == 1 and u.dtype == y.dtype
+    assert u.shape == (g.blocks, T, g.padded) and gates.shape == (g.blocks, T, 2, g.padded) and state.S.shape[1] == C
+    d = _lib.DmoeUnit()
+    d.u, d.gates, d.gate_bias, d.decay, d.y, d.y_bias = (t.data_ptr() for t in (u, gates, g.gate_b, g.decay, y, g.y_b))
+    d.state, d.out, d.multi = state.S.data_ptr(), out.data_ptr(), _lib.ptr(segs.multi)
+    d.singles = _lib.ptr(segs.singles) if segs.n_single else 0
+    d.positions, d.rows, d.kv_slots = _lib.ptr(segs.positions), _lib.ptr(segs.rows), _lib.ptr(segs.kv_slots)
+    d.ldy, d.ldo, d.block_rows = y.stride(0), out.stride(0), T
+    d.n_single, d.n_multi, d.n_slots, d.width, d.blocks, d.padded = segs.n_single, segs.n_multi, state.S.shape[0], C, g.blocks, g.padded
+    _lib.check(_lib.lib().dmoe_unit_recurrence(ctypes.c_int(int(y.dtype == torch.float32)), ctypes.byref(d),
+                                               ctypes.c_void_p(_lib.stream_ptr())), "dmoe_unit_recurrence")
     return out

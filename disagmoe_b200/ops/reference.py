@@ -59,10 +59,12 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slots: Optional[t
 def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                     bt_row: Optional[torch.Tensor], ctx_len: torch.Tensor, n_q: int, n_kv: int, hd: int,
                     scale: Optional[float] = None, window: Optional[int] = None, softcap: Optional[float] = None,
-                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None, q_temp=None,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Token t attends to the first ctx_len[t] cached tokens of block-table row bt_row[t] (default t), or to the last
     ``window`` of them, or to those in the same ``chunk`` of positions as the last one; ``softcap``: scores become cap * tanh(score / cap); ``sink`` [n_q]: the softmax denominator has
-    exp(sink) in addition."""
+    exp(sink) in addition; ``q_temp`` (coef, every): scores times the query temperature of position ctx_len - 1; ``gate`` [T, n_q]:
+    every head's output times sigmoid(gate)."""
     T = q.shape[0]
     block_size = kcache.shape[1]
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
@@ -85,6 +87,8 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
             k, v = k[-n:], v[-n:]
         qt = q[t].float().view(n_kv, gq, hd)
         s = torch.einsum("kgd,lkd->kgl", qt, k) * scale
+        if q_temp is not None:
+            s = s * (1.0 + q_temp.coef * math.log(L // q_temp.every + 1))
         if softcap:
             s = softcap * torch.tanh(s / softcap)
         if sink is not None:
@@ -92,6 +96,8 @@ def paged_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         p = torch.softmax(s, dim=-1)[..., :k.shape[0]]
         o = torch.einsum("kgl,lkd->kgd", p, v)
         out[t] = o.reshape(-1)
+    if gate is not None:
+        out = (out.view(T, n_q, vd) * torch.sigmoid(gate.float())[..., None]).reshape(T, -1)
     return out.to(q.dtype)
 
 
@@ -143,9 +149,12 @@ def sort_by_expert(topk_ids: torch.Tensor) -> torch.Tensor:
     return pos.int()
 
 
-def swiglu(h: torch.Tensor, act: str = "silu") -> torch.Tensor:
+def swiglu(h: torch.Tensor, act: str = "silu", limit: float = 0.0) -> torch.Tensor:
     I = h.shape[-1] // 2
     g = h[..., :I].float()
+    if act == "clamped":
+        g = g.clamp(max=limit)
+        return g * torch.sigmoid(1.702 * g) * (h[..., I:].float().clamp(-limit, limit) + 1.0)
     g = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
     return g * h[..., I:].float()
 
@@ -200,19 +209,25 @@ def resid_norm(resid, y, post, pre, eps, dtype, out_scale=1.0, rows=None):
     return None if pre is None else (_rms_scale(x, eps) * pre * out_scale).to(dtype)
 
 
-def sum_norm(resid, y, parts, w, eps, dtype, centred, rows=None, mult=1.0):
+def sum_norm(resid, y, parts, w, eps, dtype, centred, rows=None, mult=1.0, bias=None, gate=None, sides=None):
     """resid += mult * (y + parts.sum(1)) (either may be None; ``rows``: only these rows are returned, resid untouched); returns the
-    RMS norm of resid times w, or with ``centred`` its layer norm (mean taken off) times w."""
+    RMS norm of resid times w, or with ``centred`` its layer norm (mean taken off) times w, plus ``bias``. ``gate``: what is added is
+    multiplied by sigmoid(gate.z + gate.bias) first. ``sides``: y is the scaled sum of two rows, each normed with its weight."""
     x = resid if rows is None else resid[rows.long()]
+    pick = lambda a: a if rows is None else a[rows.long()]
+    g = mult if gate is None else mult * torch.sigmoid(pick(gate.z).float() + gate.bias)
+    if sides is not None:
+        y = sides.scale * sum(_rms_scale(sides.rows[i].float(), eps) * sides.weights[i] for i in range(2))
     for a in (y, parts):
         if a is not None:
-            a = a if rows is None else a[rows.long()]
-            x = x + mult * (a.float() if a.dim() == 2 else a.float().sum(1))
+            a = pick(a)
+            x = x + g * (a.float() if a.dim() == 2 else a.float().sum(1))
     if rows is None:
         resid.copy_(x)
     if centred:
         x = x - x.mean(-1, keepdim=True)
-    return (_rms_scale(x, eps) * w).to(dtype)
+    h = _rms_scale(x, eps) * w
+    return (h if bias is None else h + bias).to(dtype)
 
 
 def _turn(x, table, positions, interleaved):
@@ -229,9 +244,10 @@ def _turn(x, table, positions, interleaved):
 
 
 def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table, qw, kw, eps, interleaved=False,
-                 v_first=None, v_lambda=0.0, tied=False) -> None:
+                 v_first=None, v_lambda=0.0, tied=False, v_norm=0) -> None:
     """Per-head norm (where weights are given) + partial rotation of q (in place) and k, K / V append at slots >= 0; with
-    ``v_first`` [T, n_kv, >= dv] the values appended are (1 - v_lambda) v + v_lambda v_first, ``tied`` those of the raw keys."""
+    ``v_first`` [T, n_kv, >= dv] the values appended are (1 - v_lambda) v + v_lambda v_first, ``tied`` those of the raw keys,
+    ``v_norm`` > 0: divided by their root mean square over that many dimensions."""
     T = qkv.shape[0]
 
     def turn(x, w):
@@ -248,6 +264,8 @@ def qk_norm_rope(qkv, positions, slots, kcache, vcache, n_q, n_kv, dk, dv, table
             qkv[ok][:, qs + ks:qs + ks + n_kv * dv].reshape(-1, n_kv, dv)
         if v_first is not None:
             v = ((1.0 - v_lambda) * v.float() + v_lambda * v_first[ok][..., :dv].float()).to(v.dtype)
+        if v_norm:
+            v = (v.float() / torch.sqrt(v.float().pow(2).sum(-1, keepdim=True) / v_norm + eps)).to(v.dtype)
         vcache.view(-1, n_kv, dv)[slots[ok]] = v
     qkv[:, :qs] = q.reshape(T, qs).clone()
 
@@ -288,6 +306,56 @@ def conv_segment(x: torch.Tensor, w: torch.Tensor, ring: Optional[torch.Tensor],
     for j in range(max(0, n - taps + 1), n):
         ring[(pos0 + j) % taps] = x[j]
     return torch.nn.functional.silu(acc).to(x.dtype)
+
+
+def seq_conv(x, w, ring, segs, in_bias, out_bias, residual):
+    """See :func:`disagmoe_b200.ops.functional.seq_conv`: fp32 [T, C]."""
+    taps, out = w.shape[0], torch.zeros(x.shape, dtype=torch.float32)
+    add = 0.0 if in_bias is None else in_bias
+    for a, n, slot, pos0 in segs.table():
+        hist = [ring[slot, (pos0 - j) % taps].float() + add if pos0 - j >= 0 else torch.zeros(x.shape[1]) for j in range(taps - 1, 0, -1)]
+        seg = x[a:a + n].float() + add
+        full = torch.cat([torch.stack(hist), seg]) if hist else seg
+        acc = sum(full[j:j + n] * w[j] for j in range(taps))
+        if out_bias is not None:
+            acc = acc + out_bias
+        out[a:a + n] = seg + acc if residual else acc
+        for j in range(max(0, n - taps + 1), n):
+            ring[slot, (pos0 + j) % taps] = x[a + j]
+    return out
+
+
+def diagonal_segment(u, r, i, decay, state, pos0):
+    """u, r, i [n, C] fp32, decay [C] (log decay of an open gate); ``state`` [C] is read (zero where pos0 = 0) and updated."""
+    S = state.clone() if pos0 > 0 else torch.zeros_like(state)
+    out = []
+    for t in range(u.shape[0]):
+        log_a = decay * r[t]
+        S = torch.exp(log_a) * S + torch.sqrt(-torch.expm1(2.0 * log_a)) * (i[t] * u[t])
+        out.append(S)
+    state.copy_(S)
+    return torch.stack(out)
+
+
+def memory_segment(q, k, v, i, f, S, n, m, pos0, qscale):
+    """q, k [T, H, D], v [T, H, V], i, f [T, H] logs of the gates; the state S [H, D, V], n [H, D] and the running maxima
+    m [2, H] (at the position's parity) are read (zero where pos0 = 0) and updated. Returns fp32 read-outs [T, H, V]."""
+    q, k, v = q.float() * qscale, k.float(), v.float()
+    zero = pos0 == 0
+    A, b, top = (torch.zeros_like(t) if zero else t.clone() for t in (S, n, m[(pos0 - 1) % 2]))
+    out = []
+    for t in range(q.shape[0]):
+        new = torch.maximum(f[t] + top, i[t])
+        keep, put = torch.exp(f[t] + top - new), torch.exp(i[t] - new)
+        A = keep[:, None, None] * A + put[:, None, None] * k[t][..., None] * v[t][:, None, :]
+        b = keep[:, None] * b + put[:, None] * k[t]
+        top = new
+        size = torch.maximum((b * q[t]).sum(-1).abs(), torch.exp(-top)) + 1e-6
+        out.append(torch.einsum("hdv,hd->hv", A, q[t]) / size[:, None])
+    S.copy_(A)
+    n.copy_(b)
+    m[(pos0 + q.shape[0] - 1) % 2] = top
+    return torch.stack(out)
 
 
 def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, segs) -> torch.Tensor:
