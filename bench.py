@@ -146,7 +146,7 @@ def main():
                          "continuous batching; prints output tokens/s with p50 / p99 time per output token per rate")
     ap.add_argument("--rates", default="2,8,16,32")
     ap.add_argument("--duration", type=float, default=60.0)
-    ap.add_argument("--layer-list", nargs="?", const="rurunex", choices=["rurunex", "supinex", "vufinex"],
+    ap.add_argument("--layer-list", nargs="?", const="rurunex", choices=["rurunex", "supinex", "vufinex", "panarax"],
                     help="1 GPU: prefill and decode throughput of layer-list decoders of this design beside the closest "
                          "decoder of equal size (benchmark/layer_list.py) instead of the headline workload")
     ap.add_argument("--layer-list-sizes", default="", help="comma-separated widths for --layer-list")

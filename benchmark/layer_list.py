@@ -1,6 +1,6 @@
 """Prefill and decode throughput of layer-list decoders beside the closest decoder of the package at equal size.
 
-    python bench.py --layer-list [rurunex | supinex | vufinex] [--steps K --warmup W]
+    python bench.py --layer-list [rurunex | supinex | vufinex | panarax] [--steps K --warmup W]
 
 Both run through the same engine classes with random weights.
   rurunex  repeats (gated linear attention, channel-wise delta rule, windowed attention), every layer with a gated
@@ -10,19 +10,23 @@ Both run through the same engine classes with random weights.
            decoder with the same width, heads, experts and number of layers
   vufinex  repeats (RWKV-style time mixing, gated latent attention, chunked attention), experts in every layer; beside the MoE
            decoder with the same width, heads, experts and number of layers
+  panarax  repeats (attention beside a matrix memory with a dense feed-forward, gated diagonal recurrence, lightning attention, both
+           with experts); beside the MoE decoder with the same width, heads, experts and numbers of dense and expert layers
 Prints one JSON line per (size, phase, model): tokens/s from device-timed steps (CUDA events, L2 flushed between steps), and
 one per (size, phase) with the device time per kernel.
 """
 from __future__ import annotations
 
 import json
+import math
 import statistics
 from typing import Dict, List
 
 import torch
 
-from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, LatentAttentionSpec,
-                                  LayerListConfig, LayerSpec, ModelConfig, RotarySpec, RoutedSpec, WkvSpec)
+from disagmoe_b200.config import (AttentionSpec, CacheConfig, ChannelDeltaSpec, GatedLinearSpec, GatedUnitSpec, HeadDecaySpec,
+                                  LatentAttentionSpec, LayerListConfig, LayerSpec, MatrixMemorySpec, ModelConfig, QueryTemperature,
+                                  RotarySpec, RoutedSpec, SideBySideSpec, WkvSpec)
 from disagmoe_b200.frontend.colocated import ColocatedEngine
 from disagmoe_b200.ops import _lib, gemm
 
@@ -69,6 +73,17 @@ def prenorm_config(size: str, chunk: int = 1024, max_seq_len: int = 8192) -> Lay
               AttentionSpec(H, G, D, D, D ** -0.5, RotarySpec(D // 2, 5e5), qk_norm=False, chunk=chunk, tied_values=True))
     return LayerListConfig.make(W, VOCAB, [LayerSpec(mixers[i % 3], routed=moe) for i in range(n)], max_seq_len=max_seq_len,
                                 block="prenorm", embed_scale=32.0, residual_mult=0.5, name="vufinex-" + size)
+
+
+def gated_config(size: str, max_seq_len: int = 8192) -> LayerListConfig:
+    W, H, G, D, ff, n, _, E, K = MOE_SIZES[size]
+    moe = RoutedSpec(E, K, ff, act="clamped", scoring="sigmoid", limit=7.0, weigh_input=True)
+    both = SideBySideSpec(AttentionSpec(H, G, D, D, D ** -0.5, qk_norm=False, value_norm=True, gate=True, q_temp=QueryTemperature(0.1, 1024)),
+                          MatrixMemorySpec(H // 2, D, D, 15.0))
+    decays = HeadDecaySpec(H, D, D, tuple(math.exp(-2.0 ** (-8.0 * (i + 1) / H)) for i in range(H)))
+    layers = [LayerSpec(both, 4 * ff), LayerSpec(GatedUnitSpec(H * D, H, 4), routed=moe), LayerSpec(decays, routed=moe)]
+    return LayerListConfig.make(W, VOCAB, layers * (n // 3), max_seq_len=max_seq_len, block="prenorm", layer_norm=True, residual_gate=True,
+                                input_conv=4, positions=max_seq_len, tied_head=True, name="panarax-" + size)
 
 
 def moe_config(size: str, max_seq_len: int = 8192, dense_layers: int = 1) -> ModelConfig:
@@ -144,7 +159,8 @@ def main(args) -> int:
         for phase, n, length in (("prefill", 1, 4096), ("prefill", 4, 2048), ("decode", 16, 2048), ("decode", 256, 1024)):
             for cfg in {"rurunex": lambda: (hybrid_config(size), dense_config(size)),
                         "supinex": lambda: (parallel_config(size), moe_config(size)),
-                        "vufinex": lambda: (prenorm_config(size), moe_config(size, dense_layers=0))}[args.layer_list]():
+                        "vufinex": lambda: (prenorm_config(size), moe_config(size, dense_layers=0)),
+                        "panarax": lambda: (gated_config(size), moe_config(size, dense_layers=2))}[args.layer_list]():
                 B = n if phase == "decode" else 8
                 eng = make_engine(cfg, B, n * length if phase == "prefill" else B, length if phase == "decode" else 16, 8)
                 ex = eng.executor

@@ -1,7 +1,8 @@
-"""Recurrent layers alone: prompts (chunked kernels) and decode steps; gated linear attention, the channel-wise delta rule and
-RWKV-style time mixing (wkv), the last with its token shift on its own.
+"""Recurrent layers alone: prompts (chunked kernels) and decode steps; gated linear attention, the channel-wise delta rule,
+RWKV-style time mixing (wkv, with its token shift on its own), lightning attention, the matrix memory, and Griffin's block (unit: its
+convolution and its recurrence).
 
-    python -m benchmark.ops.recurrence [--kinds gla,delta,wkv] [--heads 16] [--dim 128] [--tokens 4096] [--batch 256]
+    python -m benchmark.ops.recurrence [--kinds gla,delta,wkv,lightning,memory,unit] [--heads 16] [--dim 128] [--tokens 4096] [--batch 256]
 
 Device time (CUDA events, L2 flushed in between) beside the bytes the operation has to move: projections in, output out and,
 for a decode step, every state read and written once.
@@ -17,7 +18,8 @@ import torch
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))))
 
 from disagmoe_b200.ops import functional as F
-from disagmoe_b200.ops.recurrent import Recurrence, build_segments, decode_segments, recurrent_attention
+from disagmoe_b200.ops.recurrent import (GatedUnit, Recurrence, build_segments, decode_segments, recurrent_attention,
+                                         unit_recurrence)
 
 
 def layer(kind, H, D, V, dev="cuda"):
@@ -27,6 +29,15 @@ def layer(kind, H, D, V, dev="cuda"):
     if kind == "wkv":
         return Recurrence(H, H, D, V, False, r(H * D) - 3.0, 1 + 0.1 * r(H * D), 1e-6, exp_decay=True, bonus=0.5 * r(H, D), qscale=1.0,
                           shift_width=H * D)
+    if kind == "lightning":
+        return Recurrence(H, H, D, V, False, None, 1 + 0.1 * r(H * V), 1e-6, sigmoid_gate=True, qscale=1.0, joint_norm=True,
+                          head_decay=-torch.exp2(-8.0 * (torch.arange(H, device=dev) + 1) / H))
+    if kind == "memory":
+        return Recurrence(H, H, D, V, False, None, 1 + 0.1 * r(H * V), 1e-6, sigmoid_gate=True, gate_cap=15.0,
+                          gate_bias=torch.cat([r(H), r(H) + 4.0]))
+    if kind == "unit":
+        C = H * D
+        return GatedUnit(C, H, 0.5 * r(4, C), r(C), r(C), r(H, 2, D), -8.0 * torch.nn.functional.softplus(r(C) - 4.0), r(C))
     return Recurrence(H, H, D, V, True, 0.5 * r(H * D) - 4.0, 1 + 0.1 * r(V), 1e-6, a_log=0.3 * r(H),
                       conv_w=0.5 * r(2 * H * D + H * V, 4), sigmoid_gate=True)
 
@@ -40,7 +51,7 @@ def main():
     p.add_argument("--batch", type=int, default=256, help="decoding sequences")
     p.add_argument("--iters", type=int, default=10)
     p.add_argument("--only", default="", help="prompt | decode")
-    p.add_argument("--kinds", default="gla,delta,wkv")
+    p.add_argument("--kinds", default="gla,delta,wkv,lightning,memory,unit")
     a = p.parse_args()
     H, D = a.heads, a.dim
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
@@ -63,8 +74,17 @@ def main():
             else:
                 i = torch.arange(T, device="cuda")
                 segs = decode_segments(torch.full((T,), 100, dtype=torch.int32, device="cuda"), i.int(), i)
-            cases = [(kind, T * H * D * (2 * 5 + 4) + (2 * state.S.numel() * 4 if phase == "decode" else 0),
-                      lambda: recurrent_attention(r, q, k, v, gate, beta if kind == "delta" else None, z, state, segs))]
+            if kind == "memory":
+                z = z[:, :2 * H].contiguous()
+            if kind == "unit":
+                u, zz = torch.randn(H, T, D, device="cuda").bfloat16(), torch.randn(H, T, 2, D, device="cuda")
+            cases = [] if kind == "unit" else [(kind, T * H * D * (2 * 5 + (0 if kind in ("lightning", "memory") else 4)) + (2 * state.S.numel() * 4 if phase == "decode" else 0),
+                      lambda: recurrent_attention(r, q, k, v, gate, beta if kind == "delta" else None,
+                                                  None if kind == "lightning" else z, state, segs))]
+            if kind == "unit":
+                cases = [("convolution", T * H * D * 2 * (2 if phase == "prompt" else 6),
+                          lambda: F.seq_conv(q, r.conv_w, state.ring, segs, r.in_b, r.conv_b, blocks=H)),
+                         ("unit", T * H * D * (2 * 3 + 8 + (8 if phase == "decode" else 0)), lambda: unit_recurrence(r, u, zz, k, state, segs))]
             if kind == "wkv":
                 W = H * D
                 mu, w, resid = torch.rand(5, W, device="cuda"), torch.ones(W, device="cuda"), torch.randn(T, W, device="cuda")

@@ -618,30 +618,30 @@ def _conv_descriptor(w, ring, segs, in_bias=None, out_bias=None, residual=True, 
 
 
 def seq_conv(x: torch.Tensor, w: torch.Tensor, ring: torch.Tensor, segs, in_bias: Optional[torch.Tensor] = None,
-             out_bias: Optional[torch.Tensor] = None, residual: bool = False, blocks: int = 1,
+             out_bias: Optional[torch.Tensor] = None, residual: bool = False, blocks: int = 0,
              out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal convolution over time of every column of x [T, C] + in_bias within its segment: sum_j w[j] x_(t - taps + 1 + j) +
     out_bias, with ``residual`` plus x itself. ``ring`` [slots, taps, C] keeps the last rows of x of every sequence by position modulo
-    taps. blocks > 1: returns the equal blocks of columns one after the other, [blocks, T, n] with n = C / blocks padded with
+    taps. blocks > 0: returns the equal blocks of columns one after the other, [blocks, T, n] with n = C / blocks padded with
     zeros to a multiple of 8."""
     T, C = x.shape
-    n = C // blocks
-    padded = (n + 7) // 8 * 8 if blocks > 1 else n
+    n = C // max(1, blocks)
+    padded = (n + 7) // 8 * 8 if blocks else n
     if not x.is_cuda:
         y = reference.seq_conv(x, w, ring, segs, in_bias, out_bias, residual).to(x.dtype)
-        if blocks > 1:
+        if blocks:
             y = torch.nn.functional.pad(y.view(T, blocks, n).transpose(0, 1), (0, padded - n)).contiguous()
         if out is not None:
             return out.copy_(y)
         return y
     if out is None:
-        shape = (blocks, T, padded) if blocks > 1 else (T, C)
+        shape = (blocks, T, padded) if blocks else (T, C)
         out = (torch.empty if padded == n else torch.zeros)(shape, dtype=x.dtype, device=x.device)
     assert x.stride(1) == 1 and ring.dtype == x.dtype == out.dtype and out.stride(-1) == 1 and C == w.shape[1]
-    d = _conv_descriptor(w, ring, segs, in_bias, out_bias, residual, blocks, padded)
+    d = _conv_descriptor(w, ring, segs, in_bias, out_bias, residual, max(1, blocks), padded)
     _lib.check(_lib.lib().dmoe_seq_conv(_f32(x.dtype), _vp(x), c_ll(x.stride(0)), ctypes.byref(d), _vp(segs.multi), c_int(segs.n_multi),
                                         _vp(segs.chunks), c_int(segs.n_chunks), _vp(out), c_ll(out.stride(-2)),
-                                        c_ll(out.stride(0) if blocks > 1 else 0), c_int(C), _st()), "dmoe_seq_conv")
+                                        c_ll(out.stride(0) if blocks else 0), c_int(C), _st()), "dmoe_seq_conv")
     return out
 
 

@@ -52,13 +52,13 @@ MODELS = {
     # nothing aligned: widths, heads, vocabulary, blocks, experts; two taps
     "odd": model(44, 101, [lightning(10, 7, (0.5, 0.97, 0.999), moe(6, 3, 11, 2.5)), both(left(6, 3, 10, 14, 0.31, (0.2, 5)), right(3, 12, 9),
                            dense(37)), unit(45, 3, 3, moe(5, 5, 8)), both(left(3, 3, 20, 6, None, None), right(1, 6, 22, 20.0), None),
-                           unit(26, 2, 1, dense(13))], taps=2),
+                           unit(26, 2, 1, dense(13)), unit(21, 1, 5, None)], taps=2),
     # one of everything: heads, blocks, experts, one tap
     "ones": model(64, 80, [unit(32, 1, 4, moe(1, 1, 16)), lightning(16, 16, (0.9,), moe(4, 4, 16)),
                            both(left(1, 1, 16, 16, 1.0, (0.7, 1)), right(1, 16, 16, 1.0), dense(24)), unit(64, 64, 2, None)], taps=1),
     # many heads, long convolutions, large states
-    "wide": model(96, 90, [both(left(16, 2, 128, 128, None, (0.1, 64)), right(5, 128, 64), moe(16, 8, 32, 3.0)),
-                           unit(320, 5, 8, moe(64, 6, 24)), lightning(128, 128, (0.2, 0.9, 0.99, 0.9995, 0.6), dense(200)),
+    "wide": model(96, 90, [both(left(16, 2, 128, 128, None, (0.1, 64)), right(5, 128, 64), moe(16, 16, 32, 3.0)),
+                           unit(320, 5, 8, moe(64, 1, 24)), lightning(128, 128, (0.2, 0.9, 0.99, 0.9995, 0.6), dense(200)),
                            both(left(35, 5, 24, 32), right(9, 8, 8), None)], taps=8),
 }
 
