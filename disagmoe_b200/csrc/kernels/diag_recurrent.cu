@@ -97,18 +97,34 @@ seq_conv_kernel(const T* __restrict__ x, long long ldx, const DmoeConv a, const 
 }
 
 // ---- the recurrence ----------------------------------------------------------------------------------------------------
-__device__ __forceinline__ float sigmoid32(float x) { return 1.f / (1.f + expf(-x)); }
-// tanh form of gelu: z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)); FAST: with the approximate exponential and division
+// x sigmoid(z); FAST: with the approximate exponential and division (fp32 to a few ulp)
+template <bool FAST>
+__device__ __forceinline__ float times_sigmoid(float x, float z) {
+  return FAST ? __fdividef(x, 1.f + __expf(-z)) : x / (1.f + expf(-z));
+}
+// tanh form of gelu: z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
 template <bool FAST>
 __device__ __forceinline__ float gelu_gate(float z) {
-  const float p = 1.5957691216057308f * (z + 0.044715f * z * z * z);
-  return FAST ? __fdividef(z, 1.f + __expf(-p)) : z / (1.f + expf(-p));
+  return times_sigmoid<FAST>(z, 1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+// exp(x) - 1 for x <= 0: the Taylor series near zero (relative error below 2e-8 there), the exponential elsewhere
+__device__ __forceinline__ float expm1_below(float x) {
+  float p = 1.f / 5040.f;
+  p = p * x + 1.f / 720.f;
+  p = p * x + 1.f / 120.f;
+  p = p * x + 1.f / 24.f;
+  p = p * x + 1.f / 6.f;
+  p = p * x + 0.5f;
+  p = p * x + 1.f;
+  return x > -0.35f ? p * x : __expf(x) - 1.f;
 }
 // a token's step: S <- a S + b. 1 - a^2 = -(a - 1) (a + 1) from a - 1 = expm1(log a), exact where a is near one
+template <bool FAST>
 __device__ __forceinline__ void unit_step(float r, float i, float u, float decay, float& a, float& b) {
-  const float e = expm1f(decay * sigmoid32(r));
+  const float x = times_sigmoid<FAST>(decay, r), e = FAST ? expm1_below(x) : expm1f(x);
   a = 1.f + e;
-  b = sqrtf(-e * (2.f + e)) * (sigmoid32(i) * u);
+  const float w = -e * (2.f + e);
+  b = (FAST ? w * rsqrtf(fmaxf(w, 1e-37f)) : sqrtf(w)) * times_sigmoid<FAST>(u, i);
 }
 
 constexpr int kUnitThreads = 256;
@@ -136,7 +152,7 @@ __global__ void __launch_bounds__(kUnitThreads) unit_step_kernel(const DmoeUnit 
 #pragma unroll
   for (int e = 0; e < VEC; ++e) {
     float a, b;
-    unit_step(r[e] + rb[e], i[e] + ib[e], u[e], dec[e], a, b);
+    unit_step<sizeof(T) == 2>(r[e] + rb[e], i[e] + ib[e], u[e], dec[e], a, b);
     S[e] = a * S[e] + b;
     y[e] = S[e] * gelu_gate<sizeof(T) == 2>(y[e] + yb[e]);
   }
@@ -157,52 +173,71 @@ __global__ void __launch_bounds__(kScanThreads) unit_scan_kernel(const DmoeUnit 
   const int c = blockIdx.y * CH + ch, cc = min(c, d.width - 1);
   const bool on = c < d.width;
   const int blk = cc / per, o = cc % per;
-  const T* up = static_cast<const T*>(d.u) + (blk * d.block_rows + seg.x) * d.padded + o;
-  const float* gp = d.gates + (blk * d.block_rows + seg.x) * 2 * d.padded + o;
-  const T* yp = static_cast<const T*>(d.y) + seg.x * d.ldy + cc;
-  T* op = static_cast<T*>(d.out) + seg.x * d.ldo + cc;
+  // this run's rows, one pass further each time
+  const long long row = seg.x + run * kRun;
+  const T* up = static_cast<const T*>(d.u) + (blk * d.block_rows + row) * d.padded + o;
+  const float* gp = d.gates + (blk * d.block_rows + row) * 2 * d.padded + o;
+  const T* yp = static_cast<const T*>(d.y) + row * d.ldy + cc;
+  T* op = static_cast<T*>(d.out) + row * d.ldo + cc;
   const float rb = d.gate_bias[2 * blk * d.padded + o], ib = d.gate_bias[(2 * blk + 1) * d.padded + o];
   const float yb = d.y_bias[cc], dec = d.decay[cc];
   float* sp = d.state + static_cast<long long>(seg.z) * d.width + cc;
   if (run == 0) s_carry[0][ch] = seg.w > 0 ? *sp : 0.f;
 
   float u[kRun], r[kRun], i[kRun], y[kRun];
-  auto fetch = [&](int t0) {
+  const int p = d.padded, ldy = static_cast<int>(d.ldy), ldo = static_cast<int>(d.ldo);
+  auto fetch = [&](int left) {                       // left: tokens of the segment from the run's first on
+    if (left >= kRun) {
 #pragma unroll
-    for (int k = 0; k < kRun; ++k) {
-      const long long t = t0 + run * kRun + k;
-      const bool in = t < seg.y;
-      u[k] = in ? static_cast<float>(up[t * d.padded]) : 0.f;
-      r[k] = in ? gp[t * 2 * d.padded] : 0.f;
-      i[k] = in ? gp[t * 2 * d.padded + d.padded] : 0.f;
-      y[k] = in ? static_cast<float>(yp[t * d.ldy]) : 0.f;
+      for (int k = 0; k < kRun; ++k) {
+        u[k] = static_cast<float>(up[k * p]);
+        r[k] = gp[2 * k * p];
+        i[k] = gp[2 * k * p + p];
+        y[k] = static_cast<float>(yp[k * ldy]);
+      }
+    } else {
+#pragma unroll
+      for (int k = 0; k < kRun; ++k) {
+        const bool in = k < left;
+        u[k] = in ? static_cast<float>(up[k * p]) : 0.f;
+        r[k] = in ? gp[2 * k * p] : 0.f;
+        i[k] = in ? gp[2 * k * p + p] : 0.f;
+        y[k] = in ? static_cast<float>(yp[k * ldy]) : 0.f;
+      }
     }
+    up += static_cast<long long>(PASS) * p;
+    gp += 2ll * PASS * p;
+    yp += PASS * d.ldy;
   };
-  fetch(0);
+  fetch(seg.y - run * kRun);
   int buf = 0;
   for (int t0 = 0; t0 < seg.y; t0 += PASS, buf ^= 1) {
     const int left = seg.y - t0 - run * kRun;      // tokens of the segment from this run's first on
     float a[kRun], b[kRun], g[kRun], A = 1.f, B = 0.f;
 #pragma unroll
     for (int k = 0; k < kRun; ++k) {
-      a[k] = 1.f;
-      b[k] = 0.f;
-      if (k < left) unit_step(r[k] + rb, i[k] + ib, u[k], dec, a[k], b[k]);
+      unit_step<sizeof(T) == 2>(r[k] + rb, i[k] + ib, u[k], dec, a[k], b[k]);
+      if (k >= left) {
+        a[k] = 1.f;
+        b[k] = 0.f;
+      }
       g[k] = gelu_gate<sizeof(T) == 2>(y[k] + yb);
       A *= a[k];
       B = a[k] * B + b[k];
     }
     s_a[buf][run][ch] = A;
     s_b[buf][run][ch] = B;
-    if (t0 + PASS < seg.y) fetch(t0 + PASS);
+    if (t0 + PASS < seg.y) fetch(left - PASS);
     __syncthreads();
     float S = s_carry[buf][ch];
+#pragma unroll 8
     for (int j = 0; j < run; ++j) S = s_a[buf][j][ch] * S + s_b[buf][j][ch];
 #pragma unroll
     for (int k = 0; k < kRun; ++k) {
       S = a[k] * S + b[k];
-      if (on && k < left) op[(t0 + run * kRun + k) * d.ldo] = static_cast<T>(S * g[k]);
+      if (on && k < left) op[k * ldo] = static_cast<T>(S * g[k]);
     }
+    op += PASS * d.ldo;
     // tokens past the end leave S alone: the last run ends with the state of the segment's last token
     if (run == RUNS - 1) {
       s_carry[buf ^ 1][ch] = S;

@@ -331,11 +331,11 @@ typedef struct DmoeRecur {
   const float* gate_bias;   // [2 heads]
   float* norm_state;        // [n_slots, heads, dim]
   float* max_state;         // [n_slots, 2, heads]: m at the parity of its position
-  float* keep;              // [rows, heads] log decays, factors of k and running maxima of longer segments (dmoe_memory_gates)
+  float* keep;              // [heads, ldsteps] log decays, factors of k and running maxima of longer segments (dmoe_memory_gates)
   float* put;
   float* run_max;
   float* scale;             // with raw: [rows, heads] factors of the read-outs (the divisions above)
-  long long ldgates;
+  long long ldgates, ldsteps;
   float gate_cap;
 } DmoeRecur;
 // keep, put and run_max of the rows of a->segs; the running maxima in the slots move on.

@@ -24,7 +24,7 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
 }
 
 // out[t] = table[ids[t]] * scale (+ ptab[positions[t]]), fp32
-template <typename T>
+template <typename T, int VEC>
 __global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float scale,
                                  float* __restrict__ out, int W, int vocab, const int* __restrict__ positions,
                                  const T* __restrict__ ptab, int n_pos) {
@@ -33,8 +33,14 @@ __global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restric
   if (id < 0 || id >= vocab) id = 0;
   const T* src = table + static_cast<long long>(id) * W;
   const T* ps = ptab != nullptr ? ptab + static_cast<long long>(min(max(positions[t], 0), n_pos - 1)) * W : nullptr;
-  for (int i = threadIdx.x; i < W; i += blockDim.x)
-    out[t * W + i] = static_cast<float>(src[i]) * scale + (ps != nullptr ? static_cast<float>(ps[i]) : 0.f);
+  for (int i = threadIdx.x * VEC; i < W; i += blockDim.x * VEC) {
+    float x[VEC], p[VEC] = {};
+    Pack<T, VEC>::load(src + i, x);
+    if (ps != nullptr) Pack<T, VEC>::load(ps + i, p);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] = x[e] * scale + p[e];
+    Pack<float, VEC>::store(out + t * W + i, x);
+  }
 }
 
 // r = rows != NULL ? rows[i] : i;  x = resid[r] + (y != NULL ? norm(y[r]) * post : 0);  resid[r] = x where y is given and
@@ -599,7 +605,7 @@ rope_append_kernel(bf16* __restrict__ qkv, long long ld, const int* __restrict__
   bf16* row = qkv + t * ld;
   const float2* tab = table + static_cast<long long>(pos) * (rot / 2);
   const int uq = n_q * dk / 8, uk = uq + (slot >= 0 ? n_kv * dk / 8 : 0);
-  for (int u = threadIdx.x; u < uk; u += blockDim.x) {
+  for (int u = threadIdx.x + (rot == 0 ? uq : 0); u < uk; u += blockDim.x) {       // without a rotation q is in place
     const int d = u * 8 % dk;
     const bool is_q = u < uq;
     if (is_q && d >= rot) continue;           // in place already
@@ -806,13 +812,16 @@ extern "C" int dmoe_embed_f32(const int* ids, const void* table, int is_f32, flo
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (W < 1 || vocab < 1 || (pos_table != nullptr && (positions == nullptr || n_pos < 1))) return -10;
   if (T == 0) return 0;
-  const int threads = W >= 256 ? 256 : 64;
-  if (is_f32)
-    embed_f32_kernel<float><<<T, threads, 0, stream>>>(ids, static_cast<const float*>(table), scale, out, W, vocab, positions,
-                                                       static_cast<const float*>(pos_table), n_pos);
-  else
-    embed_f32_kernel<bf16><<<T, threads, 0, stream>>>(ids, static_cast<const bf16*>(table), scale, out, W, vocab, positions,
-                                                      static_cast<const bf16*>(pos_table), n_pos);
+  const bool vec = W % 8 == 0 && aligned16(table) && aligned16(pos_table) && aligned16(out);
+  const int threads = W >= (vec ? 2048 : 256) ? 256 : 64;
+#define DMOE_EMBED(T_, VEC_)                                                                                                  \
+  embed_f32_kernel<T_, VEC_><<<T, threads, 0, stream>>>(ids, static_cast<const T_*>(table), scale, out, W, vocab, positions, \
+                                                        static_cast<const T_*>(pos_table), n_pos)
+  if (is_f32 && vec) DMOE_EMBED(float, 8);
+  else if (is_f32) DMOE_EMBED(float, 1);
+  else if (vec) DMOE_EMBED(bf16, 8);
+  else DMOE_EMBED(bf16, 1);
+#undef DMOE_EMBED
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -35,7 +35,7 @@ struct TokenGates {
 __device__ __forceinline__ TokenGates token_gates(const DmoeRecur& a, long long row, int pos, int slot, int h) {
   TokenGates g;
   if (a.keep != nullptr) {
-    const long long at = row * a.heads + h;
+    const long long at = h * a.ldsteps + row;
     g.keep = expf(a.keep[at]);
     g.put = a.put[at];
     g.top = a.run_max[at];
@@ -487,47 +487,51 @@ wide_gate_norm_kernel(const int4* __restrict__ table, const float* __restrict__ 
   }
 }
 
-// Matrix memory, longer segments: log decay, factor of k and running maximum of every token, one CTA per (segment, head), 256 tokens
-// at a time. With F the running sum of the logs f, m_t = F_t + max(m_0, max_{j <= t} (i_j - F_j)).
-constexpr int kGateThreads = 256;
+// Matrix memory, longer segments: log decay, factor of k and running maximum of every token, one CTA per (segment, head), 1024 tokens
+// at a time. A run of tokens is a map m -> max(F + m, I); maps are composed along the tokens. Whatever wins the maximum is then a
+// sum over few tokens (logs of input gates are bounded), so nothing cancels.
+constexpr int kGateThreads = 1024;
+__device__ __forceinline__ void scan_max_plus(float& F, float& I, int lane) {       // over the warp, inclusive
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float fl = __shfl_up_sync(0xffffffffu, F, o), il = __shfl_up_sync(0xffffffffu, I, o);
+    if (lane >= o) {
+      I = fmaxf(il + F, I);
+      F += fl;
+    }
+  }
+}
 __global__ void __launch_bounds__(kGateThreads) memory_gates_kernel(const DmoeRecur a) {
-  __shared__ float s_sum[kGateThreads / 32], s_max[kGateThreads / 32], s_top[kGateThreads];
+  __shared__ float s_F[kGateThreads / 32], s_I[kGateThreads / 32], s_top[kGateThreads];
   const int4 seg = static_cast<const int4*>(a.segs)[blockIdx.x];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, slot = seg.z;
   if (seg.y <= 0 || slot < 0 || slot >= a.n_slots) return;
   float top = seg.w > 0 ? *max_state(a, slot, seg.w - 1, h) : 0.f;       // before the pass
-  float i = 0.f, f = 0.f;
+  float i = -INFINITY, f = 0.f;
   if (tid < seg.y) memory_logs(a, seg.x + tid, h, i, f);
   for (int t0 = 0; t0 < seg.y; t0 += kGateThreads) {
     const int t = t0 + tid;
-    const bool on = t < seg.y;
-    float ni = 0.f, nf = 0.f;
+    float ni = -INFINITY, nf = 0.f;
     if (t + kGateThreads < seg.y) memory_logs(a, seg.x + t + kGateThreads, h, ni, nf);
-    float F = on ? f : 0.f;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, F, o);
-      if (lane >= o) F += v;
+    float F = f, I = i;
+    scan_max_plus(F, I, lane);
+    if (lane == 31) {
+      s_F[warp] = F;
+      s_I[warp] = I;
     }
-    if (lane == 31) s_sum[warp] = F;
     __syncthreads();
-    for (int w = 0; w < warp; ++w) F += s_sum[w];
-    float best = on ? i - F : -INFINITY;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, best, o);
-      if (lane >= o) best = fmaxf(best, v);
-    }
-    if (lane == 31) s_max[warp] = best;
-    __syncthreads();
-    for (int w = 0; w < warp; ++w) best = fmaxf(best, s_max[w]);
-    const float m = F + fmaxf(top, best);
+    float wF = s_F[lane], wI = s_I[lane];
+    scan_max_plus(wF, wI, lane);
+    wF = __shfl_sync(0xffffffffu, wF, max(warp - 1, 0));
+    wI = __shfl_sync(0xffffffffu, wI, max(warp - 1, 0));
+    const float base = warp > 0 ? fmaxf(wF + top, wI) : top;               // before this warp's tokens
+    const float m = fmaxf(F + base, I);
     s_top[tid] = m;
     __syncthreads();
-    if (on) {
+    if (t < seg.y) {
       const float before = tid > 0 ? s_top[tid - 1] : top;
-      const long long at = static_cast<long long>(seg.x + t) * a.heads + h;
-      // the maximum is only a scale: whatever its rounding, the steps below are exactly those between the stored values
+      const long long at = h * a.ldsteps + seg.x + t;
+      // the steps are those between the stored maxima, whatever their rounding
       a.keep[at] = f + before - m;
       a.put[at] = expf(i - m);
       a.run_max[at] = m;
@@ -536,7 +540,7 @@ __global__ void __launch_bounds__(kGateThreads) memory_gates_kernel(const DmoeRe
     top = s_top[kGateThreads - 1];
     i = ni;
     f = nf;
-    __syncthreads();                                     // s_top and the partial sums are rewritten
+    __syncthreads();                                     // s_top and the warps' maps are rewritten
   }
 }
 

@@ -635,7 +635,7 @@ chunk_prep_head_kernel(const DmoeRecur a, const int4* __restrict__ chunks, uint8
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int t = 2 * lane + e;
-      const long long at = (row0 + t) * a.heads + h;
+      const long long at = h * a.ldsteps + row0 + t;
       b[e] = t < n ? kLog2e * (MEM ? a.keep[at] : a.head_decay[h]) : 0.f;
       p[e] = t < n ? (MEM ? a.put[at] : 1.f) : 0.f;
     }
@@ -806,6 +806,7 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
       }
     }
   };
+  float top0 = 0.f, top1 = 0.f;                                  // normaliser: running maxima of the rows r0 and r1
   auto fetch_v = [&](int c) {
     if (!DELTA && tid < kChunk * NT) {
       const int t = tid / NT, cc = v0 + tid % NT * 8;
@@ -817,9 +818,17 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
                                                 static_cast<long long>(seg.x + c * kChunk + t) * a.ldv + h * V + cc);
     }
   };
+  auto fetch_top = [&](int c) {
+    if (MEM && ones && reads && tq == 0) {
+      const float* p = a.run_max + h * a.ldsteps + seg.x + c * kChunk;
+      if (c * kChunk + r0 < seg.y) top0 = p[r0];
+      if (c * kChunk + r1 < seg.y) top1 = p[r1];
+    }
+  };
   fetch_a(0);
   fetch_b(0);
   fetch_v(0);
+  fetch_top(0);
 
   // the state tile: rows d = warp * 16 + g (+ 8), columns v0 + nt * 8 + 2 tq (+ 1)
   float* sp = a.state + (static_cast<long long>(slot) * a.heads + h) * D * V;
@@ -936,11 +945,10 @@ chunk_scan_kernel(const DmoeRecur a, const uint8_t* __restrict__ ws, long long w
     if (reads) {
       const int t0 = c * kChunk + r0, t1 = c * kChunk + r1;
       if (ones && tq == 0) {
-        const long long at = static_cast<long long>(seg.x) * a.heads + h;
-        if (t0 < seg.y) a.scale[at + static_cast<long long>(t0) * a.heads] =
-            memory_scale(acc[0][0] + cross[0][0], a.run_max[at + static_cast<long long>(t0) * a.heads]);
-        if (t1 < seg.y) a.scale[at + static_cast<long long>(t1) * a.heads] =
-            memory_scale(acc[0][2] + cross[0][2], a.run_max[at + static_cast<long long>(t1) * a.heads]);
+        float* sc = a.scale + static_cast<long long>(seg.x) * a.heads + h;
+        if (t0 < seg.y) sc[static_cast<long long>(t0) * a.heads] = memory_scale(acc[0][0] + cross[0][0], top0);
+        if (t1 < seg.y) sc[static_cast<long long>(t1) * a.heads] = memory_scale(acc[0][2] + cross[0][2], top1);
+        if (c + 1 < nc) fetch_top(c + 1);
       }
       float* o0 = a.raw + static_cast<long long>(seg.x + t0) * a.ldraw + h * V;
       float* o1 = a.raw + static_cast<long long>(seg.x + t1) * a.ldraw + h * V;

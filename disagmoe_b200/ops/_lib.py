@@ -73,7 +73,7 @@ class DmoeRecur(ctypes.Structure):
                                   "gate_kind", "is_f32", "one_token")] + \
                [(n, _f) for n in ("qscale", "inv_tau", "eps")] + [("status", _vp), ("bonus", _vp), ("norm_ld", _i)] + \
                [(n, _vp) for n in ("head_decay", "gates", "gate_bias", "norm_state", "max_state", "keep", "put", "run_max", "scale")] + \
-               [("ldgates", _ll), ("gate_cap", _f)]
+               [("ldgates", _ll), ("ldsteps", _ll), ("gate_cap", _f)]
 
 
 class DmoeRouter(ctypes.Structure):

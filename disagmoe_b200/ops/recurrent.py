@@ -237,8 +237,8 @@ def recurrent_attention(r: Recurrence, q, k, v, gate, beta, z, state: RecurrentS
         d.segs, d.n_segs = segs.multi.data_ptr(), segs.n_multi
         raw_rows(d)
         if memory:
-            steps = torch.empty(3, T, r.heads, dtype=torch.float32, device=q.device)
-            d.keep, d.put, d.run_max = (t.data_ptr() for t in steps)
+            steps = torch.empty(3, r.heads, T, dtype=torch.float32, device=q.device)
+            d.keep, d.put, d.run_max, d.ldsteps = *(t.data_ptr() for t in steps), T
             _lib.check(lib.dmoe_memory_gates(ctypes.byref(d), st), "dmoe_memory_gates")
         if q.dtype == torch.bfloat16 and lib.dmoe_recur_chunk_ok(r.dim, r.vdim):
             per_head = lib.dmoe_recur_chunk_bytes(r.dim, r.vdim, int(r.delta), segs.n_chunks)
