@@ -920,6 +920,10 @@ extern "C" int dmoe_qk_norm_rope(int is_f32, void* qkv, long long ld, const int*
   if (!is_f32 && qw == nullptr && n_kv > 0 && (v_norm == 0 || dv <= 256) && dk % 8 == 0 && dv % 8 == 0 && rot % (interleaved ? 8 : 16) == 0 &&
       ld % 8 == 0 && first_head % 8 == 0 && ld_first % 8 == 0 && aligned16(qkv) && aligned16(kcache) && aligned16(vcache) &&
       aligned16(v_first)) {
+    if (rot == 0) {                              // only what is appended moves
+      threads = (n_kv * (dk > dv ? dk : dv) / 8 + 31) / 32 * 32;
+      if (threads > 256) threads = 256;
+    }
     rope_append_kernel<<<T, threads, 0, stream>>>(
         static_cast<bf16*>(qkv), ld, positions, slots, static_cast<bf16*>(kcache), static_cast<bf16*>(vcache), n_q, n_kv, dk, dv,
         rot, interleaved, static_cast<const float2*>(table), max_pos, static_cast<const bf16*>(v_first), ld_first, first_head,

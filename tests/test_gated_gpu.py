@@ -95,7 +95,7 @@ def test_mixed_batches_reuse_pages(name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_long_decoding_over_pages_and_temperatures(dtype):
-    raw = model(128, 200, [both(left(4, 2, 64, 64, None, (0.5, 32)), right(2, 32, 64), moe(8, 2, 48)), unit(128, 2, 4, dense(96)),
+    raw = model(128, 200, [both(left(4, 2, 64, 64, None, (0.5, 32)), right(2, 40, 64), moe(8, 2, 48)), unit(128, 2, 4, dense(96)),
                            lightning(64, 32, (0.5, 0.99, 0.9999), moe(8, 2, 48)), both(left(4, 1, 48, 80), right(3, 64, 32), None)], taps=3)
     w = oracle.random_weights(raw, seed=8)
     toks = tokens(400, raw["vocab"], 2)
